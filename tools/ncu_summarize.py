@@ -1,5 +1,5 @@
 #!/usr/bin/env python
-"""Condense `ncu --page raw --csv` / `--page source --csv` exports (tools/ncu_capture.sh) into the text summaries
+"""Condense `ncu --page raw --csv` exports (tools/ncu_capture.sh) into the text summaries
 tracked under profiles/.  usage: python tools/ncu_summarize.py <case> [<case> ...]"""
 import csv
 import json
@@ -37,42 +37,16 @@ def load_raw(case):
     return {h: (u, v) for h, u, v in zip(hdr, units, vals)}
 
 
-def top_source(case, n=14):
-    path = os.path.join(SRC, f"ncu_{case}_source.csv")
-    if not os.path.exists(path):
-        return []
-    rows = list(csv.reader(open(path)))
-    hdr = rows[1]
-    i_src, i_s, i_ex = hdr.index("Source"), hdr.index("# Samples"), hdr.index("Instructions Executed")
-    stall_cols = [(i, h) for i, h in enumerate(hdr) if h.startswith("stall_") and "Not Issued" not in h]
-    body = []
-    for r in rows[2:]:
-        if len(r) <= i_s or not r[i_s].isdigit():
-            continue
-        stalls = sorted(((int(r[i]) if r[i].isdigit() else 0, h) for i, h in stall_cols), reverse=True)[:2]
-        body.append((int(r[i_s]), r[i_src].strip(), r[i_ex], ", ".join(f"{h[6:]}={c}" for c, h in stalls if c)))
-    total = sum(b[0] for b in body) or 1
-    body.sort(reverse=True)
-    return [(s, 100.0 * s / total, src, ex, st) for s, src, ex, st in body[:n]], total
-
-
 def main(cases):
     os.makedirs(OUT, exist_ok=True)
     for case in cases:
         d = load_raw(case)
-        lines = [f"# ncu --set full --clock-control none --import-source on : case '{case}' (tools/ncu_case.py {case})",
+        lines = [f"# ncu --set full --clock-control none : case '{case}' (tools/ncu_case.py {case})",
                  f"kernel : {d['Kernel Name'][1]}",
                  f"grid {d.get('Grid Size', ('', '?'))[1]} block {d.get('Block Size', ('', '?'))[1]}  device {d.get('Device', ('', '?'))[1]} cc {d.get('CC', ('', '?'))[1]}", ""]
         for k in KEYS:
             if k in d:
                 lines.append(f"{k:92s} {d[k][1]:>18s} {d[k][0]}")
-        ts = top_source(case)
-        if ts:
-            rows, total = ts
-            lines += ["", f"## hottest SASS instructions by warp-stall samples (total samples {total})",
-                      f"{'samples':>8s} {'%':>6s}  {'executed':>9s}  instruction   [top stall reasons]"]
-            for s, pct, src, ex, st in rows:
-                lines.append(f"{s:8d} {pct:6.2f}  {ex:>9s}  {src[:90]}   [{st}]")
         with open(os.path.join(OUT, f"ncu_{case}.txt"), "w") as f:
             f.write("\n".join(lines) + "\n")
         print("wrote", f"profiles/ncu_{case}.txt")
