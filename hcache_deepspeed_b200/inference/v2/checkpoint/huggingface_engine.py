@@ -17,14 +17,43 @@ from ....utils.logging import inference_logger
 from .base_engine import CheckpointEngineBase
 
 
+class NativeConfig(dict):
+    """A config.json that names an architecture of this framework (``"architecture"``) instead of a HuggingFace model type.
+    Keys are attributes too; ``model_type`` is the architecture's name in the registries (``models/arch.py``)."""
+
+    def __init__(self, d) -> None:
+        super().__init__(d)
+        self["model_type"] = d["architecture"].lower()
+
+    def __getattr__(self, k):
+        try:
+            return self[k]
+        except KeyError as e:
+            raise AttributeError(k) from e
+
+    @staticmethod
+    def load(path: str) -> Optional["NativeConfig"]:
+        """The folder's config when it is a native one, else None."""
+        file = os.path.join(path, "config.json")
+        if not os.path.isfile(file):
+            return None
+        with open(file) as f:
+            d = json.load(f)
+        if "model_type" in d or not isinstance(d.get("architecture"), str):
+            return None
+        return NativeConfig(d)
+
+
 class HuggingFaceCheckpointEngine(CheckpointEngineBase):
 
     def __init__(self, model_name_or_path: str, auth_token: Optional[str] = None, **hf_kwargs) -> None:
         super().__init__()
-        from transformers import AutoConfig
         self.model_name_or_path = model_name_or_path
         self.auth_token = auth_token
-        self.model_config = AutoConfig.from_pretrained(model_name_or_path, **hf_kwargs)
+        self.model_config = NativeConfig.load(model_name_or_path)
+        if self.model_config is None:
+            from transformers import AutoConfig
+            self.model_config = AutoConfig.from_pretrained(model_name_or_path, **hf_kwargs)
         if not hasattr(self.model_config, "max_seq_length"):
             for attr in ("max_position_embeddings", "n_positions", "seq_length"):
                 if hasattr(self.model_config, attr):

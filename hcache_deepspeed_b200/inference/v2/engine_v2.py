@@ -61,12 +61,13 @@ class InferenceEngineV2:
         self._model = self._policy.build_model(self._config, self._base_mp_group)
         inference_logger().info("Model built.")
         kv_cfg = self._model.kv_cache_config()
-        group = max(1, self._model.n_q // max(1, self._model.n_kv))
+        group = self._model.attention_group()
         self._batch = RaggedBatchWrapper(self._config.state_manager, block_size=kv_cfg[0].block_size,
                                          max_blocks_per_seq=kv_cfg[0].max_blocks_per_allocation_group, group=group,
                                          device=self._model.device)
         self._state_manager = DSStateManager(self._config.state_manager, kv_cfg, base_mp_group=self._base_mp_group,
-                                             device=self._model.device)
+                                             device=self._model.device,
+                                             recurrent_layers=self._model.recurrent_state_config())
         self._model.set_state_manager(self._state_manager)
         self._capture_stream = torch.cuda.Stream(device=self._model.device) if self._model.device.type == "cuda" else None
         self.last_put_stats = {}
@@ -216,10 +217,13 @@ class InferenceEngineV2:
     # forward
     # ------------------------------------------------------------------------------------------------
     def put(self, batch_uids: Iterable[int], batch_tokens: Iterable[torch.Tensor], do_checks: bool = True,
-            capture_latents: Optional[bool] = None, all_logits: bool = False) -> Tuple[torch.Tensor, List]:
+            capture_latents: Optional[bool] = None, all_logits: bool = False,
+            logits_at: Optional[Sequence[Sequence[int]]] = None) -> Tuple[torch.Tensor, List]:
         """One forward over a ragged batch. Returns ``(logits [len(batch_uids), vocab], latents)`` where
         ``latents[i]`` is sequence i's ``[n_layers, n_tokens_i, hidden]`` host tensor (pinned), a
-        :class:`LatentHandle` in async mode, or None when capture is off."""
+        :class:`LatentHandle` in async mode, or None when capture is off. ``logits_at[i]``: the places among sequence i's
+        tokens to return logits for (in this order, all sequences concatenated; None instead of logits when there are none)
+        in place of each sequence's last one."""
         uids, toks = list(batch_uids), list(batch_tokens)
         if do_checks:
             check = self.can_schedule(uids, [int(t.numel()) for t in toks])
@@ -240,13 +244,24 @@ class InferenceEngineV2:
             capture = hc.enabled and hc.capture != "off"
             if capture and not hc.capture_decode_steps and self._batch.current_tokens == self._batch.current_sequences:
                 capture = False
-        if (not capture and not all_logits and self._config.use_cuda_graph_decode and self._model.device.type == "cuda"
-                and self._batch.current_tokens == self._batch.current_sequences and self._batch.n_items_large == 0):
+        rows = None
+        if logits_at is not None:
+            picks = [list(map(int, p)) for p in logits_at]
+            if len(picks) != len(uids) or any(not 0 <= p < n for (_, n, _), ps in
+                                              zip(self._batch.inflight_seq_descriptors_shadow, picks) for p in ps):
+                raise ValueError("logits_at must list, for every sequence, places among its tokens")
+            rows = [b + p for (b, _, _), ps in zip(self._batch.inflight_seq_descriptors_shadow, picks) for p in ps]
+            if self._batch.current_tokens == self._batch.current_sequences and len(rows) == len(uids):
+                rows = None    # a decode step that wants every sequence's logits: the ordinary path
+        if (not capture and not all_logits and rows is None and self._config.use_cuda_graph_decode and self._model.device.type == "cuda"
+                and self._batch.current_tokens == self._batch.current_sequences and self._model.graphable_decode(self._batch)):
             logits, latent_dev = self._graphed_decode(), None
         else:
-            logits, latent_dev = self._model.forward(self._batch, capture=bool(capture), all_logits=all_logits)
+            row_t = None if rows is None else torch.tensor(rows, dtype=torch.int32).to(self._model.device)
+            logits, latent_dev = self._model.forward(self._batch, capture=bool(capture), all_logits=all_logits, logit_rows=row_t)
         latents = self._export_latents(latent_dev) if capture else [None] * len(uids)
-        assert logits.shape[0] == (self._batch.current_tokens if all_logits else self._batch.current_sequences)
+        assert logits is None or rows is not None or \
+            logits.shape[0] == (self._batch.current_tokens if all_logits else self._batch.current_sequences)
         for uid in uids:
             seq = self._state_manager.get_sequence(uid)
             seq.post_forward()
@@ -257,12 +272,9 @@ class InferenceEngineV2:
         """Pure decode step through a CUDA graph. The batch metadata (token ids, slots, block tables, work items)
         lives in fixed device buffers refreshed by ``finalize`` before every replay; only launch geometry is baked
         in, so one graph serves a given (sequence count, KV split count) until the heuristic wants more splits."""
-        from ...ops.backend import pick_decode_splits, pick_packed_splits, use_packed_decode
         model, batch = self._model, self._batch
         model.finish_pending_restore()
-        pick = pick_packed_splits if use_packed_decode(model.n_q, model.n_kv, model.d) else pick_decode_splits
-        key = (batch.current_sequences, pick(batch.n_items_small, model.n_kv, batch.max_kv_len_small),
-               batch.rows_per_small_item)
+        key = model.decode_graph_key(batch)
         entry = self._decode_graphs.get(key)
         if entry is None:
             seen = self._decode_warm.get(key, 0)
@@ -347,7 +359,7 @@ class InferenceEngineV2:
         """Tokens and KV blocks that scheduling up to ``max_request_tokens`` for ``uid`` would take."""
         seq = self._state_manager.get_sequence(uid)
         if seq is None:
-            if self._state_manager.n_tracked_sequences == self._config.state_manager.max_tracked_sequences:
+            if self._state_manager.free_sequences == 0:
                 return (0, 0)
             seq = PlaceholderSequenceDescriptor()
         return self._model.get_kv_requirements(seq, max_request_tokens, max_request_blocks)
@@ -373,7 +385,7 @@ class InferenceEngineV2:
                 return SchedulingResult.KVCacheLimitExceeded
             batch_len += length
             free_blocks -= sched_blocks
-        if cur_seqs > cfg.max_tracked_sequences:
+        if cur_seqs > cfg.max_tracked_sequences or cur_seqs - self._state_manager.n_tracked_sequences > self._state_manager.free_sequences:
             return SchedulingResult.EngineSequenceLimitExceeded
         if batch_len > cfg.max_ragged_batch_size:
             return SchedulingResult.BatchTokenLimitExceeded

@@ -90,9 +90,12 @@ class InferenceV2Policy:
         if tp_size > 1 and device.type == "cuda" and engine_config.tensor_parallel.fused_collectives:
             from ....parallel.tp_comm import make_tp_comm
             comm = make_tp_comm(mp_group, tp_size, tp_rank, device)
-        model = RaggedTransformer(self.arch, weights, engine_config.state_manager, dtype=dtype, device=device,
-                                  tp_rank=tp_rank, tp_size=tp_size, comm=comm,
-                                  capture_latents=engine_config.hcache.enabled and engine_config.hcache.capture != "off")
+        executor = RaggedTransformer
+        if self.arch.layers is not None:
+            from ....models.hybrid import HybridTransformer as executor
+        model = executor(self.arch, weights, engine_config.state_manager, dtype=dtype, device=device,
+                         tp_rank=tp_rank, tp_size=tp_size, comm=comm,
+                         capture_latents=engine_config.hcache.enabled and engine_config.hcache.capture != "off")
         mode = getattr(getattr(engine_config, "quantization", None), "quantization_mode", None)
         if mode == "wf8af8":
             model.quantize_weights_fp8()
@@ -167,7 +170,12 @@ class BloomPolicy(InferenceV2Policy):
     """ALiBi attention (``hds_attention_next_alibi``) + LayerNorm on the embeddings."""
 
 
+class NipolornPolicy(InferenceV2Policy):
+    """Windowed attention with kept first tokens beside a Mamba-2 mixer in every layer; experts chosen by token id."""
+
+
 MODEL_TYPE_TO_POLICY = {
+    "nipolorn": NipolornPolicy,
     "gpt2": GPT2Policy, "gptj": GPTJPolicy, "gpt_neox": GPTNeoXPolicy, "bloom": BloomPolicy, "gpt_neo": GPTNeoPolicy,
     "llama": Llama2Policy, "opt": OPTPolicy, "mistral": MistralPolicy, "mixtral": MixtralPolicy, "falcon": FalconPolicy,
     "phi": PhiPolicy, "phi3": Phi3Policy, "qwen": QwenPolicy, "qwen2": Qwen2Policy, "qwen2_moe": Qwen2MoePolicy,

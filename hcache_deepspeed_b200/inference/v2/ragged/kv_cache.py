@@ -52,8 +52,12 @@ class BlockedKVCache:
             dtype = DtypeEnum(dtype).value
         self._dtype = dtype
         elem = torch.tensor([], dtype=dtype).element_size()
+        shapes = cfg.layer_shapes if cfg.layer_shapes is not None else [(n_heads, head_dim)] * num_layers
+        self._layer_shapes = shapes
+        self._uniform = all(s == shapes[0] and s is not None for s in shapes)
         self._block_bytes_per_layer = 2 * n_heads * cfg.block_size * head_dim * elem
-        per_block_bytes = num_layers * self._block_bytes_per_layer
+        per_block_bytes = max(1, sum(2 * s[0] * cfg.block_size * s[1] * elem for s in shapes if s is not None))
+        self._per_block_bytes = per_block_bytes
 
         mode = memory_config.mode
         mode = mode if isinstance(mode, AllocationMode) else AllocationMode(mode)
@@ -68,6 +72,8 @@ class BlockedKVCache:
         else:
             usable = memory_config.size
         num_blocks = int(usable // per_block_bytes)
+        if mode == AllocationMode.TOKENS:
+            num_blocks = -(-int(memory_config.size) // cfg.block_size)
         if mp_group is not None:
             # every tensor-parallel rank must agree on the block count
             import torch.distributed as dist
@@ -81,8 +87,12 @@ class BlockedKVCache:
         inference_logger().info(
             f"Allocating KV-cache: {num_blocks} blocks x {per_block_bytes} B = {num_blocks * per_block_bytes / 2**30:.2f} GiB "
             f"(layers={num_layers}, kv_heads={n_heads}, block={cfg.block_size}, head_dim={head_dim}, {dtype})")
-        self._cache = torch.zeros((num_layers, num_blocks, 2, n_heads, cfg.block_size, head_dim), dtype=dtype,
-                                 device=self._device)
+        if self._uniform:
+            self._cache = torch.zeros((num_layers, num_blocks, 2, shapes[0][0], cfg.block_size, shapes[0][1]), dtype=dtype,
+                                      device=self._device)
+        else:   # unlike layers: the same block ids, one tensor per layer
+            self._cache = [None if s is None else torch.zeros((num_blocks, 2, s[0], cfg.block_size, s[1]), dtype=dtype,
+                                                              device=self._device) for s in shapes]
 
     # ---- accessors ---------------------------------------------------------------------------
     @property
@@ -99,7 +109,7 @@ class BlockedKVCache:
 
     @property
     def block_bytes_all_layers(self) -> int:
-        return self._configs[0].cache_shape[0] * self._block_bytes_per_layer
+        return self._per_block_bytes
 
     def get_cache(self, cache_id: int = 0, cache_group: int = 0) -> torch.Tensor:
         """Layer ``cache_id``'s pages: ``[blocks, 2, heads, block_size, head_dim]``."""
@@ -107,6 +117,8 @@ class BlockedKVCache:
 
     @property
     def full_cache(self) -> torch.Tensor:
+        if not self._uniform:
+            raise NotImplementedError("KV offload needs layers with pages of one shape")
         return self._cache
 
     # ---- whole-block offload / restore ------------------------------------------------------------
@@ -114,15 +126,15 @@ class BlockedKVCache:
         """Copy the listed blocks (all layers) into pinned host memory ``[n, layers, 2, heads, bs, d]``."""
         ids = torch.as_tensor(list(blocks) if not isinstance(blocks, torch.Tensor) else blocks, dtype=torch.int32)
         n = ids.numel()
-        shape = (n, ) + (self._cache.shape[0], ) + tuple(self._cache.shape[2:])
+        shape = (n, ) + (self.full_cache.shape[0], ) + tuple(self.full_cache.shape[2:])
         if host_out is None:
             host_out = pinned_empty(shape, self._dtype)
         if self._device.type != "cuda":
-            host_out.copy_(self._cache[:, ids.long()].permute(1, 0, 2, 3, 4, 5))
+            host_out.copy_(self.full_cache[:, ids.long()].permute(1, 0, 2, 3, 4, 5))
             return host_out
         from ....ops import kernels
         staging = torch.empty(shape, dtype=self._dtype, device=self._device)
-        kernels.kv_blocks_copy(self._cache, staging, ids.to(self._device), to_staging=True)
+        kernels.kv_blocks_copy(self.full_cache, staging, ids.to(self._device), to_staging=True)
         host_out.copy_(staging, non_blocking=True)
         return host_out
 
@@ -132,7 +144,7 @@ class BlockedKVCache:
         streams). The KV half of a mixed HCache plan; cold path — runs once at the end of a turn."""
         ids = torch.as_tensor(list(blocks) if not isinstance(blocks, torch.Tensor) else blocks, dtype=torch.long)
         lay = torch.as_tensor(list(layers), dtype=torch.long)
-        sel = self._cache[lay.to(self._device)][:, ids.to(self._device)]          # [n_l, n_b, 2, h, bs, d]
+        sel = self.full_cache[lay.to(self._device)][:, ids.to(self._device)]          # [n_l, n_b, 2, h, bs, d]
         sel = sel.contiguous() if layer_major else sel.permute(1, 0, 2, 3, 4, 5).contiguous()
         host = pinned_empty(tuple(sel.shape), self._dtype)
         host.copy_(sel)
@@ -156,8 +168,8 @@ class BlockedKVCache:
         """Inverse of :meth:`offload` into (possibly different) block ids."""
         ids = torch.as_tensor(list(blocks) if not isinstance(blocks, torch.Tensor) else blocks, dtype=torch.int32)
         if self._device.type != "cuda":
-            self._cache[:, ids.long()] = host_in.permute(1, 0, 2, 3, 4, 5).to(self._dtype)
+            self.full_cache[:, ids.long()] = host_in.permute(1, 0, 2, 3, 4, 5).to(self._dtype)
             return
         from ....ops import kernels
         staging = host_in.to(self._device, non_blocking=True)
-        kernels.kv_blocks_copy(self._cache, staging, ids.to(self._device), to_staging=False)
+        kernels.kv_blocks_copy(self.full_cache, staging, ids.to(self._device), to_staging=False)

@@ -7,7 +7,7 @@ reference accepts it but its KV offload raises NotImplementedError, ``ragged/kv_
 from __future__ import annotations
 
 from enum import Enum
-from typing import Tuple
+from typing import List, Optional, Tuple
 
 from pydantic import PositiveInt, model_validator
 
@@ -31,6 +31,18 @@ class KVCacheConfig(DeepSpeedConfigModel):
     cache_dtype: DtypeEnum = DtypeEnum.fp16
     max_blocks_per_allocation_group: PositiveInt = 64
     """Upper bound of blocks one sequence may own (= ceil(max_context / block_size))."""
+    layer_shapes: Optional[List[Optional[Tuple[PositiveInt, PositiveInt]]]] = None
+    """(kv_heads, head_dim) of every layer when they differ (None = a layer without attention); ``cache_shape`` otherwise."""
+
+
+class RecurrentLayerConfig(DeepSpeedConfigModel):
+    """Per-sequence state of one recurrent layer: a ``heads`` x ``vdim`` x ``state`` matrix stack and the latest ``taps``
+    inputs of ``conv_dim`` convolution channels."""
+    heads: PositiveInt
+    vdim: PositiveInt
+    state: PositiveInt
+    conv_dim: PositiveInt
+    taps: PositiveInt
 
 
 class AllocationMode(Enum):
@@ -38,6 +50,8 @@ class AllocationMode(Enum):
     """Use all free device memory except ``size`` bytes."""
     ALLOCATE = "allocate"
     """Use exactly ``size`` bytes."""
+    TOKENS = "tokens"
+    """Hold ``size`` tokens (rounded up to whole blocks)."""
 
 
 class MemoryConfig(DeepSpeedConfigModel):
@@ -54,6 +68,9 @@ class DSStateManagerConfig(DeepSpeedConfigModel):
     """Sequences per forward."""
     max_context: PositiveInt = 8192
     """Longest sequence (prompt + generation) the engine will hold."""
+    max_state_slots: Optional[PositiveInt] = None
+    """Models with recurrent layers: sequences whose recurrent state may be resident (default: every tracked sequence, as
+    far as an eighth of the free device memory holds them)."""
     memory_config: MemoryConfig = MemoryConfig()
     offload: bool = False
     """Allow whole-sequence KV offload to pinned host memory (``DSStateManager.offload_sequence``)."""

@@ -5,23 +5,29 @@ whole-sequence KV offload / reload implemented (the reference's ``offload`` conf
 """
 from __future__ import annotations
 
-from typing import Any, Dict, Optional, Tuple
+from typing import Any, Dict, Optional, Sequence, Tuple
 
 import torch
 
 from ....utils.logging import inference_logger
 from .blocked_allocator import BlockedAllocator
 from .kv_cache import BlockedKVCache
-from .manager_configs import DSStateManagerConfig, KVCacheConfig
+from .manager_configs import DSStateManagerConfig, KVCacheConfig, RecurrentLayerConfig
 from .sequence_descriptor import DSSequenceDescriptor
+from .state_cache import RecurrentStateCache
 
 
 class DSStateManager:
 
     def __init__(self, config: DSStateManagerConfig, kv_configs: Tuple[KVCacheConfig, ...], base_mp_group: Optional[Any] = None,
-                 device: Optional[torch.device] = None) -> None:
+                 device: Optional[torch.device] = None,
+                 recurrent_layers: Optional[Sequence[Optional[RecurrentLayerConfig]]] = None) -> None:
         self._config = config
         self._kv_configs = kv_configs
+        self._states: Optional[RecurrentStateCache] = None
+        if recurrent_layers is not None:    # before the KV cache, which may take all memory that is left
+            self._states = RecurrentStateCache(recurrent_layers, config.max_tracked_sequences,
+                                               device if device is not None else torch.device("cpu"), config.max_state_slots)
         self._seqs: Dict[int, DSSequenceDescriptor] = {}
         self._free_tracking_ids = list(range(config.max_tracked_sequences - 1, -1, -1))
         self._kv_cache = BlockedKVCache(kv_configs, config.memory_config, mp_group=base_mp_group, offload=config.offload,
@@ -44,8 +50,12 @@ class DSStateManager:
             raise ValueError(f"Sequence {uid} already exists.")
         if not self._free_tracking_ids:
             raise RuntimeError(f"Unable to create tracking slot for sequence {uid} since the metadata buffers are full.")
+        if self._states is not None and self._states.free_slots == 0:
+            raise RuntimeError(f"Unable to admit sequence {uid}: every recurrent-state slot is in use.")
         tid = self._free_tracking_ids.pop()
         seq = DSSequenceDescriptor(tid, self._kv_configs[0].max_blocks_per_allocation_group)
+        if self._states is not None:
+            seq.state_slot = self._states.allocate()
         self._seqs[uid] = seq
         return seq
 
@@ -58,7 +68,20 @@ class DSStateManager:
         ids = seq.free_kv_cache()
         if ids.numel():
             self._allocator.free(ids)
+        if seq.state_slot >= 0:
+            self._states.free(seq.state_slot)
+            seq.state_slot = -1
         self._free_tracking_ids.append(seq.tracking_id)
+
+    @property
+    def recurrent_states(self) -> Optional[RecurrentStateCache]:
+        return self._states
+
+    @property
+    def free_sequences(self) -> int:
+        """Sequences that can still be admitted (tracking entries and, with recurrent layers, state slots)."""
+        n = len(self._free_tracking_ids)
+        return n if self._states is None else min(n, self._states.free_slots)
 
     @property
     def tracked_sequences(self) -> Dict[int, DSSequenceDescriptor]:

@@ -60,7 +60,7 @@ class RaggedBatchWrapper:
         off = 0
         self._off = {}
         for name, n in (("ids", T), ("pos", T), ("slot", T), ("seq", T), ("last", S), ("small", 4 * self._I),
-                        ("large", 4 * self._I), ("tables", S * self._stride)):
+                        ("large", 4 * self._I), ("spans", 4 * S), ("tables", S * self._stride)):
             self._off[name] = (off, n)
             off += n
         mode = fast_host_buffer.staging_mode() if self._device.type == "cuda" else None
@@ -73,13 +73,20 @@ class RaggedBatchWrapper:
         self._dev = self._host if self._device.type == "cpu" else torch.zeros(off, dtype=torch.int32,
                                                                                device=self._device)
 
+        self._h2d_done = torch.cuda.Event() if self._device.type == "cuda" else None
+        self._h2d_pending = False
+
     # ---- building ---------------------------------------------------------------------------------
     def clear(self) -> None:
+        if self._h2d_pending:      # the staging memory is about to be rewritten: the previous upload must have left it
+            self._h2d_done.synchronize()
+            self._h2d_pending = False
         self._n_tokens = 0
         self._n_seqs = 0
         self._finalized = False
         self._inflight: List[Tuple[int, int, int]] = []
         self._descs: List[DSSequenceDescriptor] = []
+        self._n_single = 0
         self._n_small = self._n_large = self._rows_small = self._max_kv_small = self._max_kv_large = 0
 
     def insert_sequence(self, seq_descriptor: DSSequenceDescriptor, tokens: torch.Tensor, do_checks: bool = True) -> None:
@@ -103,6 +110,9 @@ class RaggedBatchWrapper:
         s.seen = seq_descriptor.seen_tokens
         s.n_blocks = seq_descriptor.cur_allocated_blocks
         s.block_ids = seq_descriptor.kv_blocks_ptr()
+        span = self._off["spans"][0] + 4 * self._n_seqs
+        self._host_np[span:span + 4] = (self._n_tokens, n, seq_descriptor.seen_tokens, getattr(seq_descriptor, "state_slot", -1))
+        self._n_single += n == 1
         self._inflight.append((self._n_tokens, n, seq_descriptor.seen_tokens))
         self._descs.append(seq_descriptor)
         self._n_tokens += n
@@ -133,6 +143,8 @@ class RaggedBatchWrapper:
         if self._dev is not self._host:
             used = self._off["tables"][0] + self._n_seqs * self._stride
             self._dev[:used].copy_(self._host[:used], non_blocking=True)
+            self._h2d_done.record()
+            self._h2d_pending = True
         self._finalized = True
 
     # ---- views (device unless on_device=False) --------------------------------------------------------
@@ -164,6 +176,10 @@ class RaggedBatchWrapper:
     def items_large(self, on_device: bool = True) -> torch.Tensor:
         return self._view("large", 4 * self._n_large, on_device).view(self._n_large, 4)
 
+    def spans(self, on_device: bool = True) -> torch.Tensor:
+        """int32 ``[n_seqs, 4]``: (first row in the batch, new tokens, tokens seen before, recurrent-state slot)."""
+        return self._view("spans", 4 * self._n_seqs, on_device).view(self._n_seqs, 4)
+
     # ---- scalars -------------------------------------------------------------------------------------
     @property
     def current_tokens(self) -> int:
@@ -172,6 +188,11 @@ class RaggedBatchWrapper:
     @property
     def current_sequences(self) -> int:
         return self._n_seqs
+
+    @property
+    def n_single_token_seqs(self) -> int:
+        """Sequences of the batch that bring exactly one token (decode steps)."""
+        return self._n_single
 
     @property
     def tensor_toks(self) -> int:

@@ -55,6 +55,8 @@ class DSSequenceDescriptor(BaseSequenceDescriptor):
         self._block_ids = torch.zeros(max_blocks, dtype=torch.int32)  # host; read by hds_build_batch
         self._n_blocks = 0
         self._max_blocks = max_blocks
+        #: slot in the recurrent-state cache (-1: the model has no recurrent layers)
+        self.state_slot = -1
         #: set while the sequence's KV lives in host memory (whole-sequence KV offload)
         self.offloaded_kv: Optional[torch.Tensor] = None
 

@@ -13,6 +13,87 @@ from dataclasses import dataclass, field, replace
 from typing import Any, Callable, Dict, List, Optional
 
 
+# ---------------------------------------------------------------------------------------------------
+# layer descriptions of stacks whose layers are not all alike (ArchSpec.layers)
+# ---------------------------------------------------------------------------------------------------
+@dataclass
+class AttentionSpec:
+    """Grouped-query softmax attention. ``window`` > 0: a query at position p sees the keys (p - window, p] and, always,
+    the first ``keep_first`` positions of its sequence. Positions enter through the mask only (no rotation)."""
+    heads: int
+    kv_heads: int
+    dim: int                 # query / key size of a head
+    vdim: int                # value size of a head
+    scale: float
+    window: int = 0
+    keep_first: int = 0
+
+    @property
+    def page_dim(self) -> int:
+        """Head size of the KV pages (and of q and of the attention output): the kernels' tile sizes 64 and 128, zero
+        padded; larger heads are served unpadded (rounded up to 8) by the generic kernel."""
+        d = max(self.dim, self.vdim)
+        return 64 if d <= 64 else 128 if d <= 128 else -(-d // 8) * 8
+
+    @property
+    def group(self) -> int:
+        return self.heads // self.kv_heads
+
+
+@dataclass
+class StateSpaceSpec:
+    """Mamba-2 mixer: heads of size ``vdim`` with a ``state`` x ``vdim`` recurrent state each; B and C are shared by the
+    heads of a group; a causal convolution of ``conv`` taps in front, a gated norm of ``norm_groups`` parts behind."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int = 1
+    conv: int = 4
+    norm_groups: int = 1
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_dim(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+    @property
+    def in_dim(self) -> int:
+        """Rows of the input projection: z | x | B | C | dt."""
+        return self.inner + self.conv_dim + self.heads
+
+
+@dataclass
+class MixerSpec:
+    """Token mixer of a layer: attention, a state-space mixer, or both side by side on the same input, each with a weight."""
+    attn: Optional[AttentionSpec] = None
+    ssm: Optional[StateSpaceSpec] = None
+    attn_weight: float = 1.0
+    ssm_weight: float = 1.0
+
+
+@dataclass
+class FeedForwardSpec:
+    """``experts`` = 0: dense gated MLP of size ``ff``. Otherwise a mixture of experts of size ``ff`` each, ``top`` per token.
+    ``routing`` = "table": a table gives every token id its experts, all with weight 1 / top. ``shared_ff`` > 0: one more
+    expert that sees every token. ``act`` = "swiglu_clamped" clamps gate and up to ``limit`` (see ops.reference)."""
+    ff: int
+    act: str = "silu"
+    limit: float = 0.0
+    experts: int = 0
+    top: int = 0
+    routing: str = "table"
+    shared_ff: int = 0
+
+
+@dataclass
+class LayerSpec:
+    mixer: MixerSpec
+    mlp: Optional[FeedForwardSpec] = None
+
+
 @dataclass
 class ArchSpec:
     model_type: str
@@ -58,6 +139,9 @@ class ArchSpec:
     moe_intermediate: int = 0
     shared_expert_intermediate: int = 0  # Qwen2-MoE shared expert (with sigmoid gate)
     norm_topk_prob: bool = True
+    #: one entry per layer for stacks of unlike layers; the scalar sizes above then hold the largest values. Such stacks
+    #: keep the residual stream in fp32 and norm every sublayer's input AND output (models/hybrid.py)
+    layers: Optional[List[LayerSpec]] = None
     extras: Dict[str, Any] = field(default_factory=dict)
 
     # ---- derived -------------------------------------------------------------------------------
@@ -79,11 +163,20 @@ class ArchSpec:
 
     def hidden_state_bytes_per_token_layer(self, elem: int = 2) -> int:
         """Bytes HCache stores per token per layer (the QKV GEMM input)."""
-        return self.hidden * elem
+        return self.padded_hidden * elem
 
     def kv_bytes_per_token_layer(self, elem: int = 2) -> int:
         """Bytes plain KV offload stores per token per layer."""
         return 2 * self.kv_dim * elem
+
+    @property
+    def padded_hidden(self) -> int:
+        """Row width of the activation buffers of a ``layers`` stack (16-byte rows for every operand type)."""
+        return self.hidden if self.layers is None else -(-self.hidden // 8) * 8
+
+    @property
+    def has_recurrent_state(self) -> bool:
+        return self.layers is not None and any(l.mixer.ssm is not None for l in self.layers)
 
     def window_of(self, layer: int) -> int:
         return int(self.layer_windows[layer]) if self.layer_windows is not None else int(self.sliding_window)
@@ -93,6 +186,18 @@ class ArchSpec:
 
     def param_count(self) -> int:
         h, i = self.hidden, self.intermediate
+        if self.layers is not None:
+            total = self.vocab * h * (1 if self.tie_word_embeddings else 2) + h
+            for l in self.layers:
+                a, m, f = l.mixer.attn, l.mixer.ssm, l.mlp
+                total += 2 * h
+                if a is not None:
+                    total += h * (a.heads * (a.dim + a.vdim) + a.kv_heads * (a.dim + a.vdim))
+                if m is not None:
+                    total += h * (m.in_dim + m.inner) + m.conv_dim * (m.conv + 1) + 3 * m.heads + m.inner
+                if f is not None:
+                    total += 2 * h + 3 * h * (f.ff * max(1, f.experts) + f.shared_ff) + self.vocab * (f.top if f.experts else 0)
+            return total
         attn = h * (self.q_dim + 2 * self.kv_dim) + self.q_dim * h
         if self.is_moe:
             mlp = self.n_experts * (3 if self.gated_mlp else 2) * h * self.moe_intermediate + h * self.n_experts
@@ -357,6 +462,56 @@ def _qwen2_moe(cfg) -> ArchSpec:
                        top_k=_get(cfg, "num_experts_per_tok"), moe_intermediate=_get(cfg, "moe_intermediate_size"),
                        shared_expert_intermediate=_get(cfg, "shared_expert_intermediate_size", default=0),
                        norm_topk_prob=bool(_get(cfg, "norm_topk_prob", default=False)))
+
+
+@register_arch("nipolorn")
+def _nipolorn(cfg) -> ArchSpec:
+    """Nipolorn: every layer runs windowed attention with kept first tokens beside a Mamba-2 mixer; feed-forwards are dense
+    (clamped gate) or mixtures of experts chosen by token id; norms before and after each sublayer. Everything is per layer
+    in config.json (``layers``), so the scalar fields only carry the largest values."""
+
+    def ff(m) -> Optional[FeedForwardSpec]:
+        if m is None:
+            return None
+        if m["kind"] == "dense":
+            return FeedForwardSpec(ff=int(m["ff"]), act="swiglu_clamped", limit=float(m["limit"]))
+        if m["kind"] != "moe":
+            raise ValueError(f"nipolorn: unknown feed-forward kind {m['kind']!r}")
+        shared = m.get("shared") or {}
+        return FeedForwardSpec(ff=int(m["expert"]["ff"]), act="silu", experts=int(m["router"]["experts"]), top=int(m["router"]["top"]),
+                               routing="table", shared_ff=int(shared.get("ff", 0)))
+
+    layers = []
+    for lc in _get(cfg, "layers"):
+        if lc["type"] != "parallel":
+            raise ValueError(f"nipolorn: unknown layer type {lc['type']!r}")
+        mx = lc["mixer"]
+        a, r = mx["left"], mx["right"]
+        layers.append(LayerSpec(
+            mixer=MixerSpec(
+                attn=AttentionSpec(heads=int(a["heads"]), kv_heads=int(a["kv_heads"]), dim=int(a["dim"]), vdim=int(a["vdim"]),
+                                   scale=float(a["scale"]), window=int(a["mask"]["size"]), keep_first=int(a["mask"]["keep_first"])),
+                ssm=StateSpaceSpec(heads=int(r["heads"]), vdim=int(r["vdim"]), state=int(r["state"]), groups=int(r["groups"]),
+                                   conv=int(r["conv"]), norm_groups=int(r["norm_groups"])),
+                attn_weight=float(mx["left_scale"]), ssm_weight=float(mx["right_scale"])),
+            mlp=ff(lc.get("mlp"))))
+    return stack_arch("nipolorn", layers, hidden=int(_get(cfg, "width")), vocab=int(_get(cfg, "vocab")),
+                      norm_eps=float(_get(cfg, "norm")["eps"]))
+
+
+def stack_arch(model_type: str, layers: List[LayerSpec], hidden: int, vocab: int, norm_eps: float, **kw) -> ArchSpec:
+    """ArchSpec of a stack of unlike layers; its scalar sizes are the largest of any layer."""
+    attn = [l.mixer.attn for l in layers if l.mixer.attn is not None]
+    mlps = [l.mlp for l in layers if l.mlp is not None]
+    widest = max(attn, key=lambda a: a.kv_heads * a.page_dim, default=AttentionSpec(1, 1, 64, 64, 1.0))
+    return ArchSpec(model_type=model_type, n_layers=len(layers), hidden=hidden, n_heads=max((a.heads for a in attn), default=1),
+                    n_kv_heads=widest.kv_heads, head_dim=widest.page_dim,
+                    intermediate=max((m.ff for m in mlps if not m.experts), default=0), vocab=vocab, norm="rms",
+                    norm_eps=norm_eps, act="silu", gated_mlp=True, pos_emb="none",
+                    sliding_window=max((a.window for a in attn), default=0), max_positions=1 << 30,
+                    n_experts=max((m.experts for m in mlps), default=0), top_k=max((m.top for m in mlps), default=0),
+                    moe_intermediate=max((m.ff for m in mlps if m.experts), default=0),
+                    shared_expert_intermediate=max((m.shared_ff for m in mlps), default=0), layers=layers, **kw)
 
 
 # ---------------------------------------------------------------------------------------------------

@@ -467,3 +467,34 @@ def map_gpt_neo(name: str, t: torch.Tensor, spec: ArchSpec) -> List[Piece]:
         if parts[1] == "c_proj":
             return [(layer, f"mlp.down{sfx}", t)]
     return []
+
+
+# ---------------------------------------------------------------------------------------------------
+_NIPOLORN_LAYER = re.compile(r"l(\d+)\.(.+)$")
+_NIPOLORN_MIXER = {"left.q": "attn.q", "left.k": "attn.k", "left.v": "attn.v", "left.o": "attn.o", "right.in": "ssm.in",
+                   "right.conv": "ssm.conv", "right.conv.b": "ssm.conv_b", "right.dt_bias": "ssm.dt_bias",
+                   "right.A_log": "ssm.A_log", "right.D": "ssm.D", "right.norm": "ssm.norm", "right.o": "ssm.o"}
+
+
+@register_mapper("nipolorn")
+def map_nipolorn(name: str, t: torch.Tensor, spec: ArchSpec) -> List[Piece]:
+    if name in ("embed", "final.norm", "head"):
+        return [(None, {"embed": "embed", "final.norm": "final_norm.g", "head": "lm_head"}[name], t)]
+    m = _NIPOLORN_LAYER.match(name)
+    if not m:
+        return []
+    li, rest = int(m.group(1)), m.group(2)
+    if rest.startswith("norm"):
+        return [(li, rest + ".g", t)]
+    part, _, leaf = rest.partition(".")
+    if part == "mix" and leaf in _NIPOLORN_MIXER:
+        return [(li, _NIPOLORN_MIXER[leaf], t)]
+    if part == "mlp":
+        if leaf in ("gate", "up", "down"):
+            return [(li, "mlp." + leaf, t)]
+        if leaf == "table" or leaf.startswith("shared."):
+            return [(li, "moe." + leaf, t)]
+        m = re.match(r"e(\d+)\.(gate|up|down)$", leaf)
+        if m:
+            return [(li, f"moe.experts.{m.group(1)}.{m.group(2)}", t)]
+    return []

@@ -15,7 +15,7 @@ import torch
 from .weights import ExpertWeights, LayerWeights, ModelWeights
 
 ALIGN = 256
-_DTYPES = {"bfloat16": torch.bfloat16, "float16": torch.float16, "float32": torch.float32}
+_DTYPES = {"bfloat16": torch.bfloat16, "float16": torch.float16, "float32": torch.float32, "int32": torch.int32}
 
 
 def pad_to_aligned_offset(offset: int, alignment: int = ALIGN) -> int:

@@ -1,0 +1,379 @@
+"""Layers of stacks that mix attention with recurrent state (``ArchSpec.layers``), for the one executor.
+
+The executor's loop, cache, state manager, batch, capture and restore are those of :class:`RaggedTransformer`; this module
+supplies what such a layer does between them, and how its checkpoint pieces are laid out for the kernels:
+
+* ``w_qkv`` stacks every projection that reads the layer's normed input: ``[q heads | k heads | v heads | z | x | B | C | dt]``.
+  Decode-size batches run it as ONE GEMM; larger ones as two (the QKV rows keep their fused paged-KV epilogue).
+* head sizes are zero padded to the page size of the attention kernels (``AttentionSpec.page_dim``): padded rows of the
+  projections make the GEMM itself produce the zeros, padded columns of the output projection ignore them.
+* ``w_o`` is ``[attention columns | state-space columns]``: both mixers write into one buffer and ONE GEMM projects and adds
+  them. Of their two weights only the ratio is applied there (to the state-space part, in fp32, inside its gated norm); the
+  common factor goes into the norm behind the mixer, which reads its input times that factor.
+* rows and columns of width ``hidden`` are zero padded to 16-byte rows.
+
+The residual stream is fp32. A sublayer leaves ``(output, factor, weight of the norm behind it)`` pending; the next norm kernel
+applies that norm, adds to the stream, and norms the stream for its own sublayer in the same pass.
+"""
+from __future__ import annotations
+
+from typing import Dict, List, NamedTuple, Optional, Tuple
+
+import torch
+
+from ..inference.v2.ragged import RaggedBatchWrapper, RecurrentLayerConfig
+from ..inference.v2.ragged.manager_configs import KVCacheConfig
+from ..ops.backend import pick_decode_splits, pick_packed_splits, pick_prefill_splits, use_packed_decode, windowed_len
+from ..ops.kernels import ACT_CODES
+from .arch import ArchSpec, AttentionSpec, FeedForwardSpec, LayerSpec, MixerSpec, StateSpaceSpec
+from .transformer import RaggedTransformer, ceil_div
+from .weights import ExpertWeights, LayerWeights, ModelWeights, interleave_gate_up
+
+
+def pad8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+# ---------------------------------------------------------------------------------------------------
+# weights
+# ---------------------------------------------------------------------------------------------------
+def required_pieces(l: LayerSpec) -> List[str]:
+    req = ["norm1.g", "norm1b.g"]
+    if l.mixer.attn is not None:
+        req += ["attn.q", "attn.k", "attn.v", "attn.o"]
+    if l.mixer.ssm is not None:
+        req += ["ssm." + n for n in ("in", "conv", "conv_b", "dt_bias", "A_log", "D", "norm", "o")]
+    if l.mlp is not None:
+        req += ["norm2.g", "norm2b.g"]
+        if l.mlp.experts:
+            req += [f"moe.experts.{e}.{n}" for e in range(l.mlp.experts) for n in ("gate", "up", "down")] + ["moe.table"]
+            if l.mlp.shared_ff:
+                req += ["moe.shared.gate", "moe.shared.up", "moe.shared.down"]
+        else:
+            req += ["mlp.gate", "mlp.up", "mlp.down"]
+    return req
+
+
+def _pad(t: torch.Tensor, dim: int, n: int) -> torch.Tensor:
+    if t.shape[dim] == n:
+        return t
+    shape = list(t.shape)
+    shape[dim] = n - t.shape[dim]
+    return torch.cat([t, t.new_zeros(shape)], dim=dim)
+
+
+def _head_rows(w: torch.Tensor, heads: int, d: int, page_dim: int) -> torch.Tensor:
+    """[heads * d, K] -> [heads * page_dim, K]"""
+    return _pad(w.reshape(heads, d, -1), 1, page_dim).reshape(heads * page_dim, -1)
+
+
+def mixer_factors(m: MixerSpec) -> Tuple[float, float]:
+    """(factor of the whole mixer output, weight of the state-space part inside it). The attention part has weight 1 inside
+    (its columns of the output projection are dropped when its weight is 0)."""
+    if m.attn is not None and m.attn_weight != 0.0:
+        return m.attn_weight, m.ssm_weight / m.attn_weight
+    return (m.ssm_weight if m.ssm is not None else 0.0), 1.0
+
+
+def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtype: torch.dtype, device: torch.device) -> LayerWeights:
+    """Checkpoint pieces of one layer in the kernels' layout."""
+    Hp = spec.padded_hidden
+
+    def to(t: torch.Tensor) -> torch.Tensor:
+        return t.to(device=device, dtype=dtype).contiguous()
+
+    def f32(t: torch.Tensor) -> torch.Tensor:
+        return t.to(device=device, dtype=torch.float32).contiguous()
+
+    def gamma(name: str) -> torch.Tensor:
+        return f32(_pad(1.0 + p[name].float(), 0, Hp))    # norm weights are stored as differences from one
+
+    def glu(prefix: str, ff: int) -> ExpertWeights:
+        ffp = pad8(ff)
+        up = interleave_gate_up(_pad(p[prefix + "gate"], 0, ffp), _pad(p[prefix + "up"], 0, ffp))
+        return ExpertWeights(to(_pad(up, 1, Hp)), to(_pad(_pad(p[prefix + "down"], 1, ffp), 0, Hp)))
+
+    lw = LayerWeights(norm1_g=gamma("norm1.g"), norm1b_g=gamma("norm1b.g"))
+    a, m = l.mixer.attn, l.mixer.ssm
+    rows, cols = [], []
+    if a is not None:
+        D = a.page_dim
+        # a scale of zero or less cannot be the factor of a running maximum: its sign (or zero) moves into the query rows
+        sign = 0.0 if a.scale == 0 else -1.0 if a.scale < 0 else 1.0
+        rows += [_head_rows(p["attn.q"] * sign, a.heads, a.dim, D), _head_rows(p["attn.k"], a.kv_heads, a.dim, D),
+                 _head_rows(p["attn.v"], a.kv_heads, a.vdim, D)]
+        o = _pad(p["attn.o"].reshape(spec.hidden, a.heads, a.vdim), 2, D).reshape(spec.hidden, a.heads * D)
+        cols.append(o if m is None or l.mixer.attn_weight != 0.0 else torch.zeros_like(o))
+    if m is not None:
+        rows.append(p["ssm.in"])
+        cols.append(_pad(p["ssm.o"], 1, pad8(m.inner)))
+        lw.ssm_conv_w, lw.ssm_conv_b = f32(p["ssm.conv"].t()), f32(p["ssm.conv_b"])
+        lw.ssm_dt_bias, lw.ssm_a, lw.ssm_d = f32(p["ssm.dt_bias"]), f32(-torch.exp(p["ssm.A_log"].float())), f32(p["ssm.D"])
+        lw.ssm_norm = f32(p["ssm.norm"])
+    lw.w_qkv = to(_pad(torch.cat(rows, dim=0), 1, Hp))
+    lw.w_o = to(_pad(torch.cat(cols, dim=1), 0, Hp))
+    f = l.mlp
+    if f is not None:
+        lw.norm2_g, lw.norm2b_g = gamma("norm2.g"), gamma("norm2b.g")
+        if f.experts:
+            # stacked for the grouped GEMM; the per-expert tensors are views of the stacks
+            ex = [glu(f"moe.experts.{e}.", f.ff) for e in range(f.experts)]
+            up, down = torch.cat([e.w_up for e in ex]), torch.cat([e.w_down for e in ex])
+            nu, nd = ex[0].w_up.shape[0], ex[0].w_down.shape[0]
+            lw.experts = [ExpertWeights(up[e * nu:(e + 1) * nu], down[e * nd:(e + 1) * nd]) for e in range(f.experts)]
+            lw.moe_table = p["moe.table"].to(device=device, dtype=torch.int32).contiguous()
+            if f.shared_ff:
+                lw.shared_expert = glu("moe.shared.", f.shared_ff)
+        else:
+            dense = glu("mlp.", f.ff)
+            lw.w_up, lw.w_down = dense.w_up, dense.w_down
+    return lw
+
+
+def top_weights(spec: ArchSpec, top: Dict[str, torch.Tensor], out: ModelWeights, dtype: torch.dtype,
+                device: torch.device) -> ModelWeights:
+    Hp = spec.padded_hidden
+    out.embed = _pad(top["embed"], 1, Hp).to(device=device, dtype=dtype).contiguous()
+    out.final_norm_g = _pad(1.0 + top["final_norm.g"].float(), 0, Hp).to(device=device).contiguous()
+    out.lm_head = _pad(top["lm_head"], 1, Hp).to(device=device, dtype=dtype).contiguous() if "lm_head" in top else out.embed
+    return out
+
+
+def random_pieces(spec: ArchSpec, l: LayerSpec, gen: torch.Generator, device: torch.device, std: float = 0.02) -> Dict[str, torch.Tensor]:
+    """Random checkpoint pieces of one layer."""
+    H = spec.hidden
+
+    def rnd(*shape, scale=std):
+        return torch.randn(shape, generator=gen, device=device, dtype=torch.float32) * scale
+
+    p = {"norm1.g": rnd(H, scale=0.05), "norm1b.g": rnd(H, scale=0.05)}
+    a, m, f = l.mixer.attn, l.mixer.ssm, l.mlp
+    if a is not None:
+        p.update({"attn.q": rnd(a.heads * a.dim, H), "attn.k": rnd(a.kv_heads * a.dim, H), "attn.v": rnd(a.kv_heads * a.vdim, H),
+                  "attn.o": rnd(H, a.heads * a.vdim)})
+    if m is not None:
+        p.update({"ssm.in": rnd(m.in_dim, H), "ssm.conv": rnd(m.conv_dim, m.conv, scale=0.3), "ssm.conv_b": rnd(m.conv_dim),
+                  "ssm.dt_bias": rnd(m.heads, scale=0.5) - 3.0, "ssm.A_log": rnd(m.heads, scale=0.5), "ssm.D": rnd(m.heads, scale=1.0),
+                  "ssm.norm": 1.0 + rnd(m.inner, scale=0.05), "ssm.o": rnd(H, m.inner)})
+    if f is not None:
+        p.update({"norm2.g": rnd(H, scale=0.05), "norm2b.g": rnd(H, scale=0.05)})
+
+        def glu(prefix, ff):
+            p.update({prefix + "gate": rnd(ff, H), prefix + "up": rnd(ff, H), prefix + "down": rnd(H, ff)})
+
+        if f.experts:
+            for e in range(f.experts):
+                glu(f"moe.experts.{e}.", f.ff)
+            p["moe.table"] = torch.argsort(torch.rand((spec.vocab, f.experts), generator=gen, device=device), dim=1)[:, :f.top].int()
+            if f.shared_ff:
+                glu("moe.shared.", f.shared_ff)
+        else:
+            glu("mlp.", f.ff)
+    return p
+
+
+def random_stack_weights(spec: ArchSpec, dtype: torch.dtype, device: torch.device, seed: int = 0, std: float = 0.02) -> ModelWeights:
+    gen = torch.Generator(device=device).manual_seed(seed)
+    mw = ModelWeights(layers=[layer_weights(spec, l, random_pieces(spec, l, gen, device, std), dtype, device) for l in spec.layers])
+    top = {"embed": torch.randn((spec.vocab, spec.hidden), generator=gen, device=device) * std,
+           "final_norm.g": torch.randn(spec.hidden, generator=gen, device=device) * 0.05,
+           "lm_head": torch.randn((spec.vocab, spec.hidden), generator=gen, device=device) * std}
+    return top_weights(spec, top, mw, dtype, device)
+
+
+# ---------------------------------------------------------------------------------------------------
+# executor
+# ---------------------------------------------------------------------------------------------------
+class Pending(NamedTuple):
+    """A sublayer's output on its way into the residual stream: stream += norm(factor * delta) * weight."""
+    delta: torch.Tensor
+    factor: float
+    weight: torch.Tensor
+
+
+class HybridTransformer(RaggedTransformer):
+
+    def __init__(self, spec: ArchSpec, *args, tp_size: int = 1, **kw) -> None:
+        if tp_size > 1:
+            raise NotImplementedError(f"{spec.model_type}: layers with recurrent state run on one GPU (no tensor-parallel split)")
+        super().__init__(spec, *args, tp_size=tp_size, **kw)
+
+    # ---- geometry ----------------------------------------------------------------------------------
+    @property
+    def kv_block_size(self) -> int:
+        return 64
+
+    def attention_group(self) -> int:
+        return max((l.mixer.attn.group for l in self.spec.layers if l.mixer.attn is not None), default=1)
+
+    def kv_cache_config(self) -> Tuple[KVCacheConfig, ...]:
+        base = super().kv_cache_config()[0]
+        shapes = [None if l.mixer.attn is None else (l.mixer.attn.kv_heads, l.mixer.attn.page_dim) for l in self.spec.layers]
+        return (base.model_copy(update={"layer_shapes": shapes}), )
+
+    def recurrent_state_config(self):
+        if not self.spec.has_recurrent_state:
+            return None
+        return [None if m is None else RecurrentLayerConfig(heads=m.heads, vdim=m.vdim, state=m.state, conv_dim=m.conv_dim, taps=m.conv)
+                for m in (l.mixer.ssm for l in self.spec.layers)]
+
+    def graphable_decode(self, batch: RaggedBatchWrapper) -> bool:
+        return True
+
+    def decode_graph_key(self, batch: RaggedBatchWrapper) -> tuple:
+        key = [batch.current_sequences, batch.rows_per_small_item]
+        for a in {(l.mixer.attn.heads, l.mixer.attn.kv_heads, l.mixer.attn.page_dim, l.mixer.attn.window, l.mixer.attn.keep_first)
+                  for l in self.spec.layers if l.mixer.attn is not None}:
+            n_q, n_kv, d, window, keep = a
+            if batch.n_items_small:
+                pick = pick_packed_splits if use_packed_decode(n_q, n_kv, d) else pick_decode_splits
+                key.append((a, pick(batch.n_items_small, n_kv, windowed_len(batch.max_kv_len_small, window, keep))))
+            if batch.n_items_large:
+                key.append((a, pick_prefill_splits(batch.n_items_large, n_q, windowed_len(batch.max_kv_len_large, window, keep))))
+        return tuple(key)
+
+    def _alloc_buffers(self) -> None:
+        s, c = self.spec, self._state_config
+        T, S, Hp = c.max_ragged_batch_size, c.max_ragged_sequence_count, s.padded_hidden
+        dev, dt = self.device, self.dtype
+
+        def buf(*shape, dtype=dt):
+            return torch.zeros(shape, dtype=dtype, device=dev)
+
+        self._tp_fused, self._tp_wait_next, self._tp_scatter_ok = False, False, False
+        attn = [l.mixer.attn for l in s.layers if l.mixer.attn is not None]
+        ssm = [l.mixer.ssm for l in s.layers if l.mixer.ssm is not None]
+        mlps = [l.mlp for l in s.layers if l.mlp is not None]
+        moes = [f for f in mlps if f.experts]
+        self.residual = buf(T, Hp, dtype=torch.float32)
+        self.xn, self.xn2 = buf(T, Hp), buf(T, Hp)
+        self.latent_buf = buf(s.n_layers, T, Hp) if self.capture_enabled else None
+        self.in_buf = buf(T * max(pad8(lw.w_qkv.shape[0]) for lw in self.w.layers))
+        self.q_buf = buf(T * max((a.heads * a.page_dim for a in attn), default=8))
+        self.mix_buf = buf(T * max(lw.w_o.shape[1] for lw in self.w.layers))
+        self.conv_buf = buf(T * max((pad8(m.conv_dim) for m in ssm), default=8))
+        self.dt_buf = buf(T * max((m.heads for m in ssm), default=1), dtype=torch.float32)
+        self.scan_buf = buf(T * max((m.inner for m in ssm), default=1), dtype=torch.float32)
+        self.act_buf = buf(T * max([pad8(f.ff) for f in mlps if not f.experts] + [pad8(f.shared_ff) for f in moes] + [8]))
+        self._delta_bufs = [buf(T, Hp, dtype=torch.float32)]
+        self._delta_idx = 0
+        self.delta32 = self._delta_bufs[0]
+        self.delta16 = buf(T, Hp)
+        self.hidden_last = buf(S, Hp)
+        self.logits_local = buf(S, self.info.vocab)
+        self.logits_full = self.partial16 = self.kv_scratch = None
+        self.ws_gemm = self.ws_small = self.ws_large = self.io_stream = None
+        self._moe_bufs: Dict[Tuple[int, int, int], dict] = {}
+        if dev.type != "cuda":
+            return
+        k = self.ops.k
+        for f in moes:
+            key = (f.experts, f.top, f.ff)
+            if key not in self._moe_bufs:
+                rows = k.moe_padded_rows(T, f.experts, f.top)
+                self._moe_bufs[key] = dict(
+                    scores=buf(T, f.top, dtype=torch.float32), expert_ids=buf(T, f.top, dtype=torch.int32),
+                    offsets=buf(T, f.top, dtype=torch.int32), mapped_slots=buf(T, f.top, dtype=torch.int32),
+                    counts=buf(f.experts, dtype=torch.int32), pad_off=buf(f.experts + 1, dtype=torch.int32),
+                    xs=buf(rows, Hp), hs=buf(rows, pad8(f.ff)), ys=buf(rows, Hp))
+        if dt != torch.float32:
+            n_max = max([self.info.vocab, Hp] + [lw.w_qkv.shape[0] for lw in self.w.layers] +
+                        [w.shape[0] for lw in self.w.layers for w in [lw.w_up, lw.shared_expert and lw.shared_expert.w_up] if w is not None])
+            self.ws_gemm = torch.zeros(k.gemm_splitk_workspace_bytes(128, n_max), dtype=torch.uint8, device=dev)
+            small, large = 16, 16
+            for a in {(a.heads, a.kv_heads, a.page_dim) for a in attn if a.page_dim <= 128}:
+                b_small, b_large = self._attention_workspace_bytes(S, *a, rows=8)
+                small, large = max(small, b_small), max(large, b_large)
+            self.ws_small = torch.zeros(small, dtype=torch.uint8, device=dev)
+            self.ws_large = torch.zeros(large, dtype=torch.uint8, device=dev)
+        self._alloc_restore_buffers(T, S, Hp)
+
+    def _view(self, flat: torch.Tensor, T: int, cols: int) -> torch.Tensor:
+        return flat[:T * cols].view(T, cols)
+
+    # ---- layer -------------------------------------------------------------------------------------
+    def _embed(self, batch: RaggedBatchWrapper) -> torch.Tensor:
+        return self.ops.embed_f32(batch.input_ids(), self.w.embed, self.residual[:batch.current_tokens])
+
+    def _norm_into(self, resid: torch.Tensor, gamma: torch.Tensor, out: torch.Tensor, pending: Optional[Pending],
+                   keep_resid: bool = True) -> torch.Tensor:
+        delta, factor, post = pending if pending is not None else (None, 1.0, None)
+        return self.ops.norm_residual(resid, gamma, out, delta=delta, factor=factor, post=post, cols=self.spec.hidden,
+                                      eps=self.spec.norm_eps, store_resid=keep_resid)
+
+    def _layer(self, li: int, resid: torch.Tensor, pending: Optional[Pending], xn: torch.Tensor, batch: RaggedBatchWrapper) -> Pending:
+        l, lw, ops, T = self.spec.layers[li], self.w.layers[li], self.ops, batch.current_tokens
+        kv = self._state_manager
+        self._norm_into(resid, lw.norm1_g, xn, pending)
+        self._kv_ready(li)
+        a, m = l.mixer.attn, l.mixer.ssm
+        proj = self._view(self.in_buf, T, pad8(lw.w_qkv.shape[0]))
+        mix = self._view(self.mix_buf, T, lw.w_o.shape[1])
+        n_attn = n_out = 0
+        if a is not None:
+            D = a.page_dim
+            n_attn, n_out = (a.heads + 2 * a.kv_heads) * D, a.heads * D
+            q = self._view(self.q_buf, T, n_out)
+            ops.mixer_in_proj(xn, lw.w_qkv, n_attn, proj, q, kv.get_cache(li), batch.tok_pos(), batch.tok_slot(), a.heads, a.kv_heads,
+                              D, kv.kv_block_size, workspace=self.ws_gemm)
+            ops.attention(q, mix[:, :n_out], kv.get_cache(li), batch, a.heads, a.kv_heads, D, abs(a.scale) or 1.0,
+                          ws_small=self.ws_small, ws_large=self.ws_large, window=a.window, keep_first=a.keep_first)
+        else:
+            ops.gemm(xn, lw.w_qkv, proj[:, :lw.w_qkv.shape[0]], workspace=self.ws_gemm)
+        factor, ssm_weight = mixer_factors(l.mixer)
+        if m is not None:
+            y = self._scan(li, m, lw, proj[:, n_attn:n_attn + m.in_dim], batch.spans(), batch.n_single_token_seqs)
+            ops.gated_norm(y, proj[:, n_attn:n_attn + m.inner], lw.ssm_norm, mix[:, n_out:n_out + m.inner], m.norm_groups,
+                           self.spec.norm_eps, ssm_weight)
+        pending = Pending(self._row_parallel(mix, lw.w_o, None, T, force_accum=False), factor, lw.norm1b_g)
+        if l.mlp is None:
+            return pending
+        x2 = self._norm_into(resid, lw.norm2_g, self.xn2[:T], pending)
+        return Pending(self._feed_forward(x2, l.mlp, lw, T, batch), 1.0, lw.norm2b_g)
+
+    def _scan(self, li: int, m: StateSpaceSpec, lw: LayerWeights, proj: torch.Tensor, spans: torch.Tensor, n_single: int) -> torch.Tensor:
+        """Convolution and recurrence of the tokens whose projections are ``proj`` = [z | x | B | C | dt]; advances the
+        sequences' state. Returns the recurrence's output (before gate and norm), fp32 ``[tokens, inner]``."""
+        T, st = proj.shape[0], self._state_manager.recurrent_states
+        return self.ops.state_space(proj, lw, m, st.ssm(li), st.conv(li), spans, n_single, self._view(self.conv_buf, T, pad8(m.conv_dim)),
+                                    self._view(self.dt_buf, T, m.heads), self._view(self.scan_buf, T, m.inner))
+
+    def _feed_forward(self, x: torch.Tensor, f: FeedForwardSpec, lw: LayerWeights, T: int, batch: RaggedBatchWrapper) -> torch.Tensor:
+        ops = self.ops
+        act = ACT_CODES[f.act]
+
+        def hidden(w: ExpertWeights):
+            h = self._view(self.act_buf, T, w.w_down.shape[1])
+            return ops.gemm(x, w.w_up, h, act=act, gated=True, workspace=self.ws_gemm, limit=f.limit)
+
+        if not f.experts:
+            return self._row_parallel(hidden(ExpertWeights(lw.w_up, lw.w_down)), lw.w_down, None, T, force_accum=False)
+        shared = None
+        if lw.shared_expert is not None:
+            shared = ops.gemm(hidden(lw.shared_expert), lw.shared_expert.w_down, self.delta16[:T], workspace=self.ws_gemm)
+        return ops.table_moe(x, batch.input_ids(), lw, f, act, shared, self.delta32[:T], self._moe_bufs.get((f.experts, f.top, f.ff)))
+
+    def _final_hidden(self, resid: torch.Tensor, pending: Optional[Pending], T: int) -> torch.Tensor:
+        return self._norm_into(resid, self.w.final_norm_g, self.xn2[:T], pending, keep_resid=False)
+
+    def _drop_pending(self, pending: Optional[Pending], T: int) -> None:
+        self.delta32[:T].zero_()
+
+    # ---- restore from saved hidden states ------------------------------------------------------------
+    def _restore_layer(self, li: int, latents: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, spans: torch.Tensor,
+                       n_single: int) -> None:
+        """K/V pages as for any layer; the recurrent state by projecting and scanning the saved inputs once more."""
+        l, lw, ops, T = self.spec.layers[li], self.w.layers[li], self.ops, latents.shape[0]
+        kv = self._state_manager
+        a, m = l.mixer.attn, l.mixer.ssm
+        n_attn = 0
+        proj = self._view(self.in_buf, T, pad8(lw.w_qkv.shape[0]))
+        if a is not None:
+            n_q = a.heads * a.page_dim
+            n_attn = n_q + 2 * a.kv_heads * a.page_dim
+            ops.restore_kv_proj(latents, lw.w_qkv[n_q:n_attn], None, kv.get_cache(li), pos, slot, None, a.kv_heads, a.page_dim,
+                                a.page_dim, kv.kv_block_size, scratch=proj[:, n_q:n_attn])
+        if m is not None:
+            part = proj[:, n_attn:n_attn + m.in_dim]
+            ops.gemm(latents, lw.w_qkv[n_attn:], part, workspace=self.ws_gemm)
+            self._scan(li, m, lw, part, spans, n_single)

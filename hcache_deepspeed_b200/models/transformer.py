@@ -27,7 +27,7 @@ import torch
 from ..inference.v2.ragged import DSStateManager, KVCacheConfig, RaggedBatchWrapper
 from ..inference.v2.ragged.manager_configs import DSStateManagerConfig
 from ..ops import reference as ref
-from ..ops.backend import MAX_DECODE_SPLITS, get_ops, pick_decode_splits
+from ..ops.backend import get_ops, pick_decode_splits, pick_packed_splits, use_packed_decode
 from ..ops.fp8 import Fp8Weight
 from ..ops.kernels import ACT_CODES
 from .arch import ArchSpec
@@ -151,7 +151,7 @@ class RaggedTransformer:
 
     def _alloc_buffers(self) -> None:
         s, c = self.spec, self._state_config
-        T, S, H = c.max_ragged_batch_size, c.max_ragged_sequence_count, s.hidden
+        T, S, H = c.max_ragged_batch_size, c.max_ragged_sequence_count, s.padded_hidden
         dev, dt = self.device, self.dtype
 
         def buf(*shape, dtype=dt):
@@ -195,47 +195,63 @@ class RaggedTransformer:
             k = self.ops.k
             n_max = max(qkv_cols, (2 if s.gated_mlp else 1) * inter, self.info.vocab, H)
             self.ws_gemm = torch.zeros(k.gemm_splitk_workspace_bytes(128, n_max), dtype=torch.uint8, device=dev)
-            G = max(1, self.n_q // max(1, self.n_kv))
+            small, large = self._attention_workspace_bytes(S, self.n_q, self.n_kv, self.d)
+            self.ws_small = torch.zeros(small, dtype=torch.uint8, device=dev)
+            self.ws_large = torch.zeros(large, dtype=torch.uint8, device=dev)
+            self._alloc_restore_buffers(T, S, H)
+
+    def _attention_workspace_bytes(self, S: int, n_q: int, n_kv: int, d: int, rows: Optional[int] = None) -> Tuple[int, int]:
+        """Split-KV scratch of (the decode kernel, the tensor-core kernel) for up to ``S`` sequences of one head geometry.
+        ``rows``: query rows a decode work item may hold (default: what this geometry's own group size allows)."""
+        k = self.ops.k
+        G = max(1, n_q // max(1, n_kv))
+        if rows is None:
             rows = min(8, max(1, (8 // G) * G))
-            worst = 16
-            for n in sorted({1, 2, 4, 8, 16, 32, 64, 128, 256, S}):
-                if n <= S:
-                    worst = max(worst, k.splitkv_workspace_bytes(n, self.n_q, self.n_kv, self.d,
-                                                                 pick_decode_splits(n, self.n_kv, 1 << 30), rows))
-            worst = max(worst, k.splitkv_workspace_bytes(S, self.n_q, self.n_kv, self.d, 1, rows))
-            self.ws_small = torch.zeros(worst, dtype=torch.uint8, device=dev)
-            worst_l = 16
-            for n in range(1, 149):
-                units = n * self.n_q
-                if units >= 148:
-                    break
-                sp = min(16, -(-148 // units))
-                worst_l = max(worst_l, k.prefill_workspace_bytes(n, self.n_q, self.d, sp))
-            from ..ops.backend import pick_packed_splits, use_packed_decode
-            if use_packed_decode(self.n_q, self.n_kv, self.d):   # head-packed GQA decode parks its split-KV partials here too
-                for n in range(1, S + 1):
-                    sp = pick_packed_splits(n, self.n_kv, 1 << 30)
-                    if sp > 1:
-                        worst_l = max(worst_l, k.prefill_workspace_bytes(n, self.n_kv, self.d, sp))
-            self.ws_large = torch.zeros(worst_l, dtype=torch.uint8, device=dev)
-            self.io_stream = torch.cuda.Stream(device=dev)
-            self.restore_stage = buf(RESTORE_SLOTS, T, H)
-            self.restore_stage_sym = None
-            self._slot_peer_ptrs = {}
-            if self.tp_size > 1 and getattr(self.comm, "fused", False):
-                # per-rank slice of the staging ring in symmetric memory: peers' restore kernels read it over NVLink
-                # "copy" gather: full-size slots, each rank fills its own rows and pulls the peers' rows (one P2P read of
-                # every byte); "kernel" gather: per-rank slices that the projection kernel reads through peer tensor maps
-                import os
-                self.tp_gather = os.environ.get("HDS_TP_GATHER", "copy")
-                self._sym_rows = T if self.tp_gather == "copy" else ceil_div(ceil_div(T, self.tp_size), 128) * 128
-                self.restore_stage_sym = self.comm.alloc_symmetric((RESTORE_SLOTS, self._sym_rows, H), dt)
-            self.restore_pos = torch.zeros(T, dtype=torch.int32, device=dev)
-            self.restore_slot = torch.zeros(T, dtype=torch.int32, device=dev)
-            self.ev_loaded = [torch.cuda.Event() for _ in range(RESTORE_SLOTS)]
-            self.ev_consumed = [torch.cuda.Event() for _ in range(RESTORE_SLOTS)]
-            if not (self.d in (64, 128) and (self.inv_freq is None or s.rot_dim == self.d)):
-                self.kv_scratch = buf(T, 2 * self.n_kv * self.d)
+        worst = 16
+        for n in sorted({1, 2, 4, 8, 16, 32, 64, 128, 256, S}):
+            if n <= S:
+                worst = max(worst, k.splitkv_workspace_bytes(n, n_q, n_kv, d, pick_decode_splits(n, n_kv, 1 << 30), rows))
+        worst = max(worst, k.splitkv_workspace_bytes(S, n_q, n_kv, d, 1, rows))
+        worst_l = 16
+        for n in range(1, 149):
+            units = n * n_q
+            if units >= 148:
+                break
+            sp = min(16, -(-148 // units))
+            worst_l = max(worst_l, k.prefill_workspace_bytes(n, n_q, d, sp))
+        if use_packed_decode(n_q, n_kv, d):   # head-packed GQA decode parks its split-KV partials here too
+            for n in range(1, S + 1):
+                sp = pick_packed_splits(n, n_kv, 1 << 30)
+                if sp > 1:
+                    worst_l = max(worst_l, k.prefill_workspace_bytes(n, n_kv, d, sp))
+        return worst, worst_l
+
+    def _alloc_restore_buffers(self, T: int, S: int, H: int) -> None:
+        """Staging ring, private metadata and events of the pipelined restore."""
+        s, dev, dt = self.spec, self.device, self.dtype
+
+        def buf(*shape, dtype=dt):
+            return torch.zeros(shape, dtype=dtype, device=dev)
+
+        self.io_stream = torch.cuda.Stream(device=dev)
+        self.restore_stage = buf(RESTORE_SLOTS, T, H)
+        self.restore_stage_sym = None
+        self._slot_peer_ptrs = {}
+        if self.tp_size > 1 and getattr(self.comm, "fused", False):
+            # per-rank slice of the staging ring in symmetric memory: peers' restore kernels read it over NVLink
+            # "copy" gather: full-size slots, each rank fills its own rows and pulls the peers' rows (one P2P read of
+            # every byte); "kernel" gather: per-rank slices that the projection kernel reads through peer tensor maps
+            import os
+            self.tp_gather = os.environ.get("HDS_TP_GATHER", "copy")
+            self._sym_rows = T if self.tp_gather == "copy" else ceil_div(ceil_div(T, self.tp_size), 128) * 128
+            self.restore_stage_sym = self.comm.alloc_symmetric((RESTORE_SLOTS, self._sym_rows, H), dt)
+        self.restore_pos = torch.zeros(T, dtype=torch.int32, device=dev)
+        self.restore_slot = torch.zeros(T, dtype=torch.int32, device=dev)
+        self.restore_spans = torch.zeros(S, 4, dtype=torch.int32, device=dev)
+        self.ev_loaded = [torch.cuda.Event() for _ in range(RESTORE_SLOTS)]
+        self.ev_consumed = [torch.cuda.Event() for _ in range(RESTORE_SLOTS)]
+        if not (self.d in (64, 128) and (self.inv_freq is None or s.rot_dim == self.d)):
+            self.kv_scratch = buf(T, 2 * self.n_kv * self.d)
 
     # ------------------------------------------------------------------------------------------------
     # DSInferenceModelBase-style KV accounting (ref: inference_transformer_base.py:336-387)
@@ -245,6 +261,23 @@ class RaggedTransformer:
         max_blocks = ceil_div(self._state_config.max_context, bs)
         return (KVCacheConfig(block_size=bs, cache_shape=(self.spec.n_layers, self.n_kv, self.d),
                               cache_dtype=self.dtype, max_blocks_per_allocation_group=max_blocks), )
+
+    def recurrent_state_config(self):
+        """Per-layer recurrent state of the model (None: no layer has any)."""
+        return None
+
+    def attention_group(self) -> int:
+        """Query heads per KV head: decides which work items the split-KV decode kernel may take."""
+        return max(1, self.n_q // max(1, self.n_kv))
+
+    def decode_graph_key(self, batch: RaggedBatchWrapper) -> tuple:
+        """Launch geometry of a pure decode step: one CUDA graph serves all steps with the same key."""
+        pick = pick_packed_splits if use_packed_decode(self.n_q, self.n_kv, self.d) else pick_decode_splits
+        return (batch.current_sequences, pick(batch.n_items_small, self.n_kv, batch.max_kv_len_small), batch.rows_per_small_item)
+
+    def graphable_decode(self, batch: RaggedBatchWrapper) -> bool:
+        """May a one-token-per-sequence batch run as a CUDA graph (its launch geometry is what ``decode_graph_key`` says)?"""
+        return batch.n_items_large == 0
 
     def set_state_manager(self, state_manager: DSStateManager) -> None:
         self._state_manager = state_manager
@@ -463,80 +496,55 @@ class RaggedTransformer:
         self._delta_idx = (self._delta_idx + 1) % len(self._delta_bufs)
         return d32
 
-    def forward(self, batch: RaggedBatchWrapper, capture: bool = False, all_logits: bool = False,
-                n_layers_limit: Optional[int] = None,
-                restore_interleave: float = 0.0) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
-        """One ragged forward. Returns ``(logits [n_seqs, vocab], latents)`` where latents is the device view
-        ``[n_layers, n_tokens, hidden]`` of the captured QKV inputs (None when capture is off).
-        ``all_logits``: unembed every token instead of each sequence's last one (``[n_tokens, vocab]``; v1 API).
-        ``n_layers_limit``: run only the first layers (writing their K/V) and return ``(None, latents)`` — the
-        recomputed prefix of a mixed HCache restore plan. With a deferred restore pending, ``restore_interleave``
-        saved layers are projected after each recomputed layer (their transfers complete at that rate), so the
-        copy engine never waits for a free staging slot while the GPU recomputes."""
+    def _embed(self, batch: RaggedBatchWrapper) -> torch.Tensor:
+        """Fill (and return) the residual stream of the batch's tokens with their embeddings."""
         s, w, ops = self.spec, self.w, self.ops
-        T, S = batch.current_tokens, batch.current_sequences
-        if capture and self.latent_buf is None:
-            raise RuntimeError("hidden-state capture was disabled when the model was built")
-        pos, slot = batch.tok_pos(), batch.tok_slot()
-        resid = self.residual[:T]
+        T = batch.current_tokens
+        pos, resid = batch.tok_pos(), self.residual[:T]
         if w.embed_norm_g is not None:   # Bloom: the residual stream starts from the normalised embeddings
             raw = self.embed_tmp[:T]
             ops.embed(batch.input_ids(), w.embed, raw, pos_weight=w.pos_embed, tok_pos=pos, pos_offset=s.learned_pos_offset)
             ops.norm(raw, w.embed_norm_g, resid, beta=w.embed_norm_b, eps=s.norm_eps, layer_norm=True)
         else:
             ops.embed(batch.input_ids(), w.embed, resid, pos_weight=w.pos_embed, tok_pos=pos, pos_offset=s.learned_pos_offset)
-        ln = s.norm == "layer"
-        pending = None
+        return resid
+
+    def _kv_ready(self, li: int) -> None:
+        """Layer ``li`` is about to touch its KV cache (and state): finish what a deferred restore still owes it."""
+        if self._pending_kv is not None:
+            self._kv_step(li)       # deferred reload of this layer's offloaded KV pages
+        if self._pending_restore is not None:
+            self._restore_step(li)  # deferred HCache restore: this layer's K/V must land before its attention
+
+    def _layer(self, li: int, resid: torch.Tensor, pending, xn: torch.Tensor, batch: RaggedBatchWrapper):
+        """One layer. ``pending``: what the previous layer left to be added to the residual stream (folded in by this layer's
+        first norm, which writes ``xn``); returns what this layer leaves."""
+        s, ops = self.spec, self.ops
+        lw = self.w.layers[li]
+        T = batch.current_tokens
         kv = self._state_manager
-        bs = kv.kv_block_size
-        two_norms = (not s.parallel_residual) or s.parallel_two_norms
-        n_run = s.n_layers if n_layers_limit is None else min(n_layers_limit, s.n_layers)
-        for li in range(n_run):
-            lw = w.layers[li]
-            xn = (self.latent_buf[li] if capture else self.xn)[:T]
-            self._norm(resid, lw.norm1_g, xn, beta=lw.norm1_b, delta=pending,
-                       res_out=resid if pending is not None else None)
-            kv_layer = kv.get_cache(li)
-            if self._pending_kv is not None:
-                self._kv_step(li)       # deferred reload of this layer's offloaded KV pages
-            if self._pending_restore is not None:
-                self._restore_step(li)  # deferred HCache restore: this layer's K/V must land before its attention
-            ops.qkv_rope_kv_append(xn, lw.w_qkv, lw.b_qkv, self.qkv_buf[:T], self.q_buf[:T], kv_layer, pos, slot,
-                                   self.inv_freq, self.n_q, self.n_kv, self.d, s.rot_dim, bs, workspace=self.ws_gemm,
-                                   comm=self.comm, tp_wait=self._take_tp_wait())
-            attn = self.attn_buf[:T]
-            ops.attention(self.q_buf[:T], attn, kv_layer, batch, self.n_q, self.n_kv, self.d, self.scale,
-                          ws_small=self.ws_small, ws_large=self.ws_large, alibi=self.alibi, window=s.window_of(li))
-            if s.parallel_residual:
-                xm = xn
-                if two_norms:
-                    xm = self._norm(resid, lw.norm2_g, self.xn2[:T], beta=lw.norm2_b)
-                self._row_parallel(attn, lw.w_o, lw.b_o, T, force_accum=True, last_into_delta=False)
-                pending = self._mlp(xm, lw, T, force_accum=True)
-            else:
-                d1 = self._row_parallel(attn, lw.w_o, lw.b_o, T, force_accum=False)
-                x2 = self._norm(resid, lw.norm2_g, self.xn2[:T], beta=lw.norm2_b, delta=d1, res_out=resid)
-                pending = self._mlp(x2, lw, T, force_accum=False)
-            if n_layers_limit is not None and restore_interleave > 0 and self._pending_restore is not None:
-                st = self._pending_restore
-                target = min(len(st["layers"]), int((li + 1) * restore_interleave))
-                while st["done"] < target:
-                    self._restore_project(st, st["done"])
-                if st["done"] >= len(st["layers"]):
-                    self._pending_restore = None
-        if n_layers_limit is not None:
-            if self._take_tp_wait():
-                self.comm.wait()
-            if pending is not None and pending.dtype == torch.float32:
-                # the partial sums of the last executed layer are not consumed by a norm; under pull-mode TP the
-                # previously consumed buffer is still dirty as well (every rank is past the barrier that follows
-                # the last GEMM, so nobody reads either buffer any more)
-                for b in self._delta_bufs:
-                    b[:T].zero_()
-            return None, (self.latent_buf[:n_run, :T] if capture else None)
-        if self._pending_restore is not None or self._pending_kv is not None:
-            self.finish_pending_restore()
-        # ---- last-token logits ----
+        self._norm(resid, lw.norm1_g, xn, beta=lw.norm1_b, delta=pending, res_out=resid if pending is not None else None)
+        kv_layer = kv.get_cache(li)
+        self._kv_ready(li)
+        ops.qkv_rope_kv_append(xn, lw.w_qkv, lw.b_qkv, self.qkv_buf[:T], self.q_buf[:T], kv_layer, batch.tok_pos(), batch.tok_slot(),
+                               self.inv_freq, self.n_q, self.n_kv, self.d, s.rot_dim, kv.kv_block_size, workspace=self.ws_gemm,
+                               comm=self.comm, tp_wait=self._take_tp_wait())
+        attn = self.attn_buf[:T]
+        ops.attention(self.q_buf[:T], attn, kv_layer, batch, self.n_q, self.n_kv, self.d, self.scale,
+                      ws_small=self.ws_small, ws_large=self.ws_large, alibi=self.alibi, window=s.window_of(li))
+        if s.parallel_residual:
+            xm = xn
+            if s.parallel_two_norms:
+                xm = self._norm(resid, lw.norm2_g, self.xn2[:T], beta=lw.norm2_b)
+            self._row_parallel(attn, lw.w_o, lw.b_o, T, force_accum=True, last_into_delta=False)
+            return self._mlp(xm, lw, T, force_accum=True)
+        d1 = self._row_parallel(attn, lw.w_o, lw.b_o, T, force_accum=False)
+        x2 = self._norm(resid, lw.norm2_g, self.xn2[:T], beta=lw.norm2_b, delta=d1, res_out=resid)
+        return self._mlp(x2, lw, T, force_accum=False)
+
+    def _final_hidden(self, resid: torch.Tensor, pending, T: int) -> torch.Tensor:
+        """Fold the last pending delta in and apply the final norm."""
+        s, w, ops = self.spec, self.w, self.ops
         fin = self.xn2[:T]
         if s.final_norm:
             self._norm(resid, w.final_norm_g, fin, beta=w.final_norm_b, delta=pending)
@@ -554,10 +562,64 @@ class RaggedTransformer:
                 ops.norm(resid, ones, self.xn[:T], delta=pending, zero_delta=True, res_out=fin, eps=s.norm_eps)
         if self._take_tp_wait():
             self.comm.wait()   # the peers' rows of `fin` have landed
+        return fin
+
+    def _drop_pending(self, pending, T: int) -> None:
+        """The partial sums of the last executed layer are not consumed by a norm: clear them. (Under pull-mode TP the
+        previously consumed buffer is still dirty as well; every rank is past the barrier that follows the last GEMM, so
+        nobody reads either buffer any more.)"""
+        if pending is not None and pending.dtype == torch.float32:
+            for b in self._delta_bufs:
+                b[:T].zero_()
+
+    def forward(self, batch: RaggedBatchWrapper, capture: bool = False, all_logits: bool = False,
+                n_layers_limit: Optional[int] = None, restore_interleave: float = 0.0,
+                logit_rows: Optional[torch.Tensor] = None) -> Tuple[Optional[torch.Tensor], Optional[torch.Tensor]]:
+        """One ragged forward. Returns ``(logits [n_seqs, vocab], latents)`` where latents is the device view
+        ``[n_layers, n_tokens, hidden]`` of the captured QKV inputs (None when capture is off).
+        ``all_logits``: unembed every token instead of each sequence's last one (``[n_tokens, vocab]``; v1 API).
+        ``logit_rows``: int32 device tensor of batch rows to unembed instead (empty: no logits, returns None for them).
+        ``n_layers_limit``: run only the first layers (writing their K/V) and return ``(None, latents)`` — the
+        recomputed prefix of a mixed HCache restore plan. With a deferred restore pending, ``restore_interleave``
+        saved layers are projected after each recomputed layer (their transfers complete at that rate), so the
+        copy engine never waits for a free staging slot while the GPU recomputes."""
+        s, w, ops = self.spec, self.w, self.ops
+        T, S = batch.current_tokens, batch.current_sequences
+        if capture and self.latent_buf is None:
+            raise RuntimeError("hidden-state capture was disabled when the model was built")
+        resid = self._embed(batch)
+        pending = None
+        n_run = s.n_layers if n_layers_limit is None else min(n_layers_limit, s.n_layers)
+        for li in range(n_run):
+            pending = self._layer(li, resid, pending, (self.latent_buf[li] if capture else self.xn)[:T], batch)
+            if n_layers_limit is not None and restore_interleave > 0 and self._pending_restore is not None:
+                st = self._pending_restore
+                target = min(len(st["layers"]), int((li + 1) * restore_interleave))
+                while st["done"] < target:
+                    self._restore_project(st, st["done"])
+                if st["done"] >= len(st["layers"]):
+                    self._pending_restore = None
+        if n_layers_limit is not None:
+            if self._take_tp_wait():
+                self.comm.wait()
+            self._drop_pending(pending, T)
+            return None, (self.latent_buf[:n_run, :T] if capture else None)
+        if self._pending_restore is not None or self._pending_kv is not None:
+            self.finish_pending_restore()
+        # ---- last-token logits ----
+        fin = self._final_hidden(resid, pending, T)
+        latents = self.latent_buf[:, :T] if capture else None
         if all_logits:
             out_local = torch.empty((T, self.info.vocab), dtype=self.dtype, device=self.device)
             logits = ops.gemm(fin, w.lm_head, out_local, bias=w.lm_head_b, workspace=self.ws_gemm)
             n_rows = T
+        elif logit_rows is not None:
+            n_rows = logit_rows.numel()
+            if n_rows == 0:
+                return None, latents
+            hidden = ops.gather_rows(fin, logit_rows, torch.empty((n_rows, fin.shape[1]), dtype=fin.dtype, device=self.device))
+            out_local = torch.empty((n_rows, self.info.vocab), dtype=self.dtype, device=self.device)
+            logits = ops.gemm(hidden, w.lm_head, out_local, bias=w.lm_head_b, workspace=self.ws_gemm)
         else:
             hidden = ops.gather_rows(fin, batch.last_rows(), self.hidden_last[:S])
             logits = ops.gemm(hidden, w.lm_head, self.logits_local[:S], bias=w.lm_head_b, workspace=self.ws_gemm,
@@ -565,14 +627,14 @@ class RaggedTransformer:
             n_rows = S
         if self.tp_size > 1:
             ranges = [shard_info(s, r, self.tp_size).vocab_range for r in range(self.tp_size)]
-            if self._tp_fused and not all_logits:
+            if self._tp_fused and not all_logits and logit_rows is None:
                 # vocabulary shards land straight in the final [S, vocab] layout: one pull kernel behind the GEMMs' flags
                 logits = self.comm.gather_logits(logits, self.logits_full[:S], ranges)
             else:
-                full = self.logits_full[:S] if not all_logits else torch.empty((n_rows, s.vocab), dtype=self.dtype,
-                                                                               device=self.device)
+                last = not all_logits and logit_rows is None
+                full = self.logits_full[:S] if last else torch.empty((n_rows, s.vocab), dtype=self.dtype, device=self.device)
                 logits = self.comm.all_gather_logits(logits, full, ranges)
-        return logits, (self.latent_buf[:, :T] if capture else None)
+        return logits, latents
 
     # ------------------------------------------------------------------------------------------------
     # HCache restore
@@ -621,8 +683,7 @@ class RaggedTransformer:
                 if layer_ready is not None:
                     layer_ready(i)
                 lat = torch.cat([l[i] for l in latents], dim=0).to(self.dtype)
-                wk, bk = self.kv_weight(li)
-                ops.restore_kv_proj(lat, wk, bk, kv.get_cache(li), pos, slot, self.inv_freq, self.n_kv, self.d, s.rot_dim, bs)
+                self._restore_layer(li, lat, pos, slot, batch.spans(), batch.n_single_token_seqs)
             return
         self.finish_pending_restore()
         comp = torch.cuda.current_stream()
@@ -631,7 +692,9 @@ class RaggedTransformer:
         # private copy of the per-token metadata: the batch wrapper's buffers are rewritten by the next forward
         self.restore_pos[:T].copy_(pos, non_blocking=True)
         self.restore_slot[:T].copy_(slot, non_blocking=True)
-        st = {"T": T, "layers": layers, "latents": list(latents), "issued": 0, "done": 0, "by_layer": {},
+        spans = self.restore_spans[:batch.current_sequences]
+        spans.copy_(batch.spans(), non_blocking=True)
+        st = {"T": T, "spans": spans, "n_single": batch.n_single_token_seqs, "layers": layers, "latents": list(latents), "issued": 0, "done": 0, "by_layer": {},
               "sharded": bool(sharded), "layer_ready": layer_ready}
         for i, li in enumerate(layers):
             st["by_layer"].setdefault(li, []).append(i)
@@ -640,6 +703,16 @@ class RaggedTransformer:
             self._restore_issue_h2d(st)
         if not defer:
             self.finish_pending_restore()
+
+    def _restore_layer(self, li: int, latents: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, spans: torch.Tensor,
+                       n_single: int) -> None:
+        """Rebuild what layer ``li`` caches for the tokens whose saved hidden states are ``latents`` (``spans`` / ``n_single``:
+        the batch's sequences, as :meth:`RaggedBatchWrapper.spans`; used by layers with recurrent state)."""
+        wk, bk = self.kv_weight(li)
+        kv = self._state_manager
+        self.ops.restore_kv_proj(latents, wk, bk, kv.get_cache(li), pos, slot, self.inv_freq, self.n_kv, self.d, self.spec.rot_dim,
+                                 kv.kv_block_size,
+                                 scratch=self.kv_scratch[:latents.shape[0]] if self.kv_scratch is not None else None)
 
     def _restore_issue_h2d(self, st) -> None:
         """Queue the H2D of the next saved layer into its staging slot (IO stream)."""
@@ -670,8 +743,8 @@ class RaggedTransformer:
         T = st["T"]
         comp = torch.cuda.current_stream()
         comp.wait_event(self.ev_loaded[k])
-        wk, bk = self.kv_weight(li)
         if st["sharded"]:
+            wk, bk = self.kv_weight(li)
             # My slice of this layer has landed in my HBM (the stream waited for the copy): tell the peers, then gather
             # every peer's rows over NVLink behind their flags. Slot reuse needs no second exchange: a peer issues the
             # "landed" signal of layer i+1 only after its gather of layer i, so once MY gather of layer i+1 has passed its
@@ -705,9 +778,7 @@ class RaggedTransformer:
             elif i >= 1 and st["issued"] < len(st["layers"]):
                 self._restore_issue_h2d(st)
             return
-        self.ops.restore_kv_proj(self.restore_stage[k][:T], wk, bk, kv.get_cache(li), self.restore_pos[:T],
-                                 self.restore_slot[:T], self.inv_freq, self.n_kv, self.d, s.rot_dim, kv.kv_block_size,
-                                 scratch=self.kv_scratch[:T] if self.kv_scratch is not None else None)
+        self._restore_layer(li, self.restore_stage[k][:T], self.restore_pos[:T], self.restore_slot[:T], st["spans"], st["n_single"])
         self.ev_consumed[k].record(comp)
         st["done"] = i + 1
         if st["issued"] < len(st["layers"]):

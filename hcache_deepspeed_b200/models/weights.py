@@ -51,6 +51,16 @@ class LayerWeights:
     experts: List[ExpertWeights] = field(default_factory=list)
     shared_expert: Optional[ExpertWeights] = None
     w_shared_gate: Optional[torch.Tensor] = None
+    moe_table: Optional[torch.Tensor] = None      # int32 [vocab, top]: the experts of every token id
+    # stacks of unlike layers (models/hybrid.py): norms behind the sublayers, state-space mixer (fp32 vectors)
+    norm1b_g: Optional[torch.Tensor] = None
+    norm2b_g: Optional[torch.Tensor] = None
+    ssm_conv_w: Optional[torch.Tensor] = None     # [taps, channels]
+    ssm_conv_b: Optional[torch.Tensor] = None
+    ssm_dt_bias: Optional[torch.Tensor] = None
+    ssm_a: Optional[torch.Tensor] = None          # -exp(A_log): the decay rate of each head
+    ssm_d: Optional[torch.Tensor] = None
+    ssm_norm: Optional[torch.Tensor] = None
 
     def tensors(self) -> Dict[str, torch.Tensor]:
         out = {}
@@ -172,6 +182,8 @@ class WeightAssembler:
     # -- sharding of one piece ------------------------------------------------------------------------
     def _shard(self, name: str, t: torch.Tensor) -> Optional[torch.Tensor]:
         s, info, d = self.spec, self.info, self.spec.head_dim
+        if s.layers is not None:
+            return t        # one rank (checked by the executor); heads are laid out per layer when a layer is complete
         r0 = info.tp_rank == 0
         base = name.split(".")[-1] if not name.startswith("moe.") else name
         if name in ("attn.q", "attn.q_b"):
@@ -214,8 +226,11 @@ class WeightAssembler:
             self._maybe_finalize_layer(layer)
 
     # -- completion tracking ----------------------------------------------------------------------------
-    def _required(self) -> List[str]:
+    def _required(self, li: int = 0) -> List[str]:
         s = self.spec
+        if s.layers is not None:
+            from .hybrid import required_pieces
+            return required_pieces(s.layers[li])
         req = ["attn.q", "attn.k", "attn.v", "attn.o", "norm1.g"]
         if s.qkv_bias:
             req += ["attn.q_b", "attn.k_b", "attn.v_b"]
@@ -247,9 +262,15 @@ class WeightAssembler:
         if li in self._done_layers:
             return
         p = self.layers[li]
-        if any(r not in p for r in self._required()):
+        if any(r not in p for r in self._required(li)):
             return
         s = self.spec
+        if s.layers is not None:
+            from .hybrid import layer_weights
+            self.out.layers[li] = layer_weights(s, s.layers[li], p, self.dtype, self.device)
+            self._done_layers.add(li)
+            del self.layers[li]
+            return
         lw = self.out.layers[li]
         lw.norm1_g, lw.norm1_b = self._to(p["norm1.g"]), self._to(p.get("norm1.b"))
         lw.norm2_g, lw.norm2_b = self._to(p.get("norm2.g")), self._to(p.get("norm2.b"))
@@ -285,10 +306,13 @@ class WeightAssembler:
         if missing:
             have = {i: sorted(self.layers.get(i, {})) for i in missing[:2]}
             raise ValueError(f"checkpoint is missing parameters for layers {missing[:8]}; got {have}; "
-                             f"need {self._required()}")
+                             f"need {self._required(missing[0])}")
         if "embed" not in self.top:
             raise ValueError("checkpoint has no token embedding")
         o = self.out
+        if s.layers is not None:
+            from .hybrid import top_weights
+            return top_weights(s, self.top, o, self.dtype, self.device)
         o.embed = self._to(self.top["embed"])
         o.pos_embed = self._to(self.top.get("pos_embed"))
         o.final_norm_g, o.final_norm_b = self._to(self.top.get("final_norm.g")), self._to(self.top.get("final_norm.b"))
@@ -322,6 +346,9 @@ def random_weights(spec: ArchSpec, tp_rank: int = 0, tp_size: int = 1, dtype: to
     """Random-init weights of the right shapes, generated directly on ``device`` in kernel layout (benchmarks
     have no checkpoints). Replicated tensors use a rank-independent seed so TP ranks agree on them."""
     device = device if device is not None else torch.device("cpu")
+    if spec.layers is not None:
+        from .hybrid import random_stack_weights
+        return random_stack_weights(spec, dtype, device, seed, std)
     info = shard_info(spec, tp_rank, tp_size)
     g_shared = torch.Generator(device=device).manual_seed(seed)
     g_rank = torch.Generator(device=device).manual_seed(seed * 1000003 + 17 + tp_rank)

@@ -26,13 +26,18 @@ def _fp8_emulate(a, w):
     return q.view(torch.float8_e4m3fn).float() * s[:, None], w.dequantize()
 
 
+def windowed_len(n_keys: int, window: int, keep_first: int = 0) -> int:
+    """Keys a work item really reads under a sliding window with kept first tokens (one tile of slack at both edges)."""
+    return min(n_keys, window + 256 + (keep_first + 127) // 128 * 128) if window else n_keys
+
+
 class CpuOps:
     name = "cpu-reference"
 
     # ---- linear ---------------------------------------------------------------------------------
-    def gemm(self, a, w, out, bias=None, act=0, gated=False, workspace=None, comm=None, tp_wait=False, tp_signal=False):
+    def gemm(self, a, w, out, bias=None, act=0, gated=False, workspace=None, comm=None, tp_wait=False, tp_signal=False, limit=0.0):
         a, w = _fp8_emulate(a, w)
-        out.copy_(ref.gemm(a, w, bias=bias, act=act, gated=gated, out_dtype=out.dtype))
+        out.copy_(ref.gemm(a, w, bias=bias, act=act, gated=gated, out_dtype=out.dtype, limit=limit))
         return out
 
     def gemm_accum(self, a, w, accum, bias=None, comm=None, tp_signal=False):
@@ -81,13 +86,62 @@ class CpuOps:
             k = ref.rope_rotate_half(k, tok_pos, inv_freq, rot_dim)
         ref.kv_append(kv_layer, k, v, tok_slot)
 
-    def attention(self, q, out, kv_layer, batch, n_q, n_kv, d, scale, ws_small=None, ws_large=None, alibi=None, window=0):
+    def attention(self, q, out, kv_layer, batch, n_q, n_kv, d, scale, ws_small=None, ws_large=None, alibi=None, window=0,
+                  keep_first=0):
         T = q.shape[0]
         q3, o3 = q.view(T, n_q, d), out.view(T, n_q, d)
         for items in (batch.items_small(), batch.items_large()):
             if items.shape[0]:
                 ref.paged_attention(q3, kv_layer, batch.block_tables(), items, n_q, n_kv, scale, out=o3, alibi=alibi,
-                                    window=window)
+                                    window=window, keep_first=keep_first)
+
+    # ---- stacks of unlike layers ----------------------------------------------------------------------
+    def embed_f32(self, ids, weight, out):
+        out.copy_(ref.embed(ids, weight))
+        return out
+
+    def norm_residual(self, resid, gamma, out, delta=None, factor=1.0, post=None, cols=None, eps=1e-5, store_resid=True):
+        x, y = ref.norm_residual(resid, gamma, delta, factor, post, cols, eps)
+        if delta is not None and delta.dtype == torch.float32:
+            delta.zero_()
+        if store_resid:
+            resid.copy_(x)
+        out.copy_(y)
+        return out
+
+    def mixer_in_proj(self, x, w_in, n_attn, proj, q_out, kv_layer, tok_pos, tok_slot, n_q, n_kv, d, block_size, workspace=None):
+        self.qkv_rope_kv_append(x, w_in[:n_attn], None, None, q_out, kv_layer, tok_pos, tok_slot, None, n_q, n_kv, d, d, block_size)
+        if w_in.shape[0] > n_attn:
+            self.gemm(x, w_in[n_attn:], proj[:, n_attn:w_in.shape[0]])
+
+    def state_space(self, proj, lw, m, ssm_state, conv_state, spans, n_single, conv_buf, dt_buf, out):
+        for row0, n, seen, slot in spans.tolist():
+            u = proj[row0:row0 + n]
+            if seen == 0:
+                ssm_state[slot].zero_()
+            xbc = ref.short_conv(u[:, m.inner:m.inner + m.conv_dim], conv_state[slot], lw.ssm_conv_w, lw.ssm_conv_b, seen)
+            xbc = xbc.to(proj.dtype).float()
+            GN = m.groups * m.state
+            dt = torch.nn.functional.softplus(u[:, m.inner + m.conv_dim:].float() + lw.ssm_dt_bias)
+            y = ref.selective_scan(xbc[:, :m.inner].reshape(n, m.heads, m.vdim), xbc[:, m.inner:m.inner + GN].reshape(n, m.groups, m.state),
+                                   xbc[:, m.inner + GN:].reshape(n, m.groups, m.state), dt, lw.ssm_a, lw.ssm_d, ssm_state[slot])
+            out[row0:row0 + n] = y.reshape(n, m.inner)
+        return out
+
+    def gated_norm(self, y, z, weight, out, groups, eps, scale=1.0):
+        out.copy_(ref.gated_norm(y, z, weight, groups, eps, scale))
+        return out
+
+    def table_moe(self, x, ids, lw, f, act, shared, out, bufs):
+        picked = lw.moe_table[ids.long()].long()
+        acc = torch.zeros_like(out) if shared is None else shared.float()
+        for e, ew in enumerate(lw.experts):
+            rows = (picked == e).any(-1).nonzero(as_tuple=False).flatten()
+            if rows.numel():
+                h = ref.gemm(x.index_select(0, rows), ew.w_up, act=act, gated=True, limit=f.limit)
+                acc.index_add_(0, rows, ref.gemm(h, ew.w_down).float() / f.top)
+        out.copy_(acc)
+        return out
 
     # ---- misc ---------------------------------------------------------------------------------------
     def embed(self, ids, weight, out, pos_weight=None, tok_pos=None, pos_offset=0):

@@ -18,9 +18,9 @@ import torch
 
 from . import native
 
-ACT_IDENTITY, ACT_GELU, ACT_RELU, ACT_SILU, ACT_GELU_TANH = 0, 1, 2, 3, 4
+ACT_IDENTITY, ACT_GELU, ACT_RELU, ACT_SILU, ACT_GELU_TANH, ACT_SWIGLU_CLAMPED = 0, 1, 2, 3, 4, 5
 ACT_CODES = {"identity": 0, None: 0, "gelu": 1, "relu": 2, "silu": 3, "gelu_tanh": 4, "gelu_new": 4,
-             "gelu_pytorch_tanh": 4, "swish": 3}
+             "gelu_pytorch_tanh": 4, "swish": 3, "swiglu_clamped": 5}
 
 EPI_STORE, EPI_GATED = 0, 1
 

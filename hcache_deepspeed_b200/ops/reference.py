@@ -29,12 +29,24 @@ def apply_act(x: torch.Tensor, act: int) -> torch.Tensor:
     return x
 
 
+#: sharpness of the sigmoid in the clamped gated unit
+CLAMPED_GLU_ALPHA = 1.702
+
+
+def clamped_glu(g: torch.Tensor, u: torch.Tensor, limit: float) -> torch.Tensor:
+    """Gate bounded above, up bounded on both sides: min(g, L) * sigmoid(alpha * min(g, L)) * (clamp(u, -L, L) + 1)."""
+    g = g.clamp(max=limit)
+    return g * torch.sigmoid(CLAMPED_GLU_ALPHA * g) * (u.clamp(-limit, limit) + 1.0)
+
+
 def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, act: int = 0, gated: bool = False,
-         out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+         out_dtype: Optional[torch.dtype] = None, limit: float = 0.0) -> torch.Tensor:
     y = a.float() @ w.float().t()
     if bias is not None:
         y = y + bias.float()
-    if gated:
+    if gated and act == 5:
+        y = clamped_glu(y[:, 0::2], y[:, 1::2], limit)
+    elif gated:
         y = apply_act(y[:, 0::2], act) * y[:, 1::2]
     else:
         y = apply_act(y, act)
@@ -90,10 +102,10 @@ def gather_kv(kv_cache_layer: torch.Tensor, block_table_row: torch.Tensor, kv_le
 
 def paged_attention(q: torch.Tensor, kv_cache_layer: torch.Tensor, block_tables: torch.Tensor, items: torch.Tensor,
                     n_q_heads: int, n_kv_heads: int, scale: float, out: Optional[torch.Tensor] = None,
-                    alibi: Optional[torch.Tensor] = None, window: int = 0) -> torch.Tensor:
+                    alibi: Optional[torch.Tensor] = None, window: int = 0, keep_first: int = 0) -> torch.Tensor:
     """q: [T, n_q_heads, d]; items: int32 [n, 4] rows (seq, q_row0, n_q, pos0). Causal over absolute positions.
     ``alibi``: [n_q_heads] slopes, score += slope * (key position - query position). ``window`` > 0: a query at position p
-    sees the keys (p - window, p] only."""
+    sees the keys (p - window, p] only, and the first ``keep_first`` positions of its sequence."""
     T, _, d = q.shape
     if out is None:
         out = torch.zeros_like(q)
@@ -111,7 +123,7 @@ def paged_attention(q: torch.Tensor, kv_cache_layer: torch.Tensor, block_tables:
             s = s + alibi.float().to(s.device)[:, None, None] * (kv_pos - q_pos).float()
         s = s.masked_fill(kv_pos > q_pos, float("-inf"))
         if window:
-            s = s.masked_fill(kv_pos <= q_pos - window, float("-inf"))
+            s = s.masked_fill((kv_pos <= q_pos - window) & (kv_pos >= keep_first), float("-inf"))
         p = torch.softmax(s, dim=-1)
         out[q_row0:q_row0 + n_q] = torch.einsum("hqk,khd->qhd", p, v).to(out.dtype)
     return out
@@ -143,3 +155,51 @@ def alibi_slopes(n_heads: int) -> torch.Tensor:
 
 def attention_scale(head_dim: int) -> float:
     return 1.0 / math.sqrt(head_dim)
+
+
+# ---------------------------------------------------------------------------------------------------
+# fp32 residual stream with norms on both sides of a sublayer; state-space mixer; expert choice by table
+# ---------------------------------------------------------------------------------------------------
+def norm_residual(resid: torch.Tensor, gamma: torch.Tensor, delta: Optional[torch.Tensor], factor: float,
+                  post: Optional[torch.Tensor], cols: int, eps: float):
+    """Returns (new fp32 stream, normed stream): stream += rms(factor * delta) * post, then rms(stream) * gamma. Rows hold
+    ``cols`` values and zeros behind them."""
+    x = resid
+    if delta is not None:
+        d = delta.float() * factor
+        x = x + d * torch.rsqrt((d * d).sum(-1, keepdim=True) / cols + eps) * post
+    return x, x * torch.rsqrt((x * x).sum(-1, keepdim=True) / cols + eps) * gamma
+
+
+def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, scale: float = 1.0) -> torch.Tensor:
+    """rms of each of ``groups`` equal parts of y * silu(z), times weight, times scale."""
+    g = y.float() * F.silu(z.float())
+    p = g.reshape(g.shape[0], groups, -1)
+    return (p * torch.rsqrt((p * p).mean(-1, keepdim=True) + eps)).reshape(g.shape) * weight * scale
+
+
+def short_conv(u: torch.Tensor, conv_state: torch.Tensor, w: torch.Tensor, b: torch.Tensor, pos0: int) -> torch.Tensor:
+    """Causal convolution + silu of ``u`` [n, channels] at positions pos0.. of one sequence; ``w`` [taps, channels].
+    ``conv_state`` [taps, channels] is a ring by position modulo taps, advanced in place."""
+    taps, n = w.shape[0], u.shape[0]
+    past = [conv_state[p % taps] if p >= 0 else torch.zeros_like(u[0], dtype=torch.float32) for p in range(pos0 - taps + 1, pos0)]
+    full = torch.cat([torch.stack(past), u.float()]) if past else u.float()
+    out = sum(full[k:k + n] * w[k] for k in range(taps)) + b
+    for i in range(max(0, n - taps), n):
+        conv_state[(pos0 + i) % taps] = u[i].float()
+    return F.silu(out)
+
+
+def selective_scan(x: torch.Tensor, B: torch.Tensor, C: torch.Tensor, dt: torch.Tensor, a: torch.Tensor, d: torch.Tensor,
+                   state: torch.Tensor) -> torch.Tensor:
+    """S <- exp(a dt) S + dt x B^T, y = S C + d x for every token of one sequence. x [n, heads, P], B / C [n, groups, N],
+    dt [n, heads], a / d [heads]; ``state`` [heads, P, N] fp32 is advanced in place."""
+    n, H, P = x.shape
+    rep = H // B.shape[1]
+    y = torch.empty((n, H, P), dtype=torch.float32)
+    for t in range(n):
+        Bt, Ct = B[t].repeat_interleave(rep, 0), C[t].repeat_interleave(rep, 0)
+        xt = x[t].float()
+        state.mul_(torch.exp(a * dt[t])[:, None, None]).add_((dt[t][:, None] * xt)[:, :, None] * Bt.float()[:, None, :])
+        y[t] = (state * Ct.float()[:, None, :]).sum(-1) + d[:, None] * xt
+    return y
