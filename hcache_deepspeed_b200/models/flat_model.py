@@ -87,4 +87,7 @@ def restore_model_weights(flat: torch.Tensor, meta: Dict, device: torch.device) 
         w.layers[li].experts.append(ExpertWeights(d["w_up"], d["w_down"]))
     for li, d in shared.items():
         w.layers[li].shared_expert = ExpertWeights(d["w_up"], d["w_down"])
+    for lw in w.layers:
+        if lw.moe_table is not None:
+            lw.stack_experts()
     return w

@@ -116,11 +116,8 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
     if f is not None:
         lw.norm2_g, lw.norm2b_g = gamma("norm2.g"), gamma("norm2b.g")
         if f.experts:
-            # stacked for the grouped GEMM; the per-expert tensors are views of the stacks
-            ex = [glu(f"moe.experts.{e}.", f.ff) for e in range(f.experts)]
-            up, down = torch.cat([e.w_up for e in ex]), torch.cat([e.w_down for e in ex])
-            nu, nd = ex[0].w_up.shape[0], ex[0].w_down.shape[0]
-            lw.experts = [ExpertWeights(up[e * nu:(e + 1) * nu], down[e * nd:(e + 1) * nd]) for e in range(f.experts)]
+            lw.experts = [glu(f"moe.experts.{e}.", f.ff) for e in range(f.experts)]
+            lw.stack_experts()
             lw.moe_table = p["moe.table"].to(device=device, dtype=torch.int32).contiguous()
             if f.shared_ff:
                 lw.shared_expert = glu("moe.shared.", f.shared_ff)

@@ -32,6 +32,14 @@ class ExpertWeights:
     w_down: torch.Tensor
 
 
+def _stack_of(parts: List[torch.Tensor]) -> torch.Tensor:
+    first, n = parts[0], parts[0].numel()
+    same = first.untyped_storage().data_ptr()
+    if any(t.untyped_storage().data_ptr() != same or t.storage_offset() != first.storage_offset() + i * n for i, t in enumerate(parts)):
+        raise ValueError("expert weights are not consecutive slices of one tensor (see LayerWeights.stack_experts)")
+    return torch.as_strided(first, (first.shape[0] * len(parts), first.shape[1]), (first.shape[1], 1), first.storage_offset())
+
+
 @dataclass
 class LayerWeights:
     norm1_g: Optional[torch.Tensor] = None
@@ -61,6 +69,21 @@ class LayerWeights:
     ssm_a: Optional[torch.Tensor] = None          # -exp(A_log): the decay rate of each head
     ssm_d: Optional[torch.Tensor] = None
     ssm_norm: Optional[torch.Tensor] = None
+
+    def stack_experts(self) -> None:
+        """Store the experts as consecutive slices of one tensor per matrix, the operands of the grouped GEMM."""
+        up, down = torch.cat([e.w_up for e in self.experts]), torch.cat([e.w_down for e in self.experts])
+        nu, nd = self.experts[0].w_up.shape[0], self.experts[0].w_down.shape[0]
+        self.experts = [ExpertWeights(up[e * nu:(e + 1) * nu], down[e * nd:(e + 1) * nd]) for e in range(len(self.experts))]
+
+    @property
+    def moe_up(self) -> torch.Tensor:
+        """All experts' ``w_up`` as one matrix (they are loaded as consecutive slices of one tensor)."""
+        return _stack_of([e.w_up for e in self.experts])
+
+    @property
+    def moe_down(self) -> torch.Tensor:
+        return _stack_of([e.w_down for e in self.experts])
 
     def tensors(self) -> Dict[str, torch.Tensor]:
         out = {}

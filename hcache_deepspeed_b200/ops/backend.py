@@ -186,7 +186,7 @@ class CudaOps:
             bufs[K] = (torch.empty(max_tokens, K, dtype=torch.uint8, device=device),
                        torch.empty(max_tokens, dtype=torch.float32, device=device))
 
-    def gemm(self, a, w, out, bias=None, act=0, gated=False, workspace=None, comm=None, tp_wait=False, tp_signal=False):
+    def gemm(self, a, w, out, bias=None, act=0, gated=False, workspace=None, comm=None, tp_wait=False, tp_signal=False, limit=0.0):
         """``tp_wait``: ``a`` was all-gathered into this GPU's buffer by the peers' norm kernels — the first kernel that
         reads it acquires their flags. ``tp_signal``: the GEMM's last CTA releases ``out`` to the peers."""
         if isinstance(w, Fp8Weight):
@@ -200,7 +200,7 @@ class CudaOps:
         if tp_wait or tp_signal:
             comm.arm(wait=tp_wait, signal=tp_signal)
         return self.k.gemm(a, w, bias=bias, act=act, gated=gated, out=out,
-                           workspace=workspace if a.shape[0] <= 128 else None)
+                           workspace=workspace if a.shape[0] <= 128 else None, limit=limit)
 
     def gemm_accum(self, a, w, accum, bias=None, comm=None, tp_signal=False):
         """``accum (fp32) += a @ w.T``. ``tp_signal`` (tensor parallel): the kernel's last CTA releases the partial sums
@@ -262,6 +262,9 @@ class CudaOps:
             scratch = scratch[:latents.shape[0]]
             self.gemm(latents, w_kv, scratch, bias=b_kv)
             self.k.rope_kv_append(scratch, scratch, kv_layer, tok_pos, tok_slot, inv_freq, 0, n_kv, d, rot_dim, block_size)
+        elif latents.dtype == torch.float32:
+            self.k.gemm(latents, w_kv, out=scratch)
+            self.k.kv_append_generic(scratch, scratch, kv_layer, tok_slot, 0, n_kv, d, block_size)
         elif d in (64, 128) and (inv_freq is None or rot_dim == d):
             self.k.restore_kv_proj(latents, w_kv, kv_layer, tok_pos, tok_slot, inv_freq, n_kv, d, block_size, bias_kv=b_kv)
         else:
@@ -270,30 +273,75 @@ class CudaOps:
             self.k.gemm(latents, w_kv, bias=b_kv, out=scratch)
             self.k.rope_kv_append(scratch, scratch, kv_layer, tok_pos, tok_slot, inv_freq, 0, n_kv, d, rot_dim, block_size)
 
-    def attention(self, q, out, kv_layer, batch, n_q, n_kv, d, scale, ws_small=None, ws_large=None, alibi=None, window=0):
+    def attention(self, q, out, kv_layer, batch, n_q, n_kv, d, scale, ws_small=None, ws_large=None, alibi=None, window=0,
+                  keep_first=0):
         k = self.k
         bs = batch.block_size
+        if q.dtype == torch.float32 or d not in (64, 128):
+            k.paged_attention_generic(q, out, kv_layer, batch.block_tables(), batch.tokens_to_seq(), batch.tok_pos(), n_q, n_kv, d, bs,
+                                      scale, window=window, keep_first=keep_first)
+            return
         # with a sliding window an item reads at most window + one tile of keys: size the KV split for that
-        seen = (lambda n_kv_tokens: min(n_kv_tokens, window + 256)) if window else (lambda n_kv_tokens: n_kv_tokens)
+        seen = lambda n_kv_tokens: windowed_len(n_kv_tokens, window, keep_first)  # noqa: E731
+        opts = dict(alibi=alibi, window=window, keep_first=keep_first)
         if batch.n_items_small:
             n = batch.n_items_small
             if use_packed_decode(n_q, n_kv, d):
                 # grouped-query decode: the group's query heads share one pass over the KV pages, on the tensor cores
                 splits = pick_packed_splits(n, n_kv, seen(batch.max_kv_len_small))
                 k.paged_attention_prefill(q, out, kv_layer, batch.block_tables(), batch.items_small(), n, n_q, n_kv, d, bs,
-                                          scale, n_splits=splits, workspace=ws_large if splits > 1 else None, packed=True,
-                                          alibi=alibi, window=window)
+                                          scale, n_splits=splits, workspace=ws_large if splits > 1 else None, packed=True, **opts)
             else:
                 splits = pick_decode_splits(n, n_kv, seen(batch.max_kv_len_small))
                 k.paged_attention_splitkv(q, out, kv_layer, batch.block_tables(), batch.items_small(), n,
-                                          batch.rows_per_small_item, n_q, n_kv, d, bs, splits, scale, ws_small, alibi=alibi,
-                                          window=window)
+                                          batch.rows_per_small_item, n_q, n_kv, d, bs, splits, scale, ws_small, **opts)
         if batch.n_items_large:
             n = batch.n_items_large
             splits = pick_prefill_splits(n, n_q, seen(batch.max_kv_len_large))
             k.paged_attention_prefill(q, out, kv_layer, batch.block_tables(), batch.items_large(), n, n_q, n_kv, d, bs,
-                                      scale, n_splits=splits, workspace=ws_large if splits > 1 else None, alibi=alibi,
-                                      window=window)
+                                      scale, n_splits=splits, workspace=ws_large if splits > 1 else None, **opts)
+
+    # ---- stacks of unlike layers ----------------------------------------------------------------------
+    def embed_f32(self, ids, weight, out):
+        return self.k.embed_f32(ids, weight, out)
+
+    def norm_residual(self, resid, gamma, out, **kw):
+        return self.k.norm_residual(resid, gamma, out, **kw)
+
+    def mixer_in_proj(self, x, w_in, n_attn, proj, q_out, kv_layer, tok_pos, tok_slot, n_q, n_kv, d, block_size, workspace=None):
+        """Every projection that reads the layer's input: Q to ``q_out``, K / V to their pages, the rest to ``proj``'s columns
+        behind the first ``n_attn``. Decode-size batches stream all weights in ONE GEMM; larger ones keep the QKV rows' fused
+        paged epilogue and run the others as a second GEMM."""
+        k, T, n_in = self.k, x.shape[0], w_in.shape[0]
+        if x.dtype != torch.float32 and d in (64, 128) and T >= self.FUSED_QKV_MIN_TOKENS:
+            k.qkv_rope_proj(x, w_in[:n_attn], q_out, kv_layer, tok_pos, tok_slot, None, n_q, n_kv, d, block_size)
+            if n_in > n_attn:
+                k.gemm(x, w_in[n_attn:], out=proj[:, n_attn:n_in])
+            return
+        self.gemm(x, w_in, proj[:, :n_in], workspace=workspace)
+        if x.dtype == torch.float32:
+            k.kv_append_generic(proj, q_out, kv_layer, tok_slot, n_q, n_kv, d, block_size)
+        else:
+            k.rope_kv_append(proj, q_out, kv_layer, tok_pos, tok_slot, None, n_q, n_kv, d, d, block_size)
+
+    def state_space(self, proj, lw, m, ssm_state, conv_state, spans, n_single, conv_buf, dt_buf, out):
+        return self.k.state_space(proj, lw.ssm_conv_w, lw.ssm_conv_b, lw.ssm_dt_bias, lw.ssm_a, lw.ssm_d, ssm_state, conv_state, spans,
+                                  n_single, m.groups, conv_buf, dt_buf, out)
+
+    def gated_norm(self, y, z, weight, out, groups, eps, scale=1.0):
+        return self.k.gated_norm(y, z, weight, out, groups, eps, scale)
+
+    def table_moe(self, x, ids, lw, f, act, shared, out, bufs):
+        """Experts by token id: route -> scatter -> grouped GEMM (gated) -> grouped GEMM -> combine with the shared expert."""
+        k, T, E = self.k, x.shape[0], f.experts
+        rows = k.moe_padded_rows(T, E, f.top)
+        xs, hs, ys = bufs["xs"][:rows], bufs["hs"][:rows], bufs["ys"][:rows]
+        ids_e, off, slots = bufs["expert_ids"][:T], bufs["offsets"][:T], bufs["mapped_slots"][:T]
+        k.moe_table_route(ids, lw.moe_table, E, bufs["scores"][:T], ids_e, off, bufs["counts"])
+        k.moe_scatter(x, xs, ids_e, off, bufs["counts"], bufs["pad_off"], slots, f.top)
+        k.moe_gemm(xs, lw.moe_up, bufs["pad_off"], E, hs, act=act, gated=True, limit=f.limit)
+        k.moe_gemm(hs, lw.moe_down, bufs["pad_off"], E, ys)
+        return k.moe_combine(ys, slots, bufs["scores"][:T], shared, out)
 
     def embed(self, ids, weight, out, pos_weight=None, tok_pos=None, pos_offset=0):
         return self.k.embed(ids, weight, out, pos_weight=pos_weight, tok_pos=tok_pos, pos_offset=pos_offset)

@@ -47,6 +47,8 @@ struct PrefillArgs {
     float* ws_o;        // [n_items][n_q_heads][n_splits][128][D]
     const float* alibi; // [n_q_heads] ALiBi slopes (natural-log units) or nullptr
     int window;         // sliding-window attention: a query at position p sees keys (p - window, p]; 0 = unlimited
+    int keep_first;     // with a window: the first keep_first positions stay visible to every later query
+    int64_t out_ld;     // elements between the output rows of two tokens
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -102,14 +104,18 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     const int kv_len = item.pos0 + item.n_q;
     const int tiles_total = (kv_len + kPfTok - 1) / kPfTok;
     // sliding window: key tiles wholly before the FIRST query's window are skipped (later rows see even less of them)
+    // (the tiles of the kept first tokens come before them: live tile i is key tile i, or i + tiles_skip behind the kept ones)
     const int tile_first = a.window > 0 ? max(0, item.pos0 - a.window + 1) / kPfTok : 0;
-    const int tiles_live = tiles_total - tile_first;
+    const int tiles_keep = min((a.keep_first + kPfTok - 1) / kPfTok, tile_first);
+    const int tiles_skip = tile_first - tiles_keep;
+    const int tiles_live = tiles_total - tiles_skip;
     const int tps = (tiles_live + a.n_splits - 1) / a.n_splits;
     const int eff_splits = (tiles_live + tps - 1) / tps;
     const int split = blockIdx.z;
     if (split >= eff_splits) return;
-    const int t0 = tile_first + split * tps;
-    const int n_tiles = min(tiles_total, t0 + tps) - t0;  // tiles of this split: absolute index t0 + ti
+    const int t0 = split * tps;
+    const int n_tiles = min(tiles_live, t0 + tps) - t0;  // tiles of this split: live index t0 + ti
+    auto key_tile = [&](int ti) { return t0 + ti < tiles_keep ? t0 + ti : t0 + ti + tiles_skip; };
     const int bs = a.block_size;
     const int bps = kPfTok / bs;
 
@@ -161,7 +167,7 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
                 for (int b = 0; b < bps; ++b) {
                     // past the end of the sequence re-load its last page: masked out later, but keeps
                     // every V value that meets a zero probability finite (0 * NaN would poison the row)
-                    const int bi = min((t0 + ti) * bps + b, last_blk_idx);
+                    const int bi = min(key_tile(ti) * bps + b, last_blk_idx);
                     const int blk = table[bi];
                     const int krow = ((blk * 2 + 0) * a.n_kv_heads + kvh) * bs;
                     const int vrow = ((blk * 2 + 1) * a.n_kv_heads + kvh) * bs;
@@ -244,10 +250,11 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         constexpr float kRescaleThreshold = 8.0f;    // log2 units: probabilities stay below 2^8 against a stale max
         auto pair_sync = [&]() { asm volatile("bar.sync %0, 64;" ::"r"(1 + quad) : "memory"); };
         for (int ti = 0; ti < n_tiles; ++ti) {
-            const int tok0 = (t0 + ti) * kPfTok + half * HC;
+            const int tile0 = key_tile(ti) * kPfTok;
+            const int tok0 = tile0 + half * HC;
             // warp-uniform: the tile reaches past the first query (causal edge) or starts before the last query's window
-            const bool need_mask = (t0 + ti) * kPfTok + kPfTok - 1 > item.pos0 ||
-                                   (a.window > 0 && (t0 + ti) * kPfTok <= item.pos0 + item.n_q - 1 - a.window);
+            const bool need_mask = tile0 + kPfTok - 1 > item.pos0 ||
+                                   (a.window > 0 && tile0 <= item.pos0 + item.n_q - 1 - a.window);
             const int win_lo = a.window > 0 ? q_pos - a.window : -(1 << 30);   // keys at or before this position are hidden
             mbar_wait(s_full, ti & 1);
             tc_fence_after();
@@ -288,7 +295,7 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
 #pragma unroll
                 for (int j = 0; j < HC; ++j) {
                     const int kv_pos = tok0 + j;
-                    const float sv = (kv_pos <= q_pos && kv_pos < kv_len && kv_pos > win_lo) ? __uint_as_float(sr[j]) : -INFINITY;
+                    const float sv = (kv_pos <= q_pos && kv_pos < kv_len && (kv_pos > win_lo || kv_pos < a.keep_first)) ? __uint_as_float(sr[j]) : -INFINITY;
                     sr[j] = __float_as_uint(sv);
                     tmax = fmaxf(tmax, sv);
                 }
@@ -374,7 +381,7 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         tc_fence_before();
         const bool row_valid = r < n_live_rows;
         char* dst = reinterpret_cast<char*>(a.out) +
-                    ((static_cast<int64_t>(item.q_row0 + r_tok) * a.n_q_heads + r_head) * D + half * HD2) * 2;
+                    (static_cast<int64_t>(item.q_row0 + r_tok) * a.out_ld + r_head * D + half * HD2) * 2;
         if (eff_splits == 1) {
             if (row_valid) {
                 const float inv = 1.0f / l_run;
@@ -503,11 +510,14 @@ static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tkv, const P
 using namespace hds;
 
 static inline int64_t pf_align256(int64_t x) { return (x + 255) & ~int64_t(255); }
+// The tickets lead the scratch and must read zero at every launch: one region size for all problems, so that no launch finds
+// another one's partial sums there (see counter_bytes in attention_splitkv.cu).
+static inline int64_t ticket_bytes(int64_t units) { return pf_align256((units > 4096 ? units : 4096) * 8 * 4); }
 
 extern "C" int64_t hds_paged_attention_prefill_workspace_bytes(int n_items, int n_q_heads, int head_dim, int n_splits) {
     if (n_splits <= 1) return 0;
     const int64_t units = static_cast<int64_t>(n_items) * n_q_heads;
-    return pf_align256(units * 8 * 4) + pf_align256(units * n_splits * 128 * 2 * 4) +
+    return ticket_bytes(units) + pf_align256(units * n_splits * 128 * 2 * 4) +
            pf_align256(units * n_splits * 128 * head_dim * 4);
 }
 
@@ -522,11 +532,15 @@ static int attention_tc_impl(bool packed, const void* q, void* out, const void* 
     HDS_REQUIRE(dtype == 0 || dtype == 1, "paged_attention_prefill: dtype must be 0 (bf16) or 1 (fp16)");
     const float* alibi = attn_take_alibi();
     const int window = attn_take_window();
+    const int keep_first = attn_take_keep_first();
+    const int64_t out_ld = attn_take_out_stride();
     if (n_items == 0) return HDS_OK;
     PrefillArgs a;
     memset(&a, 0, sizeof(a));
     a.alibi = alibi;
     a.window = window;
+    a.keep_first = window > 0 ? keep_first : 0;
+    a.out_ld = out_ld > 0 ? out_ld : static_cast<int64_t>(n_q_heads) * head_dim;
     a.out = out;
     a.block_tables = block_tables;
     a.items = items;
@@ -548,8 +562,8 @@ static int attention_tc_impl(bool packed, const void* q, void* out, const void* 
         const int64_t units = static_cast<int64_t>(n_items) * grid_heads;
         char* ws = reinterpret_cast<char*>(workspace);
         a.tickets = reinterpret_cast<int32_t*>(ws);
-        a.ws_ml = reinterpret_cast<float*>(ws + pf_align256(units * 8 * 4));
-        a.ws_o = reinterpret_cast<float*>(ws + pf_align256(units * 8 * 4) + pf_align256(units * n_splits * 128 * 2 * 4));
+        a.ws_ml = reinterpret_cast<float*>(ws + ticket_bytes(units));
+        a.ws_o = reinterpret_cast<float*>(ws + ticket_bytes(units) + pf_align256(units * n_splits * 128 * 2 * 4));
     }
     CUtensorMap tq, tkv;
     int rc;
@@ -570,7 +584,7 @@ static int attention_tc_impl(bool packed, const void* q, void* out, const void* 
     if (packed)
         return dtype == 0 ? launch_prefill<128, true, true>(tq, tkv, a, n_items, s)
                           : launch_prefill<128, false, true>(tq, tkv, a, n_items, s);
-    if (head_dim == 128 && block_size <= 64 && alibi == nullptr && window == 0 && prefill64_enabled())   // no ALiBi / window there
+    if (head_dim == 128 && block_size <= 64 && alibi == nullptr && window == 0 && out_ld == 0 && prefill64_enabled())   // no ALiBi / window / strided rows there
         return dtype == 0 ? launch_prefill64<true>(tq, tkv, a, n_items, s) : launch_prefill64<false>(tq, tkv, a, n_items, s);
     if (head_dim == 128)
         return dtype == 0 ? launch_prefill<128, true>(tq, tkv, a, n_items, s)

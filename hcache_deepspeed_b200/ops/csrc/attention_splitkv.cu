@@ -41,6 +41,8 @@ struct AttnArgs {
     int consumer_warps; // 8 (one CTA per SM) or 4 (two CTAs per SM); host-side choice, see attn_pick_warps
     const float* alibi; // [n_q_heads] ALiBi slopes (natural-log units) or nullptr: score += slope * (key pos - query pos)
     int window;         // sliding-window attention: a query at position p sees keys (p - window, p]; 0 = unlimited
+    int keep_first;     // with a window: the first keep_first positions stay visible to every later query
+    int64_t out_ld;     // elements between the output rows of two tokens
 };
 
 template <int D, int W>
@@ -93,13 +95,16 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
     const int kv_len = item.pos0 + item.n_q;
     const int tiles_total = (kv_len + kAttnTok - 1) / kAttnTok;
     // sliding window: tiles that lie wholly before the first query's window are never loaded
+    // (the tiles of the kept first tokens are visited before them: live tile i is tile i, or i + skipped behind the kept ones)
     const int tile_first = a.window > 0 ? max(0, item.pos0 - a.window + 1) / kAttnTok : 0;
-    const int tiles_live = tiles_total - tile_first;
+    const int tiles_keep = min((a.keep_first + kAttnTok - 1) / kAttnTok, tile_first);
+    const int tiles_skip = tile_first - tiles_keep;
+    const int tiles_live = tiles_total - tiles_skip;
     const int tps = (tiles_live + a.n_splits - 1) / a.n_splits;
     const int eff_splits = (tiles_live + tps - 1) / tps;
     if (split >= eff_splits) return;
-    const int t0 = tile_first + split * tps;
-    const int t1 = min(tiles_total, t0 + tps);
+    const int t0 = split * tps;
+    const int t1 = min(tiles_live, t0 + tps);
     const int bs = a.block_size;
 
     if (tid == 0) {
@@ -140,7 +145,7 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
                 mbar_wait(&empty_bar[stage], phase ^ 1);
                 uint8_t* kdst = stages + stage * attn_stage_bytes<D, W>();
                 uint8_t* vdst = kdst + TILE_BYTES;
-                const int tok0 = ti * kAttnTok;
+                const int tok0 = (ti < tiles_keep ? ti : ti + tiles_skip) * kAttnTok;
                 const int n_tok = min(kAttnTok, kv_len - tok0);
                 const int box = bs < kAttnTok ? bs : kAttnTok;   // rows per TMA box (host builds the map with it)
                 const int nb = (n_tok + box - 1) / box;
@@ -182,7 +187,7 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
         for (int ti = t0; ti < t1; ++ti) {
             const uint8_t* ktile = stages + stage * attn_stage_bytes<D, W>();
             const uint8_t* vtile = ktile + TILE_BYTES;
-            const int tok0 = ti * kAttnTok;
+            const int tok0 = (ti < tiles_keep ? ti : ti + tiles_skip) * kAttnTok;
             const int n_tok = min(kAttnTok, kv_len - tok0);
             const int n_mine = min(16, max(0, n_tok - warp * 16));  // valid tokens of this warp's strip (uniform)
             mbar_wait(&full_bar[stage], phase);
@@ -221,7 +226,7 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
                     float sc = part[r] + __shfl_xor_sync(0xffffffffu, part[r], 16);
                     const int q_pos = item.pos0 + r / G;
                     const bool ok = (j < n_mine) && (tok0 + rt <= q_pos) && (r < rows) &&
-                                    (a.window <= 0 || tok0 + rt > q_pos - a.window);
+                                    (a.window <= 0 || tok0 + rt > q_pos - a.window || tok0 + rt < a.keep_first);
                     sc = ok ? fmaf(slope[r], static_cast<float>(tok0 + rt - q_pos), sc) : -INFINITY;
                     float mx = sc;
 #pragma unroll
@@ -305,7 +310,7 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
         }
         if (eff_splits == 1) {
             const int qi = r / G, gg = r % G;
-            store_scalar<kBf16>(a.out, (static_cast<int64_t>(item.q_row0 + qi) * a.n_q_heads + kvh * G + gg) * D + dd,
+            store_scalar<kBf16>(a.out, static_cast<int64_t>(item.q_row0 + qi) * a.out_ld + (kvh * G + gg) * D + dd,
                                 o / l);
         } else {
             a.ws_o[((ws_base + split) * R + r) * D + dd] = o;
@@ -339,13 +344,17 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
             o += w * __ldcg(&a.ws_o[((ws_base + s) * R + r) * D + dd]);
         }
         const int qi = r / G, gg = r % G;
-        store_scalar<kBf16>(a.out, (static_cast<int64_t>(item.q_row0 + qi) * a.n_q_heads + kvh * G + gg) * D + dd,
+        store_scalar<kBf16>(a.out, static_cast<int64_t>(item.q_row0 + qi) * a.out_ld + (kvh * G + gg) * D + dd,
                             o / l);
     }
     if (tid == 0) a.counters[item_idx * a.n_kv_heads + kvh] = 0;
 }
 
 static inline int64_t align256(int64_t x) { return (x + 255) & ~int64_t(255); }
+// Arrival counters come first in the scratch and must read zero at every launch, so their region may not grow into what
+// launches of other sizes used for partial sums: it has one size for all problems up to kCounterUnits (item, KV head) pairs.
+constexpr int64_t kCounterUnits = 65536;
+static inline int64_t counter_bytes(int64_t units) { return align256((units > kCounterUnits ? units : kCounterUnits) * 4); }
 
 template <int D, int R, bool kBf16, int W>
 static int launch_splitkv_w(const CUtensorMap& tm, const AttnArgs& a, int n_items, cudaStream_t s) {
@@ -394,6 +403,8 @@ static inline int attn_pick_warps(int64_t ctas) {
 // ALiBi slopes for the NEXT paged-attention launch of this thread (either kernel family); consumed by that launch.
 static thread_local const float* g_next_alibi = nullptr;
 static thread_local int g_next_window = 0;
+static thread_local int g_next_keep_first = 0;
+static thread_local int64_t g_next_out_stride = 0;
 const float* hds::attn_take_alibi() {
     const float* p = g_next_alibi;
     g_next_alibi = nullptr;
@@ -405,7 +416,30 @@ int hds::attn_take_window() {
     return w;
 }
 
+int hds::attn_take_keep_first() {
+    const int k = g_next_keep_first;
+    g_next_keep_first = 0;
+    return k;
+}
+int64_t hds::attn_take_out_stride() {
+    const int64_t s = g_next_out_stride;
+    g_next_out_stride = 0;
+    return s;
+}
+
 using namespace hds;
+
+extern "C" int hds_attention_next_keep_first(int keep_first) {
+    HDS_REQUIRE(keep_first >= 0, "hds_attention_next_keep_first: keep_first >= 0");
+    g_next_keep_first = keep_first;
+    return HDS_OK;
+}
+
+extern "C" int hds_attention_next_out_stride(int64_t elements) {
+    HDS_REQUIRE(elements >= 0 && elements % 8 == 0, "hds_attention_next_out_stride: a multiple of 8 elements");
+    g_next_out_stride = elements;
+    return HDS_OK;
+}
 
 extern "C" int hds_attention_next_alibi(const float* slopes) {
     g_next_alibi = slopes;
@@ -423,7 +457,7 @@ extern "C" int64_t hds_paged_attention_splitkv_workspace_bytes(int n_items, int 
     (void)n_q_heads;
     const int R = rows_bucket(rows_per_item);
     const int64_t units = static_cast<int64_t>(n_items) * n_kv_heads;
-    return align256(units * 4) + align256(units * max_splits * R * 2 * 4) + align256(units * max_splits * R * head_dim * 4);
+    return counter_bytes(units) + align256(units * max_splits * R * 2 * 4) + align256(units * max_splits * R * head_dim * 4);
 }
 
 extern "C" int hds_paged_attention_splitkv(const void* q, void* out, const void* kv_cache_layer,
@@ -434,6 +468,8 @@ extern "C" int hds_paged_attention_splitkv(const void* q, void* out, const void*
                                                 int64_t workspace_bytes, int dtype, void* stream) {
     const float* alibi = attn_take_alibi();
     const int window = attn_take_window();
+    const int keep_first = attn_take_keep_first();
+    const int64_t out_ld = attn_take_out_stride();
     HDS_REQUIRE(head_dim == 64 || head_dim == 128, "paged_attention_splitkv: head_dim must be 64 or 128");
     HDS_REQUIRE(block_size == 16 || block_size == 32 || block_size == 64 || block_size == 128,
                 "paged_attention_splitkv: block_size must be 16/32/64/128");
@@ -462,11 +498,13 @@ extern "C" int hds_paged_attention_splitkv(const void* q, void* out, const void*
     a.scale_log2 = scale * 1.4426950408889634f;
     a.alibi = alibi;
     a.window = window;
+    a.keep_first = window > 0 ? keep_first : 0;
+    a.out_ld = out_ld > 0 ? out_ld : static_cast<int64_t>(n_q_heads) * head_dim;
     const int64_t units = static_cast<int64_t>(n_items) * n_kv_heads;
     char* ws = reinterpret_cast<char*>(workspace);
     a.counters = reinterpret_cast<int32_t*>(ws);
-    a.ws_ml = reinterpret_cast<float*>(ws + align256(units * 4));
-    a.ws_o = reinterpret_cast<float*>(ws + align256(units * 4) + align256(units * n_splits * R * 2 * 4));
+    a.ws_ml = reinterpret_cast<float*>(ws + counter_bytes(units));
+    a.ws_o = reinterpret_cast<float*>(ws + counter_bytes(units) + align256(units * n_splits * R * 2 * 4));
     CUtensorMap tm;
     const uint64_t rows = static_cast<uint64_t>(num_blocks) * 2 * n_kv_heads * block_size;
     a.consumer_warps = attn_pick_warps(units * n_splits);
@@ -493,7 +531,7 @@ extern "C" int hds_paged_attention_splitkv(const void* q, void* out, const void*
 // Cost and limits, so nobody is surprised:
 //   * the array is part of the library image: every GPU that loads libhds_b200.so holds
 //     HDS_STATIC_SCRATCH_BYTES (8 MiB) of device memory until the process exits, used or not;
-//   * a problem whose scratch need (hds_paged_attention_splitkv_workspace_bytes) exceeds that size is
+//   * a problem whose partial sums and counters exceed that size is
 //     refused with HDS_ERR_TOO_LARGE (-4) and a message saying how much was needed — lower n_splits or
 //     n_items, or use the caller-scratch entry point;
 //   * every call on a device shares the one array and finds whatever the previous call left in it. The
@@ -548,8 +586,9 @@ extern "C" int hds_paged_attention_splitkv_static(const void* q, void* out, cons
     HDS_REQUIRE(n_splits >= 1 && n_splits <= 64, "paged_attention_splitkv_static: n_splits in [1,64]");
     HDS_REQUIRE(dtype == 0 || dtype == 1, "paged_attention_splitkv_static: dtype must be 0 (bf16) or 1 (fp16)");
     if (n_items == 0) return HDS_OK;
-    const int64_t need =
-        hds_paged_attention_splitkv_workspace_bytes(n_items, n_q_heads, n_kv_heads, head_dim, n_splits, rows_per_item);
+    const int R = rows_bucket(rows_per_item);
+    const int64_t units = static_cast<int64_t>(n_items) * n_kv_heads;
+    const int64_t need = align256(units * 4) + align256(units * n_splits * R * 2 * 4) + align256(units * n_splits * R * head_dim * 4);
     if (need > HDS_STATIC_SCRATCH_BYTES) {
         char b[256];
         snprintf(b, sizeof(b),
@@ -563,8 +602,6 @@ extern "C" int hds_paged_attention_splitkv_static(const void* q, void* out, cons
     int rc = static_scratch_address(&ws);
     if (rc) return rc;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    const int R = rows_bucket(rows_per_item);
-    const int64_t units = static_cast<int64_t>(n_items) * n_kv_heads;
     // the counters must read zero when the kernel starts; the previous call may have left partial sums here
     HDS_CHECK_CUDA(cudaMemsetAsync(ws, 0, static_cast<size_t>(align256(units * 4)), s));
     AttnArgs a;
@@ -578,6 +615,7 @@ extern "C" int hds_paged_attention_splitkv_static(const void* q, void* out, cons
     a.n_kv_heads = n_kv_heads;
     a.block_size = block_size;
     a.n_splits = n_splits;
+    a.out_ld = static_cast<int64_t>(n_q_heads) * head_dim;
     a.scale_log2 = scale * 1.4426950408889634f;
     a.counters = reinterpret_cast<int32_t*>(ws);
     a.ws_ml = reinterpret_cast<float*>(ws + align256(units * 4));

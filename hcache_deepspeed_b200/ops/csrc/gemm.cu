@@ -206,6 +206,7 @@ static int launch_skinny(int epi, bool bf16, const void* X, int64_t ldx, const v
     a.splits = splits;
     a.kb_per_split = per;
     a.act = act;
+    a.act_limit = gemm_take_act_limit();
     a.out = out; a.ldo = ldo; a.bias = bias;
     a.accum = accum; a.ld_accum = ld_accum;
     a.sync = tp_take_armed();
@@ -283,6 +284,17 @@ static int grid_for(const GemmArgs& g, int bn) {
 
 using namespace hds;
 
+static thread_local float g_next_act_limit = 0.0f;
+float hds::gemm_take_act_limit() {
+    const float l = g_next_act_limit;
+    g_next_act_limit = 0.0f;
+    return l;
+}
+extern "C" int hds_gemm_next_act_limit(float limit) {
+    g_next_act_limit = limit;
+    return HDS_OK;
+}
+
 extern "C" const char* hds_last_error(void) { return g_last_error; }
 
 static inline int64_t align256(int64_t x) { return (x + 255) & ~int64_t(255); }
@@ -330,6 +342,7 @@ extern "C" int hds_gemm(const void* A, int64_t lda, const void* W, int64_t ldw, 
     int rc = prepare(g, ops, A, lda, W, ldw, M, N, K, dtype == 0, bn, splits);
     if (rc) return rc;
     g.act = act;
+    g.act_limit = gemm_take_act_limit();
     g.out = out;
     g.ldo = ldo;
     g.bias = bias;
@@ -400,6 +413,7 @@ extern "C" int hds_moe_gemm(const void* A, int64_t lda, const void* W_stacked, i
                           static_cast<uint64_t>(ldw) * 2, kGemmBK, bn, dtype == 0);
     if (rc) return rc;
     g.act = act;
+    g.act_limit = gemm_take_act_limit();
     g.out = out;
     g.ldo = ldo;
     g.group_pad_off = pad_off;

@@ -330,6 +330,7 @@ int gemm_2sm_dispatch(const void* A, int64_t lda_bytes, const float* a_scale, co
     fa.g.N = N;
     fa.g.K = K;
     fa.g.act = act;
+    fa.g.act_limit = gemm_take_act_limit();
     fa.g.out = out;
     fa.g.ldo = ldo;
     fa.g.bias = bias;

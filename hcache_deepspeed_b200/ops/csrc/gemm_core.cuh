@@ -67,6 +67,7 @@ struct GemmArgs {
     int debug_skip;        // experiments only (HDS_GEMM_DEBUG): bit0 = no A loads, bit1 = no MMA issue (results invalid)
     int w_tiled;           // W is stored pre-tiled [N/32][K/64][32][64]: every TMA box is one contiguous 4 KB chunk
     int act;               // Activation
+    float act_limit;       // ACT_SWIGLU_CLAMPED: the bound L
     // EPI_STORE / EPI_GATED
     void* out;
     int64_t ldo;           // elements
@@ -165,9 +166,17 @@ __device__ __forceinline__ void gated_chunk(const GemmArgs& a, int row, int n, f
             u[j] += load_scalar<kBf16>(a.bias, n + 2 * j + 1);
         }
     }
-    apply_act_vec<16>(o, a.act);
+    if (a.act == ACT_SWIGLU_CLAMPED) {
 #pragma unroll
-    for (int j = 0; j < 16; ++j) o[j] *= u[j];
+        for (int j = 0; j < 16; ++j) {
+            const float g = fminf(o[j], a.act_limit);
+            o[j] = __fdividef(g, 1.0f + __expf(-kClampedGluAlpha * g)) * (fminf(fmaxf(u[j], -a.act_limit), a.act_limit) + 1.0f);
+        }
+    } else {
+        apply_act_vec<16>(o, a.act);
+#pragma unroll
+        for (int j = 0; j < 16; ++j) o[j] *= u[j];
+    }
     const int64_t off = static_cast<int64_t>(row) * a.ldo + (n >> 1);
     char* dst = reinterpret_cast<char*>(a.out) + off * 2;
     if (n + 32 <= a.N && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {

@@ -34,6 +34,7 @@ struct SkinnyArgs {
     int M, N, K;
     int splits, kb_per_split;
     int act;
+    float act_limit;    // ACT_SWIGLU_CLAMPED: the bound L
     void* out;          // EPI_STORE / EPI_GATED
     int64_t ldo;
     const void* bias;   // [N] I/O dtype, may be null
@@ -79,7 +80,15 @@ __device__ __forceinline__ void skinny_finalize(const SkinnyArgs& a, int n, uint
     for (int t = 0; t < NT; ++t) v[t] += b;
     if constexpr (kGated) {
         // even lanes hold gate features (activated), odd lanes the matching up features (left as they are)
-        apply_act_vec<NT>(v, (lane & 1) ? static_cast<int>(ACT_IDENTITY) : a.act);
+        if (a.act == ACT_SWIGLU_CLAMPED) {
+#pragma unroll
+            for (int t = 0; t < NT; ++t) {
+                const float c = fminf(v[t], a.act_limit);
+                v[t] = (lane & 1) ? fmaxf(c, -a.act_limit) + 1.0f : __fdividef(c, 1.0f + __expf(-kClampedGluAlpha * c));
+            }
+        } else {
+            apply_act_vec<NT>(v, (lane & 1) ? static_cast<int>(ACT_IDENTITY) : a.act);
+        }
 #pragma unroll
         for (int t = 0; t < NT; ++t) {
             const float partner = __shfl_xor_sync(0xffffffffu, v[t], 1);

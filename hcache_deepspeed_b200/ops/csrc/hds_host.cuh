@@ -217,5 +217,10 @@ inline int make_tmap_3d_16b(CUtensorMap* map, const void* base, uint64_t d0, uin
 // attention_splitkv.cu); returns them once, then nullptr.
 const float* attn_take_alibi();
 int attn_take_window();   // same for hds_attention_next_window (0 = no sliding window)
+int attn_take_keep_first();       // hds_attention_next_keep_first (0 = none)
+int64_t attn_take_out_stride();   // hds_attention_next_out_stride (0 = dense rows)
+
+// Bound of ACT_SWIGLU_CLAMPED armed by hds_gemm_next_act_limit for the next GEMM launch of this thread (gemm.cu).
+float gemm_take_act_limit();
 
 }  // namespace hds

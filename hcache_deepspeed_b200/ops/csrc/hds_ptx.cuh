@@ -513,7 +513,9 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
-enum Activation : int { ACT_IDENTITY = 0, ACT_GELU = 1, ACT_RELU = 2, ACT_SILU = 3, ACT_GELU_TANH = 4 };
+enum Activation : int { ACT_IDENTITY = 0, ACT_GELU = 1, ACT_RELU = 2, ACT_SILU = 3, ACT_GELU_TANH = 4, ACT_SWIGLU_CLAMPED = 5 };
+// ACT_SWIGLU_CLAMPED (gated epilogues only): g = min(gate, L), u = clamp(up, -L, L), out = g * sigmoid(alpha g) * (u + 1)
+constexpr float kClampedGluAlpha = 1.702f;
 
 // sin / cos of a RoPE angle (position x inverse frequency: up to ~1e5 rad). Two-constant Cody-Waite reduction to
 // [-pi, pi] followed by the SFU approximations: absolute error ~1e-6, far below the 6e-8 * |x| the fp32 product

@@ -110,6 +110,40 @@ moe_topk_gating_kernel(const void* __restrict__ logits, int64_t ld, int E, int k
     }
 }
 
+// Expert choice by a table of token ids: the same outputs as the gating kernel, every choice with weight 1 / k. Ids outside
+// the vocabulary take row 0 (their rows are never read).
+__global__ void moe_table_route_kernel(const int32_t* __restrict__ ids, const int32_t* __restrict__ table, int vocab, int T, int k,
+                                       float* __restrict__ scores, int32_t* __restrict__ expert_ids,
+                                       int32_t* __restrict__ offsets, int32_t* __restrict__ counts) {
+    pdl_enter();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= T * k) return;
+    const int id = ids[c / k];
+    const int e = table[static_cast<int64_t>(id >= 0 && id < vocab ? id : 0) * k + c % k];
+    scores[c] = 1.0f / k;
+    expert_ids[c] = e;
+    offsets[c] = atomicAdd(&counts[e], 1);
+}
+
+// out[t] = base[t] + sum_j score[t, j] * y[row(t, j)]: stores (no read of out), base optional. DT: type of y and base.
+template <int DT>
+__global__ void moe_combine_kernel(const void* __restrict__ y, int64_t ldy, const int32_t* __restrict__ mapped_slots,
+                                   const float* __restrict__ scores, const void* __restrict__ base, int64_t ldb,
+                                   float* __restrict__ out, int64_t ldo, int H, int k) {
+    pdl_enter();
+    const int64_t t = blockIdx.x;
+    for (int c = threadIdx.x * 2; c < H; c += blockDim.x * 2) {
+        float a0 = base ? load_any<DT>(base, t * ldb + c) : 0.0f, a1 = base ? load_any<DT>(base, t * ldb + c + 1) : 0.0f;
+        for (int j = 0; j < k; ++j) {
+            const int64_t row = static_cast<int64_t>(mapped_slots[t * k + j]) * ldy;
+            const float s = scores[t * k + j];
+            a0 = fmaf(s, load_any<DT>(y, row + c), a0);
+            a1 = fmaf(s, load_any<DT>(y, row + c + 1), a1);
+        }
+        *reinterpret_cast<float2*>(out + t * ldo + c) = make_float2(a0, a1);
+    }
+}
+
 __global__ void moe_offsets_kernel(int32_t* __restrict__ counts, int32_t* __restrict__ pad_off, int E) {
     pdl_enter();
     if (threadIdx.x == 0 && blockIdx.x == 0) {
@@ -218,4 +252,29 @@ extern "C" int hds_moe_gather(const void* y, int64_t ldy, const int32_t* mapped_
 extern "C" int64_t hds_moe_padded_rows(int T, int E, int k) {
     // every expert's range is rounded up to the 128-row GEMM tile
     return (static_cast<int64_t>(T) * k + static_cast<int64_t>(E) * (kMoeRowPad - 1)) / kMoeRowPad * kMoeRowPad + kMoeRowPad;
+}
+
+extern "C" int hds_moe_table_route(const int32_t* ids, const int32_t* table, int vocab, int T, int E, int k, float* scores,
+                                   int32_t* expert_ids, int32_t* offsets, int32_t* counts, void* stream) {
+    HDS_REQUIRE(E >= 1 && k >= 1 && k <= E && vocab >= 1, "hds_moe_table_route: 1 <= top_k <= experts, vocab >= 1");
+    if (T == 0) return HDS_OK;
+    HDS_CHECK_CUDA(launch_kernel(moe_table_route_kernel, dim3((T * k + 255) / 256), dim3(256), 0, static_cast<cudaStream_t>(stream),
+                                 ids, table, vocab, T, k, scores, expert_ids, offsets, counts));
+    return HDS_OK;
+}
+
+extern "C" int hds_moe_combine(const void* y, int64_t ldy, const int32_t* mapped_slots, const float* scores, const void* base,
+                               int64_t ldb, float* out, int64_t ldo, int T, int k, int H, int dtype, void* stream) {
+    HDS_REQUIRE(H % 2 == 0 && ldo % 2 == 0, "hds_moe_combine: even row widths");
+    HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_moe_combine: dtype 0 bf16 / 1 fp16 / 2 fp32");
+    if (T == 0) return HDS_OK;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const dim3 block(H >= 512 ? 256 : 128);
+    if (dtype == 0)
+        HDS_CHECK_CUDA(launch_kernel(moe_combine_kernel<0>, dim3(T), block, 0, s, y, ldy, mapped_slots, scores, base, ldb, out, ldo, H, k));
+    else if (dtype == 1)
+        HDS_CHECK_CUDA(launch_kernel(moe_combine_kernel<1>, dim3(T), block, 0, s, y, ldy, mapped_slots, scores, base, ldb, out, ldo, H, k));
+    else
+        HDS_CHECK_CUDA(launch_kernel(moe_combine_kernel<2>, dim3(T), block, 0, s, y, ldy, mapped_slots, scores, base, ldb, out, ldo, H, k));
+    return HDS_OK;
 }

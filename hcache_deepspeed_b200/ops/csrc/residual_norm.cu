@@ -1,0 +1,241 @@
+// Norms of stacks that keep the residual stream in fp32 and norm every sublayer's input AND output.
+//
+//   norm_residual : one pass per sublayer boundary. The previous sublayer's output d (16-bit, or the fp32 partial sums of a
+//                   split-K GEMM, cleared while being read) is itself RMS-normed and weighted, added to the fp32 stream, and
+//                   the stream is RMS-normed for the next sublayer:
+//                       x += f d / rms(f d) * post;   out = x / rms(x) * gamma
+//                   One CTA per row; the row stays in registers between the two reductions.
+//   gated_norm    : out = rms(y * silu(z)) * weight * scale over `groups` equal parts of a row (state-space mixers)
+//   embed_f32     : embedding rows into the fp32 stream
+#include "hds_host.cuh"
+#include "hds_ptx.cuh"
+#include "../../../include/hds_b200.h"
+
+namespace hds {
+
+template <int THREADS>
+__device__ __forceinline__ float block_sum_t(float v, float* red) {
+    v = warp_sum(v);
+    const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
+    if (l == 0) red[w] = v;
+    __syncthreads();
+    float t = l < THREADS / 32 ? red[l] : 0.0f;
+    t = warp_sum(t);
+    __syncthreads();
+    return t;
+}
+
+// four consecutive values of a row; DT 0 bf16, 1 fp16, 2 fp32
+template <int DT>
+__device__ __forceinline__ float4 load4(const void* base, int64_t idx) {
+    if constexpr (DT == 2) {
+        return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(base) + idx);
+    } else {
+        const uint2 q = *reinterpret_cast<const uint2*>(reinterpret_cast<const char*>(base) + idx * 2);
+        return make_float4(unpack_lo<DT == 0>(q.x), unpack_hi<DT == 0>(q.x), unpack_lo<DT == 0>(q.y), unpack_hi<DT == 0>(q.y));
+    }
+}
+template <int DT>
+__device__ __forceinline__ void store4(void* base, int64_t idx, float4 v) {
+    if constexpr (DT == 2) {
+        *reinterpret_cast<float4*>(reinterpret_cast<float*>(base) + idx) = v;
+    } else {
+        uint2 q;
+        q.x = pack2<DT == 0>(v.x, v.y);
+        q.y = pack2<DT == 0>(v.z, v.w);
+        *reinterpret_cast<uint2*>(reinterpret_cast<char*>(base) + idx * 2) = q;
+    }
+}
+
+// `cols`: values a row's mean is taken over; `padded` >= cols: row width, zeros behind the values. DELTA 0 none, 1 fp32
+// (cleared after being read), 2 the output's type.
+template <int THREADS, int VPT, int DT, int DELTA>
+__global__ void __launch_bounds__(THREADS)
+norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const float* __restrict__ post,
+                     const float* __restrict__ gamma, void* __restrict__ out, int64_t ld, int cols, int padded, float eps,
+                     int store_x) {
+    __shared__ float red[THREADS / 32];
+    pdl_enter();
+    const int64_t row = static_cast<int64_t>(blockIdx.x) * ld;
+    const int nvec = padded >> 2;
+    float4 v[VPT], d[VPT];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+        const int c = threadIdx.x + i * THREADS;
+        v[i] = d[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < nvec) {
+            v[i] = *reinterpret_cast<const float4*>(x + row + 4 * c);
+            if constexpr (DELTA == 1) {
+                float4* p = reinterpret_cast<float4*>(reinterpret_cast<float*>(delta) + row + 4 * c);
+                d[i] = *p;
+                *p = make_float4(0.f, 0.f, 0.f, 0.f);
+            } else if constexpr (DELTA == 2) {
+                d[i] = load4<DT>(delta, row + 4 * c);
+            }
+            if constexpr (DELTA != 0) {
+                d[i].x *= factor; d[i].y *= factor; d[i].z *= factor; d[i].w *= factor;
+                ss += d[i].x * d[i].x + d[i].y * d[i].y + d[i].z * d[i].z + d[i].w * d[i].w;
+            }
+        }
+    }
+    if constexpr (DELTA != 0) {
+        const float r = 1.0f / sqrtf(block_sum_t<THREADS>(ss, red) / cols + eps);
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) {
+            const int c = threadIdx.x + i * THREADS;
+            if (c < nvec) {
+                const float4 w = *reinterpret_cast<const float4*>(post + 4 * c);
+                v[i].x += d[i].x * r * w.x; v[i].y += d[i].y * r * w.y;
+                v[i].z += d[i].z * r * w.z; v[i].w += d[i].w * r * w.w;
+                if (store_x) *reinterpret_cast<float4*>(x + row + 4 * c) = v[i];
+            }
+        }
+    }
+    ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    const float r = 1.0f / sqrtf(block_sum_t<THREADS>(ss, red) / cols + eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+        const int c = threadIdx.x + i * THREADS;
+        if (c < nvec) {
+            const float4 w = *reinterpret_cast<const float4*>(gamma + 4 * c);
+            store4<DT>(out, row + 4 * c, make_float4(v[i].x * r * w.x, v[i].y * r * w.y, v[i].z * r * w.z, v[i].w * r * w.w));
+        }
+    }
+}
+
+template <int DT, int DELTA>
+static int launch_norm_residual(float* x, void* delta, float factor, const float* post, const float* gamma, void* out, int64_t ld,
+                                int rows, int cols, int padded, float eps, int store_x, cudaStream_t s) {
+    const int nvec = padded / 4;
+#define HDS_NR(TH, V)                                                                                                       \
+    HDS_CHECK_CUDA(launch_kernel(norm_residual_kernel<TH, V, DT, DELTA>, dim3(rows), dim3(TH), 0, s, x, delta, factor, post, \
+                                 gamma, out, ld, cols, padded, eps, store_x))
+    if (nvec <= 128) HDS_NR(128, 1);
+    else if (nvec <= 256) HDS_NR(256, 1);
+    else if (nvec <= 512) HDS_NR(512, 1);
+    else if (nvec <= 1024) HDS_NR(512, 2);
+    else if (nvec <= 2048) HDS_NR(512, 4);
+    else if (nvec <= 8192) HDS_NR(1024, 8);
+    else {
+        set_error("hds_norm_residual: rows wider than 32768 are unsupported");
+        return HDS_ERR_UNSUPPORTED;
+    }
+#undef HDS_NR
+    return HDS_OK;
+}
+
+// One CTA per (row, part). y fp32, z in the I/O type; any part size.
+template <int DT>
+__global__ void __launch_bounds__(256)
+gated_norm_kernel(const float* __restrict__ y, int64_t ld_y, const void* __restrict__ z, int64_t ld_z,
+                  const float* __restrict__ w, void* __restrict__ out, int64_t ld_out, int part, float eps, float scale) {
+    extern __shared__ float vals[];
+    __shared__ float red[8];
+    pdl_enter();
+    const int64_t t = blockIdx.x;
+    const int c0 = blockIdx.y * part;
+    float ss = 0.0f;
+    const bool vec = (part & 3) == 0 && (ld_y & 3) == 0 && (ld_z & 3) == 0 && (ld_out & 3) == 0;
+    if (vec) {
+        for (int c = threadIdx.x * 4; c < part; c += 1024) {
+            const float4 a = *reinterpret_cast<const float4*>(y + t * ld_y + c0 + c);
+            const float4 b = load4<DT>(z, t * ld_z + c0 + c);
+            float4 g;
+            g.x = a.x * (b.x / (1.0f + expf(-b.x)));
+            g.y = a.y * (b.y / (1.0f + expf(-b.y)));
+            g.z = a.z * (b.z / (1.0f + expf(-b.z)));
+            g.w = a.w * (b.w / (1.0f + expf(-b.w)));
+            *reinterpret_cast<float4*>(vals + c) = g;
+            ss += g.x * g.x + g.y * g.y + g.z * g.z + g.w * g.w;
+        }
+    } else {
+        for (int c = threadIdx.x; c < part; c += 256) {
+            const float b = load_any<DT>(z, t * ld_z + c0 + c);
+            const float g = y[t * ld_y + c0 + c] * (b / (1.0f + expf(-b)));
+            vals[c] = g;
+            ss += g * g;
+        }
+    }
+    const float r = scale / sqrtf(block_sum_t<256>(ss, red) / part + eps);
+    if (vec) {
+        for (int c = threadIdx.x * 4; c < part; c += 1024) {
+            const float4 g = *reinterpret_cast<const float4*>(vals + c);
+            const float4 ww = *reinterpret_cast<const float4*>(w + c0 + c);
+            store4<DT>(out, t * ld_out + c0 + c, make_float4(g.x * r * ww.x, g.y * r * ww.y, g.z * r * ww.z, g.w * r * ww.w));
+        }
+    } else {
+        for (int c = threadIdx.x; c < part; c += 256) {
+            const float v = vals[c] * r * w[c0 + c];
+            if constexpr (DT == 2) reinterpret_cast<float*>(out)[t * ld_out + c0 + c] = v;
+            else store_scalar<DT == 0>(out, t * ld_out + c0 + c, v);
+        }
+    }
+}
+
+template <int DT>
+__global__ void embed_f32_kernel(const int32_t* __restrict__ ids, const void* __restrict__ W, float* __restrict__ out, int H, int vocab) {
+    pdl_enter();
+    const int64_t t = blockIdx.x;
+    const int id = ids[t];
+    const bool ok = id >= 0 && id < vocab;
+    for (int c = threadIdx.x * 4; c < H; c += blockDim.x * 4)
+        *reinterpret_cast<float4*>(out + t * H + c) =
+            ok ? load4<DT>(W, static_cast<int64_t>(id) * H + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+}
+
+}  // namespace hds
+
+using namespace hds;
+
+extern "C" int hds_norm_residual(float* x, void* delta, int delta_is_f32, float factor, const float* post, const float* gamma,
+                                 void* out, int64_t ld, int rows, int cols, int padded, float eps, int store_x, int dtype,
+                                 void* stream) {
+    HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_norm_residual: dtype 0 bf16 / 1 fp16 / 2 fp32");
+    HDS_REQUIRE(padded % 4 == 0 && ld % 4 == 0 && cols <= padded && padded <= ld, "hds_norm_residual: rows of 4-value vectors");
+    HDS_REQUIRE(delta == nullptr || post != nullptr, "hds_norm_residual: a delta needs its norm weight");
+    if (rows == 0) return HDS_OK;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const int mode = delta == nullptr ? 0 : delta_is_f32 ? 1 : 2;
+#define HDS_NR_ARGS x, delta, factor, post, gamma, out, ld, rows, cols, padded, eps, store_x, s
+#define HDS_NR_DT(DT)                                                            \
+    return mode == 0   ? launch_norm_residual<DT, 0>(HDS_NR_ARGS)                \
+           : mode == 1 ? launch_norm_residual<DT, 1>(HDS_NR_ARGS)                \
+                       : launch_norm_residual<DT, 2>(HDS_NR_ARGS)
+    if (dtype == 0) { HDS_NR_DT(0); }
+    if (dtype == 1) { HDS_NR_DT(1); }
+    HDS_NR_DT(2);
+#undef HDS_NR_DT
+#undef HDS_NR_ARGS
+}
+
+extern "C" int hds_gated_norm(const float* y, int64_t ld_y, const void* z, int64_t ld_z, const float* w, void* out, int64_t ld_out,
+                              int rows, int cols, int groups, float eps, float scale, int dtype, void* stream) {
+    HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_gated_norm: dtype 0 bf16 / 1 fp16 / 2 fp32");
+    HDS_REQUIRE(groups >= 1 && cols % groups == 0 && cols / groups <= 12000, "hds_gated_norm: equal parts of at most 12000 values");
+    if (rows == 0) return HDS_OK;
+    const int part = cols / groups;
+    const size_t smem = static_cast<size_t>(part) * 4;
+    const dim3 grid(rows, groups);
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (dtype == 0)
+        HDS_CHECK_CUDA(launch_kernel(gated_norm_kernel<0>, grid, dim3(256), smem, s, y, ld_y, z, ld_z, w, out, ld_out, part, eps, scale));
+    else if (dtype == 1)
+        HDS_CHECK_CUDA(launch_kernel(gated_norm_kernel<1>, grid, dim3(256), smem, s, y, ld_y, z, ld_z, w, out, ld_out, part, eps, scale));
+    else
+        HDS_CHECK_CUDA(launch_kernel(gated_norm_kernel<2>, grid, dim3(256), smem, s, y, ld_y, z, ld_z, w, out, ld_out, part, eps, scale));
+    return HDS_OK;
+}
+
+extern "C" int hds_embed_f32(const int32_t* ids, const void* W, float* out, int T, int H, int vocab, int dtype, void* stream) {
+    HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_embed_f32: dtype 0 bf16 / 1 fp16 / 2 fp32");
+    HDS_REQUIRE(H % 4 == 0, "hds_embed_f32: rows of 4-value vectors");
+    if (T == 0) return HDS_OK;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (dtype == 0) HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<0>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab));
+    else if (dtype == 1) HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<1>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab));
+    else HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<2>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab));
+    return HDS_OK;
+}

@@ -22,7 +22,7 @@ ACT_IDENTITY, ACT_GELU, ACT_RELU, ACT_SILU, ACT_GELU_TANH, ACT_SWIGLU_CLAMPED = 
 ACT_CODES = {"identity": 0, None: 0, "gelu": 1, "relu": 2, "silu": 3, "gelu_tanh": 4, "gelu_new": 4,
              "gelu_pytorch_tanh": 4, "swish": 3, "swiglu_clamped": 5}
 
-EPI_STORE, EPI_GATED = 0, 1
+EPI_STORE, EPI_GATED, EPI_ACCUM = 0, 1, 2
 
 #: counts launches of our own kernels (bench.py reports it as ``gpu_launches``)
 launch_count = 0
@@ -34,6 +34,11 @@ def _dt(t: torch.Tensor) -> int:
     if t.dtype == torch.float16:
         return 1
     raise TypeError(f"unsupported activation dtype {t.dtype}: the sm_100a kernels take bf16 or fp16")
+
+
+def _dt3(t: torch.Tensor) -> int:
+    """dtype code of the kernels that also take fp32."""
+    return 2 if t.dtype == torch.float32 else _dt(t)
 
 
 def _p(t: Optional[torch.Tensor]):
@@ -112,9 +117,10 @@ def gemm_splitk_workspace_bytes(M: int, N: int) -> int:
 
 def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, act: int = ACT_IDENTITY,
          gated: bool = False, out: Optional[torch.Tensor] = None, bn: int = 0, splits: int = 0,
-         workspace: Optional[torch.Tensor] = None) -> torch.Tensor:
+         workspace: Optional[torch.Tensor] = None, limit: float = 0.0) -> torch.Tensor:
     """``out = epilogue(a @ w.T + bias)`` on the tcgen05 GEMM. ``gated``: interleaved (gate, up) columns.
-    ``workspace`` (zero-initialised uint8 scratch) enables split-K for decode-size M."""
+    ``workspace`` (zero-initialised uint8 scratch) enables split-K for decode-size M. ``limit``: the bound of
+    ``ACT_SWIGLU_CLAMPED``. fp32 operands take the plain fp32 kernel."""
     _check_2d(a, "a")
     M, K = a.shape
     N = w.shape[0]
@@ -124,11 +130,28 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, 
     if out is None:
         out = torch.empty((M, n_out), dtype=a.dtype, device=a.device)
     _check_2d(out, "out")
+    if a.dtype == torch.float32:
+        assert bias is None
+        return _gemm_f32(a, w, out, EPI_GATED if gated else EPI_STORE, act, limit)
     lib = native.cuda_lib()
+    if act == ACT_SWIGLU_CLAMPED:
+        native.check(lib.hds_gemm_next_act_limit(limit), "hds_gemm_next_act_limit")
     rc = lib.hds_gemm(_p(a), a.stride(0), wp, ldw, M, N, K, _dt(a), EPI_GATED if gated else EPI_STORE,
                       act, _p(bias), _p(out), out.stride(0), bn, splits, _p(workspace),
                       0 if workspace is None else workspace.numel() * workspace.element_size(), _stream())
     native.check(rc, "hds_gemm")
+    _count()
+    return out
+
+
+def _gemm_f32(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, act: int, limit: float,
+              group_off: Optional[torch.Tensor] = None, n_groups: int = 0) -> torch.Tensor:
+    M, K = a.shape
+    N = w.shape[0] // max(1, n_groups)
+    assert w.dtype == torch.float32 and w.shape[1] == K and out.dtype == torch.float32
+    rc = native.cuda_lib().hds_gemm_f32(_p(a), a.stride(0), _p(w), w.stride(0), M, N, K, epilogue, act, limit, _p(out), out.stride(0),
+                                        _p(group_off), n_groups, _stream())
+    native.check(rc, "hds_gemm_f32")
     _count()
     return out
 
@@ -142,8 +165,12 @@ def gemm_accum(a: torch.Tensor, w: torch.Tensor, accum: torch.Tensor, bias: Opti
     _check_2d(a, "a")
     M, K = a.shape
     N = w.shape[0]
-    wp, ldw = _w(w)
     assert accum.dtype == torch.float32 and accum.stride(-1) == 1
+    if a.dtype == torch.float32:
+        assert bias is None and peer_ptrs is None and multicast_ptr is None
+        _gemm_f32(a, w, accum, EPI_ACCUM, ACT_IDENTITY, 0.0)
+        return
+    wp, ldw = _w(w)
     if multicast_ptr is not None:
         ptrs, mode = [multicast_ptr], 2
     elif peer_ptrs is not None:
@@ -319,7 +346,7 @@ def embed(ids: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, pos_weight
 
 def gather_rows(x: torch.Tensor, row_idx: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     lib = native.cuda_lib()
-    rc = lib.hds_gather_rows(_p(x), _p(row_idx), _p(out), row_idx.numel(), x.shape[-1], _stream())
+    rc = lib.hds_gather_rows(_p(x), _p(row_idx), _p(out), row_idx.numel(), x.shape[-1] * x.element_size() // 2, _stream())
     native.check(rc, "hds_gather_rows")
     _count()
     return out
@@ -374,9 +401,14 @@ def splitkv_workspace_bytes(n_items: int, n_q_heads: int, n_kv_heads: int, head_
                                                                              max_splits, rows_per_item))
 
 
-def _arm_alibi(lib, alibi: Optional[torch.Tensor], n_q_heads: int, window: int = 0) -> None:
-    """ALiBi slopes / sliding window for the next attention launch of this thread (``hds_attention_next_alibi``,
-    ``hds_attention_next_window``; both are consumed by that launch)."""
+def _arm_alibi(lib, alibi: Optional[torch.Tensor], n_q_heads: int, window: int = 0, keep_first: int = 0,
+               out: Optional[torch.Tensor] = None) -> None:
+    """Options of the next attention launch of this thread, consumed by that launch: ALiBi slopes, sliding window and kept
+    first tokens, and the stride of ``out`` when its rows (``[T, n_q_heads * head_dim]``) are not dense."""
+    if keep_first:
+        native.check(lib.hds_attention_next_keep_first(int(keep_first)), "hds_attention_next_keep_first")
+    if out is not None and out.dim() == 2 and out.stride(0) != out.shape[1]:
+        native.check(lib.hds_attention_next_out_stride(out.stride(0)), "hds_attention_next_out_stride")
     if window:
         native.check(lib.hds_attention_next_window(int(window)), "hds_attention_next_window")
     if alibi is None:
@@ -389,11 +421,12 @@ def paged_attention_splitkv(q: torch.Tensor, out: torch.Tensor, kv_cache_layer: 
                             block_tables: torch.Tensor, items: torch.Tensor, n_items: int, rows_per_item: int,
                             n_q_heads: int, n_kv_heads: int, head_dim: int, block_size: int, n_splits: int,
                             scale: float, workspace: Optional[torch.Tensor], alibi: Optional[torch.Tensor] = None,
-                            window: int = 0) -> None:
+                            window: int = 0, keep_first: int = 0) -> None:
     """kv_cache_layer: [blocks, 2, kvh, bs, d]; items: int32 [n, 4] = (seq, q_row0, n_q, pos0). ``alibi``: fp32 [n_q_heads]
-    slopes; score += slope * (key position - query position). ``window``: sliding-window attention, keys (p - window, p]."""
+    slopes; score += slope * (key position - query position). ``window``: sliding-window attention, keys (p - window, p] and
+    the first ``keep_first`` ones."""
     lib = native.cuda_lib()
-    _arm_alibi(lib, alibi, n_q_heads, window)
+    _arm_alibi(lib, alibi, n_q_heads, window, keep_first, out)
     rc = lib.hds_paged_attention_splitkv(_p(q), _p(out), _p(kv_cache_layer), kv_cache_layer.shape[0], _p(block_tables),
                                          block_tables.stride(0), _p(items), n_items, rows_per_item, n_q_heads,
                                          n_kv_heads, head_dim, block_size, n_splits, scale, _p(workspace),
@@ -411,12 +444,12 @@ def paged_attention_prefill(q: torch.Tensor, out: torch.Tensor, kv_cache_layer: 
                             block_tables: torch.Tensor, items: torch.Tensor, n_items: int, n_q_heads: int,
                             n_kv_heads: int, head_dim: int, block_size: int, scale: float, n_splits: int = 1,
                             workspace: Optional[torch.Tensor] = None, packed: bool = False,
-                            alibi: Optional[torch.Tensor] = None, window: int = 0) -> None:
+                            alibi: Optional[torch.Tensor] = None, window: int = 0, keep_first: int = 0) -> None:
     """tcgen05 paged attention. ``packed``: grouped-query decode form — one CTA per (item, KV head) whose MMA rows are
     the group's (token, query head) pairs (``hds_paged_attention_packed``). ``alibi``: fp32 [n_q_heads] slopes;
     ``window``: sliding-window attention."""
     lib = native.cuda_lib()
-    _arm_alibi(lib, alibi, n_q_heads, window)
+    _arm_alibi(lib, alibi, n_q_heads, window, keep_first, out)
     fn = lib.hds_paged_attention_packed if packed else lib.hds_paged_attention_prefill
     rc = fn(_p(q), _p(out), _p(kv_cache_layer), kv_cache_layer.shape[0], _p(block_tables),
                                          block_tables.stride(0), _p(items), n_items, q.shape[0], n_q_heads, n_kv_heads,
@@ -451,20 +484,26 @@ def moe_scatter(x: torch.Tensor, xs: torch.Tensor, expert_ids: torch.Tensor, off
     """Build ``pad_off`` (int32 [E+1]) from ``counts`` (re-zeroed) and copy every token row to its k expert rows."""
     T, H = x.shape
     E = counts.numel()
-    rc = native.cuda_lib().hds_moe_scatter(_p(x), x.stride(0), _p(xs), xs.stride(0), _p(expert_ids), _p(offsets), _p(counts),
+    r = x.element_size() // 2      # the kernel moves 16-bit units
+    H *= r
+    rc = native.cuda_lib().hds_moe_scatter(_p(x), x.stride(0) * r, _p(xs), xs.stride(0) * r, _p(expert_ids), _p(offsets), _p(counts),
                                            _p(pad_off), _p(mapped_slots), T, E, top_k, H, _stream())
     native.check(rc, "hds_moe_scatter")
     _count(2)
 
 
 def moe_gemm(a: torch.Tensor, w_stacked: torch.Tensor, pad_off: torch.Tensor, n_experts: int, out: torch.Tensor,
-             act: int = ACT_IDENTITY, gated: bool = False) -> torch.Tensor:
+             act: int = ACT_IDENTITY, gated: bool = False, limit: float = 0.0) -> torch.Tensor:
     """Grouped GEMM: rows of ``a`` in expert e's range times ``w_stacked[e*N:(e+1)*N]``ᵀ (``w_stacked``: [E*N, K])."""
     _check_2d(a, "a")
     _check_2d(out, "out")
     rows, K = a.shape
     N = w_stacked.shape[0] // n_experts
     assert w_stacked.shape[1] == K and rows % 128 == 0 and out.shape[0] >= rows
+    if a.dtype == torch.float32:
+        return _gemm_f32(a, w_stacked, out, EPI_GATED if gated else EPI_STORE, act, limit, pad_off, n_experts)
+    if act == ACT_SWIGLU_CLAMPED:
+        native.check(native.cuda_lib().hds_gemm_next_act_limit(limit), "hds_gemm_next_act_limit")
     rc = native.cuda_lib().hds_moe_gemm(_p(a), a.stride(0), _p(w_stacked), w_stacked.stride(0), _p(pad_off), n_experts, rows,
                                         N, K, _dt(a), EPI_GATED if gated else EPI_STORE, act, _p(out), out.stride(0),
                                         _stream())
@@ -569,4 +608,103 @@ def moe_gather(y: torch.Tensor, mapped_slots: torch.Tensor, scores: torch.Tensor
     rc = native.cuda_lib().hds_moe_gather(_p(y), y.stride(0), _p(mapped_slots), _p(scores), _p(out), out.stride(0), T, k,
                                           y.shape[1], _dt(y), _stream())
     native.check(rc, "hds_moe_gather")
+    _count()
+
+
+# ------------------------------------------------------------------------------------------------
+# expert choice by table, fp32 residual stream, state-space mixers, generic attention
+# ------------------------------------------------------------------------------------------------
+def moe_table_route(ids: torch.Tensor, table: torch.Tensor, n_experts: int, scores: torch.Tensor, expert_ids: torch.Tensor,
+                    offsets: torch.Tensor, counts: torch.Tensor) -> None:
+    """Experts of every token from ``table`` (int32 [vocab, top]) with equal weights; ``counts`` as in moe_topk_gating."""
+    assert ids.dtype == torch.int32 and table.dtype == torch.int32
+    rc = native.cuda_lib().hds_moe_table_route(_p(ids), _p(table), table.shape[0], ids.numel(), n_experts, table.shape[1], _p(scores),
+                                               _p(expert_ids), _p(offsets), _p(counts), _stream())
+    native.check(rc, "hds_moe_table_route")
+    _count()
+
+
+def moe_combine(y: torch.Tensor, mapped_slots: torch.Tensor, scores: torch.Tensor, base: Optional[torch.Tensor],
+                out: torch.Tensor) -> torch.Tensor:
+    """``out[t] = base[t] + sum_j scores[t, j] * y[mapped_slots[t, j]]`` (``out`` fp32, stored; ``base`` optional)."""
+    T, k = mapped_slots.shape
+    assert out.dtype == torch.float32
+    rc = native.cuda_lib().hds_moe_combine(_p(y), y.stride(0), _p(mapped_slots), _p(scores), _p(base),
+                                           0 if base is None else base.stride(0), _p(out), out.stride(0), T, k, y.shape[1], _dt3(y),
+                                           _stream())
+    native.check(rc, "hds_moe_combine")
+    _count()
+    return out
+
+
+def embed_f32(ids: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    assert ids.dtype == torch.int32 and out.dtype == torch.float32
+    rc = native.cuda_lib().hds_embed_f32(_p(ids), _p(weight), _p(out), ids.numel(), weight.shape[1], weight.shape[0], _dt3(weight),
+                                         _stream())
+    native.check(rc, "hds_embed_f32")
+    _count()
+    return out
+
+
+def norm_residual(resid: torch.Tensor, gamma: torch.Tensor, out: torch.Tensor, delta: Optional[torch.Tensor] = None,
+                  factor: float = 1.0, post: Optional[torch.Tensor] = None, cols: Optional[int] = None, eps: float = 1e-5,
+                  store_resid: bool = True) -> torch.Tensor:
+    """``resid += norm(factor * delta) * post`` on the fp32 stream, ``out = norm(resid) * gamma`` (``hds_norm_residual``)."""
+    rows, width = resid.shape
+    assert resid.stride(0) == out.stride(0) and (delta is None or delta.stride(0) == resid.stride(0))
+    assert delta is None or delta.dtype in (torch.float32, out.dtype)
+    rc = native.cuda_lib().hds_norm_residual(_p(resid), _p(delta), 1 if (delta is not None and delta.dtype == torch.float32) else 0,
+                                             factor, _p(post), _p(gamma), _p(out), resid.stride(0), rows,
+                                             width if cols is None else cols, width, eps, 1 if store_resid else 0, _dt3(out), _stream())
+    native.check(rc, "hds_norm_residual")
+    _count()
+    return out
+
+
+def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, groups: int, eps: float,
+               scale: float = 1.0) -> torch.Tensor:
+    """``out = scale * weight * v / rms(v)``, ``v = y * silu(z)``, rms per part of a row (``groups`` equal parts)."""
+    rc = native.cuda_lib().hds_gated_norm(_p(y), y.stride(0), _p(z), z.stride(0), _p(weight), _p(out), out.stride(0), y.shape[0],
+                                          y.shape[1], groups, eps, scale, _dt3(out), _stream())
+    native.check(rc, "hds_gated_norm")
+    _count()
+    return out
+
+
+SCAN_AUTO, SCAN_TOKENS, SCAN_CHUNKED = 0, 1, 2
+
+
+def state_space(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, dt_bias: torch.Tensor, decay: torch.Tensor,
+                skip: torch.Tensor, state: torch.Tensor, conv_state: torch.Tensor, spans: torch.Tensor, n_single: int, groups: int,
+                u: torch.Tensor, dt: torch.Tensor, y: torch.Tensor, method: int = SCAN_AUTO) -> torch.Tensor:
+    """Convolution and recurrence of a state-space mixer over a ragged batch (``hds_state_space``). ``state``
+    [slots, heads, vdim, state], ``conv_state`` [slots, taps, channels]; ``spans`` int32 [n_seqs, 4]."""
+    T = proj.shape[0]
+    _, heads, vdim, n = state.shape
+    taps = conv_w.shape[0]
+    rc = native.cuda_lib().hds_state_space(_p(proj), proj.stride(0), _p(conv_w), _p(conv_b), _p(dt_bias), _p(decay), _p(skip), _p(state),
+                                           _p(conv_state), _p(spans), spans.shape[0], n_single, T, heads, vdim, n, groups, taps, _p(u),
+                                           u.stride(0), _p(dt), _p(y), method, _dt3(proj), _stream())
+    native.check(rc, "hds_state_space")
+    n_multi = spans.shape[0] - n_single
+    _count((2 if n_multi else 0) + (1 if n_single else 0))
+    return y
+
+
+def paged_attention_generic(q: torch.Tensor, out: torch.Tensor, kv_cache_layer: torch.Tensor, block_tables: torch.Tensor,
+                            tok_seq: torch.Tensor, tok_pos: torch.Tensor, n_q_heads: int, n_kv_heads: int, head_dim: int,
+                            block_size: int, scale: float, window: int = 0, keep_first: int = 0) -> None:
+    """fp32-arithmetic attention for any operand type and head size (``hds_paged_attention_generic``)."""
+    rc = native.cuda_lib().hds_paged_attention_generic(_p(q), _p(out), out.stride(0), _p(kv_cache_layer), _p(block_tables),
+                                                       block_tables.stride(0), _p(tok_seq), _p(tok_pos), q.shape[0], n_q_heads,
+                                                       n_kv_heads, head_dim, block_size, scale, window, keep_first, _dt3(q), _stream())
+    native.check(rc, "hds_paged_attention_generic")
+    _count()
+
+
+def kv_append_generic(qkv: torch.Tensor, q_out: torch.Tensor, kv_cache_layer: torch.Tensor, tok_slot: torch.Tensor, n_q_heads: int,
+                      n_kv_heads: int, head_dim: int, block_size: int) -> None:
+    rc = native.cuda_lib().hds_kv_append_generic(_p(qkv), qkv.stride(0), _p(q_out), _p(kv_cache_layer), _p(tok_slot), qkv.shape[0],
+                                                 n_q_heads, n_kv_heads, head_dim, block_size, qkv.element_size(), _stream())
+    native.check(rc, "hds_kv_append_generic")
     _count()

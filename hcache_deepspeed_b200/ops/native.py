@@ -45,6 +45,18 @@ def _declare_cuda(lib: ctypes.CDLL) -> None:
         "hds_fp8_next_weight_format": [I],
         "hds_attention_next_alibi": [P],
         "hds_attention_next_window": [I],
+        "hds_attention_next_keep_first": [I],
+        "hds_attention_next_out_stride": [L],
+        "hds_paged_attention_generic": [P, P, L, P, P, I, P, P, I, I, I, I, I, F, I, I, I, P],
+        "hds_kv_append_generic": [P, L, P, P, P, I, I, I, I, I, I, P],
+        "hds_gemm_f32": [P, L, P, L, I, I, I, I, I, F, P, L, P, I, P],
+        "hds_gemm_next_act_limit": [F],
+        "hds_moe_table_route": [P, P, I, I, I, I, P, P, P, P, P],
+        "hds_moe_combine": [P, L, P, P, P, L, P, L, I, I, I, I, P],
+        "hds_embed_f32": [P, P, P, I, I, I, I, P],
+        "hds_norm_residual": [P, P, I, F, P, P, P, L, I, I, I, F, I, I, P],
+        "hds_gated_norm": [P, L, P, L, P, P, L, I, I, I, F, F, I, P],
+        "hds_state_space": [P, L, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, L, P, P, I, I, P],
         "hds_host_buffer_alloc": [L, I, I, P],
         "hds_host_buffer_device_ptr": [P, P],
         "hds_host_buffer_free": [P],

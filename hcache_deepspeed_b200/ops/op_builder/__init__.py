@@ -20,12 +20,14 @@ def _mk(name, lib, symbols, sources=(), depends=(), doc=""):
 
 
 InferenceCoreBuilder = _mk("inference_core_ops", "cuda", ["hds_gemm", "hds_gemm_2sm", "hds_gemm_fp8", "hds_quantize_fp8_rows", "hds_norm"],
-                           sources=_GEMM_TUS + ("elementwise.cu", ), depends=_TP)
+                           sources=_GEMM_TUS + ("elementwise.cu", "residual_norm.cu", "gemm_f32.cu"), depends=_TP)
 RaggedOpsBuilder = _mk("ragged_device_ops", "cuda", ["hds_paged_attention_splitkv", "hds_paged_attention_prefill", "hds_embed",
                                                        "hds_rope_kv_append", "hds_gather_rows", "hds_moe_topk_gating",
                                                        "hds_moe_scatter", "hds_moe_gather"],
-                       sources=("attention_splitkv.cu", "attention_prefill.cu", "elementwise.cu", "moe.cu", "host_buffer.cu"),
+                       sources=("attention_splitkv.cu", "attention_prefill.cu", "elementwise.cu", "moe.cu", "host_buffer.cu",
+                                "attention_generic.cu"),
                        depends=_TP)
+StateSpaceBuilder = _mk("state_space_ops", "cuda", ["hds_state_space"], sources=("ssm.cu", "ssm_chunk.cu"))
 InferenceCutlassBuilder = _mk("cutlass_ops", "cuda", ["hds_moe_gemm"], sources=("moe.cu", ))
 RaggedUtilsBuilder = _mk("ragged_ops", "host", ["hds_alloc_create", "hds_build_batch"], sources=("host_runtime.cpp", ))
 InferenceBuilder = _mk("transformer_inference", "cuda", ["hds_gemm", "hds_norm", "hds_rope_kv_append"],
@@ -86,7 +88,7 @@ class UtilsBuilder(OpBuilder):
         return SimpleNamespace(flatten=_flatten_dense_tensors, unflatten=_unflatten_dense_tensors)
 
 ALL_OPS: Dict[str, OpBuilder] = {b.NAME: b() for b in (
-    InferenceCoreBuilder, RaggedOpsBuilder, InferenceCutlassBuilder, RaggedUtilsBuilder, InferenceBuilder, AsyncIOBuilder,
+    InferenceCoreBuilder, RaggedOpsBuilder, StateSpaceBuilder, InferenceCutlassBuilder, RaggedUtilsBuilder, InferenceBuilder, AsyncIOBuilder,
     GDSBuilder, QuantizerBuilder, FPQuantizerBuilder, FusedAdamBuilder, FusedLionBuilder, FusedLambBuilder, CPUAdamBuilder,
     CPUAdagradBuilder, CPULionBuilder, TransformerBuilder, StochasticTransformerBuilder, SparseAttnBuilder, RandomLTDBuilder,
     SpatialInferenceBuilder, EvoformerAttnBuilder, UtilsBuilder, ShareMemCommBuilder)}

@@ -239,6 +239,24 @@ int hds_attention_next_alibi(const float* slopes);
  * loaded. 0 = unlimited. Cleared by that launch. */
 int hds_attention_next_window(int window);
 
+/* With a window, for the same launch: the first keep_first positions of a sequence stay visible to all of its later queries
+ * (their key tiles are visited although they lie before the window). Cleared by that launch. */
+int hds_attention_next_keep_first(int keep_first);
+/* Elements between the output rows of two tokens for the same launch (a multiple of 8; 0 = dense rows of n_q_heads * head_dim),
+ * so that a layer's mixers can write side by side into one buffer. Cleared by that launch. */
+int hds_attention_next_out_stride(int64_t elements);
+
+/* Paged attention in plain fp32 arithmetic for operands and head sizes the tensor-core kernels do not take: dtype 0 bf16,
+ * 1 fp16, 2 fp32, head_dim up to 512. One warp per (token, query head); tok_seq / tok_pos give each token's block-table row and
+ * position. window / keep_first as above. */
+int hds_paged_attention_generic(const void* q, void* out, int64_t ld_out, const void* kv_cache_layer, const int32_t* block_tables,
+                                int max_blocks_per_seq, const int32_t* tok_seq, const int32_t* tok_pos, int T, int n_q_heads,
+                                int n_kv_heads, int head_dim, int block_size, float scale, int window, int keep_first, int dtype,
+                                void* stream);
+/* hds_rope_kv_append without rotation, for 2- or 4-byte elements and any head_dim. */
+int hds_kv_append_generic(const void* qkv, int64_t ld_qkv, void* q_out, void* kv_cache_layer, const int32_t* tok_slot, int T,
+                          int n_q_heads, int n_kv_heads, int head_dim, int block_size, int elem_bytes, void* stream);
+
 /* tcgen05 paged attention for items with up to 128 query tokens (prefill / chunked continuation): QK^T and
  * PV on the tensor cores with TMEM accumulators, TMA page gathers, online softmax in registers.
  * n_q_rows = total rows of q (bounds the Q tensor map). n_splits > 1 splits each item's KV range over several
@@ -337,6 +355,53 @@ int hds_multi_tensor_adam(int n_tensors, void* const* params, const void* const*
 int hds_multi_tensor_lion(int n_tensors, void* const* params, const void* const* grads, float* const* exp_avg,
                           const int64_t* numels, int param_dtype, int grad_dtype, float lr, float beta1, float beta2,
                           float weight_decay, float grad_scale, void* stream);
+
+/* ---- fp32 models, expert choice by table, fp32 residual stream, state-space mixers ----------------------------------- */
+
+/* D[M,N] = A[M,K] * W[N,K]^T in true fp32. epilogue 0 store + act, 1 gated (interleaved gate / up rows, out has N/2 columns),
+ * 2 out += D. group_off (optional, as hds_moe_gemm's pad_off): rows of group e use W[e*N:(e+1)*N]. limit: see below. */
+int hds_gemm_f32(const float* A, int64_t lda, const float* W, int64_t ldw, int M, int N, int K, int epilogue, int act, float limit,
+                 float* out, int64_t ldo, const int32_t* group_off, int n_groups, void* stream);
+
+/* act = 5 of the gated epilogues of hds_gemm, hds_gemm_2sm, hds_moe_gemm and hds_gemm_f32 bounds its inputs:
+ * g = min(gate, L), u = clamp(up, -L, L), out = g * sigmoid(1.702 g) * (u + 1). This sets L for the NEXT GEMM launch of the
+ * calling thread; cleared by that launch. */
+int hds_gemm_next_act_limit(float limit);
+
+/* Expert choice by token id: expert_ids[t, j] = table[ids[t], j], scores = 1 / k; offsets / counts as hds_moe_topk_gating. */
+int hds_moe_table_route(const int32_t* ids, const int32_t* table, int vocab, int T, int E, int k, float* scores, int32_t* expert_ids,
+                        int32_t* offsets, int32_t* counts, void* stream);
+/* out[t, :] = base[t, :] + sum_j scores[t, j] * y[mapped_slots[t, j], :] (stored; base optional; dtype of y and base 0 / 1 / 2). */
+int hds_moe_combine(const void* y, int64_t ldy, const int32_t* mapped_slots, const float* scores, const void* base, int64_t ldb,
+                    float* out, int64_t ldo, int T, int k, int H, int dtype, void* stream);
+
+/* out[t] = W[ids[t]] as fp32 (rows of H values; ids outside the vocabulary give zeros). dtype of W 0 / 1 / 2. */
+int hds_embed_f32(const int32_t* ids, const void* W, float* out, int T, int H, int vocab, int dtype, void* stream);
+
+/* One sublayer boundary of a stack with norms on both sides of its sublayers, on an fp32 residual stream x [rows, ld]:
+ *   x += (factor * delta) / rms(factor * delta) * post   (delta NULL: skipped);   out = x / rms(x) * gamma
+ * rms over the first `cols` values of a row (the rest of `padded` are zeros). An fp32 delta is cleared after being read; a
+ * 16-bit one has out's dtype. store_x 0: x is only read. dtype of out 0 bf16, 1 fp16, 2 fp32. All rows ld apart. */
+int hds_norm_residual(float* x, void* delta, int delta_is_f32, float factor, const float* post, const float* gamma, void* out,
+                      int64_t ld, int rows, int cols, int padded, float eps, int store_x, int dtype, void* stream);
+
+/* out = scale * w * v / rms(v) with v = y * silu(z), rms over each of `groups` equal parts of a row. y, w fp32; z, out dtype. */
+int hds_gated_norm(const float* y, int64_t ld_y, const void* z, int64_t ld_z, const float* w, void* out, int64_t ld_out, int rows,
+                   int cols, int groups, float eps, float scale, int dtype, void* stream);
+
+/* State-space (Mamba-2) mixer between its projections, over a ragged batch of T rows. proj: [T, ld_proj] rows of
+ * z | x (heads * vdim each) | B | C (groups * state_size each) | dt (heads). A causal convolution of `taps` taps (conv_w
+ * [taps, channels], conv_b) and silu over x | B | C; dt = softplus(dt + dt_bias); per head
+ *     S = exp(decay_rate * dt) S + dt * x B^T,   y = S C + skip * x.
+ * spans: int32 [n_seqs, 4] = (first row, new tokens, tokens seen before, slot); sequences in row order, together all T rows; a
+ * sequence with 0 tokens seen starts from zero. n_single of them bring one token. state [slots, heads, vdim, state_size] and
+ * conv_state [slots, taps, channels] (ring by position % taps) are fp32 and advanced in place. Scratch: u [T, ld_u] (dtype),
+ * dt [T, heads] fp32. y [T, heads * vdim] fp32, before the gate. method 0 picks, 1 forces the token-by-token kernel, 2 the
+ * chunked tensor-core one. */
+int hds_state_space(const void* proj, int64_t ld_proj, const float* conv_w, const float* conv_b, const float* dt_bias,
+                    const float* decay_rate, const float* skip, float* state, float* conv_state, const int32_t* spans, int n_seqs,
+                    int n_single, int T, int heads, int vdim, int state_size, int groups, int taps, void* u, int64_t ld_u, float* dt,
+                    float* y, int method, int dtype, void* stream);
 
 #ifdef __cplusplus
 }
