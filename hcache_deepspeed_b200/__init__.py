@@ -32,7 +32,8 @@ def init_inference(model, config=None, **kwargs):
     """Initialize the inference engine (v1 API).
 
     ``config`` may be a dict, a path to a JSON file, or None; keyword arguments are merged into it and a key given
-    both ways with different values is an error (same rule as ``deepspeed/__init__.py:341-362``).
+    both ways with different values is an error (same rule as ``deepspeed/__init__.py:341-362``). ``model`` is a module, or the
+    path of a checkpoint folder of a supported architecture (which then runs on the ragged executor).
     Returns an :class:`hcache_deepspeed_b200.inference.engine.InferenceEngine`.
     """
     from .inference.config import DeepSpeedInferenceConfig

@@ -43,6 +43,20 @@ class _Output(dict):
         return super().__getitem__(k)
 
 
+class CheckpointModel(torch.nn.Module):
+    """Stands for a model that exists only as a checkpoint folder: its config and the engine that streams its weights. The
+    ragged executor is its only implementation (architectures of this framework have no HuggingFace module)."""
+
+    def __init__(self, path: str) -> None:
+        super().__init__()
+        from .v2.checkpoint import HuggingFaceCheckpointEngine
+        self.checkpoint = HuggingFaceCheckpointEngine(path)
+        self.config = self.checkpoint.model_config
+
+    def forward(self, *_, **__):
+        raise RuntimeError("a checkpoint folder runs through the ragged executor only")
+
+
 class InferenceEngine(torch.nn.Module):
     inference_mp_group = None
     inference_ep_group = None
@@ -50,6 +64,8 @@ class InferenceEngine(torch.nn.Module):
 
     def __init__(self, model: torch.nn.Module, config: DeepSpeedInferenceConfig):
         super().__init__()
+        if isinstance(model, (str, os.PathLike)):
+            model = CheckpointModel(os.fspath(model))
         self.module = model
         self._config = config
         self.dtype = config.dtype
@@ -74,7 +90,7 @@ class InferenceEngine(torch.nn.Module):
             self._create_model_parallel_group(config)
         if config.checkpoint is not None:
             self._load_checkpoint(config.checkpoint, base_dir=config.base_dir)
-        self.injected = bool(config.replace_with_kernel_inject or config.hcache.enabled)
+        self.injected = bool(config.replace_with_kernel_inject or config.hcache.enabled) or isinstance(model, CheckpointModel)
         self.fused_layers = 0
         if self.injected and not config.hcache.enabled and not self._has_v2_policy():
             # families outside the ragged executor: per-layer injection of the v1 fused layer
@@ -180,7 +196,9 @@ class InferenceEngine(torch.nn.Module):
             quant = {"quantization_mode": "wf8af8"}
             dtype = torch.bfloat16 if self.device.type == "cuda" else torch.float32
             log_dist("init_inference: dtype=torch.int8 -> 8-bit serving through the E4M3 tensor-core path (wf8af8)", [0])
-        if self.device.type == "cuda" and dtype not in (torch.float16, torch.bfloat16):
+        from ..models.arch import arch_from_hf_config
+        fp32_ok = dtype == torch.float32 and arch_from_hf_config(self.module.config).layers is not None   # (models/hybrid.py)
+        if self.device.type == "cuda" and dtype not in (torch.float16, torch.bfloat16) and not fp32_ok:
             raise ValueError("the sm_100a kernels take fp16 or bf16; pass dtype=torch.bfloat16")
         if cfg.use_triton:
             log_dist("init_inference: use_triton is ignored (no Triton kernels in this build; the native sm_100a kernels run)", [0])
@@ -190,8 +208,8 @@ class InferenceEngine(torch.nn.Module):
         ecfg = RaggedInferenceEngineConfig(tensor_parallel={"tp_size": cfg.tensor_parallel.tp_size}, state_manager=state,
                                            hcache={"enabled": True, "capture": "sync" if hc.enabled else "off"},
                                            **({"quantization": quant} if quant else {}))
-        policy = MODEL_TYPE_TO_POLICY[mt](self.module.config, checkpoint_engine=InMemoryModelEngine(self.module), dtype=dtype,
-                                          device=self.device)
+        ckpt = self.module.checkpoint if isinstance(self.module, CheckpointModel) else InMemoryModelEngine(self.module)
+        policy = MODEL_TYPE_TO_POLICY[mt](self.module.config, checkpoint_engine=ckpt, dtype=dtype, device=self.device)
         self._engine = InferenceEngineV2(policy, ecfg)
         log_dist(f"init_inference: transformer stack of {mt} now runs on the {self._engine.model().ops.name} executor", [0])
 

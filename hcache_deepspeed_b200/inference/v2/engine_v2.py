@@ -225,6 +225,10 @@ class InferenceEngineV2:
         tokens to return logits for (in this order, all sequences concatenated; None instead of logits when there are none)
         in place of each sequence's last one."""
         uids, toks = list(batch_uids), list(batch_tokens)
+        if logits_at is not None:
+            picks = [list(map(int, p)) for p in logits_at]
+            if len(picks) != len(uids) or any(not 0 <= p < t.numel() for t, ps in zip(toks, picks) for p in ps):
+                raise ValueError("logits_at must list, for every sequence, places among its tokens")
         if do_checks:
             check = self.can_schedule(uids, [int(t.numel()) for t in toks])
             if check != SchedulingResult.Success:
@@ -246,10 +250,6 @@ class InferenceEngineV2:
                 capture = False
         rows = None
         if logits_at is not None:
-            picks = [list(map(int, p)) for p in logits_at]
-            if len(picks) != len(uids) or any(not 0 <= p < n for (_, n, _), ps in
-                                              zip(self._batch.inflight_seq_descriptors_shadow, picks) for p in ps):
-                raise ValueError("logits_at must list, for every sequence, places among its tokens")
             rows = [b + p for (b, _, _), ps in zip(self._batch.inflight_seq_descriptors_shadow, picks) for p in ps]
             if self._batch.current_tokens == self._batch.current_sequences and len(rows) == len(uids):
                 rows = None    # a decode step that wants every sequence's logits: the ordinary path

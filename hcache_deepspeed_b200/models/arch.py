@@ -500,11 +500,11 @@ def _nipolorn(cfg) -> ArchSpec:
 
 
 def stack_arch(model_type: str, layers: List[LayerSpec], hidden: int, vocab: int, norm_eps: float, **kw) -> ArchSpec:
-    """ArchSpec of a stack of unlike layers; its scalar sizes are the largest of any layer."""
+    """ArchSpec of a stack of unlike layers; its scalar sizes are those of the layer with the widest KV pages, or the largest of any."""
     attn = [l.mixer.attn for l in layers if l.mixer.attn is not None]
     mlps = [l.mlp for l in layers if l.mlp is not None]
     widest = max(attn, key=lambda a: a.kv_heads * a.page_dim, default=AttentionSpec(1, 1, 64, 64, 1.0))
-    return ArchSpec(model_type=model_type, n_layers=len(layers), hidden=hidden, n_heads=max((a.heads for a in attn), default=1),
+    return ArchSpec(model_type=model_type, n_layers=len(layers), hidden=hidden, n_heads=widest.heads,
                     n_kv_heads=widest.kv_heads, head_dim=widest.page_dim,
                     intermediate=max((m.ff for m in mlps if not m.experts), default=0), vocab=vocab, norm="rms",
                     norm_eps=norm_eps, act="silu", gated_mlp=True, pos_emb="none",
