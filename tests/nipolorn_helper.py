@@ -146,8 +146,9 @@ def error(got, want):
     return (d.pow(2).mean(-1).sqrt().max() / (want.double() - want.double().mean(-1, keepdim=True)).pow(2).mean().sqrt()).item()
 
 
-#: what rounding alone leaves: fp32 arithmetic, or 16-bit operands through a few layers
-TOLERANCE = {torch.float32: 1e-4, torch.bfloat16: 6e-2, torch.float16: 2e-2}
+#: what rounding alone leaves at the worst position: fp32 arithmetic, or 16-bit operands (whose rounding a norm can magnify where
+#: a sublayer's output is small); the fp32 runs are the sharp test of the bookkeeping
+TOLERANCE = {torch.float32: 1e-4, torch.bfloat16: 0.15, torch.float16: 3e-2}
 
 
 # ---- scenarios shared by the CPU and GPU tests ---------------------------------------------------------------------

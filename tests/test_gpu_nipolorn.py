@@ -154,6 +154,32 @@ def test_state_space_against_reference(heads, P, N, groups, taps, dtype, method)
             torch.testing.assert_close(ring[s].cpu()[filled], ring_ref[s][filled])
 
 
+@pytest.mark.parametrize("heads,P,N,groups", [(4, 64, 128, 2), (3, 48, 32, 1), (2, 128, 64, 1), (2, 8, 16, 2), (6, 40, 96, 3)])
+def test_chunked_scan_against_token_scan(heads, P, N, groups):
+    """The tensor-core scan keeps 16 bits of every fp32 operand: far closer to the fp32 scan than 16-bit rounding would be.
+    Lengths around the chunk borders, with and without carried state, fast and slow decays."""
+    inner, C, taps = heads * P, heads * P + 2 * groups * N, 4
+    cw, cb, db = rnd(taps, C, scale=0.6), rnd(C, seed=1, scale=0.2), rnd(heads, seed=2) - 1
+    a, dsk = -torch.exp(rnd(heads, seed=3, scale=2.0)), rnd(heads, seed=4)
+    for lens in ([2], [128, 127], [129, 3, 300], [64, 256, 2]):
+        T = sum(lens)
+        proj = rnd(T, 8 * ((2 * inner + 2 * groups * N + heads + 7) // 8), seed=T, dtype=BF16)
+        spans, row = [], 0
+        for i, n in enumerate(lens):
+            spans.append([row, n, 5 if i % 2 else 0, len(lens) - 1 - i])
+            row += n
+        outs = []
+        for method in (1, 2):
+            state, ring = rnd(len(lens), heads, P, N, seed=5), rnd(len(lens), taps, C, seed=6)
+            u = torch.zeros(T, 8 * ((C + 7) // 8), dtype=BF16, device="cuda")
+            dt, y = torch.zeros(T, heads, device="cuda"), torch.zeros(T, inner, device="cuda")
+            k().state_space(proj, cw, cb, db, a, dsk, state, ring, torch.tensor(spans, dtype=torch.int32, device="cuda"), 0, groups, u, dt, y,
+                            method=method)
+            outs.append((y, state, ring))
+        for got, want in zip(outs[1], outs[0]):
+            torch.testing.assert_close(got / want.abs().max(), want / want.abs().max(), rtol=0, atol=5e-5)
+
+
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("cols,groups", [(120, 5), (256, 1), (4096, 8), (51, 3)])
 def test_gated_norm(cols, groups, dtype):
