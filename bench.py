@@ -54,6 +54,9 @@ def parse():
                         "e.g. the OPT-30B TP=4 NVMe configuration), instead of what the planner would choose")
     p.add_argument("--plan", default="hidden", choices=["auto", "hidden", "planner", "adaptive"],
                    help="hidden: every layer from hidden states (fastest measured on 1xB200: 20.4 ms vs 21.6 ms); auto: planner mix with a recomputed prefix")
+    p.add_argument("--stacks", action="store_true",
+                   help="instead of the headline workload: prefill and decode throughput of the Nipolorn stacks beside the closest plain "
+                        "families at equal sizes, and their kernels against the measured peaks (one JSON line each; one GPU)")
     return p.parse_args()
 
 
@@ -333,7 +336,10 @@ def run_reference(a):
 
 if __name__ == "__main__":
     args = parse()
-    if args.impl == "reference":
+    if args.stacks:
+        from hcache_deepspeed_b200.benchmarks.stacks import main as run_stacks
+        run_stacks(args.steps, args.warmup)
+    elif args.impl == "reference":
         run_reference(args)
     else:
         run_ours(args)

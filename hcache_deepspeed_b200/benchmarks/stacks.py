@@ -1,0 +1,178 @@
+"""Throughput of stacks that mix attention with recurrent state, beside the closest plain families at equal sizes.
+
+``bench.py --stacks``. Four layers of each size, random weights, through the public engine: one 4096-token prompt, and decode steps
+of 8 and 64 sequences at 4096 tokens of context. Then the kernels that only such stacks use, each next to its counterpart in a
+plain family: CUDA-event medians with an L2-sized flush between launches, as fractions of the measured peaks.
+"""
+from __future__ import annotations
+
+import json
+import os
+import statistics
+from typing import Callable, Dict, Optional
+
+import torch
+
+PAIRS = [("nipolorn-2048", "mistral-2048"), ("nipolorn-4096", "mistral-4096"), ("nipolorn-4096-moe", "qwen2-moe-4096")]
+PROMPT = 4096
+
+
+def peaks() -> Dict[str, float]:
+    path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
+    out = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    if os.path.exists(path):
+        with open(path) as f:
+            out.update({k: v for k, v in json.load(f).items() if k in out})
+    return out
+
+
+def _time(fn: Callable[[], None], iters: int, warmup: int, before: Optional[Callable[[], None]] = None) -> float:
+    """Median milliseconds of ``fn`` on the device; ``before`` runs untimed in front of every iteration."""
+    times = []
+    for i in range(warmup + iters):
+        if before is not None:
+            before()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        fn()
+        b.record()
+        b.synchronize()
+        if i >= warmup:
+            times.append(a.elapsed_time(b))
+    return statistics.median(times)
+
+
+def bench_engine(name: str, steps: int, warmup: int) -> Dict[str, float]:
+    from ..inference.v2 import RaggedInferenceEngineConfig, build_engine_from_arch
+    from ..models.arch import named_arch
+    spec = named_arch(name)
+    eng = build_engine_from_arch(spec, RaggedInferenceEngineConfig(
+        state_manager={"max_tracked_sequences": 66, "max_ragged_batch_size": PROMPT, "max_ragged_sequence_count": 64, "max_context": PROMPT + 256,
+                       "memory_config": {"mode": "tokens", "size": 66 * (PROMPT + 256)}, "max_state_slots": 66},
+        hcache={"enabled": False, "capture": "off"}), seed=1, dtype=torch.bfloat16, device=torch.device("cuda"))
+    g = torch.Generator().manual_seed(0)
+    prompt = torch.randint(0, spec.vocab, (PROMPT, ), generator=g)
+    out = {}
+    ms = _time(lambda: eng.put([999], [prompt]), steps, warmup, before=lambda: eng.flush(999) if eng.state_manager.get_sequence(999) else None)
+    eng.flush(999)
+    out["prefill_ms"], out["prefill_tokens_per_s"] = round(ms, 3), round(PROMPT / ms * 1e3)
+    for uid in range(64):
+        eng.put([uid], [prompt])
+    for n in (8, 64):
+        uids = list(range(n))
+        cur = [torch.randint(0, spec.vocab, (1, ), generator=g) for _ in uids]
+        ms = _time(lambda: eng.put(uids, cur), 4 * steps, warmup + 4)
+        out[f"decode{n}_ms"], out[f"decode{n}_tokens_per_s"] = round(ms, 4), round(n / ms * 1e3)
+    out["weights_MiB"] = round(eng.model().w.n_bytes() / 2**20)
+    return out
+
+
+def bench_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
+    """Kernels of a stack next to the like kernel of a plain family (``like``), with bytes or flops that the operation itself
+    needs. Sizes: width 4096, 32 / 8 attention heads of 128, 128 state-space heads of 64 x 128 in 8 groups."""
+    from ..ops import kernels as K
+    dev, bf = "cuda", torch.bfloat16
+    flush = torch.empty(512 << 20, dtype=torch.uint8, device=dev)
+    W, T = 4096, PROMPT
+
+    def rnd(*shape, dtype=bf, scale=1.0):
+        return (torch.randn(shape, device=dev) * scale).to(dtype)
+
+    def report(op, kernel, fn, bytes_=0.0, flops=0.0):
+        ms = _time(fn, iters, warmup, before=flush.zero_)
+        need = max(bytes_ / (p["hbm_gbs"] * 1e6), flops / (p["bf16_tflops"] * 1e9))     # ms at the measured peaks
+        print(json.dumps({"op": op, "kernel": kernel, "us": round(ms * 1e3, 1), "roofline_us": round(need * 1e3, 1),
+                          "bound": "memory" if bytes_ / (p["hbm_gbs"] * 1e6) >= flops / (p["bf16_tflops"] * 1e9) else "math",
+                          "of_measured_peak": round(need / ms, 3)}), flush=True)
+
+    for rows in (T, 64):
+        x32, x16, d16, out = rnd(rows, W, dtype=torch.float32), rnd(rows, W), rnd(rows, W), rnd(rows, W)
+        g32, g16 = torch.ones(W, device=dev), torch.ones(W, device=dev, dtype=bf)
+        report(f"norm {rows}x{W}", "norm_residual", lambda: K.norm_residual(x32, g32, out, delta=d16, post=g32, eps=1e-5), rows * W * (4 + 4 + 2 + 2))
+        report(f"norm {rows}x{W}", "norm (like)", lambda: K.norm(x16, g16, out, delta=d16, res_out=x16, eps=1e-5), rows * W * (2 + 2 + 2 + 2))
+    heads, P, N, G = 128, 64, 128, 8
+    inner, C = heads * P, heads * P + 2 * G * N
+    ld = 2 * inner + 2 * G * N + heads
+    vec = lambda n: torch.randn(n, device=dev) * 0.5  # noqa: E731
+    cw, cb, db, a, d = torch.randn(4, C, device=dev) * 0.5, vec(C), vec(heads) - 3, -torch.exp(vec(heads)), vec(heads)
+    for rows, seqs in ((T, 1), (T, 4), (64, 64), (8, 8)):
+        n = rows // seqs
+        proj = rnd(rows, ld)
+        state, ring = torch.zeros(seqs, heads, P, N, device=dev), torch.zeros(seqs, 4, C, device=dev)
+        spans = torch.tensor([[i * n, n, 128, i] for i in range(seqs)], dtype=torch.int32, device=dev)
+        u, dt, y = torch.zeros(rows, C, dtype=bf, device=dev), torch.zeros(rows, heads, device=dev), torch.zeros(rows, inner, device=dev)
+        single = seqs if n == 1 else 0
+        # algorithmic bytes: projections in, y out, the states in and out
+        need = rows * (C * 2 + heads * 2 + inner * 4) + 2 * seqs * (heads * P * N + 4 * C) * 4
+        report(f"state space {seqs}x{n}", "conv + chunked scan" if n > 1 else "step", lambda: K.state_space(
+            proj, cw, cb, db, a, d, state, ring, spans, single, G, u, dt, y), need)
+        mix, w = rnd(rows, inner), torch.ones(inner, device=dev)
+        report(f"gated norm {rows}x{inner}", "gated_norm", lambda: K.gated_norm(y, proj[:, :inner], w, mix, G, 1e-5, 0.5), rows * inner * (4 + 2 + 2))
+    from ..ops.backend import pick_packed_splits, windowed_len
+    nq, nkv, D, page = 32, 8, 128, 64
+    ws = torch.zeros(256 << 20, dtype=torch.uint8, device=dev)
+    for window, keep in ((0, 0), (1024, 0), (1024, 64), (4096, 64)):
+        cache = rnd(T // page + 1, 2, nkv, page, D)
+        table = torch.randperm(T // page, device=dev).to(torch.int32)[None].contiguous()
+        q, o = rnd(T, nq * D), rnd(T, nq * D)
+        items = torch.tensor([[0, i, 128, i] for i in range(0, T, 128)], dtype=torch.int32, device=dev)
+        pairs = sum(i + 1 if not window else min(i + 1, window + max(0, min(keep, i + 1 - window))) for i in range(T))
+        report(f"attention prefill {T} window {window} keep {keep}", "paged_attention_prefill" + ("" if window or keep else " (like)"), lambda:
+               K.paged_attention_prefill(q, o, cache, table, items, T // 128, nq, nkv, D, page, 0.09, window=window, keep_first=keep),
+               flops=4.0 * pairs * nq * D)
+    B = 64
+    for window, keep in ((0, 0), (1024, 0), (1024, 64)):
+        cache = rnd(B * T // page, 2, nkv, page, D)
+        tables = torch.randperm(B * T // page, device=dev).to(torch.int32).view(B, T // page).contiguous()
+        q, o = rnd(B, nq * D), rnd(B, nq * D)
+        items = torch.tensor([[i, i, 1, T - 1] for i in range(B)], dtype=torch.int32, device=dev)
+        keys = T if not window else min(T, window + keep)
+        sp = pick_packed_splits(B, nkv, windowed_len(T, window, keep))
+        report(f"attention decode {B}x{T} window {window} keep {keep}", "paged_attention_packed" + ("" if window or keep else " (like)"), lambda:
+               K.paged_attention_prefill(q, o, cache, tables, items, B, nq, nkv, D, page, 0.09, n_splits=sp, workspace=ws, packed=True,
+                                         window=window, keep_first=keep), B * keys * 2 * nkv * D * 2)
+    del cache
+    ff = 14336
+    w_up = rnd(2 * ff, W, scale=0.02)
+    wsg = torch.zeros(K.gemm_splitk_workspace_bytes(128, 2 * ff), dtype=torch.uint8, device=dev)
+    for rows in (T, 64, 8):
+        x, h = rnd(rows, W), rnd(rows, ff)
+        for act, tag in ((5, "gated GEMM, clamped"), (3, "gated GEMM, silu (like)")):
+            report(f"mlp up {rows}x{2 * ff}x{W}", tag, lambda: K.gemm(x, w_up, out=h, act=act, gated=True, limit=7.0,
+                                                                       workspace=wsg if rows <= 128 else None),
+                   2 * (2 * ff * W + rows * (W + ff)), 2.0 * rows * 2 * ff * W)
+    E, top, V = 16, 2, 32000
+    i32 = lambda *s: torch.zeros(s, dtype=torch.int32, device=dev)  # noqa: E731
+    table = torch.stack([torch.randperm(E, device=dev)[:top] for _ in range(256)]).int().repeat(V // 256, 1).contiguous()
+    for rows in (T, 64):
+        scores, e, off, slots, counts, pad = torch.zeros(rows, top, device=dev), i32(rows, top), i32(rows, top), i32(rows, top), i32(E), i32(E + 1)
+        R = K.moe_padded_rows(rows, E, top)
+        x, xs, ys, base, out, lg = rnd(rows, W), rnd(R, W), rnd(R, W), rnd(rows, W), torch.zeros(rows, W, device=dev), rnd(rows, E)
+        ids = torch.randint(0, V, (rows, ), device=dev).int()
+
+        def by_table():
+            K.moe_table_route(ids, table, E, scores, e, off, counts)
+            K.moe_scatter(x, xs, e, off, counts, pad, slots, top)
+
+        def by_gate():
+            K.moe_topk_gating(lg, top, True, scores, e, off, counts)
+            K.moe_scatter(x, xs, e, off, counts, pad, slots, top)
+
+        report(f"route + scatter {rows}", "table", by_table, rows * W * 2 * (1 + top))
+        report(f"route + scatter {rows}", "top-k gate (like)", by_gate, rows * W * 2 * (1 + top))
+        report(f"combine {rows}", "moe_combine + shared", lambda: K.moe_combine(ys, slots, scores, base, out), rows * W * (2 * top + 2 + 4))
+        report(f"combine {rows}", "moe_gather (like)", lambda: K.moe_gather(ys, slots, scores, out), rows * W * (2 * top + 4 + 4))
+
+
+def main(steps: int = 5, warmup: int = 3) -> None:
+    p = peaks()
+    for pair in PAIRS:
+        for name in pair:
+            print(json.dumps({"stack": name, "layers": 4, "prompt": PROMPT, "dtype": "bf16", "data": "random weights, synthetic tokens",
+                              **bench_engine(name, steps, warmup)}), flush=True)
+            torch.cuda.empty_cache()
+    bench_kernels(p, max(steps, 10), warmup)
+
+
+if __name__ == "__main__":
+    main()

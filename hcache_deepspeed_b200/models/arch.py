@@ -538,6 +538,31 @@ def named_arch(name: str) -> ArchSpec:
         "tiny-opt-test": ArchSpec(n_layers=2, hidden=256, n_heads=4, n_kv_heads=4, intermediate=512,
                                   **{**opt, "vocab": 512, "head_dim": 64, "max_positions": 512}),
     }
+    table.update(_stack_named())
     if n not in table:
         raise KeyError(f"unknown named architecture {name}; known: {sorted(table)}")
     return table[n]
+
+
+def _stack_named() -> Dict[str, ArchSpec]:
+    """Nipolorn stacks with layers of real sizes, and beside each the closest plain family at equal sizes (same width, heads,
+    window and feed-forward): windowed attention with a dense MLP, or with routed experts and a shared one."""
+
+    def nipolorn(width, heads, kv, window, keep, ssm_heads, groups, mlp):
+        mixer = MixerSpec(attn=AttentionSpec(heads, kv, 128, 128, 128 ** -0.5, window, keep),
+                          ssm=StateSpaceSpec(ssm_heads, 64, 128, groups, 4, groups), attn_weight=1.0, ssm_weight=0.5)
+        return stack_arch("nipolorn", [LayerSpec(mixer, mlp)] * 4, hidden=width, vocab=32000, norm_eps=1e-5)
+
+    def plain(mt, width, heads, kv, window, **kw):
+        return ArchSpec(model_type=mt, n_layers=4, hidden=width, n_heads=heads, n_kv_heads=kv, head_dim=128, vocab=32000, norm="rms",
+                        norm_eps=1e-5, act="silu", gated_mlp=True, pos_emb="rope", sliding_window=window, max_positions=1 << 20, **kw)
+
+    moe = dict(n_experts=16, top_k=2, moe_intermediate=3584, shared_expert_intermediate=3584)
+    return {
+        "nipolorn-2048": nipolorn(2048, 16, 4, 1024, 16, 64, 4, FeedForwardSpec(ff=8192, act="swiglu_clamped", limit=7.0)),
+        "mistral-2048": plain("mistral", 2048, 16, 4, 1024, intermediate=8192),
+        "nipolorn-4096": nipolorn(4096, 32, 8, 4096, 64, 128, 8, FeedForwardSpec(ff=14336, act="swiglu_clamped", limit=7.0)),
+        "mistral-4096": plain("mistral", 4096, 32, 8, 4096, intermediate=14336),
+        "nipolorn-4096-moe": nipolorn(4096, 32, 8, 2048, 64, 64, 8, FeedForwardSpec(ff=3584, experts=16, top=2, shared_ff=3584)),
+        "qwen2-moe-4096": plain("qwen2_moe", 4096, 32, 8, 2048, intermediate=3584, **moe),
+    }

@@ -132,15 +132,27 @@ __global__ void moe_combine_kernel(const void* __restrict__ y, int64_t ldy, cons
                                    float* __restrict__ out, int64_t ldo, int H, int k) {
     pdl_enter();
     const int64_t t = blockIdx.x;
-    for (int c = threadIdx.x * 2; c < H; c += blockDim.x * 2) {
-        float a0 = base ? load_any<DT>(base, t * ldb + c) : 0.0f, a1 = base ? load_any<DT>(base, t * ldb + c + 1) : 0.0f;
-        for (int j = 0; j < k; ++j) {
-            const int64_t row = static_cast<int64_t>(mapped_slots[t * k + j]) * ldy;
-            const float s = scores[t * k + j];
-            a0 = fmaf(s, load_any<DT>(y, row + c), a0);
-            a1 = fmaf(s, load_any<DT>(y, row + c + 1), a1);
+    auto add8 = [](const void* p, int64_t idx, float s, float (&v)[8]) {
+        if constexpr (DT == 2) {
+            const float4* q = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + idx);
+            const float4 x = q[0], y = q[1];
+            v[0] = fmaf(s, x.x, v[0]); v[1] = fmaf(s, x.y, v[1]); v[2] = fmaf(s, x.z, v[2]); v[3] = fmaf(s, x.w, v[3]);
+            v[4] = fmaf(s, y.x, v[4]); v[5] = fmaf(s, y.y, v[5]); v[6] = fmaf(s, y.z, v[6]); v[7] = fmaf(s, y.w, v[7]);
+        } else {
+            const uint4 x = *reinterpret_cast<const uint4*>(reinterpret_cast<const char*>(p) + idx * 2);
+            v[0] = fmaf(s, unpack_lo<DT == 0>(x.x), v[0]); v[1] = fmaf(s, unpack_hi<DT == 0>(x.x), v[1]);
+            v[2] = fmaf(s, unpack_lo<DT == 0>(x.y), v[2]); v[3] = fmaf(s, unpack_hi<DT == 0>(x.y), v[3]);
+            v[4] = fmaf(s, unpack_lo<DT == 0>(x.z), v[4]); v[5] = fmaf(s, unpack_hi<DT == 0>(x.z), v[5]);
+            v[6] = fmaf(s, unpack_lo<DT == 0>(x.w), v[6]); v[7] = fmaf(s, unpack_hi<DT == 0>(x.w), v[7]);
         }
-        *reinterpret_cast<float2*>(out + t * ldo + c) = make_float2(a0, a1);
+    };
+    for (int c = threadIdx.x * 8; c < H; c += blockDim.x * 8) {
+        float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+        if (base != nullptr) add8(base, t * ldb + c, 1.0f, v);
+        for (int j = 0; j < k; ++j) add8(y, static_cast<int64_t>(mapped_slots[t * k + j]) * ldy + c, scores[t * k + j], v);
+        float4* o = reinterpret_cast<float4*>(out + t * ldo + c);
+        o[0] = make_float4(v[0], v[1], v[2], v[3]);
+        o[1] = make_float4(v[4], v[5], v[6], v[7]);
     }
 }
 
@@ -265,11 +277,11 @@ extern "C" int hds_moe_table_route(const int32_t* ids, const int32_t* table, int
 
 extern "C" int hds_moe_combine(const void* y, int64_t ldy, const int32_t* mapped_slots, const float* scores, const void* base,
                                int64_t ldb, float* out, int64_t ldo, int T, int k, int H, int dtype, void* stream) {
-    HDS_REQUIRE(H % 2 == 0 && ldo % 2 == 0, "hds_moe_combine: even row widths");
+    HDS_REQUIRE(H % 8 == 0 && ldy % 8 == 0 && ldo % 4 == 0 && (base == nullptr || ldb % 8 == 0), "hds_moe_combine: rows of 8-value vectors");
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_moe_combine: dtype 0 bf16 / 1 fp16 / 2 fp32");
     if (T == 0) return HDS_OK;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    const dim3 block(H >= 512 ? 256 : 128);
+    const dim3 block(H / 8 >= 512 ? 512 : H / 8 >= 256 ? 256 : 128);
     if (dtype == 0)
         HDS_CHECK_CUDA(launch_kernel(moe_combine_kernel<0>, dim3(T), block, 0, s, y, ldy, mapped_slots, scores, base, ldb, out, ldo, H, k));
     else if (dtype == 1)

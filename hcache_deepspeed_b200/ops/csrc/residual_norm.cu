@@ -127,6 +127,64 @@ static int launch_norm_residual(float* x, void* delta, float factor, const float
     return HDS_OK;
 }
 
+template <int DT>
+__device__ __forceinline__ float gate_silu(float b) {
+    return DT == 2 ? b / (1.0f + expf(-b)) : __fdividef(b, 1.0f + __expf(-b));
+}
+
+// One warp per (row, part) of up to 128 * VPT values (a multiple of 4), all in registers.
+template <int DT, int VPT>
+__global__ void __launch_bounds__(256)
+gated_norm_warp_kernel(const float* __restrict__ y, int64_t ld_y, const void* __restrict__ z, int64_t ld_z, const float* __restrict__ w,
+                       void* __restrict__ out, int64_t ld_out, int rows, int groups, int part, float eps, float scale) {
+    pdl_enter();
+    const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (unit >= rows * groups) return;
+    const int64_t t = unit / groups;
+    const int c0 = unit % groups * part;
+    float4 g[VPT], b[VPT];
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+        const int c = (lane + 32 * i) * 4;
+        g[i] = b[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < part) {
+            g[i] = *reinterpret_cast<const float4*>(y + t * ld_y + c0 + c);
+            b[i] = load4<DT>(z, t * ld_z + c0 + c);
+        }
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+        g[i].x *= gate_silu<DT>(b[i].x);
+        g[i].y *= gate_silu<DT>(b[i].y);
+        g[i].z *= gate_silu<DT>(b[i].z);
+        g[i].w *= gate_silu<DT>(b[i].w);
+        ss += g[i].x * g[i].x + g[i].y * g[i].y + g[i].z * g[i].z + g[i].w * g[i].w;
+    }
+    const float r = scale / sqrtf(warp_sum(ss) / part + eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+        const int c = (lane + 32 * i) * 4;
+        if (c < part) {
+            const float4 ww = *reinterpret_cast<const float4*>(w + c0 + c);
+            store4<DT>(out, t * ld_out + c0 + c, make_float4(g[i].x * r * ww.x, g[i].y * r * ww.y, g[i].z * r * ww.z, g[i].w * r * ww.w));
+        }
+    }
+}
+
+template <int DT>
+static cudaError_t launch_gated_norm_warp(const float* y, int64_t ld_y, const void* z, int64_t ld_z, const float* w, void* out, int64_t ld_out,
+                                          int rows, int groups, int part, float eps, float scale, cudaStream_t s) {
+    const dim3 grid((static_cast<int64_t>(rows) * groups + 7) / 8), block(256);
+#define HDS_GNW(V) \
+    return launch_kernel(gated_norm_warp_kernel<DT, V>, grid, block, 0, s, y, ld_y, z, ld_z, w, out, ld_out, rows, groups, part, eps, scale)
+    if (part <= 128) HDS_GNW(1);
+    if (part <= 256) HDS_GNW(2);
+    if (part <= 512) HDS_GNW(4);
+    HDS_GNW(8);
+#undef HDS_GNW
+}
+
 // One CTA per (row, part). y fp32, z in the I/O type; any part size.
 template <int DT>
 __global__ void __launch_bounds__(256)
@@ -144,17 +202,17 @@ gated_norm_kernel(const float* __restrict__ y, int64_t ld_y, const void* __restr
             const float4 a = *reinterpret_cast<const float4*>(y + t * ld_y + c0 + c);
             const float4 b = load4<DT>(z, t * ld_z + c0 + c);
             float4 g;
-            g.x = a.x * (b.x / (1.0f + expf(-b.x)));
-            g.y = a.y * (b.y / (1.0f + expf(-b.y)));
-            g.z = a.z * (b.z / (1.0f + expf(-b.z)));
-            g.w = a.w * (b.w / (1.0f + expf(-b.w)));
+            g.x = a.x * gate_silu<DT>(b.x);
+            g.y = a.y * gate_silu<DT>(b.y);
+            g.z = a.z * gate_silu<DT>(b.z);
+            g.w = a.w * gate_silu<DT>(b.w);
             *reinterpret_cast<float4*>(vals + c) = g;
             ss += g.x * g.x + g.y * g.y + g.z * g.z + g.w * g.w;
         }
     } else {
         for (int c = threadIdx.x; c < part; c += 256) {
             const float b = load_any<DT>(z, t * ld_z + c0 + c);
-            const float g = y[t * ld_y + c0 + c] * (b / (1.0f + expf(-b)));
+            const float g = y[t * ld_y + c0 + c] * gate_silu<DT>(b);
             vals[c] = g;
             ss += g * g;
         }
@@ -220,6 +278,13 @@ extern "C" int hds_gated_norm(const float* y, int64_t ld_y, const void* z, int64
     const size_t smem = static_cast<size_t>(part) * 4;
     const dim3 grid(rows, groups);
     cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const uintptr_t al = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(z) * 2 |
+                         reinterpret_cast<uintptr_t>(out) * 2;   // 16-byte vectors of fp32, 8-byte ones of the 16-bit types
+    if (part % 4 == 0 && part <= 1024 && ld_y % 4 == 0 && ld_z % 4 == 0 && ld_out % 4 == 0 && (al & 15) == 0 && dtype != 2) {
+        HDS_CHECK_CUDA(dtype == 0 ? launch_gated_norm_warp<0>(y, ld_y, z, ld_z, w, out, ld_out, rows, groups, part, eps, scale, s)
+                                  : launch_gated_norm_warp<1>(y, ld_y, z, ld_z, w, out, ld_out, rows, groups, part, eps, scale, s));
+        return HDS_OK;
+    }
     if (dtype == 0)
         HDS_CHECK_CUDA(launch_kernel(gated_norm_kernel<0>, grid, dim3(256), smem, s, y, ld_y, z, ld_z, w, out, ld_out, part, eps, scale));
     else if (dtype == 1)

@@ -16,8 +16,9 @@ namespace hds {
 constexpr int kConvRows = 16;      // rows of the batch per block
 constexpr int kConvThreads = 256;
 
-// Thread = one channel (VEC = 1) or two neighbouring ones (VEC = 2), walking kConvRows rows with the last TAPS - 1 inputs in
-// registers. TAPS 0: any number of taps, inputs re-read. Blocks behind the channel blocks compute step sizes.
+// Thread = VEC neighbouring channels, walking kConvRows rows with the last TAPS - 1 inputs in registers. TAPS 0: any number of
+// taps, inputs re-read. Blocks whose rows all belong to one sequence load them up front (VEC 4). Blocks behind the channel
+// blocks compute step sizes.
 template <int DT, int TAPS, int VEC>
 __global__ void __launch_bounds__(kConvThreads) ssm_conv_kernel(const SsmArgs a, int channel_blocks) {
     pdl_enter();
@@ -59,6 +60,40 @@ __global__ void __launch_bounds__(kConvThreads) ssm_conv_kernel(const SsmArgs a,
     };
     SsmSpan sp = a.spans[s];
     bool fresh = true;
+    if constexpr (TAPS > 1 && VEC == 4 && DT != 2) {
+        if (sp.n > 1 && r_end - r_begin == kConvRows && r_end <= sp.row0 + sp.n) {
+            const char* src = reinterpret_cast<const char*>(a.proj) + (static_cast<int64_t>(r_begin) * a.ld_proj + inner + c) * 2;
+            uint2 q[kConvRows];
+#pragma unroll
+            for (int i = 0; i < kConvRows; ++i) q[i] = *reinterpret_cast<const uint2*>(src + static_cast<int64_t>(i) * a.ld_proj * 2);
+#pragma unroll
+            for (int k = 0; k + 1 < TAPS; ++k)
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) win[k][v] = input(sp, r_begin - sp.row0 - (TAPS - 1) + k, v);
+            char* dst = reinterpret_cast<char*>(a.u) + (static_cast<int64_t>(r_begin) * a.ld_u + c) * 2;
+#pragma unroll
+            for (int i = 0; i < kConvRows; ++i) {
+                const float x[4] = {unpack_lo<DT == 0>(q[i].x), unpack_hi<DT == 0>(q[i].x), unpack_lo<DT == 0>(q[i].y), unpack_hi<DT == 0>(q[i].y)};
+                float o[4];
+#pragma unroll
+                for (int v = 0; v < VEC; ++v) {
+                    o[v] = b[v];
+#pragma unroll
+                    for (int k = 0; k + 1 < TAPS; ++k) o[v] = fmaf(win[k][v], w[k][v], o[v]);
+                    o[v] = fmaf(x[v], w[TAPS - 1][v], o[v]);
+#pragma unroll
+                    for (int k = 0; k + 2 < TAPS; ++k) win[k][v] = win[k + 1][v];
+                    win[TAPS - 2][v] = x[v];
+                    o[v] = ssm_silu<DT>(o[v]);
+                }
+                uint2 p;
+                p.x = pack2<DT == 0>(o[0], o[1]);
+                p.y = pack2<DT == 0>(o[2], o[3]);
+                *reinterpret_cast<uint2*>(dst + static_cast<int64_t>(i) * a.ld_u * 2) = p;
+            }
+            return;
+        }
+    }
     for (int r = r_begin; r < r_end; ++r) {
         while (r >= sp.row0 + sp.n) {
             sp = a.spans[++s];
@@ -105,10 +140,10 @@ __global__ void __launch_bounds__(kConvThreads) ssm_conv_kernel(const SsmArgs a,
         }
         if constexpr (VEC == 2 && DT != 2) {
             *reinterpret_cast<uint32_t*>(reinterpret_cast<char*>(a.u) + (static_cast<int64_t>(r) * a.ld_u + c) * 2) =
-                pack2<DT == 0>(ssm_silu(out[0]), ssm_silu(out[1]));
+                pack2<DT == 0>(ssm_silu<DT>(out[0]), ssm_silu<DT>(out[1]));
         } else {
 #pragma unroll
-            for (int v = 0; v < VEC; ++v) ssm_store<DT>(a.u, static_cast<int64_t>(r) * a.ld_u + c + v, ssm_silu(out[v]));
+            for (int v = 0; v < VEC; ++v) ssm_store<DT>(a.u, static_cast<int64_t>(r) * a.ld_u + c + v, ssm_silu<DT>(out[v]));
         }
     }
 }
@@ -224,7 +259,7 @@ __global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(const SsmArgs a)
             if (p >= 0) v = fmaf(ring[static_cast<int64_t>(p % taps) * C + c], a.conv_w[static_cast<int64_t>(k) * C + c], v);
         }
         v = fmaf(x, a.conv_w[static_cast<int64_t>(taps - 1) * C + c], v);
-        sm[e] = ssm_round<DT>(ssm_silu(v));
+        sm[e] = ssm_round<DT>(ssm_silu<DT>(v));
         // the ring entry of this position is read by nobody in this launch
         if (e >= 2 * N || h % per == 0) ring[static_cast<int64_t>(pos % taps) * C + c] = x;
     }
@@ -280,9 +315,13 @@ static int launch_conv(const SsmArgs& a, cudaStream_t s) {
     const int C = a.channels();
     const bool pair = C % 2 == 0 && a.inner() % 2 == 0 && a.ld_u % 2 == 0 && a.ld_proj % 2 == 0 &&
                       (reinterpret_cast<uintptr_t>(a.proj) & 3) == 0;
-    const int cb = (C / (pair ? 2 : 1) + kConvThreads - 1) / kConvThreads;
+    const bool quad = DT != 2 && a.taps == 4 && C % 4 == 0 && a.inner() % 4 == 0 && a.ld_u % 4 == 0 && a.ld_proj % 4 == 0 &&
+                      (reinterpret_cast<uintptr_t>(a.proj) & 7) == 0;
+    const int vec = quad ? 4 : pair ? 2 : 1;
+    const int cb = (C / vec + kConvThreads - 1) / kConvThreads;
     const dim3 grid((a.T + kConvRows - 1) / kConvRows, cb + 1);
-    if (a.taps == 4 && pair) HDS_CHECK_CUDA(launch_kernel(ssm_conv_kernel<DT, 4, 2>, grid, dim3(kConvThreads), 0, s, a, cb));
+    if (quad) HDS_CHECK_CUDA(launch_kernel(ssm_conv_kernel<DT, 4, DT == 2 ? 1 : 4>, grid, dim3(kConvThreads), 0, s, a, cb));
+    else if (a.taps == 4 && pair) HDS_CHECK_CUDA(launch_kernel(ssm_conv_kernel<DT, 4, 2>, grid, dim3(kConvThreads), 0, s, a, cb));
     else if (a.taps == 4) HDS_CHECK_CUDA(launch_kernel(ssm_conv_kernel<DT, 4, 1>, grid, dim3(kConvThreads), 0, s, a, cb));
     else if (pair) HDS_CHECK_CUDA(launch_kernel(ssm_conv_kernel<DT, 0, 2>, grid, dim3(kConvThreads), 0, s, a, cb));
     else HDS_CHECK_CUDA(launch_kernel(ssm_conv_kernel<DT, 0, 1>, grid, dim3(kConvThreads), 0, s, a, cb));

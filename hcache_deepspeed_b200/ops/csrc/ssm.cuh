@@ -43,7 +43,11 @@ __device__ __forceinline__ float ssm_round(float v) {
     if constexpr (DT == 1) return __half2float(__float2half_rn(v));
     return v;
 }
-__device__ __forceinline__ float ssm_silu(float v) { return v / (1.0f + expf(-v)); }
+// (fast intrinsics where the result is rounded to 16 bits anyway)
+template <int DT>
+__device__ __forceinline__ float ssm_silu(float v) {
+    return DT == 2 ? v / (1.0f + expf(-v)) : __fdividef(v, 1.0f + __expf(-v));
+}
 __device__ __forceinline__ float ssm_softplus(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
 
 // Latest inputs of a sequence's convolution channels [c0, c1) -> the ring (all threads of the block).
