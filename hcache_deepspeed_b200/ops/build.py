@@ -25,6 +25,11 @@ OBJ_DIR = OPS_DIR / "lib" / "obj"
 REPO_INCLUDE = OPS_DIR.parent / "include" if (OPS_DIR.parent / "include" / "hds_b200.h").exists() else OPS_DIR.parent.parent / "include"
 
 CUDA_LIB = LIB_DIR / "libhds_b200.so"
+#: what a first use on a machine without the full library builds: the units a 16-bit or fp32 model is served with (no FP8 GEMMs,
+#: quantisers, optimizers, host buffers; `native.cuda_lib` builds the full library when one of those is asked for)
+SERVE_LIB = LIB_DIR / "libhds_serve.so"
+SERVE_UNITS = ("gemm", "gemm_2sm", "gemm_f32", "elementwise", "residual_norm", "attention_splitkv", "attention_prefill",
+               "attention_generic", "moe", "ssm", "ssm_chunk", "tp_comm")
 HOST_LIB = LIB_DIR / "libhds_host.so"
 
 NVCC_FLAGS = [
@@ -55,11 +60,13 @@ def _run(cmd) -> None:
         raise RuntimeError("build command failed:\n  " + " ".join(map(str, cmd)) + "\n" + res.stdout)
 
 
-def build_cuda(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every ``csrc/*.cu`` for sm_100a and link ``libhds_b200.so``."""
+def build_cuda(force: bool = False, verbose: bool = False, serve_only: bool = False) -> Path:
+    """Compile every ``csrc/*.cu`` for sm_100a and link ``libhds_b200.so``; with ``serve_only`` the serving units alone, linked
+    into ``libhds_serve.so``."""
+    lib = SERVE_LIB if serve_only else CUDA_LIB
     LIB_DIR.mkdir(exist_ok=True)
     OBJ_DIR.mkdir(exist_ok=True)
-    sources = sorted(CSRC.glob("*.cu"))
+    sources = [s for s in sorted(CSRC.glob("*.cu")) if not serve_only or s.stem in SERVE_UNITS]
     headers = sorted(CSRC.glob("*.cuh")) + sorted(REPO_INCLUDE.glob("*.h"))
     nvcc = _nvcc()
     jobs = []
@@ -73,11 +80,11 @@ def build_cuda(force: bool = False, verbose: bool = False) -> Path:
         with ThreadPoolExecutor(max_workers=min(len(jobs), os.cpu_count() or 4)) as pool:
             list(pool.map(_run, jobs))
     objs = [OBJ_DIR / (s.stem + ".o") for s in sources]
-    if force or jobs or _newer(objs, CUDA_LIB):
+    if force or jobs or _newer(objs, lib):
         # static cudart (nvcc default): no runtime dependency beyond the driver; streams and pointers
         # created by torch's runtime are driver handles and are valid here
-        _run([nvcc, "-shared", "-o", str(CUDA_LIB), *map(str, objs), "-gencode", "arch=compute_100a,code=sm_100a"])
-    return CUDA_LIB
+        _run([nvcc, "-shared", "-o", str(lib), *map(str, objs), "-gencode", "arch=compute_100a,code=sm_100a"])
+    return lib
 
 
 def build_host(force: bool = False, verbose: bool = False) -> Path:

@@ -30,7 +30,7 @@ class HdsKernelError(RuntimeError):
     pass
 
 
-def _declare_cuda(lib: ctypes.CDLL) -> None:
+def _declare_cuda(lib: ctypes.CDLL, partial: bool = False) -> None:
     P, I, L, F = c_void_p, c_int, c_int64, c_float
     lib.hds_last_error.restype = c_char_p
     lib.hds_last_error.argtypes = []
@@ -94,6 +94,8 @@ def _declare_cuda(lib: ctypes.CDLL) -> None:
         "hds_multi_tensor_lion": [I, P, P, P, P, I, I, F, F, F, F, F, P],
     }
     for name, argtypes in sigs.items():
+        if partial and not hasattr(lib, name):
+            continue
         fn = getattr(lib, name)
         fn.argtypes = argtypes
         fn.restype = c_int
@@ -116,23 +118,42 @@ def _declare_cuda(lib: ctypes.CDLL) -> None:
             fn.restype = restype
 
 
-def cuda_lib(build_if_missing: bool = True) -> ctypes.CDLL:
-    """Return the loaded sm_100a kernel library (building it in-tree first if it is absent)."""
+class _ServeLib:
+    """The serving library; an entry point it does not hold is taken from the full one, which is then built."""
+
+    def __init__(self, lib: ctypes.CDLL) -> None:
+        self._lib, self._full = lib, None
+
+    def __getattr__(self, name: str):
+        try:
+            return getattr(self._lib, name)
+        except AttributeError:
+            if self._full is None:
+                from . import build
+                self._full = ctypes.CDLL(str(build.build_cuda(verbose=True)))
+                _declare_cuda(self._full)
+            return getattr(self._full, name)
+
+
+def cuda_lib(build_if_missing: bool = True):
+    """Return the loaded sm_100a kernel library: the full one when it has been built, else the serving one (built in-tree first
+    if it is absent too)."""
     global _cuda_lib
     if _cuda_lib is not None:
         return _cuda_lib
-    path = LIB_DIR / "libhds_b200.so"
-    if not path.exists() and build_if_missing and os.environ.get("HDS_NO_AUTOBUILD") != "1":
+    path, serve = LIB_DIR / "libhds_b200.so", LIB_DIR / "libhds_serve.so"
+    if not path.exists() and not serve.exists() and build_if_missing and os.environ.get("HDS_NO_AUTOBUILD") != "1":
         from . import build
-        build.build_cuda(verbose=True)
-    if not path.exists():
+        build.build_cuda(verbose=True, serve_only=True)
+    if not path.exists() and not serve.exists():
         raise NativeLibraryError(
             f"{path} is missing: run `python -m hcache_deepspeed_b200.ops.build` (needs nvcc). "
             "The GPU path never falls back to eager PyTorch.")
-    lib = ctypes.CDLL(str(path), mode=ctypes.RTLD_GLOBAL)
-    _declare_cuda(lib)
-    _cuda_lib = lib
-    return lib
+    full = path.exists()
+    lib = ctypes.CDLL(str(path if full else serve), mode=ctypes.RTLD_GLOBAL)
+    _declare_cuda(lib, partial=not full)
+    _cuda_lib = lib if full else _ServeLib(lib)
+    return _cuda_lib
 
 
 def cuda_lib_loaded() -> bool:
