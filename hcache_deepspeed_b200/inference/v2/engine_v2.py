@@ -189,6 +189,8 @@ class InferenceEngineV2:
         model.finish_pending_restore()
         if len(rl) + len(list(hidden_layers)) + len(list(kv_layers)) != model.spec.n_layers:
             raise ValueError("the plan does not cover every layer exactly once")
+        if len(list(kv_layers)) and model.spec.has_recurrent_state:
+            raise ValueError("KV pages do not hold a layer's recurrent state: restore such models from hidden states or recompute")
         self._batch.clear()
         seq = self._state_manager.get_or_create_sequence(uid)
         if seq.seen_tokens != 0:

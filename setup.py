@@ -85,7 +85,7 @@ setup(
     package_data={PKG: ["ops/csrc/*.cu", "ops/csrc/*.cuh", "ops/csrc_host/*.cpp", "ops/csrc_host/*.h", "ops/lib/*.so",
                         ]},
     data_files=[("include", ["include/hds_b200.h", "include/hds_host.h"])],
-    scripts=["bin/hds", "bin/hds_report", "bin/hds_bench", "bin/hds_elastic", "bin/hds_ssh", "bin/hds_io", "bin/hds_nvme_tune"],
+    scripts=["bin/hds", "bin/hds_report", "bin/hds_bench", "bin/hds_elastic", "bin/hds_ssh", "bin/hds_io", "bin/hds_nvme_tune", "bin/trace_run"],
     python_requires=">=3.10",
     install_requires=["torch>=2.6", "numpy", "pydantic>=2", "packaging", "psutil", "tqdm"],
     extras_require={"hf": ["transformers", "safetensors"], "dev": ["pytest", "pytest-timeout"]},

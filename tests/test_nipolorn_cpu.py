@@ -111,6 +111,23 @@ def test_restore_from_hidden_states():
     H.check_restore(H.MIXED, F32, "cpu")
 
 
+def test_sessions_are_saved_and_restored_without_pages():
+    """Multi-turn sessions: the planner keeps to hidden states (and recomputation), which bring the recurrent state back."""
+    from hcache_deepspeed_b200.hcache import HCacheSessionManager
+    cfg = H.MIXED
+    w, t = H.weights(cfg), H.tokens(cfg, 90)
+    eng = H.engine(cfg, w, enabled=True, capture="sync")
+    m = HCacheSessionManager(eng)
+    m.prefill(3, t[:50])
+    kinds = m.end_turn(3).kinds
+    assert "kv" not in kinds
+    eng.put([8], [H.tokens(cfg, 70, seed=4)])        # another sequence takes over pages and slot meanwhile
+    eng.flush(8)
+    assert H.error(m.prefill(3, t[50:]).float(), H.expected(cfg, w, t)[-1:]) < H.TOLERANCE[F32]
+    with pytest.raises(ValueError, match="recurrent"):
+        eng.restore_session(4, t[:50], kv=None, kv_layers=[0, 1, 2, 3])
+
+
 def test_greedy_generation(tmp_path):
     H.check_greedy(H.MIXED, F32, False, tmp_path / "m")
 
