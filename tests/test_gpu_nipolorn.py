@@ -52,7 +52,7 @@ KINDS = [("split1", 64, 2, 2), ("split3", 64, 4, 2), ("split2", 128, 3, 1), ("pa
 
 
 @pytest.mark.parametrize("kind,d,n_q,n_kv", KINDS)
-@pytest.mark.parametrize("window,keep", [(40, 6), (1, 1), (128, 0), (200, 130), (300, 64), (64, 300)])
+@pytest.mark.parametrize("window,keep", [(48, 5), (1, 1), (128, 0), (200, 130), (300, 64), (64, 300)])
 def test_planted_key_is_seen_exactly_inside_its_window(kind, d, n_q, n_kv, window, keep):
     """A key of huge score is planted at one position; its value shows in the output of exactly the queries that see it:
     positions at the window's and the kept range's edges, at page borders, far back and first of all."""
@@ -227,7 +227,7 @@ def test_clamped_gate_epilogue(M, ff, K, dtype):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("E,top,shared", [(5, 2, True), (16, 1, True), (9, 3, False)])
+@pytest.mark.parametrize("E,top,shared", [(5, 2, True), (12, 1, True), (9, 3, False)])
 def test_table_moe(E, top, shared, dtype):
     from hcache_deepspeed_b200.models.arch import FeedForwardSpec
     from hcache_deepspeed_b200.models.weights import ExpertWeights, LayerWeights
