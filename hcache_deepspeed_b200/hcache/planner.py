@@ -79,8 +79,8 @@ def plan_restore(spec: ArchSpec, n_tokens: int, link: Optional[LinkModel] = None
     interleaved with the projections, so its duration belongs on the compute side of the balance.
     """
     link = link or LinkModel()
-    if spec.has_recurrent_state:
-        allow_kv = False      # pages alone do not bring a layer's recurrent state back; hidden states and recomputation do
+    if not spec.pages_hold_context:
+        allow_kv = False      # K / V pages alone do not bring a layer's context back; hidden states and recomputation do
     L = spec.n_layers
     a, b, c, f = _costs(spec, n_tokens, link, from_nvme, elem)
     best = None

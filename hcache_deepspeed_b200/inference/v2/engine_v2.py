@@ -189,8 +189,9 @@ class InferenceEngineV2:
         model.finish_pending_restore()
         if len(rl) + len(list(hidden_layers)) + len(list(kv_layers)) != model.spec.n_layers:
             raise ValueError("the plan does not cover every layer exactly once")
-        if len(list(kv_layers)) and model.spec.has_recurrent_state:
-            raise ValueError("KV pages do not hold a layer's recurrent state: restore such models from hidden states or recompute")
+        if len(list(kv_layers)) and not model.spec.pages_hold_context:
+            raise ValueError("K / V pages do not hold the context of layers with recurrent state or latents: restore such models from "
+                             "hidden states or recompute")
         self._batch.clear()
         seq = self._state_manager.get_or_create_sequence(uid)
         if seq.seen_tokens != 0:

@@ -174,8 +174,12 @@ class NipolornPolicy(InferenceV2Policy):
     """Windowed attention with kept first tokens beside a Mamba-2 mixer in every layer; experts chosen by token id."""
 
 
+class DedelornPolicy(InferenceV2Policy):
+    """Layers of a gated delta rule or of latent attention, each beside its feed-forward on one norm."""
+
+
 MODEL_TYPE_TO_POLICY = {
-    "nipolorn": NipolornPolicy,
+    "nipolorn": NipolornPolicy, "dedelorn": DedelornPolicy,
     "gpt2": GPT2Policy, "gptj": GPTJPolicy, "gpt_neox": GPTNeoXPolicy, "bloom": BloomPolicy, "gpt_neo": GPTNeoPolicy,
     "llama": Llama2Policy, "opt": OPTPolicy, "mistral": MistralPolicy, "mixtral": MixtralPolicy, "falcon": FalconPolicy,
     "phi": PhiPolicy, "phi3": Phi3Policy, "qwen": QwenPolicy, "qwen2": Qwen2Policy, "qwen2_moe": Qwen2MoePolicy,

@@ -52,11 +52,11 @@ class BlockedKVCache:
             dtype = DtypeEnum(dtype).value
         self._dtype = dtype
         elem = torch.tensor([], dtype=dtype).element_size()
-        shapes = cfg.layer_shapes if cfg.layer_shapes is not None else [(n_heads, head_dim)] * num_layers
+        shapes = cfg.layer_shapes if cfg.layer_shapes is not None else [(2, n_heads, head_dim)] * num_layers
         self._layer_shapes = shapes
         self._uniform = all(s == shapes[0] and s is not None for s in shapes)
         self._block_bytes_per_layer = 2 * n_heads * cfg.block_size * head_dim * elem
-        per_block_bytes = max(1, sum(2 * s[0] * cfg.block_size * s[1] * elem for s in shapes if s is not None))
+        per_block_bytes = max(1, sum(s[0] * s[1] * cfg.block_size * s[2] * elem for s in shapes if s is not None))
         self._per_block_bytes = per_block_bytes
 
         mode = memory_config.mode
@@ -88,10 +88,10 @@ class BlockedKVCache:
             f"Allocating KV-cache: {num_blocks} blocks x {per_block_bytes} B = {num_blocks * per_block_bytes / 2**30:.2f} GiB "
             f"(layers={num_layers}, kv_heads={n_heads}, block={cfg.block_size}, head_dim={head_dim}, {dtype})")
         if self._uniform:
-            self._cache = torch.zeros((num_layers, num_blocks, 2, shapes[0][0], cfg.block_size, shapes[0][1]), dtype=dtype,
+            self._cache = torch.zeros((num_layers, num_blocks, shapes[0][0], shapes[0][1], cfg.block_size, shapes[0][2]), dtype=dtype,
                                       device=self._device)
         else:   # unlike layers: the same block ids, one tensor per layer
-            self._cache = [None if s is None else torch.zeros((num_blocks, 2, s[0], cfg.block_size, s[1]), dtype=dtype,
+            self._cache = [None if s is None else torch.zeros((num_blocks, s[0], s[1], cfg.block_size, s[2]), dtype=dtype,
                                                               device=self._device) for s in shapes]
 
     # ---- accessors ---------------------------------------------------------------------------
@@ -112,7 +112,7 @@ class BlockedKVCache:
         return self._per_block_bytes
 
     def get_cache(self, cache_id: int = 0, cache_group: int = 0) -> torch.Tensor:
-        """Layer ``cache_id``'s pages: ``[blocks, 2, heads, block_size, head_dim]``."""
+        """Layer ``cache_id``'s pages: ``[blocks, planes, heads, block_size, head_dim]`` (planes: K and V unless configured)."""
         return self._cache[cache_id]
 
     @property

@@ -31,8 +31,9 @@ class KVCacheConfig(DeepSpeedConfigModel):
     cache_dtype: DtypeEnum = DtypeEnum.fp16
     max_blocks_per_allocation_group: PositiveInt = 64
     """Upper bound of blocks one sequence may own (= ceil(max_context / block_size))."""
-    layer_shapes: Optional[List[Optional[Tuple[PositiveInt, PositiveInt]]]] = None
-    """(kv_heads, head_dim) of every layer when they differ (None = a layer without attention); ``cache_shape`` otherwise."""
+    layer_shapes: Optional[List[Optional[Tuple[PositiveInt, PositiveInt, PositiveInt]]]] = None
+    """(planes, kv_heads, head_dim) of every layer when they differ; ``cache_shape`` with two planes, K and V, otherwise. One plane:
+    keys and values are read from the same rows. None: a layer with nothing of its own in the pages."""
 
 
 class RecurrentLayerConfig(DeepSpeedConfigModel):

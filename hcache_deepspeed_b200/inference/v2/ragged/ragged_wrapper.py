@@ -13,6 +13,7 @@ from __future__ import annotations
 import ctypes
 from typing import List, Optional, Tuple
 
+import numpy as np
 import torch
 
 from ....ops import native
@@ -87,6 +88,7 @@ class RaggedBatchWrapper:
         self._inflight: List[Tuple[int, int, int]] = []
         self._descs: List[DSSequenceDescriptor] = []
         self._n_single = 0
+        self._visible = {}
         self._n_small = self._n_large = self._rows_small = self._max_kv_small = self._max_kv_large = 0
 
     def insert_sequence(self, seq_descriptor: DSSequenceDescriptor, tokens: torch.Tensor, do_checks: bool = True) -> None:
@@ -180,7 +182,41 @@ class RaggedBatchWrapper:
         """int32 ``[n_seqs, 4]``: (first row in the batch, new tokens, tokens seen before, recurrent-state slot)."""
         return self._view("spans", 4 * self._n_seqs, on_device).view(self._n_seqs, 4)
 
+    def visible_pages(self, window: int, capacity: int) -> Optional[Tuple[torch.Tensor, torch.Tensor]]:
+        """The pages that the sequences with large items (more than ``small_item_tokens`` new tokens) see through a sliding window
+        (0: all of them), from whole 128-token tiles on: (block ids int32 ``[n]``, block tables ``[n_seqs, stride]`` that
+        name them by their place in that list), or None when there are more than ``capacity``."""
+        if window not in self._visible:
+            tables = self.block_tables(on_device=False).numpy()
+            ids, places = [], np.zeros_like(tables)
+            n = 0
+            for s, (_, new, seen) in enumerate(self._inflight):
+                if new <= self.small_item_tokens:
+                    continue
+                first = max(0, seen - window + 1) // LARGE_ITEM_TOKENS * LARGE_ITEM_TOKENS // self._block_size if window else 0
+                last = -(-(seen + new) // self._block_size)
+                ids.append(tables[s, first:last])
+                places[s, first:last] = np.arange(n, n + last - first)
+                n += last - first
+            up = lambda a: torch.from_numpy(a).to(self._device)  # noqa: E731
+            self._visible[window] = (n, up(np.concatenate(ids).copy()), up(places))
+        n, ids, places = self._visible[window]
+        return (ids, places) if n <= capacity else None
+
     # ---- scalars -------------------------------------------------------------------------------------
+    @property
+    def group(self) -> int:
+        return self._group
+
+    @property
+    def small_item_tokens(self) -> int:
+        """New tokens of a sequence up to which it is one small item."""
+        return SMALL_ITEM_ROWS // self._group
+
+    @property
+    def max_large_item_tokens(self) -> int:
+        return max((min(n, LARGE_ITEM_TOKENS) for _, n, _ in self._inflight if n > self.small_item_tokens), default=0)
+
     @property
     def current_tokens(self) -> int:
         return self._n_tokens

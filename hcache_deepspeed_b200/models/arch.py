@@ -66,19 +66,90 @@ class StateSpaceSpec:
 
 
 @dataclass
+class LatentAttentionSpec:
+    """Attention over a shared latent: every token caches one normed vector of ``kv_rank`` values and one rotated key part of
+    ``rot_dim`` values, from which each head projects its own key and value. A head's query has ``dim`` unrotated and
+    ``rot_dim`` rotated values (adjacent pairs, ``rot_base``). ``window`` as in :class:`AttentionSpec`. ``kv_from``: use what
+    that layer caches instead of an own latent (both layers' sizes and rotation agree)."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    window: int = 0
+    rot_base: float = 10000.0
+    kv_from: Optional[int] = None
+
+    @property
+    def page_width(self) -> int:
+        """Values of a cached token: latent | rotated key part, zero padded to whole 128-byte rows of 16-bit values."""
+        return -(-(self.kv_rank + self.rot_dim) // 64) * 64
+
+    @property
+    def head_width(self) -> int:
+        """Head size of q and of the attention output, and of K / V pages projected from the latents (see AttentionSpec.page_dim)."""
+        d = max(self.dim + self.rot_dim, self.vdim)
+        return 64 if d <= 64 else 128 if d <= 128 else -(-d // 8) * 8
+
+
+@dataclass
+class DeltaSpec:
+    """Gated delta rule: heads with a ``dim`` x ``vdim`` recurrent state each, which fades by a decay per head and is corrected
+    along the current key; queries and keys are shared by the value heads of a group (``kv_heads`` groups). A causal
+    convolution of ``conv`` taps in front of q, k and v; a norm per head and a gate behind."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int = 4
+
+    @property
+    def state(self) -> int:
+        return self.dim
+
+    @property
+    def groups(self) -> int:
+        return self.kv_heads
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_dim(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+    @property
+    def in_dim(self) -> int:
+        """Rows of the input projection: gate | v | k | q | decay input | step input."""
+        return self.inner + self.conv_dim + 2 * self.heads
+
+
+@dataclass
 class MixerSpec:
-    """Token mixer of a layer: attention, a state-space mixer, or both side by side on the same input, each with a weight."""
+    """Token mixer of a layer: attention, a state-space mixer, or both side by side on the same input, each with a weight; or
+    latent attention; or a gated delta rule."""
     attn: Optional[AttentionSpec] = None
     ssm: Optional[StateSpaceSpec] = None
     attn_weight: float = 1.0
     ssm_weight: float = 1.0
+    latent: Optional[LatentAttentionSpec] = None
+    delta: Optional[DeltaSpec] = None
+
+    @property
+    def recurrent(self):
+        """The part with per-sequence state, if any."""
+        return self.ssm if self.ssm is not None else self.delta
 
 
 @dataclass
 class FeedForwardSpec:
     """``experts`` = 0: dense gated MLP of size ``ff``. Otherwise a mixture of experts of size ``ff`` each, ``top`` per token.
-    ``routing`` = "table": a table gives every token id its experts, all with weight 1 / top. ``shared_ff`` > 0: one more
-    expert that sees every token. ``act`` = "swiglu_clamped" clamps gate and up to ``limit`` (see ops.reference)."""
+    ``routing`` = "table": a table gives every token id its experts, all with weight 1 / top. ``routing`` = "softmax": the
+    largest softmax scores of a router, each plus the expert's correction, choose; the scores themselves times
+    ``router_scale`` weigh. ``shared_ff`` > 0: one more expert that sees every token. ``gated`` = False: down(act(up x)).
+    ``act`` = "swiglu_clamped" clamps gate and up to ``limit`` (see ops.reference)."""
     ff: int
     act: str = "silu"
     limit: float = 0.0
@@ -86,6 +157,8 @@ class FeedForwardSpec:
     top: int = 0
     routing: str = "table"
     shared_ff: int = 0
+    gated: bool = True
+    router_scale: float = 1.0
 
 
 @dataclass
@@ -140,8 +213,10 @@ class ArchSpec:
     shared_expert_intermediate: int = 0  # Qwen2-MoE shared expert (with sigmoid gate)
     norm_topk_prob: bool = True
     #: one entry per layer for stacks of unlike layers; the scalar sizes above then hold the largest values. Such stacks
-    #: keep the residual stream in fp32 and norm every sublayer's input AND output (models/hybrid.py)
+    #: keep the residual stream in fp32 (models/hybrid.py). With ``parallel_residual`` mixer and feed-forward read one norm
     layers: Optional[List[LayerSpec]] = None
+    post_norms: bool = False  # ``layers`` stacks: every sublayer's OUTPUT is normed as well
+    norm_weight_offset: float = 0.0  # ``layers`` stacks: stored norm weights are differences from this
     extras: Dict[str, Any] = field(default_factory=dict)
 
     # ---- derived -------------------------------------------------------------------------------
@@ -176,7 +251,12 @@ class ArchSpec:
 
     @property
     def has_recurrent_state(self) -> bool:
-        return self.layers is not None and any(l.mixer.ssm is not None for l in self.layers)
+        return self.layers is not None and any(l.mixer.recurrent is not None for l in self.layers)
+
+    @property
+    def pages_hold_context(self) -> bool:
+        """Do the K / V pages of a sequence alone bring every layer's context back?"""
+        return self.layers is None or (not self.has_recurrent_state and all(l.mixer.latent is None for l in self.layers))
 
     def window_of(self, layer: int) -> int:
         return int(self.layer_windows[layer]) if self.layer_windows is not None else int(self.sliding_window)
@@ -189,14 +269,22 @@ class ArchSpec:
         if self.layers is not None:
             total = self.vocab * h * (1 if self.tie_word_embeddings else 2) + h
             for l in self.layers:
-                a, m, f = l.mixer.attn, l.mixer.ssm, l.mlp
-                total += 2 * h
+                a, m, f, c, d = l.mixer.attn, l.mixer.ssm, l.mlp, l.mixer.latent, l.mixer.delta
+                total += h * (1 + self.post_norms)
                 if a is not None:
                     total += h * (a.heads * (a.dim + a.vdim) + a.kv_heads * (a.dim + a.vdim))
                 if m is not None:
                     total += h * (m.in_dim + m.inner) + m.conv_dim * (m.conv + 1) + 3 * m.heads + m.inner
+                if c is not None:
+                    total += c.heads * (h * (c.dim + c.rot_dim + c.vdim) + c.kv_rank * (c.dim + c.vdim))
+                    total += (h * (c.kv_rank + c.rot_dim) + c.kv_rank) if c.kv_from is None else 0
+                if d is not None:
+                    total += h * (d.in_dim + d.inner) + d.conv_dim * d.conv + 2 * d.heads + d.vdim
                 if f is not None:
-                    total += 2 * h + 3 * h * (f.ff * max(1, f.experts) + f.shared_ff) + self.vocab * (f.top if f.experts else 0)
+                    total += 0 if self.parallel_residual else h * (1 + self.post_norms)
+                    total += (3 if f.gated else 2) * h * (f.ff * max(1, f.experts) + f.shared_ff)
+                    if f.experts:
+                        total += self.vocab * f.top if f.routing == "table" else (h + 1) * f.experts
             return total
         attn = h * (self.q_dim + 2 * self.kv_dim) + self.q_dim * h
         if self.is_moe:
@@ -496,19 +584,70 @@ def _nipolorn(cfg) -> ArchSpec:
                 attn_weight=float(mx["left_scale"]), ssm_weight=float(mx["right_scale"])),
             mlp=ff(lc.get("mlp"))))
     return stack_arch("nipolorn", layers, hidden=int(_get(cfg, "width")), vocab=int(_get(cfg, "vocab")),
-                      norm_eps=float(_get(cfg, "norm")["eps"]))
+                      norm_eps=float(_get(cfg, "norm")["eps"]), **NIPOLORN_NORMS)
+
+
+#: norms of Nipolorn: on both sides of every sublayer, weights stored as differences from one
+NIPOLORN_NORMS = dict(post_norms=True, norm_weight_offset=1.0)
+
+
+@register_arch("dedelorn")
+def _dedelorn(cfg) -> ArchSpec:
+    """Dedelorn: layers of a gated delta rule or of latent attention in any order, each beside its feed-forward (dense, or a
+    mixture of experts with a corrected softmax router) on one norm; latent attention layers may share another layer's cache."""
+
+    def ff(m) -> Optional[FeedForwardSpec]:
+        if m is None:
+            return None
+        if m["kind"] == "dense":
+            return FeedForwardSpec(ff=int(m["ff"]), act="gelu_tanh")
+        if m["kind"] != "moe":
+            raise ValueError(f"dedelorn: unknown feed-forward kind {m['kind']!r}")
+        r = m["router"]
+        return FeedForwardSpec(ff=int(m["expert"]["ff"]), act="gelu", experts=int(r["experts"]), top=int(r["top"]), routing="softmax",
+                               router_scale=float(r.get("scale", 1.0)), gated=False)
+
+    layers: List[LayerSpec] = []
+    for i, lc in enumerate(_get(cfg, "layers")):
+        mx = lc["mixer"]
+        if lc["type"] == "delta":
+            mixer = MixerSpec(delta=DeltaSpec(heads=int(mx["heads"]), kv_heads=int(mx["kv_heads"]), dim=int(mx["dim"]), vdim=int(mx["vdim"]),
+                                              conv=int(mx["conv"])))
+        elif lc["type"] == "latent_attention":
+            rot, src = mx["rot"], mx.get("kv_from")
+            a = LatentAttentionSpec(heads=int(mx["heads"]), dim=int(mx["dim"]), rot_dim=int(mx["rot_dim"]), vdim=int(mx["vdim"]),
+                                    kv_rank=int(mx["kv_rank"]), scale=float(mx["scale"]), window=int((mx.get("mask") or {}).get("size", 0)),
+                                    rot_base=float(rot["base"]), kv_from=None if src is None else int(src))
+            if int(rot["dims"]) != a.rot_dim:
+                raise ValueError("dedelorn: rot.dims must equal rot_dim")
+            if src is not None:
+                own = layers[a.kv_from].mixer.latent if 0 <= a.kv_from < i else None
+                if own is None or own.kv_from is not None or (own.kv_rank, own.rot_dim, own.rot_base) != (a.kv_rank, a.rot_dim, a.rot_base):
+                    raise ValueError(f"dedelorn: layer {i} cannot use the latents of layer {src}")
+            mixer = MixerSpec(latent=a)
+        else:
+            raise ValueError(f"dedelorn: unknown layer type {lc['type']!r}")
+        layers.append(LayerSpec(mixer=mixer, mlp=ff(lc.get("mlp"))))
+    return stack_arch("dedelorn", layers, hidden=int(_get(cfg, "width")), vocab=int(_get(cfg, "vocab")),
+                      norm_eps=float(_get(cfg, "norm")["eps"]), **DEDELORN_NORMS)
+
+
+#: Dedelorn: one norm per layer read by both sublayers, and a norm on the embeddings
+DEDELORN_NORMS = dict(parallel_residual=True, embed_norm=True)
 
 
 def stack_arch(model_type: str, layers: List[LayerSpec], hidden: int, vocab: int, norm_eps: float, **kw) -> ArchSpec:
     """ArchSpec of a stack of unlike layers; its scalar sizes are those of the layer with the widest KV pages, or the largest of any."""
     attn = [l.mixer.attn for l in layers if l.mixer.attn is not None]
     mlps = [l.mlp for l in layers if l.mlp is not None]
-    widest = max(attn, key=lambda a: a.kv_heads * a.page_dim, default=AttentionSpec(1, 1, 64, 64, 1.0))
-    return ArchSpec(model_type=model_type, n_layers=len(layers), hidden=hidden, n_heads=widest.heads,
-                    n_kv_heads=widest.kv_heads, head_dim=widest.page_dim,
+    latent = [l.mixer.latent for l in layers if l.mixer.latent is not None]
+    geometry = [(a.kv_heads * a.page_dim, a.heads, a.kv_heads, a.page_dim) for a in attn] + [(c.page_width, 1, 1, c.page_width) for c in latent]
+    _, n_heads, n_kv_heads, head_dim = max(geometry, default=(0, 1, 1, 64))
+    return ArchSpec(model_type=model_type, n_layers=len(layers), hidden=hidden, n_heads=n_heads,
+                    n_kv_heads=n_kv_heads, head_dim=head_dim,
                     intermediate=max((m.ff for m in mlps if not m.experts), default=0), vocab=vocab, norm="rms",
                     norm_eps=norm_eps, act="silu", gated_mlp=True, pos_emb="none",
-                    sliding_window=max((a.window for a in attn), default=0), max_positions=1 << 30,
+                    sliding_window=max((a.window for a in attn + latent), default=0), max_positions=1 << 30,
                     n_experts=max((m.experts for m in mlps), default=0), top_k=max((m.top for m in mlps), default=0),
                     moe_intermediate=max((m.ff for m in mlps if m.experts), default=0),
                     shared_expert_intermediate=max((m.shared_ff for m in mlps), default=0), layers=layers, **kw)
@@ -551,7 +690,7 @@ def _stack_named() -> Dict[str, ArchSpec]:
     def nipolorn(width, heads, kv, window, keep, ssm_heads, groups, mlp):
         mixer = MixerSpec(attn=AttentionSpec(heads, kv, 128, 128, 128 ** -0.5, window, keep),
                           ssm=StateSpaceSpec(ssm_heads, 64, 128, groups, 4, groups), attn_weight=1.0, ssm_weight=0.5)
-        return stack_arch("nipolorn", [LayerSpec(mixer, mlp)] * 4, hidden=width, vocab=32000, norm_eps=1e-5)
+        return stack_arch("nipolorn", [LayerSpec(mixer, mlp)] * 4, hidden=width, vocab=32000, norm_eps=1e-5, **NIPOLORN_NORMS)
 
     def plain(mt, width, heads, kv, window, **kw):
         return ArchSpec(model_type=mt, n_layers=4, hidden=width, n_heads=heads, n_kv_heads=kv, head_dim=128, vocab=32000, norm="rms",

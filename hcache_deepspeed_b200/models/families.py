@@ -470,7 +470,7 @@ def map_gpt_neo(name: str, t: torch.Tensor, spec: ArchSpec) -> List[Piece]:
 
 
 # ---------------------------------------------------------------------------------------------------
-_NIPOLORN_LAYER = re.compile(r"l(\d+)\.(.+)$")
+_STACK_LAYER = re.compile(r"l(\d+)\.(.+)$")
 _NIPOLORN_MIXER = {"left.q": "attn.q", "left.k": "attn.k", "left.v": "attn.v", "left.o": "attn.o", "right.in": "ssm.in",
                    "right.conv": "ssm.conv", "right.conv.b": "ssm.conv_b", "right.dt_bias": "ssm.dt_bias",
                    "right.A_log": "ssm.A_log", "right.D": "ssm.D", "right.norm": "ssm.norm", "right.o": "ssm.o"}
@@ -480,7 +480,7 @@ _NIPOLORN_MIXER = {"left.q": "attn.q", "left.k": "attn.k", "left.v": "attn.v", "
 def map_nipolorn(name: str, t: torch.Tensor, spec: ArchSpec) -> List[Piece]:
     if name in ("embed", "final.norm", "head"):
         return [(None, {"embed": "embed", "final.norm": "final_norm.g", "head": "lm_head"}[name], t)]
-    m = _NIPOLORN_LAYER.match(name)
+    m = _STACK_LAYER.match(name)
     if not m:
         return []
     li, rest = int(m.group(1)), m.group(2)
@@ -495,6 +495,39 @@ def map_nipolorn(name: str, t: torch.Tensor, spec: ArchSpec) -> List[Piece]:
         if leaf == "table" or leaf.startswith("shared."):
             return [(li, "moe." + leaf, t)]
         m = re.match(r"e(\d+)\.(gate|up|down)$", leaf)
+        if m:
+            return [(li, f"moe.experts.{m.group(1)}.{m.group(2)}", t)]
+    return []
+
+
+# ---------------------------------------------------------------------------------------------------
+_DEDELORN_DELTA = {"q": "delta.q", "k": "delta.k", "v": "delta.v", "q.conv": "delta.q_conv", "k.conv": "delta.k_conv", "v.conv": "delta.v_conv",
+                   "b": "delta.b", "a": "delta.a", "A_log": "delta.A_log", "dt_bias": "delta.dt_bias", "norm": "delta.norm", "g": "delta.g",
+                   "o": "delta.o"}
+_DEDELORN_LATENT = {"q": "latent.q", "dkv": "latent.dkv", "dkv.norm": "latent.norm", "uk": "latent.uk", "uv": "latent.uv", "o": "latent.o"}
+
+
+@register_mapper("dedelorn")
+def map_dedelorn(name: str, t: torch.Tensor, spec: ArchSpec) -> List[Piece]:
+    top = {"embed": "embed", "embed.norm": "embed_norm.g", "final.norm": "final_norm.g", "head": "lm_head"}
+    if name in top:
+        return [(None, top[name], t)]
+    m = _STACK_LAYER.match(name)
+    if not m or int(m.group(1)) >= spec.n_layers:
+        return []
+    li, rest = int(m.group(1)), m.group(2)
+    if rest == "norm1":
+        return [(li, "norm1.g", t)]
+    part, _, leaf = rest.partition(".")
+    if part == "mix":
+        table = _DEDELORN_DELTA if spec.layers[li].mixer.delta is not None else _DEDELORN_LATENT
+        return [(li, table[leaf], t)] if leaf in table else []
+    if part == "mlp":
+        if leaf in ("gate", "up", "down"):
+            return [(li, "mlp." + leaf, t)]
+        if leaf in ("router", "correction"):
+            return [(li, "moe." + leaf, t)]
+        m = re.match(r"e(\d+)\.(up|down)$", leaf)
         if m:
             return [(li, f"moe.experts.{m.group(1)}.{m.group(2)}", t)]
     return []

@@ -11,9 +11,17 @@ supplies what such a layer does between them, and how its checkpoint pieces are 
   them. Of their two weights only the ratio is applied there (to the state-space part, in fp32, inside its gated norm); the
   common factor goes into the norm behind the mixer, which reads its input times that factor.
 * rows and columns of width ``hidden`` are zero padded to 16-byte rows.
+* latent attention: ``w_qkv`` is ``[q heads | latent | rotated key part]``, heads padded to the page size of the attention kernels.
+  Short portions and decode steps attend in the latent space (``w_uk`` takes the queries there, ``w_uv`` the results back); prompts
+  project the cached rows they see to per-head K / V pages (``w_kv``, whose identity rows copy the rotated part) and use the
+  ordinary attention kernels on those.
+* a gated delta rule's ``w_qkv`` is ``[gate | v | k | q | decay input | step input]``: the columns of a state-space mixer
+  (``[z | x | B | C | dt]``) and one more per head.
+* ``parallel_residual``: mixer and dense feed-forward read the same norm, so ``w_o`` is ``[mixer columns | feed-forward columns]``
+  and ONE GEMM projects and adds both.
 
-The residual stream is fp32. A sublayer leaves ``(output, factor, weight of the norm behind it)`` pending; the next norm kernel
-applies that norm, adds to the stream, and norms the stream for its own sublayer in the same pass.
+The residual stream is fp32. A sublayer leaves ``(output, factor, weight of the norm behind it, if any)`` pending; the next norm
+kernel applies that norm, adds to the stream, and norms the stream for its own sublayer in the same pass.
 """
 from __future__ import annotations
 
@@ -23,9 +31,10 @@ import torch
 
 from ..inference.v2.ragged import RaggedBatchWrapper, RecurrentLayerConfig
 from ..inference.v2.ragged.manager_configs import KVCacheConfig
-from ..ops.backend import pick_decode_splits, pick_packed_splits, pick_prefill_splits, use_packed_decode, windowed_len
+from ..ops.backend import (LatentBuffers, latent_launches, pick_decode_splits, pick_packed_splits, pick_prefill_splits, use_packed_decode,
+                           windowed_len)
 from ..ops.kernels import ACT_CODES
-from .arch import ArchSpec, AttentionSpec, FeedForwardSpec, LayerSpec, MixerSpec, StateSpaceSpec
+from .arch import ArchSpec, AttentionSpec, DeltaSpec, FeedForwardSpec, LatentAttentionSpec, LayerSpec, MixerSpec, StateSpaceSpec
 from .transformer import RaggedTransformer, ceil_div
 from .weights import ExpertWeights, LayerWeights, ModelWeights, interleave_gate_up
 
@@ -37,20 +46,28 @@ def pad8(n: int) -> int:
 # ---------------------------------------------------------------------------------------------------
 # weights
 # ---------------------------------------------------------------------------------------------------
-def required_pieces(l: LayerSpec) -> List[str]:
-    req = ["norm1.g", "norm1b.g"]
+def required_pieces(spec: ArchSpec, l: LayerSpec) -> List[str]:
+    req = ["norm1.g"] + (["norm1b.g"] if spec.post_norms else [])
+    c = l.mixer.latent
+    if c is not None:
+        req += ["latent." + n for n in ("q", "uk", "uv", "o")] + (["latent.dkv", "latent.norm"] if c.kv_from is None else [])
+    if l.mixer.delta is not None:
+        req += ["delta." + n for n in ("q", "k", "v", "q_conv", "k_conv", "v_conv", "a", "b", "A_log", "dt_bias", "g", "norm", "o")]
     if l.mixer.attn is not None:
         req += ["attn.q", "attn.k", "attn.v", "attn.o"]
     if l.mixer.ssm is not None:
         req += ["ssm." + n for n in ("in", "conv", "conv_b", "dt_bias", "A_log", "D", "norm", "o")]
     if l.mlp is not None:
-        req += ["norm2.g", "norm2b.g"]
+        if not spec.parallel_residual:
+            req += ["norm2.g"] + (["norm2b.g"] if spec.post_norms else [])
+        parts = ("gate", "up", "down") if l.mlp.gated else ("up", "down")
         if l.mlp.experts:
-            req += [f"moe.experts.{e}.{n}" for e in range(l.mlp.experts) for n in ("gate", "up", "down")] + ["moe.table"]
+            req += [f"moe.experts.{e}.{n}" for e in range(l.mlp.experts) for n in parts]
+            req += ["moe.table"] if l.mlp.routing == "table" else ["moe.router", "moe.correction"]
             if l.mlp.shared_ff:
-                req += ["moe.shared.gate", "moe.shared.up", "moe.shared.down"]
+                req += ["moe.shared." + n for n in parts]
         else:
-            req += ["mlp.gate", "mlp.up", "mlp.down"]
+            req += ["mlp." + n for n in parts]
     return req
 
 
@@ -70,6 +87,8 @@ def _head_rows(w: torch.Tensor, heads: int, d: int, page_dim: int) -> torch.Tens
 def mixer_factors(m: MixerSpec) -> Tuple[float, float]:
     """(factor of the whole mixer output, weight of the state-space part inside it). The attention part has weight 1 inside
     (its columns of the output projection are dropped when its weight is 0)."""
+    if m.latent is not None or m.delta is not None:
+        return 1.0, 1.0
     if m.attn is not None and m.attn_weight != 0.0:
         return m.attn_weight, m.ssm_weight / m.attn_weight
     return (m.ssm_weight if m.ssm is not None else 0.0), 1.0
@@ -86,16 +105,43 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
         return t.to(device=device, dtype=torch.float32).contiguous()
 
     def gamma(name: str) -> torch.Tensor:
-        return f32(_pad(1.0 + p[name].float(), 0, Hp))    # norm weights are stored as differences from one
+        return f32(_pad(spec.norm_weight_offset + p[name].float(), 0, Hp))
 
-    def glu(prefix: str, ff: int) -> ExpertWeights:
+    def ff_weights(prefix: str, ff: int, gated: bool) -> ExpertWeights:
         ffp = pad8(ff)
-        up = interleave_gate_up(_pad(p[prefix + "gate"], 0, ffp), _pad(p[prefix + "up"], 0, ffp))
+        up = _pad(p[prefix + "up"], 0, ffp)
+        if gated:
+            up = interleave_gate_up(_pad(p[prefix + "gate"], 0, ffp), up)
         return ExpertWeights(to(_pad(up, 1, Hp)), to(_pad(_pad(p[prefix + "down"], 1, ffp), 0, Hp)))
 
-    lw = LayerWeights(norm1_g=gamma("norm1.g"), norm1b_g=gamma("norm1b.g"))
-    a, m = l.mixer.attn, l.mixer.ssm
+    lw = LayerWeights(norm1_g=gamma("norm1.g"))
+    if spec.post_norms:
+        lw.norm1b_g = gamma("norm1b.g")
+    a, m, c, d = l.mixer.attn, l.mixer.ssm, l.mixer.latent, l.mixer.delta
     rows, cols = [], []
+    if c is not None:
+        D, R = c.head_width, c.kv_rank
+        rows.append(_head_rows(p["latent.q"], c.heads, c.dim + c.rot_dim, D))
+        if c.kv_from is None:
+            rows.append(p["latent.dkv"])
+            lw.latent_norm = f32(p["latent.norm"])
+        cols.append(_pad(p["latent.o"].reshape(spec.hidden, c.heads, c.vdim), 2, D).reshape(spec.hidden, c.heads * D))
+        uk, uv = p["latent.uk"].reshape(c.heads, c.dim, R), p["latent.uv"].reshape(c.heads, c.vdim, R)
+        lw.w_uk, lw.w_uv = to(uk), to(uv.transpose(1, 2))
+        lw.rot_freq = f32(rotation_frequencies(c.rot_dim, c.rot_base))
+        if latent_expands(c, dtype):
+            w_k, w_v = uk.new_zeros(c.heads, D, c.page_width), uk.new_zeros(c.heads, D, c.page_width)
+            w_k[:, :c.dim, :R] = uk
+            w_k[:, c.dim:c.dim + c.rot_dim, R:R + c.rot_dim] = torch.eye(c.rot_dim, dtype=uk.dtype, device=uk.device)
+            w_v[:, :c.vdim, :R] = uv
+            lw.w_kv = to(torch.cat([w_k, w_v]).reshape(2 * c.heads * D, c.page_width))
+    if d is not None:
+        rows += [p["delta." + n] for n in ("g", "v", "k", "q", "a", "b")]
+        cols.append(_pad(p["delta.o"], 1, pad8(d.inner)))
+        lw.ssm_conv_w = f32(torch.cat([p[f"delta.{n}_conv"] for n in "vkq"]).t())
+        lw.ssm_conv_b = torch.zeros(d.conv_dim, dtype=torch.float32, device=device)
+        lw.ssm_dt_bias, lw.ssm_a = f32(p["delta.dt_bias"]), f32(-torch.exp(p["delta.A_log"].float()))
+        lw.ssm_norm = f32(p["delta.norm"].repeat(d.heads))
     if a is not None:
         D = a.page_dim
         # a scale of zero or less cannot be the factor of a running maximum: its sign (or zero) moves into the query rows
@@ -111,27 +157,55 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
         lw.ssm_dt_bias, lw.ssm_a, lw.ssm_d = f32(p["ssm.dt_bias"]), f32(-torch.exp(p["ssm.A_log"].float())), f32(p["ssm.D"])
         lw.ssm_norm = f32(p["ssm.norm"])
     lw.w_qkv = to(_pad(torch.cat(rows, dim=0), 1, Hp))
-    lw.w_o = to(_pad(torch.cat(cols, dim=1), 0, Hp))
     f = l.mlp
     if f is not None:
-        lw.norm2_g, lw.norm2b_g = gamma("norm2.g"), gamma("norm2b.g")
+        if not spec.parallel_residual:
+            lw.norm2_g = gamma("norm2.g")
+            if spec.post_norms:
+                lw.norm2b_g = gamma("norm2b.g")
         if f.experts:
-            lw.experts = [glu(f"moe.experts.{e}.", f.ff) for e in range(f.experts)]
+            lw.experts = [ff_weights(f"moe.experts.{e}.", f.ff, f.gated) for e in range(f.experts)]
             lw.stack_experts()
-            lw.moe_table = p["moe.table"].to(device=device, dtype=torch.int32).contiguous()
+            if f.routing == "table":
+                lw.moe_table = p["moe.table"].to(device=device, dtype=torch.int32).contiguous()
+            else:
+                lw.w_router = to(_pad(_pad(p["moe.router"], 0, pad8(f.experts)), 1, Hp))
+                lw.router_bias = f32(p["moe.correction"])
             if f.shared_ff:
-                lw.shared_expert = glu("moe.shared.", f.shared_ff)
+                lw.shared_expert = ff_weights("moe.shared.", f.shared_ff, f.gated)
         else:
-            dense = glu("mlp.", f.ff)
+            dense = ff_weights("mlp.", f.ff, f.gated)
             lw.w_up, lw.w_down = dense.w_up, dense.w_down
+            if spec.parallel_residual:
+                cols.append(lw.w_down[:spec.hidden].to(cols[0]))
+                lw.w_down = None
+    lw.w_o = to(_pad(torch.cat(cols, dim=1), 0, Hp))
     return lw
+
+
+def rotation_frequencies(dims: int, base: float) -> torch.Tensor:
+    """Angle per position of each rotated pair (computed in fp64)."""
+    return (float(base)**(-torch.arange(0, dims, 2, dtype=torch.float64) / dims)).float()
+
+
+def latent_expands(c: LatentAttentionSpec, dtype: torch.dtype) -> bool:
+    """Can prompts project cached latents to K / V pages of the tensor-core attention kernels?"""
+    return dtype != torch.float32 and c.head_width <= 128
 
 
 def top_weights(spec: ArchSpec, top: Dict[str, torch.Tensor], out: ModelWeights, dtype: torch.dtype,
                 device: torch.device) -> ModelWeights:
     Hp = spec.padded_hidden
     out.embed = _pad(top["embed"], 1, Hp).to(device=device, dtype=dtype).contiguous()
-    out.final_norm_g = _pad(1.0 + top["final_norm.g"].float(), 0, Hp).to(device=device).contiguous()
+
+    def gamma(name: str) -> torch.Tensor:
+        return _pad(spec.norm_weight_offset + top[name].float(), 0, Hp).to(device=device).contiguous()
+
+    out.final_norm_g = gamma("final_norm.g")
+    if spec.embed_norm:
+        if "embed_norm.g" not in top:
+            raise ValueError("checkpoint has no norm of the embeddings but the architecture needs one")
+        out.embed_norm_g = gamma("embed_norm.g")
     out.lm_head = _pad(top["lm_head"], 1, Hp).to(device=device, dtype=dtype).contiguous() if "lm_head" in top else out.embed
     return out
 
@@ -143,8 +217,23 @@ def random_pieces(spec: ArchSpec, l: LayerSpec, gen: torch.Generator, device: to
     def rnd(*shape, scale=std):
         return torch.randn(shape, generator=gen, device=device, dtype=torch.float32) * scale
 
-    p = {"norm1.g": rnd(H, scale=0.05), "norm1b.g": rnd(H, scale=0.05)}
-    a, m, f = l.mixer.attn, l.mixer.ssm, l.mlp
+    def norm_g(n=H):
+        return 1.0 - spec.norm_weight_offset + rnd(n, scale=0.05)
+
+    p = {"norm1.g": norm_g(), "norm1b.g": norm_g()}
+    a, m, f, c, d = l.mixer.attn, l.mixer.ssm, l.mlp, l.mixer.latent, l.mixer.delta
+    if c is not None:
+        p.update({"latent.q": rnd(c.heads * (c.dim + c.rot_dim), H), "latent.uk": rnd(c.heads * c.dim, c.kv_rank),
+                  "latent.uv": rnd(c.heads * c.vdim, c.kv_rank), "latent.o": rnd(H, c.heads * c.vdim)})
+        if c.kv_from is None:
+            p.update({"latent.dkv": rnd(c.kv_rank + c.rot_dim, H), "latent.norm": 1.0 + rnd(c.kv_rank, scale=0.05)})
+    if d is not None:
+        kd = d.kv_heads * d.dim
+        p.update({"delta.q": rnd(kd, H), "delta.k": rnd(kd, H), "delta.v": rnd(d.inner, H), "delta.g": rnd(d.inner, H),
+                  "delta.q_conv": rnd(kd, d.conv, scale=0.3), "delta.k_conv": rnd(kd, d.conv, scale=0.3),
+                  "delta.v_conv": rnd(d.inner, d.conv, scale=0.3), "delta.a": rnd(d.heads, H), "delta.b": rnd(d.heads, H),
+                  "delta.dt_bias": rnd(d.heads, scale=0.5) - 3.0, "delta.A_log": rnd(d.heads, scale=0.5),
+                  "delta.norm": 1.0 + rnd(d.vdim, scale=0.05), "delta.o": rnd(H, d.inner)})
     if a is not None:
         p.update({"attn.q": rnd(a.heads * a.dim, H), "attn.k": rnd(a.kv_heads * a.dim, H), "attn.v": rnd(a.kv_heads * a.vdim, H),
                   "attn.o": rnd(H, a.heads * a.vdim)})
@@ -153,7 +242,7 @@ def random_pieces(spec: ArchSpec, l: LayerSpec, gen: torch.Generator, device: to
                   "ssm.dt_bias": rnd(m.heads, scale=0.5) - 3.0, "ssm.A_log": rnd(m.heads, scale=0.5), "ssm.D": rnd(m.heads, scale=1.0),
                   "ssm.norm": 1.0 + rnd(m.inner, scale=0.05), "ssm.o": rnd(H, m.inner)})
     if f is not None:
-        p.update({"norm2.g": rnd(H, scale=0.05), "norm2b.g": rnd(H, scale=0.05)})
+        p.update({"norm2.g": norm_g(), "norm2b.g": norm_g()})
 
         def glu(prefix, ff):
             p.update({prefix + "gate": rnd(ff, H), prefix + "up": rnd(ff, H), prefix + "down": rnd(H, ff)})
@@ -161,7 +250,10 @@ def random_pieces(spec: ArchSpec, l: LayerSpec, gen: torch.Generator, device: to
         if f.experts:
             for e in range(f.experts):
                 glu(f"moe.experts.{e}.", f.ff)
-            p["moe.table"] = torch.argsort(torch.rand((spec.vocab, f.experts), generator=gen, device=device), dim=1)[:, :f.top].int()
+            if f.routing == "table":
+                p["moe.table"] = torch.argsort(torch.rand((spec.vocab, f.experts), generator=gen, device=device), dim=1)[:, :f.top].int()
+            else:
+                p.update({"moe.router": rnd(f.experts, H), "moe.correction": rnd(f.experts, scale=0.05)})
             if f.shared_ff:
                 glu("moe.shared.", f.shared_ff)
         else:
@@ -173,7 +265,8 @@ def random_stack_weights(spec: ArchSpec, dtype: torch.dtype, device: torch.devic
     gen = torch.Generator(device=device).manual_seed(seed)
     mw = ModelWeights(layers=[layer_weights(spec, l, random_pieces(spec, l, gen, device, std), dtype, device) for l in spec.layers])
     top = {"embed": torch.randn((spec.vocab, spec.hidden), generator=gen, device=device) * std,
-           "final_norm.g": torch.randn(spec.hidden, generator=gen, device=device) * 0.05,
+           "final_norm.g": 1.0 - spec.norm_weight_offset + torch.randn(spec.hidden, generator=gen, device=device) * 0.05,
+           "embed_norm.g": 1.0 - spec.norm_weight_offset + torch.randn(spec.hidden, generator=gen, device=device) * 0.05,
            "lm_head": torch.randn((spec.vocab, spec.hidden), generator=gen, device=device) * std}
     return top_weights(spec, top, mw, dtype, device)
 
@@ -182,10 +275,11 @@ def random_stack_weights(spec: ArchSpec, dtype: torch.dtype, device: torch.devic
 # executor
 # ---------------------------------------------------------------------------------------------------
 class Pending(NamedTuple):
-    """A sublayer's output on its way into the residual stream: stream += norm(factor * delta) * weight."""
+    """A sublayer's output on its way into the residual stream: stream += norm(factor * delta) * weight, or, without a weight,
+    stream += factor * delta."""
     delta: torch.Tensor
     factor: float
-    weight: torch.Tensor
+    weight: Optional[torch.Tensor]
 
 
 class HybridTransformer(RaggedTransformer):
@@ -205,14 +299,21 @@ class HybridTransformer(RaggedTransformer):
 
     def kv_cache_config(self) -> Tuple[KVCacheConfig, ...]:
         base = super().kv_cache_config()[0]
-        shapes = [None if l.mixer.attn is None else (l.mixer.attn.kv_heads, l.mixer.attn.page_dim) for l in self.spec.layers]
-        return (base.model_copy(update={"layer_shapes": shapes}), )
+
+        def shape(m: MixerSpec):
+            if m.attn is not None:
+                return 2, m.attn.kv_heads, m.attn.page_dim
+            if m.latent is not None and m.latent.kv_from is None:
+                return 1, 1, m.latent.page_width
+            return None
+
+        return (base.model_copy(update={"layer_shapes": [shape(l.mixer) for l in self.spec.layers]}), )
 
     def recurrent_state_config(self):
         if not self.spec.has_recurrent_state:
             return None
         return [None if m is None else RecurrentLayerConfig(heads=m.heads, vdim=m.vdim, state=m.state, conv_dim=m.conv_dim, taps=m.conv)
-                for m in (l.mixer.ssm for l in self.spec.layers)]
+                for m in (l.mixer.recurrent for l in self.spec.layers)]
 
     def graphable_decode(self, batch: RaggedBatchWrapper) -> bool:
         return True
@@ -227,6 +328,9 @@ class HybridTransformer(RaggedTransformer):
                 key.append((a, pick(batch.n_items_small, n_kv, windowed_len(batch.max_kv_len_small, window, keep))))
             if batch.n_items_large:
                 key.append((a, pick_prefill_splits(batch.n_items_large, n_q, windowed_len(batch.max_kv_len_large, window, keep))))
+        if self.dtype != torch.float32:
+            for c in {(c.heads, c.kv_rank, c.page_width, c.window) for c in (l.mixer.latent for l in self.spec.layers) if c is not None}:
+                key.append((c, latent_launches(batch, *c, batch.n_items_large > 0)))
         return tuple(key)
 
     def _alloc_buffers(self) -> None:
@@ -239,18 +343,19 @@ class HybridTransformer(RaggedTransformer):
 
         self._tp_fused, self._tp_wait_next, self._tp_scatter_ok = False, False, False
         attn = [l.mixer.attn for l in s.layers if l.mixer.attn is not None]
-        ssm = [l.mixer.ssm for l in s.layers if l.mixer.ssm is not None]
+        latents = [l.mixer.latent for l in s.layers if l.mixer.latent is not None]
+        rec = [l.mixer.recurrent for l in s.layers if l.mixer.recurrent is not None]
         mlps = [l.mlp for l in s.layers if l.mlp is not None]
         moes = [f for f in mlps if f.experts]
         self.residual = buf(T, Hp, dtype=torch.float32)
         self.xn, self.xn2 = buf(T, Hp), buf(T, Hp)
         self.latent_buf = buf(s.n_layers, T, Hp) if self.capture_enabled else None
         self.in_buf = buf(T * max(pad8(lw.w_qkv.shape[0]) for lw in self.w.layers))
-        self.q_buf = buf(T * max((a.heads * a.page_dim for a in attn), default=8))
+        self.q_buf = buf(T * max([a.heads * a.page_dim for a in attn] + [c.heads * c.head_width for c in latents] + [8]))
         self.mix_buf = buf(T * max(lw.w_o.shape[1] for lw in self.w.layers))
-        self.conv_buf = buf(T * max((pad8(m.conv_dim) for m in ssm), default=8))
-        self.dt_buf = buf(T * max((m.heads for m in ssm), default=1), dtype=torch.float32)
-        self.scan_buf = buf(T * max((m.inner for m in ssm), default=1), dtype=torch.float32)
+        self.conv_buf = buf(T * max((pad8(m.conv_dim) for m in rec), default=8))
+        self.dt_buf = buf(T * max((m.heads for m in rec), default=1), dtype=torch.float32)
+        self.scan_buf = buf(T * max((m.inner for m in rec), default=1), dtype=torch.float32)
         self.act_buf = buf(T * max([pad8(f.ff) for f in mlps if not f.experts] + [pad8(f.shared_ff) for f in moes] + [8]))
         self._delta_bufs = [buf(T, Hp, dtype=torch.float32)]
         self._delta_idx = 0
@@ -261,9 +366,16 @@ class HybridTransformer(RaggedTransformer):
         self.logits_full = self.partial16 = self.kv_scratch = None
         self.ws_gemm = self.ws_small = self.ws_large = self.io_stream = None
         self._moe_bufs: Dict[Tuple[int, int, int], dict] = {}
+        self._latent_bufs: Optional[LatentBuffers] = None
+        self._delta_ws: Optional[torch.Tensor] = None
         if dev.type != "cuda":
             return
         k = self.ops.k
+        if latents:
+            self._latent_bufs = LatentBuffers(latents, self._state_config, self.kv_block_size, dt, dev)
+        if dt != torch.float32:
+            n_ws = max((k.delta_workspace_bytes(T, min(S, 64), m.heads, m.kv_heads) for m in rec if isinstance(m, DeltaSpec)), default=0)
+            self._delta_ws = torch.empty(n_ws, dtype=torch.uint8, device=dev) if n_ws else None
         for f in moes:
             key = (f.experts, f.top, f.ff)
             if key not in self._moe_bufs:
@@ -272,6 +384,7 @@ class HybridTransformer(RaggedTransformer):
                     scores=buf(T, f.top, dtype=torch.float32), expert_ids=buf(T, f.top, dtype=torch.int32),
                     offsets=buf(T, f.top, dtype=torch.int32), mapped_slots=buf(T, f.top, dtype=torch.int32),
                     counts=buf(f.experts, dtype=torch.int32), pad_off=buf(f.experts + 1, dtype=torch.int32),
+                    logits=buf(T, pad8(f.experts), dtype=torch.float32),
                     xs=buf(rows, Hp), hs=buf(rows, pad8(f.ff)), ys=buf(rows, Hp))
         if dt != torch.float32:
             n_max = max([self.info.vocab, Hp] + [lw.w_qkv.shape[0] for lw in self.w.layers] +
@@ -281,6 +394,8 @@ class HybridTransformer(RaggedTransformer):
             for a in {(a.heads, a.kv_heads, a.page_dim) for a in attn if a.page_dim <= 128}:
                 b_small, b_large = self._attention_workspace_bytes(S, *a, rows=8)
                 small, large = max(small, b_small), max(large, b_large)
+            for c in {(c.heads, c.heads, c.head_width) for c in latents if latent_expands(c, dt)}:
+                large = max(large, self._attention_workspace_bytes(S, *c, rows=8)[1])
             self.ws_small = torch.zeros(small, dtype=torch.uint8, device=dev)
             self.ws_large = torch.zeros(large, dtype=torch.uint8, device=dev)
         self._alloc_restore_buffers(T, S, Hp)
@@ -290,7 +405,8 @@ class HybridTransformer(RaggedTransformer):
 
     # ---- layer -------------------------------------------------------------------------------------
     def _embed(self, batch: RaggedBatchWrapper) -> torch.Tensor:
-        return self.ops.embed_f32(batch.input_ids(), self.w.embed, self.residual[:batch.current_tokens])
+        return self.ops.embed_f32(batch.input_ids(), self.w.embed, self.residual[:batch.current_tokens], gamma=self.w.embed_norm_g,
+                                  cols=self.spec.hidden, eps=self.spec.norm_eps)
 
     def _norm_into(self, resid: torch.Tensor, gamma: torch.Tensor, out: torch.Tensor, pending: Optional[Pending],
                    keep_resid: bool = True) -> torch.Tensor:
@@ -300,12 +416,34 @@ class HybridTransformer(RaggedTransformer):
 
     def _layer(self, li: int, resid: torch.Tensor, pending: Optional[Pending], xn: torch.Tensor, batch: RaggedBatchWrapper) -> Pending:
         l, lw, ops, T = self.spec.layers[li], self.w.layers[li], self.ops, batch.current_tokens
-        kv = self._state_manager
         self._norm_into(resid, lw.norm1_g, xn, pending)
         self._kv_ready(li)
+        mix = self._view(self.mix_buf, T, lw.w_o.shape[1])
+        if l.mixer.latent is not None:
+            n_mix = self._latent_mixer(li, l.mixer.latent, lw, xn, mix, batch)
+        elif l.mixer.delta is not None:
+            n_mix = self._delta_mixer(li, l.mixer.delta, lw, xn, mix, batch)
+        else:
+            n_mix = self._attention_and_scan(li, l, lw, xn, mix, batch)
+        factor, f = mixer_factors(l.mixer)[0], l.mlp
+        if self.spec.parallel_residual and f is not None:
+            if not f.experts:      # both sublayers' columns meet one output projection
+                ops.gemm(xn, lw.w_up, mix[:, n_mix:], act=ACT_CODES[f.act], gated=f.gated, workspace=self.ws_gemm, limit=f.limit)
+                return Pending(self._row_parallel(mix, lw.w_o, None, T, force_accum=False), factor, None)
+            delta = self._row_parallel(mix, lw.w_o, None, T, force_accum=False)
+            return Pending(self._feed_forward(xn, f, lw, T, batch, base=delta), factor, None)
+        pending = Pending(self._row_parallel(mix, lw.w_o, None, T, force_accum=False), factor, lw.norm1b_g)
+        if f is None:
+            return pending
+        x2 = self._norm_into(resid, lw.norm2_g, self.xn2[:T], pending)
+        return Pending(self._feed_forward(x2, f, lw, T, batch), 1.0, lw.norm2b_g)
+
+    def _attention_and_scan(self, li: int, l: LayerSpec, lw: LayerWeights, xn: torch.Tensor, mix: torch.Tensor,
+                            batch: RaggedBatchWrapper) -> int:
+        """Softmax attention and / or a state-space mixer on the same input, side by side in ``mix``; returns their columns."""
+        ops, T, kv = self.ops, batch.current_tokens, self._state_manager
         a, m = l.mixer.attn, l.mixer.ssm
         proj = self._view(self.in_buf, T, pad8(lw.w_qkv.shape[0]))
-        mix = self._view(self.mix_buf, T, lw.w_o.shape[1])
         n_attn = n_out = 0
         if a is not None:
             D = a.page_dim
@@ -317,38 +455,63 @@ class HybridTransformer(RaggedTransformer):
                           ws_small=self.ws_small, ws_large=self.ws_large, window=a.window, keep_first=a.keep_first)
         else:
             ops.gemm(xn, lw.w_qkv, proj[:, :lw.w_qkv.shape[0]], workspace=self.ws_gemm)
-        factor, ssm_weight = mixer_factors(l.mixer)
-        if m is not None:
-            y = self._scan(li, m, lw, proj[:, n_attn:n_attn + m.in_dim], batch.spans(), batch.n_single_token_seqs)
-            ops.gated_norm(y, proj[:, n_attn:n_attn + m.inner], lw.ssm_norm, mix[:, n_out:n_out + m.inner], m.norm_groups,
-                           self.spec.norm_eps, ssm_weight)
-        pending = Pending(self._row_parallel(mix, lw.w_o, None, T, force_accum=False), factor, lw.norm1b_g)
-        if l.mlp is None:
-            return pending
-        x2 = self._norm_into(resid, lw.norm2_g, self.xn2[:T], pending)
-        return Pending(self._feed_forward(x2, l.mlp, lw, T, batch), 1.0, lw.norm2b_g)
+        if m is None:
+            return n_out
+        y = self._scan(li, m, lw, proj[:, n_attn:n_attn + m.in_dim], batch.spans(), batch.n_single_token_seqs)
+        ops.gated_norm(y, proj[:, n_attn:n_attn + m.inner], lw.ssm_norm, mix[:, n_out:n_out + m.inner], m.norm_groups,
+                       self.spec.norm_eps, mixer_factors(l.mixer)[1])
+        return n_out + pad8(m.inner)
 
-    def _scan(self, li: int, m: StateSpaceSpec, lw: LayerWeights, proj: torch.Tensor, spans: torch.Tensor, n_single: int) -> torch.Tensor:
-        """Convolution and recurrence of the tokens whose projections are ``proj`` = [z | x | B | C | dt]; advances the
-        sequences' state. Returns the recurrence's output (before gate and norm), fp32 ``[tokens, inner]``."""
+    def _latent_mixer(self, li: int, c: LatentAttentionSpec, lw: LayerWeights, xn: torch.Tensor, mix: torch.Tensor,
+                      batch: RaggedBatchWrapper) -> int:
+        ops, T, kv = self.ops, batch.current_tokens, self._state_manager
+        proj = self._view(self.in_buf, T, pad8(lw.w_qkv.shape[0]))
+        n_q = c.heads * c.head_width
+        q = self._view(self.q_buf, T, n_q)
+        cache = kv.get_cache(li if c.kv_from is None else c.kv_from)
+        ops.gemm(xn, lw.w_qkv, proj[:, :lw.w_qkv.shape[0]], workspace=self.ws_gemm)
+        ops.latent_append(proj, q, cache if c.kv_from is None else None, batch.tok_pos(), batch.tok_slot(), c, lw, self.spec.norm_eps)
+        ops.latent_attention(q, mix[:, :n_q], cache, batch, c, lw, self._latent_bufs, ws_large=self.ws_large)
+        return n_q
+
+    def _delta_mixer(self, li: int, d: DeltaSpec, lw: LayerWeights, xn: torch.Tensor, mix: torch.Tensor, batch: RaggedBatchWrapper) -> int:
+        proj = self._view(self.in_buf, batch.current_tokens, pad8(lw.w_qkv.shape[0]))[:, :d.in_dim]
+        self.ops.gemm(xn, lw.w_qkv, proj, workspace=self.ws_gemm)
+        self._scan(li, d, lw, proj, batch.spans(), batch.n_single_token_seqs, mix[:, :d.inner])
+        return pad8(d.inner)
+
+    def _scan(self, li: int, m, lw: LayerWeights, proj: torch.Tensor, spans: torch.Tensor, n_single: int,
+              out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Convolution and recurrence of the tokens whose projections are ``proj`` = [z | x | B | C | dt] (delta rule:
+        [gate | v | k | q | decay | step]); advances the sequences' state. Returns the recurrence's output (before gate and
+        norm), fp32 ``[tokens, inner]``; a delta rule also writes its normed and gated output to ``out`` when given."""
         T, st = proj.shape[0], self._state_manager.recurrent_states
-        return self.ops.state_space(proj, lw, m, st.ssm(li), st.conv(li), spans, n_single, self._view(self.conv_buf, T, pad8(m.conv_dim)),
-                                    self._view(self.dt_buf, T, m.heads), self._view(self.scan_buf, T, m.inner))
+        bufs = (self._view(self.conv_buf, T, pad8(m.conv_dim)), self._view(self.dt_buf, T, m.heads), self._view(self.scan_buf, T, m.inner))
+        if isinstance(m, DeltaSpec):
+            return self.ops.delta_rule(proj, lw, m, st.ssm(li), st.conv(li), spans, n_single, *bufs, out, self.spec.norm_eps, self._delta_ws)
+        return self.ops.state_space(proj, lw, m, st.ssm(li), st.conv(li), spans, n_single, *bufs)
 
-    def _feed_forward(self, x: torch.Tensor, f: FeedForwardSpec, lw: LayerWeights, T: int, batch: RaggedBatchWrapper) -> torch.Tensor:
+    def _feed_forward(self, x: torch.Tensor, f: FeedForwardSpec, lw: LayerWeights, T: int, batch: RaggedBatchWrapper,
+                      base: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``base``: the other sublayer's pending output, which a mixture of experts is added to."""
         ops = self.ops
         act = ACT_CODES[f.act]
 
         def hidden(w: ExpertWeights):
             h = self._view(self.act_buf, T, w.w_down.shape[1])
-            return ops.gemm(x, w.w_up, h, act=act, gated=True, workspace=self.ws_gemm, limit=f.limit)
+            return ops.gemm(x, w.w_up, h, act=act, gated=f.gated, workspace=self.ws_gemm, limit=f.limit)
 
         if not f.experts:
             return self._row_parallel(hidden(ExpertWeights(lw.w_up, lw.w_down)), lw.w_down, None, T, force_accum=False)
-        shared = None
         if lw.shared_expert is not None:
-            shared = ops.gemm(hidden(lw.shared_expert), lw.shared_expert.w_down, self.delta16[:T], workspace=self.ws_gemm)
-        return ops.table_moe(x, batch.input_ids(), lw, f, act, shared, self.delta32[:T], self._moe_bufs.get((f.experts, f.top, f.ff)))
+            assert base is None
+            base = ops.gemm(hidden(lw.shared_expert), lw.shared_expert.w_down, self.delta16[:T], workspace=self.ws_gemm)
+        bufs = self._moe_bufs.get((f.experts, f.top, f.ff))
+        if f.routing == "table":
+            ops.table_route(batch.input_ids(), lw, f, bufs)
+        else:
+            ops.softmax_route(x, lw, f, bufs)
+        return ops.routed_experts(x, batch.input_ids(), lw, f, act, base, self.delta32[:T], bufs)
 
     def _final_hidden(self, resid: torch.Tensor, pending: Optional[Pending], T: int) -> torch.Tensor:
         return self._norm_into(resid, self.w.final_norm_g, self.xn2[:T], pending, keep_resid=False)
@@ -362,9 +525,13 @@ class HybridTransformer(RaggedTransformer):
         """K/V pages as for any layer; the recurrent state by projecting and scanning the saved inputs once more."""
         l, lw, ops, T = self.spec.layers[li], self.w.layers[li], self.ops, latents.shape[0]
         kv = self._state_manager
-        a, m = l.mixer.attn, l.mixer.ssm
+        a, m, c = l.mixer.attn, l.mixer.recurrent, l.mixer.latent
         n_attn = 0
         proj = self._view(self.in_buf, T, pad8(lw.w_qkv.shape[0]))
+        if c is not None and c.kv_from is None:
+            part = proj[:, c.heads * c.head_width:lw.w_qkv.shape[0]]
+            ops.gemm(latents, lw.w_qkv[c.heads * c.head_width:], part, workspace=self.ws_gemm)
+            ops.latent_append(proj, None, kv.get_cache(li), pos, slot, c, lw, self.spec.norm_eps)
         if a is not None:
             n_q = a.heads * a.page_dim
             n_attn = n_q + 2 * a.kv_heads * a.page_dim

@@ -69,6 +69,13 @@ class LayerWeights:
     ssm_a: Optional[torch.Tensor] = None          # -exp(A_log): the decay rate of each head
     ssm_d: Optional[torch.Tensor] = None
     ssm_norm: Optional[torch.Tensor] = None
+    # latent attention
+    latent_norm: Optional[torch.Tensor] = None    # fp32 [kv_rank]
+    rot_freq: Optional[torch.Tensor] = None       # fp32 [rot_dim / 2]
+    w_uk: Optional[torch.Tensor] = None           # [heads, dim, kv_rank]: takes a head's query to the latent space
+    w_uv: Optional[torch.Tensor] = None           # [heads, kv_rank, vdim]: takes a head's mean latent to its value
+    w_kv: Optional[torch.Tensor] = None           # [2 * heads * head_width, page_width]: cached rows -> K / V pages (16-bit models)
+    router_bias: Optional[torch.Tensor] = None    # fp32 [experts]: added to the scores that choose, not to the weights
 
     def stack_experts(self) -> None:
         """Store the experts as consecutive slices of one tensor per matrix, the operands of the grouped GEMM."""
@@ -253,7 +260,7 @@ class WeightAssembler:
         s = self.spec
         if s.layers is not None:
             from .hybrid import required_pieces
-            return required_pieces(s.layers[li])
+            return required_pieces(s, s.layers[li])
         req = ["attn.q", "attn.k", "attn.v", "attn.o", "norm1.g"]
         if s.qkv_bias:
             req += ["attn.q_b", "attn.k_b", "attn.v_b"]

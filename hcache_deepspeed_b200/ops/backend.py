@@ -96,8 +96,9 @@ class CpuOps:
                                     window=window, keep_first=keep_first)
 
     # ---- stacks of unlike layers ----------------------------------------------------------------------
-    def embed_f32(self, ids, weight, out):
-        out.copy_(ref.embed(ids, weight))
+    def embed_f32(self, ids, weight, out, gamma=None, cols=None, eps=1e-5):
+        x = ref.embed(ids, weight).float()
+        out.copy_(x if gamma is None else x * torch.rsqrt((x * x).sum(-1, keepdim=True) / cols + eps) * gamma)
         return out
 
     def norm_residual(self, resid, gamma, out, delta=None, factor=1.0, post=None, cols=None, eps=1e-5, store_resid=True):
@@ -128,20 +129,71 @@ class CpuOps:
             out[row0:row0 + n] = y.reshape(n, m.inner)
         return out
 
+    def delta_rule(self, proj, lw, m, state, conv_state, spans, n_single, conv_buf, dt_buf, y, out, eps, workspace):
+        C, GN = m.conv_dim, m.groups * m.state
+        for row0, n, seen, slot in spans.tolist():
+            u = proj[row0:row0 + n]
+            if seen == 0:
+                state[slot].zero_()
+            vkq = ref.short_conv(u[:, m.inner:m.inner + C], conv_state[slot], lw.ssm_conv_w, lw.ssm_conv_b, seen).to(proj.dtype).float()
+            decay, beta = u[:, m.inner + C:m.inner + C + m.heads].float(), u[:, m.inner + C + m.heads:m.in_dim].float()
+            decay = torch.exp(lw.ssm_a * torch.nn.functional.softplus(decay + lw.ssm_dt_bias))
+            v, k, q = vkq.split([m.inner, GN, GN], 1)
+            o = ref.delta_scan(q.reshape(n, m.groups, m.state), k.reshape(n, m.groups, m.state), v.reshape(n, m.heads, m.vdim), decay,
+                               torch.sigmoid(beta), state[slot])
+            y[row0:row0 + n] = o.reshape(n, m.inner)
+        if out is not None:
+            out.copy_(ref.gated_norm(y, proj[:, :m.inner], lw.ssm_norm, m.heads, eps, gate_after=True))
+        return y
+
+    def latent_append(self, proj, q_out, pages, tok_pos, tok_slot, c, lw, eps):
+        n_q = c.heads * c.head_width
+        if q_out is not None:
+            q = proj[:, :n_q].reshape(-1, c.heads, c.head_width).clone()
+            q[..., c.dim:c.dim + c.rot_dim] = ref.rotate_pairs(q[..., c.dim:c.dim + c.rot_dim], tok_pos, lw.rot_freq).to(q.dtype)
+            q_out.copy_(q.reshape(q_out.shape))
+        if pages is not None:
+            rows = ref.latent_rows(proj[:, n_q:n_q + c.kv_rank + c.rot_dim], tok_pos, c.kv_rank, lw.rot_freq, lw.latent_norm, eps, c.page_width)
+            pages[:, 0, 0].view(-1, c.page_width)[tok_slot.long()] = rows.to(pages.dtype)
+
+    def latent_attention(self, q, out, pages, batch, c, lw, bufs, ws_large=None):
+        q3 = q.view(-1, c.heads, c.head_width)
+        lat = torch.cat([torch.einsum("thd,hdr->thr", q3[..., :c.dim].float(), lw.w_uk.float()), q3[..., c.dim:c.dim + c.rot_dim].float()], 2)
+        mean = torch.zeros(q3.shape[0], c.heads, c.kv_rank)
+        for items in (batch.items_small(), batch.items_large()):
+            if items.shape[0]:
+                ref.paged_latent_attention(lat, pages, batch.block_tables(), items, c.kv_rank, c.scale, c.window, out=mean)
+        v = torch.einsum("thr,hrv->thv", mean, lw.w_uv.float())
+        out.copy_(torch.nn.functional.pad(v, (0, c.head_width - c.vdim)).reshape(out.shape))
+
     def gated_norm(self, y, z, weight, out, groups, eps, scale=1.0):
         out.copy_(ref.gated_norm(y, z, weight, groups, eps, scale))
         return out
 
-    def table_moe(self, x, ids, lw, f, act, shared, out, bufs):
-        picked = lw.moe_table[ids.long()].long()
-        acc = torch.zeros_like(out) if shared is None else shared.float()
+    def table_route(self, ids, lw, f, bufs):
+        self._picked = lw.moe_table[ids.long()].long()
+        self._scores = torch.full(self._picked.shape, 1.0 / f.top)
+
+    def softmax_route(self, x, lw, f, bufs):
+        s = torch.softmax(ref.gemm(x, lw.w_router, out_dtype=torch.float32)[:, :f.experts], -1)
+        self._picked = torch.topk(s + lw.router_bias, f.top, -1).indices
+        self._scores = s.gather(-1, self._picked) * f.router_scale
+
+    def routed_experts(self, x, ids, lw, f, act, base, out, bufs):
+        """``out`` = ``base`` (None, or ``out`` itself) + the chosen experts' weighted outputs."""
+        picked = self._picked
+        acc = torch.zeros_like(out) if base is None else base.float().clone()
         for e, ew in enumerate(lw.experts):
-            rows = (picked == e).any(-1).nonzero(as_tuple=False).flatten()
+            rows, place = (picked == e).nonzero(as_tuple=True)
             if rows.numel():
-                h = ref.gemm(x.index_select(0, rows), ew.w_up, act=act, gated=True, limit=f.limit)
-                acc.index_add_(0, rows, ref.gemm(h, ew.w_down).float() / f.top)
+                h = ref.gemm(x.index_select(0, rows), ew.w_up, act=act, gated=f.gated, limit=f.limit)
+                acc.index_add_(0, rows, ref.gemm(h, ew.w_down).float() * self._scores[rows, place][:, None])
         out.copy_(acc)
         return out
+
+    def table_moe(self, x, ids, lw, f, act, shared, out, bufs):
+        self.table_route(ids, lw, f, bufs)
+        return self.routed_experts(x, ids, lw, f, act, shared, out, bufs)
 
     # ---- misc ---------------------------------------------------------------------------------------
     def embed(self, ids, weight, out, pos_weight=None, tok_pos=None, pos_offset=0):
@@ -302,8 +354,8 @@ class CudaOps:
                                       scale, n_splits=splits, workspace=ws_large if splits > 1 else None, **opts)
 
     # ---- stacks of unlike layers ----------------------------------------------------------------------
-    def embed_f32(self, ids, weight, out):
-        return self.k.embed_f32(ids, weight, out)
+    def embed_f32(self, ids, weight, out, gamma=None, cols=None, eps=1e-5):
+        return self.k.embed_f32(ids, weight, out, gamma=gamma, cols=cols, eps=eps)
 
     def norm_residual(self, resid, gamma, out, **kw):
         return self.k.norm_residual(resid, gamma, out, **kw)
@@ -331,17 +383,75 @@ class CudaOps:
     def gated_norm(self, y, z, weight, out, groups, eps, scale=1.0):
         return self.k.gated_norm(y, z, weight, out, groups, eps, scale)
 
-    def table_moe(self, x, ids, lw, f, act, shared, out, bufs):
-        """Experts by token id: route -> scatter -> grouped GEMM (gated) -> grouped GEMM -> combine with the shared expert."""
+    def table_route(self, ids, lw, f, bufs):
+        """Experts by token id."""
+        T = ids.numel()
+        self.k.moe_table_route(ids, lw.moe_table, f.experts, bufs["scores"][:T], bufs["expert_ids"][:T], bufs["offsets"][:T], bufs["counts"])
+
+    def softmax_route(self, x, lw, f, bufs):
+        """Experts by router: fp32 scores (the product accumulates in fp32 and is never rounded), corrected choice."""
+        k, T = self.k, x.shape[0]
+        logits = bufs["logits"][:T]             # zero between calls: the gating kernel clears what it has read
+        k.gemm_accum(x, lw.w_router, logits)
+        k.moe_topk_gating(logits[:, :f.experts], f.top, False, bufs["scores"][:T], bufs["expert_ids"][:T], bufs["offsets"][:T], bufs["counts"],
+                          bias=lw.router_bias, scale=f.router_scale, clear=True)
+
+    def routed_experts(self, x, ids, lw, f, act, base, out, bufs):
+        """Routed tokens: scatter -> grouped GEMM -> grouped GEMM -> weighted sum, added to ``base`` (``out`` itself: in place)."""
         k, T, E = self.k, x.shape[0], f.experts
         rows = k.moe_padded_rows(T, E, f.top)
         xs, hs, ys = bufs["xs"][:rows], bufs["hs"][:rows], bufs["ys"][:rows]
         ids_e, off, slots = bufs["expert_ids"][:T], bufs["offsets"][:T], bufs["mapped_slots"][:T]
-        k.moe_table_route(ids, lw.moe_table, E, bufs["scores"][:T], ids_e, off, bufs["counts"])
         k.moe_scatter(x, xs, ids_e, off, bufs["counts"], bufs["pad_off"], slots, f.top)
-        k.moe_gemm(xs, lw.moe_up, bufs["pad_off"], E, hs, act=act, gated=True, limit=f.limit)
+        k.moe_gemm(xs, lw.moe_up, bufs["pad_off"], E, hs, act=act, gated=f.gated, limit=f.limit)
         k.moe_gemm(hs, lw.moe_down, bufs["pad_off"], E, ys)
-        return k.moe_combine(ys, slots, bufs["scores"][:T], shared, out)
+        return k.moe_combine(ys, slots, bufs["scores"][:T], base, out)
+
+    def table_moe(self, x, ids, lw, f, act, shared, out, bufs):
+        self.table_route(ids, lw, f, bufs)
+        return self.routed_experts(x, ids, lw, f, act, shared, out, bufs)
+
+    # ---- latent attention -----------------------------------------------------------------------------
+    def latent_append(self, proj, q_out, pages, tok_pos, tok_slot, c, lw, eps):
+        self.k.latent_append(proj, q_out, pages, tok_pos, tok_slot, c.heads, c.dim, c.rot_dim, c.head_width, c.kv_rank, lw.rot_freq,
+                             lw.latent_norm, eps)
+
+    def latent_attention(self, q, out, pages, batch, c, lw, bufs, ws_large=None):
+        """Decode steps and short portions in the latent space; prompts on K / V pages projected from the cached rows they see (as
+        long as those fit the scratch pages)."""
+        k, T, bs, D = self.k, q.shape[0], batch.block_size, c.head_width
+        plan = None
+        if lw.w_kv is not None and batch.n_items_large and T > batch.current_sequences:
+            plan = batch.visible_pages(c.window, bufs.blocks)
+        generic = q.dtype == torch.float32 or not k.latent_attention_supported(c.kv_rank, c.page_width)
+        limit = batch.small_item_tokens if plan is not None else 1 << 30     # sequences with more new tokens take the other path
+        if generic or batch.n_items_small or plan is None:
+            lat, mean = bufs.queries(T, c), bufs.means(T, c)
+            k.head_matmul(q, lw.w_uk, lat, batch.tokens_to_seq(), batch.spans(), limit, in_width=D, out_width=c.page_width, copy=c.rot_dim)
+            if generic:
+                k.paged_attention_generic(lat, mean, pages, batch.block_tables(), batch.tokens_to_seq(), batch.tok_pos(), c.heads, 1,
+                                          c.page_width, bs, c.scale, window=c.window, value_dim=c.kv_rank, spans=batch.spans(), limit=limit)
+            else:
+                for items, n, tokens, splits in latent_launches(batch, c.heads, c.kv_rank, c.page_width, c.window, plan is None):
+                    k.paged_attention_latent(lat, mean, pages, batch.block_tables(), batch.items_small() if items == "small" else
+                                             batch.items_large(), n, tokens, c.heads, c.kv_rank, bs, splits, c.scale, bufs.workspace, c.window)
+            k.head_matmul(mean, lw.w_uv, out, batch.tokens_to_seq(), batch.spans(), limit, in_width=c.kv_rank, out_width=D, copy=0)
+        if plan is not None:
+            ids, tables = plan
+            n = ids.numel()
+            k.kv_blocks_copy(pages[None], bufs.rows[:n], ids, to_staging=True)
+            kv = bufs.kv_pages(n, c)
+            k.restore_kv_proj(bufs.rows.view(-1)[:n * bs * c.page_width].view(n * bs, c.page_width), lw.w_kv, kv, bufs.slots[:n * bs],
+                              bufs.slots[:n * bs], None, c.heads, D, bs)
+            n_items = batch.n_items_large
+            splits = pick_prefill_splits(n_items, c.heads, windowed_len(batch.max_kv_len_large, c.window))
+            k.paged_attention_prefill(q, out, kv, tables, batch.items_large(), n_items, c.heads, c.heads, D, bs, c.scale, n_splits=splits,
+                                      workspace=ws_large if splits > 1 else None, window=c.window)
+
+    # ---- gated delta rule -----------------------------------------------------------------------------
+    def delta_rule(self, proj, lw, m, state, conv_state, spans, n_single, conv_buf, dt_buf, y, out, eps, workspace):
+        return self.k.delta_rule(proj, lw.ssm_conv_w, lw.ssm_conv_b, lw.ssm_dt_bias, lw.ssm_a, state, conv_state, spans, n_single, m.groups,
+                                 conv_buf, dt_buf, y, out, lw.ssm_norm, eps, workspace)
 
     def embed(self, ids, weight, out, pos_weight=None, tok_pos=None, pos_offset=0):
         return self.k.embed(ids, weight, out, pos_weight=pos_weight, tok_pos=tok_pos, pos_offset=pos_offset)
@@ -411,6 +521,64 @@ def pick_prefill_splits(n_items: int, n_q_heads: int, max_kv_len: int) -> int:
     want = (N_SM + ctas - 1) // ctas
     tiles = max(1, (max_kv_len + 127) // 128)
     return int(max(1, min(want, MAX_PREFILL_SPLITS, tiles // 2 if tiles >= 2 else 1)))
+
+
+def latent_launches(batch, heads: int, rank: int, width: int, window: int, with_large: bool):
+    """Launches of the latent attention kernel for a batch: (item list, items, tokens per item at most, KV splits)."""
+    out = []
+    if batch.n_items_small:
+        out.append(("small", batch.n_items_small, batch.rows_per_small_item // batch.group, batch.max_kv_len_small))
+    if with_large and batch.n_items_large:
+        out.append(("large", batch.n_items_large, batch.max_large_item_tokens, batch.max_kv_len_large))
+    launches = []
+    for kind, n, tokens, kv_len in out:
+        ctas = n * -(-tokens * heads // 128) * -(-rank // 256)
+        tiles = max(1, -(-windowed_len(kv_len, window) // 64))
+        launches.append((kind, n, tokens, int(max(1, min(MAX_PREFILL_SPLITS, N_SM // ctas, tiles // 2)))))
+    return tuple(launches)
+
+
+class LatentBuffers:
+    """Scratch of latent attention, shared by all layers: queries and results in the latent space, and the pages that prompts
+    project their context to. ``blocks``: pages that scratch holds (a batch that sees more attends in the latent space)."""
+
+    def __init__(self, layers, state_config, block_size: int, dtype: torch.dtype, device: torch.device) -> None:
+        T, S, W = state_config.max_ragged_batch_size, state_config.max_ragged_sequence_count, max(c.page_width for c in layers)
+        self._dtype, self._device, self._bs = dtype, device, block_size
+        self._flat = {}
+        expanding = [c for c in layers if c.head_width <= 128] if dtype != torch.float32 else []
+        self.blocks = 0
+        if expanding:
+            seen = max(min(c.window or state_config.max_context, state_config.max_context) for c in expanding)
+            per_block = max(2 * c.heads * c.head_width for c in expanding) * block_size * 2
+            want = -(-T // block_size) + min(S, 8) * (-(-seen // block_size) + 3)
+            self.blocks = max(1, min(want, (2 << 30) // per_block))
+            self.rows = torch.zeros(self.blocks, 1, 1, 1, block_size, W, dtype=dtype, device=device)
+            self._kv = torch.zeros(self.blocks * per_block // 2, dtype=dtype, device=device)
+            self.slots = torch.arange(self.blocks * block_size, dtype=torch.int32, device=device)
+        self.workspace = None
+        if dtype != torch.float32:
+            from . import kernels
+            self.workspace = torch.zeros(kernels.latent_attention_workspace_bytes(), dtype=torch.uint8, device=device)
+        for c in layers:       # decode steps find their buffers in place (a graph cannot allocate them)
+            self.queries(min(T, 8 * S), c)
+            self.means(min(T, 8 * S), c)
+
+    def _get(self, name: str, n: int) -> torch.Tensor:
+        t = self._flat.get(name)
+        if t is None or t.numel() < n:
+            t = self._flat[name] = torch.zeros(n, dtype=self._dtype, device=self._device)
+        return t[:n]
+
+    def queries(self, T: int, c) -> torch.Tensor:
+        return self._get("queries", T * c.heads * c.page_width).view(T, c.heads * c.page_width)
+
+    def means(self, T: int, c) -> torch.Tensor:
+        return self._get("means", T * c.heads * c.kv_rank).view(T, c.heads * c.kv_rank)
+
+    def kv_pages(self, n: int, c) -> torch.Tensor:
+        size = 2 * c.heads * self._bs * c.head_width
+        return self._kv[:n * size].view(n, 2, c.heads, self._bs, c.head_width)
 
 
 def get_ops(device: torch.device):

@@ -1,7 +1,8 @@
 // Mixture-of-experts routing kernels for the ragged forward (tensor-parallel experts, no expert parallelism):
 //
-//   top-k gating  : softmax over the expert logits of each token, k rounds of arg-max (ties -> lower index), optional
-//                   renormalisation of the k scores, one atomic per (token, choice) to claim a row inside the expert
+//   top-k gating  : softmax over the expert logits of each token, k rounds of arg-max (ties -> lower index), optionally of the
+//                   scores plus a per-expert bias; optional renormalisation of the k scores, a factor on them, one atomic per
+//                   (token, choice) to claim a row inside the expert
 //   offsets       : per-expert row ranges padded to the GEMM's 128-row tile (so no A tile straddles two experts);
 //                   re-zeroes the counters for the next layer
 //   scatter       : copies each token's activation row to its k expert rows, records the row index per choice
@@ -17,15 +18,16 @@
 namespace hds {
 
 constexpr int kGateThreads = 128;
-constexpr int kMoeMaxK = 8;
+constexpr int kMoeMaxK = 64;
 constexpr int kMoeRowPad = 128;
 
 template <int DT>
 __global__ void __launch_bounds__(kGateThreads)
-moe_topk_gating_kernel(const void* __restrict__ logits, int64_t ld, int E, int k, int normalize,
-                       float* __restrict__ scores, int32_t* __restrict__ expert_ids, int32_t* __restrict__ offsets,
+moe_topk_gating_kernel(void* __restrict__ logits, int64_t ld, int E, int k, int normalize, const float* __restrict__ bias,
+                       float scale, int clear, float* __restrict__ scores, int32_t* __restrict__ expert_ids, int32_t* __restrict__ offsets,
                        int32_t* __restrict__ counts) {
-    extern __shared__ float probs[];  // [E]
+    extern __shared__ float probs[];  // [E] scores, [E] what chooses
+    float* choice = probs + E;
     __shared__ float red_v[kGateThreads / 32];
     __shared__ int red_i[kGateThreads / 32];
     __shared__ float sel_v[kMoeMaxK];
@@ -37,6 +39,7 @@ moe_topk_gating_kernel(const void* __restrict__ logits, int64_t ld, int E, int k
         const float v = load_any<DT>(logits, static_cast<int64_t>(t) * ld + e);
         probs[e] = v;
         mx = fmaxf(mx, v);
+        if (DT == 2 && clear) reinterpret_cast<float*>(logits)[static_cast<int64_t>(t) * ld + e] = 0.0f;
     }
     mx = warp_max(mx);
     if (lane == 0) red_v[warp] = mx;
@@ -47,7 +50,7 @@ moe_topk_gating_kernel(const void* __restrict__ logits, int64_t ld, int E, int k
     __syncthreads();
     float sum = 0.0f;
     for (int e = tid; e < E; e += kGateThreads) {
-        const float p = __expf(probs[e] - mx);
+        const float p = expf(probs[e] - mx);
         probs[e] = p;
         sum += p;
     }
@@ -58,12 +61,13 @@ moe_topk_gating_kernel(const void* __restrict__ logits, int64_t ld, int E, int k
 #pragma unroll
     for (int w = 0; w < kGateThreads / 32; ++w) sum += red_v[w];
     const float inv = 1.0f / sum;
+    for (int e = tid; e < E; e += kGateThreads) choice[e] = bias == nullptr ? probs[e] : fmaf(probs[e], inv, bias[e]);
     __syncthreads();
     for (int j = 0; j < k; ++j) {
-        float bv = -1.0f;
+        float bv = -INFINITY;
         int bi = 0x7fffffff;
         for (int e = tid; e < E; e += kGateThreads) {
-            const float p = probs[e];
+            const float p = choice[e];
             if (p > bv || (p == bv && e < bi)) {
                 bv = p;
                 bi = e;
@@ -90,9 +94,9 @@ moe_topk_gating_kernel(const void* __restrict__ logits, int64_t ld, int E, int k
                     bi = red_i[w];
                 }
             }
-            sel_v[j] = bv * inv;
+            sel_v[j] = probs[bi] * inv;
             sel_i[j] = bi;
-            probs[bi] = -1.0f;  // taken
+            choice[bi] = -INFINITY;  // taken
         }
         __syncthreads();
     }
@@ -104,7 +108,7 @@ moe_topk_gating_kernel(const void* __restrict__ logits, int64_t ld, int E, int k
             s /= tot;
         }
         const int e = sel_i[tid];
-        scores[static_cast<int64_t>(t) * k + tid] = s;
+        scores[static_cast<int64_t>(t) * k + tid] = s * scale;
         expert_ids[static_cast<int64_t>(t) * k + tid] = e;
         offsets[static_cast<int64_t>(t) * k + tid] = atomicAdd(&counts[e], 1);
     }
@@ -125,11 +129,12 @@ __global__ void moe_table_route_kernel(const int32_t* __restrict__ ids, const in
     offsets[c] = atomicAdd(&counts[e], 1);
 }
 
-// out[t] = base[t] + sum_j score[t, j] * y[row(t, j)]: stores (no read of out), base optional. DT: type of y and base.
+// out[t] = base[t] + sum_j score[t, j] * y[row(t, j)]: stores, base optional; `accumulate`: out itself is the base. DT: type of y
+// and base.
 template <int DT>
 __global__ void moe_combine_kernel(const void* __restrict__ y, int64_t ldy, const int32_t* __restrict__ mapped_slots,
                                    const float* __restrict__ scores, const void* __restrict__ base, int64_t ldb,
-                                   float* __restrict__ out, int64_t ldo, int H, int k) {
+                                   float* __restrict__ out, int64_t ldo, int H, int k, int accumulate) {
     pdl_enter();
     const int64_t t = blockIdx.x;
     auto add8 = [](const void* p, int64_t idx, float s, float (&v)[8]) {
@@ -151,6 +156,11 @@ __global__ void moe_combine_kernel(const void* __restrict__ y, int64_t ldy, cons
         if (base != nullptr) add8(base, t * ldb + c, 1.0f, v);
         for (int j = 0; j < k; ++j) add8(y, static_cast<int64_t>(mapped_slots[t * k + j]) * ldy + c, scores[t * k + j], v);
         float4* o = reinterpret_cast<float4*>(out + t * ldo + c);
+        if (accumulate) {
+            const float4 p = o[0], q = o[1];
+            v[0] += p.x; v[1] += p.y; v[2] += p.z; v[3] += p.w;
+            v[4] += q.x; v[5] += q.y; v[6] += q.z; v[7] += q.w;
+        }
         o[0] = make_float4(v[0], v[1], v[2], v[3]);
         o[1] = make_float4(v[4], v[5], v[6], v[7]);
     }
@@ -212,25 +222,26 @@ __global__ void moe_gather_kernel(const void* __restrict__ y, int64_t ldy, const
 
 using namespace hds;
 
-extern "C" int hds_moe_topk_gating(const void* logits, int64_t ld_logits, int T, int E, int k, int normalize,
-                                   int logits_dtype, float* scores, int32_t* expert_ids, int32_t* offsets,
+extern "C" int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E, int k, int normalize, const float* bias, float scale,
+                                   int clear, int logits_dtype, float* scores, int32_t* expert_ids, int32_t* offsets,
                                    int32_t* counts, void* stream) {
     HDS_REQUIRE(E >= 1 && E <= 4096, "hds_moe_topk_gating: 1..4096 experts");
-    HDS_REQUIRE(k >= 1 && k <= kMoeMaxK && k <= E, "hds_moe_topk_gating: top_k must be in 1..8 and <= experts");
+    HDS_REQUIRE(k >= 1 && k <= kMoeMaxK && k <= E, "hds_moe_topk_gating: top_k must be in 1..64 and <= experts");
     HDS_REQUIRE(logits_dtype >= 0 && logits_dtype <= 2, "hds_moe_topk_gating: logits dtype 0 bf16 / 1 fp16 / 2 fp32");
+    HDS_REQUIRE(!clear || logits_dtype == 2, "hds_moe_topk_gating: only fp32 logits are cleared");
     if (T == 0) return HDS_OK;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    const size_t smem = static_cast<size_t>(E) * sizeof(float);
+    const size_t smem = 2 * static_cast<size_t>(E) * sizeof(float);
     cudaError_t rc;
     if (logits_dtype == 0)
         rc = launch_kernel(moe_topk_gating_kernel<0>, dim3(T), dim3(kGateThreads), smem, s, logits, ld_logits, E, k,
-                           normalize, scores, expert_ids, offsets, counts);
+                           normalize, bias, scale, clear, scores, expert_ids, offsets, counts);
     else if (logits_dtype == 1)
         rc = launch_kernel(moe_topk_gating_kernel<1>, dim3(T), dim3(kGateThreads), smem, s, logits, ld_logits, E, k,
-                           normalize, scores, expert_ids, offsets, counts);
+                           normalize, bias, scale, clear, scores, expert_ids, offsets, counts);
     else
         rc = launch_kernel(moe_topk_gating_kernel<2>, dim3(T), dim3(kGateThreads), smem, s, logits, ld_logits, E, k,
-                           normalize, scores, expert_ids, offsets, counts);
+                           normalize, bias, scale, clear, scores, expert_ids, offsets, counts);
     HDS_CHECK_CUDA(rc);
     return HDS_OK;
 }
@@ -276,17 +287,17 @@ extern "C" int hds_moe_table_route(const int32_t* ids, const int32_t* table, int
 }
 
 extern "C" int hds_moe_combine(const void* y, int64_t ldy, const int32_t* mapped_slots, const float* scores, const void* base,
-                               int64_t ldb, float* out, int64_t ldo, int T, int k, int H, int dtype, void* stream) {
+                               int64_t ldb, float* out, int64_t ldo, int T, int k, int H, int accumulate, int dtype, void* stream) {
     HDS_REQUIRE(H % 8 == 0 && ldy % 8 == 0 && ldo % 4 == 0 && (base == nullptr || ldb % 8 == 0), "hds_moe_combine: rows of 8-value vectors");
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_moe_combine: dtype 0 bf16 / 1 fp16 / 2 fp32");
     if (T == 0) return HDS_OK;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     const dim3 block(H / 8 >= 512 ? 512 : H / 8 >= 256 ? 256 : 128);
     if (dtype == 0)
-        HDS_CHECK_CUDA(launch_kernel(moe_combine_kernel<0>, dim3(T), block, 0, s, y, ldy, mapped_slots, scores, base, ldb, out, ldo, H, k));
+        HDS_CHECK_CUDA(launch_kernel(moe_combine_kernel<0>, dim3(T), block, 0, s, y, ldy, mapped_slots, scores, base, ldb, out, ldo, H, k, accumulate));
     else if (dtype == 1)
-        HDS_CHECK_CUDA(launch_kernel(moe_combine_kernel<1>, dim3(T), block, 0, s, y, ldy, mapped_slots, scores, base, ldb, out, ldo, H, k));
+        HDS_CHECK_CUDA(launch_kernel(moe_combine_kernel<1>, dim3(T), block, 0, s, y, ldy, mapped_slots, scores, base, ldb, out, ldo, H, k, accumulate));
     else
-        HDS_CHECK_CUDA(launch_kernel(moe_combine_kernel<2>, dim3(T), block, 0, s, y, ldy, mapped_slots, scores, base, ldb, out, ldo, H, k));
+        HDS_CHECK_CUDA(launch_kernel(moe_combine_kernel<2>, dim3(T), block, 0, s, y, ldy, mapped_slots, scores, base, ldb, out, ldo, H, k, accumulate));
     return HDS_OK;
 }

@@ -1,12 +1,13 @@
-// Norms of stacks that keep the residual stream in fp32 and norm every sublayer's input AND output.
+// Norms of stacks that keep the residual stream in fp32.
 //
 //   norm_residual : one pass per sublayer boundary. The previous sublayer's output d (16-bit, or the fp32 partial sums of a
 //                   split-K GEMM, cleared while being read) is itself RMS-normed and weighted, added to the fp32 stream, and
 //                   the stream is RMS-normed for the next sublayer:
 //                       x += f d / rms(f d) * post;   out = x / rms(x) * gamma
-//                   One CTA per row; the row stays in registers between the two reductions.
-//   gated_norm    : out = rms(y * silu(z)) * weight * scale over `groups` equal parts of a row (state-space mixers)
-//   embed_f32     : embedding rows into the fp32 stream
+//                   (no post weight: x += f d). One CTA per row; the row stays in registers between the two reductions.
+//   gated_norm    : out = rms(y * silu(z)) * weight * scale over `groups` equal parts of a row (state-space mixers), or
+//                   rms(y) * weight * scale * silu(z) (delta rules)
+//   embed_f32     : embedding rows into the fp32 stream, optionally RMS-normed on the way
 #include "hds_host.cuh"
 #include "hds_ptx.cuh"
 #include "../../../include/hds_b200.h"
@@ -49,7 +50,7 @@ __device__ __forceinline__ void store4(void* base, int64_t idx, float4 v) {
 
 // `cols`: values a row's mean is taken over; `padded` >= cols: row width, zeros behind the values. DELTA 0 none, 1 fp32
 // (cleared after being read), 2 the output's type.
-template <int THREADS, int VPT, int DT, int DELTA>
+template <int THREADS, int VPT, int DT, int DELTA, bool kPost>
 __global__ void __launch_bounds__(THREADS)
 norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const float* __restrict__ post,
                      const float* __restrict__ gamma, void* __restrict__ out, int64_t ld, int cols, int padded, float eps,
@@ -75,17 +76,19 @@ norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const flo
             }
             if constexpr (DELTA != 0) {
                 d[i].x *= factor; d[i].y *= factor; d[i].z *= factor; d[i].w *= factor;
-                ss += d[i].x * d[i].x + d[i].y * d[i].y + d[i].z * d[i].z + d[i].w * d[i].w;
+                if constexpr (kPost) ss += d[i].x * d[i].x + d[i].y * d[i].y + d[i].z * d[i].z + d[i].w * d[i].w;
             }
         }
     }
     if constexpr (DELTA != 0) {
-        const float r = 1.0f / sqrtf(block_sum_t<THREADS>(ss, red) / cols + eps);
+        float r = 1.0f;
+        if constexpr (kPost) r = 1.0f / sqrtf(block_sum_t<THREADS>(ss, red) / cols + eps);
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
             const int c = threadIdx.x + i * THREADS;
             if (c < nvec) {
-                const float4 w = *reinterpret_cast<const float4*>(post + 4 * c);
+                float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+                if constexpr (kPost) w = *reinterpret_cast<const float4*>(post + 4 * c);
                 v[i].x += d[i].x * r * w.x; v[i].y += d[i].y * r * w.y;
                 v[i].z += d[i].z * r * w.z; v[i].w += d[i].w * r * w.w;
                 if (store_x) *reinterpret_cast<float4*>(x + row + 4 * c) = v[i];
@@ -106,12 +109,12 @@ norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const flo
     }
 }
 
-template <int DT, int DELTA>
+template <int DT, int DELTA, bool kPost>
 static int launch_norm_residual(float* x, void* delta, float factor, const float* post, const float* gamma, void* out, int64_t ld,
                                 int rows, int cols, int padded, float eps, int store_x, cudaStream_t s) {
     const int nvec = padded / 4;
 #define HDS_NR(TH, V)                                                                                                       \
-    HDS_CHECK_CUDA(launch_kernel(norm_residual_kernel<TH, V, DT, DELTA>, dim3(rows), dim3(TH), 0, s, x, delta, factor, post, \
+    HDS_CHECK_CUDA(launch_kernel(norm_residual_kernel<TH, V, DT, DELTA, kPost>, dim3(rows), dim3(TH), 0, s, x, delta, factor, post, \
                                  gamma, out, ld, cols, padded, eps, store_x))
     if (nvec <= 128) HDS_NR(128, 1);
     else if (nvec <= 256) HDS_NR(256, 1);
@@ -136,7 +139,7 @@ __device__ __forceinline__ float gate_silu(float b) {
 template <int DT, int VPT>
 __global__ void __launch_bounds__(256)
 gated_norm_warp_kernel(const float* __restrict__ y, int64_t ld_y, const void* __restrict__ z, int64_t ld_z, const float* __restrict__ w,
-                       void* __restrict__ out, int64_t ld_out, int rows, int groups, int part, float eps, float scale) {
+                       void* __restrict__ out, int64_t ld_out, int rows, int groups, int part, float eps, float scale, int gate_after) {
     pdl_enter();
     const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (unit >= rows * groups) return;
@@ -155,10 +158,11 @@ gated_norm_warp_kernel(const float* __restrict__ y, int64_t ld_y, const void* __
     float ss = 0.0f;
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
-        g[i].x *= gate_silu<DT>(b[i].x);
-        g[i].y *= gate_silu<DT>(b[i].y);
-        g[i].z *= gate_silu<DT>(b[i].z);
-        g[i].w *= gate_silu<DT>(b[i].w);
+        b[i] = make_float4(gate_silu<DT>(b[i].x), gate_silu<DT>(b[i].y), gate_silu<DT>(b[i].z), gate_silu<DT>(b[i].w));
+        if (!gate_after) {
+            g[i].x *= b[i].x; g[i].y *= b[i].y; g[i].z *= b[i].z; g[i].w *= b[i].w;
+            b[i] = make_float4(1.f, 1.f, 1.f, 1.f);
+        }
         ss += g[i].x * g[i].x + g[i].y * g[i].y + g[i].z * g[i].z + g[i].w * g[i].w;
     }
     const float r = scale / sqrtf(warp_sum(ss) / part + eps);
@@ -167,17 +171,19 @@ gated_norm_warp_kernel(const float* __restrict__ y, int64_t ld_y, const void* __
         const int c = (lane + 32 * i) * 4;
         if (c < part) {
             const float4 ww = *reinterpret_cast<const float4*>(w + c0 + c);
-            store4<DT>(out, t * ld_out + c0 + c, make_float4(g[i].x * r * ww.x, g[i].y * r * ww.y, g[i].z * r * ww.z, g[i].w * r * ww.w));
+            store4<DT>(out, t * ld_out + c0 + c, make_float4(g[i].x * r * ww.x * b[i].x, g[i].y * r * ww.y * b[i].y,
+                                                                 g[i].z * r * ww.z * b[i].z, g[i].w * r * ww.w * b[i].w));
         }
     }
 }
 
 template <int DT>
 static cudaError_t launch_gated_norm_warp(const float* y, int64_t ld_y, const void* z, int64_t ld_z, const float* w, void* out, int64_t ld_out,
-                                          int rows, int groups, int part, float eps, float scale, cudaStream_t s) {
+                                          int rows, int groups, int part, float eps, float scale, int gate_after, cudaStream_t s) {
     const dim3 grid((static_cast<int64_t>(rows) * groups + 7) / 8), block(256);
 #define HDS_GNW(V) \
-    return launch_kernel(gated_norm_warp_kernel<DT, V>, grid, block, 0, s, y, ld_y, z, ld_z, w, out, ld_out, rows, groups, part, eps, scale)
+    return launch_kernel(gated_norm_warp_kernel<DT, V>, grid, block, 0, s, y, ld_y, z, ld_z, w, out, ld_out, rows, groups, part, eps, scale, \
+                         gate_after)
     if (part <= 128) HDS_GNW(1);
     if (part <= 256) HDS_GNW(2);
     if (part <= 512) HDS_GNW(4);
@@ -189,14 +195,14 @@ static cudaError_t launch_gated_norm_warp(const float* y, int64_t ld_y, const vo
 template <int DT>
 __global__ void __launch_bounds__(256)
 gated_norm_kernel(const float* __restrict__ y, int64_t ld_y, const void* __restrict__ z, int64_t ld_z,
-                  const float* __restrict__ w, void* __restrict__ out, int64_t ld_out, int part, float eps, float scale) {
+                  const float* __restrict__ w, void* __restrict__ out, int64_t ld_out, int part, float eps, float scale, int gate_after) {
     extern __shared__ float vals[];
     __shared__ float red[8];
     pdl_enter();
     const int64_t t = blockIdx.x;
     const int c0 = blockIdx.y * part;
     float ss = 0.0f;
-    const bool vec = (part & 3) == 0 && (ld_y & 3) == 0 && (ld_z & 3) == 0 && (ld_out & 3) == 0;
+    const bool vec = !gate_after && (part & 3) == 0 && (ld_y & 3) == 0 && (ld_z & 3) == 0 && (ld_out & 3) == 0;
     if (vec) {
         for (int c = threadIdx.x * 4; c < part; c += 1024) {
             const float4 a = *reinterpret_cast<const float4*>(y + t * ld_y + c0 + c);
@@ -212,7 +218,7 @@ gated_norm_kernel(const float* __restrict__ y, int64_t ld_y, const void* __restr
     } else {
         for (int c = threadIdx.x; c < part; c += 256) {
             const float b = load_any<DT>(z, t * ld_z + c0 + c);
-            const float g = y[t * ld_y + c0 + c] * gate_silu<DT>(b);
+            const float g = gate_after ? y[t * ld_y + c0 + c] : y[t * ld_y + c0 + c] * gate_silu<DT>(b);
             vals[c] = g;
             ss += g * g;
         }
@@ -226,7 +232,8 @@ gated_norm_kernel(const float* __restrict__ y, int64_t ld_y, const void* __restr
         }
     } else {
         for (int c = threadIdx.x; c < part; c += 256) {
-            const float v = vals[c] * r * w[c0 + c];
+            float v = vals[c] * r * w[c0 + c];
+            if (gate_after) v *= gate_silu<DT>(load_any<DT>(z, t * ld_z + c0 + c));
             if constexpr (DT == 2) reinterpret_cast<float*>(out)[t * ld_out + c0 + c] = v;
             else store_scalar<DT == 0>(out, t * ld_out + c0 + c, v);
         }
@@ -244,6 +251,29 @@ __global__ void embed_f32_kernel(const int32_t* __restrict__ ids, const void* __
             ok ? load4<DT>(W, static_cast<int64_t>(id) * H + c) : make_float4(0.f, 0.f, 0.f, 0.f);
 }
 
+// the same, each row then divided by its root mean square over `cols` and weighted
+template <int DT>
+__global__ void __launch_bounds__(256)
+embed_norm_f32_kernel(const int32_t* __restrict__ ids, const void* __restrict__ W, const float* __restrict__ gamma,
+                      float* __restrict__ out, int H, int vocab, int cols, float eps) {
+    __shared__ float red[8];
+    pdl_enter();
+    const int64_t t = blockIdx.x;
+    const int id = ids[t];
+    const bool ok = id >= 0 && id < vocab;
+    float ss = 0.0f;
+    for (int c = threadIdx.x * 4; c < H; c += 1024) {
+        const float4 v = ok ? load4<DT>(W, static_cast<int64_t>(id) * H + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    const float r = 1.0f / sqrtf(block_sum_t<256>(ss, red) / cols + eps);
+    for (int c = threadIdx.x * 4; c < H; c += 1024) {
+        const float4 v = ok ? load4<DT>(W, static_cast<int64_t>(id) * H + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        const float4 g = *reinterpret_cast<const float4*>(gamma + c);
+        *reinterpret_cast<float4*>(out + t * H + c) = make_float4(v.x * r * g.x, v.y * r * g.y, v.z * r * g.z, v.w * r * g.w);
+    }
+}
+
 }  // namespace hds
 
 using namespace hds;
@@ -253,15 +283,16 @@ extern "C" int hds_norm_residual(float* x, void* delta, int delta_is_f32, float 
                                  void* stream) {
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_norm_residual: dtype 0 bf16 / 1 fp16 / 2 fp32");
     HDS_REQUIRE(padded % 4 == 0 && ld % 4 == 0 && cols <= padded && padded <= ld, "hds_norm_residual: rows of 4-value vectors");
-    HDS_REQUIRE(delta == nullptr || post != nullptr, "hds_norm_residual: a delta needs its norm weight");
     if (rows == 0) return HDS_OK;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     const int mode = delta == nullptr ? 0 : delta_is_f32 ? 1 : 2;
 #define HDS_NR_ARGS x, delta, factor, post, gamma, out, ld, rows, cols, padded, eps, store_x, s
-#define HDS_NR_DT(DT)                                                            \
-    return mode == 0   ? launch_norm_residual<DT, 0>(HDS_NR_ARGS)                \
-           : mode == 1 ? launch_norm_residual<DT, 1>(HDS_NR_ARGS)                \
-                       : launch_norm_residual<DT, 2>(HDS_NR_ARGS)
+#define HDS_NR_DT(DT)                                                                               \
+    return mode == 0         ? launch_norm_residual<DT, 0, false>(HDS_NR_ARGS)                       \
+           : post == nullptr ? (mode == 1 ? launch_norm_residual<DT, 1, false>(HDS_NR_ARGS)          \
+                                          : launch_norm_residual<DT, 2, false>(HDS_NR_ARGS))         \
+           : mode == 1       ? launch_norm_residual<DT, 1, true>(HDS_NR_ARGS)                        \
+                             : launch_norm_residual<DT, 2, true>(HDS_NR_ARGS)
     if (dtype == 0) { HDS_NR_DT(0); }
     if (dtype == 1) { HDS_NR_DT(1); }
     HDS_NR_DT(2);
@@ -270,7 +301,7 @@ extern "C" int hds_norm_residual(float* x, void* delta, int delta_is_f32, float 
 }
 
 extern "C" int hds_gated_norm(const float* y, int64_t ld_y, const void* z, int64_t ld_z, const float* w, void* out, int64_t ld_out,
-                              int rows, int cols, int groups, float eps, float scale, int dtype, void* stream) {
+                              int rows, int cols, int groups, float eps, float scale, int gate_after, int dtype, void* stream) {
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_gated_norm: dtype 0 bf16 / 1 fp16 / 2 fp32");
     HDS_REQUIRE(groups >= 1 && cols % groups == 0 && cols / groups <= 12000, "hds_gated_norm: equal parts of at most 12000 values");
     if (rows == 0) return HDS_OK;
@@ -281,24 +312,31 @@ extern "C" int hds_gated_norm(const float* y, int64_t ld_y, const void* z, int64
     const uintptr_t al = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(z) * 2 |
                          reinterpret_cast<uintptr_t>(out) * 2;   // 16-byte vectors of fp32, 8-byte ones of the 16-bit types
     if (part % 4 == 0 && part <= 1024 && ld_y % 4 == 0 && ld_z % 4 == 0 && ld_out % 4 == 0 && (al & 15) == 0 && dtype != 2) {
-        HDS_CHECK_CUDA(dtype == 0 ? launch_gated_norm_warp<0>(y, ld_y, z, ld_z, w, out, ld_out, rows, groups, part, eps, scale, s)
-                                  : launch_gated_norm_warp<1>(y, ld_y, z, ld_z, w, out, ld_out, rows, groups, part, eps, scale, s));
+        HDS_CHECK_CUDA(dtype == 0 ? launch_gated_norm_warp<0>(y, ld_y, z, ld_z, w, out, ld_out, rows, groups, part, eps, scale, gate_after, s)
+                                  : launch_gated_norm_warp<1>(y, ld_y, z, ld_z, w, out, ld_out, rows, groups, part, eps, scale, gate_after, s));
         return HDS_OK;
     }
     if (dtype == 0)
-        HDS_CHECK_CUDA(launch_kernel(gated_norm_kernel<0>, grid, dim3(256), smem, s, y, ld_y, z, ld_z, w, out, ld_out, part, eps, scale));
+        HDS_CHECK_CUDA(launch_kernel(gated_norm_kernel<0>, grid, dim3(256), smem, s, y, ld_y, z, ld_z, w, out, ld_out, part, eps, scale, gate_after));
     else if (dtype == 1)
-        HDS_CHECK_CUDA(launch_kernel(gated_norm_kernel<1>, grid, dim3(256), smem, s, y, ld_y, z, ld_z, w, out, ld_out, part, eps, scale));
+        HDS_CHECK_CUDA(launch_kernel(gated_norm_kernel<1>, grid, dim3(256), smem, s, y, ld_y, z, ld_z, w, out, ld_out, part, eps, scale, gate_after));
     else
-        HDS_CHECK_CUDA(launch_kernel(gated_norm_kernel<2>, grid, dim3(256), smem, s, y, ld_y, z, ld_z, w, out, ld_out, part, eps, scale));
+        HDS_CHECK_CUDA(launch_kernel(gated_norm_kernel<2>, grid, dim3(256), smem, s, y, ld_y, z, ld_z, w, out, ld_out, part, eps, scale, gate_after));
     return HDS_OK;
 }
 
-extern "C" int hds_embed_f32(const int32_t* ids, const void* W, float* out, int T, int H, int vocab, int dtype, void* stream) {
+extern "C" int hds_embed_f32(const int32_t* ids, const void* W, const float* gamma, float* out, int T, int H, int vocab, int cols, float eps,
+                             int dtype, void* stream) {
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_embed_f32: dtype 0 bf16 / 1 fp16 / 2 fp32");
     HDS_REQUIRE(H % 4 == 0, "hds_embed_f32: rows of 4-value vectors");
     if (T == 0) return HDS_OK;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (gamma != nullptr) {
+        if (dtype == 0) HDS_CHECK_CUDA(launch_kernel(embed_norm_f32_kernel<0>, dim3(T), dim3(256), 0, s, ids, W, gamma, out, H, vocab, cols, eps));
+        else if (dtype == 1) HDS_CHECK_CUDA(launch_kernel(embed_norm_f32_kernel<1>, dim3(T), dim3(256), 0, s, ids, W, gamma, out, H, vocab, cols, eps));
+        else HDS_CHECK_CUDA(launch_kernel(embed_norm_f32_kernel<2>, dim3(T), dim3(256), 0, s, ids, W, gamma, out, H, vocab, cols, eps));
+        return HDS_OK;
+    }
     if (dtype == 0) HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<0>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab));
     else if (dtype == 1) HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<1>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab));
     else HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<2>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab));

@@ -328,6 +328,10 @@ static int launch_conv(const SsmArgs& a, cudaStream_t s) {
     return HDS_OK;
 }
 
+int ssm_conv_launch(const SsmArgs& a, int dtype, cudaStream_t s) {
+    return dtype == 0 ? launch_conv<0>(a, s) : dtype == 1 ? launch_conv<1>(a, s) : launch_conv<2>(a, s);
+}
+
 template <int DT>
 static int launch_scan(const SsmArgs& a, cudaStream_t s) {
     const dim3 grid(a.n_seqs, a.heads, (a.P + kScanP - 1) / kScanP), block(kScanWarps * 32);

@@ -1,4 +1,5 @@
-// Shared pieces of the state-space (Mamba-2) kernels: arguments, the sequences of a ragged batch, the scan's inner steps.
+// Shared pieces of the kernels with recurrent state (state-space mixers, delta rules): arguments, the sequences of a ragged batch,
+// the inner steps. A delta rule uses the same columns, x = v, B = k, C = q, and has one more per head behind dt (its step input).
 #pragma once
 #include "hds_host.cuh"
 #include "hds_ptx.cuh"
@@ -11,7 +12,7 @@ struct SsmSpan {
 };
 
 struct SsmArgs {
-    const void* proj;        // [T][ld_proj]: z (inner) | x (inner) | B (groups * N) | C (groups * N) | dt (heads)
+    const void* proj;        // [T][ld_proj]: z (inner) | x (inner) | B (groups * N) | C (groups * N) | dt (heads) [| step (heads)]
     int64_t ld_proj;
     const float* conv_w;     // [taps][channels]
     const float* conv_b;     // [channels]
@@ -73,6 +74,8 @@ __device__ __forceinline__ void ssm_save_conv_of_head(const SsmArgs& a, const Ss
     }
 }
 
+// convolution + silu of all sequences with several new tokens into u, softplus(dt + bias) into dt (ssm.cu)
+int ssm_conv_launch(const SsmArgs& a, int dtype, cudaStream_t s);
 bool ssm_chunk_supported(const SsmArgs& a, int dtype);
 int ssm_chunk_launch(const SsmArgs& a, int dtype, cudaStream_t s);
 

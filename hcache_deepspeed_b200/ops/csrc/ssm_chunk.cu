@@ -156,7 +156,8 @@ ssm_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a) {
                 const uint32_t ph = c & 1;
                 const uint64_t dbk = d_bk + 2 * ph * PANEL, dbn = d_bn + 2 * ph * PANEL, dc = d_c + 2 * ph * PANEL;
                 const uint32_t tc = t_cb + ph * 128, ty = t_y2 + ph * 64;
-                // ---- CB = C B^T ---- (over M of chunk c - 2, whose product has been issued)
+                // ---- CB = C B^T ---- (over M of chunk c - 2, whose product must be complete)
+                if (c > 1) mbar_wait(y_done, ph);
                 mbar_wait(cb_full + ph, (c >> 1) & 1);
                 tc_fence_after();
                 if (leader) {

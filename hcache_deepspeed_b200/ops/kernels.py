@@ -469,11 +469,14 @@ def moe_padded_rows(n_tokens: int, n_experts: int, top_k: int) -> int:
 
 
 def moe_topk_gating(logits: torch.Tensor, top_k: int, normalize: bool, scores: torch.Tensor, expert_ids: torch.Tensor,
-                    offsets: torch.Tensor, counts: torch.Tensor) -> None:
-    """Softmax + top-k per token; ``counts`` (int32 [E], zero on entry) is incremented per assignment."""
+                    offsets: torch.Tensor, counts: torch.Tensor, bias: Optional[torch.Tensor] = None, scale: float = 1.0,
+                    clear: bool = False) -> None:
+    """Softmax + top-k per token; ``counts`` (int32 [E], zero on entry) is incremented per assignment. ``bias`` (fp32 [E]) is added
+    to the scores that choose, ``scale`` multiplies the scores returned, ``clear`` zeroes (fp32) logits once read."""
     T, E = logits.shape
     code = 2 if logits.dtype == torch.float32 else _dt(logits)
-    rc = native.cuda_lib().hds_moe_topk_gating(_p(logits), logits.stride(0), T, E, top_k, int(normalize), code, _p(scores),
+    rc = native.cuda_lib().hds_moe_topk_gating(_p(logits), logits.stride(0), T, E, top_k, int(normalize), _p(bias), scale,
+                                                 int(clear), code, _p(scores),
                                                _p(expert_ids), _p(offsets), _p(counts), _stream())
     native.check(rc, "hds_moe_topk_gating")
     _count()
@@ -626,21 +629,28 @@ def moe_table_route(ids: torch.Tensor, table: torch.Tensor, n_experts: int, scor
 
 def moe_combine(y: torch.Tensor, mapped_slots: torch.Tensor, scores: torch.Tensor, base: Optional[torch.Tensor],
                 out: torch.Tensor) -> torch.Tensor:
-    """``out[t] = base[t] + sum_j scores[t, j] * y[mapped_slots[t, j]]`` (``out`` fp32, stored; ``base`` optional)."""
+    """``out[t] = base[t] + sum_j scores[t, j] * y[mapped_slots[t, j]]`` (``out`` fp32, stored; ``base`` optional, or ``out``
+    itself: added in place)."""
     T, k = mapped_slots.shape
     assert out.dtype == torch.float32
+    accumulate = base is not None and base.data_ptr() == out.data_ptr()
+    if accumulate:
+        base = None
+    assert base is None or base.dtype == y.dtype
     rc = native.cuda_lib().hds_moe_combine(_p(y), y.stride(0), _p(mapped_slots), _p(scores), _p(base),
-                                           0 if base is None else base.stride(0), _p(out), out.stride(0), T, k, y.shape[1], _dt3(y),
-                                           _stream())
+                                           0 if base is None else base.stride(0), _p(out), out.stride(0), T, k, y.shape[1],
+                                             int(accumulate), _dt3(y), _stream())
     native.check(rc, "hds_moe_combine")
     _count()
     return out
 
 
-def embed_f32(ids: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+def embed_f32(ids: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gamma: Optional[torch.Tensor] = None,
+              cols: Optional[int] = None, eps: float = 1e-5) -> torch.Tensor:
+    """Embedding rows in fp32; with ``gamma`` RMS-normed over their first ``cols`` values and weighted."""
     assert ids.dtype == torch.int32 and out.dtype == torch.float32
-    rc = native.cuda_lib().hds_embed_f32(_p(ids), _p(weight), _p(out), ids.numel(), weight.shape[1], weight.shape[0], _dt3(weight),
-                                         _stream())
+    rc = native.cuda_lib().hds_embed_f32(_p(ids), _p(weight), _p(gamma), _p(out), ids.numel(), weight.shape[1], weight.shape[0],
+                                         weight.shape[1] if cols is None else cols, eps, _dt3(weight), _stream())
     native.check(rc, "hds_embed_f32")
     _count()
     return out
@@ -649,7 +659,8 @@ def embed_f32(ids: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> tor
 def norm_residual(resid: torch.Tensor, gamma: torch.Tensor, out: torch.Tensor, delta: Optional[torch.Tensor] = None,
                   factor: float = 1.0, post: Optional[torch.Tensor] = None, cols: Optional[int] = None, eps: float = 1e-5,
                   store_resid: bool = True) -> torch.Tensor:
-    """``resid += norm(factor * delta) * post`` on the fp32 stream, ``out = norm(resid) * gamma`` (``hds_norm_residual``)."""
+    """``resid += norm(factor * delta) * post`` (without ``post``: ``resid += factor * delta``) on the fp32 stream,
+    ``out = norm(resid) * gamma`` (``hds_norm_residual``)."""
     rows, width = resid.shape
     assert resid.stride(0) == out.stride(0) and (delta is None or delta.stride(0) == resid.stride(0))
     assert delta is None or delta.dtype in (torch.float32, out.dtype)
@@ -662,10 +673,11 @@ def norm_residual(resid: torch.Tensor, gamma: torch.Tensor, out: torch.Tensor, d
 
 
 def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, groups: int, eps: float,
-               scale: float = 1.0) -> torch.Tensor:
-    """``out = scale * weight * v / rms(v)``, ``v = y * silu(z)``, rms per part of a row (``groups`` equal parts)."""
+               scale: float = 1.0, gate_after: bool = False) -> torch.Tensor:
+    """``out = scale * weight * v / rms(v)``, ``v = y * silu(z)``, rms per part of a row (``groups`` equal parts); ``gate_after``:
+    ``out = scale * weight * y / rms(y) * silu(z)``."""
     rc = native.cuda_lib().hds_gated_norm(_p(y), y.stride(0), _p(z), z.stride(0), _p(weight), _p(out), out.stride(0), y.shape[0],
-                                          y.shape[1], groups, eps, scale, _dt3(out), _stream())
+                                          y.shape[1], groups, eps, scale, int(gate_after), _dt3(out), _stream())
     native.check(rc, "hds_gated_norm")
     _count()
     return out
@@ -693,11 +705,14 @@ def state_space(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, 
 
 def paged_attention_generic(q: torch.Tensor, out: torch.Tensor, kv_cache_layer: torch.Tensor, block_tables: torch.Tensor,
                             tok_seq: torch.Tensor, tok_pos: torch.Tensor, n_q_heads: int, n_kv_heads: int, head_dim: int,
-                            block_size: int, scale: float, window: int = 0, keep_first: int = 0) -> None:
-    """fp32-arithmetic attention for any operand type and head size (``hds_paged_attention_generic``)."""
+                            block_size: int, scale: float, window: int = 0, keep_first: int = 0, value_dim: int = 0,
+                            spans: Optional[torch.Tensor] = None, limit: int = 0) -> None:
+    """fp32-arithmetic attention for any operand type and head size (``hds_paged_attention_generic``). ``value_dim`` > 0: pages of
+    one plane, the first ``value_dim`` values of a key row are its value. ``spans``: skip sequences of more than ``limit`` tokens."""
     rc = native.cuda_lib().hds_paged_attention_generic(_p(q), _p(out), out.stride(0), _p(kv_cache_layer), _p(block_tables),
                                                        block_tables.stride(0), _p(tok_seq), _p(tok_pos), q.shape[0], n_q_heads,
-                                                       n_kv_heads, head_dim, block_size, scale, window, keep_first, _dt3(q), _stream())
+                                                       n_kv_heads, head_dim, block_size, scale, window, keep_first, value_dim, _p(spans),
+                                                       limit, _dt3(q), _stream())
     native.check(rc, "hds_paged_attention_generic")
     _count()
 
@@ -708,3 +723,75 @@ def kv_append_generic(qkv: torch.Tensor, q_out: torch.Tensor, kv_cache_layer: to
                                                  n_q_heads, n_kv_heads, head_dim, block_size, qkv.element_size(), _stream())
     native.check(rc, "hds_kv_append_generic")
     _count()
+
+
+# ------------------------------------------------------------------------------------------------
+# latent attention, gated delta rule
+# ------------------------------------------------------------------------------------------------
+def latent_append(proj: torch.Tensor, q_out: Optional[torch.Tensor], pages: Optional[torch.Tensor], tok_pos: torch.Tensor,
+                  tok_slot: torch.Tensor, heads: int, dim: int, rot_dim: int, head_width: int, rank: int, freq: torch.Tensor,
+                  norm_w: Optional[torch.Tensor], eps: float) -> None:
+    """Rotated queries to ``q_out`` [T, heads * head_width] and normed latents with their rotated key part to their ``pages``
+    [blocks, 1, 1, bs, width], from ``proj`` = [q heads | latent | key part] (either output optional)."""
+    width = rank + rot_dim if pages is None else pages.shape[4]
+    rc = native.cuda_lib().hds_latent_append(_p(proj), proj.stride(0), _p(q_out), _p(pages), _p(tok_pos), _p(tok_slot), proj.shape[0], heads,
+                                             dim, rot_dim, head_width, rank, width, _p(freq), _p(norm_w), eps, _dt3(proj), _stream())
+    native.check(rc, "hds_latent_append")
+    _count()
+
+
+def head_matmul(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tok_seq: torch.Tensor, spans: torch.Tensor, limit: int, in_width: int,
+                out_width: int, copy: int = 0) -> torch.Tensor:
+    """``out[t, h, :N] = x[t, h, :K] @ w[h]`` for ``w`` [heads, K, N]; then ``copy`` input values from place K on, then zeros. Rows of a
+    head are ``in_width`` / ``out_width`` wide. Tokens of sequences with more than ``limit`` new tokens are skipped."""
+    heads, K, N = w.shape
+    rc = native.cuda_lib().hds_head_matmul(_p(x), x.stride(0), in_width, _p(w), _p(out), out.stride(0), out_width, _p(tok_seq), _p(spans), limit,
+                                           x.shape[0], heads, K, N, copy, _dt3(x), _stream())
+    native.check(rc, "hds_head_matmul")
+    _count()
+    return out
+
+
+def latent_attention_supported(rank: int, page_width: int) -> bool:
+    """Does the tensor-core kernel take latents of this size (else: :func:`paged_attention_generic`)?"""
+    return bool(native.cuda_lib().hds_paged_attention_latent_supported(rank, page_width))
+
+
+def latent_attention_workspace_bytes() -> int:
+    return int(native.cuda_lib().hds_paged_attention_latent_workspace_bytes())
+
+
+def paged_attention_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tensor, block_tables: torch.Tensor, items: torch.Tensor,
+                           n_items: int, item_tokens: int, heads: int, rank: int, block_size: int, n_splits: int, scale: float,
+                           workspace: torch.Tensor, window: int = 0) -> None:
+    """tcgen05 attention in the latent space: ``q`` [T, heads * width], ``pages`` [blocks, 1, 1, bs, width], ``out`` [T, heads * rank].
+    One CTA = 128 (token, head) rows of an item (of at most ``item_tokens`` tokens) and up to 256 of the latent's values."""
+    rc = native.cuda_lib().hds_paged_attention_latent(_p(q), _p(out), _p(pages), pages.shape[0], _p(block_tables), block_tables.stride(0),
+                                                      _p(items), n_items, item_tokens, q.shape[0], heads, rank, pages.shape[4], block_size,
+                                                      scale, window, n_splits, _p(workspace), workspace.numel(), _dt(q), _stream())
+    native.check(rc, "hds_paged_attention_latent")
+    _count()
+
+
+def delta_workspace_bytes(n_tokens: int, n_seqs: int, heads: int, groups: int) -> int:
+    """Scratch of the chunked delta rule for batches of up to ``n_tokens`` tokens in ``n_seqs`` sequences."""
+    return int(native.cuda_lib().hds_delta_workspace_bytes(n_tokens, n_seqs, heads, groups))
+
+
+def delta_rule(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, dt_bias: torch.Tensor, decay: torch.Tensor, state: torch.Tensor,
+               conv_state: torch.Tensor, spans: torch.Tensor, n_single: int, groups: int, u: torch.Tensor, dt: torch.Tensor, y: torch.Tensor,
+               out: Optional[torch.Tensor], norm_w: torch.Tensor, eps: float, workspace: Optional[torch.Tensor] = None,
+               method: int = SCAN_AUTO) -> torch.Tensor:
+    """Convolution and recurrence of a gated delta rule over a ragged batch (``hds_delta_rule``), and, with ``out``, the norm and gate
+    behind it. ``state`` [slots, heads, vdim, dim]. Without ``out`` (or when sequences bring several tokens) ``y`` holds the read-outs."""
+    T = proj.shape[0]
+    _, heads, vdim, n = state.shape
+    rc = native.cuda_lib().hds_delta_rule(_p(proj), proj.stride(0), _p(conv_w), _p(conv_b), _p(dt_bias), _p(decay), _p(state), _p(conv_state),
+                                          _p(spans), spans.shape[0], n_single, T, heads, vdim, n, groups, conv_w.shape[0], _p(u), u.stride(0),
+                                          _p(dt), _p(y), _p(out), 0 if out is None else out.stride(0), _p(norm_w), eps, _p(workspace),
+                                          0 if workspace is None else workspace.numel(), method, _dt3(proj), _stream())
+    native.check(rc, "hds_delta_rule")
+    _count((2 if spans.shape[0] > n_single else 0) + (1 if n_single else 0))
+    if out is not None and n_single < spans.shape[0]:
+        gated_norm(y, proj[:, :heads * vdim], norm_w, out, heads, eps, gate_after=True)
+    return y

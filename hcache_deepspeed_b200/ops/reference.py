@@ -163,19 +163,23 @@ def attention_scale(head_dim: int) -> float:
 def norm_residual(resid: torch.Tensor, gamma: torch.Tensor, delta: Optional[torch.Tensor], factor: float,
                   post: Optional[torch.Tensor], cols: int, eps: float):
     """Returns (new fp32 stream, normed stream): stream += rms(factor * delta) * post, then rms(stream) * gamma. Rows hold
-    ``cols`` values and zeros behind them."""
+    ``cols`` values and zeros behind them. ``post`` None: stream += factor * delta."""
     x = resid
     if delta is not None:
         d = delta.float() * factor
-        x = x + d * torch.rsqrt((d * d).sum(-1, keepdim=True) / cols + eps) * post
+        x = x + (d if post is None else d * torch.rsqrt((d * d).sum(-1, keepdim=True) / cols + eps) * post)
     return x, x * torch.rsqrt((x * x).sum(-1, keepdim=True) / cols + eps) * gamma
 
 
-def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, scale: float = 1.0) -> torch.Tensor:
-    """rms of each of ``groups`` equal parts of y * silu(z), times weight, times scale."""
-    g = y.float() * F.silu(z.float())
+def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, scale: float = 1.0,
+               gate_after: bool = False) -> torch.Tensor:
+    """rms of each of ``groups`` equal parts of y * silu(z), times weight, times scale; with ``gate_after`` the norm is of y alone
+    and silu(z) multiplies its result."""
+    gate = F.silu(z.float())
+    g = y.float() if gate_after else y.float() * gate
     p = g.reshape(g.shape[0], groups, -1)
-    return (p * torch.rsqrt((p * p).mean(-1, keepdim=True) + eps)).reshape(g.shape) * weight * scale
+    out = (p * torch.rsqrt((p * p).mean(-1, keepdim=True) + eps)).reshape(g.shape) * weight * scale
+    return out * gate if gate_after else out
 
 
 def short_conv(u: torch.Tensor, conv_state: torch.Tensor, w: torch.Tensor, b: torch.Tensor, pos0: int) -> torch.Tensor:
@@ -203,3 +207,59 @@ def selective_scan(x: torch.Tensor, B: torch.Tensor, C: torch.Tensor, dt: torch.
         state.mul_(torch.exp(a * dt[t])[:, None, None]).add_((dt[t][:, None] * xt)[:, :, None] * Bt.float()[:, None, :])
         y[t] = (state * Ct.float()[:, None, :]).sum(-1) + d[:, None] * xt
     return y
+
+
+#: added under the root when the delta rule's queries and keys are made unit vectors
+DELTA_UNIT_EPS = 1e-6
+
+
+def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, beta: torch.Tensor, state: torch.Tensor) -> torch.Tensor:
+    """S <- decay S; S <- S + beta (v - S k) k^T; y = S q for every token of one sequence. q / k [n, groups, N] (as they come out of
+    the convolution: made unit vectors here, q also times N^-1/2), v [n, heads, P], decay / beta [n, heads]; ``state``
+    [heads, P, N] fp32 is advanced in place."""
+    n, H, P = v.shape
+    rep, N = H // k.shape[1], k.shape[2]
+
+    def unit(x):
+        return x.float() * torch.rsqrt((x.float()**2).sum(-1, keepdim=True) + DELTA_UNIT_EPS)
+
+    q, k = (unit(q) * N**-0.5).repeat_interleave(rep, 1), unit(k).repeat_interleave(rep, 1)
+    y = torch.empty((n, H, P), dtype=torch.float32)
+    for t in range(n):
+        state.mul_(decay[t][:, None, None])
+        u = beta[t][:, None] * (v[t].float() - (state * k[t][:, None, :]).sum(-1))
+        state.add_(u[:, :, None] * k[t][:, None, :])
+        y[t] = (state * q[t][:, None, :]).sum(-1)
+    return y
+
+
+def rotate_pairs(x: torch.Tensor, pos: torch.Tensor, freq: torch.Tensor) -> torch.Tensor:
+    """x [T, ..., dims]: the pair (2i, 2i + 1) turned by pos * freq[i]; fp32."""
+    ang = (pos.float()[:, None] * freq[None, :]).reshape((x.shape[0], ) + (1, ) * (x.dim() - 2) + (-1, ))
+    c, s = ang.cos(), ang.sin()
+    u, v = x[..., 0::2].float(), x[..., 1::2].float()
+    return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
+
+
+def latent_rows(y: torch.Tensor, pos: torch.Tensor, rank: int, freq: torch.Tensor, weight: torch.Tensor, eps: float, width: int) -> torch.Tensor:
+    """What a token caches, ``[T, width]``: the normed latent, the rotated key part, zeros. ``y`` [T, rank + rot]."""
+    c = y[:, :rank].float()
+    c = c * torch.rsqrt((c * c).mean(-1, keepdim=True) + eps) * weight
+    return F.pad(torch.cat([c, rotate_pairs(y[:, rank:], pos, freq)], 1), (0, width - y.shape[1]))
+
+
+def paged_latent_attention(q: torch.Tensor, pages: torch.Tensor, block_tables: torch.Tensor, items: torch.Tensor, rank: int, scale: float,
+                           window: int = 0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Attention in the latent space: q [T, heads, rank + rot], pages [blocks, 1, 1, bs, width]; returns the heads' mean latents
+    [T, heads, rank]. Items and windows as in :func:`paged_attention`."""
+    if out is None:
+        out = torch.zeros(q.shape[0], q.shape[1], rank, dtype=q.dtype, device=q.device)
+    bs = pages.shape[3]
+    for seq, row0, n, pos0 in items.tolist():
+        kv_len = pos0 + n
+        rows = pages[block_tables[seq, :-(-kv_len // bs)].long(), 0, 0].flatten(0, 1)[:kv_len, :q.shape[2]].float()
+        s = torch.einsum("qhd,kd->hqk", q[row0:row0 + n].float(), rows) * scale
+        back = (pos0 + torch.arange(n, device=q.device))[:, None] - torch.arange(kv_len, device=q.device)[None, :]
+        s = s.masked_fill((back < 0) | (back >= (window or kv_len)), float("-inf"))
+        out[row0:row0 + n] = torch.einsum("hqk,kd->qhd", torch.softmax(s, -1), rows[:, :rank]).to(out.dtype)
+    return out

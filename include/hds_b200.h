@@ -248,11 +248,13 @@ int hds_attention_next_out_stride(int64_t elements);
 
 /* Paged attention in plain fp32 arithmetic for operands and head sizes the tensor-core kernels do not take: dtype 0 bf16,
  * 1 fp16, 2 fp32, head_dim up to 512. One warp per (token, query head); tok_seq / tok_pos give each token's block-table row and
- * position. window / keep_first as above. */
+ * position. window / keep_first as above. value_dim > 0: pages of one plane [blocks][heads][block][head_dim], the first value_dim
+ * values of a key row are its value (and out has rows of n_q_heads * value_dim). spans (hds_state_space; optional): sequences that
+ * bring more than `limit` tokens are skipped. */
 int hds_paged_attention_generic(const void* q, void* out, int64_t ld_out, const void* kv_cache_layer, const int32_t* block_tables,
                                 int max_blocks_per_seq, const int32_t* tok_seq, const int32_t* tok_pos, int T, int n_q_heads,
-                                int n_kv_heads, int head_dim, int block_size, float scale, int window, int keep_first, int dtype,
-                                void* stream);
+                                int n_kv_heads, int head_dim, int block_size, float scale, int window, int keep_first,
+                                int value_dim, const int32_t* spans, int limit, int dtype, void* stream);
 /* hds_rope_kv_append without rotation, for 2- or 4-byte elements and any head_dim. */
 int hds_kv_append_generic(const void* qkv, int64_t ld_qkv, void* q_out, void* kv_cache_layer, const int32_t* tok_slot, int T,
                           int n_q_heads, int n_kv_heads, int head_dim, int block_size, int elem_bytes, void* stream);
@@ -283,9 +285,11 @@ int64_t hds_paged_attention_prefill_workspace_bytes(int n_items, int n_q_heads, 
 
 /* ---- mixture of experts (tensor-parallel experts; ref ragged_ops/{top_k_gating,moe_scatter,moe_gather}, moe_gemm) --- */
 /* Per token: softmax over E logits, top-k (ties -> lower index), optional renormalisation of the k scores.
- * counts[E] must be zero on entry (hds_moe_scatter re-zeroes it). offsets[t, j] = row claimed inside expert_ids[t, j]. */
-int hds_moe_topk_gating(const void* logits, int64_t ld_logits, int T, int E, int k, int normalize, int logits_dtype,
-                        float* scores, int32_t* expert_ids, int32_t* offsets, int32_t* counts, void* stream);
+ * counts[E] must be zero on entry (hds_moe_scatter re-zeroes it). offsets[t, j] = row claimed inside expert_ids[t, j].
+ * bias[E] (optional) is added to the softmax scores that choose, `scale` multiplies the returned ones, `clear` zeroes the (fp32)
+ * logits after they are read. */
+int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E, int k, int normalize, const float* bias, float scale, int clear,
+                        int logits_dtype, float* scores, int32_t* expert_ids, int32_t* offsets, int32_t* counts, void* stream);
 /* pad_off[E+1]: expert row ranges rounded up to 128 rows; xs[row] = x[t] for every (t, j); mapped_slots[t, j] = row.
  * xs needs hds_moe_padded_rows(T, E, k) rows. */
 int hds_moe_scatter(const void* x, int64_t ldx, void* xs, int64_t ld_xs, const int32_t* expert_ids,
@@ -371,23 +375,28 @@ int hds_gemm_next_act_limit(float limit);
 /* Expert choice by token id: expert_ids[t, j] = table[ids[t], j], scores = 1 / k; offsets / counts as hds_moe_topk_gating. */
 int hds_moe_table_route(const int32_t* ids, const int32_t* table, int vocab, int T, int E, int k, float* scores, int32_t* expert_ids,
                         int32_t* offsets, int32_t* counts, void* stream);
-/* out[t, :] = base[t, :] + sum_j scores[t, j] * y[mapped_slots[t, j], :] (stored; base optional; dtype of y and base 0 / 1 / 2). */
+/* out[t, :] = base[t, :] + sum_j scores[t, j] * y[mapped_slots[t, j], :] (stored; base optional; dtype of y and base 0 / 1 / 2;
+ * accumulate: out itself is one more summand). */
 int hds_moe_combine(const void* y, int64_t ldy, const int32_t* mapped_slots, const float* scores, const void* base, int64_t ldb,
-                    float* out, int64_t ldo, int T, int k, int H, int dtype, void* stream);
+                    float* out, int64_t ldo, int T, int k, int H, int accumulate, int dtype, void* stream);
 
-/* out[t] = W[ids[t]] as fp32 (rows of H values; ids outside the vocabulary give zeros). dtype of W 0 / 1 / 2. */
-int hds_embed_f32(const int32_t* ids, const void* W, float* out, int T, int H, int vocab, int dtype, void* stream);
+/* out[t] = W[ids[t]] as fp32 (rows of H values; ids outside the vocabulary give zeros). dtype of W 0 / 1 / 2. gamma (optional): each
+ * row is divided by its root mean square over `cols` values (eps inside the root) and weighted. */
+int hds_embed_f32(const int32_t* ids, const void* W, const float* gamma, float* out, int T, int H, int vocab, int cols, float eps,
+                  int dtype, void* stream);
 
-/* One sublayer boundary of a stack with norms on both sides of its sublayers, on an fp32 residual stream x [rows, ld]:
- *   x += (factor * delta) / rms(factor * delta) * post   (delta NULL: skipped);   out = x / rms(x) * gamma
+/* One sublayer boundary of a stack on an fp32 residual stream x [rows, ld]:
+ *   x += (factor * delta) / rms(factor * delta) * post   (delta NULL: skipped; post NULL: x += factor * delta)
+ *   out = x / rms(x) * gamma
  * rms over the first `cols` values of a row (the rest of `padded` are zeros). An fp32 delta is cleared after being read; a
  * 16-bit one has out's dtype. store_x 0: x is only read. dtype of out 0 bf16, 1 fp16, 2 fp32. All rows ld apart. */
 int hds_norm_residual(float* x, void* delta, int delta_is_f32, float factor, const float* post, const float* gamma, void* out,
                       int64_t ld, int rows, int cols, int padded, float eps, int store_x, int dtype, void* stream);
 
-/* out = scale * w * v / rms(v) with v = y * silu(z), rms over each of `groups` equal parts of a row. y, w fp32; z, out dtype. */
+/* out = scale * w * v / rms(v) with v = y * silu(z), rms over each of `groups` equal parts of a row; gate_after:
+ * out = scale * w * y / rms(y) * silu(z). y, w fp32; z, out dtype. */
 int hds_gated_norm(const float* y, int64_t ld_y, const void* z, int64_t ld_z, const float* w, void* out, int64_t ld_out, int rows,
-                   int cols, int groups, float eps, float scale, int dtype, void* stream);
+                   int cols, int groups, float eps, float scale, int gate_after, int dtype, void* stream);
 
 /* State-space (Mamba-2) mixer between its projections, over a ragged batch of T rows. proj: [T, ld_proj] rows of
  * z | x (heads * vdim each) | B | C (groups * state_size each) | dt (heads). A causal convolution of `taps` taps (conv_w
@@ -402,6 +411,41 @@ int hds_state_space(const void* proj, int64_t ld_proj, const float* conv_w, cons
                     const float* decay_rate, const float* skip, float* state, float* conv_state, const int32_t* spans, int n_seqs,
                     int n_single, int T, int heads, int vdim, int state_size, int groups, int taps, void* u, int64_t ld_u, float* dt,
                     float* y, int method, int dtype, void* stream);
+
+/* Gated delta rule between its projections, over a ragged batch. proj rows: gate | v (heads * vdim each) | k | q (groups * dim each) |
+ * decay input | step input (heads each). Convolution and silu over v | k | q (as hds_state_space); k and q become unit vectors
+ * (1e-6 under the root, q also times dim^-1/2); g = exp(decay_rate * softplus(decay input + dt_bias)), beta = sigmoid(step input);
+ *     S = g S,  u = beta (v - S^T k),  S = S + k u^T,  y = S^T q    per head.
+ * state [slots, heads, vdim, dim] fp32; spans, conv_state, u, dt, y, method as hds_state_space. When every sequence brings one token
+ * and out is given, out [T, ld_out] (dtype) = y / rms(y per head) * norm_w * silu(gate) is written instead of y. workspace
+ * (hds_delta_workspace_bytes; optional) enables the chunked tensor-core form for sequences with several tokens. */
+int hds_delta_rule(const void* proj, int64_t ld_proj, const float* conv_w, const float* conv_b, const float* dt_bias,
+                   const float* decay_rate, float* state, float* conv_state, const int32_t* spans, int n_seqs, int n_single, int T,
+                   int heads, int vdim, int dim, int groups, int taps, void* u, int64_t ld_u, float* dt, float* y, void* out,
+                   int64_t ld_out, const float* norm_w, float eps, void* workspace, int64_t workspace_bytes, int method, int dtype,
+                   void* stream);
+int64_t hds_delta_workspace_bytes(int T, int n_seqs, int heads, int groups);
+
+/* Latent attention, behind its input projection: proj rows = heads * head_width query values (dim unrotated, rot_dim rotated, zeros) |
+ * rank latent values | rot_dim key values. Adjacent pairs of the rotated parts turn by position * freq[i]; the latent is RMS-normed with
+ * norm_w. q_out [T, heads * head_width] and / or the tokens' page rows [latent | key part | zeros] of page_width values. */
+int hds_latent_append(const void* proj, int64_t ld, void* q_out, void* pages, const int32_t* tok_pos, const int32_t* tok_slot, int T,
+                      int heads, int dim, int rot_dim, int head_width, int rank, int page_width, const float* freq, const float* norm_w,
+                      float eps, int dtype, void* stream);
+/* out[t][h][0..N) = x[t][h][0..K) w[h] for w [heads][K][N], then `copy` values of x from K on, then zeros up to out_width. Tokens of
+ * sequences that bring more than `limit` tokens (spans, tok_seq) are skipped. dtype 0 / 1 / 2. */
+int hds_head_matmul(const void* x, int64_t ld_x, int in_width, const void* w, void* out, int64_t ld_out, int out_width,
+                    const int32_t* tok_seq, const int32_t* spans, int limit, int T, int heads, int K, int N, int copy, int dtype,
+                    void* stream);
+/* Attention of q [T][heads][page_width] over cached rows [latent | key part | zeros] shared by all heads; out [T][heads][rank] = mean
+ * latents. items: at most item_tokens tokens each. n_splits > 1: at most 148 CTAs in all. */
+int hds_paged_attention_latent(const void* q, void* out, const void* pages, int64_t num_blocks, const int32_t* block_tables,
+                               int max_blocks_per_seq, const hds_attn_item* items, int n_items, int item_tokens, int T, int heads, int rank,
+                               int page_width, int block_size, float scale, int window, int n_splits, void* workspace,
+                               int64_t workspace_bytes, int dtype, void* stream);
+int hds_paged_attention_latent_supported(int rank, int page_width);
+/* Scratch for n_splits > 1. Zero it once; the kernel leaves its tickets zeroed. */
+int64_t hds_paged_attention_latent_workspace_bytes(void);
 
 #ifdef __cplusplus
 }
