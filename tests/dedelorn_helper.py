@@ -57,7 +57,7 @@ TILED = config([(delta(heads=4, kv=2, dim=128, vdim=128, conv=4), dense(ff=192))
                 (latent(heads=4, dim=64, rot=64, vdim=64, rank=512, size=None, scale=0.08), dense(ff=128))], width=256, vocab=256)
 
 
-def make_weights(cfg, seed, dtype):
+def make_weights(cfg, seed, dtype, settled):
     """Random checkpoint tensors. Scales keep every branch audible in the logits."""
     g = torch.Generator().manual_seed(seed)
     W, V = cfg["width"], cfg["vocab"]
@@ -95,6 +95,8 @@ def make_weights(cfg, seed, dtype):
         else:
             n, ff = f["router"]["experts"], f["expert"]["ff"]
             w[q + "router"], w[q + "correction"] = rnd(n, W, scale=2 * W**-0.5), rnd(n, scale=0.3)
+            if settled:       # corrections further apart than scores can be
+                w[q + "correction"] = (1.5 * torch.randperm(n, generator=g)).to(dtype)
             for e in range(n):
                 w[f"{q}e{e}.up"], w[f"{q}e{e}.down"] = rnd(ff, W), rnd(W, ff, scale=2 * ff**-0.5)
     return w

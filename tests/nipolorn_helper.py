@@ -49,7 +49,7 @@ TILED = config([(mixer(heads=8, kv=2, dim=128, vdim=128, size=150, keep=9, scale
                        norm_groups=4), moe(ff=64, experts=8, top=2, shared=128))], width=256, vocab=256)
 
 
-def make_weights(cfg, seed, dtype):
+def make_weights(cfg, seed, dtype, settled):
     """Random checkpoint tensors. Scales keep every branch audible in the logits."""
     g = torch.Generator().manual_seed(seed)
     W, V = cfg["width"], cfg["vocab"]

@@ -5,12 +5,13 @@ import os
 
 import torch
 
-#: config "architecture" -> (weights(cfg, seed, dtype), oracle module)
+#: config "architecture" -> (weights(cfg, seed, dtype, settled), oracle module)
 DESIGNS = {}
 
 
-def weights(cfg, seed=0, dtype=torch.bfloat16):
-    return DESIGNS[cfg["architecture"]][0](cfg, seed, dtype)
+def weights(cfg, seed=0, dtype=torch.bfloat16, run_in=torch.float32):
+    """Random checkpoint tensors. For a run in 16 bits (``run_in``) no router's choice may be a close call, which rounding decides."""
+    return DESIGNS[cfg["architecture"]][0](cfg, seed, dtype, run_in != torch.float32)
 
 
 def save(folder, cfg, w):
@@ -77,7 +78,7 @@ TOLERANCE = {torch.float32: 1e-4, torch.bfloat16: 0.15, torch.float16: 3e-2}
 # ---- scenarios shared by the CPU and GPU tests ---------------------------------------------------------------------
 def check_whole_and_portions(cfg, dtype, device, n=190, tol=None):
     """One request: at once, in portions of several sizes (down to two tokens), and token by token, against the oracle."""
-    w, t = weights(cfg), tokens(cfg, n)
+    w, t = weights(cfg, run_in=dtype), tokens(cfg, n)
     want, tol = expected(cfg, w, t), tol or TOLERANCE[dtype]
     eng = engine(cfg, w, dtype, device, tokens=512)
     for uid, portions in enumerate([None, [n - 40], [2, 3, 2, 64, 1, 37, 65], [128, 2, 30], [130, 7]]):
@@ -90,7 +91,7 @@ def check_whole_and_portions(cfg, dtype, device, n=190, tol=None):
 def check_mixed_batches(cfg, dtype, device, tol=None):
     """Unequal requests in one batch: portions beside single tokens, a request left out of steps, pages and state slots freed
     and used again by others; every logit as if the request were alone."""
-    w, tol = weights(cfg, seed=3), tol or TOLERANCE[dtype]
+    w, tol = weights(cfg, seed=3, run_in=dtype), tol or TOLERANCE[dtype]
     eng = engine(cfg, w, dtype, device, tokens=512, live=3)
     lengths = {"a": 150, "b": 37, "c": 90, "d": 64, "e": 5, "f": 140, "g": 1}
     toks = {k: tokens(cfg, n, seed=ord(k)) for k, n in lengths.items()}
@@ -113,14 +114,14 @@ def check_mixed_batches(cfg, dtype, device, tol=None):
 
 
 def check_long_decode(cfg, dtype, device, n=330, tol=None):
-    w, t = weights(cfg, seed=4), tokens(cfg, n, seed=6)
+    w, t = weights(cfg, seed=4, run_in=dtype), tokens(cfg, n, seed=6)
     eng = engine(cfg, w, dtype, device, tokens=384)
     assert error(run(eng, 0, t, [7]), expected(cfg, w, t)) < (tol or TOLERANCE[dtype])
 
 
 def check_restore(cfg, dtype, device, tol=None):
     """Hidden states saved while a prompt runs rebuild pages AND recurrent state of another sequence."""
-    w, t = weights(cfg, seed=7), tokens(cfg, 150, seed=8)
+    w, t = weights(cfg, seed=7, run_in=dtype), tokens(cfg, 150, seed=8)
     eng = engine(cfg, w, dtype, device, tokens=512, enabled=True, capture="sync")
     first, lat = eng.put([0], [t[:101]])
     _, lat2 = eng.put([0], [t[101:103]])
@@ -138,7 +139,7 @@ def check_restore(cfg, dtype, device, tol=None):
 def check_greedy(cfg, dtype, device_is_gpu, folder, n_new=24):
     """Greedy generation through init_inference: every chosen token is the oracle's best (or as good, within rounding)."""
     import hcache_deepspeed_b200 as hds
-    w = weights(cfg, seed=10)
+    w = weights(cfg, seed=10, run_in=dtype)
     path = save(folder, cfg, w)
     eng = hds.init_inference(path, dtype=dtype, hcache={"max_context": 512, "max_batch_tokens": 512, "max_sessions": 8,
                                                         "kv_memory_bytes": 64 << 20})

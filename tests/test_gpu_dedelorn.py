@@ -319,7 +319,7 @@ def test_greedy_generation(dtype, tmp_path):
 
 def test_prompts_attend_in_the_latent_space_when_scratch_pages_run_out():
     cfg = H.TILED
-    w, t = H.weights(cfg, seed=5), H.tokens(cfg, 300)
+    w, t = H.weights(cfg, seed=5, run_in=BF16), H.tokens(cfg, 300)
     eng = H.engine(cfg, w, BF16, "cuda")
     eng.model()._latent_bufs.blocks = 1
     assert H.error(H.run(eng, 0, t, [150, 2, 100, 48]), H.expected(cfg, w, t)) < H.TOLERANCE[BF16]
@@ -327,7 +327,7 @@ def test_prompts_attend_in_the_latent_space_when_scratch_pages_run_out():
 
 def test_decode_runs_as_a_graph_and_fp16_is_served():
     cfg = H.TILED
-    w, t = H.weights(cfg, seed=2), H.tokens(cfg, 60)
+    w, t = H.weights(cfg, seed=2, run_in=F16), H.tokens(cfg, 60)
     eng = H.engine(cfg, w, F16, "cuda")
     assert H.error(H.run(eng, 0, t, [20]), H.expected(cfg, w, t)) < H.TOLERANCE[F16]
     assert eng.graph_replays > 20
