@@ -1,4 +1,4 @@
-"""Throughput of stacks that mix attention with recurrent state, beside the closest plain families at equal sizes.
+"""Throughput of stacks that mix attention with recurrent state, beside the closest families at equal sizes.
 
 ``bench.py --stacks``. Four layers of each size, random weights, through the public engine: one 4096-token prompt, and decode steps
 of 8 and 64 sequences at 4096 tokens of context. Then the kernels that only such stacks use, each next to its counterpart in a
@@ -13,7 +13,8 @@ from typing import Callable, Dict, Optional
 
 import torch
 
-PAIRS = [("nipolorn-2048", "mistral-2048"), ("nipolorn-4096", "mistral-4096"), ("nipolorn-4096-moe", "qwen2-moe-4096")]
+GROUPS = [("dedelorn-2048", "nipolorn-2048", "mistral-2048"), ("dedelorn-4096", "nipolorn-4096", "mistral-4096"),
+          ("dedelorn-4096-moe", "nipolorn-4096-moe", "qwen2-moe-4096")]
 PROMPT = 4096
 
 
@@ -108,7 +109,7 @@ def bench_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
             proj, cw, cb, db, a, d, state, ring, spans, single, G, u, dt, y), need)
         mix, w = rnd(rows, inner), torch.ones(inner, device=dev)
         report(f"gated norm {rows}x{inner}", "gated_norm", lambda: K.gated_norm(y, proj[:, :inner], w, mix, G, 1e-5, 0.5), rows * inner * (4 + 2 + 2))
-    from ..ops.backend import pick_packed_splits, windowed_len
+    from ..ops.backend import latent_splits, pick_packed_splits, windowed_len
     nq, nkv, D, page = 32, 8, 128, 64
     ws = torch.zeros(256 << 20, dtype=torch.uint8, device=dev)
     for window, keep in ((0, 0), (1024, 0), (1024, 64), (4096, 64)):
@@ -132,12 +133,77 @@ def bench_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
                K.paged_attention_prefill(q, o, cache, tables, items, B, nq, nkv, D, page, 0.09, n_splits=sp, workspace=ws, packed=True,
                                          window=window, keep_first=keep), B * keys * 2 * nkv * D * 2)
     del cache
+    # gated delta rule: 32 heads of 128 x 128, 16 groups; norm and gate behind it included
+    heads, P, N, G = 32, 128, 128, 16
+    inner, C = heads * P, heads * P + 2 * G * N
+    cw, cb, db, a = torch.randn(4, C, device=dev) * 0.5, torch.zeros(C, device=dev), vec(heads) - 3, -torch.exp(vec(heads))
+    for rows, seqs in ((T, 1), (T, 4), (64, 64), (8, 8)):
+        n = rows // seqs
+        proj = rnd(rows, inner + C + 2 * heads)
+        state, ring = torch.zeros(seqs, heads, P, N, device=dev), torch.zeros(seqs, 4, C, device=dev)
+        spans = torch.tensor([[i * n, n, 128, i] for i in range(seqs)], dtype=torch.int32, device=dev)
+        u, dt, y = torch.zeros(rows, C, dtype=bf, device=dev), torch.zeros(rows, heads, device=dev), torch.zeros(rows, inner, device=dev)
+        mix, w = rnd(rows, inner), torch.ones(inner, device=dev)
+        dws = torch.empty(K.delta_workspace_bytes(rows, seqs, heads, G), dtype=torch.uint8, device=dev) if n > 1 else None
+        moved = 2 * seqs * (heads * P * N + 4 * C) * 4
+        if n > 1:
+            report(f"delta rule {seqs}x{n}", "conv + chunked delta rule", lambda: K.delta_rule(
+                proj, cw, cb, db, a, state, ring, spans, 0, G, u, dt, y, None, w, 1e-5, dws), rows * (C * 2 + 2 * heads * 2 + inner * 4) + moved)
+            report(f"norm + gate {rows}x{inner}", "gated_norm", lambda: K.gated_norm(y, proj[:, :inner], w, mix, heads, 1e-5, gate_after=True),
+                   rows * inner * (4 + 2 + 2))
+        else:
+            report(f"delta rule {seqs}x{n}", "step with norm and gate", lambda: K.delta_rule(
+                proj, cw, cb, db, a, state, ring, spans, seqs, G, u, dt, y, mix, w, 1e-5), rows * (C * 2 + 2 * heads * 2 + inner * 4) + moved)
+    # latent attention: 32 heads of 96 + 32 rotated, values of 128, latents of 512
+    nh, dim, rot, rank, hw, width = 32, 96, 32, 512, 128, 576
+    from ..models.hybrid import rotation_frequencies
+    freq, gl = rotation_frequencies(rot, 1e4).to(dev), torch.ones(rank, device=dev)
+    for rows in (T, 64):
+        proj, q = rnd(rows, nh * hw + rank + rot), rnd(rows, nh * hw)
+        pages = rnd(rows // page + 1, 1, 1, page, width)
+        pos = torch.arange(rows, dtype=torch.int32, device=dev)
+        report(f"latent append {rows}", "latent_append", lambda: K.latent_append(proj, q, pages, pos, pos, nh, dim, rot, hw, rank, freq, gl, 1e-5),
+               rows * (2 * nh * hw + 2 * rank + rot + width) * 2)
+        qkv, cache = rnd(rows, (nh + 16) * 128), rnd(rows // page + 1, 2, 8, page, 128)
+        report(f"latent append {rows}", "rope_kv_append (like)", lambda: K.rope_kv_append(qkv, q, cache, pos, pos, torch.ones(64, device=dev), 32, 8, 128,
+                                                                                        128, page), rows * 2 * (nh + 16) * 128 * 2)
+    lws = torch.zeros(K.latent_attention_workspace_bytes(), dtype=torch.uint8, device=dev)
+    for B, window in ((64, 0), (64, 1024), (8, 1024)):
+        pages = rnd(B * T // page, 1, 1, page, width)
+        tables = torch.randperm(B * T // page, device=dev).to(torch.int32).view(B, T // page).contiguous()
+        lat, mean = rnd(B, nh * width, scale=0.1), rnd(B, nh * rank)
+        items = torch.tensor([[i, i, 1, T - 1] for i in range(B)], dtype=torch.int32, device=dev)
+        sp = latent_splits(B, 1, nh, rank, T, window)
+        keys = T if not window else min(T, window)
+        report(f"latent attention decode {B}x{T} window {window}", "paged_attention_latent", lambda: K.paged_attention_latent(
+            lat, mean, pages, tables, items, B, 1, nh, rank, page, sp, 0.09, lws, window), B * keys * (rank + rot) * 2)
+    del pages
+    seq, spans = torch.arange(64, dtype=torch.int32, device=dev), torch.ones(64, 4, dtype=torch.int32, device=dev)
+    wk, wv = rnd(nh, dim, rank, scale=0.02), rnd(nh, rank, 128, scale=0.02)
+    for B in (64, 8):
+        q, lat, mean, o = rnd(B, nh * hw), rnd(B, nh * width), rnd(B, nh * rank), rnd(B, nh * 128)
+        report(f"queries to latents {B}", "head_matmul", lambda: K.head_matmul(q, wk, lat, seq, spans, 8, hw, width, rot),
+               (wk.numel() + q.numel() + lat.numel()) * 2)
+        report(f"latents to values {B}", "head_matmul", lambda: K.head_matmul(mean, wv, o, seq, spans, 8, rank, 128), (wv.numel() + mean.numel() + o.numel()) * 2)
+    rows16, w_kv = rnd(T, width), rnd(2 * nh * hw, width, scale=0.02)
+    kv = rnd(T // page, 2, nh, page, hw)
+    slot = torch.arange(T, dtype=torch.int32, device=dev)
+    report(f"latents to K / V pages {T}", "restore_kv_proj", lambda: K.restore_kv_proj(rows16, w_kv, kv, slot, slot, None, nh, hw, page),
+           bytes_=(rows16.numel() + w_kv.numel() + kv.numel()) * 2, flops=2.0 * T * w_kv.numel())
+    q, o = rnd(T, nh * hw), rnd(T, nh * hw)
+    table = torch.arange(T // page, dtype=torch.int32, device=dev)[None].contiguous()
+    items = torch.tensor([[0, i, 128, i] for i in range(0, T, 128)], dtype=torch.int32, device=dev)
+    for window in (0, 1024):
+        pairs = sum(min(i + 1, window or T) for i in range(T))
+        report(f"latent attention prefill {T} window {window}", "paged_attention_prefill on projected pages", lambda: K.paged_attention_prefill(
+            q, o, kv, table, items, T // 128, nh, nh, hw, page, 0.09, window=window), flops=2.0 * pairs * nh * (dim + rot + 128))
+    del kv, q, o
     ff = 14336
     w_up = rnd(2 * ff, W, scale=0.02)
     wsg = torch.zeros(K.gemm_splitk_workspace_bytes(128, 2 * ff), dtype=torch.uint8, device=dev)
     for rows in (T, 64, 8):
         x, h = rnd(rows, W), rnd(rows, ff)
-        for act, tag in ((5, "gated GEMM, clamped"), (3, "gated GEMM, silu (like)")):
+        for act, tag in ((5, "gated GEMM, clamped"), (4, "gated GEMM, gelu"), (3, "gated GEMM, silu (like)")):
             report(f"mlp up {rows}x{2 * ff}x{W}", tag, lambda: K.gemm(x, w_up, out=h, act=act, gated=True, limit=7.0,
                                                                        workspace=wsg if rows <= 128 else None),
                    2 * (2 * ff * W + rows * (W + ff)), 2.0 * rows * 2 * ff * W)
@@ -160,14 +226,28 @@ def bench_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
 
         report(f"route + scatter {rows}", "table", by_table, rows * W * 2 * (1 + top))
         report(f"route + scatter {rows}", "top-k gate (like)", by_gate, rows * W * 2 * (1 + top))
+        wr, lg32, bias = rnd(E, W, scale=0.02), torch.zeros(rows, E, device=dev), torch.zeros(E, device=dev)
+
+        def by_corrected_gate():
+            K.gemm_accum(x, wr, lg32)
+            K.moe_topk_gating(lg32, top, False, scores, e, off, counts, bias=bias, scale=2.5, clear=True)
+            K.moe_scatter(x, xs, e, off, counts, pad, slots, top)
+
+        report(f"router + route + scatter {rows}", "fp32 scores, corrected top-k gate", by_corrected_gate, rows * W * 2 * (2 + top))
+
+        def by_gate_too():
+            K.gemm(x, wr, out=lg)
+            by_gate()
+
+        report(f"router + route + scatter {rows}", "16-bit router, top-k gate (like)", by_gate_too, rows * W * 2 * (2 + top))
         report(f"combine {rows}", "moe_combine + shared", lambda: K.moe_combine(ys, slots, scores, base, out), rows * W * (2 * top + 2 + 4))
         report(f"combine {rows}", "moe_gather (like)", lambda: K.moe_gather(ys, slots, scores, out), rows * W * (2 * top + 4 + 4))
 
 
 def main(steps: int = 5, warmup: int = 3) -> None:
     p = peaks()
-    for pair in PAIRS:
-        for name in pair:
+    for group in GROUPS:
+        for name in group:
             print(json.dumps({"stack": name, "layers": 4, "prompt": PROMPT, "dtype": "bf16", "data": "random weights, synthetic tokens",
                               **bench_engine(name, steps, warmup)}), flush=True)
             torch.cuda.empty_cache()

@@ -684,13 +684,22 @@ def named_arch(name: str) -> ArchSpec:
 
 
 def _stack_named() -> Dict[str, ArchSpec]:
-    """Nipolorn stacks with layers of real sizes, and beside each the closest plain family at equal sizes (same width, heads,
-    window and feed-forward): windowed attention with a dense MLP, or with routed experts and a shared one."""
+    """Nipolorn and Dedelorn stacks with layers of real sizes, and beside each the closest plain family at equal sizes (same width,
+    heads, window and feed-forward): windowed attention with a dense MLP, or with routed experts and a shared one."""
 
     def nipolorn(width, heads, kv, window, keep, ssm_heads, groups, mlp):
         mixer = MixerSpec(attn=AttentionSpec(heads, kv, 128, 128, 128 ** -0.5, window, keep),
                           ssm=StateSpaceSpec(ssm_heads, 64, 128, groups, 4, groups), attn_weight=1.0, ssm_weight=0.5)
         return stack_arch("nipolorn", [LayerSpec(mixer, mlp)] * 4, hidden=width, vocab=32000, norm_eps=1e-5, **NIPOLORN_NORMS)
+
+    def dedelorn(width, heads, rank, window, mlp):
+        delta = MixerSpec(delta=DeltaSpec(heads=width // 128, kv_heads=width // 256, dim=128, vdim=128, conv=4))
+
+        def latent(kv_from=None):
+            return MixerSpec(latent=LatentAttentionSpec(heads, 96, 32, 128, rank, 128**-0.5, window, 1e4, kv_from))
+
+        return stack_arch("dedelorn", [LayerSpec(m, mlp) for m in (delta, latent(), delta, latent(1))], hidden=width, vocab=32000,
+                          norm_eps=1e-5, **DEDELORN_NORMS)
 
     def plain(mt, width, heads, kv, window, **kw):
         return ArchSpec(model_type=mt, n_layers=4, hidden=width, n_heads=heads, n_kv_heads=kv, head_dim=128, vocab=32000, norm="rms",
@@ -699,6 +708,10 @@ def _stack_named() -> Dict[str, ArchSpec]:
     moe = dict(n_experts=16, top_k=2, moe_intermediate=3584, shared_expert_intermediate=3584)
     return {
         "nipolorn-2048": nipolorn(2048, 16, 4, 1024, 16, 64, 4, FeedForwardSpec(ff=8192, act="swiglu_clamped", limit=7.0)),
+        "dedelorn-2048": dedelorn(2048, 16, 256, 1024, FeedForwardSpec(ff=8192, act="gelu_tanh")),
+        "dedelorn-4096": dedelorn(4096, 32, 512, 4096, FeedForwardSpec(ff=14336, act="gelu_tanh")),
+        "dedelorn-4096-moe": dedelorn(4096, 32, 512, 2048, FeedForwardSpec(ff=5376, act="gelu", experts=16, top=2, routing="softmax", gated=False,
+                                                                            router_scale=2.5)),
         "mistral-2048": plain("mistral", 2048, 16, 4, 1024, intermediate=8192),
         "nipolorn-4096": nipolorn(4096, 32, 8, 4096, 64, 128, 8, FeedForwardSpec(ff=14336, act="swiglu_clamped", limit=7.0)),
         "mistral-4096": plain("mistral", 4096, 32, 8, 4096, intermediate=14336),

@@ -532,10 +532,15 @@ def latent_launches(batch, heads: int, rank: int, width: int, window: int, with_
         out.append(("large", batch.n_items_large, batch.max_large_item_tokens, batch.max_kv_len_large))
     launches = []
     for kind, n, tokens, kv_len in out:
-        ctas = n * -(-tokens * heads // 128) * -(-rank // 256)
-        tiles = max(1, -(-windowed_len(kv_len, window) // 64))
-        launches.append((kind, n, tokens, int(max(1, min(MAX_PREFILL_SPLITS, N_SM // ctas, tiles // 2)))))
+        launches.append((kind, n, tokens, latent_splits(n, tokens, heads, rank, kv_len, window)))
     return tuple(launches)
+
+
+def latent_splits(n_items: int, item_tokens: int, heads: int, rank: int, max_kv_len: int, window: int) -> int:
+    """KV splits of the latent attention kernel: one wave of CTAs at most, at least 2 tiles of 64 keys each."""
+    ctas = n_items * -(-item_tokens * heads // 128) * -(-rank // 256)
+    tiles = max(1, -(-windowed_len(max_kv_len, window) // 64))
+    return int(max(1, min(MAX_PREFILL_SPLITS, N_SM // ctas, tiles // 2)))
 
 
 class LatentBuffers:
