@@ -19,6 +19,7 @@
 //   1     : TMEM allocation, tcgen05.mma issue
 //   2-9   : the state's chain — two-term state, R, U
 //   10-17 : inverse -> TMEM, decayed scores in TMEM, output                 (both groups: two threads per TMEM lane)
+// The chain runs ahead: the output of a chunk is formed while the next one already solves for its U.
 // TMEM: scores 128 columns, inverse 128, S^T k and then U 64, scores x U 64, S^T q 64, state 64.
 #include "delta.cuh"
 #include "../../../include/hds_b200.h"
@@ -205,16 +206,16 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
         float x[32];
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-            float v = static_cast<int>(lane) == i ? 1.0f : 0.0f;
+            float v0 = static_cast<int>(lane) == i ? 1.0f : 0.0f, v1 = 0.0f, v2 = 0.0f, v3 = 0.0f;
 #pragma unroll
             for (int j = 0; j < i; j += 4) {
                 const float4 l = *reinterpret_cast<const float4*>(D + i * kPrepPitch + j);      // (zero on and above the diagonal)
-                v = fmaf(-l.x, x[j], v);
-                if (j + 1 < i) v = fmaf(-l.y, x[j + 1], v);
-                if (j + 2 < i) v = fmaf(-l.z, x[j + 2], v);
-                if (j + 3 < i) v = fmaf(-l.w, x[j + 3], v);
+                v0 = fmaf(-l.x, x[j], v0);
+                if (j + 1 < i) v1 = fmaf(-l.y, x[j + 1], v1);
+                if (j + 2 < i) v2 = fmaf(-l.z, x[j + 2], v2);
+                if (j + 3 < i) v3 = fmaf(-l.w, x[j + 3], v3);
             }
-            x[i] = v;
+            x[i] = (v0 + v1) + (v2 + v3);
         }
         __syncwarp();
 #pragma unroll
@@ -233,14 +234,18 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
             const float* L = step == 0 ? X21 : X22;
             const float* R = step == 0 ? X11 : T1;
             const int rp = step == 0 ? kPrepPitch : 36;
-#pragma unroll 4
-            for (int k = 0; k < 32; ++k) {
-                const float2 w = *reinterpret_cast<const float2*>(R + k * rp + j0);
+#pragma unroll 2
+            for (int k = 0; k < 32; k += 4) {
+                float2 w[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) w[e] = *reinterpret_cast<const float2*>(R + (k + e) * rp + j0);
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    const float l = L[(i0 + i) * kPrepPitch + k];
-                    acc[i][0] = fmaf(l, w.x, acc[i][0]);
-                    acc[i][1] = fmaf(l, w.y, acc[i][1]);
+                    const float4 l = *reinterpret_cast<const float4*>(L + (i0 + i) * kPrepPitch + k);
+                    acc[i][0] = fmaf(l.x, w[0].x, acc[i][0]); acc[i][1] = fmaf(l.x, w[0].y, acc[i][1]);
+                    acc[i][0] = fmaf(l.y, w[1].x, acc[i][0]); acc[i][1] = fmaf(l.y, w[1].y, acc[i][1]);
+                    acc[i][0] = fmaf(l.z, w[2].x, acc[i][0]); acc[i][1] = fmaf(l.z, w[2].y, acc[i][1]);
+                    acc[i][0] = fmaf(l.w, w[3].x, acc[i][0]); acc[i][1] = fmaf(l.w, w[3].y, acc[i][1]);
                 }
             }
             if (step == 1) __syncthreads();
@@ -260,16 +265,22 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
             const float* L = step == 0 ? X21 : X22;
             const float* R = step == 0 ? A : tmp;
             const int rp = step == 0 ? kPrepPitch : 68;
-#pragma unroll 4
-            for (int k = 0; k < 64; ++k) {
-                const float4 w = *reinterpret_cast<const float4*>(R + k * rp + j0);
+#pragma unroll 2
+            for (int k = 0; k < 64; k += 4) {
+                float4 w[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) w[e] = *reinterpret_cast<const float4*>(R + (k + e) * rp + j0);
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    const float l = L[(i0 + i) * kPrepPitch + k];
-                    acc[i][0] = fmaf(l, w.x, acc[i][0]);
-                    acc[i][1] = fmaf(l, w.y, acc[i][1]);
-                    acc[i][2] = fmaf(l, w.z, acc[i][2]);
-                    acc[i][3] = fmaf(l, w.w, acc[i][3]);
+                    const float4 l4 = *reinterpret_cast<const float4*>(L + (i0 + i) * kPrepPitch + k);
+                    const float l[4] = {l4.x, l4.y, l4.z, l4.w};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        acc[i][0] = fmaf(l[e], w[e].x, acc[i][0]);
+                        acc[i][1] = fmaf(l[e], w[e].y, acc[i][1]);
+                        acc[i][2] = fmaf(l[e], w[e].z, acc[i][2]);
+                        acc[i][3] = fmaf(l[e], w[e].w, acc[i][3]);
+                    }
                 }
             }
             if (step == 1) __syncthreads();
@@ -303,8 +314,8 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
 }
 
 // ---- chunk after chunk --------------------------------------------------------------------------------------------------
-constexpr size_t kDcSmem = 4 * kDcPanel /*k: two buffers*/ + 2 * kDcPanel /*q*/ + kDcPanel /*v*/ + 2 * kDcPanel /*S*/ + 2 * kDcPanel /*R, then U*/ +
-                           2 * kDcPanel /*weighted U*/ + 2 * kDcTok * 4 + 256;
+constexpr size_t kDcSmem = 4 * kDcPanel /*k: two buffers*/ + 2 * kDcPanel /*q*/ + kDcPanel /*v*/ + 2 * kDcPanel /*S*/ + 2 * kDcPanel /*U*/ +
+                           2 * kDcPanel /*R, then weighted U*/ + 2 * kDcTok * 4 + 256;
 
 __global__ void __launch_bounds__(kDcThreads, 1)
 delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, const DeltaWs ws) {
@@ -415,13 +426,13 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
                     if (kk < k_steps)
                         umma_f16_ss(d, rows + (kk >> 2) * PANEL + 2 * (kk & 3), d_s + t * PANEL + kk * ROWS16, IDESC_KN, (t > 0 || kk > 0) ? 1u : 0u);
         };
-        // two-term matrix in TMEM x two-term rows in u_sm: hi hi + hi lo + lo hi
-        auto times_u = [&](uint32_t d, uint32_t m) {
+        // two-term matrix in TMEM x two-term rows: hi hi + hi lo + lo hi
+        auto times_rows = [&](uint32_t d, uint32_t m, uint64_t rows) {
 #pragma unroll
             for (int t = 0; t < 3; ++t)
 #pragma unroll
                 for (int kk = 0; kk < kDcTok / 16; ++kk)
-                    umma_f16_ts(d, m + kk * 16 + (t == 2 ? 8 : 0), d_u + (t == 1 ? PANEL : 0) + kk * ROWS16, IDESC_KN, (t > 0 || kk > 0) ? 1u : 0u);
+                    umma_f16_ts(d, m + kk * 16 + (t == 2 ? 8 : 0), rows + (t == 1 ? PANEL : 0) + kk * ROWS16, IDESC_KN, (t > 0 || kk > 0) ? 1u : 0u);
         };
         for (int c = 0; c < n_chunks; ++c) {
             const uint32_t ph = c & 1;
@@ -434,6 +445,23 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
                 umma_commit(x_done);
             }
             __syncwarp();
+            if (c > 0) {      // scores x U of the chunk before, while R of this one is formed
+                mbar_wait(p_full, ph ^ 1);
+                tc_fence_after();
+                if (leader) {
+                    times_rows(t_y1, t_cb, d_u);
+                    umma_commit(y_done);
+                }
+                __syncwarp();
+            }
+            mbar_wait(t_full, ph);
+            mbar_wait(r_full, ph);
+            tc_fence_after();
+            if (leader) {
+                times_rows(t_xu, t_inv, d_w);
+                umma_commit(u_done);
+            }
+            __syncwarp();
             // (the outputs of the chunk before have been read, so its last product is complete: products of unlike shapes are not
             // ordered by themselves, and the scores below overwrite that product's operand)
             if (c > 0) mbar_wait(y_free, ph ^ 1);
@@ -442,14 +470,6 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
             if (leader) times_state(t_y2, d_q);
             __syncwarp();
             scores(c);
-            mbar_wait(t_full, ph);
-            mbar_wait(r_full, ph);
-            tc_fence_after();
-            if (leader) {
-                times_u(t_xu, t_inv);
-                umma_commit(u_done);
-            }
-            __syncwarp();
             mbar_wait(u_full, ph);
             tc_fence_after();
             if (leader) {      // (the state has been scaled in place)
@@ -462,14 +482,14 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
                 umma_commit(k_empty + (c & 1));
             }
             __syncwarp();
-            mbar_wait(p_full, ph);
-            tc_fence_after();
-            if (leader) {
-                times_u(t_y1, t_cb);
-                umma_commit(y_done);
-            }
-            __syncwarp();
         }
+        mbar_wait(p_full, (n_chunks - 1) & 1);
+        tc_fence_after();
+        if (leader) {
+            times_rows(t_y1, t_cb, d_u);
+            umma_commit(y_done);
+        }
+        __syncwarp();
     } else if (warp < 10) {
         // ===================== the state's chain: thread = (token r of the chunk and key dimension, column half) =====================
         const int quad = warp & 3, half = (warp - 2) >> 2;
@@ -482,14 +502,20 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
             __syncwarp();
             if (lane == 0) mbar_arrive(b);
         };
+        float a_last_n, a_r_n, beta_n, rk_n;      // of the next chunk, loaded a chunk ahead
+        auto load_factors = [&](int c) {
+            const int row = sp.row0 + c * kDcTok, n = min(kDcTok, sp.n - c * kDcTok);
+            const int64_t th = static_cast<int64_t>(row + r) * H + h;
+            a_last_n = __ldcg(ws.a + static_cast<int64_t>(row + n - 1) * H + h);
+            a_r_n = r < n ? __ldcg(ws.a + th) : 0.0f;
+            beta_n = r < n ? __ldcg(ws.beta + th) : 0.0f;
+            rk_n = r < n ? __ldcg(ws.rk + static_cast<int64_t>(row + r) * a.groups + g) : 0.0f;
+        };
+        load_factors(0);
         for (int c = 0; c < n_chunks; ++c) {
             const uint32_t ph = c & 1;
-            const int row = sp.row0 + c * kDcTok, n = min(kDcTok, sp.n - c * kDcTok);
-            const bool live = r < n;
-            const int64_t th = static_cast<int64_t>(row + r) * H + h;
-            const float a_last = __ldcg(ws.a + static_cast<int64_t>(row + n - 1) * H + h);
-            const float a_r = live ? __ldcg(ws.a + th) : a_last, beta = live ? __ldcg(ws.beta + th) : 0.0f;
-            const float rk = live ? __ldcg(ws.rk + static_cast<int64_t>(row + r) * a.groups + g) : 0.0f;
+            const bool live = r < min(kDcTok, sp.n - c * kDcTok);
+            const float a_last = a_last_n, a_r = live ? a_r_n : a_last, beta = beta_n, rk = rk_n;
             const float keep = dc_ex2(a_last), from_state = dc_ex2(a_r) * rk, weight = dc_ex2(a_last - a_r) * rk;
             // ---- the state: two-term copy, then scaled in place for its update ----
             uint32_t sw[32];
@@ -534,7 +560,7 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
             uint32_t x[32];
             tmem_ld_32x32(t_xu + la + half * 32, x);
             tmem_ld_wait();
-            if (c > 0) mbar_wait(y_done, ph ^ 1);      // U of the chunk before has been multiplied
+            if (c + 1 < n_chunks) load_factors(c + 1);
 #pragma unroll
             for (int ch = 0; ch < 4; ++ch) {
                 const uint32_t vv[4] = {v[ch].x, v[ch].y, v[ch].z, v[ch].w};
@@ -545,8 +571,8 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
                     const float r1 = beta * (bf16_hi(vv[e]) - from_state * __uint_as_float(x[8 * ch + 2 * e + 1]));
                     dc_split(live ? r0 : 0.0f, live ? r1 : 0.0f, hi[e], lo[e]);
                 }
-                *dc_cell(u_sm, r, half * 4 + ch) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-                *dc_cell(u_sm + kDcPanel, r, half * 4 + ch) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+                *dc_cell(w_sm, r, half * 4 + ch) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                *dc_cell(w_sm + kDcPanel, r, half * 4 + ch) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
             }
             arrive(r_full);
             if (lane == 0) mbar_arrive(v_empty);      // (all of v has been used)
@@ -555,6 +581,7 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
             tc_fence_after();
             tmem_ld_32x32(t_xu + la + half * 32, x);
             tmem_ld_wait();
+            if (c > 0) mbar_wait(y_done, ph ^ 1);      // U of the chunk before has been multiplied
 #pragma unroll
             for (int ch = 0; ch < 4; ++ch) {
                 uint32_t hi[4], lo[4], whi[4], wlo[4];
@@ -618,17 +645,8 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
             }
             __syncwarp();
         };
-        float prev = 0.0f;
-        for (int c = 0; c < n_chunks; ++c) {
-            const uint32_t ph = c & 1;
-            const int row = sp.row0 + c * kDcTok, n = min(kDcTok, sp.n - c * kDcTok);
-            const bool live = r < n;
-            const float a_last = __ldcg(ws.a + static_cast<int64_t>(row + n - 1) * H + h);
-            const float a_r = live ? __ldcg(ws.a + static_cast<int64_t>(row + r) * H + h) : a_last;
-            const float rk = live ? __ldcg(ws.rk + static_cast<int64_t>(row + r) * a.groups + g) : 1.0f;
-            const float rq = live ? __ldcg(ws.rq + static_cast<int64_t>(row + r) * a.groups + g) : 0.0f;
-            if (half == 0) b_s[ph * kDcTok + r] = a_r - __log2f(rk);
-            // ---- the inverse: my row's 64 columns, 16 at a time ----
+        // the inverse of chunk c: my row's 64 columns, 16 at a time
+        auto load_inverse = [&](int c) {
             const uint8_t* src = ws.inv + ((static_cast<int64_t>(first + c) * H + h) * kDcTok + r) * kInvRow + half * 128;
             uint4 hi[8], lo[8];
 #pragma unroll
@@ -636,7 +654,7 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
                 hi[i] = __ldcg(reinterpret_cast<const uint4*>(src + i * 16));      // (not through L1: the launch before wrote it)
                 lo[i] = __ldcg(reinterpret_cast<const uint4*>(src + 256 + i * 16));
             }
-            if (c > 0) mbar_wait(u_done, ph ^ 1);
+            if (c > 0) mbar_wait(u_done, (c - 1) & 1);
             tc_fence_after();
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
@@ -648,8 +666,23 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(t_full);
-            if (c > 0) output(c - 1, prev);
-            prev = dc_ex2(a_r) * rq;
+            __syncwarp();
+        };
+        float a_last_n, a_r_n, rk_n, rq_n;
+        auto load_factors = [&](int c) {
+            const int row = sp.row0 + c * kDcTok, n = min(kDcTok, sp.n - c * kDcTok);
+            a_last_n = __ldcg(ws.a + static_cast<int64_t>(row + n - 1) * H + h);
+            a_r_n = r < n ? __ldcg(ws.a + static_cast<int64_t>(row + r) * H + h) : 0.0f;
+            rk_n = r < n ? __ldcg(ws.rk + static_cast<int64_t>(row + r) * a.groups + g) : 1.0f;
+            rq_n = r < n ? __ldcg(ws.rq + static_cast<int64_t>(row + r) * a.groups + g) : 0.0f;
+        };
+        load_factors(0);
+        load_inverse(0);
+        for (int c = 0; c < n_chunks; ++c) {
+            const uint32_t ph = c & 1;
+            const float a_r = r < min(kDcTok, sp.n - c * kDcTok) ? a_r_n : a_last_n, rq = rq_n;
+            if (half == 0) b_s[ph * kDcTok + r] = a_r - __log2f(rk_n);
+            if (c + 1 < n_chunks) load_factors(c + 1);
             asm volatile("bar.sync 2, 256;" ::: "memory");     // b_s of this chunk is complete
             // ---- decayed scores, in place: 16 fp32 columns become 8 of leading terms and 8 of rests ----
             const float* bv = b_s + ph * kDcTok;
@@ -670,7 +703,15 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
                     const int mine = r - jp;
                     float v[16];
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) v[j] = j > mine ? 0.0f : __uint_as_float(cb[j]) * rq * dc_ex2(a_r - bv[jp + j]);
+                    for (int j = 0; j < 16; j += 4) {
+                        const float4 b = *reinterpret_cast<const float4*>(bv + jp + j);
+                        v[j + 0] = __uint_as_float(cb[j + 0]) * rq * dc_ex2(a_r - b.x);
+                        v[j + 1] = __uint_as_float(cb[j + 1]) * rq * dc_ex2(a_r - b.y);
+                        v[j + 2] = __uint_as_float(cb[j + 2]) * rq * dc_ex2(a_r - b.z);
+                        v[j + 3] = __uint_as_float(cb[j + 3]) * rq * dc_ex2(a_r - b.w);
+                    }
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) v[j] = j > mine ? 0.0f : v[j];
 #pragma unroll
                     for (int j = 0; j < 8; ++j) dc_split(v[2 * j], v[2 * j + 1], m[j], m[8 + j]);
                 }
@@ -680,8 +721,10 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(p_full);
+            __syncwarp();
+            if (c + 1 < n_chunks) load_inverse(c + 1);
+            output(c, dc_ex2(a_r) * rq);
         }
-        output(n_chunks - 1, prev);
         if (blockIdx.z == 0) ssm_save_conv_of_head<0>(a, sp, h, threadIdx.x - 320, 256);
     }
 

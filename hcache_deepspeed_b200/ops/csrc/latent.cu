@@ -4,8 +4,9 @@
 //                   the way to the dense q rows, RMS-norms the latent, rotates the shared key part and writes both into the
 //                   token's page row [latent | key part | zeros]. Statistics and angles in fp32.
 //   head_matmul   : out[t][h][n] = sum_k x[t][h][k] w[h][k][n], fp32 accumulation: takes queries to the latent space (and copies
-//                   their rotated part behind), and mean latents to values. One CTA = 16 tokens of one head; weights are read once
-//                   per CTA, x is broadcast from shared memory.
+//                   their rotated part behind), and mean latents to values. One CTA = 16 tokens of one head
+//                   and 64 columns; x is broadcast from shared memory.
+#include <type_traits>
 #include "hds_host.cuh"
 #include "hds_ptx.cuh"
 #include "../../../include/hds_b200.h"
@@ -103,21 +104,42 @@ latent_append_kernel(const void* __restrict__ proj, int64_t ld, void* __restrict
     }
 }
 
-constexpr int kHmTok = 16, kHmThreads = 256;
+constexpr int kHmTok = 16, kHmCols = 64, kHmSlices = 8, kHmBatch = 16, kHmThreads = kHmCols / 2 * kHmSlices;
 
-// Thread = two neighbouring columns of a 2 * cols-column block and one of `slices` equal parts of K; partial sums of the slices
-// meet in shared memory. Tokens of sequences that bring more than `limit` tokens are left alone.
+// Warp = one of kHmSlices equal parts of K, lane = two neighbouring columns of the CTA's 64; the parts' sums meet in shared memory.
+// A thread has kHmBatch weights in flight, the first ones before the kernel in front has finished. Tokens of sequences that bring
+// more than `limit` tokens are left alone.
 template <int DT>
 __global__ void __launch_bounds__(kHmThreads)
 head_matmul_kernel(const void* __restrict__ x, int64_t ld_x, int in_width, const void* __restrict__ w, void* __restrict__ out,
                    int64_t ld_out, int out_width, const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ spans, int limit,
-                   int T, int K, int N, int copy, int slices) {
+                   int T, int K, int N, int copy) {
     extern __shared__ float sm[];
     float* x_s = sm;                      // [K][kHmTok]
-    float* part = sm + K * kHmTok;        // [slices][kHmTok][2 * cols]
+    float* part = sm + K * kHmTok;        // [kHmSlices][kHmTok][kHmCols]
     __shared__ int live[kHmTok];
+    const int t0 = blockIdx.x * kHmTok, h = blockIdx.y, n0 = blockIdx.z * kHmCols, tid = threadIdx.x;
+    const int slice = tid >> 5, n = n0 + 2 * (tid & 31);
+    const int per = (K + kHmSlices - 1) / kHmSlices, k0 = min(K, slice * per), k1 = min(K, k0 + per);
+    const bool two = n + 1 < N, pair = two && (N & 1) == 0;
+    const int64_t wh = static_cast<int64_t>(h) * K * N + n;
+    using W = typename std::conditional<DT == 2, float2, uint32_t>::type;
+    W q[kHmBatch];
+    auto load = [&](int k) {
+#pragma unroll
+        for (int i = 0; i < kHmBatch; ++i) {
+            const bool ok = k + i < k1 && n < N;
+            const int64_t wi = wh + static_cast<int64_t>(k + i) * N;
+            if constexpr (DT == 2) {
+                q[i] = make_float2(ok ? reinterpret_cast<const float*>(w)[wi] : 0.0f, ok && two ? reinterpret_cast<const float*>(w)[wi + 1] : 0.0f);
+            } else {
+                const uint16_t* p = reinterpret_cast<const uint16_t*>(w) + wi;
+                q[i] = !ok ? 0u : pair ? *reinterpret_cast<const uint32_t*>(p) : (p[0] | (two ? static_cast<uint32_t>(p[1]) << 16 : 0u));
+            }
+        }
+    };
+    load(k0);
     pdl_enter();
-    const int t0 = blockIdx.x * kHmTok, h = blockIdx.y, tid = threadIdx.x;
     int any = 0;
     if (tid < kHmTok) {
         live[tid] = t0 + tid < T && spans[4 * tok_seq[t0 + tid] + 1] <= limit;
@@ -129,61 +151,45 @@ head_matmul_kernel(const void* __restrict__ x, int64_t ld_x, int in_width, const
         x_s[k * kHmTok + i] = live[i] ? load_any<DT>(x, static_cast<int64_t>(t0 + i) * ld_x + static_cast<int64_t>(h) * in_width + k) : 0.0f;
     }
     __syncthreads();
-    const int cols = kHmThreads / slices, slice = tid / cols, ct = tid % cols;
-    const int per = (K + slices - 1) / slices, k0 = slice * per, k1 = min(K, k0 + per);
-    const int64_t wh = static_cast<int64_t>(h) * K * N;
-    for (int n0 = 0; n0 < N; n0 += 2 * cols) {
-        const int n = n0 + 2 * ct;
-        const bool two = n + 1 < N, pair = two && (N & 1) == 0;
-        float a[kHmTok][2];
+    float a[kHmTok][2];
 #pragma unroll
-        for (int i = 0; i < kHmTok; ++i) a[i][0] = a[i][1] = 0.0f;
-        if (n < N) {
-#pragma unroll 4
-            for (int k = k0; k < k1; ++k) {
-                float w0, w1;
-                const int64_t wi = wh + static_cast<int64_t>(k) * N + n;
-                if (DT != 2 && pair) {
-                    const uint32_t q = *reinterpret_cast<const uint32_t*>(reinterpret_cast<const char*>(w) + wi * 2);
-                    w0 = unpack_lo<DT == 0>(q);
-                    w1 = unpack_hi<DT == 0>(q);
-                } else {
-                    w0 = load_any<DT>(w, wi);
-                    w1 = two ? load_any<DT>(w, wi + 1) : 0.0f;
-                }
-                const float4* xk = reinterpret_cast<const float4*>(x_s + k * kHmTok);
+    for (int i = 0; i < kHmTok; ++i) a[i][0] = a[i][1] = 0.0f;
+    for (int k = k0; k < k1; k += kHmBatch) {
+        if (k > k0) load(k);
 #pragma unroll
-                for (int i = 0; i < kHmTok / 4; ++i) {
-                    const float4 v = xk[i];
-                    a[4 * i + 0][0] = fmaf(v.x, w0, a[4 * i + 0][0]); a[4 * i + 0][1] = fmaf(v.x, w1, a[4 * i + 0][1]);
-                    a[4 * i + 1][0] = fmaf(v.y, w0, a[4 * i + 1][0]); a[4 * i + 1][1] = fmaf(v.y, w1, a[4 * i + 1][1]);
-                    a[4 * i + 2][0] = fmaf(v.z, w0, a[4 * i + 2][0]); a[4 * i + 2][1] = fmaf(v.z, w1, a[4 * i + 2][1]);
-                    a[4 * i + 3][0] = fmaf(v.w, w0, a[4 * i + 3][0]); a[4 * i + 3][1] = fmaf(v.w, w1, a[4 * i + 3][1]);
-                }
+        for (int j = 0; j < kHmBatch; ++j) {
+            if (k + j >= k1) break;
+            float w0, w1;
+            if constexpr (DT == 2) {
+                w0 = q[j].x;
+                w1 = q[j].y;
+            } else {
+                w0 = unpack_lo<DT == 0>(q[j]);
+                w1 = unpack_hi<DT == 0>(q[j]);
             }
-        }
-        if (slices > 1) {
-            __syncthreads();
+            const float4* xk = reinterpret_cast<const float4*>(x_s + (k + j) * kHmTok);
 #pragma unroll
-            for (int i = 0; i < kHmTok; ++i)
-                *reinterpret_cast<float2*>(part + (static_cast<int64_t>(slice) * kHmTok + i) * 2 * cols + 2 * ct) = make_float2(a[i][0], a[i][1]);
-            __syncthreads();
-            for (int e = tid; e < kHmTok * 2 * cols; e += kHmThreads) {
-                const int i = e / (2 * cols), c = e % (2 * cols);
-                float s = 0.0f;
-                for (int z = 0; z < slices; ++z) s += part[(static_cast<int64_t>(z) * kHmTok + i) * 2 * cols + c];
-                if (live[i] && n0 + c < N) put<DT>(out, static_cast<int64_t>(t0 + i) * ld_out + static_cast<int64_t>(h) * out_width + n0 + c, s);
+            for (int i = 0; i < kHmTok / 4; ++i) {
+                const float4 v = xk[i];
+                a[4 * i + 0][0] = fmaf(v.x, w0, a[4 * i + 0][0]); a[4 * i + 0][1] = fmaf(v.x, w1, a[4 * i + 0][1]);
+                a[4 * i + 1][0] = fmaf(v.y, w0, a[4 * i + 1][0]); a[4 * i + 1][1] = fmaf(v.y, w1, a[4 * i + 1][1]);
+                a[4 * i + 2][0] = fmaf(v.z, w0, a[4 * i + 2][0]); a[4 * i + 2][1] = fmaf(v.z, w1, a[4 * i + 2][1]);
+                a[4 * i + 3][0] = fmaf(v.w, w0, a[4 * i + 3][0]); a[4 * i + 3][1] = fmaf(v.w, w1, a[4 * i + 3][1]);
             }
-        } else if (n < N) {
-#pragma unroll
-            for (int i = 0; i < kHmTok; ++i)
-                if (live[i]) {
-                    const int64_t o = static_cast<int64_t>(t0 + i) * ld_out + static_cast<int64_t>(h) * out_width + n;
-                    put<DT>(out, o, a[i][0]);
-                    if (two) put<DT>(out, o + 1, a[i][1]);
-                }
         }
     }
+#pragma unroll
+    for (int i = 0; i < kHmTok; ++i)
+        *reinterpret_cast<float2*>(part + (slice * kHmTok + i) * kHmCols + 2 * (tid & 31)) = make_float2(a[i][0], a[i][1]);
+    __syncthreads();
+    for (int e = tid; e < kHmTok * kHmCols; e += kHmThreads) {
+        const int i = e / kHmCols, c = e % kHmCols;
+        float s = 0.0f;
+#pragma unroll
+        for (int z = 0; z < kHmSlices; ++z) s += part[(z * kHmTok + i) * kHmCols + c];
+        if (live[i] && n0 + c < N) put<DT>(out, static_cast<int64_t>(t0 + i) * ld_out + static_cast<int64_t>(h) * out_width + n0 + c, s);
+    }
+    if (blockIdx.z != 0) return;
     // behind the product: `copy` input values that follow the first K, then zeros
     const int rest = out_width - N;
     for (int e = tid; e < kHmTok * rest; e += kHmThreads) {
@@ -223,11 +229,9 @@ extern "C" int hds_head_matmul(const void* x, int64_t ld_x, int in_width, const 
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_head_matmul: dtype 0 bf16 / 1 fp16 / 2 fp32");
     HDS_REQUIRE(K >= 1 && N >= 1 && N + copy <= out_width && K + copy <= in_width, "hds_head_matmul: the product fits its rows");
     if (T == 0) return HDS_OK;
-    int slices = 1;       // parts of K: as many as leave at least N columns to the threads
-    while (slices < 8 && kHmThreads / (2 * slices) * 2 >= N && K / (2 * slices) >= 16) slices *= 2;
-    const size_t smem = static_cast<size_t>(K) * kHmTok * 4 + (slices > 1 ? static_cast<size_t>(2) * kHmThreads * kHmTok * 4 : 0);
-    HDS_REQUIRE(smem <= 220 * 1024, "hds_head_matmul: inner size up to 3000");
-    const dim3 grid((T + kHmTok - 1) / kHmTok, heads), block(kHmThreads);
+    const size_t smem = (static_cast<size_t>(K) * kHmTok + kHmSlices * kHmTok * kHmCols) * 4;
+    HDS_REQUIRE(smem <= 220 * 1024, "hds_head_matmul: inner size up to 2900");
+    const dim3 grid((T + kHmTok - 1) / kHmTok, heads, (N + kHmCols - 1) / kHmCols), block(kHmThreads);
     cudaStream_t s = static_cast<cudaStream_t>(stream);
 #define HDS_HM(DT)                                                                                                             \
     do {                                                                                                                       \
@@ -235,7 +239,7 @@ extern "C" int hds_head_matmul(const void* x, int64_t ld_x, int in_width, const 
             HDS_CHECK_CUDA(cudaFuncSetAttribute(head_matmul_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize,            \
                                                 static_cast<int>(smem)));                                                      \
         HDS_CHECK_CUDA(launch_kernel(head_matmul_kernel<DT>, grid, block, smem, s, x, ld_x, in_width, w, out, ld_out, out_width, \
-                                     tok_seq, spans, limit, T, K, N, copy, slices));                                           \
+                                     tok_seq, spans, limit, T, K, N, copy));                                                   \
     } while (0)
     if (dtype == 0) HDS_HM(0);
     else if (dtype == 1) HDS_HM(1);
