@@ -28,11 +28,12 @@ namespace hds {
 
 constexpr int kDcTok = 128, kDcPanel = kDcTok * 128, kDcP = 64;
 constexpr int kDcThreads = 576, kPrepThreads = 256, kPrepPitch = 132;
-constexpr int kInvRow = 512;                                    // bytes of a row of the inverse: 128 leading terms, 128 rests
-constexpr int64_t kInvBytes = static_cast<int64_t>(kDcTok) * kInvRow;
+// the inverse in memory: 16 pieces of leading terms and 16 of rests, a piece = 8 neighbouring values of every row
+constexpr int kInvPiece = kDcTok * 16;
+constexpr int64_t kInvBytes = 32 * kInvPiece;
 
 struct DeltaWs {
-    uint8_t* inv;      // [chunks][heads][128][512 B]
+    uint8_t* inv;      // [chunks][heads][32 pieces][128 rows][16 B]
     float* a;          // [T][heads]: running log2 decay inside the token's chunk
     float* beta;       // [T][heads]
     float* rk;         // [T][groups]: 1 / |k|
@@ -235,7 +236,7 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
             const float* R = step == 0 ? X11 : T1;
             const int rp = step == 0 ? kPrepPitch : 36;
 #pragma unroll 2
-            for (int k = 0; k < 32; k += 4) {
+            for (int k = 0; k < (step == 0 ? 32 : i0 + 4); k += 4) {      // (X22 is zero above its diagonal)
                 float2 w[4];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) w[e] = *reinterpret_cast<const float2*>(R + (k + e) * rp + j0);
@@ -266,7 +267,7 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
             const float* R = step == 0 ? A : tmp;
             const int rp = step == 0 ? kPrepPitch : 68;
 #pragma unroll 2
-            for (int k = 0; k < 64; k += 4) {
+            for (int k = 0; k < (step == 0 ? 64 : i0 + 4); k += 4) {
                 float4 w[4];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) w[e] = *reinterpret_cast<const float4*>(R + (k + e) * rp + j0);
@@ -295,15 +296,15 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
     // ---- two-term copy ----
     uint8_t* dst = ws.inv + (static_cast<int64_t>(blockIdx.x) * H + h) * kInvBytes;
     for (int e = tid; e < kDcTok * 16; e += kPrepThreads) {      // 8 values at a time
-        const int i = e >> 4, c = (e & 15) * 8;
+        const int i = e & (kDcTok - 1), p = e / kDcTok, c = p * 8;
         const float4 x = *reinterpret_cast<const float4*>(A + i * kPrepPitch + c), y = *reinterpret_cast<const float4*>(A + i * kPrepPitch + c + 4);
         uint4 hi, lo;
         dc_split(x.x, x.y, hi.x, lo.x);
         dc_split(x.z, x.w, hi.y, lo.y);
         dc_split(y.x, y.y, hi.z, lo.z);
         dc_split(y.z, y.w, hi.w, lo.w);
-        *reinterpret_cast<uint4*>(dst + i * kInvRow + c * 2) = hi;
-        *reinterpret_cast<uint4*>(dst + i * kInvRow + 256 + c * 2) = lo;
+        *reinterpret_cast<uint4*>(dst + p * kInvPiece + i * 16) = hi;
+        *reinterpret_cast<uint4*>(dst + (16 + p) * kInvPiece + i * 16) = lo;
     }
     tc_fence_before();
     __syncthreads();
@@ -647,12 +648,12 @@ delta_chunk_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, 
         };
         // the inverse of chunk c: my row's 64 columns, 16 at a time
         auto load_inverse = [&](int c) {
-            const uint8_t* src = ws.inv + ((static_cast<int64_t>(first + c) * H + h) * kDcTok + r) * kInvRow + half * 128;
+            const uint8_t* src = ws.inv + (static_cast<int64_t>(first + c) * H + h) * kInvBytes + half * 8 * kInvPiece + r * 16;
             uint4 hi[8], lo[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
-                hi[i] = __ldcg(reinterpret_cast<const uint4*>(src + i * 16));      // (not through L1: the launch before wrote it)
-                lo[i] = __ldcg(reinterpret_cast<const uint4*>(src + 256 + i * 16));
+                hi[i] = __ldcg(reinterpret_cast<const uint4*>(src + i * kInvPiece));      // (not through L1: the launch before wrote it)
+                lo[i] = __ldcg(reinterpret_cast<const uint4*>(src + (16 + i) * kInvPiece));
             }
             if (c > 0) mbar_wait(u_done, (c - 1) & 1);
             tc_fence_after();
