@@ -173,7 +173,7 @@ def bench_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
         tables = torch.randperm(B * T // page, device=dev).to(torch.int32).view(B, T // page).contiguous()
         lat, mean = rnd(B, nh * width, scale=0.1), rnd(B, nh * rank)
         items = torch.tensor([[i, i, 1, T - 1] for i in range(B)], dtype=torch.int32, device=dev)
-        sp = latent_splits(B, 1, nh, rank, T, window)
+        sp = latent_splits(B, 1, nh, rank, width, T, window)
         keys = T if not window else min(T, window)
         report(f"latent attention decode {B}x{T} window {window}", "paged_attention_latent", lambda: K.paged_attention_latent(
             lat, mean, pages, tables, items, B, 1, nh, rank, page, sp, 0.09, lws, window), B * keys * (rank + rot) * 2)

@@ -121,7 +121,8 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
     rows, cols = [], []
     if c is not None:
         D, R = c.head_width, c.kv_rank
-        rows.append(_head_rows(p["latent.q"], c.heads, c.dim + c.rot_dim, D))
+        sign = 0.0 if c.scale == 0 else -1.0 if c.scale < 0 else 1.0      # (as for ordinary attention below)
+        rows.append(_head_rows(p["latent.q"] * sign, c.heads, c.dim + c.rot_dim, D))
         if c.kv_from is None:
             rows.append(p["latent.dkv"])
             lw.latent_norm = f32(p["latent.norm"])
@@ -330,7 +331,8 @@ class HybridTransformer(RaggedTransformer):
                 key.append((a, pick_prefill_splits(batch.n_items_large, n_q, windowed_len(batch.max_kv_len_large, window, keep))))
         if self.dtype != torch.float32:
             for c in {(c.heads, c.kv_rank, c.page_width, c.window) for c in (l.mixer.latent for l in self.spec.layers) if c is not None}:
-                key.append((c, latent_launches(batch, *c, batch.n_items_large > 0)))
+                if self.ops.k.latent_attention_supported(c[1], c[2]):
+                    key.append((c, latent_launches(batch, *c, batch.n_items_large > 0)))
         return tuple(key)
 
     def _alloc_buffers(self) -> None:

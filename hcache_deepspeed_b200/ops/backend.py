@@ -162,7 +162,7 @@ class CpuOps:
         mean = torch.zeros(q3.shape[0], c.heads, c.kv_rank)
         for items in (batch.items_small(), batch.items_large()):
             if items.shape[0]:
-                ref.paged_latent_attention(lat, pages, batch.block_tables(), items, c.kv_rank, c.scale, c.window, out=mean)
+                ref.paged_latent_attention(lat, pages, batch.block_tables(), items, c.kv_rank, abs(c.scale) or 1.0, c.window, out=mean)
         v = torch.einsum("thr,hrv->thv", mean, lw.w_uv.float())
         out.copy_(torch.nn.functional.pad(v, (0, c.head_width - c.vdim)).reshape(out.shape))
 
@@ -420,7 +420,7 @@ class CudaOps:
         """Decode steps and short portions in the latent space; prompts on K / V pages projected from the cached rows they see (as
         long as those fit the scratch pages)."""
         k, T, bs, D = self.k, q.shape[0], batch.block_size, c.head_width
-        plan = None
+        plan, scale = None, abs(c.scale) or 1.0
         if lw.w_kv is not None and batch.n_items_large and T > batch.current_sequences:
             plan = batch.visible_pages(c.window, bufs.blocks)
         generic = q.dtype == torch.float32 or not k.latent_attention_supported(c.kv_rank, c.page_width)
@@ -430,11 +430,11 @@ class CudaOps:
             k.head_matmul(q, lw.w_uk, lat, batch.tokens_to_seq(), batch.spans(), limit, in_width=D, out_width=c.page_width, copy=c.rot_dim)
             if generic:
                 k.paged_attention_generic(lat, mean, pages, batch.block_tables(), batch.tokens_to_seq(), batch.tok_pos(), c.heads, 1,
-                                          c.page_width, bs, c.scale, window=c.window, value_dim=c.kv_rank, spans=batch.spans(), limit=limit)
+                                          c.page_width, bs, scale, window=c.window, value_dim=c.kv_rank, spans=batch.spans(), limit=limit)
             else:
                 for items, n, tokens, splits in latent_launches(batch, c.heads, c.kv_rank, c.page_width, c.window, plan is None):
                     k.paged_attention_latent(lat, mean, pages, batch.block_tables(), batch.items_small() if items == "small" else
-                                             batch.items_large(), n, tokens, c.heads, c.kv_rank, bs, splits, c.scale, bufs.workspace, c.window)
+                                             batch.items_large(), n, tokens, c.heads, c.kv_rank, bs, splits, scale, bufs.workspace, c.window)
             k.head_matmul(mean, lw.w_uv, out, batch.tokens_to_seq(), batch.spans(), limit, in_width=c.kv_rank, out_width=D, copy=0)
         if plan is not None:
             ids, tables = plan
@@ -445,7 +445,7 @@ class CudaOps:
                               bufs.slots[:n * bs], None, c.heads, D, bs)
             n_items = batch.n_items_large
             splits = pick_prefill_splits(n_items, c.heads, windowed_len(batch.max_kv_len_large, c.window))
-            k.paged_attention_prefill(q, out, kv, tables, batch.items_large(), n_items, c.heads, c.heads, D, bs, c.scale, n_splits=splits,
+            k.paged_attention_prefill(q, out, kv, tables, batch.items_large(), n_items, c.heads, c.heads, D, bs, scale, n_splits=splits,
                                       workspace=ws_large if splits > 1 else None, window=c.window)
 
     # ---- gated delta rule -----------------------------------------------------------------------------
@@ -532,15 +532,16 @@ def latent_launches(batch, heads: int, rank: int, width: int, window: int, with_
         out.append(("large", batch.n_items_large, batch.max_large_item_tokens, batch.max_kv_len_large))
     launches = []
     for kind, n, tokens, kv_len in out:
-        launches.append((kind, n, tokens, latent_splits(n, tokens, heads, rank, kv_len, window)))
+        launches.append((kind, n, tokens, latent_splits(n, tokens, heads, rank, width, kv_len, window)))
     return tuple(launches)
 
 
-def latent_splits(n_items: int, item_tokens: int, heads: int, rank: int, max_kv_len: int, window: int) -> int:
-    """KV splits of the latent attention kernel: one wave of CTAs at most, at least 2 tiles of 64 keys each."""
-    ctas = n_items * -(-item_tokens * heads // 128) * -(-rank // 256)
-    tiles = max(1, -(-windowed_len(max_kv_len, window) // 64))
-    return int(max(1, min(MAX_PREFILL_SPLITS, N_SM // ctas, tiles // 2)))
+def latent_splits(n_items: int, item_tokens: int, heads: int, rank: int, width: int, max_kv_len: int, window: int) -> int:
+    """KV splits of the latent attention kernel: one wave of CTAs at most, at least one tile each."""
+    from .kernels import latent_attention_ctas
+    ctas, tile = latent_attention_ctas(item_tokens, heads, rank, width)
+    tiles = max(1, -(-(min(max_kv_len, window) if window else max_kv_len) // tile))
+    return int(max(1, min(MAX_PREFILL_SPLITS, N_SM // (n_items * ctas), tiles)))
 
 
 class LatentBuffers:

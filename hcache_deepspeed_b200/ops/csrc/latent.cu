@@ -146,6 +146,21 @@ head_matmul_kernel(const void* __restrict__ x, int64_t ld_x, int in_width, const
         any = live[tid];
     }
     if (!__syncthreads_or(any)) return;
+    if (DT != 2 && (K & 7) == 0 && (in_width & 7) == 0 && (ld_x & 7) == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0) {
+        const int kv = K / 8;
+#pragma unroll 4
+        for (int e = tid; e < kv * kHmTok; e += kHmThreads) {      // lanes: tokens, so that the transposed stores spread over the banks
+            const int i = e % kHmTok, k = e / kHmTok * 8;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (live[i]) v = *reinterpret_cast<const uint4*>(reinterpret_cast<const char*>(x) +
+                                                            (static_cast<int64_t>(t0 + i) * ld_x + static_cast<int64_t>(h) * in_width + k) * 2);
+            float* d = x_s + k * kHmTok + i;
+            d[0 * kHmTok] = unpack_lo<DT == 0>(v.x); d[1 * kHmTok] = unpack_hi<DT == 0>(v.x);
+            d[2 * kHmTok] = unpack_lo<DT == 0>(v.y); d[3 * kHmTok] = unpack_hi<DT == 0>(v.y);
+            d[4 * kHmTok] = unpack_lo<DT == 0>(v.z); d[5 * kHmTok] = unpack_hi<DT == 0>(v.z);
+            d[6 * kHmTok] = unpack_lo<DT == 0>(v.w); d[7 * kHmTok] = unpack_hi<DT == 0>(v.w);
+        }
+    } else
     for (int e = tid; e < K * kHmTok; e += kHmThreads) {
         const int i = e / K, k = e % K;
         x_s[k * kHmTok + i] = live[i] ? load_any<DT>(x, static_cast<int64_t>(t0 + i) * ld_x + static_cast<int64_t>(h) * in_width + k) : 0.0f;

@@ -757,6 +757,13 @@ def latent_attention_supported(rank: int, page_width: int) -> bool:
     return bool(native.cuda_lib().hds_paged_attention_latent_supported(rank, page_width))
 
 
+def latent_attention_ctas(item_tokens: int, heads: int, rank: int, page_width: int) -> Tuple[int, int]:
+    """(CTAs per item and split, keys per tile) of :func:`paged_attention_latent`."""
+    tile = ctypes.c_int(0)
+    n = native.cuda_lib().hds_paged_attention_latent_ctas(item_tokens, heads, rank, page_width, ctypes.byref(tile))
+    return int(n), tile.value
+
+
 def latent_attention_workspace_bytes() -> int:
     return int(native.cuda_lib().hds_paged_attention_latent_workspace_bytes())
 
@@ -765,7 +772,7 @@ def paged_attention_latent(q: torch.Tensor, out: torch.Tensor, pages: torch.Tens
                            n_items: int, item_tokens: int, heads: int, rank: int, block_size: int, n_splits: int, scale: float,
                            workspace: torch.Tensor, window: int = 0) -> None:
     """tcgen05 attention in the latent space: ``q`` [T, heads * width], ``pages`` [blocks, 1, 1, bs, width], ``out`` [T, heads * rank].
-    One CTA = 128 (token, head) rows of an item (of at most ``item_tokens`` tokens) and up to 256 of the latent's values."""
+    items: at most ``item_tokens`` tokens each."""
     rc = native.cuda_lib().hds_paged_attention_latent(_p(q), _p(out), _p(pages), pages.shape[0], _p(block_tables), block_tables.stride(0),
                                                       _p(items), n_items, item_tokens, q.shape[0], heads, rank, pages.shape[4], block_size,
                                                       scale, window, n_splits, _p(workspace), workspace.numel(), _dt(q), _stream())

@@ -62,6 +62,7 @@ def _declare_cuda(lib: ctypes.CDLL, partial: bool = False) -> None:
         "hds_head_matmul": [P, L, I, P, P, L, I, P, P, I, I, I, I, I, I, I, P],
         "hds_paged_attention_latent": [P, P, P, L, P, I, P, I, I, I, I, I, I, I, F, I, I, P, L, I, P],
         "hds_paged_attention_latent_supported": [I, I],
+        "hds_paged_attention_latent_ctas": [I, I, I, I, P],
         "hds_host_buffer_alloc": [L, I, I, P],
         "hds_host_buffer_device_ptr": [P, P],
         "hds_host_buffer_free": [P],

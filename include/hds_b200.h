@@ -444,6 +444,8 @@ int hds_paged_attention_latent(const void* q, void* out, const void* pages, int6
                                int page_width, int block_size, float scale, int window, int n_splits, void* workspace,
                                int64_t workspace_bytes, int dtype, void* stream);
 int hds_paged_attention_latent_supported(int rank, int page_width);
+/* CTAs per item and split of that launch, and keys per tile. */
+int hds_paged_attention_latent_ctas(int item_tokens, int heads, int rank, int page_width, int* tile_keys);
 /* Scratch for n_splits > 1. Zero it once; the kernel leaves its tickets zeroed. */
 int64_t hds_paged_attention_latent_workspace_bytes(void);
 
