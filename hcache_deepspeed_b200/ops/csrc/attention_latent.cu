@@ -346,6 +346,19 @@ __host__ __device__ constexpr size_t fw_fixed_smem(int panels) {
     return 1024 + static_cast<size_t>(panels) * N * 128 /*Q*/ + 2 * N * 128 /*P*/ + (2 * 4 * N + 4 * N + 4 * N + 2 * N) * 4 + (8 + 2 * kFwMaxBars) * 8 + 16;
 }
 
+// key tiles that a row tile sees, and how they are split
+struct FewTiles {
+    int first, live, per, splits;
+};
+__device__ __forceinline__ FewTiles fw_tiles(const LatentArgs& a, int pos_lo, int pos_hi) {
+    FewTiles t;
+    t.first = a.window > 0 ? max(0, pos_lo - a.window + 1) / kFwKeys : 0;
+    t.live = pos_hi / kFwKeys + 1 - t.first;
+    t.per = (t.live + a.n_splits - 1) / a.n_splits;
+    t.splits = (t.live + t.per - 1) / t.per;
+    return t;
+}
+
 // v[0..31] of every lane -> lane n holds op over the lanes of v[n]
 template <typename Op>
 __device__ __forceinline__ float fw_transpose_reduce(float (&v)[32], uint32_t lane, Op op) {
@@ -382,7 +395,6 @@ paged_attn_latent_few_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
     uint64_t* bars = reinterpret_cast<uint64_t*>(inv_s + N);
     uint64_t *q_full = bars, *s_full = bars + 1 /*[2]*/, *p_full = bars + 3, *o_done = bars + 4, *k_full = bars + 8, *k_empty = k_full + kFwMaxBars;
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 5);
-    int* last_s = reinterpret_cast<int*>(bars + 6);
 
     const uint32_t warp = warp_id(), lane = lane_id();
     pdl_enter();
@@ -391,12 +403,10 @@ paged_attn_latent_few_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
     const int row0 = row_tile * N, n_rows = min(N, item.n_q * a.heads - row0);
     if (n_rows <= 0) return;
     const int pos_lo = item.pos0 + row0 / a.heads, pos_hi = item.pos0 + (row0 + n_rows - 1) / a.heads;
-    const int t_first = a.window > 0 ? max(0, pos_lo - a.window + 1) / kFwKeys : 0;
-    const int live = pos_hi / kFwKeys + 1 - t_first;
-    const int tps = (live + a.n_splits - 1) / a.n_splits, eff_splits = (live + tps - 1) / tps;
-    const int split = blockIdx.z;
+    const FewTiles ft = fw_tiles(a, pos_lo, pos_hi);
+    const int split = blockIdx.z, eff_splits = ft.splits;
     if (split >= eff_splits) return;
-    const int t0 = t_first + split * tps, n_tiles = min(tps, live - split * tps);
+    const int t0 = ft.first + split * ft.per, n_tiles = min(ft.per, ft.live - split * ft.per);
 
     if (warp == 0 && lane == 0) {
         prefetch_tmap(&tmap_q);
@@ -616,36 +626,6 @@ paged_attn_latent_few_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
             }
         }
         tc_fence_before();
-        if (eff_splits > 1) {
-            __threadfence();
-            group_sync();
-            if (tid == 0) {
-                *last_s = atomicAdd(&a.tickets[unit], 1) == eff_splits - 1;
-                if (*last_s) a.tickets[unit] = 0;
-            }
-            group_sync();
-            if (*last_s) {
-                __threadfence();
-                for (int n = 0; n < n_rows; ++n) {
-                    float mx = -INFINITY, sum = 0.0f;
-                    for (int s = 0; s < eff_splits; ++s) mx = fmaxf(mx, __ldcg(a.ws_ml + ((unit * a.n_splits + s) * kLaRows + n) * 2));
-                    float o[8] = {};      // latents of up to 1024 values
-                    for (int s = 0; s < eff_splits; ++s) {
-                        const int64_t sl = unit * a.n_splits + s;
-                        const float2 ml = __ldcg(reinterpret_cast<const float2*>(a.ws_ml + (sl * kLaRows + n) * 2));
-                        const float w = ml.x == -INFINITY ? 0.0f : la_ex2(ml.x - mx);
-                        sum = fmaf(w, ml.y, sum);
-#pragma unroll
-                        for (int b = 0; b < 8; ++b)
-                            if (b < f.v_blocks) o[b] = fmaf(w, __ldcg(a.ws_o + (sl * N + n) * width + b * 128 + tid), o[b]);
-                    }
-#pragma unroll
-                    for (int b = 0; b < 8; ++b)
-                        if (b < f.v_blocks && b * 128 + tid < a.rank)
-                            store_scalar<kBf16>(a.out, out0 + static_cast<int64_t>(n) * a.rank + b * 128 + tid, o[b] / sum);
-                }
-            }
-        }
     }
     tc_fence_before();
     __syncthreads();
@@ -653,6 +633,37 @@ paged_attn_latent_few_kernel(const __grid_constant__ CUtensorMap tmap_q, const _
         tc_fence_after();
         tmem_dealloc<TMEM_COLS>(tmem);
     }
+}
+
+// Splits of a row meet: CTA = (row tile, row), thread = value of each 128-value block.
+template <bool kBf16>
+__global__ void __launch_bounds__(128) latent_merge_kernel(const FewArgs f, int tile_rows) {
+    const LatentArgs& a = f.l;
+    pdl_enter();
+    const int unit = blockIdx.x, n = blockIdx.y;
+    const hds_attn_item item = a.items[unit / a.row_tiles];
+    const int row0 = unit % a.row_tiles * tile_rows, n_rows = min(tile_rows, item.n_q * a.heads - row0);
+    if (n >= n_rows) return;
+    const FewTiles ft = fw_tiles(a, item.pos0 + row0 / a.heads, item.pos0 + (row0 + n_rows - 1) / a.heads);
+    if (ft.splits == 1) return;       // written by the attention kernel itself
+    const int width = f.v_blocks * 128;
+    float mx = -INFINITY, sum = 0.0f;
+    for (int s = 0; s < ft.splits; ++s) mx = fmaxf(mx, a.ws_ml[((static_cast<int64_t>(unit) * a.n_splits + s) * kLaRows + n) * 2]);
+    float o[5] = {};
+#pragma unroll 4
+    for (int s = 0; s < ft.splits; ++s) {
+        const int64_t slot = static_cast<int64_t>(unit) * a.n_splits + s;
+        const float2 ml = *reinterpret_cast<const float2*>(a.ws_ml + (slot * kLaRows + n) * 2);
+        const float w = ml.x == -INFINITY ? 0.0f : la_ex2(ml.x - mx);
+        sum = fmaf(w, ml.y, sum);
+#pragma unroll
+        for (int b = 0; b < 5; ++b)
+            if (b < f.v_blocks) o[b] = fmaf(w, a.ws_o[(slot * tile_rows + n) * width + b * 128 + threadIdx.x], o[b]);
+    }
+    const int64_t out0 = (static_cast<int64_t>(item.q_row0) * a.heads + row0 + n) * a.rank;
+#pragma unroll
+    for (int b = 0; b < 5; ++b)
+        if (b < f.v_blocks && b * 128 + static_cast<int>(threadIdx.x) < a.rank) store_scalar<kBf16>(a.out, out0 + b * 128 + threadIdx.x, o[b] / sum);
 }
 
 struct FewPlan {
@@ -693,6 +704,7 @@ static int launch_few(const CUtensorMap& tq, const CUtensorMap& tk, const FewArg
         configured[dev & 63] = true;
     }
     HDS_CHECK_CUDA(launch_kernel(paged_attn_latent_few_kernel<kBf16, N>, grid, dim3(kLaThreads), smem, s, tq, tk, f));
+    if (f.l.n_splits > 1) HDS_CHECK_CUDA(launch_kernel(latent_merge_kernel<kBf16>, dim3(grid.x, N), dim3(128), 0, s, f, N));
     return HDS_OK;
 }
 
