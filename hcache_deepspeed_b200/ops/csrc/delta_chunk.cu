@@ -56,14 +56,15 @@ __device__ __forceinline__ uint4* dc_cell(uint8_t* panel, int r, int c) {   // 1
 __device__ __forceinline__ int dc_chunks(const SsmSpan& s) { return s.n > 1 ? (s.n + kDcTok - 1) / kDcTok : 0; }
 
 // ---- per chunk and head -------------------------------------------------------------------------------------------------
-constexpr size_t kPrepSmem = 2 * kDcPanel + static_cast<size_t>(kDcTok) * kPrepPitch * 4 + 3 * kDcTok * 4 + 64;
+constexpr size_t kPrepSmem = static_cast<size_t>(kDcTok) * kPrepPitch * 4 /*k panels, then A*/ + 3 * kDcTok * 4 + 64;
+static_assert(2 * kDcPanel <= kDcTok * kPrepPitch * 4, "A replaces the key panels");
 
-__global__ void __launch_bounds__(kPrepThreads)
+__global__ void __launch_bounds__(kPrepThreads, 3)
 delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, const DeltaWs ws) {
     extern __shared__ __align__(1024) uint8_t smem[];
-    uint8_t* k_sm = smem;                                           // two panels; later the products' intermediate [64][68]
-    float* tmp = reinterpret_cast<float*>(smem);
-    float* A = reinterpret_cast<float*>(smem + 2 * kDcPanel);       // [128][kPrepPitch]: A, then the inverse in place
+    uint8_t* k_sm = smem;                                           // two panels, until K K^T is done
+    float* A = reinterpret_cast<float*>(smem);                      // [128][kPrepPitch]: A, then the inverse in place
+    float* tmp = A + 64;                                            // products' intermediates: the quarter above the diagonal
     float* a_s = A + kDcTok * kPrepPitch;
     float* b_s = a_s + kDcTok;
     float* r_s = b_s + kDcTok;
@@ -168,19 +169,16 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
     const int quad = warp & 3, half = warp >> 2, r = quad * 32 + lane;
     mbar_wait(done, 0);
     tc_fence_after();
-    uint32_t s[64];
-    {
-        const uint32_t t = tmem + (static_cast<uint32_t>(quad * 32) << 16) + half * 64;
-        tmem_ld_32x32(t, *reinterpret_cast<uint32_t(*)[32]>(&s[0]));
-        tmem_ld_32x32(t + 32, *reinterpret_cast<uint32_t(*)[32]>(&s[32]));
+    const uint32_t t_row = tmem + (static_cast<uint32_t>(quad * 32) << 16);
+    if (quad / 2 == half) {      // (uniform in a warp)
+        uint32_t s[32];
+        tmem_ld_32x32(t_row + quad * 32, s);
         tmem_ld_wait();
-    }
-    {
         float kk = 0.0f;
 #pragma unroll
-        for (int j = 0; j < 64; ++j)
-            if (half * 64 + j == r) kk = __uint_as_float(s[j]);
-        if (r / 64 == half) {
+        for (int j = 0; j < 32; ++j)
+            if (j == static_cast<int>(lane)) kk = __uint_as_float(s[j]);
+        {
             const float rk = 1.0f / sqrtf(kk + kUnitEps);
             r_s[r] = rk;
             if (r < n && h % (H / a.groups) == 0) ws.rk[static_cast<int64_t>(row + r) * a.groups + g] = rk;
@@ -189,15 +187,27 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
     __syncthreads();
     {
         const float f = r < n ? b_s[r] * r_s[r] : 0.0f, ar = a_s[r];
+#pragma unroll 1
+        for (int j0 = half * 64; j0 < half * 64 + 64; j0 += 16) {
+            float* row_out = A + r * kPrepPitch + j0;
+            if (j0 > quad * 32 + 31) {      // all above the diagonal
 #pragma unroll
-        for (int j = 0; j < 64; j += 4) {
-            float v[4];
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int c = half * 64 + j + e;
-                v[e] = c < r ? f * r_s[c] * dc_ex2(ar - a_s[c]) * __uint_as_float(s[j + e]) : 0.0f;
+                for (int j = 0; j < 16; j += 4) *reinterpret_cast<float4*>(row_out + j) = make_float4(0.f, 0.f, 0.f, 0.f);
+                continue;
             }
-            *reinterpret_cast<float4*>(A + r * kPrepPitch + half * 64 + j) = make_float4(v[0], v[1], v[2], v[3]);
+            uint32_t s[16];
+            tmem_ld_32x16(t_row + j0, s);
+            tmem_ld_wait();
+#pragma unroll
+            for (int j = 0; j < 16; j += 4) {
+                const float4 rk = *reinterpret_cast<const float4*>(r_s + j0 + j), aj = *reinterpret_cast<const float4*>(a_s + j0 + j);
+                float4 v;
+                v.x = j0 + j + 0 < r ? f * rk.x * dc_ex2(ar - aj.x) * __uint_as_float(s[j + 0]) : 0.0f;
+                v.y = j0 + j + 1 < r ? f * rk.y * dc_ex2(ar - aj.y) * __uint_as_float(s[j + 1]) : 0.0f;
+                v.z = j0 + j + 2 < r ? f * rk.z * dc_ex2(ar - aj.z) * __uint_as_float(s[j + 2]) : 0.0f;
+                v.w = j0 + j + 3 < r ? f * rk.w * dc_ex2(ar - aj.w) * __uint_as_float(s[j + 3]) : 0.0f;
+                *reinterpret_cast<float4*>(row_out + j) = v;
+            }
         }
     }
     __syncthreads();
@@ -229,17 +239,16 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
         float* X11 = A + b * 64 * kPrepPitch + b * 64;
         float* X21 = X11 + 32 * kPrepPitch;
         float* X22 = X21 + 32;
-        float* T1 = tmp + b * 32 * 36;
+        float* T1 = tmp + b * 32;
         for (int step = 0; step < 2; ++step) {
             float acc[4][2] = {};
             const float* L = step == 0 ? X21 : X22;
             const float* R = step == 0 ? X11 : T1;
-            const int rp = step == 0 ? kPrepPitch : 36;
 #pragma unroll 2
             for (int k = 0; k < (step == 0 ? 32 : i0 + 4); k += 4) {      // (X22 is zero above its diagonal)
                 float2 w[4];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) w[e] = *reinterpret_cast<const float2*>(R + (k + e) * rp + j0);
+                for (int e = 0; e < 4; ++e) w[e] = *reinterpret_cast<const float2*>(R + (k + e) * kPrepPitch + j0);
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     const float4 l = *reinterpret_cast<const float4*>(L + (i0 + i) * kPrepPitch + k);
@@ -252,7 +261,7 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
             if (step == 1) __syncthreads();
 #pragma unroll
             for (int i = 0; i < 4; ++i)
-                *reinterpret_cast<float2*>((step == 0 ? T1 + (i0 + i) * 36 : X21 + (i0 + i) * kPrepPitch) + j0) =
+                *reinterpret_cast<float2*>((step == 0 ? T1 : X21) + (i0 + i) * kPrepPitch + j0) =
                     step == 0 ? make_float2(acc[i][0], acc[i][1]) : make_float2(-acc[i][0], -acc[i][1]);
             __syncthreads();
         }
@@ -265,12 +274,11 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
             float acc[4][4] = {};
             const float* L = step == 0 ? X21 : X22;
             const float* R = step == 0 ? A : tmp;
-            const int rp = step == 0 ? kPrepPitch : 68;
 #pragma unroll 2
             for (int k = 0; k < (step == 0 ? 64 : i0 + 4); k += 4) {
                 float4 w[4];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) w[e] = *reinterpret_cast<const float4*>(R + (k + e) * rp + j0);
+                for (int e = 0; e < 4; ++e) w[e] = *reinterpret_cast<const float4*>(R + (k + e) * kPrepPitch + j0);
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     const float4 l4 = *reinterpret_cast<const float4*>(L + (i0 + i) * kPrepPitch + k);
@@ -287,7 +295,7 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
             if (step == 1) __syncthreads();
 #pragma unroll
             for (int i = 0; i < 4; ++i)
-                *reinterpret_cast<float4*>((step == 0 ? tmp + (i0 + i) * 68 : X21 + (i0 + i) * kPrepPitch) + j0) =
+                *reinterpret_cast<float4*>((step == 0 ? tmp : X21) + (i0 + i) * kPrepPitch + j0) =
                     step == 0 ? make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3])
                               : make_float4(-acc[i][0], -acc[i][1], -acc[i][2], -acc[i][3]);
             __syncthreads();
@@ -298,11 +306,13 @@ delta_prep_kernel(const __grid_constant__ CUtensorMap tmap_u, const SsmArgs a, c
     for (int e = tid; e < kDcTok * 16; e += kPrepThreads) {      // 8 values at a time
         const int i = e & (kDcTok - 1), p = e / kDcTok, c = p * 8;
         const float4 x = *reinterpret_cast<const float4*>(A + i * kPrepPitch + c), y = *reinterpret_cast<const float4*>(A + i * kPrepPitch + c + 4);
-        uint4 hi, lo;
-        dc_split(x.x, x.y, hi.x, lo.x);
-        dc_split(x.z, x.w, hi.y, lo.y);
-        dc_split(y.x, y.y, hi.z, lo.z);
-        dc_split(y.z, y.w, hi.w, lo.w);
+        uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
+        if (i >= 64 || c < 64) {      // (the other quarter is zero and held intermediates)
+            dc_split(x.x, x.y, hi.x, lo.x);
+            dc_split(x.z, x.w, hi.y, lo.y);
+            dc_split(y.x, y.y, hi.z, lo.z);
+            dc_split(y.z, y.w, hi.w, lo.w);
+        }
         *reinterpret_cast<uint4*>(dst + p * kInvPiece + i * 16) = hi;
         *reinterpret_cast<uint4*>(dst + (16 + p) * kInvPiece + i * 16) = lo;
     }
