@@ -110,7 +110,8 @@ def check_mixed_batches(cfg, dtype, device, tol=None):
         for k, _ in step:
             if at[k] == len(toks[k]):
                 eng.flush(uid[k])
-    assert at == lengths and int(eng.free_blocks[0]) == 512 // 64 and eng.state_manager.recurrent_states.free_slots == 3
+    states = eng.state_manager.recurrent_states
+    assert at == lengths and int(eng.free_blocks[0]) == 512 // 64 and (states is None or states.free_slots == 3)
 
 
 def check_long_decode(cfg, dtype, device, n=330, tol=None):
