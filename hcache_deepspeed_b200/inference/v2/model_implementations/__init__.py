@@ -178,8 +178,12 @@ class DedelornPolicy(InferenceV2Policy):
     """Layers of a gated delta rule or of latent attention, each beside its feed-forward on one norm."""
 
 
+class LotelixPolicy(InferenceV2Policy):
+    """Layers of a minGRU, of windowed attention with sinks, or of sigmoid attention beside gated linear attention."""
+
+
 MODEL_TYPE_TO_POLICY = {
-    "nipolorn": NipolornPolicy, "dedelorn": DedelornPolicy,
+    "nipolorn": NipolornPolicy, "dedelorn": DedelornPolicy, "lotelix": LotelixPolicy,
     "gpt2": GPT2Policy, "gptj": GPTJPolicy, "gpt_neox": GPTNeoXPolicy, "bloom": BloomPolicy, "gpt_neo": GPTNeoPolicy,
     "llama": Llama2Policy, "opt": OPTPolicy, "mistral": MistralPolicy, "mixtral": MixtralPolicy, "falcon": FalconPolicy,
     "phi": PhiPolicy, "phi3": Phi3Policy, "qwen": QwenPolicy, "qwen2": Qwen2Policy, "qwen2_moe": Qwen2MoePolicy,

@@ -9,7 +9,7 @@ from __future__ import annotations
 from enum import Enum
 from typing import List, Optional, Tuple
 
-from pydantic import PositiveInt, model_validator
+from pydantic import NonNegativeInt, PositiveInt, model_validator
 
 from ....config import DeepSpeedConfigModel, DtypeEnum
 
@@ -38,12 +38,12 @@ class KVCacheConfig(DeepSpeedConfigModel):
 
 class RecurrentLayerConfig(DeepSpeedConfigModel):
     """Per-sequence state of one recurrent layer: a ``heads`` x ``vdim`` x ``state`` matrix stack and the latest ``taps``
-    inputs of ``conv_dim`` convolution channels."""
+    inputs of ``conv_dim`` convolution channels (0: no convolution)."""
     heads: PositiveInt
     vdim: PositiveInt
     state: PositiveInt
-    conv_dim: PositiveInt
-    taps: PositiveInt
+    conv_dim: NonNegativeInt
+    taps: NonNegativeInt
 
 
 class AllocationMode(Enum):

@@ -9,6 +9,7 @@ spec on the sm_100a kernels.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field, replace
 from typing import Any, Callable, Dict, List, Optional
 
@@ -17,9 +18,43 @@ from typing import Any, Callable, Dict, List, Optional
 # layer descriptions of stacks whose layers are not all alike (ArchSpec.layers)
 # ---------------------------------------------------------------------------------------------------
 @dataclass
+class RotationSpec:
+    """Rotation of the first ``dims`` values of every query and key head by position * base^(-2i / dims): value i is paired with
+    i + dims / 2, or, ``adjacent``, 2i with 2i + 1. ``slow_factor`` > 0: pairs whose wavelength exceeds ``original / slow_low``
+    positions turn slower by that factor, those below ``original / slow_high`` as they are, the ones between by a linear mixture."""
+    dims: int
+    base: float
+    adjacent: bool = False
+    slow_factor: float = 0.0
+    slow_low: float = 1.0
+    slow_high: float = 1.0
+    original: float = 0.0
+
+    def frequencies(self) -> List[float]:
+        out = []
+        for i in range(self.dims // 2):
+            f = float(self.base)**(-2.0 * i / self.dims)
+            if self.slow_factor:
+                wave = 2.0 * math.pi / f
+                if wave > self.original / self.slow_low:
+                    f /= self.slow_factor
+                elif wave >= self.original / self.slow_high:
+                    s = (self.original / wave - self.slow_low) / (self.slow_high - self.slow_low)
+                    f = (1.0 - s) * f / self.slow_factor + s * f
+            out.append(f)
+        return out
+
+
+@dataclass
 class AttentionSpec:
-    """Grouped-query softmax attention. ``window`` > 0: a query at position p sees the keys (p - window, p] and, always,
-    the first ``keep_first`` positions of its sequence. Positions enter through the mask only (no rotation)."""
+    """Grouped-query attention. ``window`` > 0: a query at position p sees the keys (p - window, p] and, always, the first
+    ``keep_first`` positions of its sequence. Without ``rot`` positions enter through the mask only.
+
+    ``weights`` = "softmax"; with ``sink`` its denominator holds one more term per head, exp of a learned number. "sigmoid": a
+    visible key weighs sigmoid(score + a learned number per head), not normalized over keys. ``bias``: q, k, v and the output
+    projection have biases. ``qk_norm``: all of q, and all of k, normed at once before the rotation. ``gate``: the heads are
+    multiplied by the sigmoid of one more projection of the layer's input. ``v_first``: values are mixed, by a learned share, with
+    the values that this earlier layer caches of the same token (the same heads and sizes)."""
     heads: int
     kv_heads: int
     dim: int                 # query / key size of a head
@@ -27,6 +62,13 @@ class AttentionSpec:
     scale: float
     window: int = 0
     keep_first: int = 0
+    rot: Optional[RotationSpec] = None
+    weights: str = "softmax"
+    sink: bool = False
+    bias: bool = False
+    qk_norm: bool = False
+    gate: bool = False
+    v_first: Optional[int] = None
 
     @property
     def page_dim(self) -> int:
@@ -127,20 +169,78 @@ class DeltaSpec:
 
 
 @dataclass
+class LinearAttentionSpec:
+    """Gated linear attention: heads with a ``dim`` x ``vdim`` recurrent state each, whose rows (key channels) fade by a decay of
+    their own, sigmoid(z)^(1 / tau), z a projection through ``rank`` values (0: as the checkpoint has it) plus a bias. A norm per
+    head and a gate behind."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float = 1.0
+    rank: int = 0
+
+    conv = conv_dim = 0
+
+    @property
+    def state(self) -> int:
+        return self.dim
+
+    @property
+    def keys(self) -> int:
+        """Columns of all heads' queries (keys, decays), padded to 16-byte rows."""
+        return -(-self.heads * self.dim // 8) * 8
+
+    @property
+    def inner(self) -> int:
+        return -(-self.heads * self.vdim // 8) * 8
+
+
+@dataclass
+class GRUSpec:
+    """minGRU: ``width`` independent values, S <- (1 - z) S + z c, gate z and candidate c projections of the current token only;
+    an output gate behind."""
+    width: int
+
+    heads = state = 1
+    conv = conv_dim = 0
+
+    @property
+    def vdim(self) -> int:
+        return self.inner
+
+    @property
+    def inner(self) -> int:
+        return -(-self.width // 8) * 8
+
+    @property
+    def in_dim(self) -> int:
+        """Rows of the input projection: z | candidate input | output gate."""
+        return 3 * self.inner
+
+
+@dataclass
 class MixerSpec:
     """Token mixer of a layer: attention, a state-space mixer, or both side by side on the same input, each with a weight; or
-    latent attention; or a gated delta rule."""
+    latent attention; or a gated delta rule; or a minGRU; or attention beside gated linear attention, each with an output
+    projection and a norm of its own, of which the result is the mean."""
     attn: Optional[AttentionSpec] = None
     ssm: Optional[StateSpaceSpec] = None
     attn_weight: float = 1.0
     ssm_weight: float = 1.0
     latent: Optional[LatentAttentionSpec] = None
     delta: Optional[DeltaSpec] = None
+    linear: Optional[LinearAttentionSpec] = None
+    gru: Optional[GRUSpec] = None
 
     @property
     def recurrent(self):
         """The part with per-sequence state, if any."""
-        return self.ssm if self.ssm is not None else self.delta
+        return next((m for m in (self.ssm, self.delta, self.linear, self.gru) if m is not None), None)
+
+    @property
+    def normed_mean(self) -> bool:
+        """Two outputs, each normed, instead of one?"""
+        return self.attn is not None and self.linear is not None
 
 
 @dataclass
@@ -148,7 +248,8 @@ class FeedForwardSpec:
     """``experts`` = 0: dense gated MLP of size ``ff``. Otherwise a mixture of experts of size ``ff`` each, ``top`` per token.
     ``routing`` = "table": a table gives every token id its experts, all with weight 1 / top. ``routing`` = "softmax": the
     largest softmax scores of a router, each plus the expert's correction, choose; the scores themselves times
-    ``router_scale`` weigh. ``shared_ff`` > 0: one more expert that sees every token. ``gated`` = False: down(act(up x)).
+    ``router_scale`` weigh. ``routing`` = "sigmoid": the largest sigmoid scores choose and weigh; the weight multiplies what the
+    expert reads, not what it returns. ``shared_ff`` > 0: one more expert that sees every token. ``gated`` = False: down(act(up x)).
     ``act`` = "swiglu_clamped" clamps gate and up to ``limit`` (see ops.reference)."""
     ff: int
     act: str = "silu"
@@ -159,6 +260,11 @@ class FeedForwardSpec:
     shared_ff: int = 0
     gated: bool = True
     router_scale: float = 1.0
+
+    @property
+    def weighs_inputs(self) -> bool:
+        """Does an expert's weight multiply its input instead of its output?"""
+        return self.routing == "sigmoid"
 
 
 @dataclass
@@ -217,6 +323,8 @@ class ArchSpec:
     layers: Optional[List[LayerSpec]] = None
     post_norms: bool = False  # ``layers`` stacks: every sublayer's OUTPUT is normed as well
     norm_weight_offset: float = 0.0  # ``layers`` stacks: stored norm weights are differences from this
+    norm_groups: int = 1  # ``layers`` stacks: the layers' norms and the final one norm equal consecutive parts of a row, each by itself
+    embed_scale: float = 1.0  # ``layers`` stacks: factor of the token embeddings
     extras: Dict[str, Any] = field(default_factory=dict)
 
     # ---- derived -------------------------------------------------------------------------------
@@ -256,7 +364,8 @@ class ArchSpec:
     @property
     def pages_hold_context(self) -> bool:
         """Do the K / V pages of a sequence alone bring every layer's context back?"""
-        return self.layers is None or (not self.has_recurrent_state and all(l.mixer.latent is None for l in self.layers))
+        return self.layers is None or (not self.has_recurrent_state and all(
+            l.mixer.latent is None and (l.mixer.attn is None or l.mixer.attn.v_first is None) for l in self.layers))
 
     def window_of(self, layer: int) -> int:
         return int(self.layer_windows[layer]) if self.layer_windows is not None else int(self.sliding_window)
@@ -273,6 +382,8 @@ class ArchSpec:
                 total += h * (1 + self.post_norms)
                 if a is not None:
                     total += h * (a.heads * (a.dim + a.vdim) + a.kv_heads * (a.dim + a.vdim))
+                    total += h * a.heads * a.vdim * a.gate + a.heads * (a.sink + (a.weights == "sigmoid")) + (a.v_first is not None)
+                    total += (a.heads + a.kv_heads) * a.dim * a.qk_norm + ((a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim + h) * a.bias
                 if m is not None:
                     total += h * (m.in_dim + m.inner) + m.conv_dim * (m.conv + 1) + 3 * m.heads + m.inner
                 if c is not None:
@@ -280,11 +391,16 @@ class ArchSpec:
                     total += (h * (c.kv_rank + c.rot_dim) + c.kv_rank) if c.kv_from is None else 0
                 if d is not None:
                     total += h * (d.in_dim + d.inner) + d.conv_dim * d.conv + 2 * d.heads + d.vdim
+                g, r = l.mixer.linear, l.mixer.gru
+                if g is not None:
+                    total += g.heads * (h * (2 * g.dim + 3 * g.vdim) + g.dim * (g.rank + 1)) + h * g.rank + g.vdim + 2 * h * l.mixer.normed_mean
+                if r is not None:
+                    total += r.width * (4 * h + 2)
                 if f is not None:
                     total += 0 if self.parallel_residual else h * (1 + self.post_norms)
                     total += (3 if f.gated else 2) * h * (f.ff * max(1, f.experts) + f.shared_ff)
                     if f.experts:
-                        total += self.vocab * f.top if f.routing == "table" else (h + 1) * f.experts
+                        total += self.vocab * f.top if f.routing == "table" else (h + (f.routing == "softmax")) * f.experts
             return total
         attn = h * (self.q_dim + 2 * self.kv_dim) + self.q_dim * h
         if self.is_moe:
@@ -634,6 +750,61 @@ def _dedelorn(cfg) -> ArchSpec:
 
 #: Dedelorn: one norm per layer read by both sublayers, and a norm on the embeddings
 DEDELORN_NORMS = dict(parallel_residual=True, embed_norm=True)
+
+
+@register_arch("lotelix")
+def _lotelix(cfg) -> ArchSpec:
+    """Lotelix: layers of a minGRU, of windowed attention (rotated, with sinks, an output gate and values mixed with the first such
+    layer's), or of sigmoid attention beside gated linear attention, in any order; mixtures of experts with a sigmoid router."""
+
+    def ff(m) -> Optional[FeedForwardSpec]:
+        if m is None:
+            return None
+        if m["kind"] != "moe":
+            raise ValueError(f"lotelix: unknown feed-forward kind {m['kind']!r}")
+        return FeedForwardSpec(ff=int(m["expert"]["ff"]), act="relu2", experts=int(m["router"]["experts"]), top=int(m["router"]["top"]),
+                               routing="sigmoid", gated=False)
+
+    def rotation(r, adjacent) -> RotationSpec:
+        sc = r.get("scaling")
+        slow = {} if sc is None else dict(slow_factor=float(sc["factor"]), slow_low=float(sc["low"]), slow_high=float(sc["high"]),
+                                          original=float(sc["original"]))
+        return RotationSpec(dims=int(r["dims"]), base=float(r["base"]), adjacent=adjacent, **slow)
+
+    def attention(a, adjacent, **kw) -> AttentionSpec:
+        spec = AttentionSpec(heads=int(a["heads"]), kv_heads=int(a["kv_heads"]), dim=int(a["dim"]), vdim=int(a["vdim"]), scale=float(a["scale"]),
+                             window=int((a.get("mask") or {}).get("size") or 0), rot=rotation(a["rot"], adjacent), **kw)
+        if spec.rot.dims > spec.dim or spec.rot.dims % 2 or spec.heads % spec.kv_heads:
+            raise ValueError("lotelix: rot.dims must be even and at most dim, heads a multiple of kv_heads")
+        return spec
+
+    layers: List[LayerSpec] = []
+    first = None            # the layer whose values the later ones mix in
+    for i, lc in enumerate(_get(cfg, "layers")):
+        mx = lc["mixer"]
+        if lc["type"] == "mingru":
+            mixer = MixerSpec(gru=GRUSpec(width=int(mx["width"])))
+        elif lc["type"] == "attention":
+            a = attention(mx, False, sink=True, gate=True, v_first=first if mx.get("v_mix") else None)
+            if a.v_first is not None:
+                b = layers[first].mixer.attn
+                if (b.kv_heads, b.vdim) != (a.kv_heads, a.vdim):
+                    raise ValueError(f"lotelix: layer {i} cannot mix in the values of layer {first}")
+            elif mx.get("v_mix"):
+                first = i
+            mixer = MixerSpec(attn=a)
+        elif lc["type"] == "parallel":
+            r = mx["right"]
+            mixer = MixerSpec(attn=attention(mx["left"], True, weights="sigmoid", bias=True, qk_norm=True),
+                              linear=LinearAttentionSpec(heads=int(r["heads"]), dim=int(r["dim"]), vdim=int(r["vdim"]), tau=float(r["tau"])))
+        else:
+            raise ValueError(f"lotelix: unknown layer type {lc['type']!r}")
+        layers.append(LayerSpec(mixer=mixer, mlp=ff(lc.get("mlp"))))
+    width, groups = int(_get(cfg, "width")), int(_get(cfg, "norm").get("groups", 1))
+    if width % groups:
+        raise ValueError("lotelix: width must be a multiple of norm.groups")
+    return stack_arch("lotelix", layers, hidden=width, vocab=int(_get(cfg, "vocab")), norm_eps=float(_get(cfg, "norm")["eps"]),
+                      norm_groups=groups, embed_scale=float((_get(cfg, "embedding") or {}).get("scale", 1.0)))
 
 
 def stack_arch(model_type: str, layers: List[LayerSpec], hidden: int, vocab: int, norm_eps: float, **kw) -> ArchSpec:

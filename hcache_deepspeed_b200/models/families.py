@@ -531,3 +531,38 @@ def map_dedelorn(name: str, t: torch.Tensor, spec: ArchSpec) -> List[Piece]:
         if m:
             return [(li, f"moe.experts.{m.group(1)}.{m.group(2)}", t)]
     return []
+
+
+# ---------------------------------------------------------------------------------------------------
+_LOTELIX_GRU = {"z": "gru.z", "z.b": "gru.z_b", "x": "gru.x", "x.b": "gru.x_b", "g": "gru.g", "o": "gru.o"}
+_LOTELIX_ATTENTION = {"q": "attn.q", "k": "attn.k", "v": "attn.v", "o": "attn.o", "g": "attn.g", "sink": "attn.sink", "vmix": "attn.vmix"}
+_LOTELIX_PARALLEL = {"left.q": "attn.q", "left.k": "attn.k", "left.v": "attn.v", "left.o": "attn.o", "left.q.b": "attn.q_b", "left.k.b": "attn.k_b",
+                     "left.v.b": "attn.v_b", "left.o.b": "attn.o_b", "left.q.norm": "attn.q_norm", "left.k.norm": "attn.k_norm",
+                     "left.pb": "attn.pb", "left.out": "attn.out_norm", "right.q": "linear.q", "right.k": "linear.k", "right.v": "linear.v",
+                     "right.g": "linear.g", "right.o": "linear.o", "right.norm": "linear.norm", "right.a1": "linear.a1", "right.a2": "linear.a2",
+                     "right.a2.b": "linear.a2_b", "right.out": "linear.out_norm"}
+
+
+@register_mapper("lotelix")
+def map_lotelix(name: str, t: torch.Tensor, spec: ArchSpec) -> List[Piece]:
+    top = {"embed": "embed", "final.norm": "final_norm.g", "head": "lm_head"}
+    if name in top:
+        return [(None, top[name], t)]
+    m = _STACK_LAYER.match(name)
+    if not m or int(m.group(1)) >= spec.n_layers:
+        return []
+    li, rest = int(m.group(1)), m.group(2)
+    if rest in ("norm1", "norm2"):
+        return [(li, rest + ".g", t)]
+    part, _, leaf = rest.partition(".")
+    if part == "mix":
+        mixer = spec.layers[li].mixer
+        table = _LOTELIX_GRU if mixer.gru is not None else _LOTELIX_PARALLEL if mixer.linear is not None else _LOTELIX_ATTENTION
+        return [(li, table[leaf], t)] if leaf in table else []
+    if part == "mlp":
+        if leaf == "router":
+            return [(li, "moe.router", t)]
+        m = re.match(r"e(\d+)\.(up|down)$", leaf)
+        if m:
+            return [(li, f"moe.experts.{m.group(1)}.{m.group(2)}", t)]
+    return []

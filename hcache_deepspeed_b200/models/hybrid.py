@@ -17,6 +17,13 @@ supplies what such a layer does between them, and how its checkpoint pieces are 
   ordinary attention kernels on those.
 * a gated delta rule's ``w_qkv`` is ``[gate | v | k | q | decay input | step input]``: the columns of a state-space mixer
   (``[z | x | B | C | dt]``) and one more per head.
+* rotated heads: the rows of a head's queries and keys are reordered so that the two values of pair i lie at i and at half the page
+  size + i, whatever pairing the design has; values that are not rotated fill the other places with frequency zero. The
+  kernels then know one pairing, whole heads, and every page size.
+* a minGRU's ``w_qkv`` is ``[gate | candidate | output gate]``; gated linear attention adds ``[q | k | v | gate | decay's first
+  projection]`` behind the attention's columns, each padded to 16-byte rows.
+* two mixers with a norm each: ``w_o`` and ``w_o2`` project their parts of the buffer separately; the norm kernel behind norms both,
+  with halved weights, while adding them to the stream.
 * ``parallel_residual``: mixer and dense feed-forward read the same norm, so ``w_o`` is ``[mixer columns | feed-forward columns]``
   and ONE GEMM projects and adds both.
 
@@ -34,8 +41,9 @@ from ..inference.v2.ragged.manager_configs import KVCacheConfig
 from ..ops.backend import (LatentBuffers, latent_launches, pick_decode_splits, pick_packed_splits, pick_prefill_splits, use_packed_decode,
                            windowed_len)
 from ..ops.kernels import ACT_CODES
-from .arch import ArchSpec, AttentionSpec, DeltaSpec, FeedForwardSpec, LatentAttentionSpec, LayerSpec, MixerSpec, StateSpaceSpec
-from .transformer import RaggedTransformer, ceil_div
+from .arch import (ArchSpec, AttentionSpec, DeltaSpec, FeedForwardSpec, GRUSpec, LatentAttentionSpec, LayerSpec, LinearAttentionSpec, MixerSpec,
+                   StateSpaceSpec)
+from .transformer import ACCUM_MAX_TOKENS, RaggedTransformer, ceil_div
 from .weights import ExpertWeights, LayerWeights, ModelWeights, interleave_gate_up
 
 
@@ -54,7 +62,17 @@ def required_pieces(spec: ArchSpec, l: LayerSpec) -> List[str]:
     if l.mixer.delta is not None:
         req += ["delta." + n for n in ("q", "k", "v", "q_conv", "k_conv", "v_conv", "a", "b", "A_log", "dt_bias", "g", "norm", "o")]
     if l.mixer.attn is not None:
-        req += ["attn.q", "attn.k", "attn.v", "attn.o"]
+        a = l.mixer.attn
+        req += ["attn.q", "attn.k", "attn.v", "attn.o"] + (["attn.g"] if a.gate else []) + (["attn.sink"] if a.sink else [])
+        req += ["attn.pb"] if a.weights == "sigmoid" else []
+        req += (["attn.q_b", "attn.k_b", "attn.v_b", "attn.o_b"] if a.bias else []) + (["attn.q_norm", "attn.k_norm"] if a.qk_norm else [])
+        req += ["attn.vmix"] if a.v_first is not None else []
+    if l.mixer.linear is not None:
+        req += ["linear." + n for n in ("q", "k", "v", "g", "a1", "a2", "a2_b", "norm", "o")]
+    if l.mixer.normed_mean:
+        req += ["attn.out_norm", "linear.out_norm"]
+    if l.mixer.gru is not None:
+        req += ["gru." + n for n in ("z", "z_b", "x", "x_b", "g", "o")]
     if l.mixer.ssm is not None:
         req += ["ssm." + n for n in ("in", "conv", "conv_b", "dt_bias", "A_log", "D", "norm", "o")]
     if l.mlp is not None:
@@ -63,7 +81,7 @@ def required_pieces(spec: ArchSpec, l: LayerSpec) -> List[str]:
         parts = ("gate", "up", "down") if l.mlp.gated else ("up", "down")
         if l.mlp.experts:
             req += [f"moe.experts.{e}.{n}" for e in range(l.mlp.experts) for n in parts]
-            req += ["moe.table"] if l.mlp.routing == "table" else ["moe.router", "moe.correction"]
+            req += {"table": ["moe.table"], "softmax": ["moe.router", "moe.correction"], "sigmoid": ["moe.router"]}[l.mlp.routing]
             if l.mlp.shared_ff:
                 req += ["moe.shared." + n for n in parts]
         else:
@@ -84,10 +102,33 @@ def _head_rows(w: torch.Tensor, heads: int, d: int, page_dim: int) -> torch.Tens
     return _pad(w.reshape(heads, d, -1), 1, page_dim).reshape(heads * page_dim, -1)
 
 
+def rotated_places(a: AttentionSpec) -> torch.Tensor:
+    """Place inside a page row of every value of a query or key head: the values of rotated pair i at i and page_dim / 2 + i."""
+    r, half = a.rot, a.page_dim // 2
+    i = torch.arange(r.dims // 2)
+    place = torch.empty(a.dim, dtype=torch.long)
+    u, v = (2 * i, 2 * i + 1) if r.adjacent else (i, i + r.dims // 2)
+    place[u], place[v] = i, half + i
+    free = [p for p in range(a.page_dim) if p % half >= r.dims // 2]
+    place[r.dims:] = torch.tensor(free[:a.dim - r.dims], dtype=torch.long)
+    return place
+
+
+def _query_rows(w: torch.Tensor, heads: int, a: AttentionSpec) -> torch.Tensor:
+    """Rows (or values) of query or key heads [heads * dim, ...] -> [heads * page_dim, ...], in the kernels' order."""
+    flat = w.reshape(heads, a.dim, -1)
+    if a.rot is None:
+        out = _pad(flat, 1, a.page_dim)
+    else:
+        out = flat.new_zeros(heads, a.page_dim, flat.shape[2])
+        out[:, rotated_places(a).to(flat.device)] = flat
+    return out.reshape((heads * a.page_dim, ) + tuple(w.shape[1:]))
+
+
 def mixer_factors(m: MixerSpec) -> Tuple[float, float]:
     """(factor of the whole mixer output, weight of the state-space part inside it). The attention part has weight 1 inside
     (its columns of the output projection are dropped when its weight is 0)."""
-    if m.latent is not None or m.delta is not None:
+    if m.ssm is None and m.attn is None or m.normed_mean or m.gru is not None:
         return 1.0, 1.0
     if m.attn is not None and m.attn_weight != 0.0:
         return m.attn_weight, m.ssm_weight / m.attn_weight
@@ -117,7 +158,7 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
     lw = LayerWeights(norm1_g=gamma("norm1.g"))
     if spec.post_norms:
         lw.norm1b_g = gamma("norm1b.g")
-    a, m, c, d = l.mixer.attn, l.mixer.ssm, l.mixer.latent, l.mixer.delta
+    a, m, c, d, g, r = l.mixer.attn, l.mixer.ssm, l.mixer.latent, l.mixer.delta, l.mixer.linear, l.mixer.gru
     rows, cols = [], []
     if c is not None:
         D, R = c.head_width, c.kv_rank
@@ -147,8 +188,22 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
         D = a.page_dim
         # a scale of zero or less cannot be the factor of a running maximum: its sign (or zero) moves into the query rows
         sign = 0.0 if a.scale == 0 else -1.0 if a.scale < 0 else 1.0
-        rows += [_head_rows(p["attn.q"] * sign, a.heads, a.dim, D), _head_rows(p["attn.k"], a.kv_heads, a.dim, D),
+        q_sign = 1.0 if a.qk_norm else sign       # (behind a norm it is the norm's weight that carries it)
+        rows += [_query_rows(p["attn.q"] * q_sign, a.heads, a), _query_rows(p["attn.k"], a.kv_heads, a),
                  _head_rows(p["attn.v"], a.kv_heads, a.vdim, D)]
+        if a.gate:
+            rows.append(_head_rows(p["attn.g"], a.heads, a.vdim, D))
+        if a.rot is not None:
+            lw.rot_freq = f32(torch.tensor(a.rot.frequencies() + [0.0] * (D // 2 - a.rot.dims // 2), dtype=torch.float64))
+        if a.qk_norm:
+            lw.q_norm = f32(_query_rows(p["attn.q_norm"].float() * sign, a.heads, a))
+            lw.k_norm = f32(_query_rows(p["attn.k_norm"].float(), a.kv_heads, a))
+        if a.sink:
+            lw.attn_sink = f32(p["attn.sink"])
+        if a.weights == "sigmoid":
+            lw.attn_bias = f32(p["attn.pb"])
+        if a.v_first is not None:
+            lw.v_mix = f32(p["attn.vmix"].reshape(1))
         o = _pad(p["attn.o"].reshape(spec.hidden, a.heads, a.vdim), 2, D).reshape(spec.hidden, a.heads * D)
         cols.append(o if m is None or l.mixer.attn_weight != 0.0 else torch.zeros_like(o))
     if m is not None:
@@ -157,7 +212,28 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
         lw.ssm_conv_w, lw.ssm_conv_b = f32(p["ssm.conv"].t()), f32(p["ssm.conv_b"])
         lw.ssm_dt_bias, lw.ssm_a, lw.ssm_d = f32(p["ssm.dt_bias"]), f32(-torch.exp(p["ssm.A_log"].float())), f32(p["ssm.D"])
         lw.ssm_norm = f32(p["ssm.norm"])
+    if g is not None:
+        rank = p["linear.a1"].shape[0]
+        rows += [_pad(p["linear." + n], 0, w) for n, w in (("q", g.keys), ("k", g.keys), ("v", g.inner), ("g", g.inner), ("a1", pad8(rank)))]
+        lw.w_decay = to(_pad(_pad(p["linear.a2"], 1, pad8(rank)), 0, g.keys))
+        lw.decay_bias = f32(p["linear.a2_b"])
+        lw.ssm_norm = f32(p["linear.norm"].repeat(g.heads))
+        o = _pad(p["linear.o"], 1, g.inner)
+        if l.mixer.normed_mean:
+            lw.w_o2 = to(_pad(o, 0, Hp))
+            lw.mean_g1, lw.mean_g2 = (f32(_pad(p[n].float() * 0.5, 0, Hp)) for n in ("attn.out_norm", "linear.out_norm"))
+        else:
+            cols.append(o)
+    if r is not None:
+        rows += [_pad(p["gru." + n], 0, r.inner) for n in "zxg"]
+        cols.append(_pad(p["gru.o"], 1, r.inner))
+        lw.gru_bias = f32(torch.cat([_pad(p[n], 0, r.inner) for n in ("gru.z_b", "gru.x_b")]))
     lw.w_qkv = to(_pad(torch.cat(rows, dim=0), 1, Hp))
+    if a is not None and a.bias:
+        b = [_query_rows(p["attn.q_b"] * q_sign, a.heads, a), _query_rows(p["attn.k_b"], a.kv_heads, a),
+             _head_rows(p["attn.v_b"][:, None], a.kv_heads, a.vdim, a.page_dim).reshape(-1)]
+        lw.b_qkv = to(_pad(torch.cat(b), 0, lw.w_qkv.shape[0]))
+        lw.b_o = to(_pad(p["attn.o_b"], 0, Hp))
     f = l.mlp
     if f is not None:
         if not spec.parallel_residual:
@@ -171,7 +247,7 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
                 lw.moe_table = p["moe.table"].to(device=device, dtype=torch.int32).contiguous()
             else:
                 lw.w_router = to(_pad(_pad(p["moe.router"], 0, pad8(f.experts)), 1, Hp))
-                lw.router_bias = f32(p["moe.correction"])
+                lw.router_bias = f32(p["moe.correction"]) if f.routing == "softmax" else None
             if f.shared_ff:
                 lw.shared_expert = ff_weights("moe.shared.", f.shared_ff, f.gated)
         else:
@@ -222,7 +298,17 @@ def random_pieces(spec: ArchSpec, l: LayerSpec, gen: torch.Generator, device: to
         return 1.0 - spec.norm_weight_offset + rnd(n, scale=0.05)
 
     p = {"norm1.g": norm_g(), "norm1b.g": norm_g()}
-    a, m, f, c, d = l.mixer.attn, l.mixer.ssm, l.mlp, l.mixer.latent, l.mixer.delta
+    a, m, f, c, d, g, r = l.mixer.attn, l.mixer.ssm, l.mlp, l.mixer.latent, l.mixer.delta, l.mixer.linear, l.mixer.gru
+    if g is not None:
+        kd, vd, rank = g.heads * g.dim, g.heads * g.vdim, g.rank or 16
+        p.update({"linear.q": rnd(kd, H), "linear.k": rnd(kd, H), "linear.v": rnd(vd, H), "linear.g": rnd(vd, H), "linear.a1": rnd(rank, H),
+                  "linear.a2": rnd(kd, rank, scale=0.3), "linear.a2_b": rnd(kd, scale=0.5) + 2.0, "linear.norm": 1.0 + rnd(g.vdim, scale=0.05),
+                  "linear.o": rnd(H, vd)})
+    if l.mixer.normed_mean:
+        p.update({"attn.out_norm": 1.0 + rnd(H, scale=0.05), "linear.out_norm": 1.0 + rnd(H, scale=0.05)})
+    if r is not None:
+        p.update({"gru.z": rnd(r.width, H), "gru.z_b": rnd(r.width, scale=0.5) - 1.0, "gru.x": rnd(r.width, H), "gru.x_b": rnd(r.width),
+                  "gru.g": rnd(r.width, H), "gru.o": rnd(H, r.width)})
     if c is not None:
         p.update({"latent.q": rnd(c.heads * (c.dim + c.rot_dim), H), "latent.uk": rnd(c.heads * c.dim, c.kv_rank),
                   "latent.uv": rnd(c.heads * c.vdim, c.kv_rank), "latent.o": rnd(H, c.heads * c.vdim)})
@@ -237,7 +323,10 @@ def random_pieces(spec: ArchSpec, l: LayerSpec, gen: torch.Generator, device: to
                   "delta.norm": 1.0 + rnd(d.vdim, scale=0.05), "delta.o": rnd(H, d.inner)})
     if a is not None:
         p.update({"attn.q": rnd(a.heads * a.dim, H), "attn.k": rnd(a.kv_heads * a.dim, H), "attn.v": rnd(a.kv_heads * a.vdim, H),
-                  "attn.o": rnd(H, a.heads * a.vdim)})
+                  "attn.o": rnd(H, a.heads * a.vdim), "attn.g": rnd(a.heads * a.vdim, H), "attn.sink": rnd(a.heads, scale=1.0),
+                  "attn.pb": rnd(a.heads, scale=0.5) - 4.0, "attn.vmix": 0.5 + rnd(1, scale=0.1)[0], "attn.q_b": rnd(a.heads * a.dim),
+                  "attn.k_b": rnd(a.kv_heads * a.dim), "attn.v_b": rnd(a.kv_heads * a.vdim), "attn.o_b": rnd(H),
+                  "attn.q_norm": 1.0 + rnd(a.heads * a.dim, scale=0.05), "attn.k_norm": 1.0 + rnd(a.kv_heads * a.dim, scale=0.05)})
     if m is not None:
         p.update({"ssm.in": rnd(m.in_dim, H), "ssm.conv": rnd(m.conv_dim, m.conv, scale=0.3), "ssm.conv_b": rnd(m.conv_dim),
                   "ssm.dt_bias": rnd(m.heads, scale=0.5) - 3.0, "ssm.A_log": rnd(m.heads, scale=0.5), "ssm.D": rnd(m.heads, scale=1.0),
@@ -246,7 +335,9 @@ def random_pieces(spec: ArchSpec, l: LayerSpec, gen: torch.Generator, device: to
         p.update({"norm2.g": norm_g(), "norm2b.g": norm_g()})
 
         def glu(prefix, ff):
-            p.update({prefix + "gate": rnd(ff, H), prefix + "up": rnd(ff, H), prefix + "down": rnd(H, ff)})
+            p.update({prefix + "up": rnd(ff, H), prefix + "down": rnd(H, ff)})
+            if f.gated:
+                p[prefix + "gate"] = rnd(ff, H)
 
         if f.experts:
             for e in range(f.experts):
@@ -277,10 +368,12 @@ def random_stack_weights(spec: ArchSpec, dtype: torch.dtype, device: torch.devic
 # ---------------------------------------------------------------------------------------------------
 class Pending(NamedTuple):
     """A sublayer's output on its way into the residual stream: stream += norm(factor * delta) * weight, or, without a weight,
-    stream += factor * delta."""
+    stream += factor * delta. ``delta2``: a second output, added likewise."""
     delta: torch.Tensor
     factor: float
     weight: Optional[torch.Tensor]
+    delta2: Optional[torch.Tensor] = None
+    weight2: Optional[torch.Tensor] = None
 
 
 class HybridTransformer(RaggedTransformer):
@@ -354,15 +447,19 @@ class HybridTransformer(RaggedTransformer):
         self.latent_buf = buf(s.n_layers, T, Hp) if self.capture_enabled else None
         self.in_buf = buf(T * max(pad8(lw.w_qkv.shape[0]) for lw in self.w.layers))
         self.q_buf = buf(T * max([a.heads * a.page_dim for a in attn] + [c.heads * c.head_width for c in latents] + [8]))
-        self.mix_buf = buf(T * max(lw.w_o.shape[1] for lw in self.w.layers))
+        self.mix_buf = buf(T * max(lw.w_o.shape[1] + (lw.w_o2.shape[1] if lw.w_o2 is not None else 0) for lw in self.w.layers))
         self.conv_buf = buf(T * max((pad8(m.conv_dim) for m in rec), default=8))
         self.dt_buf = buf(T * max((m.heads for m in rec), default=1), dtype=torch.float32)
-        self.scan_buf = buf(T * max((m.inner for m in rec), default=1), dtype=torch.float32)
+        self.scan_buf = buf(T * max((m.inner for m in rec if not isinstance(m, GRUSpec)), default=1), dtype=torch.float32)
+        linear = [m for m in rec if isinstance(m, LinearAttentionSpec)]
+        self.decay_buf = buf(T * max((m.keys for m in linear), default=0))
         self.act_buf = buf(T * max([pad8(f.ff) for f in mlps if not f.experts] + [pad8(f.shared_ff) for f in moes] + [8]))
         self._delta_bufs = [buf(T, Hp, dtype=torch.float32)]
         self._delta_idx = 0
         self.delta32 = self._delta_bufs[0]
         self.delta16 = buf(T, Hp)
+        two = any(l.mixer.normed_mean for l in s.layers)      # a second pending output
+        self.second32, self.second16 = (buf(min(T, ACCUM_MAX_TOKENS), Hp, dtype=torch.float32), buf(T, Hp)) if two else (None, None)
         self.hidden_last = buf(S, Hp)
         self.logits_local = buf(S, self.info.vocab)
         self.logits_full = self.partial16 = self.kv_scratch = None
@@ -370,11 +467,15 @@ class HybridTransformer(RaggedTransformer):
         self._moe_bufs: Dict[Tuple[int, int, int], dict] = {}
         self._latent_bufs: Optional[LatentBuffers] = None
         self._delta_ws: Optional[torch.Tensor] = None
+        self._scan_ws: Optional[torch.Tensor] = None
         if dev.type != "cuda":
             return
         k = self.ops.k
         if latents:
             self._latent_bufs = LatentBuffers(latents, self._state_config, self.kv_block_size, dt, dev)
+        n_ws = max([k.gru_workspace_bytes(T, S, m.inner) for m in rec if isinstance(m, GRUSpec)] +
+                   [k.linear_attention_workspace_bytes(T, S, m.heads, m.vdim, m.dim) for m in linear if dt == torch.bfloat16], default=0)
+        self._scan_ws = torch.empty(n_ws, dtype=torch.uint8, device=dev) if n_ws else None
         if dt != torch.float32:
             n_ws = max((k.delta_workspace_bytes(T, min(S, 64), m.heads, m.kv_heads) for m in rec if isinstance(m, DeltaSpec)), default=0)
             self._delta_ws = torch.empty(n_ws, dtype=torch.uint8, device=dev) if n_ws else None
@@ -408,23 +509,25 @@ class HybridTransformer(RaggedTransformer):
     # ---- layer -------------------------------------------------------------------------------------
     def _embed(self, batch: RaggedBatchWrapper) -> torch.Tensor:
         return self.ops.embed_f32(batch.input_ids(), self.w.embed, self.residual[:batch.current_tokens], gamma=self.w.embed_norm_g,
-                                  cols=self.spec.hidden, eps=self.spec.norm_eps)
+                                  cols=self.spec.hidden, eps=self.spec.norm_eps, scale=self.spec.embed_scale)
 
     def _norm_into(self, resid: torch.Tensor, gamma: torch.Tensor, out: torch.Tensor, pending: Optional[Pending],
                    keep_resid: bool = True) -> torch.Tensor:
-        delta, factor, post = pending if pending is not None else (None, 1.0, None)
+        delta, factor, post, delta2, post2 = pending if pending is not None else (None, 1.0, None, None, None)
         return self.ops.norm_residual(resid, gamma, out, delta=delta, factor=factor, post=post, cols=self.spec.hidden,
-                                      eps=self.spec.norm_eps, store_resid=keep_resid)
+                                      eps=self.spec.norm_eps, store_resid=keep_resid, groups=self.spec.norm_groups, delta2=delta2, post2=post2)
 
     def _layer(self, li: int, resid: torch.Tensor, pending: Optional[Pending], xn: torch.Tensor, batch: RaggedBatchWrapper) -> Pending:
         l, lw, ops, T = self.spec.layers[li], self.w.layers[li], self.ops, batch.current_tokens
         self._norm_into(resid, lw.norm1_g, xn, pending)
         self._kv_ready(li)
-        mix = self._view(self.mix_buf, T, lw.w_o.shape[1])
+        mix = self._view(self.mix_buf, T, lw.w_o.shape[1] + (lw.w_o2.shape[1] if lw.w_o2 is not None else 0))
         if l.mixer.latent is not None:
             n_mix = self._latent_mixer(li, l.mixer.latent, lw, xn, mix, batch)
         elif l.mixer.delta is not None:
             n_mix = self._delta_mixer(li, l.mixer.delta, lw, xn, mix, batch)
+        elif l.mixer.gru is not None:
+            n_mix = self._gru_mixer(li, l.mixer.gru, lw, xn, mix, batch)
         else:
             n_mix = self._attention_and_scan(li, l, lw, xn, mix, batch)
         factor, f = mixer_factors(l.mixer)[0], l.mlp
@@ -434,7 +537,11 @@ class HybridTransformer(RaggedTransformer):
                 return Pending(self._row_parallel(mix, lw.w_o, None, T, force_accum=False), factor, None)
             delta = self._row_parallel(mix, lw.w_o, None, T, force_accum=False)
             return Pending(self._feed_forward(xn, f, lw, T, batch, base=delta), factor, None)
-        pending = Pending(self._row_parallel(mix, lw.w_o, None, T, force_accum=False), factor, lw.norm1b_g)
+        if l.mixer.normed_mean:
+            pending = Pending(self._row_parallel(mix[:, :n_mix], lw.w_o, lw.b_o, T, force_accum=False), factor, lw.mean_g1,
+                              self._second_output(mix[:, n_mix:], lw.w_o2, T), lw.mean_g2)
+        else:
+            pending = Pending(self._row_parallel(mix, lw.w_o, lw.b_o, T, force_accum=False), factor, lw.norm1b_g)
         if f is None:
             return pending
         x2 = self._norm_into(resid, lw.norm2_g, self.xn2[:T], pending)
@@ -442,21 +549,26 @@ class HybridTransformer(RaggedTransformer):
 
     def _attention_and_scan(self, li: int, l: LayerSpec, lw: LayerWeights, xn: torch.Tensor, mix: torch.Tensor,
                             batch: RaggedBatchWrapper) -> int:
-        """Softmax attention and / or a state-space mixer on the same input, side by side in ``mix``; returns their columns."""
+        """Attention and / or a recurrent mixer on the same input, side by side in ``mix``; returns their columns (those of the
+        attention alone where the other has an output projection of its own)."""
         ops, T, kv = self.ops, batch.current_tokens, self._state_manager
-        a, m = l.mixer.attn, l.mixer.ssm
+        a, m, g = l.mixer.attn, l.mixer.ssm, l.mixer.linear
         proj = self._view(self.in_buf, T, pad8(lw.w_qkv.shape[0]))
         n_attn = n_out = 0
         if a is not None:
             D = a.page_dim
             n_attn, n_out = (a.heads + 2 * a.kv_heads) * D, a.heads * D
             q = self._view(self.q_buf, T, n_out)
-            ops.mixer_in_proj(xn, lw.w_qkv, n_attn, proj, q, kv.get_cache(li), batch.tok_pos(), batch.tok_slot(), a.heads, a.kv_heads,
-                              D, kv.kv_block_size, workspace=self.ws_gemm)
+            ops.mixer_in_proj(xn, lw, a, proj, q, kv.get_cache(li), self._first_values(a), batch.tok_pos(), batch.tok_slot(),
+                              kv.kv_block_size, self.spec.norm_eps, workspace=self.ws_gemm)
             ops.attention(q, mix[:, :n_out], kv.get_cache(li), batch, a.heads, a.kv_heads, D, abs(a.scale) or 1.0,
-                          ws_small=self.ws_small, ws_large=self.ws_large, window=a.window, keep_first=a.keep_first)
+                          ws_small=self.ws_small, ws_large=self.ws_large, window=a.window, keep_first=a.keep_first, sink=lw.attn_sink,
+                          sigmoid_bias=lw.attn_bias, gate=proj[:, n_attn:n_attn + n_out] if a.gate else None)
         else:
             ops.gemm(xn, lw.w_qkv, proj[:, :lw.w_qkv.shape[0]], workspace=self.ws_gemm)
+        if g is not None:
+            self._linear(li, g, lw, proj[:, n_attn:], batch.spans(), batch.n_single_token_seqs, mix[:, n_out:n_out + g.inner])
+            return n_out if l.mixer.normed_mean else n_out + g.inner
         if m is None:
             return n_out
         y = self._scan(li, m, lw, proj[:, n_attn:n_attn + m.in_dim], batch.spans(), batch.n_single_token_seqs)
@@ -481,6 +593,36 @@ class HybridTransformer(RaggedTransformer):
         self.ops.gemm(xn, lw.w_qkv, proj, workspace=self.ws_gemm)
         self._scan(li, d, lw, proj, batch.spans(), batch.n_single_token_seqs, mix[:, :d.inner])
         return pad8(d.inner)
+
+    def _first_values(self, a: AttentionSpec) -> Optional[torch.Tensor]:
+        """Pages of the layer whose values this one mixes in: that layer caches its values as they are, so the share of every token,
+        a restored one too, is found there."""
+        return None if a.v_first is None else self._state_manager.get_cache(a.v_first)
+
+    def _second_output(self, x: torch.Tensor, w: torch.Tensor, T: int) -> torch.Tensor:
+        """As ``_row_parallel``, into buffers of its own."""
+        if T <= ACCUM_MAX_TOKENS:
+            self.ops.gemm_accum(x, w, self.second32[:T])
+            return self.second32[:T]
+        return self.ops.gemm(x, w, self.second16[:T])
+
+    def _gru_mixer(self, li: int, r: GRUSpec, lw: LayerWeights, xn: torch.Tensor, mix: torch.Tensor, batch: RaggedBatchWrapper) -> int:
+        proj = self._view(self.in_buf, batch.current_tokens, r.in_dim)
+        self.ops.gemm(xn, lw.w_qkv, proj, workspace=self.ws_gemm)
+        self.ops.gru(proj, lw, r, self._state_manager.recurrent_states.ssm(li), batch.spans(), batch.n_single_token_seqs, mix[:, :r.inner],
+                     self._scan_ws)
+        return r.inner
+
+    def _linear(self, li: int, g: LinearAttentionSpec, lw: LayerWeights, proj: torch.Tensor, spans: torch.Tensor, n_single: int,
+                out: Optional[torch.Tensor]) -> None:
+        """Gated linear attention of the tokens whose projections are ``proj`` = [q | k | v | gate | decay's first projection]; without
+        ``out`` its state alone."""
+        T, nk, nv = proj.shape[0], g.keys, g.inner
+        low = 2 * nk + 2 * nv
+        z = self.ops.gemm(proj[:, low:low + lw.w_decay.shape[1]], lw.w_decay, self._view(self.decay_buf, T, nk), workspace=self.ws_gemm)
+        self.ops.linear_attention(proj[:, :nk], proj[:, nk:2 * nk], proj[:, 2 * nk:2 * nk + nv], proj[:, 2 * nk + nv:low], z, lw, g,
+                                  self._state_manager.recurrent_states.ssm(li), spans, n_single, self._view(self.scan_buf, T, nv), out,
+                                  self.spec.norm_eps, self._scan_ws)
 
     def _scan(self, li: int, m, lw: LayerWeights, proj: torch.Tensor, spans: torch.Tensor, n_single: int,
               out: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -511,6 +653,8 @@ class HybridTransformer(RaggedTransformer):
         bufs = self._moe_bufs.get((f.experts, f.top, f.ff))
         if f.routing == "table":
             ops.table_route(batch.input_ids(), lw, f, bufs)
+        elif f.routing == "sigmoid":
+            ops.sigmoid_route(x, lw, f, bufs)
         else:
             ops.softmax_route(x, lw, f, bufs)
         return ops.routed_experts(x, batch.input_ids(), lw, f, act, base, self.delta32[:T], bufs)
@@ -520,6 +664,8 @@ class HybridTransformer(RaggedTransformer):
 
     def _drop_pending(self, pending: Optional[Pending], T: int) -> None:
         self.delta32[:T].zero_()
+        if self.second32 is not None:
+            self.second32[:T].zero_()
 
     # ---- restore from saved hidden states ------------------------------------------------------------
     def _restore_layer(self, li: int, latents: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, spans: torch.Tensor,
@@ -537,9 +683,20 @@ class HybridTransformer(RaggedTransformer):
         if a is not None:
             n_q = a.heads * a.page_dim
             n_attn = n_q + 2 * a.kv_heads * a.page_dim
-            ops.restore_kv_proj(latents, lw.w_qkv[n_q:n_attn], None, kv.get_cache(li), pos, slot, None, a.kv_heads, a.page_dim,
-                                a.page_dim, kv.kv_block_size, scratch=proj[:, n_q:n_attn])
-        if m is not None:
+            if a.rot is not None or a.qk_norm or a.v_first is not None:
+                part = proj[:, n_q:n_attn]
+                ops.gemm(latents, lw.w_qkv[n_q:n_attn], part, bias=None if lw.b_qkv is None else lw.b_qkv[n_q:n_attn], workspace=self.ws_gemm)
+                ops.attention_append(part, lw, a, None, kv.get_cache(li), self._first_values(a), pos, slot, kv.kv_block_size, self.spec.norm_eps)
+            else:
+                ops.restore_kv_proj(latents, lw.w_qkv[n_q:n_attn], None, kv.get_cache(li), pos, slot, None, a.kv_heads, a.page_dim,
+                                    a.page_dim, kv.kv_block_size, scratch=proj[:, n_q:n_attn])
+        if isinstance(m, GRUSpec):
+            ops.gemm(latents, lw.w_qkv, proj, workspace=self.ws_gemm)
+            ops.gru(proj, lw, m, kv.recurrent_states.ssm(li), spans, n_single, None, self._scan_ws)
+        elif isinstance(m, LinearAttentionSpec):
+            ops.gemm(latents, lw.w_qkv[n_attn:], proj[:, n_attn:], workspace=self.ws_gemm)
+            self._linear(li, m, lw, proj[:, n_attn:], spans, n_single, None)
+        elif m is not None:
             part = proj[:, n_attn:n_attn + m.in_dim]
             ops.gemm(latents, lw.w_qkv[n_attn:], part, workspace=self.ws_gemm)
             self._scan(li, m, lw, part, spans, n_single)

@@ -76,6 +76,20 @@ class LayerWeights:
     w_uv: Optional[torch.Tensor] = None           # [heads, kv_rank, vdim]: takes a head's mean latent to its value
     w_kv: Optional[torch.Tensor] = None           # [2 * heads * head_width, page_width]: cached rows -> K / V pages (16-bit models)
     router_bias: Optional[torch.Tensor] = None    # fp32 [experts]: added to the scores that choose, not to the weights
+    # attention options (fp32)
+    attn_sink: Optional[torch.Tensor] = None      # [heads]: one more score in the softmax's denominator
+    attn_bias: Optional[torch.Tensor] = None      # [heads]: added to the scores of sigmoid attention
+    q_norm: Optional[torch.Tensor] = None         # [heads * page_dim] and
+    k_norm: Optional[torch.Tensor] = None         # [kv_heads * page_dim], zeros in the padding
+    v_mix: Optional[torch.Tensor] = None          # [1]: share of the first mixing layer's values
+    # two mixers with an output projection and a norm each: the second projection, half the norms' weights (fp32)
+    w_o2: Optional[torch.Tensor] = None
+    mean_g1: Optional[torch.Tensor] = None
+    mean_g2: Optional[torch.Tensor] = None
+    # gated linear attention: [keys, rank] and fp32 bias of the decays (its norm: ssm_norm); minGRU: fp32 [2 * inner] biases of z | x
+    w_decay: Optional[torch.Tensor] = None
+    decay_bias: Optional[torch.Tensor] = None
+    gru_bias: Optional[torch.Tensor] = None
 
     def stack_experts(self) -> None:
         """Store the experts as consecutive slices of one tensor per matrix, the operands of the grouped GEMM."""

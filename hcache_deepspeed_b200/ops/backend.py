@@ -87,33 +87,40 @@ class CpuOps:
         ref.kv_append(kv_layer, k, v, tok_slot)
 
     def attention(self, q, out, kv_layer, batch, n_q, n_kv, d, scale, ws_small=None, ws_large=None, alibi=None, window=0,
-                  keep_first=0):
+                  keep_first=0, sink=None, sigmoid_bias=None, gate=None):
         T = q.shape[0]
         q3, o3 = q.view(T, n_q, d), out.view(T, n_q, d)
         for items in (batch.items_small(), batch.items_large()):
             if items.shape[0]:
                 ref.paged_attention(q3, kv_layer, batch.block_tables(), items, n_q, n_kv, scale, out=o3, alibi=alibi,
-                                    window=window, keep_first=keep_first)
+                                    window=window, keep_first=keep_first, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate)
 
     # ---- stacks of unlike layers ----------------------------------------------------------------------
-    def embed_f32(self, ids, weight, out, gamma=None, cols=None, eps=1e-5):
-        x = ref.embed(ids, weight).float()
+    def embed_f32(self, ids, weight, out, gamma=None, cols=None, eps=1e-5, scale=1.0):
+        x = ref.embed(ids, weight).float() * scale
         out.copy_(x if gamma is None else x * torch.rsqrt((x * x).sum(-1, keepdim=True) / cols + eps) * gamma)
         return out
 
-    def norm_residual(self, resid, gamma, out, delta=None, factor=1.0, post=None, cols=None, eps=1e-5, store_resid=True):
-        x, y = ref.norm_residual(resid, gamma, delta, factor, post, cols, eps)
-        if delta is not None and delta.dtype == torch.float32:
-            delta.zero_()
+    def norm_residual(self, resid, gamma, out, delta=None, factor=1.0, post=None, cols=None, eps=1e-5, store_resid=True, groups=1,
+                      delta2=None, post2=None):
+        x, y = ref.norm_residual(resid, gamma, delta, factor, post, cols, eps, groups, delta2, post2)
+        for d in (delta, delta2):
+            if d is not None and d.dtype == torch.float32:
+                d.zero_()
         if store_resid:
             resid.copy_(x)
         out.copy_(y)
         return out
 
-    def mixer_in_proj(self, x, w_in, n_attn, proj, q_out, kv_layer, tok_pos, tok_slot, n_q, n_kv, d, block_size, workspace=None):
-        self.qkv_rope_kv_append(x, w_in[:n_attn], None, None, q_out, kv_layer, tok_pos, tok_slot, None, n_q, n_kv, d, d, block_size)
-        if w_in.shape[0] > n_attn:
-            self.gemm(x, w_in[n_attn:], proj[:, n_attn:w_in.shape[0]])
+    def mixer_in_proj(self, x, lw, a, proj, q_out, kv_layer, first, tok_pos, tok_slot, block_size, eps, workspace=None):
+        self.gemm(x, lw.w_qkv, proj[:, :lw.w_qkv.shape[0]], bias=lw.b_qkv)
+        self.attention_append(proj, lw, a, q_out, kv_layer, first, tok_pos, tok_slot, block_size, eps)
+
+    def attention_append(self, proj, lw, a, q_out, kv_layer, first, tok_pos, tok_slot, block_size, eps):
+        q = ref.attention_append(proj, kv_layer, tok_pos, tok_slot, a.heads if q_out is not None else 0, a.kv_heads, lw.rot_freq,
+                                 lw.q_norm, lw.k_norm, a.heads * a.dim, a.kv_heads * a.dim, eps, first, lw.v_mix)
+        if q_out is not None:
+            q_out.copy_(q)
 
     def state_space(self, proj, lw, m, ssm_state, conv_state, spans, n_single, conv_buf, dt_buf, out):
         for row0, n, seen, slot in spans.tolist():
@@ -145,6 +152,29 @@ class CpuOps:
         if out is not None:
             out.copy_(ref.gated_norm(y, proj[:, :m.inner], lw.ssm_norm, m.heads, eps, gate_after=True))
         return y
+
+    def gru(self, proj, lw, m, state, spans, n_single, out, workspace):
+        C = m.inner
+        for row0, n, seen, slot in spans.tolist():
+            u, S = proj[row0:row0 + n].float(), state[slot].view(-1)
+            if seen == 0:
+                S.zero_()
+            y = ref.gru_scan(u[:, :C] + lw.gru_bias[:C], u[:, C:2 * C] + lw.gru_bias[C:], S)
+            if out is not None:
+                out[row0:row0 + n] = y * torch.nn.functional.silu(u[:, 2 * C:3 * C])
+
+    def linear_attention(self, q, k, v, gate, z, lw, m, state, spans, n_single, y, out, eps, workspace):
+        NK, NV = m.heads * m.dim, m.heads * m.vdim
+        for row0, n, seen, slot in spans.tolist():
+            if seen == 0:
+                state[slot].zero_()
+            rows = slice(row0, row0 + n)
+            decay = ref.linear_decay(z[rows, :NK].float() + lw.decay_bias, m.tau)
+            split = lambda t, w: t[rows, :w].reshape(n, m.heads, w // m.heads)  # noqa: E731
+            y[rows, :NV] = ref.linear_scan(split(q, NK), split(k, NK), split(v, NV), decay.view(n, m.heads, m.dim), state[slot]).reshape(n, NV)
+        if out is not None:
+            out.zero_()
+            out[:, :NV] = ref.gated_norm(y[:, :NV], gate[:, :NV], lw.ssm_norm, m.heads, eps, gate_after=True)
 
     def latent_append(self, proj, q_out, pages, tok_pos, tok_slot, c, lw, eps):
         n_q = c.heads * c.head_width
@@ -179,15 +209,21 @@ class CpuOps:
         self._picked = torch.topk(s + lw.router_bias, f.top, -1).indices
         self._scores = s.gather(-1, self._picked) * f.router_scale
 
+    def sigmoid_route(self, x, lw, f, bufs):
+        s = torch.sigmoid(ref.gemm(x, lw.w_router, out_dtype=torch.float32)[:, :f.experts])
+        self._scores, self._picked = torch.topk(s, f.top, -1)
+
     def routed_experts(self, x, ids, lw, f, act, base, out, bufs):
-        """``out`` = ``base`` (None, or ``out`` itself) + the chosen experts' weighted outputs."""
-        picked = self._picked
+        """``out`` = ``base`` (None, or ``out`` itself) + the chosen experts' weighted outputs (the outputs of weighted inputs,
+        where the routing says so)."""
+        picked, inputs = self._picked, f.weighs_inputs
         acc = torch.zeros_like(out) if base is None else base.float().clone()
         for e, ew in enumerate(lw.experts):
             rows, place = (picked == e).nonzero(as_tuple=True)
             if rows.numel():
-                h = ref.gemm(x.index_select(0, rows), ew.w_up, act=act, gated=f.gated, limit=f.limit)
-                acc.index_add_(0, rows, ref.gemm(h, ew.w_down).float() * self._scores[rows, place][:, None])
+                xs, s = x.index_select(0, rows), self._scores[rows, place][:, None]
+                h = ref.gemm((xs.float() * s).to(x.dtype) if inputs else xs, ew.w_up, act=act, gated=f.gated, limit=f.limit)
+                acc.index_add_(0, rows, ref.gemm(h, ew.w_down).float() * (1.0 if inputs else s))
         out.copy_(acc)
         return out
 
@@ -326,16 +362,16 @@ class CudaOps:
             self.k.rope_kv_append(scratch, scratch, kv_layer, tok_pos, tok_slot, inv_freq, 0, n_kv, d, rot_dim, block_size)
 
     def attention(self, q, out, kv_layer, batch, n_q, n_kv, d, scale, ws_small=None, ws_large=None, alibi=None, window=0,
-                  keep_first=0):
+                  keep_first=0, sink=None, sigmoid_bias=None, gate=None):
         k = self.k
         bs = batch.block_size
         if q.dtype == torch.float32 or d not in (64, 128):
             k.paged_attention_generic(q, out, kv_layer, batch.block_tables(), batch.tokens_to_seq(), batch.tok_pos(), n_q, n_kv, d, bs,
-                                      scale, window=window, keep_first=keep_first)
+                                      scale, window=window, keep_first=keep_first, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate)
             return
         # with a sliding window an item reads at most window + one tile of keys: size the KV split for that
         seen = lambda n_kv_tokens: windowed_len(n_kv_tokens, window, keep_first)  # noqa: E731
-        opts = dict(alibi=alibi, window=window, keep_first=keep_first)
+        opts = dict(alibi=alibi, window=window, keep_first=keep_first, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate)
         if batch.n_items_small:
             n = batch.n_items_small
             if use_packed_decode(n_q, n_kv, d):
@@ -354,27 +390,47 @@ class CudaOps:
                                       scale, n_splits=splits, workspace=ws_large if splits > 1 else None, **opts)
 
     # ---- stacks of unlike layers ----------------------------------------------------------------------
-    def embed_f32(self, ids, weight, out, gamma=None, cols=None, eps=1e-5):
-        return self.k.embed_f32(ids, weight, out, gamma=gamma, cols=cols, eps=eps)
+    def embed_f32(self, ids, weight, out, **kw):
+        return self.k.embed_f32(ids, weight, out, **kw)
 
     def norm_residual(self, resid, gamma, out, **kw):
         return self.k.norm_residual(resid, gamma, out, **kw)
 
-    def mixer_in_proj(self, x, w_in, n_attn, proj, q_out, kv_layer, tok_pos, tok_slot, n_q, n_kv, d, block_size, workspace=None):
+    def mixer_in_proj(self, x, lw, a, proj, q_out, kv_layer, first, tok_pos, tok_slot, block_size, eps, workspace=None):
         """Every projection that reads the layer's input: Q to ``q_out``, K / V to their pages, the rest to ``proj``'s columns
-        behind the first ``n_attn``. Decode-size batches stream all weights in ONE GEMM; larger ones keep the QKV rows' fused
-        paged epilogue and run the others as a second GEMM."""
-        k, T, n_in = self.k, x.shape[0], w_in.shape[0]
-        if x.dtype != torch.float32 and d in (64, 128) and T >= self.FUSED_QKV_MIN_TOKENS:
-            k.qkv_rope_proj(x, w_in[:n_attn], q_out, kv_layer, tok_pos, tok_slot, None, n_q, n_kv, d, block_size)
+        behind those of the attention. Decode-size batches stream all weights in ONE GEMM; larger ones keep the QKV rows' fused
+        rotating and paged epilogue (where no norm comes before it) and run the others as a second GEMM. ``first``: pages of the
+        layer whose values are mixed in."""
+        k, T, d, w_in, b = self.k, x.shape[0], a.page_dim, lw.w_qkv, lw.b_qkv
+        n_in, n_attn = w_in.shape[0], (a.heads + 2 * a.kv_heads) * d
+        if x.dtype != torch.float32 and d in (64, 128) and T >= self.FUSED_QKV_MIN_TOKENS and not a.qk_norm:
+            k.qkv_rope_proj(x, w_in[:n_attn], q_out, kv_layer, tok_pos, tok_slot, lw.rot_freq, a.heads, a.kv_heads, d, block_size,
+                            bias_qkv=None if b is None else b[:n_attn])
             if n_in > n_attn:
-                k.gemm(x, w_in[n_attn:], out=proj[:, n_attn:n_in])
+                k.gemm(x, w_in[n_attn:], out=proj[:, n_attn:n_in], bias=None if b is None else b[n_attn:])
+            if first is not None:
+                k.mix_cached_values(kv_layer, first, tok_slot, lw.v_mix, a.kv_heads, d, block_size)
             return
-        self.gemm(x, w_in, proj[:, :n_in], workspace=workspace)
-        if x.dtype == torch.float32:
-            k.kv_append_generic(proj, q_out, kv_layer, tok_slot, n_q, n_kv, d, block_size)
+        self.gemm(x, w_in, proj[:, :n_in], bias=b, workspace=workspace)
+        self.attention_append(proj, lw, a, q_out, kv_layer, first, tok_pos, tok_slot, block_size, eps)
+
+    def attention_append(self, proj, lw, a, q_out, kv_layer, first, tok_pos, tok_slot, block_size, eps):
+        """Projected rows [q | k | v] -> rotated (and normed) queries and page rows. ``q_out`` None: keys and values only."""
+        k, d, n_q = self.k, a.page_dim, a.heads if q_out is not None else 0
+        q_out = proj if q_out is None else q_out
+        if a.rot is not None or a.qk_norm or first is not None:
+            k.attention_append(proj, q_out, kv_layer, tok_pos, tok_slot, n_q, a.kv_heads, d, block_size, lw.rot_freq, lw.q_norm, lw.k_norm,
+                               a.heads * a.dim, a.kv_heads * a.dim, eps, first, lw.v_mix)
+        elif proj.dtype == torch.float32:
+            k.kv_append_generic(proj, q_out, kv_layer, tok_slot, n_q, a.kv_heads, d, block_size)
         else:
-            k.rope_kv_append(proj, q_out, kv_layer, tok_pos, tok_slot, None, n_q, n_kv, d, d, block_size)
+            k.rope_kv_append(proj, q_out, kv_layer, tok_pos, tok_slot, None, n_q, a.kv_heads, d, d, block_size)
+
+    def gru(self, proj, lw, m, state, spans, n_single, out, workspace):
+        self.k.gru(proj, lw.gru_bias, state, spans, n_single, out, workspace)
+
+    def linear_attention(self, q, k, v, gate, z, lw, m, state, spans, n_single, y, out, eps, workspace):
+        self.k.linear_attention(q, k, v, gate, z, lw.decay_bias, 1.0 / m.tau, state, spans, n_single, y, out, lw.ssm_norm, eps, workspace)
 
     def state_space(self, proj, lw, m, ssm_state, conv_state, spans, n_single, conv_buf, dt_buf, out):
         return self.k.state_space(proj, lw.ssm_conv_w, lw.ssm_conv_b, lw.ssm_dt_bias, lw.ssm_a, lw.ssm_d, ssm_state, conv_state, spans,
@@ -396,16 +452,25 @@ class CudaOps:
         k.moe_topk_gating(logits[:, :f.experts], f.top, False, bufs["scores"][:T], bufs["expert_ids"][:T], bufs["offsets"][:T], bufs["counts"],
                           bias=lw.router_bias, scale=f.router_scale, clear=True)
 
+    def sigmoid_route(self, x, lw, f, bufs):
+        """Experts by router: the largest sigmoids of fp32 logits."""
+        k, T = self.k, x.shape[0]
+        logits = bufs["logits"][:T]
+        k.gemm_accum(x, lw.w_router, logits)
+        k.moe_topk_gating(logits[:, :f.experts], f.top, False, bufs["scores"][:T], bufs["expert_ids"][:T], bufs["offsets"][:T], bufs["counts"],
+                          clear=True, sigmoid=True)
+
     def routed_experts(self, x, ids, lw, f, act, base, out, bufs):
         """Routed tokens: scatter -> grouped GEMM -> grouped GEMM -> weighted sum, added to ``base`` (``out`` itself: in place)."""
         k, T, E = self.k, x.shape[0], f.experts
         rows = k.moe_padded_rows(T, E, f.top)
         xs, hs, ys = bufs["xs"][:rows], bufs["hs"][:rows], bufs["ys"][:rows]
         ids_e, off, slots = bufs["expert_ids"][:T], bufs["offsets"][:T], bufs["mapped_slots"][:T]
-        k.moe_scatter(x, xs, ids_e, off, bufs["counts"], bufs["pad_off"], slots, f.top)
+        scores = bufs["scores"][:T]
+        k.moe_scatter(x, xs, ids_e, off, bufs["counts"], bufs["pad_off"], slots, f.top, scores if f.weighs_inputs else None)
         k.moe_gemm(xs, lw.moe_up, bufs["pad_off"], E, hs, act=act, gated=f.gated, limit=f.limit)
         k.moe_gemm(hs, lw.moe_down, bufs["pad_off"], E, ys)
-        return k.moe_combine(ys, slots, bufs["scores"][:T], base, out)
+        return k.moe_combine(ys, slots, None if f.weighs_inputs else scores, base, out)
 
     def table_moe(self, x, ids, lw, f, act, shared, out, bufs):
         self.table_route(ids, lw, f, bufs)

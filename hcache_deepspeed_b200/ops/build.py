@@ -29,7 +29,8 @@ CUDA_LIB = LIB_DIR / "libhds_b200.so"
 #: quantisers, optimizers, host buffers; `native.cuda_lib` builds the full library when one of those is asked for)
 SERVE_LIB = LIB_DIR / "libhds_serve.so"
 SERVE_UNITS = ("gemm", "gemm_2sm", "gemm_f32", "elementwise", "residual_norm", "attention_splitkv", "attention_prefill",
-               "attention_generic", "attention_latent", "latent", "moe", "ssm", "ssm_chunk", "delta", "delta_chunk", "tp_comm")
+               "attention_generic", "attention_latent", "attention_append", "latent", "moe", "ssm", "ssm_chunk", "delta", "delta_chunk", "gru",
+               "linear_attention", "linear_chunk", "tp_comm")
 HOST_LIB = LIB_DIR / "libhds_host.so"
 
 NVCC_FLAGS = [

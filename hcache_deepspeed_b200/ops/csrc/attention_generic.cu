@@ -26,7 +26,7 @@ __global__ void __launch_bounds__(kGenWarps * 32)
 paged_attn_generic_kernel(const void* __restrict__ q, void* __restrict__ out, int64_t ld_out, const void* __restrict__ cache,
                           const int32_t* __restrict__ tables, int table_stride, const int32_t* __restrict__ tok_seq,
                           const int32_t* __restrict__ tok_pos, int n_units, int n_q, int n_kv, int D, int bs, float scale,
-                          int window, int keep_first, int DV, int64_t v_plane, const int32_t* __restrict__ spans, int limit) {
+                          int window, int keep_first, int DV, int64_t v_plane, const int32_t* __restrict__ spans, int limit, const AttnOptions opt) {
     extern __shared__ float q_s[];   // [warps][D]
     pdl_enter();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -45,7 +45,9 @@ paged_attn_generic_kernel(const void* __restrict__ q, void* __restrict__ out, in
     float acc[DIMS];
 #pragma unroll
     for (int i = 0; i < DIMS; ++i) acc[i] = 0.0f;
-    float m = -INFINITY, l = 0.0f;
+    const bool sigmoid = opt.sigmoid_bias != nullptr;      // sigmoid weights: no maximum, no denominator
+    const float bias = sigmoid ? opt.sigmoid_bias[head] : 0.0f;
+    float m = sigmoid ? 0.0f : -INFINITY, l = 0.0f;
     const int lo = window > 0 ? max(0, pos - window + 1) : 0;
     const int keep_end = min(keep_first, lo);      // the kept range ends where the window takes over
     for (int range = 0; range < 2; ++range) {
@@ -61,9 +63,9 @@ paged_attn_generic_kernel(const void* __restrict__ q, void* __restrict__ out, in
                 s = 0.0f;
                 for (int c = 0; c < D; ++c) s = fmaf(qw[c], load_any<DT>(cache, krow + c), s);
             }
-            const float m_new = fmaxf(m, warp_max(s));
+            const float m_new = sigmoid ? 0.0f : fmaxf(m, warp_max(s));
             const float keep = m == -INFINITY ? 0.0f : expf(m - m_new);
-            const float p = j < j1 ? expf(s - m_new) : 0.0f;
+            const float p = j >= j1 ? 0.0f : sigmoid ? 1.0f / (1.0f + expf(-(s + bias))) : expf(s - m_new);
             l = l * keep + warp_sum(p);
             m = m_new;
 #pragma unroll
@@ -80,10 +82,15 @@ paged_attn_generic_kernel(const void* __restrict__ q, void* __restrict__ out, in
             }
         }
     }
+    if (sigmoid) l = 1.0f;
+    else if (opt.sink != nullptr) l += expf(opt.sink[head] - m);
 #pragma unroll
     for (int i = 0; i < DIMS; ++i) {
         const int c = lane + 32 * i;
-        if (c < DV) store_any<DT>(out, t * ld_out + head * DV + c, acc[i] / l);
+        if (c >= DV) continue;
+        float o = acc[i] / l;
+        if (opt.gate != nullptr) o /= 1.0f + expf(-load_any<DT>(opt.gate, t * opt.gate_ld + head * DV + c));
+        store_any<DT>(out, t * ld_out + head * DV + c, o);
     }
 }
 
@@ -117,6 +124,7 @@ extern "C" int hds_paged_attention_generic(const void* q, void* out, int64_t ld_
                                            const int32_t* tok_pos, int T, int n_q_heads, int n_kv_heads, int head_dim,
                                            int block_size, float scale, int window, int keep_first, int value_dim,
                                            const int32_t* spans, int limit, int dtype, void* stream) {
+    const AttnOptions opt = attn_take_options();
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_paged_attention_generic: dtype 0 bf16 / 1 fp16 / 2 fp32");
     HDS_REQUIRE(head_dim >= 1 && value_dim <= head_dim && (value_dim > 0 ? value_dim : head_dim) <= 32 * kWideDims && head_dim <= 2816,
                 "hds_paged_attention_generic: values up to 2048, keys up to 2816");
@@ -133,11 +141,11 @@ extern "C" int hds_paged_attention_generic(const void* q, void* out, int64_t ld_
     if (dv <= 32 * kGenMaxDims)                                                                                               \
         HDS_CHECK_CUDA(launch_kernel(paged_attn_generic_kernel<DT, kGenMaxDims>, grid, block, smem, s, q, out, ld_out,        \
                                      kv_cache_layer, block_tables, max_blocks_per_seq, tok_seq, tok_pos, units, n_q_heads,    \
-                                     n_kv_heads, head_dim, block_size, scale, window, keep_first, dv, v_plane, spans, limit)); \
+                                     n_kv_heads, head_dim, block_size, scale, window, keep_first, dv, v_plane, spans, limit, opt)); \
     else                                                                                                                      \
         HDS_CHECK_CUDA(launch_kernel(paged_attn_generic_kernel<DT, kWideDims>, grid, block, smem, s, q, out, ld_out,          \
                                      kv_cache_layer, block_tables, max_blocks_per_seq, tok_seq, tok_pos, units, n_q_heads,    \
-                                     n_kv_heads, head_dim, block_size, scale, window, keep_first, dv, v_plane, spans, limit))
+                                     n_kv_heads, head_dim, block_size, scale, window, keep_first, dv, v_plane, spans, limit, opt))
     if (dtype == 0) { HDS_GEN(0); }
     else if (dtype == 1) { HDS_GEN(1); }
     else { HDS_GEN(2); }

@@ -10,6 +10,8 @@
 //               warps to interleave: ONE tcgen05.ld pass pulls this thread's 64 scores into
 //               registers and releases S at once (so Q K^T of the next tile runs under this tile's exponentials),
 //               causal mask, online max/sum, P -> shared (UMMA K-major swizzled layout).
+//   Sigmoid weights (kSigmoid) need neither maximum nor sum: P = sigmoid(S + a number per head), O is the plain sum of P V.
+//   A learned sink joins the row sum at the very end, where an output gate is applied too.
 //   O accumulates in TMEM across all KV tiles (PV issued with accumulate); it is rescaled in place only when a
 //   row's running max grows by more than 2^8 (lazy rescale: probabilities are computed against a slightly stale
 //   max, which is exact after the final division by the matching row sum)
@@ -49,11 +51,21 @@ struct PrefillArgs {
     int window;         // sliding-window attention: a query at position p sees keys (p - window, p]; 0 = unlimited
     int keep_first;     // with a window: the first keep_first positions stay visible to every later query
     int64_t out_ld;     // elements between the output rows of two tokens
+    const float* sink;  // [n_q_heads] or nullptr: one more score (natural-log units) in every denominator
+    const float* sigmoid_bias;  // kSigmoid: [n_q_heads], natural-log units
+    const void* gate;   // nullptr, or rows (gate_ld apart) like out's whose sigmoid multiplies it
+    int64_t gate_ld;
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+__device__ __forceinline__ float rcp_approx(float x) {   // (of infinity: zero)
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
 
@@ -64,7 +76,35 @@ __host__ __device__ constexpr size_t pf_smem_bytes() {
            2 * 2 * 128 * 4 /*row-max exchange*/ + 1024;
 }
 
-template <int D, bool kBf16, bool kPacked = false>
+// factor of a finished row: the denominator with the sink; m in log2 units
+template <bool kSigmoid>
+__device__ __forceinline__ float pf_row_factor(const PrefillArgs& a, float l, float m, int head) {
+    if constexpr (kSigmoid) return 1.0f;
+    if (a.sink != nullptr) l += exp2f(a.sink[head] * 1.4426950408889634f - m);
+    return 1.0f / l;
+}
+// eight finished values -> 16 bytes of the output, through the gate
+template <bool kBf16>
+__device__ __forceinline__ void pf_store8(const PrefillArgs& a, const float* o, float f, int64_t row, int64_t col) {
+    float x[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] = o[i] * f;
+    if (a.gate != nullptr) {
+        const uint4 g = *reinterpret_cast<const uint4*>(reinterpret_cast<const char*>(a.gate) + (row * a.gate_ld + col) * 2);
+        const uint32_t w[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            x[2 * i] = __fdividef(x[2 * i], 1.0f + ex2_approx(unpack_lo<kBf16>(w[i]) * -1.4426950408889634f));
+            x[2 * i + 1] = __fdividef(x[2 * i + 1], 1.0f + ex2_approx(unpack_hi<kBf16>(w[i]) * -1.4426950408889634f));
+        }
+    }
+    uint4 v;
+    v.x = pack2<kBf16>(x[0], x[1]); v.y = pack2<kBf16>(x[2], x[3]);
+    v.z = pack2<kBf16>(x[4], x[5]); v.w = pack2<kBf16>(x[6], x[7]);
+    st_v4(reinterpret_cast<char*>(a.out) + (row * a.out_ld + col) * 2, v);
+}
+
+template <int D, bool kBf16, bool kPacked = false, bool kSigmoid = false>
 __global__ void __launch_bounds__(kPfThreads, 1)
 paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
                           const PrefillArgs a) {
@@ -245,7 +285,8 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         const uint32_t lane_addr = (quad * 32u) << 16;
         constexpr int HC = kPfTok / 2;               // key columns per thread
         constexpr int HD2 = D / 2;                   // output dims per thread
-        float m_run = -INFINITY, l_run = 0.0f;       // l_run: this thread's columns only
+        float m_run = kSigmoid ? 0.0f : -INFINITY, l_run = 0.0f;       // l_run: this thread's columns only
+        const float sig_bias = kSigmoid ? a.sigmoid_bias[min(r_head, a.n_q_heads - 1)] * -1.4426950408889634f : 0.0f;
         uint8_t* p_row = p_sm + half * PANEL_BYTES + r * 128;   // half h owns P panel h (64 tokens = 128 B per row)
         constexpr float kRescaleThreshold = 8.0f;    // log2 units: probabilities stay below 2^8 against a stale max
         auto pair_sync = [&]() { asm volatile("bar.sync %0, 64;" ::"r"(1 + quad) : "memory"); };
@@ -291,6 +332,9 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
                     sr[j] = __float_as_uint(fmaf(sl, d0 + static_cast<float>(j), __uint_as_float(sr[j])));
             }
             float tmax = -INFINITY;
+            uint32_t packed[HC / 2];
+            float alpha = 1.0f;
+            bool rescale = false;
             if (need_mask) {
 #pragma unroll
                 for (int j = 0; j < HC; ++j) {
@@ -299,10 +343,18 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
                     sr[j] = __float_as_uint(sv);
                     tmax = fmaxf(tmax, sv);
                 }
-            } else {
+            } else if constexpr (!kSigmoid) {
 #pragma unroll
                 for (int j = 0; j < HC; ++j) tmax = fmaxf(tmax, __uint_as_float(sr[j]));
             }
+            if constexpr (kSigmoid) {
+#pragma unroll
+                for (int j = 0; j < HC; j += 2) {     // (hidden keys: 1 / (1 + inf) = 0)
+                    const float p0 = rcp_approx(1.0f + ex2_approx(fmaf(__uint_as_float(sr[j]), -a.scale_log2, sig_bias)));
+                    const float p1 = rcp_approx(1.0f + ex2_approx(fmaf(__uint_as_float(sr[j + 1]), -a.scale_log2, sig_bias)));
+                    packed[j >> 1] = pack2<kBf16>(p0, p1);
+                }
+            } else {
             // row max over both halves
             float* x = xch + (ti & 1) * 256;
             x[half * 128 + r] = tmax;
@@ -313,10 +365,9 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
             const bool grow = (m_cand > m_run + kRescaleThreshold) || (m_run == -INFINITY && m_cand != -INFINITY);
             const float m_new = grow ? m_cand : m_run;
             const bool fresh = (m_run == -INFINITY);   // nothing accumulated for this row yet
-            const float alpha = (!grow || fresh) ? (grow ? 0.0f : 1.0f) : ex2_approx(m_run - m_new);
+            alpha = (!grow || fresh) ? (grow ? 0.0f : 1.0f) : ex2_approx(m_run - m_new);
             const float m_sub = (m_new == -INFINITY) ? 0.0f : m_new;  // fully masked row: exp2(-inf - 0) = 0
             float ps0 = 0.0f, ps1 = 0.0f;
-            uint32_t packed[HC / 2];
 #pragma unroll
             for (int j = 0; j < HC; j += 2) {
                 const float p0 = ex2_approx(fmaf(__uint_as_float(sr[j]), a.scale_log2, -m_sub));
@@ -327,14 +378,15 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
             }
             l_run = l_run * alpha + (ps0 + ps1);
             m_run = m_new;
+            // (alpha may underflow to exactly 0 when the maximum jumps by > 126 log2 units, e.g. under a steep ALiBi
+            // slope: the stale accumulation must then still be wiped, so "fresh" is tracked separately)
+            rescale = grow && !fresh;
+            }
             // PV of the previous tile must be complete before P is overwritten or O is rescaled
             if (ti > 0) {
                 mbar_wait(o_full, (ti - 1) & 1);
                 tc_fence_after();
-                // (alpha may underflow to exactly 0 when the maximum jumps by > 126 log2 units, e.g. under a steep ALiBi
-                // slope: the stale accumulation must then still be wiped, so "fresh" is tracked separately)
-                const bool rescale = grow && !fresh;
-                if (__any_sync(0xffffffffu, rescale)) {
+                if (!kSigmoid && __any_sync(0xffffffffu, rescale)) {
                     const float f = rescale ? alpha : 1.0f;
 #pragma unroll
                     for (int c = 0; c < HD2; c += 32) {
@@ -361,7 +413,7 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
             if (lane == 0) mbar_arrive(p_full);
         }
         // ---- total row sum over both halves, then my half of the final O row from TMEM ----
-        if (quad_live) {
+        if (quad_live && !kSigmoid) {
             float* x = xch + (n_tiles & 1) * 256;
             x[half * 128 + r] = l_run;
             pair_sync();
@@ -380,20 +432,12 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         }
         tc_fence_before();
         const bool row_valid = r < n_live_rows;
-        char* dst = reinterpret_cast<char*>(a.out) +
-                    (static_cast<int64_t>(item.q_row0 + r_tok) * a.out_ld + r_head * D + half * HD2) * 2;
+        const int64_t out_row = item.q_row0 + r_tok, out_col = r_head * D + half * HD2;
         if (eff_splits == 1) {
             if (row_valid) {
-                const float inv = 1.0f / l_run;
+                const float inv = pf_row_factor<kSigmoid>(a, l_run, m_run, r_head);
 #pragma unroll
-                for (int c = 0; c < HD2; c += 8) {
-                    uint4 v;
-                    v.x = pack2<kBf16>(o_acc[c + 0] * inv, o_acc[c + 1] * inv);
-                    v.y = pack2<kBf16>(o_acc[c + 2] * inv, o_acc[c + 3] * inv);
-                    v.z = pack2<kBf16>(o_acc[c + 4] * inv, o_acc[c + 5] * inv);
-                    v.w = pack2<kBf16>(o_acc[c + 6] * inv, o_acc[c + 7] * inv);
-                    st_v4(dst + c * 2, v);
-                }
+                for (int c = 0; c < HD2; c += 8) pf_store8<kBf16>(a, o_acc + c, inv, out_row, out_col + c);
             }
         } else if (quad_live) {  // warp-uniform: this quadrant owns valid rows
             // ---- split-KV: park the partial (O, m, l); the last split of this (quadrant, half) merges its dims ----
@@ -434,16 +478,9 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
                             o_acc[c + 3] = fmaf(w, t.w, o_acc[c + 3]);
                         }
                     }
-                    const float inv = 1.0f / l_tot;
+                    const float inv = pf_row_factor<kSigmoid>(a, l_tot, mx, r_head);
 #pragma unroll
-                    for (int c = 0; c < HD2; c += 8) {
-                        uint4 v;
-                        v.x = pack2<kBf16>(o_acc[c + 0] * inv, o_acc[c + 1] * inv);
-                        v.y = pack2<kBf16>(o_acc[c + 2] * inv, o_acc[c + 3] * inv);
-                        v.z = pack2<kBf16>(o_acc[c + 4] * inv, o_acc[c + 5] * inv);
-                        v.w = pack2<kBf16>(o_acc[c + 6] * inv, o_acc[c + 7] * inv);
-                        st_v4(dst + c * 2, v);
-                    }
+                    for (int c = 0; c < HD2; c += 8) pf_store8<kBf16>(a, o_acc + c, inv, out_row, out_col + c);
                 }
                 __syncwarp();
                 if (lane == 0) a.tickets[(unit * 4 + quad) * 2 + half] = 0;
@@ -488,10 +525,9 @@ static bool prefill64_enabled() {
     return tile == 64;
 }
 
-template <int D, bool kBf16, bool kPacked = false>
-static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tkv, const PrefillArgs& a, int n_items,
-                          cudaStream_t s) {
-    auto kern = paged_attn_prefill_kernel<D, kBf16, kPacked>;
+template <int D, bool kBf16, bool kPacked, bool kSigmoid>
+static int launch_prefill_as(const CUtensorMap& tq, const CUtensorMap& tkv, const PrefillArgs& a, int n_items, cudaStream_t s) {
+    auto kern = paged_attn_prefill_kernel<D, kBf16, kPacked, kSigmoid>;
     static bool configured[64] = {false};
     int dev = 0;
     cudaGetDevice(&dev);
@@ -503,6 +539,12 @@ static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tkv, const P
     dim3 grid(n_items, kPacked ? a.n_kv_heads : a.n_q_heads, a.n_splits);
     HDS_CHECK_CUDA(launch_kernel(kern, grid, dim3(kPfThreads), pf_smem_bytes<D>(), s, tq, tkv, a));
     return HDS_OK;
+}
+
+template <int D, bool kBf16, bool kPacked = false>
+static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tkv, const PrefillArgs& a, int n_items, cudaStream_t s) {
+    return a.sigmoid_bias != nullptr ? launch_prefill_as<D, kBf16, kPacked, true>(tq, tkv, a, n_items, s)
+                                     : launch_prefill_as<D, kBf16, kPacked, false>(tq, tkv, a, n_items, s);
 }
 
 }  // namespace hds
@@ -534,10 +576,15 @@ static int attention_tc_impl(bool packed, const void* q, void* out, const void* 
     const int window = attn_take_window();
     const int keep_first = attn_take_keep_first();
     const int64_t out_ld = attn_take_out_stride();
+    const AttnOptions opt = attn_take_options();
     if (n_items == 0) return HDS_OK;
     PrefillArgs a;
     memset(&a, 0, sizeof(a));
     a.alibi = alibi;
+    a.sink = opt.sink;
+    a.sigmoid_bias = opt.sigmoid_bias;
+    a.gate = opt.gate;
+    a.gate_ld = opt.gate_ld;
     a.window = window;
     a.keep_first = window > 0 ? keep_first : 0;
     a.out_ld = out_ld > 0 ? out_ld : static_cast<int64_t>(n_q_heads) * head_dim;
@@ -584,7 +631,8 @@ static int attention_tc_impl(bool packed, const void* q, void* out, const void* 
     if (packed)
         return dtype == 0 ? launch_prefill<128, true, true>(tq, tkv, a, n_items, s)
                           : launch_prefill<128, false, true>(tq, tkv, a, n_items, s);
-    if (head_dim == 128 && block_size <= 64 && alibi == nullptr && window == 0 && out_ld == 0 && prefill64_enabled())   // no ALiBi / window / strided rows there
+    if (head_dim == 128 && block_size <= 64 && alibi == nullptr && window == 0 && out_ld == 0 && opt.sink == nullptr && opt.sigmoid_bias == nullptr &&
+        opt.gate == nullptr && prefill64_enabled())   // none of the options there
         return dtype == 0 ? launch_prefill64<true>(tq, tkv, a, n_items, s) : launch_prefill64<false>(tq, tkv, a, n_items, s);
     if (head_dim == 128)
         return dtype == 0 ? launch_prefill<128, true>(tq, tkv, a, n_items, s)

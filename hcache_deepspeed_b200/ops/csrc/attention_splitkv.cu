@@ -43,7 +43,25 @@ struct AttnArgs {
     int window;         // sliding-window attention: a query at position p sees keys (p - window, p]; 0 = unlimited
     int keep_first;     // with a window: the first keep_first positions stay visible to every later query
     int64_t out_ld;     // elements between the output rows of two tokens
+    const float* sink;  // [n_q_heads] or nullptr: one more score (natural-log units) in every denominator
+    const float* sigmoid_bias;  // [n_q_heads] or nullptr: keys weigh sigmoid(score + bias), no denominator
+    const void* gate;   // nullptr, or rows (gate_ld apart) like out's whose sigmoid multiplies it
+    int64_t gate_ld;
 };
+
+// a finished output value, behind the denominator (sink included) and the gate; m in log2 units
+template <bool kBf16>
+__device__ __forceinline__ float attn_finish(const AttnArgs& a, float o, float l, float m, int64_t row, int head, int col) {
+    if (a.sigmoid_bias == nullptr) {
+        if (a.sink != nullptr) l += exp2f(a.sink[head] * 1.4426950408889634f - m);
+        o /= l;
+    }
+    if (a.gate != nullptr) {
+        const float g = load_scalar<kBf16>(a.gate, row * a.gate_ld + col);
+        o /= 1.0f + exp2f(g * -1.4426950408889634f);
+    }
+    return o;
+}
 
 template <int D, int W>
 __host__ __device__ constexpr size_t attn_stage_bytes() {
@@ -130,7 +148,7 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
     float m_run[R], l_run[R], acc[R][EPL];
 #pragma unroll
     for (int r = 0; r < R; ++r) {
-        m_run[r] = -INFINITY;
+        m_run[r] = a.sigmoid_bias != nullptr ? 0.0f : -INFINITY;   // (sigmoid weights have no maximum to be relative to)
         l_run[r] = 0.0f;
 #pragma unroll
         for (int i = 0; i < EPL; ++i) acc[r][i] = 0.0f;
@@ -183,6 +201,10 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
         float slope[R];
 #pragma unroll
         for (int r = 0; r < R; ++r) slope[r] = a.alibi ? a.alibi[kvh * G + r % G] * 1.4426950408889634f : 0.0f;
+        const bool sigmoid = a.sigmoid_bias != nullptr;
+        float bias[R];
+#pragma unroll
+        for (int r = 0; r < R; ++r) bias[r] = sigmoid ? a.sigmoid_bias[kvh * G + r % G] * 1.4426950408889634f : 0.0f;
         uint32_t stage = 0, phase = 0;
         for (int ti = t0; ti < t1; ++ti) {
             const uint8_t* ktile = stages + stage * attn_stage_bytes<D, W>();
@@ -228,6 +250,10 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
                     const bool ok = (j < n_mine) && (tok0 + rt <= q_pos) && (r < rows) &&
                                     (a.window <= 0 || tok0 + rt > q_pos - a.window || tok0 + rt < a.keep_first);
                     sc = ok ? fmaf(slope[r], static_cast<float>(tok0 + rt - q_pos), sc) : -INFINITY;
+                    if (sigmoid) {
+                        p[r] = 1.0f / (1.0f + ex2f(-(sc + bias[r])));
+                        continue;
+                    }
                     float mx = sc;
 #pragma unroll
                     for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -310,8 +336,9 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
         }
         if (eff_splits == 1) {
             const int qi = r / G, gg = r % G;
-            store_scalar<kBf16>(a.out, static_cast<int64_t>(item.q_row0 + qi) * a.out_ld + (kvh * G + gg) * D + dd,
-                                o / l);
+            const int64_t row = item.q_row0 + qi;
+            const int hd = kvh * G + gg, col = hd * D + dd;
+            store_scalar<kBf16>(a.out, row * a.out_ld + col, attn_finish<kBf16>(a, o, l, mx, row, hd, col));
         } else {
             a.ws_o[((ws_base + split) * R + r) * D + dd] = o;
         }
@@ -344,8 +371,9 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
             o += w * __ldcg(&a.ws_o[((ws_base + s) * R + r) * D + dd]);
         }
         const int qi = r / G, gg = r % G;
-        store_scalar<kBf16>(a.out, static_cast<int64_t>(item.q_row0 + qi) * a.out_ld + (kvh * G + gg) * D + dd,
-                            o / l);
+        const int64_t row = item.q_row0 + qi;
+        const int hd = kvh * G + gg, col = hd * D + dd;
+        store_scalar<kBf16>(a.out, row * a.out_ld + col, attn_finish<kBf16>(a, o, l, mx, row, hd, col));
     }
     if (tid == 0) a.counters[item_idx * a.n_kv_heads + kvh] = 0;
 }
@@ -405,6 +433,12 @@ static thread_local const float* g_next_alibi = nullptr;
 static thread_local int g_next_window = 0;
 static thread_local int g_next_keep_first = 0;
 static thread_local int64_t g_next_out_stride = 0;
+static thread_local hds::AttnOptions g_next_options = {nullptr, nullptr, nullptr, 0};
+hds::AttnOptions hds::attn_take_options() {
+    const AttnOptions o = g_next_options;
+    g_next_options = {nullptr, nullptr, nullptr, 0};
+    return o;
+}
 const float* hds::attn_take_alibi() {
     const float* p = g_next_alibi;
     g_next_alibi = nullptr;
@@ -441,6 +475,24 @@ extern "C" int hds_attention_next_out_stride(int64_t elements) {
     return HDS_OK;
 }
 
+extern "C" int hds_attention_next_sink(const float* sink) {
+    g_next_options.sink = sink;
+    return HDS_OK;
+}
+
+extern "C" int hds_attention_next_sigmoid(const float* bias) {
+    g_next_options.sigmoid_bias = bias;
+    return HDS_OK;
+}
+
+extern "C" int hds_attention_next_gate(const void* gate, int64_t ld) {
+    HDS_REQUIRE(gate == nullptr || (ld > 0 && ld % 8 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0),
+                "hds_attention_next_gate: 16-byte rows");
+    g_next_options.gate = gate;
+    g_next_options.gate_ld = ld;
+    return HDS_OK;
+}
+
 extern "C" int hds_attention_next_alibi(const float* slopes) {
     g_next_alibi = slopes;
     return HDS_OK;
@@ -470,6 +522,7 @@ extern "C" int hds_paged_attention_splitkv(const void* q, void* out, const void*
     const int window = attn_take_window();
     const int keep_first = attn_take_keep_first();
     const int64_t out_ld = attn_take_out_stride();
+    const AttnOptions opt = attn_take_options();
     HDS_REQUIRE(head_dim == 64 || head_dim == 128, "paged_attention_splitkv: head_dim must be 64 or 128");
     HDS_REQUIRE(block_size == 16 || block_size == 32 || block_size == 64 || block_size == 128,
                 "paged_attention_splitkv: block_size must be 16/32/64/128");
@@ -500,6 +553,10 @@ extern "C" int hds_paged_attention_splitkv(const void* q, void* out, const void*
     a.window = window;
     a.keep_first = window > 0 ? keep_first : 0;
     a.out_ld = out_ld > 0 ? out_ld : static_cast<int64_t>(n_q_heads) * head_dim;
+    a.sink = opt.sink;
+    a.sigmoid_bias = opt.sigmoid_bias;
+    a.gate = opt.gate;
+    a.gate_ld = opt.gate_ld;
     const int64_t units = static_cast<int64_t>(n_items) * n_kv_heads;
     char* ws = reinterpret_cast<char*>(workspace);
     a.counters = reinterpret_cast<int32_t*>(ws);

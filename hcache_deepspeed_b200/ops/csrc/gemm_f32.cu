@@ -18,11 +18,13 @@ struct GemmF32Args {
     float limit;
     const int32_t* group_off;   // as GemmArgs::group_pad_off
     int n_groups;
+    const float* bias;          // [N] or nullptr
 };
 
 __device__ __forceinline__ float act_f32(float x, int act) {
     if (act == ACT_SILU) return x / (1.0f + expf(-x));
     if (act == ACT_RELU) return fmaxf(x, 0.0f);
+    if (act == ACT_RELU2) return fmaxf(x, 0.0f) * fmaxf(x, 0.0f);
     if (act == ACT_GELU) return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f));
     if (act == ACT_GELU_TANH) return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
     return x;
@@ -90,6 +92,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Args g) {
             for (int j = 0; j < 4; ++j) {
                 const int n = n0 + tx * 4 + j;
                 if (n >= g.N) continue;
+                if (g.bias != nullptr) acc[i][j] += g.bias[n];
                 if (g.epilogue == EPI_RED_F32) row[n] += acc[i][j];
                 else row[n] = act_f32(acc[i][j], g.act);
             }
@@ -102,12 +105,13 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Args g) {
 using namespace hds;
 
 extern "C" int hds_gemm_f32(const float* A, int64_t lda, const float* W, int64_t ldw, int M, int N, int K, int epilogue, int act,
-                            float limit, float* out, int64_t ldo, const int32_t* group_off, int n_groups, void* stream) {
+                            float limit, float* out, int64_t ldo, const int32_t* group_off, int n_groups, const float* bias, void* stream) {
     HDS_REQUIRE(epilogue == EPI_STORE || epilogue == EPI_GATED || epilogue == EPI_RED_F32, "hds_gemm_f32: epilogue 0 / 1 / 2");
     HDS_REQUIRE(epilogue != EPI_GATED || N % 2 == 0, "hds_gemm_f32: gated epilogue needs an even N");
     HDS_REQUIRE(group_off == nullptr || M % 128 == 0, "hds_gemm_f32: grouped rows come in multiples of 128");
+    HDS_REQUIRE(bias == nullptr || (epilogue != EPI_GATED && group_off == nullptr), "hds_gemm_f32: a bias goes with plain rows");
     if (M == 0 || N == 0) return HDS_OK;
-    GemmF32Args g{A, lda, W, ldw, out, ldo, M, N, K, epilogue, act, limit, group_off, n_groups};
+    GemmF32Args g{A, lda, W, ldw, out, ldo, M, N, K, epilogue, act, limit, group_off, n_groups, bias};
     const dim3 grid((N + kF32Tile - 1) / kF32Tile, (M + kF32Tile - 1) / kF32Tile);
     HDS_REQUIRE(grid.y <= 65535, "hds_gemm_f32: too many rows");
     HDS_CHECK_CUDA(launch_kernel(gemm_f32_kernel, grid, dim3(256), 0, static_cast<cudaStream_t>(stream), g));

@@ -219,6 +219,13 @@ const float* attn_take_alibi();
 int attn_take_window();   // same for hds_attention_next_window (0 = no sliding window)
 int attn_take_keep_first();       // hds_attention_next_keep_first (0 = none)
 int64_t attn_take_out_stride();   // hds_attention_next_out_stride (0 = dense rows)
+struct AttnOptions {              // hds_attention_next_sink / _sigmoid / _gate
+    const float* sink;
+    const float* sigmoid_bias;
+    const void* gate;
+    int64_t gate_ld;
+};
+AttnOptions attn_take_options();
 
 // Bound of ACT_SWIGLU_CLAMPED armed by hds_gemm_next_act_limit for the next GEMM launch of this thread (gemm.cu).
 float gemm_take_act_limit();

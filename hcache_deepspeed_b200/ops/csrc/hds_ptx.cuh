@@ -535,7 +535,7 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
-enum Activation : int { ACT_IDENTITY = 0, ACT_GELU = 1, ACT_RELU = 2, ACT_SILU = 3, ACT_GELU_TANH = 4, ACT_SWIGLU_CLAMPED = 5 };
+enum Activation : int { ACT_IDENTITY = 0, ACT_GELU = 1, ACT_RELU = 2, ACT_SILU = 3, ACT_GELU_TANH = 4, ACT_SWIGLU_CLAMPED = 5, ACT_RELU2 = 6 };
 // ACT_SWIGLU_CLAMPED (gated epilogues only): g = min(gate, L), u = clamp(up, -L, L), out = g * sigmoid(alpha g) * (u + 1)
 constexpr float kClampedGluAlpha = 1.702f;
 
@@ -560,6 +560,7 @@ __device__ __forceinline__ float apply_act(float x, int act) {
     if (act == ACT_SILU) return __fdividef(x, 1.0f + __expf(-x));
     if (act == ACT_IDENTITY) return x;
     if (act == ACT_RELU) return fmaxf(x, 0.0f);
+    if (act == ACT_RELU2) return fmaxf(x, 0.0f) * fmaxf(x, 0.0f);
     if (act == ACT_GELU_TANH) {
         // 0.5 x (1 + tanh(u)) == x * sigmoid(2u)
         const float u = 0.7978845608028654f * (x + 0.044715f * x * x * x);
@@ -580,6 +581,9 @@ __device__ __forceinline__ void apply_act_vec(float (&v)[N], int act) {
     } else if (act == ACT_RELU) {
 #pragma unroll
         for (int j = 0; j < N; ++j) v[j] = fmaxf(v[j], 0.0f);
+    } else if (act == ACT_RELU2) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[j] = fmaxf(v[j], 0.0f) * fmaxf(v[j], 0.0f);
     } else if (act == ACT_GELU_TANH) {
 #pragma unroll
         for (int j = 0; j < N; ++j) {

@@ -1,0 +1,43 @@
+// Shared pieces of the gated linear attention kernels (linear_attention.cu, linear_chunk.cu).
+#pragma once
+#include "recurrent.cuh"
+
+namespace hds {
+
+struct LinArgs {
+    const void* q;          // [T][ld]: heads * N columns each of q, k; heads * P of v, gate
+    const void* k;
+    const void* v;
+    const void* gate;
+    int64_t ld;
+    const void* z;          // [T][ld_z]: heads * N inputs of the decays, without their bias
+    int64_t ld_z;
+    const float* bias;      // [heads * N]
+    float inv_tau;
+    float* state;           // [slots][heads][P][N]
+    const SsmSpan* spans;
+    int n_seqs, T, heads, P, N;
+    float* y;               // [T][ld_y] read-outs, where they are not finished at once
+    int64_t ld_y;
+    void* out;              // [T][ld_out], or nullptr: the state alone
+    int64_t ld_out;
+    const float* norm_w;    // [heads * P]
+    float eps;
+    int write_y;            // steps leave read-outs in y instead of finished rows in out
+};
+
+// log2 of sigmoid(x)^(1 / tau); below 2^-200 a decay is zero to everything behind it
+template <int DT>
+__device__ __forceinline__ float lin_log2_decay(float x, float inv_tau) {
+    constexpr float kLog2e = 1.4426950408889634f;
+    float l;
+    if constexpr (DT == 2) l = (fminf(x, 0.0f) - log1pf(expf(-fabsf(x)))) * kLog2e;
+    else l = fminf(x, 0.0f) * kLog2e - __log2f(1.0f + __expf(-fabsf(x)));
+    return fmaxf(l * inv_tau, -200.0f);
+}
+
+bool lin_chunk_supported(const LinArgs& a, int dtype, const void* ws, int64_t ws_bytes);
+int lin_chunk_launch(const LinArgs& a, int n_multi, void* ws, int64_t ws_bytes, cudaStream_t s);
+int64_t lin_chunk_workspace(int T, int n_seqs, int heads, int P, int N);
+
+}  // namespace hds

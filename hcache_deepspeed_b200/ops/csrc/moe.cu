@@ -2,10 +2,11 @@
 //
 //   top-k gating  : softmax over the expert logits of each token, k rounds of arg-max (ties -> lower index), optionally of the
 //                   scores plus a per-expert bias; optional renormalisation of the k scores, a factor on them, one atomic per
-//                   (token, choice) to claim a row inside the expert
+//                   (token, choice) to claim a row inside the expert. Sigmoid scores (each expert by itself) likewise
 //   offsets       : per-expert row ranges padded to the GEMM's 128-row tile (so no A tile straddles two experts);
 //                   re-zeroes the counters for the next layer
-//   scatter       : copies each token's activation row to its k expert rows, records the row index per choice
+//   scatter       : copies each token's activation row (optionally times the choice's score) to its k expert rows, records the row
+//                   index per choice
 //   gather        : out[t] += sum_j score[t, j] * y[row(t, j)]   (fp32, straight into the pending residual delta)
 //
 // The expert GEMMs in between are ONE grouped tcgen05 launch each (gemm_core.cuh, GemmArgs::group_pad_off).
@@ -23,7 +24,7 @@ constexpr int kMoeRowPad = 128;
 
 template <int DT>
 __global__ void __launch_bounds__(kGateThreads)
-moe_topk_gating_kernel(void* __restrict__ logits, int64_t ld, int E, int k, int normalize, const float* __restrict__ bias,
+moe_topk_gating_kernel(void* __restrict__ logits, int64_t ld, int E, int k, int normalize, int sigmoid, const float* __restrict__ bias,
                        float scale, int clear, float* __restrict__ scores, int32_t* __restrict__ expert_ids, int32_t* __restrict__ offsets,
                        int32_t* __restrict__ counts) {
     extern __shared__ float probs[];  // [E] scores, [E] what chooses
@@ -50,7 +51,8 @@ moe_topk_gating_kernel(void* __restrict__ logits, int64_t ld, int E, int k, int 
     __syncthreads();
     float sum = 0.0f;
     for (int e = tid; e < E; e += kGateThreads) {
-        const float p = expf(probs[e] - mx);
+        if (sigmoid) choice[e] = probs[e];      // (logits choose as sigmoids do, and still where those have all become 1)
+        const float p = sigmoid ? 1.0f / (1.0f + expf(-probs[e])) : expf(probs[e] - mx);
         probs[e] = p;
         sum += p;
     }
@@ -60,8 +62,10 @@ moe_topk_gating_kernel(void* __restrict__ logits, int64_t ld, int E, int k, int 
     sum = 0.0f;
 #pragma unroll
     for (int w = 0; w < kGateThreads / 32; ++w) sum += red_v[w];
-    const float inv = 1.0f / sum;
-    for (int e = tid; e < E; e += kGateThreads) choice[e] = bias == nullptr ? probs[e] : fmaf(probs[e], inv, bias[e]);
+    const float inv = sigmoid ? 1.0f : 1.0f / sum;
+    for (int e = tid; e < E; e += kGateThreads)
+        if (bias != nullptr) choice[e] = fmaf(probs[e], inv, bias[e]);
+        else if (!sigmoid) choice[e] = probs[e];
     __syncthreads();
     for (int j = 0; j < k; ++j) {
         float bv = -INFINITY;
@@ -129,7 +133,7 @@ __global__ void moe_table_route_kernel(const int32_t* __restrict__ ids, const in
     offsets[c] = atomicAdd(&counts[e], 1);
 }
 
-// out[t] = base[t] + sum_j score[t, j] * y[row(t, j)]: stores, base optional; `accumulate`: out itself is the base. DT: type of y
+// out[t] = base[t] + sum_j score[t, j] * y[row(t, j)]: stores, base optional, scores too (1); `accumulate`: out itself is the base. DT: type of y
 // and base.
 template <int DT>
 __global__ void moe_combine_kernel(const void* __restrict__ y, int64_t ldy, const int32_t* __restrict__ mapped_slots,
@@ -154,7 +158,7 @@ __global__ void moe_combine_kernel(const void* __restrict__ y, int64_t ldy, cons
     for (int c = threadIdx.x * 8; c < H; c += blockDim.x * 8) {
         float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
         if (base != nullptr) add8(base, t * ldb + c, 1.0f, v);
-        for (int j = 0; j < k; ++j) add8(y, static_cast<int64_t>(mapped_slots[t * k + j]) * ldy + c, scores[t * k + j], v);
+        for (int j = 0; j < k; ++j) add8(y, static_cast<int64_t>(mapped_slots[t * k + j]) * ldy + c, scores == nullptr ? 1.0f : scores[t * k + j], v);
         float4* o = reinterpret_cast<float4*>(out + t * ldo + c);
         if (accumulate) {
             const float4 p = o[0], q = o[1];
@@ -176,6 +180,30 @@ __global__ void moe_offsets_kernel(int32_t* __restrict__ counts, int32_t* __rest
             pad_off[e + 1] = acc;
             counts[e] = 0;
         }
+    }
+}
+
+// DT: type of the rows where they are weighted (0 bf16, 1 fp16, 2 fp32); without weights H, ldx and lds count 16-bit units of any type
+template <int DT>
+__global__ void moe_scatter_scaled_kernel(const void* __restrict__ x, int64_t ldx, void* __restrict__ xs, int64_t lds,
+                                          const int32_t* __restrict__ expert_ids, const int32_t* __restrict__ offsets,
+                                          const int32_t* __restrict__ pad_off, const float* __restrict__ scores,
+                                          int32_t* __restrict__ mapped_slots, int H, int k) {
+    pdl_enter();
+    const int t = blockIdx.x, j = blockIdx.y;
+    const int64_t c = static_cast<int64_t>(t) * k + j;
+    const int slot = pad_off[expert_ids[c]] + offsets[c];
+    const float s = scores[c];
+    if (threadIdx.x == 0) mapped_slots[c] = slot;
+    const uint4* src = reinterpret_cast<const uint4*>(reinterpret_cast<const char*>(x) + static_cast<int64_t>(t) * ldx * 2);
+    uint4* dst = reinterpret_cast<uint4*>(reinterpret_cast<char*>(xs) + static_cast<int64_t>(slot) * lds * 2);
+    auto times = [&](uint32_t v) {
+        if constexpr (DT == 2) return __float_as_uint(__uint_as_float(v) * s);
+        else return pack2<DT == 0>(unpack_lo<DT == 0>(v) * s, unpack_hi<DT == 0>(v) * s);
+    };
+    for (int i = threadIdx.x; i < (H >> 3); i += blockDim.x) {
+        const uint4 v = src[i];
+        dst[i] = make_uint4(times(v.x), times(v.y), times(v.z), times(v.w));
     }
 }
 
@@ -222,8 +250,8 @@ __global__ void moe_gather_kernel(const void* __restrict__ y, int64_t ldy, const
 
 using namespace hds;
 
-extern "C" int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E, int k, int normalize, const float* bias, float scale,
-                                   int clear, int logits_dtype, float* scores, int32_t* expert_ids, int32_t* offsets,
+extern "C" int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E, int k, int normalize, int sigmoid, const float* bias,
+                                   float scale, int clear, int logits_dtype, float* scores, int32_t* expert_ids, int32_t* offsets,
                                    int32_t* counts, void* stream) {
     HDS_REQUIRE(E >= 1 && E <= 4096, "hds_moe_topk_gating: 1..4096 experts");
     HDS_REQUIRE(k >= 1 && k <= kMoeMaxK && k <= E, "hds_moe_topk_gating: top_k must be in 1..64 and <= experts");
@@ -235,26 +263,34 @@ extern "C" int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E
     cudaError_t rc;
     if (logits_dtype == 0)
         rc = launch_kernel(moe_topk_gating_kernel<0>, dim3(T), dim3(kGateThreads), smem, s, logits, ld_logits, E, k,
-                           normalize, bias, scale, clear, scores, expert_ids, offsets, counts);
+                           normalize, sigmoid, bias, scale, clear, scores, expert_ids, offsets, counts);
     else if (logits_dtype == 1)
         rc = launch_kernel(moe_topk_gating_kernel<1>, dim3(T), dim3(kGateThreads), smem, s, logits, ld_logits, E, k,
-                           normalize, bias, scale, clear, scores, expert_ids, offsets, counts);
+                           normalize, sigmoid, bias, scale, clear, scores, expert_ids, offsets, counts);
     else
         rc = launch_kernel(moe_topk_gating_kernel<2>, dim3(T), dim3(kGateThreads), smem, s, logits, ld_logits, E, k,
-                           normalize, bias, scale, clear, scores, expert_ids, offsets, counts);
+                           normalize, sigmoid, bias, scale, clear, scores, expert_ids, offsets, counts);
     HDS_CHECK_CUDA(rc);
     return HDS_OK;
 }
 
 extern "C" int hds_moe_scatter(const void* x, int64_t ldx, void* xs, int64_t ld_xs, const int32_t* expert_ids,
                                const int32_t* offsets, int32_t* counts, int32_t* pad_off, int32_t* mapped_slots, int T,
-                               int E, int k, int H, void* stream) {
+                               int E, int k, int H, const float* scores, int dtype, void* stream) {
     HDS_REQUIRE(H % 8 == 0 && ldx % 8 == 0 && ld_xs % 8 == 0, "hds_moe_scatter: H and strides must be multiples of 8");
     if (T == 0) return HDS_OK;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     HDS_CHECK_CUDA(launch_kernel(moe_offsets_kernel, dim3(1), dim3(32), 0, s, counts, pad_off, E));
-    HDS_CHECK_CUDA(launch_kernel(moe_scatter_kernel, dim3(T, k), dim3(H / 8 >= 256 ? 256 : 128), 0, s, x, ldx, xs, ld_xs,
-                                 expert_ids, offsets, static_cast<const int32_t*>(pad_off), mapped_slots, H, k));
+    const dim3 grid(T, k), block(H / 8 >= 256 ? 256 : 128);
+    const int32_t* off = pad_off;
+    if (scores == nullptr)
+        HDS_CHECK_CUDA(launch_kernel(moe_scatter_kernel, grid, block, 0, s, x, ldx, xs, ld_xs, expert_ids, offsets, off, mapped_slots, H, k));
+    else if (dtype == 0)
+        HDS_CHECK_CUDA(launch_kernel(moe_scatter_scaled_kernel<0>, grid, block, 0, s, x, ldx, xs, ld_xs, expert_ids, offsets, off, scores, mapped_slots, H, k));
+    else if (dtype == 1)
+        HDS_CHECK_CUDA(launch_kernel(moe_scatter_scaled_kernel<1>, grid, block, 0, s, x, ldx, xs, ld_xs, expert_ids, offsets, off, scores, mapped_slots, H, k));
+    else
+        HDS_CHECK_CUDA(launch_kernel(moe_scatter_scaled_kernel<2>, grid, block, 0, s, x, ldx, xs, ld_xs, expert_ids, offsets, off, scores, mapped_slots, H, k));
     return HDS_OK;
 }
 

@@ -5,6 +5,8 @@
 //                   the stream is RMS-normed for the next sublayer:
 //                       x += f d / rms(f d) * post;   out = x / rms(x) * gamma
 //                   (no post weight: x += f d). One CTA per row; the row stays in registers between the two reductions.
+//                   A second output may be normed, weighted and added in the same pass; the stream's norm may be taken over
+//                   equal consecutive parts of a row, each by itself.
 //   gated_norm    : out = rms(y * silu(z)) * weight * scale over `groups` equal parts of a row (state-space mixers), or
 //                   rms(y) * weight * scale * silu(z) (delta rules)
 //   embed_f32     : embedding rows into the fp32 stream, optionally RMS-normed on the way
@@ -49,30 +51,40 @@ __device__ __forceinline__ void store4(void* base, int64_t idx, float4 v) {
 }
 
 // `cols`: values a row's mean is taken over; `padded` >= cols: row width, zeros behind the values. DELTA 0 none, 1 fp32
-// (cleared after being read), 2 the output's type.
-template <int THREADS, int VPT, int DT, int DELTA, bool kPost>
+// (cleared after being read), 2 the output's type. kTwo: a second output of the same kind. groups > 1: the last norm is taken over
+// that many equal parts of the `cols` values (dynamic shared memory: groups * (THREADS / 32 + 1) floats).
+template <int THREADS, int VPT, int DT, int DELTA, bool kPost, bool kTwo>
 __global__ void __launch_bounds__(THREADS)
 norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const float* __restrict__ post,
                      const float* __restrict__ gamma, void* __restrict__ out, int64_t ld, int cols, int padded, float eps,
-                     int store_x) {
+                     int store_x, int groups, void* delta2, const float* __restrict__ post2) {
     __shared__ float red[THREADS / 32];
+    extern __shared__ float group_s[];
     pdl_enter();
     const int64_t row = static_cast<int64_t>(blockIdx.x) * ld;
     const int nvec = padded >> 2;
-    float4 v[VPT], d[VPT];
-    float ss = 0.0f;
+    float4 v[VPT], d[VPT], d2[kTwo ? VPT : 1];
+    float ss = 0.0f, ss2 = 0.0f;
+    auto take = [&](void* from, int c) {
+        if constexpr (DELTA == 1) {
+            float4* p = reinterpret_cast<float4*>(reinterpret_cast<float*>(from) + row + 4 * c);
+            const float4 q = *p;
+            *p = make_float4(0.f, 0.f, 0.f, 0.f);
+            return q;
+        } else {
+            return load4<DT>(from, row + 4 * c);
+        }
+    };
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
         const int c = threadIdx.x + i * THREADS;
         v[i] = d[i] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (c < nvec) {
             v[i] = *reinterpret_cast<const float4*>(x + row + 4 * c);
-            if constexpr (DELTA == 1) {
-                float4* p = reinterpret_cast<float4*>(reinterpret_cast<float*>(delta) + row + 4 * c);
-                d[i] = *p;
-                *p = make_float4(0.f, 0.f, 0.f, 0.f);
-            } else if constexpr (DELTA == 2) {
-                d[i] = load4<DT>(delta, row + 4 * c);
+            if constexpr (DELTA != 0) d[i] = take(delta, c);
+            if constexpr (kTwo) {
+                d2[i] = take(delta2, c);
+                ss2 += d2[i].x * d2[i].x + d2[i].y * d2[i].y + d2[i].z * d2[i].z + d2[i].w * d2[i].w;
             }
             if constexpr (DELTA != 0) {
                 d[i].x *= factor; d[i].y *= factor; d[i].z *= factor; d[i].w *= factor;
@@ -83,6 +95,8 @@ norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const flo
     if constexpr (DELTA != 0) {
         float r = 1.0f;
         if constexpr (kPost) r = 1.0f / sqrtf(block_sum_t<THREADS>(ss, red) / cols + eps);
+        float r2 = 0.0f;
+        if constexpr (kTwo) r2 = 1.0f / sqrtf(block_sum_t<THREADS>(ss2, red) / cols + eps);
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
             const int c = threadIdx.x + i * THREADS;
@@ -91,9 +105,49 @@ norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const flo
                 if constexpr (kPost) w = *reinterpret_cast<const float4*>(post + 4 * c);
                 v[i].x += d[i].x * r * w.x; v[i].y += d[i].y * r * w.y;
                 v[i].z += d[i].z * r * w.z; v[i].w += d[i].w * r * w.w;
+                if constexpr (kTwo) {
+                    const float4 u = *reinterpret_cast<const float4*>(post2 + 4 * c);
+                    v[i].x += d2[i].x * r2 * u.x; v[i].y += d2[i].y * r2 * u.y;
+                    v[i].z += d2[i].z * r2 * u.z; v[i].w += d2[i].w * r2 * u.w;
+                }
                 if (store_x) *reinterpret_cast<float4*>(x + row + 4 * c) = v[i];
             }
         }
+    }
+    if (groups > 1) {
+        const int part = cols / groups, warp = threadIdx.x >> 5;
+        float* r_s = group_s + groups * (THREADS / 32);
+        for (int g = 0; g < groups; ++g) {
+            const int g0 = g * part, g1 = g0 + part;
+            float s = 0.0f;
+#pragma unroll
+            for (int i = 0; i < VPT; ++i) {
+                const int e = 4 * (threadIdx.x + i * THREADS);
+                if (e + 3 < g0 || e >= g1) continue;
+                s += (e >= g0 ? v[i].x * v[i].x : 0.0f) + (e + 1 >= g0 && e + 1 < g1 ? v[i].y * v[i].y : 0.0f) +
+                     (e + 2 >= g0 && e + 2 < g1 ? v[i].z * v[i].z : 0.0f) + (e + 3 < g1 ? v[i].w * v[i].w : 0.0f);
+            }
+            s = warp_sum(s);
+            if ((threadIdx.x & 31) == 0) group_s[g * (THREADS / 32) + warp] = s;
+        }
+        __syncthreads();
+        for (int g = threadIdx.x; g < groups; g += THREADS) {
+            float s = 0.0f;
+            for (int w = 0; w < THREADS / 32; ++w) s += group_s[g * (THREADS / 32) + w];
+            r_s[g] = 1.0f / sqrtf(s / part + eps);
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) {
+            const int c = threadIdx.x + i * THREADS, e = 4 * c;
+            if (c < nvec) {
+                const float4 w = *reinterpret_cast<const float4*>(gamma + e);
+                auto of = [&](int x) { return r_s[min(x / part, groups - 1)]; };    // (past the values: zeros)
+                store4<DT>(out, row + e, make_float4(v[i].x * of(e) * w.x, v[i].y * of(e + 1) * w.y, v[i].z * of(e + 2) * w.z,
+                                                     v[i].w * of(e + 3) * w.w));
+            }
+        }
+        return;
     }
     ss = 0.0f;
 #pragma unroll
@@ -109,13 +163,15 @@ norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const flo
     }
 }
 
-template <int DT, int DELTA, bool kPost>
+template <int DT, int DELTA, bool kPost, bool kTwo = false>
 static int launch_norm_residual(float* x, void* delta, float factor, const float* post, const float* gamma, void* out, int64_t ld,
-                                int rows, int cols, int padded, float eps, int store_x, cudaStream_t s) {
+                                int rows, int cols, int padded, float eps, int store_x, int groups, void* delta2, const float* post2,
+                                cudaStream_t s) {
     const int nvec = padded / 4;
 #define HDS_NR(TH, V)                                                                                                       \
-    HDS_CHECK_CUDA(launch_kernel(norm_residual_kernel<TH, V, DT, DELTA, kPost>, dim3(rows), dim3(TH), 0, s, x, delta, factor, post, \
-                                 gamma, out, ld, cols, padded, eps, store_x))
+    HDS_CHECK_CUDA(launch_kernel(norm_residual_kernel<TH, V, DT, DELTA, kPost, kTwo>, dim3(rows), dim3(TH),                        \
+                                 groups > 1 ? sizeof(float) * groups * (TH / 32 + 1) : 0, s, x, delta, factor, post, gamma, out, ld, \
+                                 cols, padded, eps, store_x, groups, delta2, post2))
     if (nvec <= 128) HDS_NR(128, 1);
     else if (nvec <= 256) HDS_NR(256, 1);
     else if (nvec <= 512) HDS_NR(512, 1);
@@ -241,14 +297,15 @@ gated_norm_kernel(const float* __restrict__ y, int64_t ld_y, const void* __restr
 }
 
 template <int DT>
-__global__ void embed_f32_kernel(const int32_t* __restrict__ ids, const void* __restrict__ W, float* __restrict__ out, int H, int vocab) {
+__global__ void embed_f32_kernel(const int32_t* __restrict__ ids, const void* __restrict__ W, float* __restrict__ out, int H, int vocab, float scale) {
     pdl_enter();
     const int64_t t = blockIdx.x;
     const int id = ids[t];
     const bool ok = id >= 0 && id < vocab;
-    for (int c = threadIdx.x * 4; c < H; c += blockDim.x * 4)
-        *reinterpret_cast<float4*>(out + t * H + c) =
-            ok ? load4<DT>(W, static_cast<int64_t>(id) * H + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int c = threadIdx.x * 4; c < H; c += blockDim.x * 4) {
+        const float4 v = ok ? load4<DT>(W, static_cast<int64_t>(id) * H + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        *reinterpret_cast<float4*>(out + t * H + c) = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+    }
 }
 
 // the same, each row then divided by its root mean square over `cols` and weighted
@@ -279,18 +336,23 @@ embed_norm_f32_kernel(const int32_t* __restrict__ ids, const void* __restrict__ 
 using namespace hds;
 
 extern "C" int hds_norm_residual(float* x, void* delta, int delta_is_f32, float factor, const float* post, const float* gamma,
-                                 void* out, int64_t ld, int rows, int cols, int padded, float eps, int store_x, int dtype,
-                                 void* stream) {
+                                 void* out, int64_t ld, int rows, int cols, int padded, float eps, int store_x, int groups, void* delta2,
+                                 const float* post2, int dtype, void* stream) {
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_norm_residual: dtype 0 bf16 / 1 fp16 / 2 fp32");
     HDS_REQUIRE(padded % 4 == 0 && ld % 4 == 0 && cols <= padded && padded <= ld, "hds_norm_residual: rows of 4-value vectors");
+    HDS_REQUIRE(groups >= 1 && groups <= 256 && cols % groups == 0, "hds_norm_residual: 1..256 equal parts");
+    HDS_REQUIRE(delta2 == nullptr || (delta != nullptr && post != nullptr && post2 != nullptr),
+                "hds_norm_residual: a second output comes behind a first one, both with weights");
     if (rows == 0) return HDS_OK;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     const int mode = delta == nullptr ? 0 : delta_is_f32 ? 1 : 2;
-#define HDS_NR_ARGS x, delta, factor, post, gamma, out, ld, rows, cols, padded, eps, store_x, s
+#define HDS_NR_ARGS x, delta, factor, post, gamma, out, ld, rows, cols, padded, eps, store_x, groups, delta2, post2, s
 #define HDS_NR_DT(DT)                                                                               \
     return mode == 0         ? launch_norm_residual<DT, 0, false>(HDS_NR_ARGS)                       \
            : post == nullptr ? (mode == 1 ? launch_norm_residual<DT, 1, false>(HDS_NR_ARGS)          \
                                           : launch_norm_residual<DT, 2, false>(HDS_NR_ARGS))         \
+           : delta2 != nullptr ? (mode == 1 ? launch_norm_residual<DT, 1, true, true>(HDS_NR_ARGS)   \
+                                            : launch_norm_residual<DT, 2, true, true>(HDS_NR_ARGS))  \
            : mode == 1       ? launch_norm_residual<DT, 1, true>(HDS_NR_ARGS)                        \
                              : launch_norm_residual<DT, 2, true>(HDS_NR_ARGS)
     if (dtype == 0) { HDS_NR_DT(0); }
@@ -326,19 +388,20 @@ extern "C" int hds_gated_norm(const float* y, int64_t ld_y, const void* z, int64
 }
 
 extern "C" int hds_embed_f32(const int32_t* ids, const void* W, const float* gamma, float* out, int T, int H, int vocab, int cols, float eps,
-                             int dtype, void* stream) {
+                             float scale, int dtype, void* stream) {
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_embed_f32: dtype 0 bf16 / 1 fp16 / 2 fp32");
     HDS_REQUIRE(H % 4 == 0, "hds_embed_f32: rows of 4-value vectors");
     if (T == 0) return HDS_OK;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
+    HDS_REQUIRE(gamma == nullptr || scale == 1.0f, "hds_embed_f32: a norm or a factor");
     if (gamma != nullptr) {
         if (dtype == 0) HDS_CHECK_CUDA(launch_kernel(embed_norm_f32_kernel<0>, dim3(T), dim3(256), 0, s, ids, W, gamma, out, H, vocab, cols, eps));
         else if (dtype == 1) HDS_CHECK_CUDA(launch_kernel(embed_norm_f32_kernel<1>, dim3(T), dim3(256), 0, s, ids, W, gamma, out, H, vocab, cols, eps));
         else HDS_CHECK_CUDA(launch_kernel(embed_norm_f32_kernel<2>, dim3(T), dim3(256), 0, s, ids, W, gamma, out, H, vocab, cols, eps));
         return HDS_OK;
     }
-    if (dtype == 0) HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<0>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab));
-    else if (dtype == 1) HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<1>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab));
-    else HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<2>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab));
+    if (dtype == 0) HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<0>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab, scale));
+    else if (dtype == 1) HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<1>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab, scale));
+    else HDS_CHECK_CUDA(launch_kernel(embed_f32_kernel<2>, dim3(T), dim3(256), 0, s, ids, W, out, H, vocab, scale));
     return HDS_OK;
 }

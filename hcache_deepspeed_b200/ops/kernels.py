@@ -18,9 +18,9 @@ import torch
 
 from . import native
 
-ACT_IDENTITY, ACT_GELU, ACT_RELU, ACT_SILU, ACT_GELU_TANH, ACT_SWIGLU_CLAMPED = 0, 1, 2, 3, 4, 5
+ACT_IDENTITY, ACT_GELU, ACT_RELU, ACT_SILU, ACT_GELU_TANH, ACT_SWIGLU_CLAMPED, ACT_RELU2 = 0, 1, 2, 3, 4, 5, 6
 ACT_CODES = {"identity": 0, None: 0, "gelu": 1, "relu": 2, "silu": 3, "gelu_tanh": 4, "gelu_new": 4,
-             "gelu_pytorch_tanh": 4, "swish": 3, "swiglu_clamped": 5}
+             "gelu_pytorch_tanh": 4, "swish": 3, "swiglu_clamped": 5, "relu2": 6}
 
 EPI_STORE, EPI_GATED, EPI_ACCUM = 0, 1, 2
 
@@ -131,8 +131,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, 
         out = torch.empty((M, n_out), dtype=a.dtype, device=a.device)
     _check_2d(out, "out")
     if a.dtype == torch.float32:
-        assert bias is None
-        return _gemm_f32(a, w, out, EPI_GATED if gated else EPI_STORE, act, limit)
+        return _gemm_f32(a, w, out, EPI_GATED if gated else EPI_STORE, act, limit, bias=bias)
     lib = native.cuda_lib()
     if act == ACT_SWIGLU_CLAMPED:
         native.check(lib.hds_gemm_next_act_limit(limit), "hds_gemm_next_act_limit")
@@ -145,12 +144,12 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, 
 
 
 def _gemm_f32(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, act: int, limit: float,
-              group_off: Optional[torch.Tensor] = None, n_groups: int = 0) -> torch.Tensor:
+              group_off: Optional[torch.Tensor] = None, n_groups: int = 0, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     M, K = a.shape
     N = w.shape[0] // max(1, n_groups)
     assert w.dtype == torch.float32 and w.shape[1] == K and out.dtype == torch.float32
     rc = native.cuda_lib().hds_gemm_f32(_p(a), a.stride(0), _p(w), w.stride(0), M, N, K, epilogue, act, limit, _p(out), out.stride(0),
-                                        _p(group_off), n_groups, _stream())
+                                        _p(group_off), n_groups, _p(bias), _stream())
     native.check(rc, "hds_gemm_f32")
     _count()
     return out
@@ -167,8 +166,8 @@ def gemm_accum(a: torch.Tensor, w: torch.Tensor, accum: torch.Tensor, bias: Opti
     N = w.shape[0]
     assert accum.dtype == torch.float32 and accum.stride(-1) == 1
     if a.dtype == torch.float32:
-        assert bias is None and peer_ptrs is None and multicast_ptr is None
-        _gemm_f32(a, w, accum, EPI_ACCUM, ACT_IDENTITY, 0.0)
+        assert peer_ptrs is None and multicast_ptr is None
+        _gemm_f32(a, w, accum, EPI_ACCUM, ACT_IDENTITY, 0.0, bias=bias)
         return
     wp, ldw = _w(w)
     if multicast_ptr is not None:
@@ -402,9 +401,18 @@ def splitkv_workspace_bytes(n_items: int, n_q_heads: int, n_kv_heads: int, head_
 
 
 def _arm_alibi(lib, alibi: Optional[torch.Tensor], n_q_heads: int, window: int = 0, keep_first: int = 0,
-               out: Optional[torch.Tensor] = None) -> None:
+               out: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, sigmoid_bias: Optional[torch.Tensor] = None,
+               gate: Optional[torch.Tensor] = None) -> None:
     """Options of the next attention launch of this thread, consumed by that launch: ALiBi slopes, sliding window and kept
-    first tokens, and the stride of ``out`` when its rows (``[T, n_q_heads * head_dim]``) are not dense."""
+    first tokens, the stride of ``out`` when its rows (``[T, n_q_heads * head_dim]``) are not dense, softmax sinks, the biases of
+    sigmoid weights, the output gate."""
+    for t, fn in ((sink, "hds_attention_next_sink"), (sigmoid_bias, "hds_attention_next_sigmoid")):
+        if t is not None:
+            assert t.dtype == torch.float32 and t.is_cuda and t.is_contiguous() and t.numel() == n_q_heads
+            native.check(getattr(lib, fn)(_p(t)), fn)
+    if gate is not None:
+        _check_2d(gate, "gate")
+        native.check(lib.hds_attention_next_gate(_p(gate), gate.stride(0)), "hds_attention_next_gate")
     if keep_first:
         native.check(lib.hds_attention_next_keep_first(int(keep_first)), "hds_attention_next_keep_first")
     if out is not None and out.dim() == 2 and out.stride(0) != out.shape[1]:
@@ -421,12 +429,14 @@ def paged_attention_splitkv(q: torch.Tensor, out: torch.Tensor, kv_cache_layer: 
                             block_tables: torch.Tensor, items: torch.Tensor, n_items: int, rows_per_item: int,
                             n_q_heads: int, n_kv_heads: int, head_dim: int, block_size: int, n_splits: int,
                             scale: float, workspace: Optional[torch.Tensor], alibi: Optional[torch.Tensor] = None,
-                            window: int = 0, keep_first: int = 0) -> None:
+                            window: int = 0, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
+                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """kv_cache_layer: [blocks, 2, kvh, bs, d]; items: int32 [n, 4] = (seq, q_row0, n_q, pos0). ``alibi``: fp32 [n_q_heads]
     slopes; score += slope * (key position - query position). ``window``: sliding-window attention, keys (p - window, p] and
-    the first ``keep_first`` ones."""
+    the first ``keep_first`` ones. ``sink``, ``sigmoid_bias`` (fp32 [n_q_heads]) and ``gate`` (rows like ``out``'s): see
+    ``hds_attention_next_sink``."""
     lib = native.cuda_lib()
-    _arm_alibi(lib, alibi, n_q_heads, window, keep_first, out)
+    _arm_alibi(lib, alibi, n_q_heads, window, keep_first, out, sink, sigmoid_bias, gate)
     rc = lib.hds_paged_attention_splitkv(_p(q), _p(out), _p(kv_cache_layer), kv_cache_layer.shape[0], _p(block_tables),
                                          block_tables.stride(0), _p(items), n_items, rows_per_item, n_q_heads,
                                          n_kv_heads, head_dim, block_size, n_splits, scale, _p(workspace),
@@ -444,12 +454,13 @@ def paged_attention_prefill(q: torch.Tensor, out: torch.Tensor, kv_cache_layer: 
                             block_tables: torch.Tensor, items: torch.Tensor, n_items: int, n_q_heads: int,
                             n_kv_heads: int, head_dim: int, block_size: int, scale: float, n_splits: int = 1,
                             workspace: Optional[torch.Tensor] = None, packed: bool = False,
-                            alibi: Optional[torch.Tensor] = None, window: int = 0, keep_first: int = 0) -> None:
+                            alibi: Optional[torch.Tensor] = None, window: int = 0, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
+                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """tcgen05 paged attention. ``packed``: grouped-query decode form — one CTA per (item, KV head) whose MMA rows are
     the group's (token, query head) pairs (``hds_paged_attention_packed``). ``alibi``: fp32 [n_q_heads] slopes;
     ``window``: sliding-window attention."""
     lib = native.cuda_lib()
-    _arm_alibi(lib, alibi, n_q_heads, window, keep_first, out)
+    _arm_alibi(lib, alibi, n_q_heads, window, keep_first, out, sink, sigmoid_bias, gate)
     fn = lib.hds_paged_attention_packed if packed else lib.hds_paged_attention_prefill
     rc = fn(_p(q), _p(out), _p(kv_cache_layer), kv_cache_layer.shape[0], _p(block_tables),
                                          block_tables.stride(0), _p(items), n_items, q.shape[0], n_q_heads, n_kv_heads,
@@ -470,12 +481,12 @@ def moe_padded_rows(n_tokens: int, n_experts: int, top_k: int) -> int:
 
 def moe_topk_gating(logits: torch.Tensor, top_k: int, normalize: bool, scores: torch.Tensor, expert_ids: torch.Tensor,
                     offsets: torch.Tensor, counts: torch.Tensor, bias: Optional[torch.Tensor] = None, scale: float = 1.0,
-                    clear: bool = False) -> None:
-    """Softmax + top-k per token; ``counts`` (int32 [E], zero on entry) is incremented per assignment. ``bias`` (fp32 [E]) is added
+                    clear: bool = False, sigmoid: bool = False) -> None:
+    """Softmax (or ``sigmoid``) + top-k per token; ``counts`` (int32 [E], zero on entry) is incremented per assignment. ``bias`` (fp32 [E]) is added
     to the scores that choose, ``scale`` multiplies the scores returned, ``clear`` zeroes (fp32) logits once read."""
     T, E = logits.shape
     code = 2 if logits.dtype == torch.float32 else _dt(logits)
-    rc = native.cuda_lib().hds_moe_topk_gating(_p(logits), logits.stride(0), T, E, top_k, int(normalize), _p(bias), scale,
+    rc = native.cuda_lib().hds_moe_topk_gating(_p(logits), logits.stride(0), T, E, top_k, int(normalize), int(sigmoid), _p(bias), scale,
                                                  int(clear), code, _p(scores),
                                                _p(expert_ids), _p(offsets), _p(counts), _stream())
     native.check(rc, "hds_moe_topk_gating")
@@ -483,14 +494,15 @@ def moe_topk_gating(logits: torch.Tensor, top_k: int, normalize: bool, scores: t
 
 
 def moe_scatter(x: torch.Tensor, xs: torch.Tensor, expert_ids: torch.Tensor, offsets: torch.Tensor, counts: torch.Tensor,
-                pad_off: torch.Tensor, mapped_slots: torch.Tensor, top_k: int) -> None:
-    """Build ``pad_off`` (int32 [E+1]) from ``counts`` (re-zeroed) and copy every token row to its k expert rows."""
+                pad_off: torch.Tensor, mapped_slots: torch.Tensor, top_k: int, scores: Optional[torch.Tensor] = None) -> None:
+    """Build ``pad_off`` (int32 [E+1]) from ``counts`` (re-zeroed) and copy every token row, times its ``scores`` if given, to its k
+    expert rows."""
     T, H = x.shape
     E = counts.numel()
     r = x.element_size() // 2      # the kernel moves 16-bit units
     H *= r
     rc = native.cuda_lib().hds_moe_scatter(_p(x), x.stride(0) * r, _p(xs), xs.stride(0) * r, _p(expert_ids), _p(offsets), _p(counts),
-                                           _p(pad_off), _p(mapped_slots), T, E, top_k, H, _stream())
+                                           _p(pad_off), _p(mapped_slots), T, E, top_k, H, _p(scores), _dt3(x), _stream())
     native.check(rc, "hds_moe_scatter")
     _count(2)
 
@@ -627,10 +639,10 @@ def moe_table_route(ids: torch.Tensor, table: torch.Tensor, n_experts: int, scor
     _count()
 
 
-def moe_combine(y: torch.Tensor, mapped_slots: torch.Tensor, scores: torch.Tensor, base: Optional[torch.Tensor],
+def moe_combine(y: torch.Tensor, mapped_slots: torch.Tensor, scores: Optional[torch.Tensor], base: Optional[torch.Tensor],
                 out: torch.Tensor) -> torch.Tensor:
     """``out[t] = base[t] + sum_j scores[t, j] * y[mapped_slots[t, j]]`` (``out`` fp32, stored; ``base`` optional, or ``out``
-    itself: added in place)."""
+    itself: added in place; ``scores`` None: ones)."""
     T, k = mapped_slots.shape
     assert out.dtype == torch.float32
     accumulate = base is not None and base.data_ptr() == out.data_ptr()
@@ -646,11 +658,11 @@ def moe_combine(y: torch.Tensor, mapped_slots: torch.Tensor, scores: torch.Tenso
 
 
 def embed_f32(ids: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gamma: Optional[torch.Tensor] = None,
-              cols: Optional[int] = None, eps: float = 1e-5) -> torch.Tensor:
-    """Embedding rows in fp32; with ``gamma`` RMS-normed over their first ``cols`` values and weighted."""
+              cols: Optional[int] = None, eps: float = 1e-5, scale: float = 1.0) -> torch.Tensor:
+    """Embedding rows in fp32, times ``scale``; with ``gamma`` RMS-normed over their first ``cols`` values and weighted instead."""
     assert ids.dtype == torch.int32 and out.dtype == torch.float32
     rc = native.cuda_lib().hds_embed_f32(_p(ids), _p(weight), _p(gamma), _p(out), ids.numel(), weight.shape[1], weight.shape[0],
-                                         weight.shape[1] if cols is None else cols, eps, _dt3(weight), _stream())
+                                         weight.shape[1] if cols is None else cols, eps, scale, _dt3(weight), _stream())
     native.check(rc, "hds_embed_f32")
     _count()
     return out
@@ -658,15 +670,18 @@ def embed_f32(ids: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gamma:
 
 def norm_residual(resid: torch.Tensor, gamma: torch.Tensor, out: torch.Tensor, delta: Optional[torch.Tensor] = None,
                   factor: float = 1.0, post: Optional[torch.Tensor] = None, cols: Optional[int] = None, eps: float = 1e-5,
-                  store_resid: bool = True) -> torch.Tensor:
-    """``resid += norm(factor * delta) * post`` (without ``post``: ``resid += factor * delta``) on the fp32 stream,
-    ``out = norm(resid) * gamma`` (``hds_norm_residual``)."""
+                  store_resid: bool = True, groups: int = 1, delta2: Optional[torch.Tensor] = None,
+                  post2: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``resid += norm(factor * delta) * post`` (without ``post``: ``resid += factor * delta``), ``+= norm(delta2) * post2`` on the
+    fp32 stream, ``out = norm(resid) * gamma``, that norm over each of ``groups`` equal parts of a row (``hds_norm_residual``)."""
     rows, width = resid.shape
     assert resid.stride(0) == out.stride(0) and (delta is None or delta.stride(0) == resid.stride(0))
     assert delta is None or delta.dtype in (torch.float32, out.dtype)
+    assert delta2 is None or (delta2.dtype == delta.dtype and delta2.stride(0) == resid.stride(0))
     rc = native.cuda_lib().hds_norm_residual(_p(resid), _p(delta), 1 if (delta is not None and delta.dtype == torch.float32) else 0,
                                              factor, _p(post), _p(gamma), _p(out), resid.stride(0), rows,
-                                             width if cols is None else cols, width, eps, 1 if store_resid else 0, _dt3(out), _stream())
+                                             width if cols is None else cols, width, eps, 1 if store_resid else 0, groups, _p(delta2), _p(post2),
+                                             _dt3(out), _stream())
     native.check(rc, "hds_norm_residual")
     _count()
     return out
@@ -706,9 +721,11 @@ def state_space(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, 
 def paged_attention_generic(q: torch.Tensor, out: torch.Tensor, kv_cache_layer: torch.Tensor, block_tables: torch.Tensor,
                             tok_seq: torch.Tensor, tok_pos: torch.Tensor, n_q_heads: int, n_kv_heads: int, head_dim: int,
                             block_size: int, scale: float, window: int = 0, keep_first: int = 0, value_dim: int = 0,
-                            spans: Optional[torch.Tensor] = None, limit: int = 0) -> None:
+                            spans: Optional[torch.Tensor] = None, limit: int = 0, sink: Optional[torch.Tensor] = None,
+                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """fp32-arithmetic attention for any operand type and head size (``hds_paged_attention_generic``). ``value_dim`` > 0: pages of
     one plane, the first ``value_dim`` values of a key row are its value. ``spans``: skip sequences of more than ``limit`` tokens."""
+    _arm_alibi(native.cuda_lib(), None, n_q_heads, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate)
     rc = native.cuda_lib().hds_paged_attention_generic(_p(q), _p(out), out.stride(0), _p(kv_cache_layer), _p(block_tables),
                                                        block_tables.stride(0), _p(tok_seq), _p(tok_pos), q.shape[0], n_q_heads,
                                                        n_kv_heads, head_dim, block_size, scale, window, keep_first, value_dim, _p(spans),
@@ -802,3 +819,73 @@ def delta_rule(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, d
     if out is not None and n_single < spans.shape[0]:
         gated_norm(y, proj[:, :heads * vdim], norm_w, out, heads, eps, gate_after=True)
     return y
+
+
+# ------------------------------------------------------------------------------------------------
+# attention inputs, minGRU, gated linear attention
+# ------------------------------------------------------------------------------------------------
+def attention_append(qkv: torch.Tensor, q_out: torch.Tensor, kv_cache_layer: torch.Tensor, tok_pos: torch.Tensor, tok_slot: torch.Tensor,
+                     n_q_heads: int, n_kv_heads: int, head_dim: int, block_size: int, freq: Optional[torch.Tensor],
+                     q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None, q_cols: int = 0, k_cols: int = 0,
+                     eps: float = 0.0, first: Optional[torch.Tensor] = None, share: Optional[torch.Tensor] = None) -> None:
+    """Projected rows ``qkv`` = [q heads | k heads | v heads] -> normed and rotated queries, page rows with mixed values
+    (``hds_attention_append``)."""
+    _check_2d(qkv, "qkv")
+    assert kv_cache_layer.shape[4] == head_dim and kv_cache_layer.shape[3] == block_size
+    assert first is None or (first.shape[:4] == kv_cache_layer.shape[:4] and first.is_contiguous())
+    rc = native.cuda_lib().hds_attention_append(_p(qkv), qkv.stride(0), _p(q_out), _p(kv_cache_layer), _p(tok_pos), _p(tok_slot), qkv.shape[0],
+                                                n_q_heads, n_kv_heads, head_dim, block_size, _p(freq), _p(q_norm), _p(k_norm), q_cols, k_cols,
+                                                eps, _p(first), 0 if first is None else first.shape[4], _p(share), _dt3(qkv), _stream())
+    native.check(rc, "hds_attention_append")
+    _count()
+
+
+def mix_cached_values(kv_cache_layer: torch.Tensor, first: torch.Tensor, tok_slot: torch.Tensor, share: torch.Tensor, n_kv_heads: int,
+                      head_dim: int, block_size: int) -> None:
+    """The tokens' cached values become (1 - share) of themselves plus ``share`` of those in ``first``."""
+    assert first.shape[:4] == kv_cache_layer.shape[:4] and kv_cache_layer.shape[3] == block_size
+    rc = native.cuda_lib().hds_mix_cached_values(_p(kv_cache_layer), _p(first), first.shape[4], _p(tok_slot), _p(share), tok_slot.numel(),
+                                                 n_kv_heads, head_dim, block_size, _dt3(kv_cache_layer), _stream())
+    native.check(rc, "hds_mix_cached_values")
+    _count()
+
+
+def gru_workspace_bytes(n_tokens: int, n_seqs: int, width: int) -> int:
+    return int(native.cuda_lib().hds_gru_workspace_bytes(n_tokens, n_seqs, width))
+
+
+def gru(proj: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, spans: torch.Tensor, n_single: int, out: Optional[torch.Tensor],
+        workspace: Optional[torch.Tensor]) -> None:
+    """minGRU of ``proj`` = [z | u | output gate] over a ragged batch (``hds_gru``); ``state`` [slots, ..., width] fp32."""
+    _check_2d(proj, "proj")
+    width = bias.numel() // 2
+    assert proj.shape[1] == 3 * width and state[0].numel() == width
+    rc = native.cuda_lib().hds_gru(_p(proj), proj.stride(0), _p(bias), _p(state), _p(spans), spans.shape[0], n_single, proj.shape[0], width,
+                                   _p(out), 0 if out is None else out.stride(0), _p(workspace), 0 if workspace is None else workspace.numel(),
+                                   _dt3(proj), _stream())
+    native.check(rc, "hds_gru")
+    _count((3 if out is not None else 2) * (spans.shape[0] > n_single) + (n_single > 0))
+
+
+def linear_attention_workspace_bytes(n_tokens: int, n_seqs: int, heads: int, vdim: int, dim: int) -> int:
+    """Scratch of the chunked form for batches of up to ``n_tokens`` tokens in ``n_seqs`` sequences (0: not for this shape)."""
+    return int(native.cuda_lib().hds_linear_attention_workspace_bytes(n_tokens, n_seqs, heads, vdim, dim))
+
+
+def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, z: torch.Tensor, bias: torch.Tensor, inv_tau: float,
+                     state: torch.Tensor, spans: torch.Tensor, n_single: int, y: torch.Tensor, out: Optional[torch.Tensor],
+                     norm_w: torch.Tensor, eps: float, workspace: Optional[torch.Tensor] = None, method: int = SCAN_AUTO) -> None:
+    """Gated linear attention over a ragged batch, with the norm and gate behind (``hds_linear_attention``). ``state``
+    [slots, heads, vdim, dim] fp32; ``y`` fp32 scratch; ``out`` None: advance the state alone."""
+    T = q.shape[0]
+    _, heads, vdim, dim = state.shape
+    assert q.stride(0) == k.stride(0) == v.stride(0) == gate.stride(0) and bias.numel() == heads * dim
+    done = ctypes.c_int(1)
+    rc = native.cuda_lib().hds_linear_attention(_p(q), _p(k), _p(v), _p(gate), q.stride(0), _p(z), z.stride(0), _p(bias), inv_tau, _p(state),
+                                                _p(spans), spans.shape[0], n_single, T, heads, vdim, dim, _p(y), y.stride(0), _p(out),
+                                                0 if out is None else out.stride(0), _p(norm_w), eps, _p(workspace),
+                                                0 if workspace is None else workspace.numel(), method, ctypes.addressof(done), _dt3(q), _stream())
+    native.check(rc, "hds_linear_attention")
+    _count((3 if out is not None else 2) * (spans.shape[0] > n_single) + (n_single > 0))
+    if out is not None and not done.value:
+        gated_norm(y[:, :heads * vdim], gate[:, :heads * vdim], norm_w, out, heads, eps, gate_after=True)

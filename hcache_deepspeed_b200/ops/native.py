@@ -49,12 +49,19 @@ def _declare_cuda(lib: ctypes.CDLL, partial: bool = False) -> None:
         "hds_attention_next_out_stride": [L],
         "hds_paged_attention_generic": [P, P, L, P, P, I, P, P, I, I, I, I, I, F, I, I, I, P, I, I, P],
         "hds_kv_append_generic": [P, L, P, P, P, I, I, I, I, I, I, P],
-        "hds_gemm_f32": [P, L, P, L, I, I, I, I, I, F, P, L, P, I, P],
+        "hds_gemm_f32": [P, L, P, L, I, I, I, I, I, F, P, L, P, I, P, P],
+        "hds_attention_next_sink": [P],
+        "hds_attention_next_sigmoid": [P],
+        "hds_attention_next_gate": [P, L],
+        "hds_attention_append": [P, L, P, P, P, P, I, I, I, I, I, P, P, P, I, I, F, P, I, P, I, P],
+        "hds_mix_cached_values": [P, P, I, P, P, I, I, I, I, I, P],
+        "hds_gru": [P, L, P, P, P, I, I, I, I, P, L, P, L, I, P],
+        "hds_linear_attention": [P, P, P, P, L, P, L, P, F, P, P, I, I, I, I, I, I, P, L, P, L, P, F, P, L, I, P, I, P],
         "hds_gemm_next_act_limit": [F],
         "hds_moe_table_route": [P, P, I, I, I, I, P, P, P, P, P],
         "hds_moe_combine": [P, L, P, P, P, L, P, L, I, I, I, I, I, P],
-        "hds_embed_f32": [P, P, P, P, I, I, I, I, F, I, P],
-        "hds_norm_residual": [P, P, I, F, P, P, P, L, I, I, I, F, I, I, P],
+        "hds_embed_f32": [P, P, P, P, I, I, I, I, F, F, I, P],
+        "hds_norm_residual": [P, P, I, F, P, P, P, L, I, I, I, F, I, I, P, P, I, P],
         "hds_gated_norm": [P, L, P, L, P, P, L, I, I, I, F, F, I, I, P],
         "hds_state_space": [P, L, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, L, P, P, I, I, P],
         "hds_delta_rule": [P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, L, P, P, P, L, P, F, P, L, I, I, P],
@@ -84,8 +91,8 @@ def _declare_cuda(lib: ctypes.CDLL, partial: bool = False) -> None:
         "hds_paged_attention_splitkv": [P, P, P, L, P, I, P, I, I, I, I, I, I, I, F, P, L, I, P],
         "hds_paged_attention_prefill": [P, P, P, L, P, I, P, I, I, I, I, I, I, F, I, P, L, I, P],
         "hds_paged_attention_packed": [P, P, P, L, P, I, P, I, I, I, I, I, I, F, I, P, L, I, P],
-        "hds_moe_topk_gating": [P, L, I, I, I, I, P, F, I, I, P, P, P, P, P],
-        "hds_moe_scatter": [P, L, P, L, P, P, P, P, P, I, I, I, I, P],
+        "hds_moe_topk_gating": [P, L, I, I, I, I, I, P, F, I, I, P, P, P, P, P],
+        "hds_moe_scatter": [P, L, P, L, P, P, P, P, P, I, I, I, I, P, I, P],
         "hds_moe_gemm": [P, L, P, L, P, I, I, I, I, I, I, I, P, L, P],
         "hds_moe_gather": [P, L, P, P, P, L, I, I, I, I, P],
         "hds_gemm_2sm": [P, L, P, L, I, I, I, I, I, I, P, P, L, I, P],
@@ -115,6 +122,10 @@ def _declare_cuda(lib: ctypes.CDLL, partial: bool = False) -> None:
     lib.hds_paged_attention_latent_workspace_bytes.restype = c_int64
     lib.hds_delta_workspace_bytes.argtypes = [I, I, I, I]
     lib.hds_delta_workspace_bytes.restype = c_int64
+    lib.hds_gru_workspace_bytes.argtypes = [I, I, I]
+    lib.hds_gru_workspace_bytes.restype = c_int64
+    lib.hds_linear_attention_workspace_bytes.argtypes = [I, I, I, I, I]
+    lib.hds_linear_attention_workspace_bytes.restype = c_int64
     lib.hds_moe_padded_rows.argtypes = [I, I, I]
     lib.hds_moe_padded_rows.restype = c_int64
     # optional entry points (declared when present so older builds keep loading)

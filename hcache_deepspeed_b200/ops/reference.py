@@ -26,6 +26,8 @@ def apply_act(x: torch.Tensor, act: int) -> torch.Tensor:
         return F.silu(x)
     if act == 4:
         return F.gelu(x, approximate="tanh")
+    if act == 6:
+        return F.relu(x)**2
     return x
 
 
@@ -102,10 +104,13 @@ def gather_kv(kv_cache_layer: torch.Tensor, block_table_row: torch.Tensor, kv_le
 
 def paged_attention(q: torch.Tensor, kv_cache_layer: torch.Tensor, block_tables: torch.Tensor, items: torch.Tensor,
                     n_q_heads: int, n_kv_heads: int, scale: float, out: Optional[torch.Tensor] = None,
-                    alibi: Optional[torch.Tensor] = None, window: int = 0, keep_first: int = 0) -> torch.Tensor:
+                    alibi: Optional[torch.Tensor] = None, window: int = 0, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
+                    sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q: [T, n_q_heads, d]; items: int32 [n, 4] rows (seq, q_row0, n_q, pos0). Causal over absolute positions.
     ``alibi``: [n_q_heads] slopes, score += slope * (key position - query position). ``window`` > 0: a query at position p
-    sees the keys (p - window, p] only, and the first ``keep_first`` positions of its sequence."""
+    sees the keys (p - window, p] only, and the first ``keep_first`` positions of its sequence. ``sink`` [n_q_heads]: one more
+    score in every softmax, without a key. ``sigmoid_bias`` [n_q_heads]: weights are sigmoid(score + bias) instead, not
+    normalized. ``gate`` [T, n_q_heads * d]: the output is multiplied by its sigmoid."""
     T, _, d = q.shape
     if out is None:
         out = torch.zeros_like(q)
@@ -124,8 +129,16 @@ def paged_attention(q: torch.Tensor, kv_cache_layer: torch.Tensor, block_tables:
         s = s.masked_fill(kv_pos > q_pos, float("-inf"))
         if window:
             s = s.masked_fill((kv_pos <= q_pos - window) & (kv_pos >= keep_first), float("-inf"))
-        p = torch.softmax(s, dim=-1)
-        out[q_row0:q_row0 + n_q] = torch.einsum("hqk,khd->qhd", p, v).to(out.dtype)
+        if sigmoid_bias is not None:
+            p = torch.sigmoid(s + sigmoid_bias[:, None, None])
+        elif sink is not None:
+            p = torch.softmax(torch.cat([s, sink[:, None, None].expand(-1, n_q, 1)], dim=-1), dim=-1)[..., :-1]
+        else:
+            p = torch.softmax(s, dim=-1)
+        o = torch.einsum("hqk,khd->qhd", p, v)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[q_row0:q_row0 + n_q].float().reshape(o.shape))
+        out[q_row0:q_row0 + n_q] = o.to(out.dtype)
     return out
 
 
@@ -161,14 +174,26 @@ def attention_scale(head_dim: int) -> float:
 # fp32 residual stream with norms on both sides of a sublayer; state-space mixer; expert choice by table
 # ---------------------------------------------------------------------------------------------------
 def norm_residual(resid: torch.Tensor, gamma: torch.Tensor, delta: Optional[torch.Tensor], factor: float,
-                  post: Optional[torch.Tensor], cols: int, eps: float):
-    """Returns (new fp32 stream, normed stream): stream += rms(factor * delta) * post, then rms(stream) * gamma. Rows hold
-    ``cols`` values and zeros behind them. ``post`` None: stream += factor * delta."""
+                  post: Optional[torch.Tensor], cols: int, eps: float, groups: int = 1, delta2: Optional[torch.Tensor] = None,
+                  post2: Optional[torch.Tensor] = None):
+    """Returns (new fp32 stream, normed stream): stream += rms(factor * delta) * post (+ rms(delta2) * post2), then
+    rms(stream) * gamma, the latter over each of ``groups`` equal parts of a row. Rows hold ``cols`` values and zeros behind them.
+    ``post`` None: stream += factor * delta."""
+
+    def rms(d):
+        return d * torch.rsqrt((d * d).sum(-1, keepdim=True) / cols + eps)
+
     x = resid
     if delta is not None:
         d = delta.float() * factor
-        x = x + (d if post is None else d * torch.rsqrt((d * d).sum(-1, keepdim=True) / cols + eps) * post)
-    return x, x * torch.rsqrt((x * x).sum(-1, keepdim=True) / cols + eps) * gamma
+        x = x + (d if post is None else rms(d) * post)
+    if delta2 is not None:
+        x = x + rms(delta2.float()) * post2
+    if groups == 1:
+        return x, rms(x) * gamma
+    p = x[:, :cols].reshape(x.shape[0], groups, -1)
+    y = (p * torch.rsqrt((p * p).mean(-1, keepdim=True) + eps)).reshape(x.shape[0], cols)
+    return x, F.pad(y, (0, x.shape[1] - cols)) * gamma
 
 
 def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, scale: float = 1.0,
@@ -263,3 +288,62 @@ def paged_latent_attention(q: torch.Tensor, pages: torch.Tensor, block_tables: t
         s = s.masked_fill((back < 0) | (back >= (window or kv_len)), float("-inf"))
         out[row0:row0 + n] = torch.einsum("hqk,kd->qhd", torch.softmax(s, -1), rows[:, :rank]).to(out.dtype)
     return out
+
+
+def attention_append(qkv: torch.Tensor, kv_cache_layer: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, n_q: int, n_kv: int,
+                     freq: Optional[torch.Tensor], q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], q_cols: int, k_cols: int,
+                     eps: float, first: Optional[torch.Tensor], share: Optional[torch.Tensor]) -> torch.Tensor:
+    """What lies between a layer's projections ``qkv`` = [q heads | k heads | v heads] and its attention: all of q (k) normed over its
+    ``q_cols`` (``k_cols``) values, heads rotated by halves with the angles pos * freq, values mixed with those that the layer with
+    the pages ``first`` cached of the same tokens. K and V go to their pages; returns q, fp32 [T, n_q * D]."""
+    T, D = qkv.shape[0], kv_cache_layer.shape[4]
+    q, k, v = qkv[:, :(n_q + 2 * n_kv) * D].float().split([n_q * D, n_kv * D, n_kv * D], 1)
+
+    def normed(x, w, cols):
+        return x if w is None else x * torch.rsqrt((x * x).sum(-1, keepdim=True) / cols + eps) * w
+
+    def rotated(x):
+        return x if freq is None else rope_rotate_half(x, pos, freq, D)
+
+    q, k = normed(q, q_norm, q_cols).reshape(T, n_q, D), normed(k, k_norm, k_cols).reshape(T, n_kv, D)
+    v = v.reshape(T, n_kv, D)
+    if first is not None:
+        v = mixed_values(v, first, slot, share)
+    kv_append(kv_cache_layer, rotated(k), v, slot)
+    return rotated(q).reshape(T, n_q * D)
+
+
+def mixed_values(v: torch.Tensor, first: torch.Tensor, slot: torch.Tensor, share: torch.Tensor) -> torch.Tensor:
+    """v [T, n_kv, D] and the values of the same tokens in another layer's pages, by ``share``; widths may be padded differently."""
+    bs, s = first.shape[3], slot.long().clamp_min(0)
+    n = min(v.shape[2], first.shape[4])
+    other = F.pad(first[s // bs, 1, :, s % bs, :n].float(), (0, v.shape[2] - n))
+    return (1.0 - share) * v.float() + share * other
+
+
+def gru_scan(z: torch.Tensor, u: torch.Tensor, state: torch.Tensor) -> torch.Tensor:
+    """S <- (1 - sigmoid(z)) S + sigmoid(z) c for every token of one sequence, c = u + 1/2 where u >= 0, else sigmoid(u); z, u
+    [n, width], ``state`` [width] fp32 is advanced in place."""
+    z, u = torch.sigmoid(z.float()), u.float()
+    c = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+    out = torch.empty_like(z)
+    for t in range(z.shape[0]):
+        state.copy_((1.0 - z[t]) * state + z[t] * c[t])
+        out[t] = state
+    return out
+
+
+def linear_decay(z: torch.Tensor, tau: float) -> torch.Tensor:
+    """sigmoid(z)^(1 / tau)"""
+    return torch.exp(F.logsigmoid(z.float()) / tau)
+
+
+def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor) -> torch.Tensor:
+    """S <- S diag(decay) + v k^T, y = S q dim^-1/2 for every token of one sequence; q / k / decay [n, heads, N], v [n, heads, P];
+    ``state`` [heads, P, N] fp32 is advanced in place."""
+    y = torch.empty(v.shape, dtype=torch.float32)
+    q = q.float() * q.shape[2]**-0.5
+    for t in range(v.shape[0]):
+        state.mul_(decay[t][:, None, :]).add_(v[t].float()[:, :, None] * k[t].float()[:, None, :])
+        y[t] = (state * q[t][:, None, :]).sum(-1)
+    return y

@@ -245,6 +245,13 @@ int hds_attention_next_keep_first(int keep_first);
 /* Elements between the output rows of two tokens for the same launch (a multiple of 8; 0 = dense rows of n_q_heads * head_dim),
  * so that a layer's mixers can write side by side into one buffer. Cleared by that launch. */
 int hds_attention_next_out_stride(int64_t elements);
+/* Further options of the same launch (all three kernel families; device pointers, cleared by that launch):
+ *   sink    n_q_heads floats: one more score, without key or value and not scaled, in the denominator of every softmax
+ *   sigmoid n_q_heads floats: a visible key weighs sigmoid(score + bias[head]); weights are not normalized
+ *   gate    rows like the output's (operand type, ld elements apart): the output is multiplied by its sigmoid */
+int hds_attention_next_sink(const float* sink);
+int hds_attention_next_sigmoid(const float* bias);
+int hds_attention_next_gate(const void* gate, int64_t ld);
 
 /* Paged attention in plain fp32 arithmetic for operands and head sizes the tensor-core kernels do not take: dtype 0 bf16,
  * 1 fp16, 2 fp32, head_dim up to 512. One warp per (token, query head); tok_seq / tok_pos give each token's block-table row and
@@ -286,15 +293,16 @@ int64_t hds_paged_attention_prefill_workspace_bytes(int n_items, int n_q_heads, 
 /* ---- mixture of experts (tensor-parallel experts; ref ragged_ops/{top_k_gating,moe_scatter,moe_gather}, moe_gemm) --- */
 /* Per token: softmax over E logits, top-k (ties -> lower index), optional renormalisation of the k scores.
  * counts[E] must be zero on entry (hds_moe_scatter re-zeroes it). offsets[t, j] = row claimed inside expert_ids[t, j].
- * bias[E] (optional) is added to the softmax scores that choose, `scale` multiplies the returned ones, `clear` zeroes the (fp32)
- * logits after they are read. */
-int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E, int k, int normalize, const float* bias, float scale, int clear,
-                        int logits_dtype, float* scores, int32_t* expert_ids, int32_t* offsets, int32_t* counts, void* stream);
-/* pad_off[E+1]: expert row ranges rounded up to 128 rows; xs[row] = x[t] for every (t, j); mapped_slots[t, j] = row.
+ * bias[E] (optional) is added to the scores that choose, `scale` multiplies the returned ones, `clear` zeroes the (fp32)
+ * logits after they are read. `sigmoid`: the scores are the logits' sigmoids, each by itself. */
+int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E, int k, int normalize, int sigmoid, const float* bias, float scale,
+                        int clear, int logits_dtype, float* scores, int32_t* expert_ids, int32_t* offsets, int32_t* counts, void* stream);
+/* pad_off[E+1]: expert row ranges rounded up to 128 rows; xs[row] = x[t] for every (t, j); mapped_slots[t, j] = row. scores
+ * (optional): xs[row] = scores[t, j] * x[t] in the rows' type (dtype 0 / 1 / 2). H and strides count 16-bit units.
  * xs needs hds_moe_padded_rows(T, E, k) rows. */
 int hds_moe_scatter(const void* x, int64_t ldx, void* xs, int64_t ld_xs, const int32_t* expert_ids,
                     const int32_t* offsets, int32_t* counts, int32_t* pad_off, int32_t* mapped_slots, int T, int E, int k,
-                    int H, void* stream);
+                    int H, const float* scores, int dtype, void* stream);
 int64_t hds_moe_padded_rows(int T, int E, int k);
 /* Grouped tcgen05 GEMM: rows [pad_off[e], pad_off[e+1]) of A times W_stacked[e*N:(e+1)*N, :]^T; epilogue as hds_gemm
  * (no bias). max_rows = row capacity of A and out (multiple of 128). */
@@ -363,9 +371,9 @@ int hds_multi_tensor_lion(int n_tensors, void* const* params, const void* const*
 /* ---- fp32 models, expert choice by table, fp32 residual stream, state-space mixers ----------------------------------- */
 
 /* D[M,N] = A[M,K] * W[N,K]^T in true fp32. epilogue 0 store + act, 1 gated (interleaved gate / up rows, out has N/2 columns),
- * 2 out += D. group_off (optional, as hds_moe_gemm's pad_off): rows of group e use W[e*N:(e+1)*N]. limit: see below. */
+ * 2 out += D; bias (optional, plain rows): [N], added to D. group_off (optional, as hds_moe_gemm's pad_off): rows of group e use W[e*N:(e+1)*N]. limit: see below. */
 int hds_gemm_f32(const float* A, int64_t lda, const float* W, int64_t ldw, int M, int N, int K, int epilogue, int act, float limit,
-                 float* out, int64_t ldo, const int32_t* group_off, int n_groups, void* stream);
+                 float* out, int64_t ldo, const int32_t* group_off, int n_groups, const float* bias, void* stream);
 
 /* act = 5 of the gated epilogues of hds_gemm, hds_gemm_2sm, hds_moe_gemm and hds_gemm_f32 bounds its inputs:
  * g = min(gate, L), u = clamp(up, -L, L), out = g * sigmoid(1.702 g) * (u + 1). This sets L for the NEXT GEMM launch of the
@@ -375,23 +383,25 @@ int hds_gemm_next_act_limit(float limit);
 /* Expert choice by token id: expert_ids[t, j] = table[ids[t], j], scores = 1 / k; offsets / counts as hds_moe_topk_gating. */
 int hds_moe_table_route(const int32_t* ids, const int32_t* table, int vocab, int T, int E, int k, float* scores, int32_t* expert_ids,
                         int32_t* offsets, int32_t* counts, void* stream);
-/* out[t, :] = base[t, :] + sum_j scores[t, j] * y[mapped_slots[t, j], :] (stored; base optional; dtype of y and base 0 / 1 / 2;
+/* out[t, :] = base[t, :] + sum_j scores[t, j] * y[mapped_slots[t, j], :] (stored; base optional, scores too: 1; dtype of y and base 0 / 1 / 2;
  * accumulate: out itself is one more summand). */
 int hds_moe_combine(const void* y, int64_t ldy, const int32_t* mapped_slots, const float* scores, const void* base, int64_t ldb,
                     float* out, int64_t ldo, int T, int k, int H, int accumulate, int dtype, void* stream);
 
 /* out[t] = W[ids[t]] as fp32 (rows of H values; ids outside the vocabulary give zeros). dtype of W 0 / 1 / 2. gamma (optional): each
- * row is divided by its root mean square over `cols` values (eps inside the root) and weighted. */
+ * row is divided by its root mean square over `cols` values (eps inside the root) and weighted. Without: times scale. */
 int hds_embed_f32(const int32_t* ids, const void* W, const float* gamma, float* out, int T, int H, int vocab, int cols, float eps,
-                  int dtype, void* stream);
+                  float scale, int dtype, void* stream);
 
 /* One sublayer boundary of a stack on an fp32 residual stream x [rows, ld]:
  *   x += (factor * delta) / rms(factor * delta) * post   (delta NULL: skipped; post NULL: x += factor * delta)
  *   out = x / rms(x) * gamma
  * rms over the first `cols` values of a row (the rest of `padded` are zeros). An fp32 delta is cleared after being read; a
- * 16-bit one has out's dtype. store_x 0: x is only read. dtype of out 0 bf16, 1 fp16, 2 fp32. All rows ld apart. */
+ * 16-bit one has out's dtype. delta2 (optional; needs delta and post): x += delta2 / rms(delta2) * post2 as well. groups > 1: the
+ * norm of x is taken over that many equal parts of the `cols` values, each by itself. store_x 0: x is only read. dtype of out 0 bf16, 1 fp16, 2 fp32. All rows ld apart. */
 int hds_norm_residual(float* x, void* delta, int delta_is_f32, float factor, const float* post, const float* gamma, void* out,
-                      int64_t ld, int rows, int cols, int padded, float eps, int store_x, int dtype, void* stream);
+                      int64_t ld, int rows, int cols, int padded, float eps, int store_x, int groups, void* delta2, const float* post2,
+                      int dtype, void* stream);
 
 /* out = scale * w * v / rms(v) with v = y * silu(z), rms over each of `groups` equal parts of a row; gate_after:
  * out = scale * w * y / rms(y) * silu(z). y, w fp32; z, out dtype. */
@@ -448,6 +458,39 @@ int hds_paged_attention_latent_supported(int rank, int page_width);
 int hds_paged_attention_latent_ctas(int item_tokens, int heads, int rank, int page_width, int* tile_keys);
 /* Scratch for n_splits > 1. Zero it once; the kernel leaves its tickets zeroed. */
 int64_t hds_paged_attention_latent_workspace_bytes(void);
+
+/* ---- attention inputs, minGRU, gated linear attention --------------------------------------------------------------- */
+
+/* Projected rows qkv = [n_q heads | n_kv heads | n_kv heads] of head_dim values -> q_out [T, n_q * head_dim] and the tokens' K / V page
+ * rows (tok_slot < 0: none). q_norm / k_norm (optional, together; fp32 per column): all of a row's q (k) divided by its root mean
+ * square over q_cols (k_cols) values and weighted. freq (optional, [head_dim / 2]): value c turns with value head_dim / 2 + c by
+ * position * freq[c]. first (optional): pages [blocks][2][n_kv][block][first_dim] of another layer; v = (1 - share) v + share *
+ * its cached value of the same token. dtype 0 / 1 / 2. n_q_heads 0: keys and values alone. */
+int hds_attention_append(const void* qkv, int64_t ld_qkv, void* q_out, void* kv_cache_layer, const int32_t* tok_pos,
+                         const int32_t* tok_slot, int T, int n_q_heads, int n_kv_heads, int head_dim, int block_size, const float* freq,
+                         const float* q_norm, const float* k_norm, int q_cols, int k_cols, float eps, const void* first, int first_dim,
+                         const float* share, int dtype, void* stream);
+/* The same mixing of the tokens' values, in place in their pages. */
+int hds_mix_cached_values(void* kv_cache_layer, const void* first, int first_dim, const int32_t* tok_slot, const float* share, int T,
+                          int n_kv_heads, int head_dim, int block_size, int dtype, void* stream);
+
+/* minGRU over a ragged batch: proj rows z | u | g (width each), bias [2 * width] of z and u;  S = (1 - sigmoid(z)) S + sigmoid(z) c,
+ * c = u + 1/2 where u >= 0, else sigmoid(u);  out = S * silu(g) (out NULL: the state alone). state [slots, width] fp32 advanced in
+ * place; spans and n_single as hds_state_space. workspace: for batches with sequences of several tokens. */
+int hds_gru(const void* proj, int64_t ld_proj, const float* bias, float* state, const int32_t* spans, int n_seqs, int n_single, int T,
+            int width, void* out, int64_t ld_out, void* workspace, int64_t workspace_bytes, int dtype, void* stream);
+int64_t hds_gru_workspace_bytes(int T, int n_seqs, int width);
+
+/* Gated linear attention over a ragged batch: q, k [T, ld] of heads * dim columns, v and gate of heads * vdim, decay inputs z [T, ld_z]
+ * and their bias [heads * dim];  S = S diag(sigmoid(z + bias)^inv_tau) + v k^T,  y = S q dim^-1/2  per head, state
+ * [slots, heads, vdim, dim] fp32 advanced in place. *finished = 1: out [T, ld_out] = y / rms(y per head) * norm_w * silu(gate) has been
+ * written (norm_w [heads * vdim]); 0: y [T, ld_y] fp32 holds the read-outs. out NULL: the state alone. method as hds_state_space.
+ * workspace (optional) enables the chunked form (bf16; dim a multiple of 16 up to 256, vdim of 16); a larger one needs fewer passes. */
+int hds_linear_attention(const void* q, const void* k, const void* v, const void* gate, int64_t ld, const void* z, int64_t ld_z,
+                         const float* bias, float inv_tau, float* state, const int32_t* spans, int n_seqs, int n_single, int T, int heads,
+                         int vdim, int dim, float* y, int64_t ld_y, void* out, int64_t ld_out, const float* norm_w, float eps,
+                         void* workspace, int64_t workspace_bytes, int method, int* finished, int dtype, void* stream);
+int64_t hds_linear_attention_workspace_bytes(int T, int n_seqs, int heads, int vdim, int dim);
 
 #ifdef __cplusplus
 }
