@@ -14,7 +14,7 @@ from typing import Callable, Dict, Optional
 import torch
 
 GROUPS = [("dedelorn-2048", "nipolorn-2048", "mistral-2048"), ("dedelorn-4096", "nipolorn-4096", "mistral-4096"),
-          ("dedelorn-4096-moe", "nipolorn-4096-moe", "qwen2-moe-4096")]
+          ("lotelix-2048", "dedelorn-2048-moe"), ("lotelix-4096", "dedelorn-4096-moe", "nipolorn-4096-moe", "qwen2-moe-4096")]
 PROMPT = 4096
 
 
@@ -68,16 +68,12 @@ def bench_engine(name: str, steps: int, warmup: int) -> Dict[str, float]:
     return out
 
 
-def bench_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
-    """Kernels of a stack next to the like kernel of a plain family (``like``), with bytes or flops that the operation itself
-    needs. Sizes: width 4096, 32 / 8 attention heads of 128, 128 state-space heads of 64 x 128 in 8 groups."""
-    from ..ops import kernels as K
-    dev, bf = "cuda", torch.bfloat16
-    flush = torch.empty(512 << 20, dtype=torch.uint8, device=dev)
-    W, T = 4096, PROMPT
+def _rnd(*shape, dtype=torch.bfloat16, scale=1.0):
+    return (torch.randn(shape, device="cuda") * scale).to(dtype)
 
-    def rnd(*shape, dtype=bf, scale=1.0):
-        return (torch.randn(shape, device=dev) * scale).to(dtype)
+
+def _reporter(p: Dict[str, float], iters: int, warmup: int):
+    flush = torch.empty(512 << 20, dtype=torch.uint8, device="cuda")
 
     def report(op, kernel, fn, bytes_=0.0, flops=0.0):
         ms = _time(fn, iters, warmup, before=flush.zero_)
@@ -85,6 +81,16 @@ def bench_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
         print(json.dumps({"op": op, "kernel": kernel, "us": round(ms * 1e3, 1), "roofline_us": round(need * 1e3, 1),
                           "bound": "memory" if bytes_ / (p["hbm_gbs"] * 1e6) >= flops / (p["bf16_tflops"] * 1e9) else "math",
                           "of_measured_peak": round(need / ms, 3)}), flush=True)
+
+    return report
+
+
+def bench_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
+    """Kernels of a stack next to the like kernel of a plain family (``like``), with bytes or flops that the operation itself
+    needs. Sizes: width 4096, 32 / 8 attention heads of 128, 128 state-space heads of 64 x 128 in 8 groups."""
+    from ..ops import kernels as K
+    dev, bf, rnd, report = "cuda", torch.bfloat16, _rnd, _reporter(p, iters, warmup)
+    W, T = 4096, PROMPT
 
     for rows in (T, 64):
         x32, x16, d16, out = rnd(rows, W, dtype=torch.float32), rnd(rows, W), rnd(rows, W), rnd(rows, W)
@@ -244,6 +250,94 @@ def bench_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
         report(f"combine {rows}", "moe_gather (like)", lambda: K.moe_gather(ys, slots, scores, out), rows * W * (2 * top + 4 + 4))
 
 
+def bench_lotelix_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
+    """The same for what Lotelix adds: minGRU, gated linear attention (32 heads of 128 x 128), sinks, sigmoid weights, gates, normed and
+    rotated inputs, mixed values, grouped norms, weighted expert inputs."""
+    from ..ops import kernels as K
+    from ..ops.backend import pick_packed_splits, windowed_len
+    dev, bf, f32, rnd, report = "cuda", torch.bfloat16, torch.float32, _rnd, _reporter(p, iters, warmup)
+    W, T = 4096, PROMPT
+    for rows in (T, 64):
+        x, g, g2, out = rnd(rows, W, dtype=f32), torch.ones(W, device=dev), torch.ones(W, device=dev), rnd(rows, W)
+        a, b, h = rnd(rows, W), rnd(rows, W), rnd(rows, W)
+        report(f"norm {rows}x{W}", "norm_residual, 2 groups", lambda: K.norm_residual(x, g, out, delta=a, eps=1e-5, groups=2), rows * W * (4 + 4 + 2 + 2))
+        report(f"norm {rows}x{W}", "norm_residual, two normed outputs", lambda: K.norm_residual(
+            x, g, out, delta=a, post=g, eps=1e-5, groups=2, delta2=b, post2=g2), rows * W * (4 + 4 + 2 + 2 + 2))
+        report(f"norm {rows}x{W}", "norm (like)", lambda: K.norm(h, g.to(bf), out, delta=a, res_out=h, eps=1e-5), rows * W * (2 + 2 + 2 + 2))
+    bias = rnd(2 * W, dtype=f32)
+    heads, N, P = 32, 128, 128
+    for rows, seqs in ((T, 1), (T, 4), (64, 64), (8, 8)):
+        n = rows // seqs
+        single = seqs if n == 1 else 0
+        spans = torch.tensor([[i * n, n, 128, i] for i in range(seqs)], dtype=torch.int32, device=dev)
+        proj, state, mix = rnd(rows, 3 * W), torch.zeros(seqs, W, device=dev), rnd(rows, W)
+        ws = torch.empty(K.gru_workspace_bytes(rows, seqs, W), dtype=torch.uint8, device=dev)
+        report(f"minGRU {seqs}x{n}", "chunks" if n > 1 else "step", lambda: K.gru(proj, bias, state, spans, single, mix, ws), rows * W * 8 + 8 * seqs * W)
+        proj, z, state = rnd(rows, 4 * heads * N), rnd(rows, heads * N), torch.zeros(seqs, heads, P, N, device=dev)
+        q, k, v, gate = proj.split(heads * N, 1)
+        b, w, y = torch.ones(heads * N, device=dev), torch.ones(heads * P, device=dev), torch.zeros(rows, heads * P, device=dev)
+        lws = torch.empty(K.linear_attention_workspace_bytes(rows, seqs, heads, P, N), dtype=torch.uint8, device=dev)
+        report(f"linear attention {seqs}x{n}", "chunks, norm and gate" if n > 1 else "step, norm and gate", lambda: K.linear_attention(
+            q, k, v, gate, z, b, 1 / 16, state, spans, single, y, mix, w, 1e-5, lws), rows * heads * N * 2 * 6 + 2 * seqs * heads * P * N * 4)
+        del lws
+    nq, nkv, D, page = 32, 8, 128, 64
+    ws = torch.zeros(256 << 20, dtype=torch.uint8, device=dev)
+    sink, sbias = torch.zeros(nq, device=dev), torch.full((nq, ), -6.0, device=dev)
+    cache = rnd(T // page + 1, 2, nkv, page, D)
+    table = torch.randperm(T // page, device=dev).to(torch.int32)[None].contiguous()
+    q, o, gate = rnd(T, nq * D), rnd(T, nq * D), rnd(T, nq * D)
+    items = torch.tensor([[0, i, 128, i] for i in range(0, T, 128)], dtype=torch.int32, device=dev)
+    cases = [("softmax (like)", 0, {}), ("sigmoid weights", 0, {"sigmoid_bias": sbias}), ("softmax (like)", 2048, {}),
+             ("sink and gate", 2048, {"sink": sink, "gate": gate})]
+    for tag, window, opts in cases:
+        pairs = sum(min(i + 1, window or T) for i in range(T))
+        report(f"attention prefill {T} window {window}", tag, lambda: K.paged_attention_prefill(
+            q, o, cache, table, items, T // 128, nq, nkv, D, page, 0.09, window=window, **opts), flops=4.0 * pairs * nq * D)
+    B = 64
+    cache = rnd(B * T // page, 2, nkv, page, D)
+    tables = torch.randperm(B * T // page, device=dev).to(torch.int32).view(B, T // page).contiguous()
+    items = torch.tensor([[i, i, 1, T - 1] for i in range(B)], dtype=torch.int32, device=dev)
+    qd, od, gd = rnd(B, nq * D), rnd(B, nq * D), rnd(B, nq * D)
+    for tag, window, opts in cases:
+        sp = pick_packed_splits(B, nkv, windowed_len(T, window))
+        opts = dict(opts, gate=gd) if "gate" in opts else opts
+        report(f"attention decode {B}x{T} window {window}", tag, lambda: K.paged_attention_prefill(
+            qd, od, cache, tables, items, B, nq, nkv, D, page, 0.09, n_splits=sp, workspace=ws, packed=True, window=window, **opts),
+               B * min(T, window or T) * 2 * nkv * D * 2)
+    del cache, q, o, gate
+    freq, qn, kn, share = torch.ones(64, device=dev), torch.ones(nq * D, device=dev), torch.ones(nkv * D, device=dev), torch.ones(1, device=dev)
+    for rows in (T, 64):
+        qkv, q, pages, first = rnd(rows, (nq + 2 * nkv) * D), rnd(rows, nq * D), rnd(rows // page + 1, 2, nkv, page, D), rnd(rows // page + 1, 2, nkv, page, D)
+        pos = torch.arange(rows, dtype=torch.int32, device=dev)
+        need = rows * 2 * (nq + 2 * nkv) * D * 2
+        report(f"attention inputs {rows}", "norms, rotation, pages", lambda: K.attention_append(
+            qkv, q, pages, pos, pos, nq, nkv, D, page, freq, qn, kn, nq * D, nkv * D, 1e-5), need)
+        report(f"attention inputs {rows}", "rotation, pages, mixed values", lambda: K.attention_append(
+            qkv, q, pages, pos, pos, nq, nkv, D, page, freq, first=first, share=share), need + rows * nkv * D * 2)
+        report(f"attention inputs {rows}", "rope_kv_append (like)", lambda: K.rope_kv_append(qkv, q, pages, pos, pos, freq, nq, nkv, D, D, page), need)
+        report(f"mix values {rows}", "mix_cached_values", lambda: K.mix_cached_values(pages, first, pos, share, nkv, D, page), rows * 3 * nkv * D * 2)
+    E, top, ff = 16, 2, 5376
+    i32 = lambda *s: torch.zeros(s, dtype=torch.int32, device=dev)  # noqa: E731
+    for rows in (T, 64):
+        scores, e, off, slots, counts, pad = torch.zeros(rows, top, device=dev), i32(rows, top), i32(rows, top), i32(rows, top), i32(E), i32(E + 1)
+        R = K.moe_padded_rows(rows, E, top)
+        x, xs, ys, out, wr, lg = rnd(rows, W), rnd(R, W), rnd(R, W), torch.zeros(rows, W, device=dev), rnd(E, W, scale=0.02), torch.zeros(rows, E, device=dev)
+        hs, wu, wd = rnd(R, ff), rnd(E * ff, W, scale=0.02), rnd(E * W, ff, scale=0.02)
+
+        def route(sigmoid):
+            K.gemm_accum(x, wr, lg)
+            K.moe_topk_gating(lg, top, False, scores, e, off, counts, clear=True, sigmoid=sigmoid)
+            K.moe_scatter(x, xs, e, off, counts, pad, slots, top, scores if sigmoid else None)
+
+        for tag, sigmoid in (("sigmoid scores, weighted rows", True), ("softmax scores (like)", False)):
+            report(f"router + route + scatter {rows}", tag, lambda: route(sigmoid), rows * W * 2 * (2 + top))
+        for tag, act in (("grouped GEMM, squared relu", 6), ("grouped GEMM, gelu (like)", 1)):
+            report(f"experts up {rows}", tag, lambda: K.moe_gemm(xs, wu, pad, E, hs, act=act), 2 * (wu.numel() + rows * top * (W + ff)), 2.0 * rows * top * W * ff)
+        report(f"experts down {rows}", "grouped GEMM", lambda: K.moe_gemm(hs, wd, pad, E, ys), 2 * (wd.numel() + rows * top * (W + ff)), 2.0 * rows * top * W * ff)
+        report(f"combine {rows}", "moe_combine, plain sum", lambda: K.moe_combine(ys, slots, None, None, out), rows * W * (2 * top + 4))
+        report(f"combine {rows}", "moe_combine, weighted (like)", lambda: K.moe_combine(ys, slots, scores, None, out), rows * W * (2 * top + 4))
+
+
 def main(steps: int = 5, warmup: int = 3) -> None:
     p = peaks()
     for group in GROUPS:
@@ -252,6 +346,8 @@ def main(steps: int = 5, warmup: int = 3) -> None:
                               **bench_engine(name, steps, warmup)}), flush=True)
             torch.cuda.empty_cache()
     bench_kernels(p, max(steps, 10), warmup)
+    torch.cuda.empty_cache()
+    bench_lotelix_kernels(p, max(steps, 10), warmup)
 
 
 if __name__ == "__main__":

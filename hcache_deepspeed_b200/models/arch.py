@@ -855,8 +855,8 @@ def named_arch(name: str) -> ArchSpec:
 
 
 def _stack_named() -> Dict[str, ArchSpec]:
-    """Nipolorn and Dedelorn stacks with layers of real sizes, and beside each the closest plain family at equal sizes (same width,
-    heads, window and feed-forward): windowed attention with a dense MLP, or with routed experts and a shared one."""
+    """Nipolorn, Dedelorn and Lotelix stacks with layers of real sizes, and beside each the closest plain family at equal sizes (same
+    width, heads, window and feed-forward): windowed attention with a dense MLP, or with routed experts and a shared one."""
 
     def nipolorn(width, heads, kv, window, keep, ssm_heads, groups, mlp):
         mixer = MixerSpec(attn=AttentionSpec(heads, kv, 128, 128, 128 ** -0.5, window, keep),
@@ -872,6 +872,17 @@ def _stack_named() -> Dict[str, ArchSpec]:
         return stack_arch("dedelorn", [LayerSpec(m, mlp) for m in (delta, latent(), delta, latent(1))], hidden=width, vocab=32000,
                           norm_eps=1e-5, **DEDELORN_NORMS)
 
+    def lotelix(width, heads, kv, window, ff):
+        def attn(v_first=None):
+            return MixerSpec(attn=AttentionSpec(heads, kv, 128, 128, 128**-0.5, window, rot=RotationSpec(128, 1e6, False, 8.0, 1.0, 4.0, 8192), sink=True,
+                                                gate=True, v_first=v_first))
+
+        both = MixerSpec(attn=AttentionSpec(heads, kv, 128, 128, 128**-0.5, rot=RotationSpec(128, 1e6, True), weights="sigmoid", bias=True, qk_norm=True),
+                         linear=LinearAttentionSpec(heads=width // 128, dim=128, vdim=128, tau=16.0, rank=16))
+        mlp = FeedForwardSpec(ff=ff, act="relu2", experts=16, top=2, routing="sigmoid", gated=False)
+        return stack_arch("lotelix", [LayerSpec(m, mlp) for m in (MixerSpec(gru=GRUSpec(width)), attn(), both, attn(1))], hidden=width, vocab=32000,
+                          norm_eps=1e-5, norm_groups=2, embed_scale=1.0)
+
     def plain(mt, width, heads, kv, window, **kw):
         return ArchSpec(model_type=mt, n_layers=4, hidden=width, n_heads=heads, n_kv_heads=kv, head_dim=128, vocab=32000, norm="rms",
                         norm_eps=1e-5, act="silu", gated_mlp=True, pos_emb="rope", sliding_window=window, max_positions=1 << 20, **kw)
@@ -883,6 +894,10 @@ def _stack_named() -> Dict[str, ArchSpec]:
         "dedelorn-4096": dedelorn(4096, 32, 512, 4096, FeedForwardSpec(ff=14336, act="gelu_tanh")),
         "dedelorn-4096-moe": dedelorn(4096, 32, 512, 2048, FeedForwardSpec(ff=5376, act="gelu", experts=16, top=2, routing="softmax", gated=False,
                                                                             router_scale=2.5)),
+        "dedelorn-2048-moe": dedelorn(2048, 16, 256, 1024, FeedForwardSpec(ff=2688, act="gelu", experts=16, top=2, routing="softmax", gated=False,
+                                                                            router_scale=2.5)),
+        "lotelix-2048": lotelix(2048, 16, 4, 1024, 2688),
+        "lotelix-4096": lotelix(4096, 32, 8, 2048, 5376),
         "mistral-2048": plain("mistral", 2048, 16, 4, 1024, intermediate=8192),
         "nipolorn-4096": nipolorn(4096, 32, 8, 4096, 64, 128, 8, FeedForwardSpec(ff=14336, act="swiglu_clamped", limit=7.0)),
         "mistral-4096": plain("mistral", 4096, 32, 8, 4096, intermediate=14336),

@@ -305,7 +305,7 @@ def attention_append(qkv: torch.Tensor, kv_cache_layer: torch.Tensor, pos: torch
     def rotated(x):
         return x if freq is None else rope_rotate_half(x, pos, freq, D)
 
-    q, k = normed(q, q_norm, q_cols).reshape(T, n_q, D), normed(k, k_norm, k_cols).reshape(T, n_kv, D)
+    q, k = normed(q, q_norm if n_q else None, q_cols).reshape(T, n_q, D), normed(k, k_norm, k_cols).reshape(T, n_kv, D)
     v = v.reshape(T, n_kv, D)
     if first is not None:
         v = mixed_values(v, first, slot, share)

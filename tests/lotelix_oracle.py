@@ -183,9 +183,10 @@ def mixture(h, w, p, router):
     """A token's weight for an expert multiplies what the expert reads."""
     chosen, weight = route(h, w, p, router)
     out = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for e, f in zip(chosen[t].tolist(), weight[t]):
-            out[t] += expert(f * h[t:t + 1], w, f"{p}e{e}.")[0]
+    for e in range(w[p + "router"].shape[0]):
+        for j in range(router["top"]):
+            t = chosen[:, j] == e
+            out[t] += expert(weight[t, j, None] * h[t], w, f"{p}e{e}.")
     return out
 
 
