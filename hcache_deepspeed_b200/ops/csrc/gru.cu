@@ -6,6 +6,8 @@
 //   gru_chain : states in front of every chunk, from the (A, B) of the chunks before it; advances the state pool
 //   gru_out   : the tokens of a chunk from the state in front of it
 // The gates depend on the token alone, so only gru_chain walks along a sequence, a step per 32 tokens.
+#include <type_traits>
+
 #include "recurrent.cuh"
 #include "../../../include/hds_b200.h"
 
@@ -26,24 +28,37 @@ struct GruArgs {
     float4* b;
 };
 
+// four neighbouring values as they are stored, and as fp32
 template <int DT>
-__device__ __forceinline__ float4 gru_load(const void* p, int64_t i) {
-    if constexpr (DT == 2) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + i);
-    else {
-        const uint2 q = *reinterpret_cast<const uint2*>(reinterpret_cast<const char*>(p) + i * 2);
-        return make_float4(unpack_lo<DT == 0>(q.x), unpack_hi<DT == 0>(q.x), unpack_lo<DT == 0>(q.y), unpack_hi<DT == 0>(q.y));
+struct GruRaw {
+    typename std::conditional<DT == 2, float4, uint2>::type v;
+    __device__ __forceinline__ void load(const void* p, int64_t i) {
+        v = *reinterpret_cast<const decltype(v)*>(reinterpret_cast<const char*>(p) + i * (DT == 2 ? 4 : 2));
     }
-}
+    __device__ __forceinline__ float4 get() const {
+        if constexpr (DT == 2) return v;
+        else return make_float4(unpack_lo<DT == 0>(v.x), unpack_hi<DT == 0>(v.x), unpack_lo<DT == 0>(v.y), unpack_hi<DT == 0>(v.y));
+    }
+};
 template <int DT>
 __device__ __forceinline__ float gru_sigmoid(float v) {
     return DT == 2 ? 1.0f / (1.0f + expf(-v)) : __fdividef(1.0f, 1.0f + __expf(-v));
 }
-// gates of one value: kept share of the state, and what is added
+// gates of one value: kept share of the state, and what is added. 16-bit inputs: both sigmoids from one reciprocal (inputs below -40,
+// whose sigmoid is zero to any state, count as -40 so that the product of the denominators stays finite).
 template <int DT>
 __device__ __forceinline__ void gru_gate(float z, float u, float& keep, float& add) {
-    const float s = gru_sigmoid<DT>(z);
+    float s, c;
+    if constexpr (DT == 2) {
+        s = gru_sigmoid<2>(z);
+        c = gru_sigmoid<2>(u);
+    } else {
+        const float a = 1.0f + __expf(-fmaxf(z, -40.0f)), b = 1.0f + __expf(-fmaxf(u, -40.0f)), r = __fdividef(1.0f, a * b);
+        s = r * b;
+        c = r * a;
+    }
     keep = 1.0f - s;
-    add = s * (u >= 0.0f ? u + 0.5f : gru_sigmoid<DT>(u));
+    add = s * (u >= 0.0f ? u + 0.5f : c);
 }
 template <int DT>
 __device__ __forceinline__ void gru_gates(float4 z, float4 u, float4 bz, float4 bu, float4& keep, float4& add) {
@@ -72,13 +87,16 @@ __global__ void __launch_bounds__(kGruThreads) gru_step_kernel(const GruArgs a) 
     if (sp.n != 1 || c >= a.C) return;
     float4* st = reinterpret_cast<float4*>(a.state + static_cast<int64_t>(sp.slot) * a.C + c);
     const int64_t at = static_cast<int64_t>(sp.row0) * a.ld + c;
-    const float4 z = gru_load<DT>(a.proj, at), u = gru_load<DT>(a.proj, at + a.C);
+    GruRaw<DT> z, u, g;
+    z.load(a.proj, at);
+    u.load(a.proj, at + a.C);
+    g.load(a.proj, at + 2 * a.C);
     float4 keep, add, S = make_float4(0.f, 0.f, 0.f, 0.f);
     if (sp.seen > 0) S = *st;
-    gru_gates<DT>(z, u, *reinterpret_cast<const float4*>(a.bias + c), *reinterpret_cast<const float4*>(a.bias + a.C + c), keep, add);
+    gru_gates<DT>(z.get(), u.get(), *reinterpret_cast<const float4*>(a.bias + c), *reinterpret_cast<const float4*>(a.bias + a.C + c), keep, add);
     S = gru_fma(keep, S, add);
     *st = S;
-    if (a.out != nullptr) gru_emit<DT>(a, sp.row0, c, S, gru_load<DT>(a.proj, at + 2 * a.C));
+    if (a.out != nullptr) gru_emit<DT>(a, sp.row0, c, S, g.get());
 }
 
 // kOut false: (A, B) of the chunk; true: its outputs from the state in front
@@ -94,24 +112,28 @@ __global__ void __launch_bounds__(kGruThreads) gru_chunk_kernel(const GruArgs a)
     const float4 bz = *reinterpret_cast<const float4*>(a.bias + c), bu = *reinterpret_cast<const float4*>(a.bias + a.C + c);
     float4 A = make_float4(1.f, 1.f, 1.f, 1.f), S = make_float4(0.f, 0.f, 0.f, 0.f);
     if constexpr (kOut) S = a.a[cell];
-    constexpr int U = 8;        // tokens in flight
+    constexpr int U = 4;        // tokens loaded ahead of those being worked on
+    GruRaw<DT> z[U], u[U], g[kOut ? U : 1];
+    auto load = [&](int t, int i) {
+        const int64_t at = (row + min(t, n - 1)) * a.ld + c;
+        z[i].load(a.proj, at);
+        u[i].load(a.proj, at + a.C);
+        if constexpr (kOut) g[i].load(a.proj, at + 2 * a.C);
+    };
+#pragma unroll
+    for (int i = 0; i < U; ++i) load(i, i);
     for (int t = 0; t < n; t += U) {
-        float4 z[U], u[U], g[kOut ? U : 1];
 #pragma unroll
         for (int i = 0; i < U; ++i) {
-            const int64_t at = (row + min(t + i, n - 1)) * a.ld + c;
-            z[i] = gru_load<DT>(a.proj, at);
-            u[i] = gru_load<DT>(a.proj, at + a.C);
-            if constexpr (kOut) g[i] = gru_load<DT>(a.proj, at + 2 * a.C);
-        }
-#pragma unroll
-        for (int i = 0; i < U; ++i) {
-            if (t + i >= n) break;
-            float4 keep, add;
-            gru_gates<DT>(z[i], u[i], bz, bu, keep, add);
-            S = gru_fma(keep, S, add);
-            if constexpr (kOut) gru_emit<DT>(a, row + t + i, c, S, g[i]);
-            else A = make_float4(A.x * keep.x, A.y * keep.y, A.z * keep.z, A.w * keep.w);
+            const GruRaw<DT> zi = z[i], ui = u[i], gi = g[kOut ? i : 0];
+            load(t + i + U, i);
+            if (t + i < n) {
+                float4 keep, add;
+                gru_gates<DT>(zi.get(), ui.get(), bz, bu, keep, add);
+                S = gru_fma(keep, S, add);
+                if constexpr (kOut) gru_emit<DT>(a, row + t + i, c, S, gi.get());
+                else A = make_float4(A.x * keep.x, A.y * keep.y, A.z * keep.z, A.w * keep.w);
+            }
         }
     }
     if constexpr (!kOut) {
@@ -120,32 +142,37 @@ __global__ void __launch_bounds__(kGruThreads) gru_chunk_kernel(const GruArgs a)
     }
 }
 
+// One value per thread; the loads of 16 chunks run ahead of the chain.
 __global__ void __launch_bounds__(kGruThreads) gru_chain_kernel(const GruArgs a) {
     pdl_enter();
     const SsmSpan sp = a.spans[blockIdx.x];
-    const int c = (blockIdx.y * kGruThreads + threadIdx.x) * 4;
+    const int c = blockIdx.y * kGruThreads + threadIdx.x;
     if (sp.n <= 1 || c >= a.C) return;
-    const int n = span_chunks(sp, kGruTok), stride = a.C / 4;
-    float4* st = reinterpret_cast<float4*>(a.state + static_cast<int64_t>(sp.slot) * a.C + c);
-    float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (sp.seen > 0) S = *st;
-    int64_t cell = static_cast<int64_t>(first_chunk(a.spans, blockIdx.x, kGruTok)) * stride + c / 4;
-    constexpr int U = 8;
+    const int n = span_chunks(sp, kGruTok);
+    float* st = a.state + static_cast<int64_t>(sp.slot) * a.C + c;
+    float S = sp.seen > 0 ? *st : 0.0f;
+    const int64_t cell = static_cast<int64_t>(first_chunk(a.spans, blockIdx.x, kGruTok)) * a.C + c;
+    float* pa = reinterpret_cast<float*>(a.a) + cell;
+    const float* pb = reinterpret_cast<const float*>(a.b) + cell;
+    constexpr int U = 16;
+    float A[U], B[U];
+    auto load = [&](int i, int j) {
+        const int64_t at = static_cast<int64_t>(min(i, n - 1)) * a.C;
+        A[j] = __ldcg(pa + at);
+        B[j] = __ldcg(pb + at);
+    };
+#pragma unroll
+    for (int j = 0; j < U; ++j) load(j, j);
     for (int i = 0; i < n; i += U) {
-        float4 A[U], B[U];
 #pragma unroll
         for (int j = 0; j < U; ++j) {
-            const int64_t at = cell + static_cast<int64_t>(min(j, n - 1 - i)) * stride;
-            A[j] = a.a[at];
-            B[j] = a.b[at];
+            const float aj = A[j], bj = B[j];
+            load(i + j + U, j);
+            if (i + j < n) {
+                pa[static_cast<int64_t>(i + j) * a.C] = S;
+                S = fmaf(aj, S, bj);
+            }
         }
-#pragma unroll
-        for (int j = 0; j < U; ++j) {
-            if (i + j >= n) break;
-            a.a[cell + static_cast<int64_t>(j) * stride] = S;
-            S = gru_fma(A[j], S, B[j]);
-        }
-        cell += static_cast<int64_t>(U) * stride;
     }
     *st = S;
 }
@@ -158,7 +185,7 @@ static int launch_gru(const GruArgs& a, int n_single, int T, cudaStream_t s) {
     if (n_multi > 0) {
         const dim3 grid(T / kGruTok + n_multi, blocks);      // (at least as many as there are chunks)
         HDS_CHECK_CUDA(launch_kernel(gru_chunk_kernel<DT, false>, grid, block, 0, s, a));
-        HDS_CHECK_CUDA(launch_kernel(gru_chain_kernel, dim3(a.n_seqs, blocks), block, 0, s, a));
+        HDS_CHECK_CUDA(launch_kernel(gru_chain_kernel, dim3(a.n_seqs, (a.C + kGruThreads - 1) / kGruThreads), block, 0, s, a));
         if (a.out != nullptr) HDS_CHECK_CUDA(launch_kernel(gru_chunk_kernel<DT, true>, grid, block, 0, s, a));
     }
     if (n_single > 0) HDS_CHECK_CUDA(launch_kernel(gru_step_kernel<DT>, dim3(a.n_seqs, blocks), block, 0, s, a));

@@ -16,6 +16,21 @@
 
 namespace hds {
 
+// two sums at once; red: 2 * THREADS / 32 floats
+template <int THREADS>
+__device__ __forceinline__ void block_sums_t(float& a, float& b, float* red) {
+    a = warp_sum(a);
+    b = warp_sum(b);
+    const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
+    if (l == 0) {
+        red[w] = a;
+        red[THREADS / 32 + w] = b;
+    }
+    __syncthreads();
+    a = warp_sum(l < THREADS / 32 ? red[l] : 0.0f);
+    b = warp_sum(l < THREADS / 32 ? red[THREADS / 32 + l] : 0.0f);
+}
+
 template <int THREADS>
 __device__ __forceinline__ float block_sum_t(float v, float* red) {
     v = warp_sum(v);
@@ -58,7 +73,7 @@ __global__ void __launch_bounds__(THREADS)
 norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const float* __restrict__ post,
                      const float* __restrict__ gamma, void* __restrict__ out, int64_t ld, int cols, int padded, float eps,
                      int store_x, int groups, void* delta2, const float* __restrict__ post2) {
-    __shared__ float red[THREADS / 32];
+    __shared__ float red[THREADS / 32], red2[kTwo ? THREADS / 16 : 1];
     extern __shared__ float group_s[];
     pdl_enter();
     const int64_t row = static_cast<int64_t>(blockIdx.x) * ld;
@@ -66,14 +81,12 @@ norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const flo
     float4 v[VPT], d[VPT], d2[kTwo ? VPT : 1];
     float ss = 0.0f, ss2 = 0.0f;
     auto take = [&](void* from, int c) {
-        if constexpr (DELTA == 1) {
-            float4* p = reinterpret_cast<float4*>(reinterpret_cast<float*>(from) + row + 4 * c);
-            const float4 q = *p;
-            *p = make_float4(0.f, 0.f, 0.f, 0.f);
-            return q;
-        } else {
-            return load4<DT>(from, row + 4 * c);
-        }
+        if constexpr (DELTA == 1) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(from) + row + 4 * c);
+        else return load4<DT>(from, row + 4 * c);
+    };
+    // (a store right behind the load of the same line, while that is still on its way, costs several times the transfer: clear later)
+    auto clear = [&](void* from, int c) {
+        if constexpr (DELTA == 1) *reinterpret_cast<float4*>(reinterpret_cast<float*>(from) + row + 4 * c) = make_float4(0.f, 0.f, 0.f, 0.f);
     };
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
@@ -94,9 +107,14 @@ norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const flo
     }
     if constexpr (DELTA != 0) {
         float r = 1.0f;
-        if constexpr (kPost) r = 1.0f / sqrtf(block_sum_t<THREADS>(ss, red) / cols + eps);
         float r2 = 0.0f;
-        if constexpr (kTwo) r2 = 1.0f / sqrtf(block_sum_t<THREADS>(ss2, red) / cols + eps);
+        if constexpr (kTwo) {
+            block_sums_t<THREADS>(ss, ss2, red2);
+            r = 1.0f / sqrtf(ss / cols + eps);
+            r2 = 1.0f / sqrtf(ss2 / cols + eps);
+        } else if constexpr (kPost) {
+            r = 1.0f / sqrtf(block_sum_t<THREADS>(ss, red) / cols + eps);
+        }
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
             const int c = threadIdx.x + i * THREADS;
@@ -111,6 +129,8 @@ norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const flo
                     v[i].z += d2[i].z * r2 * u.z; v[i].w += d2[i].w * r2 * u.w;
                 }
                 if (store_x) *reinterpret_cast<float4*>(x + row + 4 * c) = v[i];
+                clear(delta, c);
+                if constexpr (kTwo) clear(delta2, c);
             }
         }
     }
@@ -143,8 +163,12 @@ norm_residual_kernel(float* __restrict__ x, void* delta, float factor, const flo
             if (c < nvec) {
                 const float4 w = *reinterpret_cast<const float4*>(gamma + e);
                 auto of = [&](int x) { return r_s[min(x / part, groups - 1)]; };    // (past the values: zeros)
-                store4<DT>(out, row + e, make_float4(v[i].x * of(e) * w.x, v[i].y * of(e + 1) * w.y, v[i].z * of(e + 2) * w.z,
-                                                     v[i].w * of(e + 3) * w.w));
+                const float r0 = of(e);
+                if ((part & 3) == 0)
+                    store4<DT>(out, row + e, make_float4(v[i].x * r0 * w.x, v[i].y * r0 * w.y, v[i].z * r0 * w.z, v[i].w * r0 * w.w));
+                else
+                    store4<DT>(out, row + e, make_float4(v[i].x * r0 * w.x, v[i].y * of(e + 1) * w.y, v[i].z * of(e + 2) * w.z,
+                                                         v[i].w * of(e + 3) * w.w));
             }
         }
         return;

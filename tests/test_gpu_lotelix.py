@@ -266,7 +266,7 @@ def test_chunked_linear_attention_against_token_scan(heads, N, P, decay, tau, ce
             spans.append([row, n, 5 if i % 2 else 0, len(lens) - 1 - i])
             row += n
         single = sum(n == 1 for n in lens)
-        n_ws = k().linear_attention_workspace_bytes(T, len(lens), heads, P, N) if not cells else cells * heads * N * (P + 1) * 4
+        n_ws = k().linear_attention_workspace_bytes(T, len(lens), heads, P, N) if not cells else cells * heads * N * (P + 64) * 4
         ws = torch.empty(n_ws, dtype=torch.uint8, device="cuda")
         res = []
         for method in (1, 2):
