@@ -55,7 +55,7 @@ def parse():
     p.add_argument("--plan", default="hidden", choices=["auto", "hidden", "planner", "adaptive"],
                    help="hidden: every layer from hidden states (fastest measured on 1xB200: 20.4 ms vs 21.6 ms); auto: planner mix with a recomputed prefix")
     p.add_argument("--stacks", action="store_true",
-                   help="instead of the headline workload: prefill and decode throughput of the Dedelorn and Nipolorn stacks beside the "
+                   help="instead of the headline workload: prefill and decode throughput of the Lotelix, Dedelorn and Nipolorn stacks beside the "
                         "closest plain families at equal sizes, and their kernels against the measured peaks (one JSON line each; one GPU)")
     return p.parse_args()
 

@@ -213,7 +213,7 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
         lw.ssm_dt_bias, lw.ssm_a, lw.ssm_d = f32(p["ssm.dt_bias"]), f32(-torch.exp(p["ssm.A_log"].float())), f32(p["ssm.D"])
         lw.ssm_norm = f32(p["ssm.norm"])
     if g is not None:
-        rank = p["linear.a1"].shape[0]
+        g.rank = rank = p["linear.a1"].shape[0]       # (a checkpoint's own; its config does not say)
         rows += [_pad(p["linear." + n], 0, w) for n, w in (("q", g.keys), ("k", g.keys), ("v", g.inner), ("g", g.inner), ("a1", pad8(rank)))]
         lw.w_decay = to(_pad(_pad(p["linear.a2"], 1, pad8(rank)), 0, g.keys))
         lw.decay_bias = f32(p["linear.a2_b"])
