@@ -182,8 +182,12 @@ class LotelixPolicy(InferenceV2Policy):
     """Layers of a minGRU, of windowed attention with sinks, or of sigmoid attention beside gated linear attention."""
 
 
+class RelulixPolicy(InferenceV2Policy):
+    """Layers of retention or of windowed attention with bounded scores, each beside its experts on one norm."""
+
+
 MODEL_TYPE_TO_POLICY = {
-    "nipolorn": NipolornPolicy, "dedelorn": DedelornPolicy, "lotelix": LotelixPolicy,
+    "nipolorn": NipolornPolicy, "dedelorn": DedelornPolicy, "lotelix": LotelixPolicy, "relulix": RelulixPolicy,
     "gpt2": GPT2Policy, "gptj": GPTJPolicy, "gpt_neox": GPTNeoXPolicy, "bloom": BloomPolicy, "gpt_neo": GPTNeoPolicy,
     "llama": Llama2Policy, "opt": OPTPolicy, "mistral": MistralPolicy, "mixtral": MixtralPolicy, "falcon": FalconPolicy,
     "phi": PhiPolicy, "phi3": Phi3Policy, "qwen": QwenPolicy, "qwen2": Qwen2Policy, "qwen2_moe": Qwen2MoePolicy,

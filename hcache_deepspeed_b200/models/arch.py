@@ -21,7 +21,9 @@ from typing import Any, Callable, Dict, List, Optional
 class RotationSpec:
     """Rotation of the first ``dims`` values of every query and key head by position * base^(-2i / dims): value i is paired with
     i + dims / 2, or, ``adjacent``, 2i with 2i + 1. ``slow_factor`` > 0: pairs whose wavelength exceeds ``original / slow_low``
-    positions turn slower by that factor, those below ``original / slow_high`` as they are, the ones between by a linear mixture."""
+    positions turn slower by that factor, those below ``original / slow_high`` as they are, the ones between by a linear mixture;
+    with ``ramp`` that mixture is linear in the pair's index, between the whole indices next to those two wavelengths. ``amplitude``
+    multiplies the rotated values."""
     dims: int
     base: float
     adjacent: bool = False
@@ -29,12 +31,22 @@ class RotationSpec:
     slow_low: float = 1.0
     slow_high: float = 1.0
     original: float = 0.0
+    ramp: bool = False
+    amplitude: float = 1.0
+
+    def index_of(self, turns: float) -> float:
+        """Index of the pair (a real number) that turns this often within ``original`` positions."""
+        return self.dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
 
     def frequencies(self) -> List[float]:
         out = []
         for i in range(self.dims // 2):
             f = float(self.base)**(-2.0 * i / self.dims)
-            if self.slow_factor:
+            if self.slow_factor and self.ramp:
+                lo, hi = max(math.floor(self.index_of(self.slow_high)), 0), min(math.ceil(self.index_of(self.slow_low)), self.dims - 1)
+                s = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+                f = f / self.slow_factor * s + f * (1.0 - s)
+            elif self.slow_factor:
                 wave = 2.0 * math.pi / f
                 if wave > self.original / self.slow_low:
                     f /= self.slow_factor
@@ -44,6 +56,17 @@ class RotationSpec:
             out.append(f)
         return out
 
+    def places(self, dim: int, width: int) -> List[int]:
+        """Place of every value of a head of ``dim`` in rows of ``width`` whose value c is paired with c + width / 2: the values of
+        rotated pair i at i and width / 2 + i, the others in what is free."""
+        half, n = width // 2, self.dims // 2
+        place = [0] * dim
+        for i in range(n):
+            u, v = (2 * i, 2 * i + 1) if self.adjacent else (i, i + n)
+            place[u], place[v] = i, half + i
+        place[self.dims:] = [p for p in range(width) if p % half >= n][:dim - self.dims]
+        return place
+
 
 @dataclass
 class AttentionSpec:
@@ -51,10 +74,14 @@ class AttentionSpec:
     ``keep_first`` positions of its sequence. Without ``rot`` positions enter through the mask only.
 
     ``weights`` = "softmax"; with ``sink`` its denominator holds one more term per head, exp of a learned number. "sigmoid": a
-    visible key weighs sigmoid(score + a learned number per head), not normalized over keys. ``bias``: q, k, v and the output
-    projection have biases. ``qk_norm``: all of q, and all of k, normed at once before the rotation. ``gate``: the heads are
+    visible key weighs sigmoid(score + a learned number per head), not normalized over keys. ``bias``: q, k and v have
+    biases. ``qk_norm``: all of q, and all of k, normed at once before the rotation. ``gate``: the heads are
     multiplied by the sigmoid of one more projection of the layer's input. ``v_first``: values are mixed, by a learned share, with
-    the values that this earlier layer caches of the same token (the same heads and sizes)."""
+    the values that this earlier layer caches of the same token (the same heads and sizes).
+
+    ``one_more``: the softmax's denominator holds a one more (a score of zero without a value). ``softcap`` > 0: scores are bounded,
+    softcap * tanh(score / softcap). ``o_bias``: the output projection has a bias. ``kv_from``: use the keys and values that this
+    earlier layer caches instead of own ones (both layers' heads, sizes and rotation agree)."""
     heads: int
     kv_heads: int
     dim: int                 # query / key size of a head
@@ -69,6 +96,15 @@ class AttentionSpec:
     qk_norm: bool = False
     gate: bool = False
     v_first: Optional[int] = None
+    one_more: bool = False
+    softcap: float = 0.0
+    o_bias: bool = False
+    kv_from: Optional[int] = None
+
+    @property
+    def cached_heads(self) -> int:
+        """Key / value heads of its own."""
+        return 0 if self.kv_from is not None else self.kv_heads
 
     @property
     def page_dim(self) -> int:
@@ -196,6 +232,40 @@ class LinearAttentionSpec:
 
 
 @dataclass
+class RetentionSpec:
+    """Retention: linear attention whose heads' ``dim`` x ``vdim`` states fade by a constant each (``decay``); queries and keys
+    rotated by position; a norm per head and a gate behind. Heads are zero padded to multiples of 16."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: List[float]
+    rot: Optional[RotationSpec] = None
+
+    conv = conv_dim = 0
+
+    @property
+    def width(self) -> int:
+        """Size of a query or key row of a head."""
+        return -(-self.dim // 16) * 16
+
+    @property
+    def vwidth(self) -> int:
+        return -(-self.vdim // 16) * 16
+
+    @property
+    def keys(self) -> int:
+        return self.heads * self.width
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vwidth
+
+    @property
+    def state(self) -> int:
+        return self.width
+
+
+@dataclass
 class GRUSpec:
     """minGRU: ``width`` independent values, S <- (1 - z) S + z c, gate z and candidate c projections of the current token only;
     an output gate behind."""
@@ -221,8 +291,8 @@ class GRUSpec:
 @dataclass
 class MixerSpec:
     """Token mixer of a layer: attention, a state-space mixer, or both side by side on the same input, each with a weight; or
-    latent attention; or a gated delta rule; or a minGRU; or attention beside gated linear attention, each with an output
-    projection and a norm of its own, of which the result is the mean."""
+    latent attention; or a gated delta rule; or a minGRU; or retention; or attention beside gated linear attention, each with an
+    output projection and a norm of its own, of which the result is the mean."""
     attn: Optional[AttentionSpec] = None
     ssm: Optional[StateSpaceSpec] = None
     attn_weight: float = 1.0
@@ -231,11 +301,12 @@ class MixerSpec:
     delta: Optional[DeltaSpec] = None
     linear: Optional[LinearAttentionSpec] = None
     gru: Optional[GRUSpec] = None
+    retention: Optional[RetentionSpec] = None
 
     @property
     def recurrent(self):
         """The part with per-sequence state, if any."""
-        return next((m for m in (self.ssm, self.delta, self.linear, self.gru) if m is not None), None)
+        return next((m for m in (self.ssm, self.delta, self.linear, self.gru, self.retention) if m is not None), None)
 
     @property
     def normed_mean(self) -> bool:
@@ -249,7 +320,8 @@ class FeedForwardSpec:
     ``routing`` = "table": a table gives every token id its experts, all with weight 1 / top. ``routing`` = "softmax": the
     largest softmax scores of a router, each plus the expert's correction, choose; the scores themselves times
     ``router_scale`` weigh. ``routing`` = "sigmoid": the largest sigmoid scores choose and weigh; the weight multiplies what the
-    expert reads, not what it returns. ``shared_ff`` > 0: one more expert that sees every token. ``gated`` = False: down(act(up x)).
+    expert reads, not what it returns. ``routing`` = "chosen": the largest logits (a bias per expert included) choose, the softmax over
+    the chosen ones alone weighs. ``shared_ff`` > 0: one more expert that sees every token. ``gated`` = False: down(act(up x)).
     ``act`` = "swiglu_clamped" clamps gate and up to ``limit`` (see ops.reference)."""
     ff: int
     act: str = "silu"
@@ -323,6 +395,7 @@ class ArchSpec:
     layers: Optional[List[LayerSpec]] = None
     post_norms: bool = False  # ``layers`` stacks: every sublayer's OUTPUT is normed as well
     norm_weight_offset: float = 0.0  # ``layers`` stacks: stored norm weights are differences from this
+    norm_scalar: bool = False  # ``layers`` stacks: the weight of a norm is one number for all coordinates
     norm_groups: int = 1  # ``layers`` stacks: the layers' norms and the final one norm equal consecutive parts of a row, each by itself
     embed_scale: float = 1.0  # ``layers`` stacks: factor of the token embeddings
     extras: Dict[str, Any] = field(default_factory=dict)
@@ -365,7 +438,8 @@ class ArchSpec:
     def pages_hold_context(self) -> bool:
         """Do the K / V pages of a sequence alone bring every layer's context back?"""
         return self.layers is None or (not self.has_recurrent_state and all(
-            l.mixer.latent is None and (l.mixer.attn is None or l.mixer.attn.v_first is None) for l in self.layers))
+            l.mixer.latent is None and (l.mixer.attn is None or (l.mixer.attn.v_first is None and l.mixer.attn.kv_from is None))
+            for l in self.layers))
 
     def window_of(self, layer: int) -> int:
         return int(self.layer_windows[layer]) if self.layer_windows is not None else int(self.sliding_window)
@@ -376,14 +450,15 @@ class ArchSpec:
     def param_count(self) -> int:
         h, i = self.hidden, self.intermediate
         if self.layers is not None:
-            total = self.vocab * h * (1 if self.tie_word_embeddings else 2) + h
+            n = 1 if self.norm_scalar else h
+            total = self.vocab * h * (1 if self.tie_word_embeddings else 2) + n
             for l in self.layers:
                 a, m, f, c, d = l.mixer.attn, l.mixer.ssm, l.mlp, l.mixer.latent, l.mixer.delta
-                total += h * (1 + self.post_norms)
+                total += n * (1 + self.post_norms)
                 if a is not None:
-                    total += h * (a.heads * (a.dim + a.vdim) + a.kv_heads * (a.dim + a.vdim))
+                    total += h * (a.heads * (a.dim + a.vdim) + a.cached_heads * (a.dim + a.vdim))
                     total += h * a.heads * a.vdim * a.gate + a.heads * (a.sink + (a.weights == "sigmoid")) + (a.v_first is not None)
-                    total += (a.heads + a.kv_heads) * a.dim * a.qk_norm + ((a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim + h) * a.bias
+                    total += (a.heads + a.kv_heads) * a.dim * a.qk_norm + ((a.heads + a.cached_heads) * a.dim + a.cached_heads * a.vdim) * a.bias + h * a.o_bias
                 if m is not None:
                     total += h * (m.in_dim + m.inner) + m.conv_dim * (m.conv + 1) + 3 * m.heads + m.inner
                 if c is not None:
@@ -396,11 +471,14 @@ class ArchSpec:
                     total += g.heads * (h * (2 * g.dim + 3 * g.vdim) + g.dim * (g.rank + 1)) + h * g.rank + g.vdim + 2 * h * l.mixer.normed_mean
                 if r is not None:
                     total += r.width * (4 * h + 2)
+                t = l.mixer.retention
+                if t is not None:
+                    total += h * t.heads * (2 * t.dim + 3 * t.vdim)
                 if f is not None:
-                    total += 0 if self.parallel_residual else h * (1 + self.post_norms)
+                    total += 0 if self.parallel_residual else n * (1 + self.post_norms)
                     total += (3 if f.gated else 2) * h * (f.ff * max(1, f.experts) + f.shared_ff)
                     if f.experts:
-                        total += self.vocab * f.top if f.routing == "table" else (h + (f.routing == "softmax")) * f.experts
+                        total += self.vocab * f.top if f.routing == "table" else (h + (f.routing in ("softmax", "chosen"))) * f.experts
             return total
         attn = h * (self.q_dim + 2 * self.kv_dim) + self.q_dim * h
         if self.is_moe:
@@ -795,7 +873,7 @@ def _lotelix(cfg) -> ArchSpec:
             mixer = MixerSpec(attn=a)
         elif lc["type"] == "parallel":
             r = mx["right"]
-            mixer = MixerSpec(attn=attention(mx["left"], True, weights="sigmoid", bias=True, qk_norm=True),
+            mixer = MixerSpec(attn=attention(mx["left"], True, weights="sigmoid", bias=True, o_bias=True, qk_norm=True),
                               linear=LinearAttentionSpec(heads=int(r["heads"]), dim=int(r["dim"]), vdim=int(r["vdim"]), tau=float(r["tau"])))
         else:
             raise ValueError(f"lotelix: unknown layer type {lc['type']!r}")
@@ -805,6 +883,65 @@ def _lotelix(cfg) -> ArchSpec:
         raise ValueError("lotelix: width must be a multiple of norm.groups")
     return stack_arch("lotelix", layers, hidden=width, vocab=int(_get(cfg, "vocab")), norm_eps=float(_get(cfg, "norm")["eps"]),
                       norm_groups=groups, embed_scale=float((_get(cfg, "embedding") or {}).get("scale", 1.0)))
+
+
+@register_arch("relulix")
+def _relulix(cfg) -> ArchSpec:
+    """Relulix: layers of retention or of windowed attention (biases, partly rotated heads, bounded scores, a one more in the
+    denominator; some on another layer's keys and values) in any order, each beside its feed-forward on one norm whose weight is a
+    single number; mixtures of clamped gated experts weighed by the softmax over the chosen ones."""
+
+    def ff(m) -> Optional[FeedForwardSpec]:
+        if m is None:
+            return None
+        if m["kind"] != "moe":
+            raise ValueError(f"relulix: unknown feed-forward kind {m['kind']!r}")
+        f = FeedForwardSpec(ff=int(m["expert"]["ff"]), act="swiglu_clamped", limit=float(m["expert"]["limit"]),
+                            experts=int(m["router"]["experts"]), top=int(m["router"]["top"]), routing="chosen")
+        if not 1 <= f.top <= f.experts:
+            raise ValueError("relulix: a token's experts are at least one and at most all")
+        return f
+
+    def rotation(r, dim) -> RotationSpec:
+        sc = r.get("scaling")
+        slow = {} if sc is None else dict(slow_factor=float(sc["factor"]), slow_low=float(sc["slow"]), slow_high=float(sc["fast"]),
+                                          original=float(sc["original"]), ramp=True, amplitude=0.1 * math.log(sc["factor"]) + 1.0)
+        spec = RotationSpec(dims=int(r["dims"]), base=float(r["base"]), **slow)
+        if spec.dims > dim or spec.dims % 2:
+            raise ValueError("relulix: rot.dims must be even and at most dim")
+        return spec
+
+    layers: List[LayerSpec] = []
+    for i, lc in enumerate(_get(cfg, "layers")):
+        mx = lc["mixer"]
+        if lc["type"] == "retention":
+            m = RetentionSpec(heads=int(mx["heads"]), dim=int(mx["dim"]), vdim=int(mx["vdim"]), decay=[float(d) for d in mx["decay"]],
+                              rot=rotation(mx["rot"], int(mx["dim"])))
+            if len(m.decay) != m.heads:
+                raise ValueError(f"relulix: layer {i} has {m.heads} heads and {len(m.decay)} decays")
+            mixer = MixerSpec(retention=m)
+        elif lc["type"] == "attention":
+            src = mx.get("kv_from")
+            a = AttentionSpec(heads=int(mx["heads"]), kv_heads=int(mx["kv_heads"]), dim=int(mx["dim"]), vdim=int(mx["vdim"]),
+                              scale=float(mx["scale"]), window=int((mx.get("mask") or {}).get("size") or 0),
+                              rot=rotation(mx["rot"], int(mx["dim"])), bias=True, one_more=True, softcap=float(mx.get("softcap") or 0.0),
+                              kv_from=None if src is None else int(src))
+            if a.heads % a.kv_heads:
+                raise ValueError("relulix: heads must be a multiple of kv_heads")
+            if src is not None:
+                own = layers[a.kv_from].mixer.attn if 0 <= a.kv_from < i else None
+                if own is None or own.kv_from is not None or (own.kv_heads, own.dim, own.vdim, own.rot) != (a.kv_heads, a.dim, a.vdim, a.rot):
+                    raise ValueError(f"relulix: layer {i} cannot use the keys and values of layer {src}")
+            mixer = MixerSpec(attn=a)
+        else:
+            raise ValueError(f"relulix: unknown layer type {lc['type']!r}")
+        layers.append(LayerSpec(mixer=mixer, mlp=ff(lc.get("mlp"))))
+    return stack_arch("relulix", layers, hidden=int(_get(cfg, "width")), vocab=int(_get(cfg, "vocab")), norm_eps=float(_get(cfg, "norm")["eps"]),
+                      embed_scale=float((_get(cfg, "embedding") or {}).get("scale", 1.0)), **RELULIX_NORMS)
+
+
+#: Relulix: one norm per layer read by both sublayers, its weight a single number
+RELULIX_NORMS = dict(parallel_residual=True, norm_scalar=True)
 
 
 def stack_arch(model_type: str, layers: List[LayerSpec], hidden: int, vocab: int, norm_eps: float, **kw) -> ArchSpec:
@@ -877,7 +1014,7 @@ def _stack_named() -> Dict[str, ArchSpec]:
             return MixerSpec(attn=AttentionSpec(heads, kv, 128, 128, 128**-0.5, window, rot=RotationSpec(128, 1e6, False, 8.0, 1.0, 4.0, 8192), sink=True,
                                                 gate=True, v_first=v_first))
 
-        both = MixerSpec(attn=AttentionSpec(heads, kv, 128, 128, 128**-0.5, rot=RotationSpec(128, 1e6, True), weights="sigmoid", bias=True, qk_norm=True),
+        both = MixerSpec(attn=AttentionSpec(heads, kv, 128, 128, 128**-0.5, rot=RotationSpec(128, 1e6, True), weights="sigmoid", bias=True, o_bias=True, qk_norm=True),
                          linear=LinearAttentionSpec(heads=width // 128, dim=128, vdim=128, tau=16.0, rank=16))
         mlp = FeedForwardSpec(ff=ff, act="relu2", experts=16, top=2, routing="sigmoid", gated=False)
         return stack_arch("lotelix", [LayerSpec(m, mlp) for m in (MixerSpec(gru=GRUSpec(width)), attn(), both, attn(1))], hidden=width, vocab=32000,

@@ -566,3 +566,32 @@ def map_lotelix(name: str, t: torch.Tensor, spec: ArchSpec) -> List[Piece]:
         if m:
             return [(li, f"moe.experts.{m.group(1)}.{m.group(2)}", t)]
     return []
+
+
+# ---------------------------------------------------------------------------------------------------
+_RELULIX_RETENTION = {n: "retention." + n for n in "qkvgo"}
+_RELULIX_ATTENTION = {"q": "attn.q", "k": "attn.k", "v": "attn.v", "o": "attn.o", "q.b": "attn.q_b", "k.b": "attn.k_b", "v.b": "attn.v_b"}
+
+
+@register_mapper("relulix")
+def map_relulix(name: str, t: torch.Tensor, spec: ArchSpec) -> List[Piece]:
+    top = {"embed": "embed", "final.norm": "final_norm.g", "head": "lm_head"}
+    if name in top:
+        return [(None, top[name], t)]
+    m = _STACK_LAYER.match(name)
+    if not m or int(m.group(1)) >= spec.n_layers:
+        return []
+    li, rest = int(m.group(1)), m.group(2)
+    if rest == "norm1":
+        return [(li, "norm1.g", t)]
+    part, _, leaf = rest.partition(".")
+    if part == "mix":
+        table = _RELULIX_RETENTION if spec.layers[li].mixer.retention is not None else _RELULIX_ATTENTION
+        return [(li, table[leaf], t)] if leaf in table else []
+    if part == "mlp":
+        if leaf in ("router", "router.b"):
+            return [(li, "moe.router" if leaf == "router" else "moe.router_b", t)]
+        m = re.match(r"e(\d+)\.(gate|up|down)$", leaf)
+        if m:
+            return [(li, f"moe.experts.{m.group(1)}.{m.group(2)}", t)]
+    return []

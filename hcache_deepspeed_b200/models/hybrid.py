@@ -22,6 +22,9 @@ supplies what such a layer does between them, and how its checkpoint pieces are 
   kernels then know one pairing, whole heads, and every page size.
 * a minGRU's ``w_qkv`` is ``[gate | candidate | output gate]``; gated linear attention adds ``[q | k | v | gate | decay's first
   projection]`` behind the attention's columns, each padded to 16-byte rows.
+* attention on another layer's keys and values: ``w_qkv`` holds the queries alone, the pages are those of that layer.
+* retention: ``w_qkv`` = ``[q | k | v | gate]``, heads padded to multiples of 16, queries and keys reordered like those of attention;
+  their rotation happens inside the recurrence's kernels, in fp32.
 * two mixers with a norm each: ``w_o`` and ``w_o2`` project their parts of the buffer separately; the norm kernel behind norms both,
   with halved weights, while adding them to the stream.
 * ``parallel_residual``: mixer and dense feed-forward read the same norm, so ``w_o`` is ``[mixer columns | feed-forward columns]``
@@ -42,7 +45,7 @@ from ..ops.backend import (LatentBuffers, latent_launches, pick_decode_splits, p
                            windowed_len)
 from ..ops.kernels import ACT_CODES
 from .arch import (ArchSpec, AttentionSpec, DeltaSpec, FeedForwardSpec, GRUSpec, LatentAttentionSpec, LayerSpec, LinearAttentionSpec, MixerSpec,
-                   StateSpaceSpec)
+                   RetentionSpec, RotationSpec, StateSpaceSpec)
 from .transformer import ACCUM_MAX_TOKENS, RaggedTransformer, ceil_div
 from .weights import ExpertWeights, LayerWeights, ModelWeights, interleave_gate_up
 
@@ -63,9 +66,11 @@ def required_pieces(spec: ArchSpec, l: LayerSpec) -> List[str]:
         req += ["delta." + n for n in ("q", "k", "v", "q_conv", "k_conv", "v_conv", "a", "b", "A_log", "dt_bias", "g", "norm", "o")]
     if l.mixer.attn is not None:
         a = l.mixer.attn
-        req += ["attn.q", "attn.k", "attn.v", "attn.o"] + (["attn.g"] if a.gate else []) + (["attn.sink"] if a.sink else [])
+        own = "qkv" if a.kv_from is None else "q"
+        req += ["attn." + n for n in own + "o"] + (["attn.g"] if a.gate else []) + (["attn.sink"] if a.sink else [])
         req += ["attn.pb"] if a.weights == "sigmoid" else []
-        req += (["attn.q_b", "attn.k_b", "attn.v_b", "attn.o_b"] if a.bias else []) + (["attn.q_norm", "attn.k_norm"] if a.qk_norm else [])
+        req += ([f"attn.{n}_b" for n in own] if a.bias else []) + (["attn.o_b"] if a.o_bias else [])
+        req += ["attn.q_norm", "attn.k_norm"] if a.qk_norm else []
         req += ["attn.vmix"] if a.v_first is not None else []
     if l.mixer.linear is not None:
         req += ["linear." + n for n in ("q", "k", "v", "g", "a1", "a2", "a2_b", "norm", "o")]
@@ -73,6 +78,8 @@ def required_pieces(spec: ArchSpec, l: LayerSpec) -> List[str]:
         req += ["attn.out_norm", "linear.out_norm"]
     if l.mixer.gru is not None:
         req += ["gru." + n for n in ("z", "z_b", "x", "x_b", "g", "o")]
+    if l.mixer.retention is not None:
+        req += ["retention." + n for n in "qkvgo"]
     if l.mixer.ssm is not None:
         req += ["ssm." + n for n in ("in", "conv", "conv_b", "dt_bias", "A_log", "D", "norm", "o")]
     if l.mlp is not None:
@@ -81,7 +88,8 @@ def required_pieces(spec: ArchSpec, l: LayerSpec) -> List[str]:
         parts = ("gate", "up", "down") if l.mlp.gated else ("up", "down")
         if l.mlp.experts:
             req += [f"moe.experts.{e}.{n}" for e in range(l.mlp.experts) for n in parts]
-            req += {"table": ["moe.table"], "softmax": ["moe.router", "moe.correction"], "sigmoid": ["moe.router"]}[l.mlp.routing]
+            req += {"table": ["moe.table"], "softmax": ["moe.router", "moe.correction"], "sigmoid": ["moe.router"],
+                    "chosen": ["moe.router", "moe.router_b"]}[l.mlp.routing]
             if l.mlp.shared_ff:
                 req += ["moe.shared." + n for n in parts]
         else:
@@ -103,26 +111,30 @@ def _head_rows(w: torch.Tensor, heads: int, d: int, page_dim: int) -> torch.Tens
 
 
 def rotated_places(a: AttentionSpec) -> torch.Tensor:
-    """Place inside a page row of every value of a query or key head: the values of rotated pair i at i and page_dim / 2 + i."""
-    r, half = a.rot, a.page_dim // 2
-    i = torch.arange(r.dims // 2)
-    place = torch.empty(a.dim, dtype=torch.long)
-    u, v = (2 * i, 2 * i + 1) if r.adjacent else (i, i + r.dims // 2)
-    place[u], place[v] = i, half + i
-    free = [p for p in range(a.page_dim) if p % half >= r.dims // 2]
-    place[r.dims:] = torch.tensor(free[:a.dim - r.dims], dtype=torch.long)
-    return place
+    """Place inside a page row of every value of a query or key head."""
+    return torch.tensor(a.rot.places(a.dim, a.page_dim), dtype=torch.long)
+
+
+def _rotated_rows(w: torch.Tensor, heads: int, dim: int, width: int, rot: Optional[RotationSpec]) -> torch.Tensor:
+    """Rows (or values) of query or key heads [heads * dim, ...] -> [heads * width, ...], in the kernels' order."""
+    flat = w.reshape(heads, dim, -1)
+    if rot is None:
+        out = _pad(flat, 1, width)
+    else:
+        out = flat.new_zeros(heads, width, flat.shape[2])
+        out[:, torch.tensor(rot.places(dim, width), dtype=torch.long, device=flat.device)] = flat
+    return out.reshape((heads * width, ) + tuple(w.shape[1:]))
 
 
 def _query_rows(w: torch.Tensor, heads: int, a: AttentionSpec) -> torch.Tensor:
-    """Rows (or values) of query or key heads [heads * dim, ...] -> [heads * page_dim, ...], in the kernels' order."""
-    flat = w.reshape(heads, a.dim, -1)
-    if a.rot is None:
-        out = _pad(flat, 1, a.page_dim)
-    else:
-        out = flat.new_zeros(heads, a.page_dim, flat.shape[2])
-        out[:, rotated_places(a).to(flat.device)] = flat
-    return out.reshape((heads * a.page_dim, ) + tuple(w.shape[1:]))
+    return _rotated_rows(w, heads, a.dim, a.page_dim, a.rot)
+
+
+def rotation_table(rot: RotationSpec, width: int) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """(angle per position, amplitude) of the value pairs (c, width / 2 + c) of a row, fp64; amplitudes None: all one."""
+    n, half = rot.dims // 2, width // 2
+    freq = torch.tensor(rot.frequencies() + [0.0] * (half - n), dtype=torch.float64)
+    return freq, None if rot.amplitude == 1.0 else torch.tensor([rot.amplitude] * n + [1.0] * (half - n), dtype=torch.float64)
 
 
 def mixer_factors(m: MixerSpec) -> Tuple[float, float]:
@@ -146,7 +158,7 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
         return t.to(device=device, dtype=torch.float32).contiguous()
 
     def gamma(name: str) -> torch.Tensor:
-        return f32(_pad(spec.norm_weight_offset + p[name].float(), 0, Hp))
+        return f32(_pad(norm_weight(spec, p[name]), 0, Hp))
 
     def ff_weights(prefix: str, ff: int, gated: bool) -> ExpertWeights:
         ffp = pad8(ff)
@@ -189,17 +201,21 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
         # a scale of zero or less cannot be the factor of a running maximum: its sign (or zero) moves into the query rows
         sign = 0.0 if a.scale == 0 else -1.0 if a.scale < 0 else 1.0
         q_sign = 1.0 if a.qk_norm else sign       # (behind a norm it is the norm's weight that carries it)
-        rows += [_query_rows(p["attn.q"] * q_sign, a.heads, a), _query_rows(p["attn.k"], a.kv_heads, a),
-                 _head_rows(p["attn.v"], a.kv_heads, a.vdim, D)]
+        rows.append(_query_rows(p["attn.q"] * q_sign, a.heads, a))
+        if a.kv_from is None:
+            rows += [_query_rows(p["attn.k"], a.kv_heads, a), _head_rows(p["attn.v"], a.kv_heads, a.vdim, D)]
         if a.gate:
             rows.append(_head_rows(p["attn.g"], a.heads, a.vdim, D))
         if a.rot is not None:
-            lw.rot_freq = f32(torch.tensor(a.rot.frequencies() + [0.0] * (D // 2 - a.rot.dims // 2), dtype=torch.float64))
+            freq, amp = rotation_table(a.rot, D)
+            lw.rot_freq, lw.rot_amp = f32(freq), None if amp is None else f32(amp)
         if a.qk_norm:
             lw.q_norm = f32(_query_rows(p["attn.q_norm"].float() * sign, a.heads, a))
             lw.k_norm = f32(_query_rows(p["attn.k_norm"].float(), a.kv_heads, a))
         if a.sink:
             lw.attn_sink = f32(p["attn.sink"])
+        elif a.one_more:
+            lw.attn_sink = torch.zeros(a.heads, dtype=torch.float32, device=device)
         if a.weights == "sigmoid":
             lw.attn_bias = f32(p["attn.pb"])
         if a.v_first is not None:
@@ -228,11 +244,23 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
         rows += [_pad(p["gru." + n], 0, r.inner) for n in "zxg"]
         cols.append(_pad(p["gru.o"], 1, r.inner))
         lw.gru_bias = f32(torch.cat([_pad(p[n], 0, r.inner) for n in ("gru.z_b", "gru.x_b")]))
+    t = l.mixer.retention
+    if t is not None:
+        rows += [_rotated_rows(p["retention." + n], t.heads, t.dim, t.width, t.rot) for n in "qk"]
+        rows += [_head_rows(p["retention." + n], t.heads, t.vdim, t.vwidth) for n in "vg"]
+        cols.append(_pad(p["retention.o"].reshape(spec.hidden, t.heads, t.vdim), 2, t.vwidth).reshape(spec.hidden, t.inner))
+        # (logarithms to base 2 from fp64: a power of the decay is one rounded product away)
+        lw.ret_decay = f32(torch.tensor(t.decay, dtype=torch.float64).clamp(min=0).log2().clamp(min=RETENTION_LOG_FLOOR))
+        lw.ssm_norm = torch.ones(t.inner, dtype=torch.float32, device=device)
+        freq, amp = rotation_table(t.rot or RotationSpec(0, 1.0), t.width)
+        lw.rot_freq, lw.rot_amp = f32(freq), None if amp is None else f32(amp)
     lw.w_qkv = to(_pad(torch.cat(rows, dim=0), 1, Hp))
     if a is not None and a.bias:
-        b = [_query_rows(p["attn.q_b"] * q_sign, a.heads, a), _query_rows(p["attn.k_b"], a.kv_heads, a),
-             _head_rows(p["attn.v_b"][:, None], a.kv_heads, a.vdim, a.page_dim).reshape(-1)]
+        b = [_query_rows(p["attn.q_b"] * q_sign, a.heads, a)]
+        if a.kv_from is None:
+            b += [_query_rows(p["attn.k_b"], a.kv_heads, a), _head_rows(p["attn.v_b"][:, None], a.kv_heads, a.vdim, a.page_dim).reshape(-1)]
         lw.b_qkv = to(_pad(torch.cat(b), 0, lw.w_qkv.shape[0]))
+    if a is not None and a.o_bias:
         lw.b_o = to(_pad(p["attn.o_b"], 0, Hp))
     f = l.mlp
     if f is not None:
@@ -247,7 +275,8 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
                 lw.moe_table = p["moe.table"].to(device=device, dtype=torch.int32).contiguous()
             else:
                 lw.w_router = to(_pad(_pad(p["moe.router"], 0, pad8(f.experts)), 1, Hp))
-                lw.router_bias = f32(p["moe.correction"]) if f.routing == "softmax" else None
+                bias = {"softmax": "moe.correction", "chosen": "moe.router_b"}.get(f.routing)
+                lw.router_bias = f32(p[bias]) if bias else None
             if f.shared_ff:
                 lw.shared_expert = ff_weights("moe.shared.", f.shared_ff, f.gated)
         else:
@@ -258,6 +287,16 @@ def layer_weights(spec: ArchSpec, l: LayerSpec, p: Dict[str, torch.Tensor], dtyp
                 lw.w_down = None
     lw.w_o = to(_pad(torch.cat(cols, dim=1), 0, Hp))
     return lw
+
+
+#: log2 of the least decay per token: what it leaves is zero to everything behind it
+RETENTION_LOG_FLOOR = -200.0
+
+
+def norm_weight(spec: ArchSpec, t: torch.Tensor) -> torch.Tensor:
+    """A stored norm weight as one value per coordinate."""
+    t = spec.norm_weight_offset + t.float()
+    return t.reshape(1).expand(spec.hidden) if spec.norm_scalar else t
 
 
 def rotation_frequencies(dims: int, base: float) -> torch.Tensor:
@@ -276,7 +315,7 @@ def top_weights(spec: ArchSpec, top: Dict[str, torch.Tensor], out: ModelWeights,
     out.embed = _pad(top["embed"], 1, Hp).to(device=device, dtype=dtype).contiguous()
 
     def gamma(name: str) -> torch.Tensor:
-        return _pad(spec.norm_weight_offset + top[name].float(), 0, Hp).to(device=device).contiguous()
+        return _pad(norm_weight(spec, top[name]), 0, Hp).to(device=device).contiguous()
 
     out.final_norm_g = gamma("final_norm.g")
     if spec.embed_norm:
@@ -294,8 +333,8 @@ def random_pieces(spec: ArchSpec, l: LayerSpec, gen: torch.Generator, device: to
     def rnd(*shape, scale=std):
         return torch.randn(shape, generator=gen, device=device, dtype=torch.float32) * scale
 
-    def norm_g(n=H):
-        return 1.0 - spec.norm_weight_offset + rnd(n, scale=0.05)
+    def norm_g():
+        return 1.0 - spec.norm_weight_offset + rnd(1 if spec.norm_scalar else H, scale=0.05)
 
     p = {"norm1.g": norm_g(), "norm1b.g": norm_g()}
     a, m, f, c, d, g, r = l.mixer.attn, l.mixer.ssm, l.mlp, l.mixer.latent, l.mixer.delta, l.mixer.linear, l.mixer.gru
@@ -327,6 +366,10 @@ def random_pieces(spec: ArchSpec, l: LayerSpec, gen: torch.Generator, device: to
                   "attn.pb": rnd(a.heads, scale=0.5) - 4.0, "attn.vmix": 0.5 + rnd(1, scale=0.1)[0], "attn.q_b": rnd(a.heads * a.dim),
                   "attn.k_b": rnd(a.kv_heads * a.dim), "attn.v_b": rnd(a.kv_heads * a.vdim), "attn.o_b": rnd(H),
                   "attn.q_norm": 1.0 + rnd(a.heads * a.dim, scale=0.05), "attn.k_norm": 1.0 + rnd(a.kv_heads * a.dim, scale=0.05)})
+    t = l.mixer.retention
+    if t is not None:
+        p.update({"retention.q": rnd(t.heads * t.dim, H), "retention.k": rnd(t.heads * t.dim, H), "retention.v": rnd(t.heads * t.vdim, H),
+                  "retention.g": rnd(t.heads * t.vdim, H), "retention.o": rnd(H, t.heads * t.vdim)})
     if m is not None:
         p.update({"ssm.in": rnd(m.in_dim, H), "ssm.conv": rnd(m.conv_dim, m.conv, scale=0.3), "ssm.conv_b": rnd(m.conv_dim),
                   "ssm.dt_bias": rnd(m.heads, scale=0.5) - 3.0, "ssm.A_log": rnd(m.heads, scale=0.5), "ssm.D": rnd(m.heads, scale=1.0),
@@ -345,7 +388,7 @@ def random_pieces(spec: ArchSpec, l: LayerSpec, gen: torch.Generator, device: to
             if f.routing == "table":
                 p["moe.table"] = torch.argsort(torch.rand((spec.vocab, f.experts), generator=gen, device=device), dim=1)[:, :f.top].int()
             else:
-                p.update({"moe.router": rnd(f.experts, H), "moe.correction": rnd(f.experts, scale=0.05)})
+                p.update({"moe.router": rnd(f.experts, H), "moe.correction": rnd(f.experts, scale=0.05), "moe.router_b": rnd(f.experts, scale=0.05)})
             if f.shared_ff:
                 glu("moe.shared.", f.shared_ff)
         else:
@@ -357,7 +400,7 @@ def random_stack_weights(spec: ArchSpec, dtype: torch.dtype, device: torch.devic
     gen = torch.Generator(device=device).manual_seed(seed)
     mw = ModelWeights(layers=[layer_weights(spec, l, random_pieces(spec, l, gen, device, std), dtype, device) for l in spec.layers])
     top = {"embed": torch.randn((spec.vocab, spec.hidden), generator=gen, device=device) * std,
-           "final_norm.g": 1.0 - spec.norm_weight_offset + torch.randn(spec.hidden, generator=gen, device=device) * 0.05,
+           "final_norm.g": 1.0 - spec.norm_weight_offset + torch.randn(1 if spec.norm_scalar else spec.hidden, generator=gen, device=device) * 0.05,
            "embed_norm.g": 1.0 - spec.norm_weight_offset + torch.randn(spec.hidden, generator=gen, device=device) * 0.05,
            "lm_head": torch.randn((spec.vocab, spec.hidden), generator=gen, device=device) * std}
     return top_weights(spec, top, mw, dtype, device)
@@ -396,7 +439,7 @@ class HybridTransformer(RaggedTransformer):
 
         def shape(m: MixerSpec):
             if m.attn is not None:
-                return 2, m.attn.kv_heads, m.attn.page_dim
+                return (2, m.attn.kv_heads, m.attn.page_dim) if m.attn.kv_from is None else None
             if m.latent is not None and m.latent.kv_from is None:
                 return 1, 1, m.latent.page_width
             return None
@@ -406,7 +449,7 @@ class HybridTransformer(RaggedTransformer):
     def recurrent_state_config(self):
         if not self.spec.has_recurrent_state:
             return None
-        return [None if m is None else RecurrentLayerConfig(heads=m.heads, vdim=m.vdim, state=m.state, conv_dim=m.conv_dim, taps=m.conv)
+        return [None if m is None else RecurrentLayerConfig(heads=m.heads, vdim=m.vwidth if isinstance(m, RetentionSpec) else m.vdim, state=m.state, conv_dim=m.conv_dim, taps=m.conv)
                 for m in (l.mixer.recurrent for l in self.spec.layers)]
 
     def graphable_decode(self, batch: RaggedBatchWrapper) -> bool:
@@ -474,6 +517,7 @@ class HybridTransformer(RaggedTransformer):
         if latents:
             self._latent_bufs = LatentBuffers(latents, self._state_config, self.kv_block_size, dt, dev)
         n_ws = max([k.gru_workspace_bytes(T, S, m.inner) for m in rec if isinstance(m, GRUSpec)] +
+                   [k.retention_workspace_bytes(T, S, m.heads, m.vwidth, m.width) for m in rec if isinstance(m, RetentionSpec) and dt == torch.bfloat16] +
                    [k.linear_attention_workspace_bytes(T, S, m.heads, m.vdim, m.dim) for m in linear if dt == torch.bfloat16], default=0)
         self._scan_ws = torch.empty(n_ws, dtype=torch.uint8, device=dev) if n_ws else None
         if dt != torch.float32:
@@ -528,6 +572,8 @@ class HybridTransformer(RaggedTransformer):
             n_mix = self._delta_mixer(li, l.mixer.delta, lw, xn, mix, batch)
         elif l.mixer.gru is not None:
             n_mix = self._gru_mixer(li, l.mixer.gru, lw, xn, mix, batch)
+        elif l.mixer.retention is not None:
+            n_mix = self._retention_mixer(li, l.mixer.retention, lw, xn, mix, batch)
         else:
             n_mix = self._attention_and_scan(li, l, lw, xn, mix, batch)
         factor, f = mixer_factors(l.mixer)[0], l.mlp
@@ -557,13 +603,14 @@ class HybridTransformer(RaggedTransformer):
         n_attn = n_out = 0
         if a is not None:
             D = a.page_dim
-            n_attn, n_out = (a.heads + 2 * a.kv_heads) * D, a.heads * D
+            n_attn, n_out = (a.heads + 2 * a.cached_heads) * D, a.heads * D
             q = self._view(self.q_buf, T, n_out)
             ops.mixer_in_proj(xn, lw, a, proj, q, kv.get_cache(li), self._first_values(a), batch.tok_pos(), batch.tok_slot(),
                               kv.kv_block_size, self.spec.norm_eps, workspace=self.ws_gemm)
-            ops.attention(q, mix[:, :n_out], kv.get_cache(li), batch, a.heads, a.kv_heads, D, abs(a.scale) or 1.0,
-                          ws_small=self.ws_small, ws_large=self.ws_large, window=a.window, keep_first=a.keep_first, sink=lw.attn_sink,
-                          sigmoid_bias=lw.attn_bias, gate=proj[:, n_attn:n_attn + n_out] if a.gate else None)
+            ops.attention(q, mix[:, :n_out], kv.get_cache(li if a.kv_from is None else a.kv_from), batch, a.heads, a.kv_heads, D,
+                          abs(a.scale) or 1.0, ws_small=self.ws_small, ws_large=self.ws_large, window=a.window, keep_first=a.keep_first,
+                          sink=lw.attn_sink, sigmoid_bias=lw.attn_bias, gate=proj[:, n_attn:n_attn + n_out] if a.gate else None,
+                          softcap=a.softcap)
         else:
             ops.gemm(xn, lw.w_qkv, proj[:, :lw.w_qkv.shape[0]], workspace=self.ws_gemm)
         if g is not None:
@@ -613,6 +660,20 @@ class HybridTransformer(RaggedTransformer):
                      self._scan_ws)
         return r.inner
 
+    def _retention_mixer(self, li: int, t: RetentionSpec, lw: LayerWeights, xn: torch.Tensor, mix: torch.Tensor, batch: RaggedBatchWrapper) -> int:
+        proj = self._view(self.in_buf, batch.current_tokens, lw.w_qkv.shape[0])
+        self.ops.gemm(xn, lw.w_qkv, proj, workspace=self.ws_gemm)
+        self._retention(li, t, lw, proj, batch.spans(), batch.n_single_token_seqs, mix[:, :t.inner])
+        return t.inner
+
+    def _retention(self, li: int, t: RetentionSpec, lw: LayerWeights, proj: torch.Tensor, spans: torch.Tensor, n_single: int,
+                   out: Optional[torch.Tensor]) -> None:
+        """Retention of the tokens whose projections are ``proj`` = [q | k | v | gate]; without ``out`` its state alone."""
+        nk, nv = t.keys, t.inner
+        self.ops.retention(proj[:, :nk], proj[:, nk:2 * nk], proj[:, 2 * nk:2 * nk + nv], proj[:, 2 * nk + nv:], lw, t,
+                           self._state_manager.recurrent_states.ssm(li), spans, n_single, self._view(self.scan_buf, proj.shape[0], nv), out,
+                           self.spec.norm_eps, self._scan_ws)
+
     def _linear(self, li: int, g: LinearAttentionSpec, lw: LayerWeights, proj: torch.Tensor, spans: torch.Tensor, n_single: int,
                 out: Optional[torch.Tensor]) -> None:
         """Gated linear attention of the tokens whose projections are ``proj`` = [q | k | v | gate | decay's first projection]; without
@@ -655,6 +716,8 @@ class HybridTransformer(RaggedTransformer):
             ops.table_route(batch.input_ids(), lw, f, bufs)
         elif f.routing == "sigmoid":
             ops.sigmoid_route(x, lw, f, bufs)
+        elif f.routing == "chosen":
+            ops.chosen_route(x, lw, f, bufs)
         else:
             ops.softmax_route(x, lw, f, bufs)
         return ops.routed_experts(x, batch.input_ids(), lw, f, act, base, self.delta32[:T], bufs)
@@ -680,7 +743,7 @@ class HybridTransformer(RaggedTransformer):
             part = proj[:, c.heads * c.head_width:lw.w_qkv.shape[0]]
             ops.gemm(latents, lw.w_qkv[c.heads * c.head_width:], part, workspace=self.ws_gemm)
             ops.latent_append(proj, None, kv.get_cache(li), pos, slot, c, lw, self.spec.norm_eps)
-        if a is not None:
+        if a is not None and a.kv_from is None:
             n_q = a.heads * a.page_dim
             n_attn = n_q + 2 * a.kv_heads * a.page_dim
             if a.rot is not None or a.qk_norm or a.v_first is not None:
@@ -693,6 +756,10 @@ class HybridTransformer(RaggedTransformer):
         if isinstance(m, GRUSpec):
             ops.gemm(latents, lw.w_qkv, proj, workspace=self.ws_gemm)
             ops.gru(proj, lw, m, kv.recurrent_states.ssm(li), spans, n_single, None, self._scan_ws)
+        elif isinstance(m, RetentionSpec):
+            proj = self._view(self.in_buf, T, lw.w_qkv.shape[0])
+            ops.gemm(latents, lw.w_qkv, proj, workspace=self.ws_gemm)
+            self._retention(li, m, lw, proj, spans, n_single, None)
         elif isinstance(m, LinearAttentionSpec):
             ops.gemm(latents, lw.w_qkv[n_attn:], proj[:, n_attn:], workspace=self.ws_gemm)
             self._linear(li, m, lw, proj[:, n_attn:], spans, n_single, None)

@@ -72,6 +72,7 @@ class LayerWeights:
     # latent attention
     latent_norm: Optional[torch.Tensor] = None    # fp32 [kv_rank]
     rot_freq: Optional[torch.Tensor] = None       # fp32 [rot_dim / 2]
+    rot_amp: Optional[torch.Tensor] = None        # fp32, like rot_freq: factors of the rotated pairs
     w_uk: Optional[torch.Tensor] = None           # [heads, dim, kv_rank]: takes a head's query to the latent space
     w_uv: Optional[torch.Tensor] = None           # [heads, kv_rank, vdim]: takes a head's mean latent to its value
     w_kv: Optional[torch.Tensor] = None           # [2 * heads * head_width, page_width]: cached rows -> K / V pages (16-bit models)
@@ -90,6 +91,7 @@ class LayerWeights:
     w_decay: Optional[torch.Tensor] = None
     decay_bias: Optional[torch.Tensor] = None
     gru_bias: Optional[torch.Tensor] = None
+    ret_decay: Optional[torch.Tensor] = None      # fp32 [heads]: log2 of retention's decays
 
     def stack_experts(self) -> None:
         """Store the experts as consecutive slices of one tensor per matrix, the operands of the grouped GEMM."""

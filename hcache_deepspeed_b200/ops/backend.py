@@ -31,6 +31,12 @@ def windowed_len(n_keys: int, window: int, keep_first: int = 0) -> int:
     return min(n_keys, window + 256 + (keep_first + 127) // 128 * 128) if window else n_keys
 
 
+def padded_head_norm(m, eps: float):
+    """(eps, factor) that make a norm over the zero-padded rows of retention's heads one over their own values."""
+    r = m.vwidth / m.vdim
+    return eps / r, r**-0.5
+
+
 class CpuOps:
     name = "cpu-reference"
 
@@ -87,13 +93,13 @@ class CpuOps:
         ref.kv_append(kv_layer, k, v, tok_slot)
 
     def attention(self, q, out, kv_layer, batch, n_q, n_kv, d, scale, ws_small=None, ws_large=None, alibi=None, window=0,
-                  keep_first=0, sink=None, sigmoid_bias=None, gate=None):
+                  keep_first=0, sink=None, sigmoid_bias=None, gate=None, softcap=0.0):
         T = q.shape[0]
         q3, o3 = q.view(T, n_q, d), out.view(T, n_q, d)
         for items in (batch.items_small(), batch.items_large()):
             if items.shape[0]:
                 ref.paged_attention(q3, kv_layer, batch.block_tables(), items, n_q, n_kv, scale, out=o3, alibi=alibi,
-                                    window=window, keep_first=keep_first, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate)
+                                    window=window, keep_first=keep_first, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate, softcap=softcap)
 
     # ---- stacks of unlike layers ----------------------------------------------------------------------
     def embed_f32(self, ids, weight, out, gamma=None, cols=None, eps=1e-5, scale=1.0):
@@ -117,8 +123,8 @@ class CpuOps:
         self.attention_append(proj, lw, a, q_out, kv_layer, first, tok_pos, tok_slot, block_size, eps)
 
     def attention_append(self, proj, lw, a, q_out, kv_layer, first, tok_pos, tok_slot, block_size, eps):
-        q = ref.attention_append(proj, kv_layer, tok_pos, tok_slot, a.heads if q_out is not None else 0, a.kv_heads, lw.rot_freq,
-                                 lw.q_norm, lw.k_norm, a.heads * a.dim, a.kv_heads * a.dim, eps, first, lw.v_mix)
+        q = ref.attention_append(proj, kv_layer, tok_pos, tok_slot, a.heads if q_out is not None else 0, a.cached_heads, lw.rot_freq,
+                                 lw.q_norm, lw.k_norm, a.heads * a.dim, a.kv_heads * a.dim, eps, first, lw.v_mix, lw.rot_amp, a.page_dim)
         if q_out is not None:
             q_out.copy_(q)
 
@@ -176,6 +182,18 @@ class CpuOps:
             out.zero_()
             out[:, :NV] = ref.gated_norm(y[:, :NV], gate[:, :NV], lw.ssm_norm, m.heads, eps, gate_after=True)
 
+    def retention(self, q, k, v, gate, lw, m, state, spans, n_single, y, out, eps, workspace):
+        for row0, n, seen, slot in spans.tolist():
+            if seen == 0:
+                state[slot].zero_()
+            pos = torch.arange(seen, seen + n)
+            turned = lambda t: ref.rotate_halves(t[row0:row0 + n].reshape(n, m.heads, m.width), pos, lw.rot_freq, lw.rot_amp)  # noqa: E731
+            y[row0:row0 + n] = ref.retention_scan(turned(q), turned(k), v[row0:row0 + n].reshape(n, m.heads, m.vwidth), lw.ret_decay, m.dim**-0.5,
+                                                  state[slot]).reshape(n, m.inner)
+        if out is not None:
+            head_eps, scale = padded_head_norm(m, eps)
+            out.copy_(ref.gated_norm(y, gate, lw.ssm_norm, m.heads, head_eps, scale, gate_after=True))
+
     def latent_append(self, proj, q_out, pages, tok_pos, tok_slot, c, lw, eps):
         n_q = c.heads * c.head_width
         if q_out is not None:
@@ -212,6 +230,10 @@ class CpuOps:
     def sigmoid_route(self, x, lw, f, bufs):
         s = torch.sigmoid(ref.gemm(x, lw.w_router, out_dtype=torch.float32)[:, :f.experts])
         self._scores, self._picked = torch.topk(s, f.top, -1)
+
+    def chosen_route(self, x, lw, f, bufs):
+        z, self._picked = torch.topk(ref.gemm(x, lw.w_router, out_dtype=torch.float32)[:, :f.experts] + lw.router_bias, f.top, -1)
+        self._scores = torch.softmax(z, -1)
 
     def routed_experts(self, x, ids, lw, f, act, base, out, bufs):
         """``out`` = ``base`` (None, or ``out`` itself) + the chosen experts' weighted outputs (the outputs of weighted inputs,
@@ -362,16 +384,16 @@ class CudaOps:
             self.k.rope_kv_append(scratch, scratch, kv_layer, tok_pos, tok_slot, inv_freq, 0, n_kv, d, rot_dim, block_size)
 
     def attention(self, q, out, kv_layer, batch, n_q, n_kv, d, scale, ws_small=None, ws_large=None, alibi=None, window=0,
-                  keep_first=0, sink=None, sigmoid_bias=None, gate=None):
+                  keep_first=0, sink=None, sigmoid_bias=None, gate=None, softcap=0.0):
         k = self.k
         bs = batch.block_size
         if q.dtype == torch.float32 or d not in (64, 128):
             k.paged_attention_generic(q, out, kv_layer, batch.block_tables(), batch.tokens_to_seq(), batch.tok_pos(), n_q, n_kv, d, bs,
-                                      scale, window=window, keep_first=keep_first, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate)
+                                      scale, window=window, keep_first=keep_first, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate, softcap=softcap)
             return
         # with a sliding window an item reads at most window + one tile of keys: size the KV split for that
         seen = lambda n_kv_tokens: windowed_len(n_kv_tokens, window, keep_first)  # noqa: E731
-        opts = dict(alibi=alibi, window=window, keep_first=keep_first, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate)
+        opts = dict(alibi=alibi, window=window, keep_first=keep_first, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate, softcap=softcap)
         if batch.n_items_small:
             n = batch.n_items_small
             if use_packed_decode(n_q, n_kv, d):
@@ -402,10 +424,10 @@ class CudaOps:
         rotating and paged epilogue (where no norm comes before it) and run the others as a second GEMM. ``first``: pages of the
         layer whose values are mixed in."""
         k, T, d, w_in, b = self.k, x.shape[0], a.page_dim, lw.w_qkv, lw.b_qkv
-        n_in, n_attn = w_in.shape[0], (a.heads + 2 * a.kv_heads) * d
+        n_in, n_attn, n_kv = w_in.shape[0], (a.heads + 2 * a.cached_heads) * d, a.cached_heads
         if x.dtype != torch.float32 and d in (64, 128) and T >= self.FUSED_QKV_MIN_TOKENS and not a.qk_norm:
-            k.qkv_rope_proj(x, w_in[:n_attn], q_out, kv_layer, tok_pos, tok_slot, lw.rot_freq, a.heads, a.kv_heads, d, block_size,
-                            bias_qkv=None if b is None else b[:n_attn])
+            k.qkv_rope_proj(x, w_in[:n_attn], q_out, kv_layer, tok_pos, tok_slot, lw.rot_freq, a.heads, n_kv, d, block_size,
+                            bias_qkv=None if b is None else b[:n_attn], amp=lw.rot_amp)
             if n_in > n_attn:
                 k.gemm(x, w_in[n_attn:], out=proj[:, n_attn:n_in], bias=None if b is None else b[n_attn:])
             if first is not None:
@@ -418,9 +440,9 @@ class CudaOps:
         """Projected rows [q | k | v] -> rotated (and normed) queries and page rows. ``q_out`` None: keys and values only."""
         k, d, n_q = self.k, a.page_dim, a.heads if q_out is not None else 0
         q_out = proj if q_out is None else q_out
-        if a.rot is not None or a.qk_norm or first is not None:
-            k.attention_append(proj, q_out, kv_layer, tok_pos, tok_slot, n_q, a.kv_heads, d, block_size, lw.rot_freq, lw.q_norm, lw.k_norm,
-                               a.heads * a.dim, a.kv_heads * a.dim, eps, first, lw.v_mix)
+        if a.rot is not None or a.qk_norm or first is not None or a.kv_from is not None:
+            k.attention_append(proj, q_out, kv_layer, tok_pos, tok_slot, n_q, a.cached_heads, d, block_size, lw.rot_freq, lw.q_norm, lw.k_norm,
+                               a.heads * a.dim, a.kv_heads * a.dim, eps, first, lw.v_mix, lw.rot_amp)
         elif proj.dtype == torch.float32:
             k.kv_append_generic(proj, q_out, kv_layer, tok_slot, n_q, a.kv_heads, d, block_size)
         else:
@@ -431,6 +453,10 @@ class CudaOps:
 
     def linear_attention(self, q, k, v, gate, z, lw, m, state, spans, n_single, y, out, eps, workspace):
         self.k.linear_attention(q, k, v, gate, z, lw.decay_bias, 1.0 / m.tau, state, spans, n_single, y, out, lw.ssm_norm, eps, workspace)
+
+    def retention(self, q, k, v, gate, lw, m, state, spans, n_single, y, out, eps, workspace):
+        self.k.retention(q, k, v, gate, lw.ret_decay, lw.rot_freq, lw.rot_amp, m.dim**-0.5, m.vdim, state, spans, n_single, y, out, lw.ssm_norm, eps,
+                         workspace)
 
     def state_space(self, proj, lw, m, ssm_state, conv_state, spans, n_single, conv_buf, dt_buf, out):
         return self.k.state_space(proj, lw.ssm_conv_w, lw.ssm_conv_b, lw.ssm_dt_bias, lw.ssm_a, lw.ssm_d, ssm_state, conv_state, spans,
@@ -459,6 +485,14 @@ class CudaOps:
         k.gemm_accum(x, lw.w_router, logits)
         k.moe_topk_gating(logits[:, :f.experts], f.top, False, bufs["scores"][:T], bufs["expert_ids"][:T], bufs["offsets"][:T], bufs["counts"],
                           clear=True, sigmoid=True)
+
+    def chosen_route(self, x, lw, f, bufs):
+        """Experts by router: the largest fp32 logits, bias included, weighed by the softmax over them."""
+        k, T = self.k, x.shape[0]
+        logits = bufs["logits"][:T]
+        k.gemm_accum(x, lw.w_router, logits)
+        k.moe_topk_gating(logits[:, :f.experts], f.top, True, bufs["scores"][:T], bufs["expert_ids"][:T], bufs["offsets"][:T], bufs["counts"],
+                          bias=lw.router_bias, clear=True, biased=True)
 
     def routed_experts(self, x, ids, lw, f, act, base, out, bufs):
         """Routed tokens: scatter -> grouped GEMM -> grouped GEMM -> weighted sum, added to ``base`` (``out`` itself: in place)."""

@@ -30,7 +30,7 @@ CUDA_LIB = LIB_DIR / "libhds_b200.so"
 SERVE_LIB = LIB_DIR / "libhds_serve.so"
 SERVE_UNITS = ("gemm", "gemm_2sm", "gemm_f32", "elementwise", "residual_norm", "attention_splitkv", "attention_prefill",
                "attention_generic", "attention_latent", "attention_append", "latent", "moe", "ssm", "ssm_chunk", "delta", "delta_chunk", "gru",
-               "linear_attention", "linear_chunk", "tp_comm")
+               "linear_attention", "linear_chunk", "retention", "tp_comm")
 HOST_LIB = LIB_DIR / "libhds_host.so"
 
 NVCC_FLAGS = [

@@ -20,6 +20,7 @@ struct AppendArgs {
     const int32_t* tok_pos;
     const int32_t* tok_slot;    // negative: nothing is cached
     const float* freq;          // [D / 2] or nullptr
+    const float* amp;           // [D / 2] factors of sines and cosines, or nullptr
     const float* q_norm;        // [n_q * D] and [n_kv * D], or nullptr
     const float* k_norm;
     int q_cols, k_cols;         // values the two means are taken over (padding excluded)
@@ -85,7 +86,13 @@ __global__ void __launch_bounds__(kAaThreads) attention_append_kernel(const Appe
     const int64_t row = t * a.ld;
     if (a.freq != nullptr) {
         const float pos = static_cast<float>(a.tok_pos[t]);
-        for (int c = threadIdx.x; c < half; c += kAaThreads) aa_sincos<DT>(pos * a.freq[c], &cs[half + c], &cs[c]);
+        for (int c = threadIdx.x; c < half; c += kAaThreads) {
+            float s, co;
+            aa_sincos<DT>(pos * a.freq[c], &s, &co);
+            const float m = a.amp != nullptr ? a.amp[c] : 1.0f;
+            cs[half + c] = s * m;
+            cs[c] = co * m;
+        }
     }
     float rq = 1.0f, rk = 1.0f;
     if (a.k_norm != nullptr) {
@@ -128,7 +135,7 @@ __global__ void __launch_bounds__(kAaThreads) attention_append_kernel(const Appe
         aa_store<DT>(dst, o, x);
         aa_store<DT>(dst, o + half, y);
     }
-    if (slot < 0) return;
+    if (slot < 0 || a.n_kv == 0) return;
     const float share = a.first != nullptr ? *a.share : 0.0f;
     for (int u = threadIdx.x * 4; u < a.n_kv * D; u += kAaThreads * 4) {
         const int h = u / D, c = u - h * D;
@@ -166,7 +173,7 @@ using namespace hds;
 
 extern "C" int hds_attention_append(const void* qkv, int64_t ld_qkv, void* q_out, void* kv_cache_layer, const int32_t* tok_pos,
                                     const int32_t* tok_slot, int T, int n_q_heads, int n_kv_heads, int head_dim, int block_size,
-                                    const float* freq, const float* q_norm, const float* k_norm, int q_cols, int k_cols, float eps,
+                                    const float* freq, const float* amp, const float* q_norm, const float* k_norm, int q_cols, int k_cols, float eps,
                                     const void* first, int first_dim, const float* share, int dtype, void* stream) {
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_attention_append: dtype 0 bf16 / 1 fp16 / 2 fp32");
     HDS_REQUIRE(head_dim >= 8 && head_dim % 8 == 0 && head_dim <= 8192 && ld_qkv % 4 == 0, "hds_attention_append: heads of 8-value multiples");
@@ -174,7 +181,8 @@ extern "C" int hds_attention_append(const void* qkv, int64_t ld_qkv, void* q_out
     HDS_REQUIRE(k_norm == nullptr || (k_cols > 0 && q_cols > 0 && (q_norm != nullptr || n_q_heads == 0)), "hds_attention_append: norms of q and k");
     HDS_REQUIRE(first == nullptr || (share != nullptr && first_dim % 4 == 0), "hds_attention_append: a share for the mixed values");
     if (T == 0) return HDS_OK;
-    const AppendArgs a{qkv, ld_qkv, q_out, kv_cache_layer, tok_pos, tok_slot, freq, q_norm, k_norm, q_cols, k_cols, eps,
+    HDS_REQUIRE(n_kv_heads == 0 || kv_cache_layer != nullptr, "hds_attention_append: pages for the keys and values");
+    const AppendArgs a{qkv, ld_qkv, q_out, kv_cache_layer, tok_pos, tok_slot, freq, amp, q_norm, k_norm, q_cols, k_cols, eps,
                        first, first_dim, share, n_q_heads, n_kv_heads, head_dim, block_size};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     const size_t smem = static_cast<size_t>(head_dim) * 4;

@@ -62,6 +62,7 @@ paged_attn_generic_kernel(const void* __restrict__ q, void* __restrict__ out, in
                 vrow = krow + v_plane;
                 s = 0.0f;
                 for (int c = 0; c < D; ++c) s = fmaf(qw[c], load_any<DT>(cache, krow + c), s);
+                if (opt.softcap > 0.0f) s = opt.softcap * tanhf(s / opt.softcap);
             }
             const float m_new = sigmoid ? 0.0f : fmaxf(m, warp_max(s));
             const float keep = m == -INFINITY ? 0.0f : expf(m - m_new);

@@ -10,6 +10,7 @@
 //               warps to interleave: ONE tcgen05.ld pass pulls this thread's 64 scores into
 //               registers and releases S at once (so Q K^T of the next tile runs under this tile's exponentials),
 //               causal mask, online max/sum, P -> shared (UMMA K-major swizzled layout).
+//   Bounded scores (kCapped) replace the raw ones in registers, in log2 units, before the mask.
 //   Sigmoid weights (kSigmoid) need neither maximum nor sum: P = sigmoid(S + a number per head), O is the plain sum of P V.
 //   A learned sink joins the row sum at the very end, where an output gate is applied too.
 //   O accumulates in TMEM across all KV tiles (PV issued with accumulate); it is rescaled in place only when a
@@ -55,7 +56,11 @@ struct PrefillArgs {
     const float* sigmoid_bias;  // kSigmoid: [n_q_heads], natural-log units
     const void* gate;   // nullptr, or rows (gate_ld apart) like out's whose sigmoid multiplies it
     int64_t gate_ld;
+    float cap_log2, cap_k;      // kCapped: bounded scores (softcap_log2 of raw ones)
 };
+
+// what turns scores into weights: softmax, sigmoids, softmax of bounded scores
+enum PrefillWeights : int { PF_SOFTMAX = 0, PF_SIGMOID = 1, PF_CAPPED = 2 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
     float y;
@@ -104,10 +109,11 @@ __device__ __forceinline__ void pf_store8(const PrefillArgs& a, const float* o, 
     st_v4(reinterpret_cast<char*>(a.out) + (row * a.out_ld + col) * 2, v);
 }
 
-template <int D, bool kBf16, bool kPacked = false, bool kSigmoid = false>
+template <int D, bool kBf16, bool kPacked = false, int kWeights = PF_SOFTMAX>
 __global__ void __launch_bounds__(kPfThreads, 1)
 paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
                           const PrefillArgs a) {
+    constexpr bool kSigmoid = kWeights == PF_SIGMOID, kCapped = kWeights == PF_CAPPED;
     constexpr int PANELS = D / 64;
     constexpr int PANEL_BYTES = kPfTok * 128;  // [128 rows x 128 B]
     constexpr int TILE_BYTES = PANELS * PANEL_BYTES;
@@ -285,6 +291,7 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         const uint32_t lane_addr = (quad * 32u) << 16;
         constexpr int HC = kPfTok / 2;               // key columns per thread
         constexpr int HD2 = D / 2;                   // output dims per thread
+        const float to_log2 = kCapped ? 1.0f : a.scale_log2;
         float m_run = kSigmoid ? 0.0f : -INFINITY, l_run = 0.0f;       // l_run: this thread's columns only
         const float sig_bias = kSigmoid ? a.sigmoid_bias[min(r_head, a.n_q_heads - 1)] * -1.4426950408889634f : 0.0f;
         uint8_t* p_row = p_sm + half * PANEL_BYTES + r * 128;   // half h owns P panel h (64 tokens = 128 B per row)
@@ -322,7 +329,11 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(s_empty);
-            if (a.alibi != nullptr) {
+            if constexpr (kCapped) {
+#pragma unroll
+                for (int j = 0; j < HC; ++j) sr[j] = __float_as_uint(softcap_log2(__uint_as_float(sr[j]), a.cap_k, a.cap_log2));
+            }
+            if (!kCapped && a.alibi != nullptr) {
                 // ALiBi: raw score += slope * (key - query position), expressed in raw-score units so that the scaling below
                 // stays one multiply-add per element (kernel-uniform branch; slopes differ per row only in packed mode)
                 const float sl = a.alibi[r_head] * 1.4426950408889634f / a.scale_log2;
@@ -361,7 +372,7 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
             pair_sync();
             tmax = fmaxf(tmax, x[(half ^ 1) * 128 + r]);
             // lazy rescale: move the reference max only when it grew by more than the threshold
-            const float m_cand = fmaxf(m_run, tmax * a.scale_log2);
+            const float m_cand = fmaxf(m_run, tmax * to_log2);
             const bool grow = (m_cand > m_run + kRescaleThreshold) || (m_run == -INFINITY && m_cand != -INFINITY);
             const float m_new = grow ? m_cand : m_run;
             const bool fresh = (m_run == -INFINITY);   // nothing accumulated for this row yet
@@ -370,8 +381,8 @@ paged_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
             float ps0 = 0.0f, ps1 = 0.0f;
 #pragma unroll
             for (int j = 0; j < HC; j += 2) {
-                const float p0 = ex2_approx(fmaf(__uint_as_float(sr[j]), a.scale_log2, -m_sub));
-                const float p1 = ex2_approx(fmaf(__uint_as_float(sr[j + 1]), a.scale_log2, -m_sub));
+                const float p0 = ex2_approx(fmaf(__uint_as_float(sr[j]), to_log2, -m_sub));
+                const float p1 = ex2_approx(fmaf(__uint_as_float(sr[j + 1]), to_log2, -m_sub));
                 ps0 += p0;
                 ps1 += p1;
                 packed[j >> 1] = pack2<kBf16>(p0, p1);
@@ -525,9 +536,9 @@ static bool prefill64_enabled() {
     return tile == 64;
 }
 
-template <int D, bool kBf16, bool kPacked, bool kSigmoid>
+template <int D, bool kBf16, bool kPacked, int kWeights>
 static int launch_prefill_as(const CUtensorMap& tq, const CUtensorMap& tkv, const PrefillArgs& a, int n_items, cudaStream_t s) {
-    auto kern = paged_attn_prefill_kernel<D, kBf16, kPacked, kSigmoid>;
+    auto kern = paged_attn_prefill_kernel<D, kBf16, kPacked, kWeights>;
     static bool configured[64] = {false};
     int dev = 0;
     cudaGetDevice(&dev);
@@ -543,8 +554,9 @@ static int launch_prefill_as(const CUtensorMap& tq, const CUtensorMap& tkv, cons
 
 template <int D, bool kBf16, bool kPacked = false>
 static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tkv, const PrefillArgs& a, int n_items, cudaStream_t s) {
-    return a.sigmoid_bias != nullptr ? launch_prefill_as<D, kBf16, kPacked, true>(tq, tkv, a, n_items, s)
-                                     : launch_prefill_as<D, kBf16, kPacked, false>(tq, tkv, a, n_items, s);
+    return a.sigmoid_bias != nullptr ? launch_prefill_as<D, kBf16, kPacked, PF_SIGMOID>(tq, tkv, a, n_items, s)
+           : a.cap_log2 > 0.0f       ? launch_prefill_as<D, kBf16, kPacked, PF_CAPPED>(tq, tkv, a, n_items, s)
+                                     : launch_prefill_as<D, kBf16, kPacked, PF_SOFTMAX>(tq, tkv, a, n_items, s);
 }
 
 }  // namespace hds
@@ -585,6 +597,9 @@ static int attention_tc_impl(bool packed, const void* q, void* out, const void* 
     a.sigmoid_bias = opt.sigmoid_bias;
     a.gate = opt.gate;
     a.gate_ld = opt.gate_ld;
+    HDS_REQUIRE(opt.softcap == 0.0f || (alibi == nullptr && opt.sigmoid_bias == nullptr), "paged_attention_prefill: bounded scores without other terms");
+    a.cap_log2 = opt.softcap * 1.4426950408889634f;
+    a.cap_k = opt.softcap > 0.0f ? 2.0f * 1.4426950408889634f * scale / opt.softcap : 0.0f;
     a.window = window;
     a.keep_first = window > 0 ? keep_first : 0;
     a.out_ld = out_ld > 0 ? out_ld : static_cast<int64_t>(n_q_heads) * head_dim;
@@ -632,7 +647,7 @@ static int attention_tc_impl(bool packed, const void* q, void* out, const void* 
         return dtype == 0 ? launch_prefill<128, true, true>(tq, tkv, a, n_items, s)
                           : launch_prefill<128, false, true>(tq, tkv, a, n_items, s);
     if (head_dim == 128 && block_size <= 64 && alibi == nullptr && window == 0 && out_ld == 0 && opt.sink == nullptr && opt.sigmoid_bias == nullptr &&
-        opt.gate == nullptr && prefill64_enabled())   // none of the options there
+        opt.gate == nullptr && opt.softcap == 0.0f && prefill64_enabled())   // none of the options there
         return dtype == 0 ? launch_prefill64<true>(tq, tkv, a, n_items, s) : launch_prefill64<false>(tq, tkv, a, n_items, s);
     if (head_dim == 128)
         return dtype == 0 ? launch_prefill<128, true>(tq, tkv, a, n_items, s)

@@ -47,6 +47,7 @@ struct AttnArgs {
     const float* sigmoid_bias;  // [n_q_heads] or nullptr: keys weigh sigmoid(score + bias), no denominator
     const void* gate;   // nullptr, or rows (gate_ld apart) like out's whose sigmoid multiplies it
     int64_t gate_ld;
+    float cap_log2, cap_k;      // cap_log2 > 0: bounded scores (softcap_log2; scores come scaled, in log2 units)
 };
 
 // a finished output value, behind the denominator (sink included) and the gate; m in log2 units
@@ -246,6 +247,7 @@ paged_attn_splitkv_kernel(const __grid_constant__ CUtensorMap tmap_kv, const Att
 #pragma unroll
                 for (int r = 0; r < R; ++r) {
                     float sc = part[r] + __shfl_xor_sync(0xffffffffu, part[r], 16);
+                    if (a.cap_log2 > 0.0f) sc = softcap_log2(sc, a.cap_k, a.cap_log2);
                     const int q_pos = item.pos0 + r / G;
                     const bool ok = (j < n_mine) && (tok0 + rt <= q_pos) && (r < rows) &&
                                     (a.window <= 0 || tok0 + rt > q_pos - a.window || tok0 + rt < a.keep_first);
@@ -433,10 +435,10 @@ static thread_local const float* g_next_alibi = nullptr;
 static thread_local int g_next_window = 0;
 static thread_local int g_next_keep_first = 0;
 static thread_local int64_t g_next_out_stride = 0;
-static thread_local hds::AttnOptions g_next_options = {nullptr, nullptr, nullptr, 0};
+static thread_local hds::AttnOptions g_next_options = {nullptr, nullptr, nullptr, 0, 0.0f};
 hds::AttnOptions hds::attn_take_options() {
     const AttnOptions o = g_next_options;
-    g_next_options = {nullptr, nullptr, nullptr, 0};
+    g_next_options = {nullptr, nullptr, nullptr, 0, 0.0f};
     return o;
 }
 const float* hds::attn_take_alibi() {
@@ -490,6 +492,12 @@ extern "C" int hds_attention_next_gate(const void* gate, int64_t ld) {
                 "hds_attention_next_gate: 16-byte rows");
     g_next_options.gate = gate;
     g_next_options.gate_ld = ld;
+    return HDS_OK;
+}
+
+extern "C" int hds_attention_next_softcap(float cap) {
+    HDS_REQUIRE(cap >= 0.0f, "hds_attention_next_softcap: cap >= 0 (0 = none)");
+    g_next_options.softcap = cap;
     return HDS_OK;
 }
 
@@ -557,6 +565,9 @@ extern "C" int hds_paged_attention_splitkv(const void* q, void* out, const void*
     a.sigmoid_bias = opt.sigmoid_bias;
     a.gate = opt.gate;
     a.gate_ld = opt.gate_ld;
+    HDS_REQUIRE(opt.softcap == 0.0f || (alibi == nullptr && opt.sigmoid_bias == nullptr), "paged_attention_splitkv: bounded scores without other terms");
+    a.cap_log2 = opt.softcap * 1.4426950408889634f;
+    a.cap_k = opt.softcap > 0.0f ? 2.0f / opt.softcap : 0.0f;
     const int64_t units = static_cast<int64_t>(n_items) * n_kv_heads;
     char* ws = reinterpret_cast<char*>(workspace);
     a.counters = reinterpret_cast<int32_t*>(ws);

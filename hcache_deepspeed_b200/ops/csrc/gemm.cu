@@ -436,10 +436,10 @@ extern "C" int hds_moe_gemm(const void* A, int64_t lda, const void* W_stacked, i
 static int gemm_rope_common(bool has_q, const void* A, int64_t lda, const void* W, int64_t ldw, int M, int K,
                             int dtype, const void* bias, void* q_out, void* kv_cache_layer, const int32_t* tok_pos,
                             const int32_t* tok_slot, const float* inv_freq, int n_q_heads, int n_kv_heads,
-                            int head_dim, int block_size, int do_rope, void* stream) {
+                            int head_dim, int block_size, int do_rope, void* stream, const float* rot_amp = nullptr) {
     HDS_REQUIRE(dtype == 0 || dtype == 1, "gemm_rope: dtype must be 0 (bf16) or 1 (fp16)");
     HDS_REQUIRE(head_dim == 64 || head_dim == 128, "gemm_rope: fused epilogue supports head_dim 64 / 128");
-    HDS_REQUIRE(n_kv_heads > 0 && block_size > 0, "gemm_rope: bad head/block geometry");
+    HDS_REQUIRE((n_kv_heads > 0 || (has_q && n_kv_heads == 0)) && block_size > 0, "gemm_rope: bad head/block geometry");
     HDS_REQUIRE(!do_rope || inv_freq != nullptr, "gemm_rope: inv_freq required when do_rope");
     GemmArgs g;
     memset(&g, 0, sizeof(g));
@@ -470,6 +470,7 @@ static int gemm_rope_common(bool has_q, const void* A, int64_t lda, const void* 
     g.tok_pos = tok_pos;
     g.tok_slot = tok_slot;
     g.inv_freq = inv_freq;
+    g.rot_amp = rot_amp;
     g.n_q_heads = has_q ? n_q_heads : 0;
     g.n_kv_heads = n_kv_heads;
     g.block_size = block_size;
@@ -528,9 +529,9 @@ extern "C" int hds_restore_kv_proj_peers(const void* const* latent_ptrs, int n_p
 
 extern "C" int hds_qkv_rope_proj(const void* x, int64_t ldx, const void* w_qkv, int64_t ldw, int T, int H, int dtype,
                                  const void* bias_qkv, void* q_out, void* kv_cache_layer, const int32_t* tok_pos,
-                                 const int32_t* tok_slot, const float* inv_freq, int n_q_heads, int n_kv_heads,
+                                 const int32_t* tok_slot, const float* inv_freq, const float* rot_amp, int n_q_heads, int n_kv_heads,
                                  int head_dim, int block_size, int do_rope, void* stream) {
     HDS_REQUIRE(q_out != nullptr && n_q_heads > 0, "hds_qkv_rope_proj: q_out and n_q_heads required");
     return gemm_rope_common(true, x, ldx, w_qkv, ldw, T, H, dtype, bias_qkv, q_out, kv_cache_layer, tok_pos,
-                            tok_slot, inv_freq, n_q_heads, n_kv_heads, head_dim, block_size, do_rope, stream);
+                            tok_slot, inv_freq, n_q_heads, n_kv_heads, head_dim, block_size, do_rope, stream, rot_amp);
 }

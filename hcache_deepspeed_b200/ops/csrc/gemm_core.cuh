@@ -87,6 +87,7 @@ struct GemmArgs {
     const int32_t* tok_pos;   // [M] absolute position of each token in its sequence
     const int32_t* tok_slot;  // [M] block_id * block_size + in-block offset; < 0 = skip token
     const float* inv_freq;    // [rotary_dim / 2]
+    const float* rot_amp;     // [rotary_dim / 2] factors of sines and cosines, or nullptr
     int n_q_heads, n_kv_heads, block_size, do_rope;
     // grouped (mixture-of-experts) mode: A rows [group_pad_off[e], group_pad_off[e+1]) belong to expert e (ranges are
     // multiples of 128 so no tile straddles two experts); W stacks the experts' [N, K] matrices along its rows.
@@ -378,6 +379,10 @@ __device__ __forceinline__ void epilogue_kv_rope(const GemmArgs& a, uint32_t tad
                     for (int j = 0; j < 32; ++j) {
                         float sn, co;
                         rope_sincos(static_cast<float>(pos) * a.inv_freq[c + j], &sn, &co);
+                        if (a.rot_amp != nullptr) {
+                            sn *= a.rot_amp[c + j];
+                            co *= a.rot_amp[c + j];
+                        }
                         const float x = lo[j], y = hi[j];
                         lo[j] = x * co - y * sn;
                         hi[j] = y * co + x * sn;

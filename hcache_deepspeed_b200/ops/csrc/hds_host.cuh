@@ -219,11 +219,12 @@ const float* attn_take_alibi();
 int attn_take_window();   // same for hds_attention_next_window (0 = no sliding window)
 int attn_take_keep_first();       // hds_attention_next_keep_first (0 = none)
 int64_t attn_take_out_stride();   // hds_attention_next_out_stride (0 = dense rows)
-struct AttnOptions {              // hds_attention_next_sink / _sigmoid / _gate
+struct AttnOptions {              // hds_attention_next_sink / _sigmoid / _gate / _softcap
     const float* sink;
     const float* sigmoid_bias;
     const void* gate;
     int64_t gate_ld;
+    float softcap;
 };
 AttnOptions attn_take_options();
 

@@ -550,6 +550,15 @@ __device__ __forceinline__ void rope_sincos(float x, float* s, float* c) {
     __sincosf(r, s, c);
 }
 
+// Bounded scores, cap * tanh(score / cap), by tanh(x) = 1 - 2 / (1 + e^(2x)): absolute error about 2^-23 cap. `k` and `c` turn a raw
+// score into the exponent and the result into log2 units: k = 2 log2(e) scale / cap, c = cap log2(e).
+__device__ __forceinline__ float softcap_log2(float raw, float k, float c) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * k));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+    return fmaf(-2.0f * c, r, c);
+}
+
 // Activations are applied inside unrolled epilogue loops (16-64 copies per kernel), so the body must stay small: the
 // erf form of GELU is an out-of-line call, everything else is a handful of instructions on the fast-math intrinsics
 // (an inlined switch over erff / tanhf made the epilogues instruction-fetch bound: a 4160 x 22016 store epilogue took

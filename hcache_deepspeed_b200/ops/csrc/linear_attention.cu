@@ -1,10 +1,12 @@
 // Gated linear attention over a ragged batch, per head:  S <- S diag(alpha) + v k^T,  o = S q dim^-1/2, with a decay per key channel,
 // alpha = s(z + bias)^(1 / tau) (s the logistic function), then o / rms(o) * weight * silu(gate). The state is kept as [vdim][dim].
+// Retention (kRet) has one constant decay per head and turns q and k by position on the way in.
 //
 //   lin_step : sequences with one new token (decode), norm and gate included
 //   lin_scan : sequences with several, token by token in fp32 (fp32 models, and shapes the chunked form does not take)
 //   the chunked form (linear_chunk.cu): prompts of bf16 models on the tensor cores
 #include "linear_attention.cuh"
+#include <math.h>
 #include "../../../include/hds_b200.h"
 
 namespace hds {
@@ -12,7 +14,7 @@ namespace hds {
 constexpr int kLsThreads = 256, kLsWarps = kLsThreads / 32;
 
 // CTA = (sequence, head). NV > 0: state rows of up to 128 * NV values (a multiple of 4) as float4, R rows in flight per warp; 0: any.
-template <int DT, int NV>
+template <int DT, int NV, bool kRet>
 __global__ void __launch_bounds__(kLsThreads) lin_step_kernel(const LinArgs a) {
     extern __shared__ float sm[];
     __shared__ float red[kLsWarps];
@@ -41,11 +43,28 @@ __global__ void __launch_bounds__(kLsThreads) lin_step_kernel(const LinArgs a) {
             }
     };
     if constexpr (NV > 0) load_rows(warp * R);
-    const float scale = rsqrtf(static_cast<float>(N));
-    for (int n = threadIdx.x; n < N; n += kLsThreads) {
-        q_s[n] = load_any<DT>(a.q, row * a.ld + h * N + n) * scale;
-        k_s[n] = load_any<DT>(a.k, row * a.ld + h * N + n);
-        d_s[n] = exp2f(lin_log2_decay<DT>(load_any<DT>(a.z, row * a.ld_z + h * N + n) + a.bias[h * N + n], a.inv_tau));
+    const float keep = kRet ? exp2f(a.log2_decay[h]) : 0.0f;
+    if constexpr (kRet) {
+        const float pos = static_cast<float>(sp.seen);
+        for (int c = threadIdx.x; c < N >> 1; c += kLsThreads) {
+            float s, co;
+            lin_sincos<DT>(pos * a.freq[c], &s, &co);
+            if (a.amp != nullptr) {
+                s *= a.amp[c];
+                co *= a.amp[c];
+            }
+            const float2 q = lin_turned<DT>(a, a.q, row * a.ld + h * N, c, s, co), k = lin_turned<DT>(a, a.k, row * a.ld + h * N, c, s, co);
+            q_s[c] = q.x * a.q_scale;
+            q_s[c + (N >> 1)] = q.y * a.q_scale;
+            k_s[c] = k.x * a.k_scale;
+            k_s[c + (N >> 1)] = k.y * a.k_scale;
+        }
+    } else {
+        for (int n = threadIdx.x; n < N; n += kLsThreads) {
+            q_s[n] = load_any<DT>(a.q, row * a.ld + h * N + n) * a.q_scale;
+            k_s[n] = load_any<DT>(a.k, row * a.ld + h * N + n) * a.k_scale;
+            d_s[n] = exp2f(lin_log2_decay<DT>(load_any<DT>(a.z, row * a.ld_z + h * N + n) + a.bias[h * N + n], a.inv_tau));
+        }
     }
     for (int p = threadIdx.x; p < P; p += kLsThreads) o_s[p] = load_any<DT>(a.v, row * a.ld + h * P + p);
     __syncthreads();
@@ -61,7 +80,7 @@ __global__ void __launch_bounds__(kLsThreads) lin_step_kernel(const LinArgs a) {
                 const int n = (lane + 32 * j) * 4;
                 if (n >= N) continue;
                 const float4 q = *reinterpret_cast<const float4*>(q_s + n), k = *reinterpret_cast<const float4*>(k_s + n),
-                             d = *reinterpret_cast<const float4*>(d_s + n);
+                             d = kRet ? make_float4(keep, keep, keep, keep) : *reinterpret_cast<const float4*>(d_s + n);
 #pragma unroll
                 for (int r = 0; r < R; ++r) {
                     float4 x = S[r][j];
@@ -88,7 +107,7 @@ __global__ void __launch_bounds__(kLsThreads) lin_step_kernel(const LinArgs a) {
             const float v = o_s[p];
             float* r = st + static_cast<int64_t>(p) * N;
             for (int n = lane; n < N; n += 32) {
-                const float x = fmaf(v, k_s[n], carry ? d_s[n] * r[n] : 0.0f);
+                const float x = fmaf(v, k_s[n], carry ? (kRet ? keep : d_s[n]) * r[n] : 0.0f);
                 r[n] = x;
                 sq = fmaf(x, q_s[n], sq);
             }
@@ -112,7 +131,7 @@ __global__ void __launch_bounds__(kLsThreads) lin_step_kernel(const LinArgs a) {
     ss = 0.0f;
 #pragma unroll
     for (int w = 0; w < kLsWarps; ++w) ss += red[w];
-    const float r = 1.0f / sqrtf(ss / P + a.eps);
+    const float r = 1.0f / sqrtf(ss / a.norm_cols + a.eps);
     for (int p = threadIdx.x; p < P; p += kLsThreads) {
         const float g = load_any<DT>(a.gate, row * a.ld + h * P + p);
         ssm_store<DT>(a.out, row * a.ld_out + h * P + p, o_s[p] * r * a.norm_w[h * P + p] * ssm_silu<DT>(g));
@@ -122,7 +141,7 @@ __global__ void __launch_bounds__(kLsThreads) lin_step_kernel(const LinArgs a) {
 // CTA = (sequence, head, 16 rows): a warp keeps 4 rows, NL state values of each per lane.
 constexpr int kLcWarps = 4, kLcRows = 4, kLcP = kLcWarps * kLcRows, kLcTok = 16;
 
-template <int DT, int NL>
+template <int DT, int NL, bool kRet>
 __global__ void __launch_bounds__(kLcWarps * 32) lin_scan_kernel(const LinArgs a) {
     extern __shared__ float sm[];
     pdl_enter();
@@ -134,7 +153,7 @@ __global__ void __launch_bounds__(kLcWarps * 32) lin_scan_kernel(const LinArgs a
     float* d_s = q_s + kLcTok * N;
     float* v_s = d_s + kLcTok * N;          // [tok][kLcP]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const float scale = rsqrtf(static_cast<float>(N));
+    const float keep = kRet ? exp2f(a.log2_decay[h]) : 0.0f;
     float S[kLcRows][NL];
     float* st = a.state + (static_cast<int64_t>(sp.slot) * a.heads + h) * P * N;
 #pragma unroll
@@ -148,11 +167,29 @@ __global__ void __launch_bounds__(kLcWarps * 32) lin_scan_kernel(const LinArgs a
         const int nt = min(kLcTok, sp.n - t0);
         const int64_t row = sp.row0 + t0;
         __syncthreads();
-        for (int e = threadIdx.x; e < nt * N; e += blockDim.x) {
+        if constexpr (kRet) {
+            const int half = N >> 1;
+            for (int e = threadIdx.x; e < nt * half; e += blockDim.x) {
+                const int t = e / half, c = e - t * half;
+                const int64_t at = (row + t) * a.ld + h * N;
+                float s, co;
+                lin_sincos<DT>(static_cast<float>(sp.seen + t0 + t) * a.freq[c], &s, &co);
+                if (a.amp != nullptr) {
+                    s *= a.amp[c];
+                    co *= a.amp[c];
+                }
+                const float2 q = lin_turned<DT>(a, a.q, at, c, s, co), k = lin_turned<DT>(a, a.k, at, c, s, co);
+                q_s[t * N + c] = q.x * a.q_scale;
+                q_s[t * N + half + c] = q.y * a.q_scale;
+                k_s[t * N + c] = k.x * a.k_scale;
+                k_s[t * N + half + c] = k.y * a.k_scale;
+            }
+        }
+        for (int e = threadIdx.x; !kRet && e < nt * N; e += blockDim.x) {
             const int t = e / N, n = e - t * N;
             const int64_t at = (row + t) * a.ld + h * N + n;
-            k_s[e] = load_any<DT>(a.k, at);
-            q_s[e] = load_any<DT>(a.q, at) * scale;
+            k_s[e] = load_any<DT>(a.k, at) * a.k_scale;
+            q_s[e] = load_any<DT>(a.q, at) * a.q_scale;
             d_s[e] = exp2f(lin_log2_decay<DT>(load_any<DT>(a.z, (row + t) * a.ld_z + h * N + n) + a.bias[h * N + n], a.inv_tau));
         }
         for (int e = threadIdx.x; e < nt * kLcP; e += blockDim.x) {
@@ -165,7 +202,7 @@ __global__ void __launch_bounds__(kLcWarps * 32) lin_scan_kernel(const LinArgs a
 #pragma unroll
             for (int j = 0; j < NL; ++j) {
                 const int n = lane + 32 * j;
-                const float k = n < N ? k_s[t * N + n] : 0.0f, q = n < N ? q_s[t * N + n] : 0.0f, d = n < N ? d_s[t * N + n] : 0.0f;
+                const float k = n < N ? k_s[t * N + n] : 0.0f, q = n < N ? q_s[t * N + n] : 0.0f, d = kRet ? keep : n < N ? d_s[t * N + n] : 0.0f;
 #pragma unroll
                 for (int r = 0; r < kLcRows; ++r) {
                     S[r][j] = fmaf(v_s[t * kLcP + warp * kLcRows + r], k, d * S[r][j]);
@@ -189,11 +226,11 @@ __global__ void __launch_bounds__(kLcWarps * 32) lin_scan_kernel(const LinArgs a
         }
 }
 
-template <int DT>
+template <int DT, bool kRet>
 static int launch_step(const LinArgs& a, cudaStream_t s) {
     const dim3 grid(a.n_seqs, a.heads), block(kLsThreads);
     const size_t smem = (3 * static_cast<size_t>(a.N) + a.P) * 4;
-#define HDS_LS(NV) HDS_CHECK_CUDA(launch_kernel(lin_step_kernel<DT, NV>, grid, block, smem, s, a))
+#define HDS_LS(NV) HDS_CHECK_CUDA(launch_kernel(lin_step_kernel<DT, NV, kRet>, grid, block, smem, s, a))
     if (a.N % 4 != 0 || a.N > 512) HDS_LS(0);
     else if (a.N <= 128) HDS_LS(1);
     else if (a.N <= 256) HDS_LS(2);
@@ -202,14 +239,14 @@ static int launch_step(const LinArgs& a, cudaStream_t s) {
     return HDS_OK;
 }
 
-template <int DT>
+template <int DT, bool kRet>
 static int launch_scan(const LinArgs& a, cudaStream_t s) {
     const dim3 grid(a.n_seqs, a.heads, (a.P + kLcP - 1) / kLcP), block(kLcWarps * 32);
     const size_t smem = static_cast<size_t>(kLcTok) * (3 * a.N + kLcP) * 4;
-#define HDS_LC(NL)                                                                                                                          \
-    do {                                                                                                                                    \
-        HDS_CHECK_CUDA(cudaFuncSetAttribute(lin_scan_kernel<DT, NL>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
-        HDS_CHECK_CUDA(launch_kernel(lin_scan_kernel<DT, NL>, grid, block, smem, s, a));                                                    \
+#define HDS_LC(NL)                                                                                                                                \
+    do {                                                                                                                                          \
+        HDS_CHECK_CUDA(cudaFuncSetAttribute(lin_scan_kernel<DT, NL, kRet>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
+        HDS_CHECK_CUDA(launch_kernel(lin_scan_kernel<DT, NL, kRet>, grid, block, smem, s, a));                                                    \
     } while (0)
     if (a.N <= 32) HDS_LC(1);
     else if (a.N <= 64) HDS_LC(2);
@@ -219,6 +256,18 @@ static int launch_scan(const LinArgs& a, cudaStream_t s) {
     else HDS_LC(32);
 #undef HDS_LC
     return HDS_OK;
+}
+
+template <bool kRet>
+static int launch_tokens(bool step, const LinArgs& a, int dtype, cudaStream_t s) {
+    if (step) return dtype == 0 ? launch_step<0, kRet>(a, s) : dtype == 1 ? launch_step<1, kRet>(a, s) : launch_step<2, kRet>(a, s);
+    return dtype == 0 ? launch_scan<0, kRet>(a, s) : dtype == 1 ? launch_scan<1, kRet>(a, s) : launch_scan<2, kRet>(a, s);
+}
+int lin_launch_step(const LinArgs& a, int dtype, bool retention, cudaStream_t s) {
+    return retention ? launch_tokens<true>(true, a, dtype, s) : launch_tokens<false>(true, a, dtype, s);
+}
+int lin_launch_scan(const LinArgs& a, int dtype, bool retention, cudaStream_t s) {
+    return retention ? launch_tokens<true>(false, a, dtype, s) : launch_tokens<false>(false, a, dtype, s);
 }
 
 }  // namespace hds
@@ -240,7 +289,7 @@ extern "C" int hds_linear_attention(const void* q, const void* k, const void* v,
     *finished = 1;
     if (T == 0 || n_seqs == 0) return HDS_OK;
     LinArgs a{q, k, v, gate, ld, z, ld_z, bias, inv_tau, state, reinterpret_cast<const SsmSpan*>(spans), n_seqs, T, heads, vdim, dim,
-              y, ld_y, out, ld_out, norm_w, eps, 0};
+              y, ld_y, out, ld_out, norm_w, eps, 0, vdim, 1.0f / sqrtf(static_cast<float>(dim)), 1.0f, nullptr, nullptr, nullptr};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     const int n_multi = n_seqs - n_single;
     int rc = HDS_OK;
@@ -256,9 +305,9 @@ extern "C" int hds_linear_attention(const void* q, const void* k, const void* v,
         } else {
             *finished = 0;
             a.write_y = 1;      // by every row of the batch: one norm finishes them all
-            rc = dtype == 0 ? launch_scan<0>(a, s) : dtype == 1 ? launch_scan<1>(a, s) : launch_scan<2>(a, s);
+            rc = lin_launch_scan(a, dtype, false, s);
         }
     }
     if (rc != HDS_OK || n_single == 0) return rc;
-    return dtype == 0 ? launch_step<0>(a, s) : dtype == 1 ? launch_step<1>(a, s) : launch_step<2>(a, s);
+    return lin_launch_step(a, dtype, false, s);
 }

@@ -1,4 +1,4 @@
-// Shared pieces of the gated linear attention kernels (linear_attention.cu, linear_chunk.cu).
+// Shared pieces of the linear attention kernels (linear_attention.cu, linear_chunk.cu, retention.cu).
 #pragma once
 #include "recurrent.cuh"
 
@@ -24,7 +24,26 @@ struct LinArgs {
     const float* norm_w;    // [heads * P]
     float eps;
     int write_y;            // steps leave read-outs in y instead of finished rows in out
+    int norm_cols;          // values of a head that its norm averages over
+    float q_scale, k_scale;
+    // retention: a constant decay per head instead of z; q and k turned by position
+    const float* log2_decay;    // [heads]
+    const float* freq;          // [N / 2]
+    const float* amp;           // [N / 2] or nullptr
 };
+
+template <int DT>
+__device__ __forceinline__ void lin_sincos(float x, float* s, float* c) {
+    if constexpr (DT == 2) sincosf(x, s, c);
+    else rope_sincos(x, s, c);
+}
+
+// values c and N / 2 + c of a head's row, turned for position pos
+template <int DT>
+__device__ __forceinline__ float2 lin_turned(const LinArgs& a, const void* x, int64_t head_row, int c, float s, float co) {
+    const float u = load_any<DT>(x, head_row + c), v = load_any<DT>(x, head_row + (a.N >> 1) + c);
+    return make_float2(u * co - v * s, v * co + u * s);
+}
 
 // log2 of sigmoid(x)^(1 / tau); below 2^-200 a decay is zero to everything behind it
 template <int DT>
@@ -35,6 +54,10 @@ __device__ __forceinline__ float lin_log2_decay(float x, float inv_tau) {
     else l = fminf(x, 0.0f) * kLog2e - __log2f(1.0f + __expf(-fabsf(x)));
     return fmaxf(l * inv_tau, -200.0f);
 }
+
+// token by token (linear_attention.cu): sequences with one new token; with several, which leave their read-outs in y
+int lin_launch_step(const LinArgs& a, int dtype, bool retention, cudaStream_t s);
+int lin_launch_scan(const LinArgs& a, int dtype, bool retention, cudaStream_t s);
 
 bool lin_chunk_supported(const LinArgs& a, int dtype, const void* ws, int64_t ws_bytes);
 int lin_chunk_launch(const LinArgs& a, int n_multi, void* ws, int64_t ws_bytes, cudaStream_t s);

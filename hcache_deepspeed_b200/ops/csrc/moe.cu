@@ -2,7 +2,8 @@
 //
 //   top-k gating  : softmax over the expert logits of each token, k rounds of arg-max (ties -> lower index), optionally of the
 //                   scores plus a per-expert bias; optional renormalisation of the k scores, a factor on them, one atomic per
-//                   (token, choice) to claim a row inside the expert. Sigmoid scores (each expert by itself) likewise
+//                   (token, choice) to claim a row inside the expert. Sigmoid scores (each expert by itself) likewise; or the
+//                   bias joins the logits, which choose as they are
 //   offsets       : per-expert row ranges padded to the GEMM's 128-row tile (so no A tile straddles two experts);
 //                   re-zeroes the counters for the next layer
 //   scatter       : copies each token's activation row (optionally times the choice's score) to its k expert rows, records the row
@@ -21,10 +22,12 @@ namespace hds {
 constexpr int kGateThreads = 128;
 constexpr int kMoeMaxK = 64;
 constexpr int kMoeRowPad = 128;
+// softmax scores (+ bias) choose; sigmoids do; softmax scores of logits + bias, chosen by those
+enum MoeScores : int { MOE_SOFTMAX = 0, MOE_SIGMOID = 1, MOE_BIASED = 2 };
 
 template <int DT>
 __global__ void __launch_bounds__(kGateThreads)
-moe_topk_gating_kernel(void* __restrict__ logits, int64_t ld, int E, int k, int normalize, int sigmoid, const float* __restrict__ bias,
+moe_topk_gating_kernel(void* __restrict__ logits, int64_t ld, int E, int k, int normalize, int kind, const float* __restrict__ bias,
                        float scale, int clear, float* __restrict__ scores, int32_t* __restrict__ expert_ids, int32_t* __restrict__ offsets,
                        int32_t* __restrict__ counts) {
     extern __shared__ float probs[];  // [E] scores, [E] what chooses
@@ -35,9 +38,11 @@ moe_topk_gating_kernel(void* __restrict__ logits, int64_t ld, int E, int k, int 
     __shared__ int sel_i[kMoeMaxK];
     pdl_enter();
     const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const bool sigmoid = kind == MOE_SIGMOID, biased = kind == MOE_BIASED;
     float mx = -INFINITY;
     for (int e = tid; e < E; e += kGateThreads) {
-        const float v = load_any<DT>(logits, static_cast<int64_t>(t) * ld + e);
+        float v = load_any<DT>(logits, static_cast<int64_t>(t) * ld + e);
+        if (biased) v += bias[e];
         probs[e] = v;
         mx = fmaxf(mx, v);
         if (DT == 2 && clear) reinterpret_cast<float*>(logits)[static_cast<int64_t>(t) * ld + e] = 0.0f;
@@ -51,7 +56,7 @@ moe_topk_gating_kernel(void* __restrict__ logits, int64_t ld, int E, int k, int 
     __syncthreads();
     float sum = 0.0f;
     for (int e = tid; e < E; e += kGateThreads) {
-        if (sigmoid) choice[e] = probs[e];      // (logits choose as sigmoids do, and still where those have all become 1)
+        if (sigmoid || biased) choice[e] = probs[e];    // (logits choose as scores do, and still where those are all 1 or 0)
         const float p = sigmoid ? 1.0f / (1.0f + expf(-probs[e])) : expf(probs[e] - mx);
         probs[e] = p;
         sum += p;
@@ -64,7 +69,8 @@ moe_topk_gating_kernel(void* __restrict__ logits, int64_t ld, int E, int k, int 
     for (int w = 0; w < kGateThreads / 32; ++w) sum += red_v[w];
     const float inv = sigmoid ? 1.0f : 1.0f / sum;
     for (int e = tid; e < E; e += kGateThreads)
-        if (bias != nullptr) choice[e] = fmaf(probs[e], inv, bias[e]);
+        if (biased) continue;
+        else if (bias != nullptr) choice[e] = fmaf(probs[e], inv, bias[e]);
         else if (!sigmoid) choice[e] = probs[e];
     __syncthreads();
     for (int j = 0; j < k; ++j) {
@@ -250,12 +256,13 @@ __global__ void moe_gather_kernel(const void* __restrict__ y, int64_t ldy, const
 
 using namespace hds;
 
-extern "C" int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E, int k, int normalize, int sigmoid, const float* bias,
+extern "C" int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E, int k, int normalize, int kind, const float* bias,
                                    float scale, int clear, int logits_dtype, float* scores, int32_t* expert_ids, int32_t* offsets,
                                    int32_t* counts, void* stream) {
     HDS_REQUIRE(E >= 1 && E <= 4096, "hds_moe_topk_gating: 1..4096 experts");
     HDS_REQUIRE(k >= 1 && k <= kMoeMaxK && k <= E, "hds_moe_topk_gating: top_k must be in 1..64 and <= experts");
     HDS_REQUIRE(logits_dtype >= 0 && logits_dtype <= 2, "hds_moe_topk_gating: logits dtype 0 bf16 / 1 fp16 / 2 fp32");
+    HDS_REQUIRE(kind >= 0 && kind <= 2 && (kind != 2 || bias != nullptr), "hds_moe_topk_gating: kind 0 / 1 / 2, the last with a bias");
     HDS_REQUIRE(!clear || logits_dtype == 2, "hds_moe_topk_gating: only fp32 logits are cleared");
     if (T == 0) return HDS_OK;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -263,13 +270,13 @@ extern "C" int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E
     cudaError_t rc;
     if (logits_dtype == 0)
         rc = launch_kernel(moe_topk_gating_kernel<0>, dim3(T), dim3(kGateThreads), smem, s, logits, ld_logits, E, k,
-                           normalize, sigmoid, bias, scale, clear, scores, expert_ids, offsets, counts);
+                           normalize, kind, bias, scale, clear, scores, expert_ids, offsets, counts);
     else if (logits_dtype == 1)
         rc = launch_kernel(moe_topk_gating_kernel<1>, dim3(T), dim3(kGateThreads), smem, s, logits, ld_logits, E, k,
-                           normalize, sigmoid, bias, scale, clear, scores, expert_ids, offsets, counts);
+                           normalize, kind, bias, scale, clear, scores, expert_ids, offsets, counts);
     else
         rc = launch_kernel(moe_topk_gating_kernel<2>, dim3(T), dim3(kGateThreads), smem, s, logits, ld_logits, E, k,
-                           normalize, sigmoid, bias, scale, clear, scores, expert_ids, offsets, counts);
+                           normalize, kind, bias, scale, clear, scores, expert_ids, offsets, counts);
     HDS_CHECK_CUDA(rc);
     return HDS_OK;
 }

@@ -217,14 +217,16 @@ def restore_kv_proj_peers(peer_ptrs: Sequence[int], rows_per_peer: int, T: int, 
 
 def qkv_rope_proj(x: torch.Tensor, w_qkv: torch.Tensor, q_out: torch.Tensor, kv_cache_layer: torch.Tensor,
                   tok_pos: torch.Tensor, tok_slot: torch.Tensor, inv_freq: Optional[torch.Tensor], n_q_heads: int,
-                  n_kv_heads: int, head_dim: int, block_size: int, bias_qkv: Optional[torch.Tensor] = None) -> None:
-    """Forward QKV projection with RoPE + KV-append fused into the GEMM epilogue."""
+                  n_kv_heads: int, head_dim: int, block_size: int, bias_qkv: Optional[torch.Tensor] = None,
+                  amp: Optional[torch.Tensor] = None) -> None:
+    """Forward QKV projection with RoPE + KV-append fused into the GEMM epilogue. ``n_kv_heads`` = 0: queries alone, no pages.
+    ``amp`` (like ``inv_freq``): factors of the rotated pairs."""
     _check_2d(x, "x")
     T, H = x.shape
     lib = native.cuda_lib()
     wp, ldw = _w(w_qkv)
     rc = lib.hds_qkv_rope_proj(_p(x), x.stride(0), wp, ldw, T, H, _dt(x), _p(bias_qkv), _p(q_out),
-                               _p(kv_cache_layer), _p(tok_pos), _p(tok_slot), _p(inv_freq), n_q_heads, n_kv_heads,
+                               _p(kv_cache_layer), _p(tok_pos), _p(tok_slot), _p(inv_freq), _p(amp), n_q_heads, n_kv_heads,
                                head_dim, block_size, 0 if inv_freq is None else 1, _stream())
     native.check(rc, "hds_qkv_rope_proj")
     _count()
@@ -402,10 +404,12 @@ def splitkv_workspace_bytes(n_items: int, n_q_heads: int, n_kv_heads: int, head_
 
 def _arm_alibi(lib, alibi: Optional[torch.Tensor], n_q_heads: int, window: int = 0, keep_first: int = 0,
                out: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, sigmoid_bias: Optional[torch.Tensor] = None,
-               gate: Optional[torch.Tensor] = None) -> None:
+               gate: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
     """Options of the next attention launch of this thread, consumed by that launch: ALiBi slopes, sliding window and kept
     first tokens, the stride of ``out`` when its rows (``[T, n_q_heads * head_dim]``) are not dense, softmax sinks, the biases of
-    sigmoid weights, the output gate."""
+    sigmoid weights, the output gate, the bound of the scores."""
+    if softcap:
+        native.check(lib.hds_attention_next_softcap(float(softcap)), "hds_attention_next_softcap")
     for t, fn in ((sink, "hds_attention_next_sink"), (sigmoid_bias, "hds_attention_next_sigmoid")):
         if t is not None:
             assert t.dtype == torch.float32 and t.is_cuda and t.is_contiguous() and t.numel() == n_q_heads
@@ -430,13 +434,13 @@ def paged_attention_splitkv(q: torch.Tensor, out: torch.Tensor, kv_cache_layer: 
                             n_q_heads: int, n_kv_heads: int, head_dim: int, block_size: int, n_splits: int,
                             scale: float, workspace: Optional[torch.Tensor], alibi: Optional[torch.Tensor] = None,
                             window: int = 0, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
-                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
     """kv_cache_layer: [blocks, 2, kvh, bs, d]; items: int32 [n, 4] = (seq, q_row0, n_q, pos0). ``alibi``: fp32 [n_q_heads]
     slopes; score += slope * (key position - query position). ``window``: sliding-window attention, keys (p - window, p] and
     the first ``keep_first`` ones. ``sink``, ``sigmoid_bias`` (fp32 [n_q_heads]) and ``gate`` (rows like ``out``'s): see
     ``hds_attention_next_sink``."""
     lib = native.cuda_lib()
-    _arm_alibi(lib, alibi, n_q_heads, window, keep_first, out, sink, sigmoid_bias, gate)
+    _arm_alibi(lib, alibi, n_q_heads, window, keep_first, out, sink, sigmoid_bias, gate, softcap)
     rc = lib.hds_paged_attention_splitkv(_p(q), _p(out), _p(kv_cache_layer), kv_cache_layer.shape[0], _p(block_tables),
                                          block_tables.stride(0), _p(items), n_items, rows_per_item, n_q_heads,
                                          n_kv_heads, head_dim, block_size, n_splits, scale, _p(workspace),
@@ -455,12 +459,12 @@ def paged_attention_prefill(q: torch.Tensor, out: torch.Tensor, kv_cache_layer: 
                             n_kv_heads: int, head_dim: int, block_size: int, scale: float, n_splits: int = 1,
                             workspace: Optional[torch.Tensor] = None, packed: bool = False,
                             alibi: Optional[torch.Tensor] = None, window: int = 0, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
-                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
     """tcgen05 paged attention. ``packed``: grouped-query decode form — one CTA per (item, KV head) whose MMA rows are
     the group's (token, query head) pairs (``hds_paged_attention_packed``). ``alibi``: fp32 [n_q_heads] slopes;
     ``window``: sliding-window attention."""
     lib = native.cuda_lib()
-    _arm_alibi(lib, alibi, n_q_heads, window, keep_first, out, sink, sigmoid_bias, gate)
+    _arm_alibi(lib, alibi, n_q_heads, window, keep_first, out, sink, sigmoid_bias, gate, softcap)
     fn = lib.hds_paged_attention_packed if packed else lib.hds_paged_attention_prefill
     rc = fn(_p(q), _p(out), _p(kv_cache_layer), kv_cache_layer.shape[0], _p(block_tables),
                                          block_tables.stride(0), _p(items), n_items, q.shape[0], n_q_heads, n_kv_heads,
@@ -481,12 +485,12 @@ def moe_padded_rows(n_tokens: int, n_experts: int, top_k: int) -> int:
 
 def moe_topk_gating(logits: torch.Tensor, top_k: int, normalize: bool, scores: torch.Tensor, expert_ids: torch.Tensor,
                     offsets: torch.Tensor, counts: torch.Tensor, bias: Optional[torch.Tensor] = None, scale: float = 1.0,
-                    clear: bool = False, sigmoid: bool = False) -> None:
+                    clear: bool = False, sigmoid: bool = False, biased: bool = False) -> None:
     """Softmax (or ``sigmoid``) + top-k per token; ``counts`` (int32 [E], zero on entry) is incremented per assignment. ``bias`` (fp32 [E]) is added
-    to the scores that choose, ``scale`` multiplies the scores returned, ``clear`` zeroes (fp32) logits once read."""
+    to the scores that choose (``biased``: to the logits, which choose), ``scale`` multiplies the scores returned, ``clear`` zeroes (fp32) logits once read."""
     T, E = logits.shape
     code = 2 if logits.dtype == torch.float32 else _dt(logits)
-    rc = native.cuda_lib().hds_moe_topk_gating(_p(logits), logits.stride(0), T, E, top_k, int(normalize), int(sigmoid), _p(bias), scale,
+    rc = native.cuda_lib().hds_moe_topk_gating(_p(logits), logits.stride(0), T, E, top_k, int(normalize), 2 if biased else int(sigmoid), _p(bias), scale,
                                                  int(clear), code, _p(scores),
                                                _p(expert_ids), _p(offsets), _p(counts), _stream())
     native.check(rc, "hds_moe_topk_gating")
@@ -722,10 +726,10 @@ def paged_attention_generic(q: torch.Tensor, out: torch.Tensor, kv_cache_layer: 
                             tok_seq: torch.Tensor, tok_pos: torch.Tensor, n_q_heads: int, n_kv_heads: int, head_dim: int,
                             block_size: int, scale: float, window: int = 0, keep_first: int = 0, value_dim: int = 0,
                             spans: Optional[torch.Tensor] = None, limit: int = 0, sink: Optional[torch.Tensor] = None,
-                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
     """fp32-arithmetic attention for any operand type and head size (``hds_paged_attention_generic``). ``value_dim`` > 0: pages of
     one plane, the first ``value_dim`` values of a key row are its value. ``spans``: skip sequences of more than ``limit`` tokens."""
-    _arm_alibi(native.cuda_lib(), None, n_q_heads, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate)
+    _arm_alibi(native.cuda_lib(), None, n_q_heads, sink=sink, sigmoid_bias=sigmoid_bias, gate=gate, softcap=softcap)
     rc = native.cuda_lib().hds_paged_attention_generic(_p(q), _p(out), out.stride(0), _p(kv_cache_layer), _p(block_tables),
                                                        block_tables.stride(0), _p(tok_seq), _p(tok_pos), q.shape[0], n_q_heads,
                                                        n_kv_heads, head_dim, block_size, scale, window, keep_first, value_dim, _p(spans),
@@ -824,17 +828,18 @@ def delta_rule(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, d
 # ------------------------------------------------------------------------------------------------
 # attention inputs, minGRU, gated linear attention
 # ------------------------------------------------------------------------------------------------
-def attention_append(qkv: torch.Tensor, q_out: torch.Tensor, kv_cache_layer: torch.Tensor, tok_pos: torch.Tensor, tok_slot: torch.Tensor,
+def attention_append(qkv: torch.Tensor, q_out: torch.Tensor, kv_cache_layer: Optional[torch.Tensor], tok_pos: torch.Tensor, tok_slot: torch.Tensor,
                      n_q_heads: int, n_kv_heads: int, head_dim: int, block_size: int, freq: Optional[torch.Tensor],
                      q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None, q_cols: int = 0, k_cols: int = 0,
-                     eps: float = 0.0, first: Optional[torch.Tensor] = None, share: Optional[torch.Tensor] = None) -> None:
+                     eps: float = 0.0, first: Optional[torch.Tensor] = None, share: Optional[torch.Tensor] = None,
+                     amp: Optional[torch.Tensor] = None) -> None:
     """Projected rows ``qkv`` = [q heads | k heads | v heads] -> normed and rotated queries, page rows with mixed values
-    (``hds_attention_append``)."""
+    (``hds_attention_append``). ``n_kv_heads`` = 0: queries alone, no pages."""
     _check_2d(qkv, "qkv")
-    assert kv_cache_layer.shape[4] == head_dim and kv_cache_layer.shape[3] == block_size
+    assert n_kv_heads == 0 or (kv_cache_layer.shape[4] == head_dim and kv_cache_layer.shape[3] == block_size)
     assert first is None or (first.shape[:4] == kv_cache_layer.shape[:4] and first.is_contiguous())
     rc = native.cuda_lib().hds_attention_append(_p(qkv), qkv.stride(0), _p(q_out), _p(kv_cache_layer), _p(tok_pos), _p(tok_slot), qkv.shape[0],
-                                                n_q_heads, n_kv_heads, head_dim, block_size, _p(freq), _p(q_norm), _p(k_norm), q_cols, k_cols,
+                                                n_q_heads, n_kv_heads, head_dim, block_size, _p(freq), _p(amp), _p(q_norm), _p(k_norm), q_cols, k_cols,
                                                 eps, _p(first), 0 if first is None else first.shape[4], _p(share), _dt3(qkv), _stream())
     native.check(rc, "hds_attention_append")
     _count()
@@ -889,3 +894,28 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: to
     _count((3 if out is not None else 2) * (spans.shape[0] > n_single) + (n_single > 0))
     if out is not None and not done.value:
         gated_norm(y[:, :heads * vdim], gate[:, :heads * vdim], norm_w, out, heads, eps, gate_after=True)
+
+
+def retention_workspace_bytes(n_tokens: int, n_seqs: int, heads: int, vdim: int, dim: int) -> int:
+    """Scratch of the chunked form for batches of up to ``n_tokens`` tokens in ``n_seqs`` sequences (0: not for this shape)."""
+    return int(native.cuda_lib().hds_retention_workspace_bytes(n_tokens, n_seqs, heads, vdim, dim))
+
+
+def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, log2_decay: torch.Tensor, freq: torch.Tensor,
+              amp: Optional[torch.Tensor], k_scale: float, norm_cols: int, state: torch.Tensor, spans: torch.Tensor, n_single: int, y: torch.Tensor,
+              out: Optional[torch.Tensor], norm_w: torch.Tensor, eps: float, workspace: Optional[torch.Tensor] = None, method: int = SCAN_AUTO) -> None:
+    """Retention over a ragged batch, with the norm and gate behind (``hds_retention``). ``state`` [slots, heads, vdim, dim] fp32; heads
+    hold ``norm_cols`` values and zeros; ``y`` fp32 scratch; ``out`` None: advance the state alone."""
+    T = q.shape[0]
+    _, heads, vdim, dim = state.shape
+    assert q.stride(0) == k.stride(0) == v.stride(0) == gate.stride(0) and log2_decay.numel() == heads and freq.numel() == dim // 2
+    done = ctypes.c_int(1)
+    rc = native.cuda_lib().hds_retention(_p(q), _p(k), _p(v), _p(gate), q.stride(0), _p(log2_decay), _p(freq), _p(amp), k_scale, norm_cols, _p(state),
+                                         _p(spans), spans.shape[0], n_single, T, heads, vdim, dim, _p(y), y.stride(0), _p(out),
+                                         0 if out is None else out.stride(0), _p(norm_w), eps, _p(workspace),
+                                         0 if workspace is None else workspace.numel(), method, ctypes.addressof(done), _dt3(q), _stream())
+    native.check(rc, "hds_retention")
+    _count((3 if out is not None else 2) * (spans.shape[0] > n_single) + (n_single > 0))
+    if out is not None and not done.value:
+        r = vdim / norm_cols          # mean over a padded row * r = mean over the head
+        gated_norm(y[:, :heads * vdim], gate, norm_w, out, heads, eps / r, r**-0.5, gate_after=True)

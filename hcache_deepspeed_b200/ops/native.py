@@ -38,7 +38,7 @@ def _declare_cuda(lib: ctypes.CDLL, partial: bool = False) -> None:
         "hds_gemm": [P, L, P, L, I, I, I, I, I, I, P, P, L, I, I, P, L, P],
         "hds_gemm_accum": [P, L, P, L, I, I, I, I, P, P, I, I, L, I, I, P],
         "hds_restore_kv_proj": [P, L, P, L, I, I, I, P, P, P, P, P, I, I, I, I, P],
-        "hds_qkv_rope_proj": [P, L, P, L, I, I, I, P, P, P, P, P, P, I, I, I, I, I, P],
+        "hds_qkv_rope_proj": [P, L, P, L, I, I, I, P, P, P, P, P, P, P, I, I, I, I, I, P],
         "hds_restore_kv_proj_peers": [P, I, I, L, P, L, I, I, I, P, P, P, P, P, I, I, I, I, P],
         "hds_norm": [P, L, P, I, I, P, P, L, P, P, P, I, I, F, I, I, I, P],
         "hds_norm_tp": [I, I, I, P, L, P, P, I, P, P, P, L, P, P, I, I, I, P, P, I, F, I, I, P],
@@ -53,9 +53,11 @@ def _declare_cuda(lib: ctypes.CDLL, partial: bool = False) -> None:
         "hds_attention_next_sink": [P],
         "hds_attention_next_sigmoid": [P],
         "hds_attention_next_gate": [P, L],
-        "hds_attention_append": [P, L, P, P, P, P, I, I, I, I, I, P, P, P, I, I, F, P, I, P, I, P],
+        "hds_attention_next_softcap": [F],
+        "hds_attention_append": [P, L, P, P, P, P, I, I, I, I, I, P, P, P, P, I, I, F, P, I, P, I, P],
         "hds_mix_cached_values": [P, P, I, P, P, I, I, I, I, I, P],
         "hds_gru": [P, L, P, P, P, I, I, I, I, P, L, P, L, I, P],
+        "hds_retention": [P, P, P, P, L, P, P, P, F, I, P, P, I, I, I, I, I, I, P, L, P, L, P, F, P, L, I, P, I, P],
         "hds_linear_attention": [P, P, P, P, L, P, L, P, F, P, P, I, I, I, I, I, I, P, L, P, L, P, F, P, L, I, P, I, P],
         "hds_gemm_next_act_limit": [F],
         "hds_moe_table_route": [P, P, I, I, I, I, P, P, P, P, P],
@@ -126,6 +128,8 @@ def _declare_cuda(lib: ctypes.CDLL, partial: bool = False) -> None:
     lib.hds_gru_workspace_bytes.restype = c_int64
     lib.hds_linear_attention_workspace_bytes.argtypes = [I, I, I, I, I]
     lib.hds_linear_attention_workspace_bytes.restype = c_int64
+    lib.hds_retention_workspace_bytes.argtypes = [I, I, I, I, I]
+    lib.hds_retention_workspace_bytes.restype = c_int64
     lib.hds_moe_padded_rows.argtypes = [I, I, I]
     lib.hds_moe_padded_rows.restype = c_int64
     # optional entry points (declared when present so older builds keep loading)

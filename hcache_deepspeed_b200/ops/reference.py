@@ -105,12 +105,13 @@ def gather_kv(kv_cache_layer: torch.Tensor, block_table_row: torch.Tensor, kv_le
 def paged_attention(q: torch.Tensor, kv_cache_layer: torch.Tensor, block_tables: torch.Tensor, items: torch.Tensor,
                     n_q_heads: int, n_kv_heads: int, scale: float, out: Optional[torch.Tensor] = None,
                     alibi: Optional[torch.Tensor] = None, window: int = 0, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
-                    sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, softcap: float = 0.0) -> torch.Tensor:
     """q: [T, n_q_heads, d]; items: int32 [n, 4] rows (seq, q_row0, n_q, pos0). Causal over absolute positions.
     ``alibi``: [n_q_heads] slopes, score += slope * (key position - query position). ``window`` > 0: a query at position p
     sees the keys (p - window, p] only, and the first ``keep_first`` positions of its sequence. ``sink`` [n_q_heads]: one more
     score in every softmax, without a key. ``sigmoid_bias`` [n_q_heads]: weights are sigmoid(score + bias) instead, not
-    normalized. ``gate`` [T, n_q_heads * d]: the output is multiplied by its sigmoid."""
+    normalized. ``gate`` [T, n_q_heads * d]: the output is multiplied by its sigmoid. ``softcap`` > 0: scaled scores are bounded by
+    softcap * tanh(score / softcap) before anything else."""
     T, _, d = q.shape
     if out is None:
         out = torch.zeros_like(q)
@@ -122,6 +123,8 @@ def paged_attention(q: torch.Tensor, kv_cache_layer: torch.Tensor, block_tables:
         v = v.float().repeat_interleave(G, dim=1)
         qq = q[q_row0:q_row0 + n_q].float()  # [n_q, H, d]
         s = torch.einsum("qhd,khd->hqk", qq, k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         kv_pos = torch.arange(kv_len, device=q.device)[None, None, :]
         q_pos = (pos0 + torch.arange(n_q, device=q.device))[None, :, None]
         if alibi is not None:
@@ -292,25 +295,35 @@ def paged_latent_attention(q: torch.Tensor, pages: torch.Tensor, block_tables: t
 
 def attention_append(qkv: torch.Tensor, kv_cache_layer: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, n_q: int, n_kv: int,
                      freq: Optional[torch.Tensor], q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], q_cols: int, k_cols: int,
-                     eps: float, first: Optional[torch.Tensor], share: Optional[torch.Tensor]) -> torch.Tensor:
+                     eps: float, first: Optional[torch.Tensor], share: Optional[torch.Tensor], amp: Optional[torch.Tensor] = None,
+                     head_dim: int = 0) -> torch.Tensor:
     """What lies between a layer's projections ``qkv`` = [q heads | k heads | v heads] and its attention: all of q (k) normed over its
-    ``q_cols`` (``k_cols``) values, heads rotated by halves with the angles pos * freq, values mixed with those that the layer with
-    the pages ``first`` cached of the same tokens. K and V go to their pages; returns q, fp32 [T, n_q * D]."""
-    T, D = qkv.shape[0], kv_cache_layer.shape[4]
+    ``q_cols`` (``k_cols``) values, heads rotated by halves with the angles pos * freq (and times ``amp``), values mixed with those that
+    the layer with the pages ``first`` cached of the same tokens. K and V go to their pages; returns q, fp32 [T, n_q * D].
+    ``n_kv`` = 0: queries alone, heads of ``head_dim``, no pages."""
+    T, D = qkv.shape[0], kv_cache_layer.shape[4] if n_kv else head_dim
     q, k, v = qkv[:, :(n_q + 2 * n_kv) * D].float().split([n_q * D, n_kv * D, n_kv * D], 1)
 
     def normed(x, w, cols):
         return x if w is None else x * torch.rsqrt((x * x).sum(-1, keepdim=True) / cols + eps) * w
 
     def rotated(x):
-        return x if freq is None else rope_rotate_half(x, pos, freq, D)
+        return x if freq is None else rotate_halves(x, pos, freq, amp)
 
+    if n_kv == 0:
+        return rotated(normed(q, q_norm, q_cols).reshape(T, n_q, D)).reshape(T, n_q * D)
     q, k = normed(q, q_norm if n_q else None, q_cols).reshape(T, n_q, D), normed(k, k_norm, k_cols).reshape(T, n_kv, D)
     v = v.reshape(T, n_kv, D)
     if first is not None:
         v = mixed_values(v, first, slot, share)
     kv_append(kv_cache_layer, rotated(k), v, slot)
     return rotated(q).reshape(T, n_q * D)
+
+
+def rotate_halves(x: torch.Tensor, pos: torch.Tensor, freq: torch.Tensor, amp: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x [T, heads, D]: the values c and D / 2 + c turned by pos * freq[c] and multiplied by amp[c]; fp32."""
+    y = rope_rotate_half(x.float(), pos, freq, x.shape[-1])
+    return y if amp is None else y * torch.cat([amp, amp])
 
 
 def mixed_values(v: torch.Tensor, first: torch.Tensor, slot: torch.Tensor, share: torch.Tensor) -> torch.Tensor:
@@ -346,4 +359,15 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.
     for t in range(v.shape[0]):
         state.mul_(decay[t][:, None, :]).add_(v[t].float()[:, :, None] * k[t].float()[:, None, :])
         y[t] = (state * q[t][:, None, :]).sum(-1)
+    return y
+
+
+def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log2_decay: torch.Tensor, scale: float, state: torch.Tensor) -> torch.Tensor:
+    """S <- decay S + v (scale k)^T, y = S q for every token of one sequence; q / k [n, heads, N], v [n, heads, P], log2_decay [heads];
+    ``state`` [heads, P, N] fp32 is advanced in place."""
+    y, decay = torch.empty(v.shape, dtype=torch.float32), torch.exp2(log2_decay)[:, None, None]
+    k = k.float() * scale
+    for t in range(v.shape[0]):
+        state.mul_(decay).add_(v[t].float()[:, :, None] * k[t][:, None, :])
+        y[t] = (state * q[t].float()[:, None, :]).sum(-1)
     return y

@@ -71,10 +71,10 @@ int hds_restore_kv_proj_peers(const void* const* latent_ptrs, int n_peers, int r
                               void* stream);
 
 /* Forward QKV projection with the same fused epilogue: Q (RoPE) -> q_out[T, n_q*d]; K (RoPE), V -> paged cache.
- * w_qkv rows: Q heads, K heads, V heads. */
+ * w_qkv rows: Q heads, K heads, V heads (n_kv_heads 0: Q alone). rot_amp (optional, like inv_freq): factors of the rotated pairs. */
 int hds_qkv_rope_proj(const void* x, int64_t ldx, const void* w_qkv, int64_t ldw, int T, int H, int dtype,
                       const void* bias_qkv, void* q_out, void* kv_cache_layer, const int32_t* tok_pos,
-                      const int32_t* tok_slot, const float* inv_freq, int n_q_heads, int n_kv_heads, int head_dim,
+                      const int32_t* tok_slot, const float* inv_freq, const float* rot_amp, int n_q_heads, int n_kv_heads, int head_dim,
                       int block_size, int do_rope, void* stream);
 
 /* ---- normalisation ------------------------------------------------------------------------- */
@@ -248,10 +248,12 @@ int hds_attention_next_out_stride(int64_t elements);
 /* Further options of the same launch (all three kernel families; device pointers, cleared by that launch):
  *   sink    n_q_heads floats: one more score, without key or value and not scaled, in the denominator of every softmax
  *   sigmoid n_q_heads floats: a visible key weighs sigmoid(score + bias[head]); weights are not normalized
- *   gate    rows like the output's (operand type, ld elements apart): the output is multiplied by its sigmoid */
+ *   gate    rows like the output's (operand type, ld elements apart): the output is multiplied by its sigmoid
+ *   softcap > 0: scaled scores become cap * tanh(score / cap) (not with alibi or sigmoid) */
 int hds_attention_next_sink(const float* sink);
 int hds_attention_next_sigmoid(const float* bias);
 int hds_attention_next_gate(const void* gate, int64_t ld);
+int hds_attention_next_softcap(float cap);
 
 /* Paged attention in plain fp32 arithmetic for operands and head sizes the tensor-core kernels do not take: dtype 0 bf16,
  * 1 fp16, 2 fp32, head_dim up to 512. One warp per (token, query head); tok_seq / tok_pos give each token's block-table row and
@@ -294,8 +296,9 @@ int64_t hds_paged_attention_prefill_workspace_bytes(int n_items, int n_q_heads, 
 /* Per token: softmax over E logits, top-k (ties -> lower index), optional renormalisation of the k scores.
  * counts[E] must be zero on entry (hds_moe_scatter re-zeroes it). offsets[t, j] = row claimed inside expert_ids[t, j].
  * bias[E] (optional) is added to the scores that choose, `scale` multiplies the returned ones, `clear` zeroes the (fp32)
- * logits after they are read. `sigmoid`: the scores are the logits' sigmoids, each by itself. */
-int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E, int k, int normalize, int sigmoid, const float* bias, float scale,
+ * logits after they are read. kind 1: the scores are the logits' sigmoids, each by itself; 2: bias is added to the logits themselves,
+ * the largest of which are chosen. */
+int hds_moe_topk_gating(void* logits, int64_t ld_logits, int T, int E, int k, int normalize, int kind, const float* bias, float scale,
                         int clear, int logits_dtype, float* scores, int32_t* expert_ids, int32_t* offsets, int32_t* counts, void* stream);
 /* pad_off[E+1]: expert row ranges rounded up to 128 rows; xs[row] = x[t] for every (t, j); mapped_slots[t, j] = row. scores
  * (optional): xs[row] = scores[t, j] * x[t] in the rows' type (dtype 0 / 1 / 2). H and strides count 16-bit units.
@@ -464,11 +467,11 @@ int64_t hds_paged_attention_latent_workspace_bytes(void);
 /* Projected rows qkv = [n_q heads | n_kv heads | n_kv heads] of head_dim values -> q_out [T, n_q * head_dim] and the tokens' K / V page
  * rows (tok_slot < 0: none). q_norm / k_norm (optional, together; fp32 per column): all of a row's q (k) divided by its root mean
  * square over q_cols (k_cols) values and weighted. freq (optional, [head_dim / 2]): value c turns with value head_dim / 2 + c by
- * position * freq[c]. first (optional): pages [blocks][2][n_kv][block][first_dim] of another layer; v = (1 - share) v + share *
- * its cached value of the same token. dtype 0 / 1 / 2. n_q_heads 0: keys and values alone. */
+ * position * freq[c], both times amp[c] (optional). first (optional): pages [blocks][2][n_kv][block][first_dim] of another layer; v = (1 - share) v + share *
+ * its cached value of the same token. dtype 0 / 1 / 2. n_q_heads 0: keys and values alone; n_kv_heads 0: queries alone, no pages. */
 int hds_attention_append(const void* qkv, int64_t ld_qkv, void* q_out, void* kv_cache_layer, const int32_t* tok_pos,
                          const int32_t* tok_slot, int T, int n_q_heads, int n_kv_heads, int head_dim, int block_size, const float* freq,
-                         const float* q_norm, const float* k_norm, int q_cols, int k_cols, float eps, const void* first, int first_dim,
+                         const float* amp, const float* q_norm, const float* k_norm, int q_cols, int k_cols, float eps, const void* first, int first_dim,
                          const float* share, int dtype, void* stream);
 /* The same mixing of the tokens' values, in place in their pages. */
 int hds_mix_cached_values(void* kv_cache_layer, const void* first, int first_dim, const int32_t* tok_slot, const float* share, int T,
@@ -491,6 +494,15 @@ int hds_linear_attention(const void* q, const void* k, const void* v, const void
                          int vdim, int dim, float* y, int64_t ld_y, void* out, int64_t ld_out, const float* norm_w, float eps,
                          void* workspace, int64_t workspace_bytes, int method, int* finished, int dtype, void* stream);
 int64_t hds_linear_attention_workspace_bytes(int T, int n_seqs, int heads, int vdim, int dim);
+
+/* Retention over a ragged batch: as hds_linear_attention, but every head's state fades by a constant: S = 2^log2_decay[head] S + v k'^T,
+ * y = S q'. q' and k' are q and k whose values c and dim / 2 + c of a head are turned by position * freq[c] and multiplied by amp[c]
+ * (optional); k' also by k_scale. norm_cols: values of a head that its norm averages over (the others are zero padding). */
+int hds_retention(const void* q, const void* k, const void* v, const void* gate, int64_t ld, const float* log2_decay, const float* freq,
+                  const float* amp, float k_scale, int norm_cols, float* state, const int32_t* spans, int n_seqs, int n_single, int T, int heads,
+                  int vdim, int dim, float* y, int64_t ld_y, void* out, int64_t ld_out, const float* norm_w, float eps, void* workspace,
+                  int64_t workspace_bytes, int method, int* finished, int dtype, void* stream);
+int64_t hds_retention_workspace_bytes(int T, int n_seqs, int heads, int vdim, int dim);
 
 #ifdef __cplusplus
 }
