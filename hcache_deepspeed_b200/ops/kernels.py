@@ -919,3 +919,10 @@ def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Ten
     if out is not None and not done.value:
         r = vdim / norm_cols          # mean over a padded row * r = mean over the head
         gated_norm(y[:, :heads * vdim], gate, norm_w, out, heads, eps / r, r**-0.5, gate_after=True)
+
+
+def retention_stuck() -> bool:
+    """Has a wait inside retention's kernels ever run out of time? (Synchronizes.)"""
+    flag = ctypes.c_int(0)
+    native.check(native.cuda_lib().hds_retention_status(ctypes.addressof(flag)), "hds_retention_status")
+    return bool(flag.value)

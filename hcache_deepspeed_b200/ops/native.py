@@ -57,6 +57,7 @@ def _declare_cuda(lib: ctypes.CDLL, partial: bool = False) -> None:
         "hds_attention_append": [P, L, P, P, P, P, I, I, I, I, I, P, P, P, P, I, I, F, P, I, P, I, P],
         "hds_mix_cached_values": [P, P, I, P, P, I, I, I, I, I, P],
         "hds_gru": [P, L, P, P, P, I, I, I, I, P, L, P, L, I, P],
+        "hds_retention_status": [P],
         "hds_retention": [P, P, P, P, L, P, P, P, F, I, P, P, I, I, I, I, I, I, P, L, P, L, P, F, P, L, I, P, I, P],
         "hds_linear_attention": [P, P, P, P, L, P, L, P, F, P, P, I, I, I, I, I, I, P, L, P, L, P, F, P, L, I, P, I, P],
         "hds_gemm_next_act_limit": [F],

@@ -87,6 +87,8 @@ def make_weights(cfg, seed, dtype, settled):
         if lc["type"] == "retention":
             for n, rows in (("q", m["heads"] * m["dim"]), ("k", m["heads"] * m["dim"]), ("v", n_o), ("g", n_o)):
                 w[q + n] = rnd(rows, W)
+            if settled:       # (a token's own key answers its query: no head's output is so small that its norm magnifies rounding)
+                w[q + "k"] = (0.8 * w[q + "q"].float() + 0.6 * w[q + "k"].float()).to(dtype)
         else:
             own = [("q", m["heads"] * m["dim"])]
             if m.get("kv_from") is None:
@@ -104,7 +106,7 @@ def make_weights(cfg, seed, dtype, settled):
             for x, t in like.items():
                 own = rnd(*t.shape, scale=(2 if x == "down" else 1) * t.shape[1]**-0.5)
                 # (settled: experts so alike that a choice which rounding decides makes no difference to speak of)
-                w[f"{q}e{e}.{x}"] = t + own * 0.1 if settled else own
+                w[f"{q}e{e}.{x}"] = t + own * 0.05 if settled else own
     return w
 
 
