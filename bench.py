@@ -54,9 +54,10 @@ def parse():
                         "e.g. the OPT-30B TP=4 NVMe configuration), instead of what the planner would choose")
     p.add_argument("--plan", default="hidden", choices=["auto", "hidden", "planner", "adaptive"],
                    help="hidden: every layer from hidden states (fastest measured on 1xB200: 20.4 ms vs 21.6 ms); auto: planner mix with a recomputed prefix")
-    p.add_argument("--stacks", action="store_true",
-                   help="instead of the headline workload: prefill and decode throughput of the Lotelix, Dedelorn and Nipolorn stacks beside the "
-                        "closest plain families at equal sizes, and their kernels against the measured peaks (one JSON line each; one GPU)")
+    p.add_argument("--stacks", nargs="?", const="all", default=None, metavar="FAMILY",
+                   help="instead of the headline workload: prefill and decode throughput of the Relulix, Lotelix, Dedelorn and Nipolorn stacks beside "
+                        "the closest plain families at equal sizes, and their kernels against the measured peaks (one JSON line each; one GPU); with "
+                        "a family (relulix, lotelix) only its sizes and kernels and their like")
     return p.parse_args()
 
 
@@ -338,7 +339,7 @@ if __name__ == "__main__":
     args = parse()
     if args.stacks:
         from hcache_deepspeed_b200.benchmarks.stacks import main as run_stacks
-        run_stacks(args.steps, args.warmup)
+        run_stacks(args.steps, args.warmup, only="" if args.stacks == "all" else args.stacks)
     elif args.impl == "reference":
         run_reference(args)
     else:

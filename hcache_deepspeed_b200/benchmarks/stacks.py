@@ -14,7 +14,7 @@ from typing import Callable, Dict, Optional
 import torch
 
 GROUPS = [("dedelorn-2048", "nipolorn-2048", "mistral-2048"), ("dedelorn-4096", "nipolorn-4096", "mistral-4096"),
-          ("lotelix-2048", "dedelorn-2048-moe"), ("lotelix-4096", "dedelorn-4096-moe", "nipolorn-4096-moe", "qwen2-moe-4096")]
+          ("relulix-2048", "lotelix-2048", "dedelorn-2048-moe"), ("relulix-4096", "lotelix-4096", "dedelorn-4096-moe", "nipolorn-4096-moe", "qwen2-moe-4096")]
 PROMPT = 4096
 
 
@@ -338,16 +338,106 @@ def bench_lotelix_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
         report(f"combine {rows}", "moe_combine, weighted (like)", lambda: K.moe_combine(ys, slots, scores, None, out), rows * W * (2 * top + 4))
 
 
-def main(steps: int = 5, warmup: int = 3) -> None:
+def bench_relulix_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
+    """The same for what Relulix adds: retention (32 heads of 128 x 128 and of 64 x 128), bounded scores with a one more, rotation with amplitudes,
+    queries alone, experts weighed among the chosen, clamped gated experts."""
+    from ..ops import kernels as K
+    from ..ops.backend import pick_packed_splits, windowed_len
+    dev, rnd, report = "cuda", _rnd, _reporter(p, iters, warmup)
+    W, T, heads, P = 4096, PROMPT, 32, 128
+    i32 = lambda *s: torch.zeros(s, dtype=torch.int32, device=dev)  # noqa: E731
+    for N in (128, 64):
+        decay, freq = torch.linspace(-0.05, -1e-3, heads, device=dev), 1e6**(-torch.arange(N // 2, device=dev) / (N // 2))
+        for rows, seqs in ((T, 1), (T, 4), (64, 64), (8, 8)):
+            n = rows // seqs
+            single = seqs if n == 1 else 0
+            spans = torch.tensor([[i * n, n, 128, i] for i in range(seqs)], dtype=torch.int32, device=dev)
+            proj, z, state, mix = rnd(rows, 2 * heads * (N + P)), rnd(rows, heads * N), torch.zeros(seqs, heads, P, N, device=dev), rnd(rows, heads * P)
+            q, k, v, gate = proj.split([heads * N, heads * N, heads * P, heads * P], 1)
+            b, w, y = torch.ones(heads * N, device=dev), torch.ones(heads * P, device=dev), torch.zeros(rows, heads * P, device=dev)
+            moved = rows * heads * (2 * N + 3 * P) * 2 + 2 * seqs * heads * P * N * 4
+            tag = "chunks, norm and gate" if n > 1 else "step, norm and gate"
+            ws = torch.empty(K.retention_workspace_bytes(rows, seqs, heads, P, N), dtype=torch.uint8, device=dev)
+            report(f"retention {seqs}x{n}, heads {N}x{P}", tag, lambda: K.retention(
+                q, k, v, gate, decay, freq, None, N**-0.5, P, state, spans, single, y, mix, w, 1e-5, ws), moved)
+            ws = torch.empty(K.linear_attention_workspace_bytes(rows, seqs, heads, P, N), dtype=torch.uint8, device=dev)
+            report(f"retention {seqs}x{n}, heads {N}x{P}", "linear attention, norm and gate (like)", lambda: K.linear_attention(
+                q, k, v, gate, z, b, 1 / 16, state, spans, single, y, mix, w, 1e-5, ws), moved + rows * heads * N * 2)
+            del ws
+    nq, nkv, D, page, window = 32, 8, 128, 64, 2048
+    ws = torch.zeros(256 << 20, dtype=torch.uint8, device=dev)
+    sink = torch.zeros(nq, device=dev)
+    cases = [("softmax (like)", {}), ("sink (like)", {"sink": sink}), ("bounded, one more", {"sink": sink, "softcap": 30.0})]
+    cache, q, o = rnd(T // page + 1, 2, nkv, page, D), rnd(T, nq * D), rnd(T, nq * D)
+    table = torch.randperm(T // page, device=dev).to(torch.int32)[None].contiguous()
+    items = torch.tensor([[0, i, 128, i] for i in range(0, T, 128)], dtype=torch.int32, device=dev)
+    pairs = sum(min(i + 1, window) for i in range(T))
+    for tag, opts in cases:
+        report(f"attention prefill {T} window {window}", tag, lambda: K.paged_attention_prefill(
+            q, o, cache, table, items, T // 128, nq, nkv, D, page, 0.09, window=window, **opts), flops=4.0 * pairs * nq * D)
+    B = 64
+    for kvh in (nkv, nq):         # head-packed on the tensor cores, and one query head per key head
+        cache = rnd(B * T // page // (kvh // nkv), 2, kvh, page, D)
+        tables = torch.arange(cache.shape[0], device=dev).to(torch.int32).view(-1, T // page).contiguous()
+        n = tables.shape[0]
+        items = torch.tensor([[i, i, 1, T - 1] for i in range(n)], dtype=torch.int32, device=dev)
+        qd, od = rnd(n, nq * D), rnd(n, nq * D)
+        for tag, opts in cases:
+            need = n * window * 2 * kvh * D * 2
+            if kvh == nkv:
+                sp = pick_packed_splits(n, kvh, windowed_len(T, window))
+                report(f"attention decode {n}x{T} window {window}, {nq} / {kvh} heads", tag, lambda: K.paged_attention_prefill(
+                    qd, od, cache, tables, items, n, nq, kvh, D, page, 0.09, n_splits=sp, workspace=ws, packed=True, window=window, **opts), need)
+            else:
+                report(f"attention decode {n}x{T} window {window}, {nq} / {kvh} heads", tag, lambda: K.paged_attention_splitkv(
+                    qd, od, cache, tables, items, n, 1, nq, kvh, D, page, 1, 0.09, ws, window=window, **opts), need)
+    del cache
+    freq, amp = 1e4**(-torch.arange(64, device=dev) / 64), torch.full((64, ), 1.1, device=dev)
+    x, w, b = rnd(T, W), rnd((nq + 2 * nkv) * D, W, scale=0.02), rnd((nq + 2 * nkv) * D)
+    pages, pos = rnd(T // page, 2, nkv, page, D), torch.arange(T, dtype=torch.int32, device=dev)
+    for tag, n, kw in (("biases, rotation with amplitudes, pages", nkv, {"bias_qkv": b, "amp": amp}), ("the same, queries alone", 0, {"bias_qkv": b, "amp": amp}),
+                       ("rotation, pages (like)", nkv, {})):
+        rows = (nq + 2 * n) * D
+        report(f"q, k, v of {T}", tag, lambda: K.qkv_rope_proj(x, w[:rows], q, pages, pos, pos, freq, nq, n, D, page, **kw), flops=2.0 * T * rows * W)
+    for rows in (64, ):
+        qkv, n_all = rnd(rows, (nq + 2 * nkv) * D), (nq + 2 * nkv) * D
+        for tag, n, kw in (("rotation with amplitudes, pages", nkv, {"amp": amp}), ("the same, queries alone", 0, {"amp": amp})):
+            report(f"attention inputs {rows}", tag, lambda: K.attention_append(qkv, q, pages, pos, pos, nq, n, D, page, freq, **kw), rows * 4 * (nq + 2 * n) * D)
+        report(f"attention inputs {rows}", "rope_kv_append (like)", lambda: K.rope_kv_append(qkv, q, pages, pos, pos, freq, nq, nkv, D, D, page), rows * 4 * n_all)
+    del x, w, pages
+    E, top, ff = 16, 2, 3584
+    for rows in (T, 64):
+        scores, e, off, slots, counts, pad = torch.zeros(rows, top, device=dev), i32(rows, top), i32(rows, top), i32(rows, top), i32(E), i32(E + 1)
+        R = K.moe_padded_rows(rows, E, top)
+        x, xs, wr, lg, bias = rnd(rows, W), rnd(R, W), rnd(E, W, scale=0.02), torch.zeros(rows, E, device=dev), torch.zeros(E, device=dev)
+        hs, wu = rnd(R, ff), rnd(E * 2 * ff, W, scale=0.02)
+
+        def route(**kw):
+            K.gemm_accum(x, wr, lg)
+            K.moe_topk_gating(lg, top, bool(kw), scores, e, off, counts, clear=True, **kw)
+            K.moe_scatter(x, xs, e, off, counts, pad, slots, top)
+
+        for tag, kw in (("logits with a bias choose", {"bias": bias, "biased": True}), ("softmax scores (like)", {})):
+            report(f"router + route + scatter {rows}", tag, lambda: route(**kw), rows * W * 2 * (2 + top))
+        for tag, act in (("grouped GEMM, clamped gate", 5), ("grouped GEMM, silu gate (like)", 3)):
+            report(f"experts up {rows}", tag, lambda: K.moe_gemm(xs, wu, pad, E, hs, act=act, gated=True, limit=7.0),
+                   2 * (wu.numel() + rows * top * (W + ff)), 2.0 * rows * top * W * 2 * ff)
+        ys, d32, out = rnd(R, W), torch.zeros(rows, W, device=dev), torch.zeros(rows, W, device=dev)
+        report(f"combine {rows}", "moe_combine onto the mixer's output", lambda: K.moe_combine(ys, slots, scores, d32, d32), rows * W * (2 * top + 8))
+        report(f"combine {rows}", "moe_combine (like)", lambda: K.moe_combine(ys, slots, scores, None, out), rows * W * (2 * top + 4))
+
+
+def main(steps: int = 5, warmup: int = 3, only: str = "") -> None:
     p = peaks()
     for group in GROUPS:
-        for name in group:
+        for name in group if not only or any(n.startswith(only) for n in group) else ():
             print(json.dumps({"stack": name, "layers": 4, "prompt": PROMPT, "dtype": "bf16", "data": "random weights, synthetic tokens",
                               **bench_engine(name, steps, warmup)}), flush=True)
             torch.cuda.empty_cache()
-    bench_kernels(p, max(steps, 10), warmup)
-    torch.cuda.empty_cache()
-    bench_lotelix_kernels(p, max(steps, 10), warmup)
+    for prefix, kernels in (("", bench_kernels), ("lotelix", bench_lotelix_kernels), ("relulix", bench_relulix_kernels)):
+        if not only or only == prefix:
+            kernels(p, max(steps, 10), warmup)
+            torch.cuda.empty_cache()
 
 
 if __name__ == "__main__":

@@ -992,7 +992,7 @@ def named_arch(name: str) -> ArchSpec:
 
 
 def _stack_named() -> Dict[str, ArchSpec]:
-    """Nipolorn, Dedelorn and Lotelix stacks with layers of real sizes, and beside each the closest plain family at equal sizes (same
+    """Nipolorn, Dedelorn, Lotelix and Relulix stacks with layers of real sizes, and beside each the closest plain family at equal sizes (same
     width, heads, window and feed-forward): windowed attention with a dense MLP, or with routed experts and a shared one."""
 
     def nipolorn(width, heads, kv, window, keep, ssm_heads, groups, mlp):
@@ -1020,6 +1020,18 @@ def _stack_named() -> Dict[str, ArchSpec]:
         return stack_arch("lotelix", [LayerSpec(m, mlp) for m in (MixerSpec(gru=GRUSpec(width)), attn(), both, attn(1))], hidden=width, vocab=32000,
                           norm_eps=1e-5, norm_groups=2, embed_scale=1.0)
 
+    def relulix(width, heads, kv, window, ff):
+        rot = RotationSpec(64, 1e6, False, 4.0, 1.0, 32.0, 8192, True, 0.1 * math.log(4.0) + 1.0)
+
+        def attn(kv_from=None):
+            return MixerSpec(attn=AttentionSpec(heads, kv, 128, 128, 128**-0.5, window, rot=rot, bias=True, one_more=True, softcap=30.0, kv_from=kv_from))
+
+        n = width // 128
+        ret = MixerSpec(retention=RetentionSpec(n, 128, 128, [1.0 - 2.0**(-5.0 - 7.0 * i / n) for i in range(n)], RotationSpec(128, 1e6)))
+        mlp = FeedForwardSpec(ff=ff, act="swiglu_clamped", limit=7.0, experts=16, top=2, routing="chosen")
+        return stack_arch("relulix", [LayerSpec(m, mlp) for m in (ret, attn(), ret, attn(1))], hidden=width, vocab=32000, norm_eps=1e-5, embed_scale=1.0,
+                          **RELULIX_NORMS)
+
     def plain(mt, width, heads, kv, window, **kw):
         return ArchSpec(model_type=mt, n_layers=4, hidden=width, n_heads=heads, n_kv_heads=kv, head_dim=128, vocab=32000, norm="rms",
                         norm_eps=1e-5, act="silu", gated_mlp=True, pos_emb="rope", sliding_window=window, max_positions=1 << 20, **kw)
@@ -1035,6 +1047,8 @@ def _stack_named() -> Dict[str, ArchSpec]:
                                                                             router_scale=2.5)),
         "lotelix-2048": lotelix(2048, 16, 4, 1024, 2688),
         "lotelix-4096": lotelix(4096, 32, 8, 2048, 5376),
+        "relulix-2048": relulix(2048, 16, 4, 1024, 1792),
+        "relulix-4096": relulix(4096, 32, 8, 2048, 3584),
         "mistral-2048": plain("mistral", 2048, 16, 4, 1024, intermediate=8192),
         "nipolorn-4096": nipolorn(4096, 32, 8, 4096, 64, 128, 8, FeedForwardSpec(ff=14336, act="swiglu_clamped", limit=7.0)),
         "mistral-4096": plain("mistral", 4096, 32, 8, 4096, intermediate=14336),
