@@ -347,7 +347,7 @@ def bench_relulix_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
     W, T, heads, P = 4096, PROMPT, 32, 128
     i32 = lambda *s: torch.zeros(s, dtype=torch.int32, device=dev)  # noqa: E731
     for N in (128, 64):
-        decay, freq = torch.linspace(-0.05, -1e-3, heads, device=dev), 1e6**(-torch.arange(N // 2, device=dev) / (N // 2))
+        decay = torch.linspace(-0.05, -1e-3, heads, device=dev)
         for rows, seqs in ((T, 1), (T, 4), (64, 64), (8, 8)):
             n = rows // seqs
             single = seqs if n == 1 else 0
@@ -359,7 +359,7 @@ def bench_relulix_kernels(p: Dict[str, float], iters: int, warmup: int) -> None:
             tag = "chunks, norm and gate" if n > 1 else "step, norm and gate"
             ws = torch.empty(K.retention_workspace_bytes(rows, seqs, heads, P, N), dtype=torch.uint8, device=dev)
             report(f"retention {seqs}x{n}, heads {N}x{P}", tag, lambda: K.retention(
-                q, k, v, gate, decay, freq, None, N**-0.5, P, state, spans, single, y, mix, w, 1e-5, ws), moved)
+                q, k, v, gate, decay, None, None, N**-0.5, P, state, spans, single, y, mix, w, 1e-5, ws), moved)
             ws = torch.empty(K.linear_attention_workspace_bytes(rows, seqs, heads, P, N), dtype=torch.uint8, device=dev)
             report(f"retention {seqs}x{n}, heads {N}x{P}", "linear attention, norm and gate (like)", lambda: K.linear_attention(
                 q, k, v, gate, z, b, 1 / 16, state, spans, single, y, mix, w, 1e-5, ws), moved + rows * heads * N * 2)

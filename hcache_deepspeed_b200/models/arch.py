@@ -234,7 +234,8 @@ class LinearAttentionSpec:
 @dataclass
 class RetentionSpec:
     """Retention: linear attention whose heads' ``dim`` x ``vdim`` states fade by a constant each (``decay``); queries and keys
-    rotated by position; a norm per head and a gate behind. Heads are zero padded to multiples of 16."""
+    rotated by position; a norm per head and a gate behind. Queries and keys are zero padded to the kernels' tile sizes 64 and 128
+    (larger ones, and values, to multiples of 16)."""
     heads: int
     dim: int
     vdim: int
@@ -246,7 +247,7 @@ class RetentionSpec:
     @property
     def width(self) -> int:
         """Size of a query or key row of a head."""
-        return -(-self.dim // 16) * 16
+        return 64 if self.dim <= 64 else 128 if self.dim <= 128 else -(-self.dim // 16) * 16
 
     @property
     def vwidth(self) -> int:

@@ -23,8 +23,8 @@ supplies what such a layer does between them, and how its checkpoint pieces are 
 * a minGRU's ``w_qkv`` is ``[gate | candidate | output gate]``; gated linear attention adds ``[q | k | v | gate | decay's first
   projection]`` behind the attention's columns, each padded to 16-byte rows.
 * attention on another layer's keys and values: ``w_qkv`` holds the queries alone, the pages are those of that layer.
-* retention: ``w_qkv`` = ``[q | k | v | gate]``, heads padded to multiples of 16, queries and keys reordered like those of attention;
-  their rotation happens inside the recurrence's kernels, in fp32.
+* retention: ``w_qkv`` = ``[q | k | v | gate]``, heads padded, queries and keys reordered like those of attention. Prompts rotate them
+  in the projection's epilogue, decode steps and fp32 models inside the recurrence's kernels.
 * two mixers with a norm each: ``w_o`` and ``w_o2`` project their parts of the buffer separately; the norm kernel behind norms both,
   with halved weights, while adding them to the stream.
 * ``parallel_residual``: mixer and dense feed-forward read the same norm, so ``w_o`` is ``[mixer columns | feed-forward columns]``
@@ -489,7 +489,8 @@ class HybridTransformer(RaggedTransformer):
         self.xn, self.xn2 = buf(T, Hp), buf(T, Hp)
         self.latent_buf = buf(s.n_layers, T, Hp) if self.capture_enabled else None
         self.in_buf = buf(T * max(pad8(lw.w_qkv.shape[0]) for lw in self.w.layers))
-        self.q_buf = buf(T * max([a.heads * a.page_dim for a in attn] + [c.heads * c.head_width for c in latents] + [8]))
+        self.q_buf = buf(T * max([a.heads * a.page_dim for a in attn] + [c.heads * c.head_width for c in latents] +
+                                 [2 * m.keys for m in rec if isinstance(m, RetentionSpec)] + [8]))
         self.mix_buf = buf(T * max(lw.w_o.shape[1] + (lw.w_o2.shape[1] if lw.w_o2 is not None else 0) for lw in self.w.layers))
         self.conv_buf = buf(T * max((pad8(m.conv_dim) for m in rec), default=8))
         self.dt_buf = buf(T * max((m.heads for m in rec), default=1), dtype=torch.float32)
@@ -661,18 +662,17 @@ class HybridTransformer(RaggedTransformer):
         return r.inner
 
     def _retention_mixer(self, li: int, t: RetentionSpec, lw: LayerWeights, xn: torch.Tensor, mix: torch.Tensor, batch: RaggedBatchWrapper) -> int:
-        proj = self._view(self.in_buf, batch.current_tokens, lw.w_qkv.shape[0])
-        self.ops.gemm(xn, lw.w_qkv, proj, workspace=self.ws_gemm)
-        self._retention(li, t, lw, proj, batch.spans(), batch.n_single_token_seqs, mix[:, :t.inner])
+        self._retention(li, t, lw, xn, batch.tok_pos(), batch.spans(), batch.n_single_token_seqs, mix[:, :t.inner])
         return t.inner
 
-    def _retention(self, li: int, t: RetentionSpec, lw: LayerWeights, proj: torch.Tensor, spans: torch.Tensor, n_single: int,
+    def _retention(self, li: int, t: RetentionSpec, lw: LayerWeights, x: torch.Tensor, pos: torch.Tensor, spans: torch.Tensor, n_single: int,
                    out: Optional[torch.Tensor]) -> None:
-        """Retention of the tokens whose projections are ``proj`` = [q | k | v | gate]; without ``out`` its state alone."""
-        nk, nv = t.keys, t.inner
-        self.ops.retention(proj[:, :nk], proj[:, nk:2 * nk], proj[:, 2 * nk:2 * nk + nv], proj[:, 2 * nk + nv:], lw, t,
-                           self._state_manager.recurrent_states.ssm(li), spans, n_single, self._view(self.scan_buf, proj.shape[0], nv), out,
-                           self.spec.norm_eps, self._scan_ws)
+        """Retention of the tokens whose normed inputs are ``x``; without ``out`` its state alone."""
+        T = x.shape[0]
+        q, k, v, gate, turned = self.ops.retention_in_proj(x, lw, t, self._view(self.in_buf, T, lw.w_qkv.shape[0]), self._view(self.q_buf, T, 2 * t.keys),
+                                                           pos, n_single < spans.shape[0], workspace=self.ws_gemm)
+        self.ops.retention(q, k, v, gate, lw, t, turned, self._state_manager.recurrent_states.ssm(li), spans, n_single,
+                           self._view(self.scan_buf, T, t.inner), out, self.spec.norm_eps, self._scan_ws)
 
     def _linear(self, li: int, g: LinearAttentionSpec, lw: LayerWeights, proj: torch.Tensor, spans: torch.Tensor, n_single: int,
                 out: Optional[torch.Tensor]) -> None:
@@ -757,9 +757,7 @@ class HybridTransformer(RaggedTransformer):
             ops.gemm(latents, lw.w_qkv, proj, workspace=self.ws_gemm)
             ops.gru(proj, lw, m, kv.recurrent_states.ssm(li), spans, n_single, None, self._scan_ws)
         elif isinstance(m, RetentionSpec):
-            proj = self._view(self.in_buf, T, lw.w_qkv.shape[0])
-            ops.gemm(latents, lw.w_qkv, proj, workspace=self.ws_gemm)
-            self._retention(li, m, lw, proj, spans, n_single, None)
+            self._retention(li, m, lw, latents, pos, spans, n_single, None)
         elif isinstance(m, LinearAttentionSpec):
             ops.gemm(latents, lw.w_qkv[n_attn:], proj[:, n_attn:], workspace=self.ws_gemm)
             self._linear(li, m, lw, proj[:, n_attn:], spans, n_single, None)

@@ -182,7 +182,11 @@ class CpuOps:
             out.zero_()
             out[:, :NV] = ref.gated_norm(y[:, :NV], gate[:, :NV], lw.ssm_norm, m.heads, eps, gate_after=True)
 
-    def retention(self, q, k, v, gate, lw, m, state, spans, n_single, y, out, eps, workspace):
+    def retention_in_proj(self, x, lw, m, proj, qk, tok_pos, prompts, workspace=None):
+        self.gemm(x, lw.w_qkv, proj)
+        return (*proj.split([m.keys, m.keys, m.inner, m.inner], 1), False)
+
+    def retention(self, q, k, v, gate, lw, m, turned, state, spans, n_single, y, out, eps, workspace):
         for row0, n, seen, slot in spans.tolist():
             if seen == 0:
                 state[slot].zero_()
@@ -454,8 +458,19 @@ class CudaOps:
     def linear_attention(self, q, k, v, gate, z, lw, m, state, spans, n_single, y, out, eps, workspace):
         self.k.linear_attention(q, k, v, gate, z, lw.decay_bias, 1.0 / m.tau, state, spans, n_single, y, out, lw.ssm_norm, eps, workspace)
 
-    def retention(self, q, k, v, gate, lw, m, state, spans, n_single, y, out, eps, workspace):
-        self.k.retention(q, k, v, gate, lw.ret_decay, lw.rot_freq, lw.rot_amp, m.dim**-0.5, m.vdim, state, spans, n_single, y, out, lw.ssm_norm, eps,
+    def retention_in_proj(self, x, lw, m, proj, qk, tok_pos, prompts, workspace=None):
+        """q, k, v, gate of retention, and whether q and k have been turned: in the epilogue of batches with ``prompts`` that are large
+        enough, for the chunked kernels (which take them so); else the recurrence does it in fp32."""
+        k, nk, nv = self.k, m.keys, m.inner
+        if prompts and x.dtype == torch.bfloat16 and m.width in (64, 128) and x.shape[0] >= self.FUSED_QKV_MIN_TOKENS:
+            k.qkv_rope_proj(x, lw.w_qkv[:2 * nk], qk, None, tok_pos, tok_pos, lw.rot_freq, 2 * m.heads, 0, m.width, 1, amp=lw.rot_amp)
+            k.gemm(x, lw.w_qkv[2 * nk:], out=proj[:, 2 * nk:])
+            return qk[:, :nk], qk[:, nk:], proj[:, 2 * nk:2 * nk + nv], proj[:, 2 * nk + nv:], True
+        self.gemm(x, lw.w_qkv, proj, workspace=workspace)
+        return (*proj.split([nk, nk, nv, nv], 1), False)
+
+    def retention(self, q, k, v, gate, lw, m, turned, state, spans, n_single, y, out, eps, workspace):
+        self.k.retention(q, k, v, gate, lw.ret_decay, None if turned else lw.rot_freq, lw.rot_amp, m.dim**-0.5, m.vdim, state, spans, n_single, y, out, lw.ssm_norm, eps,
                          workspace)
 
     def state_space(self, proj, lw, m, ssm_state, conv_state, spans, n_single, conv_buf, dt_buf, out):

@@ -48,12 +48,9 @@ __global__ void __launch_bounds__(kLsThreads) lin_step_kernel(const LinArgs a) {
         const float pos = static_cast<float>(sp.seen);
         for (int c = threadIdx.x; c < N >> 1; c += kLsThreads) {
             float s, co;
-            lin_sincos<DT>(pos * a.freq[c], &s, &co);
-            if (a.amp != nullptr) {
-                s *= a.amp[c];
-                co *= a.amp[c];
-            }
-            const float2 q = lin_turned<DT>(a, a.q, row * a.ld + h * N, c, s, co), k = lin_turned<DT>(a, a.k, row * a.ld + h * N, c, s, co);
+            lin_turn<DT>(a, pos, c, &s, &co);
+            const int64_t at = row * a.ld_qk + h * N;
+            const float2 q = lin_turned<DT>(a, a.q, at, c, s, co), k = lin_turned<DT>(a, a.k, at, c, s, co);
             q_s[c] = q.x * a.q_scale;
             q_s[c + (N >> 1)] = q.y * a.q_scale;
             k_s[c] = k.x * a.k_scale;
@@ -61,8 +58,8 @@ __global__ void __launch_bounds__(kLsThreads) lin_step_kernel(const LinArgs a) {
         }
     } else {
         for (int n = threadIdx.x; n < N; n += kLsThreads) {
-            q_s[n] = load_any<DT>(a.q, row * a.ld + h * N + n) * a.q_scale;
-            k_s[n] = load_any<DT>(a.k, row * a.ld + h * N + n) * a.k_scale;
+            q_s[n] = load_any<DT>(a.q, row * a.ld_qk + h * N + n) * a.q_scale;
+            k_s[n] = load_any<DT>(a.k, row * a.ld_qk + h * N + n) * a.k_scale;
             d_s[n] = exp2f(lin_log2_decay<DT>(load_any<DT>(a.z, row * a.ld_z + h * N + n) + a.bias[h * N + n], a.inv_tau));
         }
     }
@@ -134,7 +131,7 @@ __global__ void __launch_bounds__(kLsThreads) lin_step_kernel(const LinArgs a) {
     const float r = 1.0f / sqrtf(ss / a.norm_cols + a.eps);
     for (int p = threadIdx.x; p < P; p += kLsThreads) {
         const float g = load_any<DT>(a.gate, row * a.ld + h * P + p);
-        ssm_store<DT>(a.out, row * a.ld_out + h * P + p, o_s[p] * r * a.norm_w[h * P + p] * ssm_silu<DT>(g));
+        ssm_store<DT>(a.out, row * a.ld_out + h * P + p, o_s[p] * r * (a.norm_w != nullptr ? a.norm_w[h * P + p] : 1.0f) * ssm_silu<DT>(g));
     }
 }
 
@@ -171,13 +168,9 @@ __global__ void __launch_bounds__(kLcWarps * 32) lin_scan_kernel(const LinArgs a
             const int half = N >> 1;
             for (int e = threadIdx.x; e < nt * half; e += blockDim.x) {
                 const int t = e / half, c = e - t * half;
-                const int64_t at = (row + t) * a.ld + h * N;
+                const int64_t at = (row + t) * a.ld_qk + h * N;
                 float s, co;
-                lin_sincos<DT>(static_cast<float>(sp.seen + t0 + t) * a.freq[c], &s, &co);
-                if (a.amp != nullptr) {
-                    s *= a.amp[c];
-                    co *= a.amp[c];
-                }
+                lin_turn<DT>(a, static_cast<float>(sp.seen + t0 + t), c, &s, &co);
                 const float2 q = lin_turned<DT>(a, a.q, at, c, s, co), k = lin_turned<DT>(a, a.k, at, c, s, co);
                 q_s[t * N + c] = q.x * a.q_scale;
                 q_s[t * N + half + c] = q.y * a.q_scale;
@@ -187,7 +180,7 @@ __global__ void __launch_bounds__(kLcWarps * 32) lin_scan_kernel(const LinArgs a
         }
         for (int e = threadIdx.x; !kRet && e < nt * N; e += blockDim.x) {
             const int t = e / N, n = e - t * N;
-            const int64_t at = (row + t) * a.ld + h * N + n;
+            const int64_t at = (row + t) * a.ld_qk + h * N + n;
             k_s[e] = load_any<DT>(a.k, at) * a.k_scale;
             q_s[e] = load_any<DT>(a.q, at) * a.q_scale;
             d_s[e] = exp2f(lin_log2_decay<DT>(load_any<DT>(a.z, (row + t) * a.ld_z + h * N + n) + a.bias[h * N + n], a.inv_tau));
@@ -289,7 +282,7 @@ extern "C" int hds_linear_attention(const void* q, const void* k, const void* v,
     *finished = 1;
     if (T == 0 || n_seqs == 0) return HDS_OK;
     LinArgs a{q, k, v, gate, ld, z, ld_z, bias, inv_tau, state, reinterpret_cast<const SsmSpan*>(spans), n_seqs, T, heads, vdim, dim,
-              y, ld_y, out, ld_out, norm_w, eps, 0, vdim, 1.0f / sqrtf(static_cast<float>(dim)), 1.0f, nullptr, nullptr, nullptr};
+              y, ld_y, out, ld_out, norm_w, eps, 0, vdim, 1.0f / sqrtf(static_cast<float>(dim)), 1.0f, ld, nullptr, nullptr, nullptr};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     const int n_multi = n_seqs - n_single;
     int rc = HDS_OK;

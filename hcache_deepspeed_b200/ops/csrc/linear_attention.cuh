@@ -5,7 +5,7 @@
 namespace hds {
 
 struct LinArgs {
-    const void* q;          // [T][ld]: heads * N columns each of q, k; heads * P of v, gate
+    const void* q;          // [T][ld_qk]: heads * N columns each of q, k; [T][ld]: heads * P of v, gate
     const void* k;
     const void* v;
     const void* gate;
@@ -21,14 +21,15 @@ struct LinArgs {
     int64_t ld_y;
     void* out;              // [T][ld_out], or nullptr: the state alone
     int64_t ld_out;
-    const float* norm_w;    // [heads * P]
+    const float* norm_w;    // [heads * P], or nullptr: ones
     float eps;
     int write_y;            // steps leave read-outs in y instead of finished rows in out
     int norm_cols;          // values of a head that its norm averages over
     float q_scale, k_scale;
-    // retention: a constant decay per head instead of z; q and k turned by position
+    int64_t ld_qk;              // of q and k
+    // retention: a constant decay per head instead of z; q and k are turned by position (freq nullptr: they have been)
     const float* log2_decay;    // [heads]
-    const float* freq;          // [N / 2]
+    const float* freq;          // [N / 2] or nullptr
     const float* amp;           // [N / 2] or nullptr
 };
 
@@ -38,7 +39,20 @@ __device__ __forceinline__ void lin_sincos(float x, float* s, float* c) {
     else rope_sincos(x, s, c);
 }
 
-// values c and N / 2 + c of a head's row, turned for position pos
+// sine and cosine of pair c at a position
+template <int DT>
+__device__ __forceinline__ void lin_turn(const LinArgs& a, float pos, int c, float* s, float* co) {
+    *s = 0.0f;
+    *co = 1.0f;
+    if (a.freq == nullptr) return;
+    lin_sincos<DT>(pos * a.freq[c], s, co);
+    if (a.amp != nullptr) {
+        *s *= a.amp[c];
+        *co *= a.amp[c];
+    }
+}
+
+// values c and N / 2 + c of a head's row, turned
 template <int DT>
 __device__ __forceinline__ float2 lin_turned(const LinArgs& a, const void* x, int64_t head_row, int c, float s, float co) {
     const float u = load_any<DT>(x, head_row + c), v = load_any<DT>(x, head_row + (a.N >> 1) + c);

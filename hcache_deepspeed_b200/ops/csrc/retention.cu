@@ -1,26 +1,26 @@
 // Retention over a ragged batch, per head:  S <- decay S + v k^T,  o = S q  (q and k turned by position), then o / rms(o) * silu(gate).
-// Sequences with one new token are stepped, and fp32 / fp16 models and odd sizes scanned, by the kernels of linear_attention.cu. Prompts of
-// bf16 models run here on tcgen05, 128 tokens at a time. With S the state in front of a chunk and d the head's decay:
+// Sequences with one new token are stepped, and batches whose q and k still have to be turned scanned, by the kernels of
+// linear_attention.cu. Prompts of bf16 models, whose projection has turned them already, run here on tcgen05, 128 tokens at a time. With S
+// the state in front of a chunk and d the head's decay:
 //
 //   o_i = d^(i + 1) S q_i + sum_{j <= i} d^(i - j) (q_i . k_j) v_j          S <- d^n S + sum_j d^(n - 1 - j) v_j k_j^T
 //
 //   ret_local : per (chunk, head): what the chunk's tokens add to the state. Independent of other chunks
 //   ret_chain : states in front of every chunk, in place of those sums; advances the state pool. A plain stream along the chunks
-//   ret_out   : per (chunk, head): scores, state and value products, norm and gate
+//   ret_out   : per (chunk, head): scores, state and value products, norm and gate. Persistent blocks
 //
-// v enters products exactly as it is. Everything fp32 that becomes an operand (turned q and k, decayed keys and scores, the state) is a bf16
-// value plus the bf16 rest, 16 significant bits; sums are fp32 in TMEM, the carried state is never rounded. A thread turns runs of
-// consecutive tokens: one sine and cosine of its first position, then a step by the pair's own angle per token (runs of 64 at most).
-// The sums are [P][N] rows of 32-byte groups (8 values); a state takes their place as 8 leading terms and 8 rests, the 16-byte pieces of
-// swizzled operand rows. Long batches run in segments, which bounds the workspace.
+// q, k and v enter products exactly as they are. Everything fp32 that becomes an operand (decayed values, decayed scores, the state) is a bf16
+// value plus the bf16 rest, 16 significant bits; sums are fp32 in TMEM, the carried state is never rounded. Sums are [P][N] rows; a state
+// takes a row's place as N leading terms and N rests, which TMA reads as two tiles. Long batches run in segments, which bounds the workspace.
 #include "linear_attention.cuh"
 #include "../../../include/hds_b200.h"
 
 namespace hds {
 
 constexpr int kRtTok = 128, kRtThreads = 256, kRtP = 128, kRtPanel = kRtTok * 128;       // a panel: 128 rows of 128 bytes
+constexpr uint64_t kRtRows16 = (16 * 128) >> 4;     // 16 rows of a panel, in descriptor units
 
-//: set when a wait ran out (a fault of the kernel's own protocol); read by hds_retention_status
+//: set when a wait ran out (a fault of the kernels' own protocol); read by hds_retention_status
 __device__ int g_ret_stuck = 0;
 
 // Wait for a phase; gives up after about a second, records it and never waits again.
@@ -40,146 +40,90 @@ __device__ __forceinline__ float rt_ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+__device__ __forceinline__ float rt_rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rt_silu(float g) { return g * rt_rcp(1.0f + rt_ex2(g * -1.4426950408889634f)); }
 __device__ __forceinline__ void rt_split(float v0, float v1, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(v0, v1);
     lo = pack_bf16(v0 - bf16_lo(hi), v1 - bf16_hi(hi));
 }
-// byte of column c (of 64-column panels) in row r of a 128-byte-swizzled tile
-__device__ __forceinline__ uint32_t rt_byte(int r, int c) {
-    return static_cast<uint32_t>((c >> 6) * kRtPanel + r * 128 + ((((c & 63) >> 3) ^ (r & 7)) << 4) + (c & 7) * 2);
-}
-__device__ __forceinline__ void rt_copy16(void* dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-
-// Which tokens and columns a thread turns: columns c, c + 1 and their partners half a row behind, tokens t0 .. t0 + run - 1.
-struct RtPlace {
-    int c, t0, run;
-};
-__device__ __forceinline__ RtPlace rt_place(int N) {
-    const int lanes = N >> 2, runs = kRtThreads / lanes, run = (kRtTok + runs - 1) / runs, u = threadIdx.x / lanes;
-    RtPlace p;
-    p.c = (threadIdx.x - u * lanes) * 2;
-    p.t0 = u < runs ? u * run : kRtTok;
-    p.run = run;
-    return p;
-}
-
-// Rows of q or k of one head (fp32 once turned) -> two operand tiles. weight(t): factor of token t. Tokens from n on are zeros.
-// RUN: tokens per run where that is known (8 loads in flight at a time otherwise).
-template <int RUN, typename F>
-__device__ __forceinline__ void rt_turn(const LinArgs& a, const void* x, int64_t row, int64_t head_col, int N, int n, float pos0, uint8_t* hi_t,
-                                        uint8_t* lo_t, F weight) {
-    const RtPlace p = rt_place(N);
-    if (p.t0 >= kRtTok) return;
-    const int half = N >> 1;
-    const char* src = static_cast<const char*>(x) + ((row + p.t0) * a.ld + head_col + p.c) * 2;
-    float s0, c0, s1, c1, fs0, fc0, fs1, fc1;
-    const float f0 = a.freq[p.c], f1 = a.freq[p.c + 1];
-    rope_sincos((pos0 + p.t0) * f0, &s0, &c0);
-    rope_sincos((pos0 + p.t0) * f1, &s1, &c1);
-    rope_sincos(f0, &fs0, &fc0);
-    rope_sincos(f1, &fs1, &fc1);
-    if (a.amp != nullptr) {
-        s0 *= a.amp[p.c]; c0 *= a.amp[p.c];
-        s1 *= a.amp[p.c + 1]; c1 *= a.amp[p.c + 1];
-    }
-    constexpr int U = RUN > 0 ? RUN : 8;
-    for (int b = 0; b < (RUN > 0 ? RUN : p.run); b += U) {
-        uint32_t u[U], v[U];
-#pragma unroll
-        for (int i = 0; i < U; ++i) {
-            u[i] = v[i] = 0u;
-            if (b + i < p.run && p.t0 + b + i < n) {
-                const char* at = src + static_cast<int64_t>(b + i) * a.ld * 2;
-                u[i] = *reinterpret_cast<const uint32_t*>(at);
-                v[i] = *reinterpret_cast<const uint32_t*>(at + half * 2);
-            }
-        }
-#pragma unroll
-        for (int i = 0; i < U; ++i) {
-            const int t = p.t0 + b + i;
-            if (b + i >= p.run || t >= kRtTok) break;
-            const float w = weight(t);
-            const float x0 = bf16_lo(u[i]), x1 = bf16_hi(u[i]), y0 = bf16_lo(v[i]), y1 = bf16_hi(v[i]);
-            uint32_t hi, lo;
-            rt_split(w * (x0 * c0 - y0 * s0), w * (x1 * c1 - y1 * s1), hi, lo);
-            uint32_t at = rt_byte(t, p.c);
-            *reinterpret_cast<uint32_t*>(hi_t + at) = hi;
-            *reinterpret_cast<uint32_t*>(lo_t + at) = lo;
-            rt_split(w * (y0 * c0 + x0 * s0), w * (y1 * c1 + x1 * s1), hi, lo);
-            at = rt_byte(t, p.c + half);
-            *reinterpret_cast<uint32_t*>(hi_t + at) = hi;
-            *reinterpret_cast<uint32_t*>(lo_t + at) = lo;
-            const float n0 = c0 * fc0 - s0 * fs0, n1 = c1 * fc1 - s1 * fs1;
-            s0 = s0 * fc0 + c0 * fs0;
-            s1 = s1 * fc1 + c1 * fs1;
-            c0 = n0;
-            c1 = n1;
-        }
-    }
-}
+// 16-byte piece c (8 values) of row r in a swizzled panel
+__device__ __forceinline__ uint4* rt_cell(uint8_t* panel, int r, int c) { return reinterpret_cast<uint4*>(panel + r * 128 + ((c ^ (r & 7)) << 4)); }
 
 struct RetWs {
     float* s;           // [chunks][heads][P][N]: sums, then states (see above)
     int c0, n;          // chunks [c0, c0 + n) of the batch
 };
+struct RetMaps {
+    CUtensorMap q, k, v, s;     // [T][heads * N] twice, [T][heads * P]; [cells * P][2 N] rows of states
+};
 
-__host__ __device__ constexpr int rt_panels(int cols) { return (cols + 63) / 64; }
-// k (two terms) and v
-__host__ __device__ constexpr size_t rt_local_smem(int N) { return static_cast<size_t>(2 * rt_panels(N) + 2) * kRtPanel + 1024; }
+// k; v, which its leading terms replace; its rests
+__host__ __device__ constexpr size_t rt_local_smem(int N) { return static_cast<size_t>(N / 64 + 4) * kRtPanel + 1024; }
 
-// NT: the number of key channels where it is known, 0: any
-template <int NT>
-__global__ void __launch_bounds__(kRtThreads, 2)
-ret_local_kernel(const __grid_constant__ CUtensorMap tmap_v, const LinArgs a, const RetWs ws) {
+template <int N>
+__global__ void __launch_bounds__(kRtThreads, 2) ret_local_kernel(const __grid_constant__ RetMaps maps, const LinArgs a, const RetWs ws) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ ChunkPlace place;
-    __shared__ uint64_t v_full, done;
+    __shared__ uint64_t full, done;
     __shared__ uint32_t tmem_slot;
     pdl_enter();
     if (!find_chunk(a.spans, a.n_seqs, kRtTok, ws.c0 + blockIdx.x, &place)) return;
-    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    const int N = NT > 0 ? NT : a.N, P = a.P, h = blockIdx.y, p0 = blockIdx.z * kRtP, Pb = min(kRtP, P - p0);
-    const int t0 = place.chunk * kRtTok, n = min(kRtTok, place.span.n - t0);
-    const int64_t row = place.span.row0 + t0;
-    uint8_t* k_hi = smem;
-    uint8_t* k_lo = k_hi + rt_panels(N) * kRtPanel;
-    uint8_t* v_sm = k_lo + rt_panels(N) * kRtPanel;
+    uint8_t* k_sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+    uint8_t* v_hi = k_sm + N / 64 * kRtPanel;
+    uint8_t* v_lo = v_hi + 2 * kRtPanel;
+    const int P = a.P, h = blockIdx.y, p0 = blockIdx.z * kRtP, Pb = min(kRtP, P - p0);
+    const int t0 = place.chunk * kRtTok, n = min(kRtTok, place.span.n - t0), row = place.span.row0 + t0, panels = (Pb + 63) >> 6;
     const uint32_t warp = warp_id(), lane = lane_id();
     bool stuck = false;
     if (threadIdx.x == 0) {
-        prefetch_tmap(&tmap_v);
-        mbar_init(&v_full, 1);
+        mbar_init(&full, 1);
         mbar_init(&done, 1);
         fence_barrier_init();
-        const int panels = rt_panels(Pb);
-        mbar_expect_tx(&v_full, panels * kRtPanel);
-        for (int p = 0; p < panels; ++p) tma_load_2d(v_sm + p * kRtPanel, &tmap_v, &v_full, h * P + p0 + p * 64, static_cast<int>(row), kEvictNormal);
+        mbar_expect_tx(&full, (N / 64 + panels) * kRtPanel);
+        for (int p = 0; p < panels; ++p) tma_load_2d(v_hi + p * kRtPanel, &maps.v, &full, h * P + p0 + p * 64, row, kEvictNormal);
+        for (int p = 0; p < N / 64; ++p) tma_load_2d(k_sm + p * kRtPanel, &maps.k, &full, h * N + p * 64, row, kEvictNormal);
     }
     if (warp == 1) {
         tmem_alloc<128>(&tmem_slot);
         tmem_relinquish();
     }
-    const float ld = a.log2_decay[h], last = static_cast<float>(n - 1);
-    rt_turn<NT == 128 ? 16 : NT == 64 ? 8 : 0>(a, a.k, row, static_cast<int64_t>(h) * N, N, n, static_cast<float>(place.span.seen + t0), k_hi, k_lo,
-                                               [&](int t) { return a.k_scale * rt_ex2(ld * fmaxf(last - t, 0.0f)); });
-    fence_proxy_async_smem();
+    const float ld = a.log2_decay[h];
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = tmem_slot;
+    rt_wait(&full, 0, stuck);
+    for (int e = threadIdx.x; e < kRtTok * panels * 8; e += kRtThreads) {       // values, each faded to the end of the chunk
+        const int t = e / (panels * 8), c = e - t * panels * 8;
+        uint8_t* hi_p = v_hi + (c >> 3) * kRtPanel;
+        uint4* at = rt_cell(hi_p, t, c & 7);
+        uint4 hi = make_uint4(0, 0, 0, 0), lo = hi;
+        if (t < n) {
+            const uint4 x = *at;
+            const float w = a.k_scale * rt_ex2(ld * static_cast<float>(n - 1 - t));
+            rt_split(w * bf16_lo(x.x), w * bf16_hi(x.x), hi.x, lo.x);
+            rt_split(w * bf16_lo(x.y), w * bf16_hi(x.y), hi.y, lo.y);
+            rt_split(w * bf16_lo(x.z), w * bf16_hi(x.z), hi.z, lo.z);
+            rt_split(w * bf16_lo(x.w), w * bf16_hi(x.w), hi.w, lo.w);
+        }
+        *at = hi;
+        *rt_cell(v_lo + (c >> 3) * kRtPanel, t, c & 7) = lo;
+    }
+    fence_proxy_async_smem();
+    __syncthreads();
     if (threadIdx.x == 0) {      // sums [P][N] = V^T K, both operands as they lie (tokens are rows)
-        rt_wait(&v_full, 0, stuck);
         tc_fence_after();
-        const uint32_t idesc = make_idesc_f16(128, N, true, true, true);
-        const uint64_t dv = make_desc_mnmajor_sw128(smem_u32(v_sm), kRtPanel);
-        constexpr uint64_t ROWS16 = (16 * 128) >> 4;
+        constexpr uint32_t idesc = make_idesc_f16(128, N, true, true, true);
+        const uint64_t dk = make_desc_mnmajor_sw128(smem_u32(k_sm), kRtPanel);
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
-            const uint64_t dk = make_desc_mnmajor_sw128(smem_u32(t ? k_lo : k_hi), kRtPanel);
+            const uint64_t dv = make_desc_mnmajor_sw128(smem_u32(t ? v_lo : v_hi), kRtPanel);
 #pragma unroll
-            for (int kk = 0; kk < kRtTok / 16; ++kk) umma_f16_ss(tmem, dv + kk * ROWS16, dk + kk * ROWS16, idesc, (t > 0 || kk > 0) ? 1u : 0u);
+            for (int kk = 0; kk < kRtTok / 16; ++kk) umma_f16_ss(tmem, dv + kk * kRtRows16, dk + kk * kRtRows16, idesc, (t > 0 || kk > 0) ? 1u : 0u);
         }
         umma_commit(&done);
     }
@@ -189,7 +133,8 @@ ret_local_kernel(const __grid_constant__ CUtensorMap tmap_v, const LinArgs a, co
     tc_fence_after();
     const int quad = warp & 3, half = warp >> 2, p = quad * 32 + lane;
     float* out = ws.s + ((static_cast<int64_t>(blockIdx.x) * a.heads + h) * P + p0 + p) * N;
-    for (int b = half; b < N >> 4; b += 2) {
+#pragma unroll
+    for (int b = half; b < N / 16; b += 2) {
         uint32_t r[16];
         tmem_ld_32x16(tmem + (static_cast<uint32_t>(quad * 32) << 16) + b * 16, r);
         tmem_ld_wait();
@@ -211,292 +156,405 @@ ret_local_kernel(const __grid_constant__ CUtensorMap tmap_v, const LinArgs a, co
     }
 }
 
-// A thread keeps eight state values along the chunks of a sequence that lie in the segment; loads run ahead of the stores.
+// A thread keeps four values of a state row along the chunks of a sequence that lie in the segment; loads run ahead of the stores. A row
+// belongs to one warp (or half of one): its sums have all been read when its two terms take their place.
+template <int N>
 __global__ void __launch_bounds__(kRtThreads) ret_chain_kernel(const LinArgs a, const RetWs ws) {
     pdl_enter();
     const SsmSpan sp = a.spans[blockIdx.x];
     if (sp.n <= 1) return;
     const int total = span_chunks(sp, kRtTok), base = first_chunk(a.spans, blockIdx.x, kRtTok);
-    const int i0 = max(0, ws.c0 - base), i1 = min(total, ws.c0 + ws.n - base);
-    const int h = blockIdx.y, PN = a.P * a.N, e = (blockIdx.z * kRtThreads + threadIdx.x) * 8;
-    if (i0 >= i1 || e >= PN) return;
+    const int i0 = max(0, ws.c0 - base), n = min(total, ws.c0 + ws.n - base) - i0;
+    if (n <= 0) return;
+    const int h = blockIdx.y, PN = a.P * N, e = (blockIdx.z * kRtThreads + threadIdx.x) * 4;
+    const bool live = e < PN;       // (whole rows: a warp's idle lanes only keep its barrier)
+    const int row = e / N, c = e % N;
     float* st = a.state + (static_cast<int64_t>(sp.slot) * a.heads + h) * PN + e;
-    float4 S = make_float4(0.f, 0.f, 0.f, 0.f), R = S;
-    if (sp.seen > 0 || i0 > 0) {
-        S = *reinterpret_cast<const float4*>(st);
-        R = *reinterpret_cast<const float4*>(st + 4);
-    }
+    float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (live && (sp.seen > 0 || i0 > 0)) S = *reinterpret_cast<const float4*>(st);
     const float ld = a.log2_decay[h], keep = rt_ex2(ld * kRtTok), keep_last = rt_ex2(ld * (sp.n - (total - 1) * kRtTok));
     const int64_t step = static_cast<int64_t>(a.heads) * PN;
-    float* s = ws.s + (base + i0 - ws.c0) * step + static_cast<int64_t>(h) * PN + e;
+    float* cell = ws.s + (base + i0 - ws.c0) * step + static_cast<int64_t>(h) * PN + static_cast<int64_t>(row) * N;
+    const float* next = cell + c;
     constexpr int U = 4;
-    float4 x[U], y[U];
-    const float* sl = s;
-    auto load = [&](int j, bool live) {
-        if (!live) return;
-        x[j] = __ldcg(reinterpret_cast<const float4*>(sl));
-        y[j] = __ldcg(reinterpret_cast<const float4*>(sl + 4));
-        sl += step;
+    float4 x[U];
+    auto load = [&](int j, bool more) {
+        if (more && live) x[j] = __ldcg(reinterpret_cast<const float4*>(next));
+        next += step;
     };
-    const int n = i1 - i0;
 #pragma unroll
-    for (int j = 0; j < U; ++j) load(j, j < n);
+    for (int j = 0; j < U; ++j) {
+        x[j] = S;
+        load(j, j < n);
+    }
     for (int i = 0; i < n; i += U) {
 #pragma unroll
         for (int j = 0; j < U; ++j) {
             if (i + j >= n) break;
-            uint4 hi, lo;
+            uint2 hi, lo;
             rt_split(S.x, S.y, hi.x, lo.x);
             rt_split(S.z, S.w, hi.y, lo.y);
-            rt_split(R.x, R.y, hi.z, lo.z);
-            rt_split(R.z, R.w, hi.w, lo.w);
-            reinterpret_cast<uint4*>(s)[0] = hi;
-            reinterpret_cast<uint4*>(s)[1] = lo;
-            s += step;
             const float f = i0 + i + j == total - 1 ? keep_last : keep;
             S = make_float4(fmaf(f, S.x, x[j].x), fmaf(f, S.y, x[j].y), fmaf(f, S.z, x[j].z), fmaf(f, S.w, x[j].w));
-            R = make_float4(fmaf(f, R.x, y[j].x), fmaf(f, R.y, y[j].y), fmaf(f, R.z, y[j].z), fmaf(f, R.w, y[j].w));
+            asm volatile("" ::"f"(S.x), "f"(S.w) : "memory");
+            __syncwarp();
+            if (live) {
+                uint16_t* r = reinterpret_cast<uint16_t*>(cell) + c;
+                *reinterpret_cast<uint2*>(r) = hi;
+                *reinterpret_cast<uint2*>(r + N) = lo;
+            }
+            cell += step;
             load(j, i + j + U < n);
         }
     }
-    *reinterpret_cast<float4*>(st) = S;
-    *reinterpret_cast<float4*>(st + 4) = R;
+    if (live) *reinterpret_cast<float4*>(st) = S;
 }
 
-// q, k and the state (two terms each) and v. Up to 64 key channels two blocks share an SM: the state takes the place of the keys, once
-// those have been multiplied.
-__host__ __device__ constexpr bool rt_shares(int N) { return N <= 64; }
+// ret_out: warp 0 loads, warp 1 issues products, 16 warps form weights and outputs (a thread: a row and a quarter of its columns).
+// q and k have two buffers, v and the state one (two of each up to 64 channels); scores and outputs have two places in TMEM, so that the
+// products of one item run under the arithmetic of the other.
+constexpr int kRtOutWarps = 16, kRtOutThreads = 64 + kRtOutWarps * 32;
+__host__ __device__ constexpr int rt_stages(int N) { return N == 64 ? 2 : 1; }
 __host__ __device__ constexpr size_t rt_out_smem(int N) {
-    const int p = rt_panels(N);
-    return static_cast<size_t>((rt_shares(N) ? 4 : 6) * p + 2) * kRtPanel + 1024;
+    return static_cast<size_t>(2 * 2 * (N / 64) + rt_stages(N) * (2 + 2 * (N / 64))) * kRtPanel + 256 + 4 * kRtTok * 4;
 }
 
-template <int NT>
-__global__ void __launch_bounds__(kRtThreads, NT == 64 ? 2 : 1)
-ret_out_kernel(const __grid_constant__ CUtensorMap tmap_v, const LinArgs a, const RetWs ws) {
-    extern __shared__ uint8_t smem_raw[];
-    __shared__ ChunkPlace place;
-    __shared__ uint64_t v_full, s_done, y_done, o_done;
-    __shared__ uint32_t tmem_slot;
-    __shared__ float ss_s[2][kRtTok];
+struct RtItem {
+    int row, n, h, p0, Pb, cell;
+    bool fresh, valid;      // fresh: nothing in front, the state is zero
+};
+// Item number `index`: (chunk of the segment, head, block of values), by a whole warp.
+__device__ __forceinline__ RtItem rt_item(const LinArgs& a, const RetWs& ws, int index, int blocks) {
+    const int lane = threadIdx.x & 31, per = a.heads * blocks, local = index / per, rest = index - local * per;
+    const int target = ws.c0 + local;
+    int base = 0, seq = -1, chunk = 0;
+    for (int s0 = 0; s0 < a.n_seqs && seq < 0; s0 += 32) {
+        const int s = s0 + lane, mine = s < a.n_seqs ? span_chunks(a.spans[s], kRtTok) : 0;
+        int incl = mine;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int up = __shfl_up_sync(0xffffffffu, incl, o);
+            if (lane >= o) incl += up;
+        }
+        const unsigned hit = __ballot_sync(0xffffffffu, target < base + incl);
+        if (hit) {
+            const int l = __ffs(hit) - 1;
+            seq = s0 + l;
+            chunk = target - base - __shfl_sync(0xffffffffu, incl - mine, l);
+        }
+        base += __shfl_sync(0xffffffffu, incl, 31);
+    }
+    RtItem it;
+    it.valid = seq >= 0;
+    const SsmSpan sp = a.spans[max(seq, 0)];
+    it.row = sp.row0 + chunk * kRtTok;
+    it.n = min(kRtTok, sp.n - chunk * kRtTok);
+    it.fresh = sp.seen == 0 && chunk == 0;
+    it.h = rest / blocks;
+    it.p0 = (rest - it.h * blocks) * kRtP;
+    it.Pb = min(kRtP, a.P - it.p0);
+    it.cell = local * a.heads + it.h;
+    return it;
+}
+
+template <int N>
+__global__ void __launch_bounds__(kRtOutThreads, 1)
+ret_out_kernel(const __grid_constant__ RetMaps maps, const LinArgs a, const RetWs ws, const int items, const int blocks) {
+    constexpr int KP = N / 64, VS = rt_stages(N);
+    extern __shared__ __align__(1024) uint8_t smem[];       // (no room for alignment slack: the tiles need 1024-byte bases)
     pdl_enter();
-    if (!find_chunk(a.spans, a.n_seqs, kRtTok, ws.c0 + blockIdx.x, &place)) return;
-    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    const int N = NT > 0 ? NT : a.N, P = a.P, h = blockIdx.y, p0 = blockIdx.z * kRtP, Pb = min(kRtP, P - p0);
-    const int t0 = place.chunk * kRtTok, n = min(kRtTok, place.span.n - t0);
-    const int64_t row = place.span.row0 + t0;
-    const int tile = rt_panels(N) * kRtPanel;
-    uint8_t* q_hi = smem;
-    uint8_t* q_lo = q_hi + tile;
-    uint8_t* k_hi = q_lo + tile;
-    uint8_t* k_lo = k_hi + tile;
-    uint8_t* s_hi = rt_shares(N) ? k_hi : k_lo + tile;
-    uint8_t* s_lo = s_hi + tile;
-    uint8_t* v_sm = s_lo + tile;
+    uint8_t* qk_sm = smem;                                  // [2][q, k]
+    uint8_t* v_sm = qk_sm + 4 * KP * kRtPanel;              // [VS][2 panels]
+    uint8_t* s_sm = v_sm + VS * 2 * kRtPanel;               // [VS][leading terms, rests]
+    uint64_t* bars = reinterpret_cast<uint64_t*>(s_sm + VS * 2 * KP * kRtPanel);     // two of each
+    uint64_t *qk_full = bars, *qk_free = bars + 2, *v_full = bars + 4, *v_free = bars + 6, *s_full = bars + 8, *s_free = bars + 10,
+             *sc_done = bars + 12, *y_done = bars + 14, *o_done = bars + 16, *a_full = bars + 18, *t_free = bars + 20;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 22);
+    float* ss_s = reinterpret_cast<float*>(bars + 32);      // [4][128]
     const uint32_t warp = warp_id(), lane = lane_id();
-    const bool fresh = place.span.seen == 0 && place.chunk == 0;        // (nothing in front: the state is zero)
-    bool stuck = false;
+    if ((smem_u32(smem) & 1023u) != 0u) {
+        g_ret_stuck = 2;
+        return;
+    }
     if (threadIdx.x == 0) {
-        prefetch_tmap(&tmap_v);
-        mbar_init(&v_full, 1);
-        mbar_init(&s_done, 1);
-        mbar_init(&y_done, 1);
-        mbar_init(&o_done, 1);
+        for (int i = 0; i < 18; ++i) mbar_init(bars + i, 1);
+        for (int i = 18; i < 22; ++i) mbar_init(bars + i, kRtOutWarps);
         fence_barrier_init();
-        const int panels = rt_panels(Pb);
-        mbar_expect_tx(&v_full, panels * kRtPanel);
-        for (int p = 0; p < panels; ++p) tma_load_2d(v_sm + p * kRtPanel, &tmap_v, &v_full, h * P + p0 + p * 64, static_cast<int>(row), kEvictNormal);
     }
     if (warp == 1) {
-        tmem_alloc<256>(&tmem_slot);
+        tmem_alloc<512>(tmem_slot);
         tmem_relinquish();
     }
-    auto fetch_state = [&]() {
-        const char* src = reinterpret_cast<const char*>(ws.s + ((static_cast<int64_t>(blockIdx.x) * a.heads + h) * P + p0) * N);
-        const int groups = N >> 3;
-        for (int e = threadIdx.x; e < Pb * groups; e += kRtThreads) {
-            const int r = e / groups, at = rt_byte(r, (e - r * groups) * 8);
-            rt_copy16(s_hi + at, src + static_cast<int64_t>(e) * 32);
-            rt_copy16(s_lo + at, src + static_cast<int64_t>(e) * 32 + 16);
-        }
-    };
-    if (!fresh && !rt_shares(N)) fetch_state();
-    const float ld = a.log2_decay[h], pos0 = static_cast<float>(place.span.seen + t0);
-    constexpr int RUN = NT == 128 ? 16 : NT == 64 ? 8 : 0;
-    rt_turn<RUN>(a, a.k, row, static_cast<int64_t>(h) * N, N, n, pos0, k_hi, k_lo, [&](int) { return a.k_scale; });
-    rt_turn<RUN>(a, a.q, row, static_cast<int64_t>(h) * N, N, n, pos0, q_hi, q_lo, [&](int) { return 1.0f; });
-    if (!rt_shares(N)) asm volatile("cp.async.wait_all;" ::: "memory");
-    fence_proxy_async_smem();
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
-    const uint32_t t_a = tmem_slot, t_y = t_a + 128;        // scores, then their two terms (per 16 tokens: 8 columns each); output
-    constexpr uint64_t PANEL = kRtPanel >> 4, ROWS16 = (16 * 128) >> 4;
-    // the three products of two operands of two terms each that matter
-    auto three = [&](uint32_t d, const uint8_t* x_hi, const uint8_t* x_lo, const uint8_t* y_hi, const uint8_t* y_lo, uint32_t idesc) {
-        const uint64_t dx[2] = {make_desc_kmajor_sw128(smem_u32(x_hi)), make_desc_kmajor_sw128(smem_u32(x_lo))};
-        const uint64_t dy[2] = {make_desc_kmajor_sw128(smem_u32(y_hi)), make_desc_kmajor_sw128(smem_u32(y_lo))};
-#pragma unroll
-        for (int t = 0; t < 3; ++t)
-#pragma unroll
-            for (int kk = 0; kk < 8; ++kk)
-                if (kk < N >> 4) {
-                    const uint64_t at = (kk >> 2) * PANEL + 2 * (kk & 3);
-                    umma_f16_ss(d, dx[t == 2] + at, dy[t == 1] + at, idesc, (t > 0 || kk > 0) ? 1u : 0u);
-                }
-    };
-    if (threadIdx.x == 0) {
-        three(t_a, q_hi, q_lo, k_hi, k_lo, make_idesc_f16(128, 128, true, false, false));
-        umma_commit(&s_done);
-        if (!fresh && !rt_shares(N)) {
-            three(t_y, q_hi, q_lo, s_hi, s_lo, make_idesc_f16(128, Pb, true, false, false));
-            umma_commit(&y_done);
-        }
-    }
-    __syncwarp();
-    const int quad = warp & 3, half = warp >> 2, r = quad * 32 + lane;
-    const uint32_t la = static_cast<uint32_t>(quad * 32) << 16;
-    rt_wait(&s_done, 0, stuck);
-    __syncwarp();
-    tc_fence_after();
-    if (!fresh && rt_shares(N)) {
-        fetch_state();
-        asm volatile("cp.async.wait_all;" ::: "memory");
-        fence_proxy_async_smem();
-        __syncthreads();
-        if (threadIdx.x == 0) {
-            three(t_y, q_hi, q_lo, s_hi, s_lo, make_idesc_f16(128, Pb, true, false, false));
-            umma_commit(&y_done);
-        }
-        __syncwarp();
-    }
-    // ---- scores, decayed, in place: 16 fp32 columns become 8 of leading terms and 8 of rests ----
-    const float d = rt_ex2(ld);
-#pragma unroll 1
-    for (int part = 0; part < 4; ++part) {
-        const int j0 = half * 64 + part * 16;
-        uint32_t m[16];
-        if (j0 > quad * 32 + 31) {          // every column lies in the future
-#pragma unroll
-            for (int j = 0; j < 16; ++j) m[j] = 0u;
-        } else {
-            uint32_t x[16];
-            tmem_ld_32x16(t_a + la + j0, x);
-            tmem_ld_wait();
-            float v[16];
-            if (j0 + 15 > quad * 32) {      // the diagonal
-#pragma unroll
-                for (int j = 0; j < 16; ++j) {
-                    const int back = r - j0 - j;
-                    v[j] = back < 0 ? 0.0f : __uint_as_float(x[j]) * rt_ex2(ld * back);
-                }
-            } else {
-                float f = rt_ex2(ld * (r - j0 - 15));
-#pragma unroll
-                for (int j = 15; j >= 0; --j) {
-                    v[j] = __uint_as_float(x[j]) * f;
-                    f *= d;
+    const uint32_t tmem = *tmem_slot;       // twice: scores, then their two terms (per 16 tokens: 8 columns each); output
+    bool stuck = false;
+    const int stride = gridDim.x;
+
+    if (warp == 0) {
+        const bool leader = elect_one();
+        int i = 0, si = 0;      // items; items with a state
+        auto load_qk = [&](const RtItem& it, int k) {
+            if (k > 1) rt_wait(qk_free + (k & 1), ((k >> 1) - 1) & 1, stuck);
+            if (leader) {
+                uint8_t* q = qk_sm + (k & 1) * 2 * KP * kRtPanel;
+                mbar_expect_tx(qk_full + (k & 1), 2 * KP * kRtPanel);
+                for (int p = 0; p < KP; ++p) {
+                    tma_load_2d(q + p * kRtPanel, &maps.q, qk_full + (k & 1), it.h * N + p * 64, it.row, kEvictNormal);
+                    tma_load_2d(q + (KP + p) * kRtPanel, &maps.k, qk_full + (k & 1), it.h * N + p * 64, it.row, kEvictNormal);
                 }
             }
-#pragma unroll
-            for (int j = 0; j < 8; ++j) rt_split(v[2 * j], v[2 * j + 1], m[j], m[8 + j]);
+            __syncwarp();
+        };
+        RtItem it, next;
+        next.valid = false;
+        int at = blockIdx.x;
+        if (at < items) next = rt_item(a, ws, at, blocks);
+        if (next.valid) load_qk(next, 0);
+        while (next.valid) {
+            it = next;
+            at += stride;
+            next.valid = false;
+            if (at < items) next = rt_item(a, ws, at, blocks);
+            if (next.valid) load_qk(next, i + 1);
+            if (!it.fresh) {
+                const int b = si % VS;
+                if (si >= VS) rt_wait(s_free + b, (si / VS - 1) & 1, stuck);
+                if (leader) {
+                    uint8_t* s = s_sm + b * 2 * KP * kRtPanel;
+                    // (a box of 128 rows: where the head's block has fewer, the rest are the next head's and are not used)
+                    mbar_expect_tx(s_full + b, 2 * KP * kRtPanel);
+                    for (int p = 0; p < 2 * KP; ++p)
+                        tma_load_2d(s + p * kRtPanel, &maps.s, s_full + b, p * 64, it.cell * a.P + it.p0, kEvictFirst);
+                }
+                __syncwarp();
+                ++si;
+            }
+            const int b = i % VS, panels = (it.Pb + 63) >> 6;
+            if (i >= VS) rt_wait(v_free + b, (i / VS - 1) & 1, stuck);
+            if (leader) {
+                mbar_expect_tx(v_full + b, panels * kRtPanel);
+                for (int p = 0; p < panels; ++p)
+                    tma_load_2d(v_sm + (2 * b + p) * kRtPanel, &maps.v, v_full + b, it.h * a.P + it.p0 + p * 64, it.row, kEvictNormal);
+            }
+            __syncwarp();
+            ++i;
         }
-        tmem_st_32x16(t_a + la + j0, m);
-    }
-    // ---- what the state gives, decayed, in place; the scores' product adds to it ----
-    const int blocks = Pb >> 4;
-    if (!fresh) {
-        rt_wait(&y_done, 0, stuck);
-        __syncwarp();
-        tc_fence_after();
-        const float g = rt_ex2(ld * (r + 1));
+    } else if (warp == 1) {
+        const bool leader = elect_one();
+        constexpr uint64_t PANEL = kRtPanel >> 4;
+        constexpr uint32_t IDESC_QK = make_idesc_f16(128, 128, true, false, false);
+        const uint64_t d_qk = make_desc_kmajor_sw128(smem_u32(qk_sm)), d_s = make_desc_kmajor_sw128(smem_u32(s_sm)),
+                       d_v = make_desc_mnmajor_sw128(smem_u32(v_sm), kRtPanel);
+        int i = 0, si = 0;
+        bool prev_fresh = false;
+        int prev_pb = 0;
+        auto values = [&](int k, bool fresh, int pb) {     // output += weights of item k times its values
+            const int b = k & 1, vb = k % VS;
+            rt_wait(v_full + vb, (k / VS) & 1, stuck);
+            rt_wait(a_full + b, (k >> 1) & 1, stuck);
+            tc_fence_after();
+            const uint32_t t_a = tmem + b * 256;
+            const uint32_t idesc = make_idesc_f16(128, pb, true, false, true);
+            if (leader) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int b = half + 2 * i;
-            if (b >= blocks) break;
-            uint32_t x[16];
-            tmem_ld_32x16(t_y + la + b * 16, x);
-            tmem_ld_wait();
+                for (int t = 0; t < 2; ++t)
 #pragma unroll
-            for (int j = 0; j < 16; ++j) x[j] = __float_as_uint(__uint_as_float(x[j]) * g);
-            tmem_st_32x16(t_y + la + b * 16, x);
+                    for (int kk = 0; kk < kRtTok / 16; ++kk)
+                        umma_f16_ts(t_a + 128, t_a + kk * 16 + t * 8, d_v + 2 * vb * PANEL + kk * kRtRows16, idesc, (!fresh || t > 0 || kk > 0) ? 1u : 0u);
+                umma_commit(o_done + b);
+                umma_commit(v_free + vb);
+            }
+            __syncwarp();
+        };
+        for (int at = blockIdx.x; at < items; at += stride) {
+            const RtItem it = rt_item(a, ws, at, blocks);
+            if (!it.valid) break;
+            const int b = i & 1;
+            const uint32_t t_a = tmem + b * 256;
+            const uint64_t dq = d_qk + b * 2 * KP * PANEL, dk = dq + KP * PANEL;
+            rt_wait(qk_full + b, (i >> 1) & 1, stuck);
+            if (i > 1) rt_wait(t_free + b, ((i >> 1) - 1) & 1, stuck);       // (its output has been read)
+            tc_fence_after();
+            if (leader) {
+#pragma unroll
+                for (int kk = 0; kk < N / 16; ++kk) {
+                    const uint64_t o = (kk >> 2) * PANEL + 2 * (kk & 3);
+                    umma_f16_ss(t_a, dq + o, dk + o, IDESC_QK, kk > 0 ? 1u : 0u);
+                }
+                umma_commit(sc_done + b);
+            }
+            __syncwarp();
+            if (!it.fresh) {
+                const int sb = si % VS;
+                rt_wait(s_full + sb, (si / VS) & 1, stuck);
+                tc_fence_after();
+                const uint32_t idesc = make_idesc_f16(128, it.Pb, true, false, false);
+                if (leader) {
+#pragma unroll
+                    for (int t = 0; t < 2; ++t)
+#pragma unroll
+                        for (int kk = 0; kk < N / 16; ++kk) {
+                            const uint64_t o = (kk >> 2) * PANEL + 2 * (kk & 3);
+                            umma_f16_ss(t_a + 128, dq + o, d_s + (2 * sb + t) * KP * PANEL + o, idesc, (t > 0 || kk > 0) ? 1u : 0u);
+                        }
+                    umma_commit(y_done + b);
+                    umma_commit(s_free + sb);
+                }
+                __syncwarp();
+                ++si;
+            }
+            if (leader) umma_commit(qk_free + b);
+            __syncwarp();
+            if (i > 0) values(i - 1, prev_fresh, prev_pb);
+            prev_fresh = it.fresh;
+            prev_pb = it.Pb;
+            ++i;
         }
+        if (i > 0) values(i - 1, prev_fresh, prev_pb);
+    } else {
+        const int quad = warp & 3, part0 = (warp - 2) >> 2, r = quad * 32 + lane;
+        const uint32_t la = static_cast<uint32_t>(quad * 32) << 16;
+        int i = 0, yc[2] = {0, 0};      // items; those with a state, by place
+        auto output = [&](const RtItem& it, int k) {
+            const int b = k & 1, n_blocks = it.Pb >> 4;
+            const bool live = r < it.n;
+            const uint32_t t_y = tmem + b * 256 + 128 + la;
+            const int64_t col = static_cast<int64_t>(it.h) * a.P + it.p0;
+            uint4 gate[2][2];
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                const int blk = part0 + 4 * x;
+                gate[x][0] = gate[x][1] = make_uint4(0, 0, 0, 0);
+                if (!a.write_y && live && blk < n_blocks) {
+                    const uint4* src = reinterpret_cast<const uint4*>(static_cast<const char*>(a.gate) + ((it.row + r) * a.ld + col + blk * 16) * 2);
+                    gate[x][0] = src[0];
+                    gate[x][1] = src[1];
+                }
+            }
+            rt_wait(o_done + b, (k >> 1) & 1, stuck);
+            __syncwarp();
+            tc_fence_after();
+            float o[2][16], ss = 0.0f;
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                const int blk = part0 + 4 * x;
+                uint32_t y[16];
+                if (blk < n_blocks) {
+                    tmem_ld_32x16(t_y + blk * 16, y);
+                    tmem_ld_wait();
+                }
+#pragma unroll
+                for (int j = 0; j < 16; ++j) {
+                    o[x][j] = blk < n_blocks ? __uint_as_float(y[j]) : 0.0f;
+                    ss = fmaf(o[x][j], o[x][j], ss);
+                }
+            }
+            tc_fence_before();
+            auto rows_sync = [&]() { asm volatile("bar.sync %0, 128;" ::"r"(1 + quad) : "memory"); };       // the four warps of these rows
+            rows_sync();        // (the sums of the item before have been read)
+            ss_s[part0 * kRtTok + r] = ss;
+            __syncwarp();
+            if (lane == 0) mbar_arrive(t_free + b);
+            rows_sync();
+            const float f = rsqrtf((ss_s[r] + ss_s[kRtTok + r] + ss_s[2 * kRtTok + r] + ss_s[3 * kRtTok + r]) / a.norm_cols + a.eps);
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                const int blk = part0 + 4 * x;
+                if (blk >= n_blocks || !live) continue;
+                if (a.write_y) {
+#pragma unroll
+                    for (int j = 0; j < 16; j += 4)
+                        *reinterpret_cast<float4*>(a.y + (it.row + r) * a.ld_y + col + blk * 16 + j) = make_float4(o[x][j], o[x][j + 1], o[x][j + 2], o[x][j + 3]);
+                    continue;
+                }
+                const uint32_t gw[8] = {gate[x][0].x, gate[x][0].y, gate[x][0].z, gate[x][0].w, gate[x][1].x, gate[x][1].y, gate[x][1].z, gate[x][1].w};
+                uint32_t res[8];
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                    res[j] = pack_bf16(o[x][2 * j] * f * rt_silu(bf16_lo(gw[j])), o[x][2 * j + 1] * f * rt_silu(bf16_hi(gw[j])));
+                char* dst = static_cast<char*>(a.out) + ((it.row + r) * a.ld_out + col + blk * 16) * 2;
+                st_v4(dst, make_uint4(res[0], res[1], res[2], res[3]));
+                st_v4(dst + 16, make_uint4(res[4], res[5], res[6], res[7]));
+            }
+        };
+        RtItem prev;
+        for (int at = blockIdx.x; at < items; at += stride) {
+            const RtItem it = rt_item(a, ws, at, blocks);
+            if (!it.valid) break;
+            const int b = i & 1;
+            const uint32_t t_a = tmem + b * 256 + la;
+            const float ld = a.log2_decay[it.h], d = rt_ex2(ld);
+            rt_wait(sc_done + b, (i >> 1) & 1, stuck);
+            __syncwarp();
+            tc_fence_after();
+            // ---- scores, decayed, in place: 16 fp32 columns become 8 of leading terms and 8 of rests ----
+#pragma unroll
+            for (int part = part0; part < 8; part += 4) {
+                const int j0 = part * 16;
+                uint32_t m[16];
+                if (j0 > quad * 32 + 31) {          // every column lies in the future
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) m[j] = 0u;
+                } else {
+                    uint32_t x[16];
+                    tmem_ld_32x16(t_a + j0, x);
+                    tmem_ld_wait();
+                    float v[16];
+                    if (j0 + 15 > quad * 32) {      // the diagonal
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) {
+                            const int back = r - j0 - j;
+                            v[j] = back < 0 ? 0.0f : __uint_as_float(x[j]) * (a.k_scale * rt_ex2(ld * static_cast<float>(back)));
+                        }
+                    } else {
+                        float f = a.k_scale * rt_ex2(ld * static_cast<float>(r - j0 - 15));
+#pragma unroll
+                        for (int j = 15; j >= 0; --j) {
+                            v[j] = __uint_as_float(x[j]) * f;
+                            f *= d;
+                        }
+                    }
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) rt_split(v[2 * j], v[2 * j + 1], m[j], m[8 + j]);
+                }
+                tmem_st_32x16(t_a + j0, m);
+            }
+            // ---- what the state gives, decayed, in place; the product with the values adds to it ----
+            if (!it.fresh) {
+                rt_wait(y_done + b, yc[b] & 1, stuck);
+                ++yc[b];
+                __syncwarp();
+                tc_fence_after();
+                const float g = rt_ex2(ld * static_cast<float>(r + 1));
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    const int blk = part0 + 4 * x;
+                    if (blk >= it.Pb >> 4) break;
+                    uint32_t y[16];
+                    tmem_ld_32x16(t_a + 128 + blk * 16, y);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) y[j] = __float_as_uint(__uint_as_float(y[j]) * g);
+                    tmem_st_32x16(t_a + 128 + blk * 16, y);
+                }
+            }
+            tmem_st_wait();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(a_full + b);
+            if (i > 0) output(prev, i - 1);
+            prev = it;
+            ++i;
+        }
+        if (i > 0) output(prev, i - 1);
     }
-    tmem_st_wait();
     tc_fence_before();
     __syncthreads();
-    if (threadIdx.x == 0) {
-        rt_wait(&v_full, 0, stuck);
-        tc_fence_after();
-        const uint32_t idesc = make_idesc_f16(128, Pb, true, false, true);
-        const uint64_t dv = make_desc_mnmajor_sw128(smem_u32(v_sm), kRtPanel);
-#pragma unroll
-        for (int t = 0; t < 2; ++t)
-#pragma unroll
-            for (int kk = 0; kk < kRtTok / 16; ++kk)
-                umma_f16_ts(t_y, t_a + kk * 16 + t * 8, dv + kk * ROWS16, idesc, (!fresh || t > 0 || kk > 0) ? 1u : 0u);
-        umma_commit(&o_done);
-    }
-    __syncwarp();
-    const bool live = r < n;
-    const int64_t col = static_cast<int64_t>(h) * P + p0;
-    uint4 gate[4][2];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        const int b = half + 2 * i;
-        gate[i][0] = gate[i][1] = make_uint4(0, 0, 0, 0);
-        if (!a.write_y && live && b < blocks) {
-            const uint4* src = reinterpret_cast<const uint4*>(static_cast<const char*>(a.gate) + ((row + r) * a.ld + col + b * 16) * 2);
-            gate[i][0] = src[0];
-            gate[i][1] = src[1];
-        }
-    }
-    rt_wait(&o_done, 0, stuck);
-    __syncwarp();
-    tc_fence_after();
-    float o[4][16], ss = 0.0f;
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        const int b = half + 2 * i;
-        if (b >= blocks) break;
-        uint32_t x[16];
-        tmem_ld_32x16(t_y + la + b * 16, x);
-        tmem_ld_wait();
-#pragma unroll
-        for (int j = 0; j < 16; ++j) {
-            o[i][j] = __uint_as_float(x[j]);
-            ss = fmaf(o[i][j], o[i][j], ss);
-        }
-    }
-    ss_s[half][r] = ss;
-    tc_fence_before();
-    __syncthreads();
-    const float f = rsqrtf((ss_s[0][r] + ss_s[1][r]) / a.norm_cols + a.eps);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        const int b = half + 2 * i;
-        if (b >= blocks || !live) break;
-        if (a.write_y) {
-#pragma unroll
-            for (int j = 0; j < 16; j += 4)
-                *reinterpret_cast<float4*>(a.y + (row + r) * a.ld_y + col + b * 16 + j) = make_float4(o[i][j], o[i][j + 1], o[i][j + 2], o[i][j + 3]);
-            continue;
-        }
-        const uint32_t* gw = reinterpret_cast<const uint32_t*>(gate[i]);
-        const float* w = a.norm_w + col + b * 16;
-        uint32_t res[8];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const float2 nw = *reinterpret_cast<const float2*>(w + 2 * j);
-            res[j] = pack_bf16(o[i][2 * j] * f * nw.x * ssm_silu<0>(bf16_lo(gw[j])), o[i][2 * j + 1] * f * nw.y * ssm_silu<0>(bf16_hi(gw[j])));
-        }
-        char* dst = static_cast<char*>(a.out) + ((row + r) * a.ld_out + col + b * 16) * 2;
-        st_v4(dst, make_uint4(res[0], res[1], res[2], res[3]));
-        st_v4(dst + 16, make_uint4(res[4], res[5], res[6], res[7]));
-    }
     if (warp == 1) {
         tc_fence_after();
-        tmem_dealloc<256>(t_a);
+        tmem_dealloc<512>(tmem);
     }
 }
 
@@ -510,41 +568,42 @@ static int64_t rt_segment(int64_t chunks, int heads, int P, int N) {
 
 static bool rt_chunk_supported(const LinArgs& a, int dtype, const void* ws, int64_t ws_bytes) {
     auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    return dtype == 0 && a.N % 16 == 0 && a.N <= 128 && a.P % 16 == 0 && ws != nullptr && ws_bytes >= rt_cell_bytes(a.heads, a.P, a.N) &&
+    return dtype == 0 && a.freq == nullptr && (a.N == 64 || a.N == 128) && a.P % 16 == 0 && ws != nullptr && ws_bytes >= rt_cell_bytes(a.heads, a.P, a.N) &&
            (reinterpret_cast<uintptr_t>(ws) & 31) == 0 && aligned(a.q) && aligned(a.k) && aligned(a.v) && aligned(a.gate) && aligned(a.out) &&
-           aligned(a.state) && aligned(a.y) && a.ld % 8 == 0 && a.ld_out % 8 == 0 && a.ld_y % 4 == 0;
+           aligned(a.state) && aligned(a.y) && a.ld % 8 == 0 && a.ld_qk % 8 == 0 && a.ld_out % 8 == 0 && a.ld_y % 4 == 0;
 }
 
-template <int NT>
-static int rt_chunk_launch_as(const LinArgs& a, const CUtensorMap& tv, int64_t bound, int step, void* ws, cudaStream_t s) {
-    auto local = ret_local_kernel<NT>;
-    auto out = ret_out_kernel<NT>;
-    HDS_CHECK_CUDA(cudaFuncSetAttribute(local, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(rt_local_smem(a.N))));
-    HDS_CHECK_CUDA(cudaFuncSetAttribute(out, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(rt_out_smem(a.N))));
+template <int N>
+static int rt_chunk_launch(const LinArgs& a, int n_multi, void* ws, int64_t ws_bytes, cudaStream_t s) {
+    const int64_t bound = a.T / kRtTok + n_multi;           // at least as many as there are chunks
+    const int64_t fits = ws_bytes / rt_cell_bytes(a.heads, a.P, N), seg = rt_segment(bound, a.heads, a.P, N);
+    const int step = static_cast<int>(seg < fits ? seg : fits);
+    RetMaps m;
+    const uint64_t T = static_cast<uint64_t>(a.T), keys = static_cast<uint64_t>(a.heads) * N, vals = static_cast<uint64_t>(a.heads) * a.P;
+    int rc = make_tmap_2d_16b(&m.q, a.q, keys, T, static_cast<uint64_t>(a.ld_qk) * 2, 64, kRtTok, true);
+    if (!rc) rc = make_tmap_2d_16b(&m.k, a.k, keys, T, static_cast<uint64_t>(a.ld_qk) * 2, 64, kRtTok, true);
+    if (!rc) rc = make_tmap_2d_16b(&m.v, a.v, vals, T, static_cast<uint64_t>(a.ld) * 2, 64, kRtTok, true);
+    if (!rc) rc = make_tmap_2d_16b(&m.s, ws, 2 * N, static_cast<uint64_t>(step) * vals, 4 * N, 64, kRtTok, true);
+    if (rc) return rc;
+    auto local = ret_local_kernel<N>;
+    auto chain = ret_chain_kernel<N>;
+    auto out = ret_out_kernel<N>;
+    HDS_CHECK_CUDA(cudaFuncSetAttribute(local, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(rt_local_smem(N))));
+    HDS_CHECK_CUDA(cudaFuncSetAttribute(out, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(rt_out_smem(N))));
     const unsigned blocks = (a.P + kRtP - 1) / kRtP;
     for (int64_t c0 = 0; c0 < bound; c0 += step) {
         RetWs w;
         w.s = static_cast<float*>(ws);
         w.c0 = static_cast<int>(c0);
         w.n = static_cast<int>(step < bound - c0 ? step : bound - c0);
-        const dim3 grid(w.n, a.heads, blocks), block(kRtThreads);
-        HDS_CHECK_CUDA(launch_kernel(local, grid, block, rt_local_smem(a.N), s, tv, a, w));
-        HDS_CHECK_CUDA(launch_kernel(ret_chain_kernel, dim3(a.n_seqs, a.heads, (a.P * a.N / 8 + kRtThreads - 1) / kRtThreads), block, 0, s, a, w));
-        if (a.out != nullptr || a.write_y) HDS_CHECK_CUDA(launch_kernel(out, grid, block, rt_out_smem(a.N), s, tv, a, w));
+        HDS_CHECK_CUDA(launch_kernel(local, dim3(w.n, a.heads, blocks), dim3(kRtThreads), rt_local_smem(N), s, m, a, w));
+        HDS_CHECK_CUDA(launch_kernel(chain, dim3(a.n_seqs, a.heads, (a.P * N / 4 + kRtThreads - 1) / kRtThreads), dim3(kRtThreads), 0, s, a, w));
+        if (a.out != nullptr || a.write_y) {
+            const int items = w.n * a.heads * static_cast<int>(blocks), sms = sm_count();
+            HDS_CHECK_CUDA(launch_kernel(out, dim3(items < sms ? items : sms), dim3(kRtOutThreads), rt_out_smem(N), s, m, a, w, items, static_cast<int>(blocks)));
+        }
     }
     return HDS_OK;
-}
-
-static int rt_chunk_launch(const LinArgs& a, int n_multi, void* ws, int64_t ws_bytes, cudaStream_t s) {
-    const int64_t bound = a.T / kRtTok + n_multi;           // at least as many as there are chunks
-    const int64_t fits = ws_bytes / rt_cell_bytes(a.heads, a.P, a.N), seg = rt_segment(bound, a.heads, a.P, a.N);
-    const int step = static_cast<int>(seg < fits ? seg : fits);
-    CUtensorMap tv;      // columns of all heads' values; a box that reaches past them reads zeros
-    const int rc = make_tmap_2d_16b(&tv, a.v, static_cast<uint64_t>(a.heads) * a.P, static_cast<uint64_t>(a.T), static_cast<uint64_t>(a.ld) * 2, 64, kRtTok, true);
-    if (rc) return rc;
-    return a.N == 128 ? rt_chunk_launch_as<128>(a, tv, bound, step, ws, s)
-           : a.N == 64 ? rt_chunk_launch_as<64>(a, tv, bound, step, ws, s)
-                       : rt_chunk_launch_as<0>(a, tv, bound, step, ws, s);
 }
 
 }  // namespace hds
@@ -552,7 +611,7 @@ static int rt_chunk_launch(const LinArgs& a, int n_multi, void* ws, int64_t ws_b
 using namespace hds;
 
 extern "C" int64_t hds_retention_workspace_bytes(int T, int n_seqs, int heads, int vdim, int dim) {
-    if (dim % 16 != 0 || dim > 128 || vdim % 16 != 0) return 0;
+    if ((dim != 64 && dim != 128) || vdim % 16 != 0) return 0;
     const int64_t all = T / kRtTok + (n_seqs < T / 2 ? n_seqs : T / 2);
     return rt_segment(all > 0 ? all : 1, heads, vdim, dim) * rt_cell_bytes(heads, vdim, dim);
 }
@@ -563,11 +622,10 @@ extern "C" int hds_retention_status(int* stuck) {
 }
 
 // Returns in *finished 1 when out holds the finished rows, 0 when y holds the read-outs (out still to be normed and gated).
-extern "C" int hds_retention(const void* q, const void* k, const void* v, const void* gate, int64_t ld, const float* log2_decay,
+extern "C" int hds_retention(const void* q, const void* k, int64_t ld_qk, const void* v, const void* gate, int64_t ld, const float* log2_decay,
                              const float* freq, const float* amp, float k_scale, int norm_cols, float* state, const int32_t* spans, int n_seqs,
-                             int n_single, int T, int heads, int vdim, int dim, float* y, int64_t ld_y, void* out, int64_t ld_out,
-                             const float* norm_w, float eps, void* workspace, int64_t workspace_bytes, int method, int* finished, int dtype,
-                             void* stream) {
+                             int n_single, int T, int heads, int vdim, int dim, float* y, int64_t ld_y, void* out, int64_t ld_out, float eps,
+                             void* workspace, int64_t workspace_bytes, int method, int* finished, int dtype, void* stream) {
     HDS_REQUIRE(dtype >= 0 && dtype <= 2, "hds_retention: dtype 0 bf16 / 1 fp16 / 2 fp32");
     HDS_REQUIRE(heads >= 1 && vdim >= 1 && vdim <= 8192 && dim >= 2 && dim <= 1024 && dim % 2 == 0, "hds_retention: heads of up to 1024 x 8192");
     HDS_REQUIRE(norm_cols >= 1 && norm_cols <= vdim, "hds_retention: 1 <= norm_cols <= vdim");
@@ -575,7 +633,7 @@ extern "C" int hds_retention(const void* q, const void* k, const void* v, const 
     *finished = 1;
     if (T == 0 || n_seqs == 0) return HDS_OK;
     LinArgs a{q, k, v, gate, ld, nullptr, 0, nullptr, 0.0f, state, reinterpret_cast<const SsmSpan*>(spans), n_seqs, T, heads, vdim, dim,
-              y, ld_y, out, ld_out, norm_w, eps, 0, norm_cols, 1.0f, k_scale, log2_decay, freq, amp};
+              y, ld_y, out, ld_out, nullptr, eps, 0, norm_cols, 1.0f, k_scale, ld_qk, log2_decay, freq, amp};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     int rc = HDS_OK;
     if (n_seqs > n_single) {
@@ -586,7 +644,8 @@ extern "C" int hds_retention(const void* q, const void* k, const void* v, const 
                 *finished = 0;
                 a.write_y = 1;
             }
-            rc = rt_chunk_launch(a, n_seqs - n_single, workspace, workspace_bytes, s);
+            rc = dim == 64 ? rt_chunk_launch<64>(a, n_seqs - n_single, workspace, workspace_bytes, s)
+                           : rt_chunk_launch<128>(a, n_seqs - n_single, workspace, workspace_bytes, s);
         } else {
             *finished = 0;
             a.write_y = 1;      // by every row of the batch: one norm finishes them all

@@ -901,24 +901,25 @@ def retention_workspace_bytes(n_tokens: int, n_seqs: int, heads: int, vdim: int,
     return int(native.cuda_lib().hds_retention_workspace_bytes(n_tokens, n_seqs, heads, vdim, dim))
 
 
-def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, log2_decay: torch.Tensor, freq: torch.Tensor,
+def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, log2_decay: torch.Tensor, freq: Optional[torch.Tensor],
               amp: Optional[torch.Tensor], k_scale: float, norm_cols: int, state: torch.Tensor, spans: torch.Tensor, n_single: int, y: torch.Tensor,
-              out: Optional[torch.Tensor], norm_w: torch.Tensor, eps: float, workspace: Optional[torch.Tensor] = None, method: int = SCAN_AUTO) -> None:
+              out: Optional[torch.Tensor], ones: torch.Tensor, eps: float, workspace: Optional[torch.Tensor] = None, method: int = SCAN_AUTO) -> None:
     """Retention over a ragged batch, with the norm and gate behind (``hds_retention``). ``state`` [slots, heads, vdim, dim] fp32; heads
-    hold ``norm_cols`` values and zeros; ``y`` fp32 scratch; ``out`` None: advance the state alone."""
+    hold ``norm_cols`` values and zeros; ``freq`` None: q and k have been turned; ``y`` fp32 scratch; ``out`` None: advance the state
+    alone; ``ones``: as many as a row of v has values."""
     T = q.shape[0]
     _, heads, vdim, dim = state.shape
-    assert q.stride(0) == k.stride(0) == v.stride(0) == gate.stride(0) and log2_decay.numel() == heads and freq.numel() == dim // 2
+    assert q.stride(0) == k.stride(0) and v.stride(0) == gate.stride(0) and log2_decay.numel() == heads and (freq is None or freq.numel() == dim // 2)
     done = ctypes.c_int(1)
-    rc = native.cuda_lib().hds_retention(_p(q), _p(k), _p(v), _p(gate), q.stride(0), _p(log2_decay), _p(freq), _p(amp), k_scale, norm_cols, _p(state),
-                                         _p(spans), spans.shape[0], n_single, T, heads, vdim, dim, _p(y), y.stride(0), _p(out),
-                                         0 if out is None else out.stride(0), _p(norm_w), eps, _p(workspace),
-                                         0 if workspace is None else workspace.numel(), method, ctypes.addressof(done), _dt3(q), _stream())
+    rc = native.cuda_lib().hds_retention(_p(q), _p(k), q.stride(0), _p(v), _p(gate), v.stride(0), _p(log2_decay), _p(freq), _p(amp), k_scale, norm_cols,
+                                         _p(state), _p(spans), spans.shape[0], n_single, T, heads, vdim, dim, _p(y), y.stride(0), _p(out),
+                                         0 if out is None else out.stride(0), eps, _p(workspace), 0 if workspace is None else workspace.numel(),
+                                         method, ctypes.addressof(done), _dt3(q), _stream())
     native.check(rc, "hds_retention")
     _count((3 if out is not None else 2) * (spans.shape[0] > n_single) + (n_single > 0))
     if out is not None and not done.value:
         r = vdim / norm_cols          # mean over a padded row * r = mean over the head
-        gated_norm(y[:, :heads * vdim], gate, norm_w, out, heads, eps / r, r**-0.5, gate_after=True)
+        gated_norm(y[:, :heads * vdim], gate, ones, out, heads, eps / r, r**-0.5, gate_after=True)
 
 
 def retention_stuck() -> bool:

@@ -58,7 +58,7 @@ def _declare_cuda(lib: ctypes.CDLL, partial: bool = False) -> None:
         "hds_mix_cached_values": [P, P, I, P, P, I, I, I, I, I, P],
         "hds_gru": [P, L, P, P, P, I, I, I, I, P, L, P, L, I, P],
         "hds_retention_status": [P],
-        "hds_retention": [P, P, P, P, L, P, P, P, F, I, P, P, I, I, I, I, I, I, P, L, P, L, P, F, P, L, I, P, I, P],
+        "hds_retention": [P, P, L, P, P, L, P, P, P, F, I, P, P, I, I, I, I, I, I, P, L, P, L, F, P, L, I, P, I, P],
         "hds_linear_attention": [P, P, P, P, L, P, L, P, F, P, P, I, I, I, I, I, I, P, L, P, L, P, F, P, L, I, P, I, P],
         "hds_gemm_next_act_limit": [F],
         "hds_moe_table_route": [P, P, I, I, I, I, P, P, P, P, P],

@@ -495,13 +495,14 @@ int hds_linear_attention(const void* q, const void* k, const void* v, const void
                          void* workspace, int64_t workspace_bytes, int method, int* finished, int dtype, void* stream);
 int64_t hds_linear_attention_workspace_bytes(int T, int n_seqs, int heads, int vdim, int dim);
 
-/* Retention over a ragged batch: as hds_linear_attention, but every head's state fades by a constant: S = 2^log2_decay[head] S + v k'^T,
- * y = S q'. q' and k' are q and k whose values c and dim / 2 + c of a head are turned by position * freq[c] and multiplied by amp[c]
- * (optional); k' also by k_scale. norm_cols: values of a head that its norm averages over (the others are zero padding). The chunked form
- * takes bf16, dim a multiple of 16 up to 128, vdim of 16. */
-int hds_retention(const void* q, const void* k, const void* v, const void* gate, int64_t ld, const float* log2_decay, const float* freq,
-                  const float* amp, float k_scale, int norm_cols, float* state, const int32_t* spans, int n_seqs, int n_single, int T, int heads,
-                  int vdim, int dim, float* y, int64_t ld_y, void* out, int64_t ld_out, const float* norm_w, float eps, void* workspace,
+/* Retention over a ragged batch: q, k [T, ld_qk] of heads * dim columns, v and gate [T, ld] of heads * vdim. As hds_linear_attention, but
+ * every head's state fades by a constant: S = 2^log2_decay[head] S + v k'^T, y = S q'. q' and k' are q and k whose values c and dim / 2 + c
+ * of a head are turned by position * freq[c] and multiplied by amp[c] (optional; freq NULL: they have been already, see hds_qkv_rope_proj);
+ * k' also by k_scale. norm_cols: values of a head that its norm averages over (the others are zero padding). The chunked form takes turned
+ * bf16 rows, dim 64 or 128, vdim a multiple of 16. */
+int hds_retention(const void* q, const void* k, int64_t ld_qk, const void* v, const void* gate, int64_t ld, const float* log2_decay,
+                  const float* freq, const float* amp, float k_scale, int norm_cols, float* state, const int32_t* spans, int n_seqs, int n_single,
+                  int T, int heads, int vdim, int dim, float* y, int64_t ld_y, void* out, int64_t ld_out, float eps, void* workspace,
                   int64_t workspace_bytes, int method, int* finished, int dtype, void* stream);
 int64_t hds_retention_workspace_bytes(int T, int n_seqs, int heads, int vdim, int dim);
 /* *stuck = 1 when a wait inside one of its kernels ever ran out of time (their results are then wrong). Synchronizes. */

@@ -268,7 +268,7 @@ def test_pages_and_state_of_each_layer():
     assert [None if c.get_cache(i) is None else tuple(c.get_cache(i).shape[1:]) for i in range(8)] == [
         None, (2, 2, 64, 64), None, None, (2, 4, 64, 128), None, None, None]
     assert [None if s.ssm(i) is None else tuple(s.ssm(i).shape[1:]) for i in range(8)] == [
-        (3, 32, 32), None, None, (2, 32, 48), None, None, (5, 48, 16), None]
+        (3, 32, 64), None, None, (2, 32, 64), None, None, (5, 48, 64), None]
 
 
 def test_errors_name_what_is_wrong():
@@ -297,7 +297,8 @@ def test_parameter_count_matches_the_checkpoint():
 
 def test_specs_of_one_layer():
     m = RetentionSpec(3, 7, 33, [0.5] * 3)
-    assert (m.width, m.vwidth, m.keys, m.inner, m.state) == (16, 48, 48, 144, 16)
+    assert (m.width, m.vwidth, m.keys, m.inner, m.state) == (64, 48, 192, 144, 64)
+    assert [RetentionSpec(1, d, 16, [0.5]).width for d in (64, 65, 128, 130)] == [64, 128, 128, 144]
     assert AttentionSpec(4, 2, 64, 64, 1.0, kv_from=0).cached_heads == 0 and AttentionSpec(4, 2, 64, 64, 1.0).cached_heads == 2
 
 
