@@ -5,19 +5,19 @@
 //
 //   o_i = d^(i + 1) S q_i + sum_{j <= i} d^(i - j) (q_i . k_j) v_j          S <- d^n S + sum_j d^(n - 1 - j) v_j k_j^T
 //
-//   ret_local : per (chunk, head): what the chunk's tokens add to the state. Independent of other chunks
-//   ret_chain : states in front of every chunk, in place of those sums; advances the state pool. A plain stream along the chunks
+//   ret_state : per (sequence, head, 32 values): walks the chunks with the state in TMEM and leaves the state in front of every chunk in the
+//               workspace; advances the state pool
 //   ret_out   : per (chunk, head): scores, state and value products, norm and gate. Persistent blocks
 //
 // q, k and v enter products exactly as they are. Everything fp32 that becomes an operand (decayed values, decayed scores, the state) is a bf16
-// value plus the bf16 rest, 16 significant bits; sums are fp32 in TMEM, the carried state is never rounded. Sums are [P][N] rows; a state
-// takes a row's place as N leading terms and N rests, which TMA reads as two tiles. Long batches run in segments, which bounds the workspace.
+// value plus the bf16 rest, 16 significant bits; sums are fp32 in TMEM, the carried state is never rounded. A state in the workspace is N rows
+// of P leading terms and P rests, which TMA reads as two tiles. Long batches run in segments, which bounds the workspace.
 #include "linear_attention.cuh"
 #include "../../../include/hds_b200.h"
 
 namespace hds {
 
-constexpr int kRtTok = 128, kRtThreads = 256, kRtP = 128, kRtPanel = kRtTok * 128;       // a panel: 128 rows of 128 bytes
+constexpr int kRtTok = 128, kRtP = 128, kRtPanel = kRtTok * 128;       // a panel: 128 rows of 128 bytes
 constexpr uint64_t kRtRows16 = (16 * 128) >> 4;     // 16 rows of a panel, in descriptor units
 
 //: set when a wait ran out (a fault of the kernels' own protocol); read by hds_retention_status
@@ -50,164 +50,193 @@ __device__ __forceinline__ void rt_split(float v0, float v1, uint32_t& hi, uint3
     hi = pack_bf16(v0, v1);
     lo = pack_bf16(v0 - bf16_lo(hi), v1 - bf16_hi(hi));
 }
+__device__ __forceinline__ void rt_store32(void* p, const uint32_t (&v)[8]) {
+    asm volatile("st.global.v8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(p), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]),
+                 "r"(v[5]), "r"(v[6]), "r"(v[7])
+                 : "memory");
+}
 // 16-byte piece c (8 values) of row r in a swizzled panel
 __device__ __forceinline__ uint4* rt_cell(uint8_t* panel, int r, int c) { return reinterpret_cast<uint4*>(panel + r * 128 + ((c ^ (r & 7)) << 4)); }
 
 struct RetWs {
-    float* s;           // [chunks][heads][P][N]: sums, then states (see above)
+    uint16_t* s;        // [chunks][heads][N][2 P]: states in front of the chunks (see above), or nullptr: not wanted
     int c0, n;          // chunks [c0, c0 + n) of the batch
 };
 struct RetMaps {
-    CUtensorMap q, k, v, s;     // [T][heads * N] twice, [T][heads * P]; [cells * P][2 N] rows of states
+    CUtensorMap q, k, v, s;     // [T][heads * N] twice, [T][heads * P]; [cells * N][2 P] rows of states
 };
 
-// k; v, which its leading terms replace; its rests
-__host__ __device__ constexpr size_t rt_local_smem(int N) { return static_cast<size_t>(N / 64 + 4) * kRtPanel + 1024; }
+// ret_state: warp 0 loads keys, warp 1 issues products, 8 warps keep the chain (a thread: a key channel of the state, half of the 32
+// columns), 8 warps decay values (a thread: a token, half of the columns), ahead of it. Between two products lies only the state's own
+// decay; the state in front of a chunk is written out while the chunk's product runs.
+constexpr int kRsP = 32, kRsThreads = 64 + 2 * 256, kRsStages = 4;
+__host__ __device__ constexpr size_t rt_state_smem(int N) { return static_cast<size_t>(kRsStages * (N / 64) + 2 * 2) * kRtPanel + 1024; }
 
 template <int N>
-__global__ void __launch_bounds__(kRtThreads, 2) ret_local_kernel(const __grid_constant__ RetMaps maps, const LinArgs a, const RetWs ws) {
+__global__ void __launch_bounds__(kRsThreads, 1) ret_state_kernel(const __grid_constant__ RetMaps maps, const LinArgs a, const RetWs ws) {
+    constexpr int KP = N / 64;
     extern __shared__ uint8_t smem_raw[];
-    __shared__ ChunkPlace place;
-    __shared__ uint64_t full, done;
+    __shared__ uint64_t k_full[kRsStages], k_free[kRsStages], w_full[2], w_free[2], s_ready, s_done;
     __shared__ uint32_t tmem_slot;
-    pdl_enter();
-    if (!find_chunk(a.spans, a.n_seqs, kRtTok, ws.c0 + blockIdx.x, &place)) return;
-    uint8_t* k_sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    uint8_t* v_hi = k_sm + N / 64 * kRtPanel;
-    uint8_t* v_lo = v_hi + 2 * kRtPanel;
-    const int P = a.P, h = blockIdx.y, p0 = blockIdx.z * kRtP, Pb = min(kRtP, P - p0);
-    const int t0 = place.chunk * kRtTok, n = min(kRtTok, place.span.n - t0), row = place.span.row0 + t0, panels = (Pb + 63) >> 6;
-    const uint32_t warp = warp_id(), lane = lane_id();
-    bool stuck = false;
-    if (threadIdx.x == 0) {
-        mbar_init(&full, 1);
-        mbar_init(&done, 1);
-        fence_barrier_init();
-        mbar_expect_tx(&full, (N / 64 + panels) * kRtPanel);
-        for (int p = 0; p < panels; ++p) tma_load_2d(v_hi + p * kRtPanel, &maps.v, &full, h * P + p0 + p * 64, row, kEvictNormal);
-        for (int p = 0; p < N / 64; ++p) tma_load_2d(k_sm + p * kRtPanel, &maps.k, &full, h * N + p * 64, row, kEvictNormal);
-    }
-    if (warp == 1) {
-        tmem_alloc<128>(&tmem_slot);
-        tmem_relinquish();
-    }
-    const float ld = a.log2_decay[h];
-    tc_fence_before();
-    __syncthreads();
-    tc_fence_after();
-    const uint32_t tmem = tmem_slot;
-    rt_wait(&full, 0, stuck);
-    for (int e = threadIdx.x; e < kRtTok * panels * 8; e += kRtThreads) {       // values, each faded to the end of the chunk
-        const int t = e / (panels * 8), c = e - t * panels * 8;
-        uint8_t* hi_p = v_hi + (c >> 3) * kRtPanel;
-        uint4* at = rt_cell(hi_p, t, c & 7);
-        uint4 hi = make_uint4(0, 0, 0, 0), lo = hi;
-        if (t < n) {
-            const uint4 x = *at;
-            const float w = a.k_scale * rt_ex2(ld * static_cast<float>(n - 1 - t));
-            rt_split(w * bf16_lo(x.x), w * bf16_hi(x.x), hi.x, lo.x);
-            rt_split(w * bf16_lo(x.y), w * bf16_hi(x.y), hi.y, lo.y);
-            rt_split(w * bf16_lo(x.z), w * bf16_hi(x.z), hi.z, lo.z);
-            rt_split(w * bf16_lo(x.w), w * bf16_hi(x.w), hi.w, lo.w);
-        }
-        *at = hi;
-        *rt_cell(v_lo + (c >> 3) * kRtPanel, t, c & 7) = lo;
-    }
-    fence_proxy_async_smem();
-    __syncthreads();
-    if (threadIdx.x == 0) {      // sums [P][N] = V^T K, both operands as they lie (tokens are rows)
-        tc_fence_after();
-        constexpr uint32_t idesc = make_idesc_f16(128, N, true, true, true);
-        const uint64_t dk = make_desc_mnmajor_sw128(smem_u32(k_sm), kRtPanel);
-#pragma unroll
-        for (int t = 0; t < 2; ++t) {
-            const uint64_t dv = make_desc_mnmajor_sw128(smem_u32(t ? v_lo : v_hi), kRtPanel);
-#pragma unroll
-            for (int kk = 0; kk < kRtTok / 16; ++kk) umma_f16_ss(tmem, dv + kk * kRtRows16, dk + kk * kRtRows16, idesc, (t > 0 || kk > 0) ? 1u : 0u);
-        }
-        umma_commit(&done);
-    }
-    __syncwarp();
-    rt_wait(&done, 0, stuck);
-    __syncwarp();
-    tc_fence_after();
-    const int quad = warp & 3, half = warp >> 2, p = quad * 32 + lane;
-    float* out = ws.s + ((static_cast<int64_t>(blockIdx.x) * a.heads + h) * P + p0 + p) * N;
-#pragma unroll
-    for (int b = half; b < N / 16; b += 2) {
-        uint32_t r[16];
-        tmem_ld_32x16(tmem + (static_cast<uint32_t>(quad * 32) << 16) + b * 16, r);
-        tmem_ld_wait();
-        if (p < Pb) {
-#pragma unroll
-            for (int g = 0; g < 2; ++g) {
-                float o[8];
-#pragma unroll
-                for (int j = 0; j < 8; ++j) o[j] = __uint_as_float(r[8 * g + j]);
-                st_v8_f32(out + b * 16 + g * 8, o);
-            }
-        }
-    }
-    tc_fence_before();
-    __syncthreads();
-    if (warp == 1) {
-        tc_fence_after();
-        tmem_dealloc<128>(tmem);
-    }
-}
-
-// A thread keeps four values of a state row along the chunks of a sequence that lie in the segment; loads run ahead of the stores. A row
-// belongs to one warp (or half of one): its sums have all been read when its two terms take their place.
-template <int N>
-__global__ void __launch_bounds__(kRtThreads) ret_chain_kernel(const LinArgs a, const RetWs ws) {
     pdl_enter();
     const SsmSpan sp = a.spans[blockIdx.x];
     if (sp.n <= 1) return;
     const int total = span_chunks(sp, kRtTok), base = first_chunk(a.spans, blockIdx.x, kRtTok);
-    const int i0 = max(0, ws.c0 - base), n = min(total, ws.c0 + ws.n - base) - i0;
-    if (n <= 0) return;
-    const int h = blockIdx.y, PN = a.P * N, e = (blockIdx.z * kRtThreads + threadIdx.x) * 4;
-    const bool live = e < PN;       // (whole rows: a warp's idle lanes only keep its barrier)
-    const int row = e / N, c = e % N;
-    float* st = a.state + (static_cast<int64_t>(sp.slot) * a.heads + h) * PN + e;
-    float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (live && (sp.seen > 0 || i0 > 0)) S = *reinterpret_cast<const float4*>(st);
-    const float ld = a.log2_decay[h], keep = rt_ex2(ld * kRtTok), keep_last = rt_ex2(ld * (sp.n - (total - 1) * kRtTok));
-    const int64_t step = static_cast<int64_t>(a.heads) * PN;
-    float* cell = ws.s + (base + i0 - ws.c0) * step + static_cast<int64_t>(h) * PN + static_cast<int64_t>(row) * N;
-    const float* next = cell + c;
-    constexpr int U = 4;
-    float4 x[U];
-    auto load = [&](int j, bool more) {
-        if (more && live) x[j] = __ldcg(reinterpret_cast<const float4*>(next));
-        next += step;
-    };
-#pragma unroll
-    for (int j = 0; j < U; ++j) {
-        x[j] = S;
-        load(j, j < n);
+    const int i0 = max(0, ws.c0 - base), n_chunks = min(total, ws.c0 + ws.n - base) - i0;       // those of the segment
+    if (n_chunks <= 0) return;
+    const int P = a.P, h = blockIdx.y, p0 = blockIdx.z * kRsP;
+    uint8_t* k_sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));     // [stages]
+    uint8_t* w_sm = k_sm + kRsStages * KP * kRtPanel;       // [2][leading terms, rests]: 32 of a panel's columns
+    const uint32_t warp = warp_id(), lane = lane_id();
+    bool stuck = false;
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < kRsStages; ++i) {
+            mbar_init(k_full + i, 1);
+            mbar_init(k_free + i, 1);
+        }
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(w_full + i, 8);
+            mbar_init(w_free + i, 1);
+        }
+        mbar_init(&s_ready, 8);
+        mbar_init(&s_done, 1);
+        fence_barrier_init();
     }
-    for (int i = 0; i < n; i += U) {
-#pragma unroll
-        for (int j = 0; j < U; ++j) {
-            if (i + j >= n) break;
-            uint2 hi, lo;
-            rt_split(S.x, S.y, hi.x, lo.x);
-            rt_split(S.z, S.w, hi.y, lo.y);
-            const float f = i0 + i + j == total - 1 ? keep_last : keep;
-            S = make_float4(fmaf(f, S.x, x[j].x), fmaf(f, S.y, x[j].y), fmaf(f, S.z, x[j].z), fmaf(f, S.w, x[j].w));
-            asm volatile("" ::"f"(S.x), "f"(S.w) : "memory");
-            __syncwarp();
-            if (live) {
-                uint16_t* r = reinterpret_cast<uint16_t*>(cell) + c;
-                *reinterpret_cast<uint2*>(r) = hi;
-                *reinterpret_cast<uint2*>(r + N) = lo;
+    if (warp == 1) {
+        tmem_alloc<32>(&tmem_slot);
+        tmem_relinquish();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = tmem_slot;
+    if (warp == 0) {
+        if (lane == 0) {
+            for (int c = 0; c < n_chunks; ++c) {
+                const int b = c % kRsStages;
+                if (c >= kRsStages) rt_wait(k_free + b, (c / kRsStages - 1) & 1, stuck);
+                mbar_expect_tx(k_full + b, KP * kRtPanel);
+                for (int p = 0; p < KP; ++p)
+                    tma_load_2d(k_sm + (b * KP + p) * kRtPanel, &maps.k, k_full + b, h * N + p * 64, sp.row0 + (i0 + c) * kRtTok, kEvictNormal);
             }
-            cell += step;
-            load(j, i + j + U < n);
+        }
+    } else if (warp == 1) {
+        const bool leader = elect_one();
+        constexpr uint32_t idesc = make_idesc_f16(128, kRsP, true, true, true);     // S [N][32] += K^T V, both operands as they lie (tokens are rows)
+        constexpr uint64_t PANEL = kRtPanel >> 4;
+        const uint64_t d_k = make_desc_mnmajor_sw128(smem_u32(k_sm), kRtPanel), d_w = make_desc_mnmajor_sw128(smem_u32(w_sm), kRtPanel);
+        for (int c = 0; c < n_chunks; ++c) {
+            const int b = c & 1, kb = c % kRsStages;
+            rt_wait(k_full + kb, (c / kRsStages) & 1, stuck);
+            rt_wait(w_full + b, (c >> 1) & 1, stuck);
+            rt_wait(&s_ready, c & 1, stuck);
+            tc_fence_after();
+            if (leader) {
+#pragma unroll
+                for (int t = 0; t < 2; ++t)
+#pragma unroll
+                    for (int kk = 0; kk < kRtTok / 16; ++kk)
+                        umma_f16_ss(tmem, d_k + kb * KP * PANEL + kk * kRtRows16, d_w + (2 * b + t) * PANEL + kk * kRtRows16, idesc, 1u);
+                umma_commit(&s_done);
+                umma_commit(w_free + b);
+                umma_commit(k_free + kb);
+            }
+            __syncwarp();
+        }
+    } else if (warp < 10) {
+        const int quad = warp & 3, half = (warp - 2) >> 2, r = quad * 32 + lane, p = p0 + half * 16;
+        const uint32_t t_s = tmem + (static_cast<uint32_t>(quad * 32) << 16) + half * 16;
+        const bool mine = r < N && p < P;       // (P is a multiple of 16)
+        const float ld = a.log2_decay[h];
+        float* st = a.state + ((static_cast<int64_t>(sp.slot) * a.heads + h) * P + p) * N + r;
+        uint32_t sw[16];
+        for (int c = 0; c < n_chunks; ++c) {
+            if (c == 0) {
+#pragma unroll
+                for (int j = 0; j < 16; ++j) sw[j] = __float_as_uint((sp.seen > 0 || i0 > 0) && mine ? st[static_cast<int64_t>(j) * N] : 0.0f);
+            } else {
+                rt_wait(&s_done, (c - 1) & 1, stuck);
+                __syncwarp();
+                tc_fence_after();
+                tmem_ld_32x16(t_s, sw);
+                tmem_ld_wait();
+            }
+            const float keep = rt_ex2(ld * static_cast<float>(min(kRtTok, sp.n - (i0 + c) * kRtTok)));
+            uint32_t sc[16];
+#pragma unroll
+            for (int j = 0; j < 16; ++j) sc[j] = __float_as_uint(__uint_as_float(sw[j]) * keep);
+            tmem_st_32x16(t_s, sc);
+            tmem_st_wait();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&s_ready);
+            if (ws.s != nullptr && mine) {
+                uint32_t hi[8], lo[8];
+#pragma unroll
+                for (int j = 0; j < 8; ++j) rt_split(__uint_as_float(sw[2 * j]), __uint_as_float(sw[2 * j + 1]), hi[j], lo[j]);
+                uint16_t* dst = ws.s + ((static_cast<int64_t>(base + i0 + c - ws.c0) * a.heads + h) * N + r) * 2 * P + p;
+                rt_store32(dst, hi);        // whole sectors
+                rt_store32(dst + P, lo);
+            }
+        }
+        rt_wait(&s_done, (n_chunks - 1) & 1, stuck);
+        __syncwarp();
+        tc_fence_after();
+        tmem_ld_32x16(t_s, sw);
+        tmem_ld_wait();
+        tc_fence_before();
+        if (mine)
+#pragma unroll
+            for (int j = 0; j < 16; ++j) st[static_cast<int64_t>(j) * N] = __uint_as_float(sw[j]);
+    } else {
+        const int quad = warp & 3, half = (warp - 10) >> 2, r = quad * 32 + lane, p = p0 + half * 16;
+        const float ld = a.log2_decay[h];
+        constexpr int U = 3;        // chunks whose values are on their way
+        uint4 x[U][2];
+        auto fetch = [&](int c, uint4 (&v)[2]) {       // this token's values
+            const int t = (i0 + c) * kRtTok + r;
+            v[0] = v[1] = make_uint4(0, 0, 0, 0);
+            if (c < n_chunks && t < sp.n && p < P) {
+                const uint4* src = reinterpret_cast<const uint4*>(static_cast<const char*>(a.v) +
+                                                                 (static_cast<int64_t>(sp.row0 + t) * a.ld + static_cast<int64_t>(h) * P + p) * 2);
+                v[0] = ld_nc_v4(src);
+                v[1] = ld_nc_v4(src + 1);
+            }
+        };
+#pragma unroll
+        for (int u = 0; u < U; ++u) fetch(u, x[u]);
+        for (int c0 = 0; c0 < n_chunks; c0 += U) {
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int c = c0 + u;
+                if (c >= n_chunks) break;
+                const int n = min(kRtTok, sp.n - (i0 + c) * kRtTok);
+                const float w = r < n ? a.k_scale * rt_ex2(ld * static_cast<float>(n - 1 - r)) : 0.0f;      // faded to the end of the chunk
+                uint8_t* hi_p = w_sm + (c & 1) * 2 * kRtPanel;
+                if (c > 1) rt_wait(w_free + (c & 1), ((c >> 1) - 1) & 1, stuck);
+#pragma unroll
+                for (int g = 0; g < 2; ++g) {
+                    const uint4 v = x[u][g];
+                    uint4 hi, lo;
+                    rt_split(w * bf16_lo(v.x), w * bf16_hi(v.x), hi.x, lo.x);
+                    rt_split(w * bf16_lo(v.y), w * bf16_hi(v.y), hi.y, lo.y);
+                    rt_split(w * bf16_lo(v.z), w * bf16_hi(v.z), hi.z, lo.z);
+                    rt_split(w * bf16_lo(v.w), w * bf16_hi(v.w), hi.w, lo.w);
+                    *rt_cell(hi_p, r, half * 2 + g) = hi;
+                    *rt_cell(hi_p + kRtPanel, r, half * 2 + g) = lo;
+                }
+                fence_proxy_async_smem();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(w_full + (c & 1));
+                fetch(c + U, x[u]);
+            }
         }
     }
-    if (live) *reinterpret_cast<float4*>(st) = S;
+    __syncthreads();
+    if (warp == 1) {
+        tc_fence_after();
+        tmem_dealloc<32>(tmem);
+    }
 }
 
 // ret_out: warp 0 loads, warp 1 issues products, 16 warps form weights and outputs (a thread: a row and a quarter of its columns).
@@ -260,12 +289,12 @@ __device__ __forceinline__ RtItem rt_item(const LinArgs& a, const RetWs& ws, int
 template <int N>
 __global__ void __launch_bounds__(kRtOutThreads, 1)
 ret_out_kernel(const __grid_constant__ RetMaps maps, const LinArgs a, const RetWs ws, const int items, const int blocks) {
-    constexpr int KP = N / 64, VS = rt_stages(N);
+    constexpr int KP = N / 64, VS = rt_stages(N), SPANEL = N * 128;
     extern __shared__ __align__(1024) uint8_t smem[];       // (no room for alignment slack: the tiles need 1024-byte bases)
     pdl_enter();
     uint8_t* qk_sm = smem;                                  // [2][q, k]
     uint8_t* v_sm = qk_sm + 4 * KP * kRtPanel;              // [VS][2 panels]
-    uint8_t* s_sm = v_sm + VS * 2 * kRtPanel;               // [VS][leading terms, rests]
+    uint8_t* s_sm = v_sm + VS * 2 * kRtPanel;               // [VS][leading terms, rests][2 panels of N rows]
     uint64_t* bars = reinterpret_cast<uint64_t*>(s_sm + VS * 2 * KP * kRtPanel);     // two of each
     uint64_t *qk_full = bars, *qk_free = bars + 2, *v_full = bars + 4, *v_free = bars + 6, *s_full = bars + 8, *s_free = bars + 10,
              *sc_done = bars + 12, *y_done = bars + 14, *o_done = bars + 16, *a_full = bars + 18, *t_free = bars + 20;
@@ -322,11 +351,12 @@ ret_out_kernel(const __grid_constant__ RetMaps maps, const LinArgs a, const RetW
                 const int b = si % VS;
                 if (si >= VS) rt_wait(s_free + b, (si / VS - 1) & 1, stuck);
                 if (leader) {
-                    uint8_t* s = s_sm + b * 2 * KP * kRtPanel;
-                    // (a box of 128 rows: where the head's block has fewer, the rest are the next head's and are not used)
-                    mbar_expect_tx(s_full + b, 2 * KP * kRtPanel);
-                    for (int p = 0; p < 2 * KP; ++p)
-                        tma_load_2d(s + p * kRtPanel, &maps.s, s_full + b, p * 64, it.cell * a.P + it.p0, kEvictFirst);
+                    uint8_t* s = s_sm + b * 4 * SPANEL;
+                    const int panels = (it.Pb + 63) >> 6;       // (columns past the head's own values are never used)
+                    mbar_expect_tx(s_full + b, 2 * panels * SPANEL);
+                    for (int t = 0; t < 2; ++t)
+                        for (int p = 0; p < panels; ++p)
+                            tma_load_2d(s + (2 * t + p) * SPANEL, &maps.s, s_full + b, t * a.P + it.p0 + p * 64, it.cell * N, kEvictFirst);
                 }
                 __syncwarp();
                 ++si;
@@ -345,7 +375,7 @@ ret_out_kernel(const __grid_constant__ RetMaps maps, const LinArgs a, const RetW
         const bool leader = elect_one();
         constexpr uint64_t PANEL = kRtPanel >> 4;
         constexpr uint32_t IDESC_QK = make_idesc_f16(128, 128, true, false, false);
-        const uint64_t d_qk = make_desc_kmajor_sw128(smem_u32(qk_sm)), d_s = make_desc_kmajor_sw128(smem_u32(s_sm)),
+        const uint64_t d_qk = make_desc_kmajor_sw128(smem_u32(qk_sm)), d_s = make_desc_mnmajor_sw128(smem_u32(s_sm), SPANEL),
                        d_v = make_desc_mnmajor_sw128(smem_u32(v_sm), kRtPanel);
         int i = 0, si = 0;
         bool prev_fresh = false;
@@ -390,14 +420,14 @@ ret_out_kernel(const __grid_constant__ RetMaps maps, const LinArgs a, const RetW
                 const int sb = si % VS;
                 rt_wait(s_full + sb, (si / VS) & 1, stuck);
                 tc_fence_after();
-                const uint32_t idesc = make_idesc_f16(128, it.Pb, true, false, false);
+                const uint32_t idesc = make_idesc_f16(128, it.Pb, true, false, true);
                 if (leader) {
 #pragma unroll
                     for (int t = 0; t < 2; ++t)
 #pragma unroll
                         for (int kk = 0; kk < N / 16; ++kk) {
                             const uint64_t o = (kk >> 2) * PANEL + 2 * (kk & 3);
-                            umma_f16_ss(t_a + 128, dq + o, d_s + (2 * sb + t) * KP * PANEL + o, idesc, (t > 0 || kk > 0) ? 1u : 0u);
+                            umma_f16_ss(t_a + 128, dq + o, d_s + (2 * sb + t) * (2 * SPANEL >> 4) + kk * kRtRows16, idesc, (t > 0 || kk > 0) ? 1u : 0u);
                         }
                     umma_commit(y_done + b);
                     umma_commit(s_free + sb);
@@ -583,22 +613,21 @@ static int rt_chunk_launch(const LinArgs& a, int n_multi, void* ws, int64_t ws_b
     int rc = make_tmap_2d_16b(&m.q, a.q, keys, T, static_cast<uint64_t>(a.ld_qk) * 2, 64, kRtTok, true);
     if (!rc) rc = make_tmap_2d_16b(&m.k, a.k, keys, T, static_cast<uint64_t>(a.ld_qk) * 2, 64, kRtTok, true);
     if (!rc) rc = make_tmap_2d_16b(&m.v, a.v, vals, T, static_cast<uint64_t>(a.ld) * 2, 64, kRtTok, true);
-    if (!rc) rc = make_tmap_2d_16b(&m.s, ws, 2 * N, static_cast<uint64_t>(step) * vals, 4 * N, 64, kRtTok, true);
+    if (!rc) rc = make_tmap_2d_16b(&m.s, ws, 2 * static_cast<uint64_t>(a.P), static_cast<uint64_t>(step) * keys, 4 * static_cast<uint64_t>(a.P), 64, N, true);
     if (rc) return rc;
-    auto local = ret_local_kernel<N>;
-    auto chain = ret_chain_kernel<N>;
+    auto chain = ret_state_kernel<N>;
     auto out = ret_out_kernel<N>;
-    HDS_CHECK_CUDA(cudaFuncSetAttribute(local, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(rt_local_smem(N))));
+    HDS_CHECK_CUDA(cudaFuncSetAttribute(chain, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(rt_state_smem(N))));
     HDS_CHECK_CUDA(cudaFuncSetAttribute(out, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(rt_out_smem(N))));
     const unsigned blocks = (a.P + kRtP - 1) / kRtP;
+    const bool reads = a.out != nullptr || a.write_y;
     for (int64_t c0 = 0; c0 < bound; c0 += step) {
         RetWs w;
-        w.s = static_cast<float*>(ws);
+        w.s = reads ? static_cast<uint16_t*>(ws) : nullptr;
         w.c0 = static_cast<int>(c0);
         w.n = static_cast<int>(step < bound - c0 ? step : bound - c0);
-        HDS_CHECK_CUDA(launch_kernel(local, dim3(w.n, a.heads, blocks), dim3(kRtThreads), rt_local_smem(N), s, m, a, w));
-        HDS_CHECK_CUDA(launch_kernel(chain, dim3(a.n_seqs, a.heads, (a.P * N / 4 + kRtThreads - 1) / kRtThreads), dim3(kRtThreads), 0, s, a, w));
-        if (a.out != nullptr || a.write_y) {
+        HDS_CHECK_CUDA(launch_kernel(chain, dim3(a.n_seqs, a.heads, (a.P + kRsP - 1) / kRsP), dim3(kRsThreads), rt_state_smem(N), s, m, a, w));
+        if (reads) {
             const int items = w.n * a.heads * static_cast<int>(blocks), sms = sm_count();
             HDS_CHECK_CUDA(launch_kernel(out, dim3(items < sms ? items : sms), dim3(kRtOutThreads), rt_out_smem(N), s, m, a, w, items, static_cast<int>(blocks)));
         }

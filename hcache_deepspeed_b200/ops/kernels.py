@@ -916,7 +916,7 @@ def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Ten
                                          0 if out is None else out.stride(0), eps, _p(workspace), 0 if workspace is None else workspace.numel(),
                                          method, ctypes.addressof(done), _dt3(q), _stream())
     native.check(rc, "hds_retention")
-    _count((3 if out is not None else 2) * (spans.shape[0] > n_single) + (n_single > 0))
+    _count((2 if out is not None else 1) * (spans.shape[0] > n_single) + (n_single > 0))
     if out is not None and not done.value:
         r = vdim / norm_cols          # mean over a padded row * r = mean over the head
         gated_norm(y[:, :heads * vdim], gate, ones, out, heads, eps / r, r**-0.5, gate_after=True)
